@@ -37,6 +37,9 @@ NVCC_FLAGS = [
     "-Wno-unused-function",
     "--expt-relaxed-constexpr",
 ]
+# Sources compiled without --use_fast_math: their exponentials, logarithms, divisions and roots feed recurrent state or
+# serve the 32-bit mode.
+PRECISE_SOURCES = {"hybrid_ops.cu", "delta_rule.cu"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-pthread"]
 
 
@@ -74,6 +77,8 @@ def lib_path(flavour: str = "") -> Path:
 def _compile_one(src: Path, verbose: bool, ptxas_verbose: bool, flavour: str = "") -> Path:
     is_cu = src.suffix == ".cu"
     flags = (NVCC_FLAGS if is_cu else CXX_FLAGS) + FLAVOUR_FLAGS[flavour]
+    if src.name in PRECISE_SOURCES:
+        flags = [f for f in flags if f != "--use_fast_math"]
     obj_dir = OBJ_DIR if not flavour else OBJ_DIR.parent / f"build_{flavour}"
     obj = obj_dir / (src.name + ".o")
     stamp = obj_dir / (src.name + ".sha1")

@@ -9,6 +9,11 @@
 //    waiting sequences for (chunked) prefill within the token budget. When pages run out the most
 //    recently admitted running sequence is preempted (its pages are released; it is re-prefilled later
 //    with the tokens generated so far).
+//  * State slots: every running sequence owns one of max_num_seqs slots (recurrent state, convolution inputs) from its
+//    admission until it finishes, is preempted or is removed. A sequence that (re)starts at position 0 ignores what the
+//    slot held.
+//  * Fed sequences: the caller brings the tokens of every step itself (replays, scoring); vb_sched_feed plans exactly
+//    the given tokens, all or nothing, and never preempts. They end with vb_sched_remove.
 //  * Abort / finish release pages immediately. All state is host memory; the Python side copies the
 //    step description (token ids, positions, slot mapping, block tables) into pinned buffers.
 //
@@ -32,6 +37,7 @@ struct Seq {
   int num_cached_pages = 0;      // leading pages obtained from the prefix cache
   bool running = false;
   bool finished = false;
+  int state_slot = -1;           // slot of the per-sequence state while running
   int preempt_count = 0;
   std::vector<uint64_t> page_hashes;  // hash chain of the full prompt pages
 };
@@ -52,6 +58,7 @@ struct Scheduler {
   std::unordered_map<int64_t, Seq> seqs;
   std::deque<int64_t> waiting;
   std::vector<int64_t> running;                       // admission order
+  std::vector<int32_t> free_slots;                    // state slots no running sequence owns
   int64_t clock = 0;
   int64_t total_preempted = 0;
   int64_t prefix_hits = 0, prefix_queries = 0;
@@ -109,6 +116,16 @@ void release_seq_pages(Scheduler* s, Seq& q) {
   q.blocks.clear();
   q.computed = 0;
   q.num_cached_pages = 0;
+  if (q.state_slot >= 0) {
+    s->free_slots.push_back(q.state_slot);
+    q.state_slot = -1;
+  }
+}
+
+void take_slot(Scheduler* s, Seq& q) {
+  if (q.state_slot >= 0 || s->free_slots.empty()) return;
+  q.state_slot = s->free_slots.back();
+  s->free_slots.pop_back();
 }
 
 void compute_hashes(Scheduler* s, Seq& q) {
@@ -197,6 +214,7 @@ void* vb_sched_create(int num_blocks, int block_size, int max_num_seqs, int max_
   s->prefix_caching = prefix_caching != 0;
   s->pages.resize(num_blocks);
   for (int i = num_blocks - 1; i >= 0; --i) s->free_list.push_back(i);
+  for (int i = max_num_seqs - 1; i >= 0; --i) s->free_slots.push_back(i);
   return s;
 }
 
@@ -297,6 +315,7 @@ int vb_sched_step(void* h) {
     if (!ensure_pages(s, q, q.computed + want)) { release_seq_pages(s, q); break; }
     s->waiting.erase(s->waiting.begin() + wi);
     q.running = true;
+    take_slot(s, q);
     s->running.push_back(id);
     s->step_seq_ids.push_back(id);
     s->step_num_tokens.push_back(want);
@@ -306,6 +325,59 @@ int vb_sched_step(void* h) {
     if ((int)q.page_hashes.size() > q.num_cached_pages) inflight.push_back(q.page_hashes[0]);
   }
   return (int)s->step_seq_ids.size();
+}
+
+// Plan a step of exactly these tokens: counts[i] >= 1 of sequence ids[i], concatenated in `tokens`. A sequence that does
+// not exist yet starts here. Returns 0, or without having changed anything: -1 a repeated id, an empty entry or too many
+// tokens, -2 the sequence would exceed max_model_len, -3 no free place for a new sequence, -4 not enough free pages.
+int vb_sched_feed(void* h, int n, const int64_t* ids, const int32_t* counts, const int32_t* tokens) {
+  auto* s = static_cast<Scheduler*>(h);
+  long long need = 0, total = 0;
+  int fresh = 0;
+  for (int i = 0; i < n; ++i) {
+    for (int j = 0; j < i; ++j)
+      if (ids[j] == ids[i]) return -1;
+    if (counts[i] <= 0) return -1;
+    total += counts[i];
+    auto it = s->seqs.find(ids[i]);
+    const int have = it == s->seqs.end() ? 0 : (int)it->second.tokens.size();
+    if (have + counts[i] > s->max_model_len) return -2;
+    fresh += it == s->seqs.end();
+    need += (have + counts[i] + s->block_size - 1) / s->block_size - (it == s->seqs.end() ? 0 : (int)it->second.blocks.size());
+  }
+  if (total > s->max_batched_tokens) return -1;
+  if ((int)s->running.size() + fresh > s->max_num_seqs) return -3;
+  if (need > free_pages(s)) return -4;
+  s->clock++;
+  s->step_seq_ids.clear();
+  s->step_num_tokens.clear();
+  s->step_start.clear();
+  s->step_is_prefill.clear();
+  for (int i = 0; i < n; ++i) {
+    Seq& q = s->seqs[ids[i]];
+    if (!q.running) {
+      q.id = ids[i];
+      q.running = true;
+      q.max_total = s->max_model_len + 1;  // only the caller ends it
+      take_slot(s, q);
+      s->running.push_back(ids[i]);
+    }
+    q.tokens.insert(q.tokens.end(), tokens, tokens + counts[i]);
+    q.prompt_len = (int)q.tokens.size();
+    tokens += counts[i];
+    ensure_pages(s, q, (int)q.tokens.size());
+    s->step_seq_ids.push_back(ids[i]);
+    s->step_num_tokens.push_back(counts[i]);
+    s->step_start.push_back(q.computed);
+    s->step_is_prefill.push_back(counts[i] > 1 || q.computed == 0 ? 1 : 0);
+  }
+  return 0;
+}
+
+// State slots of the sequences of the last planned step.
+void vb_sched_step_slots(void* h, int32_t* slots) {
+  auto* s = static_cast<Scheduler*>(h);
+  for (size_t i = 0; i < s->step_seq_ids.size(); ++i) slots[i] = s->seqs[s->step_seq_ids[i]].state_slot;
 }
 
 // Copy the plan of the last step. ``tokens``/``positions``/``slots`` have one entry per scheduled token,

@@ -10,6 +10,8 @@ from dataclasses import asdict, dataclass, field
 from pathlib import Path
 from typing import Any
 
+from .layer_specs import AttentionSpec, DeltaSpec, GluSpec, LayerSpec
+
 _ARCH_TO_TYPE = {
     "LlamaForCausalLM": "llama",
     "MistralForCausalLM": "llama",
@@ -29,6 +31,8 @@ _TYPE_TO_ARCH = {"llama": "LlamaForCausalLM", "qwen2": "Qwen2ForCausalLM", "qwen
                  "qwen3_moe": "Qwen3MoeForCausalLM", "qwen2_vl": "Qwen2VLForConditionalGeneration",
                  "qwen2_5_vl": "Qwen2_5_VLForConditionalGeneration", "apertus": "ApertusForCausalLM",
                  "qwen3_vl": "Qwen3VLForConditionalGeneration", "qwen3_vl_moe": "Qwen3VLMoeForConditionalGeneration"}
+# designs whose config.json lists its layers one by one (``architecture`` instead of ``architectures``)
+_LAYER_LIST_ARCHS = {"Fuganex": "fuganex"}
 _VL_TYPES = ("qwen2_vl", "qwen2_5_vl", "qwen3_vl", "qwen3_vl_moe")
 
 
@@ -61,9 +65,15 @@ class ModelConfig:
     bos_token_id: int | None = None
     eos_token_id: int | None = 2
     pad_token_id: int | None = None
+    # layer-list designs: one LayerSpec per layer (empty: all layers alike, described by the fields above)
+    layer_specs: tuple = ()
+    embedding_scale: float = 1.0
     extra: dict = field(default_factory=dict)
 
     def __post_init__(self):
+        self.layer_specs = tuple(self.layer_specs)
+        if self.layer_specs:
+            self.num_hidden_layers = len(self.layer_specs)
         if self.head_dim is None:
             self.head_dim = self.hidden_size // self.num_attention_heads
         if self.attention_bias is None:
@@ -77,6 +87,15 @@ class ModelConfig:
     @property
     def is_moe(self) -> bool:
         return self.num_experts > 0
+
+    @property
+    def is_layer_list(self) -> bool:
+        return bool(self.layer_specs)
+
+    @property
+    def has_recurrent_state(self) -> bool:
+        """Some layer carries a state per sequence that pages cannot share."""
+        return any(s.kind == "delta" for s in self.layer_specs)
 
     @property
     def mlp_gated(self) -> bool:
@@ -112,6 +131,9 @@ class ModelConfig:
 
     def num_parameters(self, include_embedding: bool = True) -> int:
         H, L = self.hidden_size, self.num_hidden_layers
+        if self.is_layer_list:
+            total = H + sum(s.num_parameters(H) for s in self.layer_specs)
+            return total + (2 * self.vocab_size * H if include_embedding else 0)
         attn = H * (self.q_size + 2 * self.kv_size) + self.q_size * H
         if self.attention_bias:
             attn += self.q_size + 2 * self.kv_size
@@ -129,6 +151,8 @@ class ModelConfig:
     # --------------------------------------------------------------- (de)serialise
     @classmethod
     def from_hf_dict(cls, d: dict[str, Any]) -> "ModelConfig":
+        if d.get("architecture") in _LAYER_LIST_ARCHS:
+            return cls._from_layer_list(d)
         mt = d.get("model_type")
         if mt is None:
             archs = d.get("architectures") or ["Qwen2ForCausalLM"]
@@ -181,6 +205,30 @@ class ModelConfig:
         return cfg
 
     @classmethod
+    def _from_layer_list(cls, d: dict[str, Any]) -> "ModelConfig":
+        specs = tuple(LayerSpec.from_dict(x) for x in d["layers"])
+        att = [s.mixer for s in specs if s.kind == "attention"]
+        kw = {k: int(d[k]) for k in ("bos_token_id", "eos_token_id", "pad_token_id") if d.get(k) is not None}
+        kw.setdefault("eos_token_id", None)
+        known = ("architecture", "vocab", "width", "layers", "norm", "embedding", *kw)
+        return cls(model_type=_LAYER_LIST_ARCHS[d["architecture"]], vocab_size=int(d["vocab"]), hidden_size=int(d["width"]),
+                   intermediate_size=max([s.mlp.ff for s in specs if s.mlp] or [0]),
+                   num_attention_heads=max([a.heads for a in att] or [1]),
+                   num_key_value_heads=max([a.kv_heads for a in att] or [1]), head_dim=max([a.dim for a in att] or [1]),
+                   rms_norm_eps=float(d["norm"]["eps"]), embedding_scale=float(d["embedding"]["scale"]),
+                   layer_specs=specs, extra={k: v for k, v in d.items() if k not in known}, **kw)
+
+    def _to_layer_list(self) -> dict[str, Any]:
+        arch = {v: k for k, v in _LAYER_LIST_ARCHS.items()}[self.model_type]
+        d = {"architecture": arch, "vocab": self.vocab_size, "width": self.hidden_size,
+             "layers": [s.to_dict() for s in self.layer_specs], "norm": {"eps": self.rms_norm_eps},
+             "embedding": {"scale": self.embedding_scale}, **self.extra}
+        for k in ("bos_token_id", "eos_token_id", "pad_token_id"):
+            if getattr(self, k) is not None:
+                d[k] = getattr(self, k)
+        return d
+
+    @classmethod
     def from_pretrained(cls, path: str | Path) -> "ModelConfig":
         p = Path(path)
         if p.is_dir():
@@ -188,7 +236,10 @@ class ModelConfig:
         return cls.from_hf_dict(json.loads(p.read_text()))
 
     def to_hf_dict(self) -> dict[str, Any]:
+        if self.is_layer_list:
+            return self._to_layer_list()
         d = asdict(self)
+        del d["layer_specs"], d["embedding_scale"]
         extra = d.pop("extra")
         if self.model_type in _VL_TYPES:
             moe_keys = () if self.is_moe else ("num_experts", "num_experts_per_tok", "moe_intermediate_size", "norm_topk_prob",
@@ -224,6 +275,15 @@ class ModelConfig:
         p = Path(path)
         p.mkdir(parents=True, exist_ok=True)
         (p / "config.json").write_text(json.dumps(self.to_hf_dict(), indent=2))
+
+
+def _fuganex_specs(groups: int, heads: int, kv_heads: int, dim: int, window: int, keep_first: int, ff: int, d_heads: int,
+                   d_kv_heads: int, d_dim: int) -> tuple:
+    """``groups`` x (two delta-rule layers, one attention layer), a feed-forward after each."""
+    mlp = GluSpec(ff, 7.0)
+    delta = LayerSpec(DeltaSpec(d_heads, d_kv_heads, d_dim, d_dim, 4), mlp)
+    att = LayerSpec(AttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, window, keep_first, 128.0, 32), mlp)
+    return (delta, delta, att) * groups
 
 
 # Named architectures used by the benchmarks and tests (random-init, no download needed).
@@ -324,6 +384,12 @@ PRESETS: dict[str, dict] = {
                        rms_norm_eps=1e-5, eos_token_id=2, max_position_embeddings=65536,
                        extra={"rope_scaling": {"rope_type": "llama3", "factor": 8.0, "original_max_position_embeddings": 8192,
                                                "low_freq_factor": 1.0, "high_freq_factor": 4.0}}),
+    "tiny-fuganex": dict(model_type="fuganex", vocab_size=640, hidden_size=192, eos_token_id=2, rms_norm_eps=1e-6,
+                         layer_specs=_fuganex_specs(1, 6, 2, 32, 40, 6, 320, 6, 3, 32)),
+    # real-model sizes for benchmarks: the widths of llama-3-8b, a third of the layers with windowed attention
+    "fuganex-8b": dict(model_type="fuganex", vocab_size=128256, hidden_size=4096, eos_token_id=None, rms_norm_eps=1e-5,
+                       num_attention_heads=32, num_key_value_heads=8, head_dim=128, intermediate_size=14336,
+                       layer_specs=_fuganex_specs(10, 32, 8, 128, 1024, 4, 14336, 32, 16, 128)),
     "llama-3-8b": dict(model_type="llama", vocab_size=128256, hidden_size=4096, intermediate_size=14336,
                        num_hidden_layers=32, num_attention_heads=32, num_key_value_heads=8, rope_theta=5e5,
                        rms_norm_eps=1e-5, eos_token_id=128001),

@@ -70,6 +70,8 @@ def _normalise_vl_keys(hf_sd: dict) -> dict:
 
 def hf_to_native_state_dict(cfg: ModelConfig, hf_sd: dict[str, torch.Tensor]) -> dict[str, torch.Tensor]:
     """Fuse an HF state dict into native parameter names/shapes."""
+    if cfg.is_layer_list:
+        return _layer_list_to_native(cfg, hf_sd)
     out: dict[str, torch.Tensor] = {}
     if cfg.is_vl or any(k.startswith(("model.language_model.", "model.visual.", "visual.")) for k in hf_sd):
         hf_sd = _normalise_vl_keys(hf_sd)
@@ -131,6 +133,10 @@ def hf_to_native_state_dict(cfg: ModelConfig, hf_sd: dict[str, torch.Tensor]) ->
 def native_to_hf_items(cfg: ModelConfig, named: Iterable[tuple[str, torch.Tensor]]) -> Iterator[tuple[str, torch.Tensor]]:
     """Stream (hf_name, tensor) pairs from native (name, tensor) pairs, splitting fused tensors.
     Works one parameter at a time so it can drive a weight-sync generator."""
+    if cfg.is_layer_list:
+        for name, t in named:
+            yield from _layer_list_to_ckpt(cfg, name, t)
+        return
     vl = cfg.is_vl
     lm = "model.language_model." if vl else "model."
     for name, t in named:
@@ -197,6 +203,72 @@ def native_to_hf_items(cfg: ModelConfig, named: Iterable[tuple[str, torch.Tensor
                 yield p + rest, t
         else:
             yield name, t
+
+
+# ------------------------------------------------------------- layer-list checkpoints (models/hybrid.py)
+# native name -> checkpoint name of the tensors that are stored alike
+_LIST_TOP = {"embed_tokens.weight": "embed", "norm.weight": "final.norm", "lm_head.weight": "head"}
+_LIST_PLAIN = {"norm1.weight": "norm1", "norm2.weight": "norm2", "mlp.down_proj.weight": "mlp.down",
+               "mixer.o_proj.weight": "mix.o", "mixer.q_norm.weight": "mix.q.norm", "mixer.k_norm.weight": "mix.k.norm",
+               "mixer.rel": "mix.rel", "mixer.A_log": "mix.A_log", "mixer.dt_bias": "mix.dt_bias",
+               "mixer.norm.weight": "mix.norm"}
+
+
+def _list_fused(spec) -> dict[str, list[tuple[str, int]]]:
+    """Native fused matrices of a layer: name -> [(checkpoint name, rows), ...] in row order."""
+    m = spec.mixer
+    if spec.kind == "attention":
+        out = {"mixer.qkv_proj.weight": [("mix.q", m.q_size), ("mix.k", m.k_size), ("mix.v", m.v_size)]}
+    else:
+        qk, v = m.kv_heads * m.dim, m.heads * m.vdim
+        out = {"mixer.in_proj.weight": [("mix.q", qk), ("mix.k", qk), ("mix.v", v), ("mix.g", v), ("mix.b", m.heads),
+                                        ("mix.a", m.heads)],
+               "mixer.conv": [("mix.q.conv", qk), ("mix.k.conv", qk), ("mix.v.conv", v)]}
+    if spec.mlp is not None:
+        out["mlp.gate_up_proj.weight"] = [("mlp.gate", spec.mlp.ff), ("mlp.up", spec.mlp.ff)]
+    return out
+
+
+def _layer_list_to_native(cfg: ModelConfig, sd: dict[str, torch.Tensor]) -> dict[str, torch.Tensor]:
+    out = {n: sd[c] for n, c in _LIST_TOP.items()}
+    for i, spec in enumerate(cfg.layer_specs):
+        fused = _list_fused(spec)
+        for n, parts in fused.items():
+            ts = []
+            for c, rows in parts:
+                t = sd[f"l{i}.{c}"]
+                if t.shape[0] != rows:
+                    raise ValueError(f"l{i}.{c}: {t.shape[0]} rows, the configuration says {rows}")
+                ts.append(t)
+            w = torch.cat(ts, 0)
+            if n.endswith("_proj.weight") and w.shape[0] % 8:  # padded with zero rows
+                w = torch.cat([w, w.new_zeros(8 - w.shape[0] % 8, w.shape[1])], 0)
+            out[f"layers.{i}.{n}"] = w
+        for n, c in _LIST_PLAIN.items():
+            if f"l{i}.{c}" in sd:
+                out[f"layers.{i}.{n}"] = sd[f"l{i}.{c}"]
+    return out
+
+
+def _layer_list_to_ckpt(cfg: ModelConfig, name: str, t: torch.Tensor) -> Iterator[tuple[str, torch.Tensor]]:
+    if name in _LIST_TOP:
+        yield _LIST_TOP[name], t
+        return
+    _, i, rest = name.split(".", 2)
+    if rest in _LIST_PLAIN:
+        yield f"l{i}.{_LIST_PLAIN[rest]}", t
+        return
+    lo = 0
+    for c, rows in _list_fused(cfg.layer_specs[int(i)])[rest]:
+        yield f"l{i}.{c}", t[lo : lo + rows]
+        lo += rows
+
+
+def _sizes_from_tensors(cfg: ModelConfig, sd: dict[str, torch.Tensor]) -> None:
+    """Sizes that only the tensors' shapes give: the rows of the distance-bias tables."""
+    cfg.layer_specs = tuple(
+        s.with_bias_rows(sd[f"l{i}.mix.rel"].shape[0] if f"l{i}.mix.rel" in sd else 0) if s.kind == "attention" else s
+        for i, s in enumerate(cfg.layer_specs))
 
 
 def _vis_native_to_hf(name: str, gated: bool = False) -> str:
@@ -267,4 +339,6 @@ def load_hf_checkpoint(path: str | Path) -> tuple[ModelConfig, dict[str, torch.T
         raise FileNotFoundError(f"no safetensors files under {path}")
     for f in files:
         hf_sd.update(load_file(str(f)))
+    if cfg.is_layer_list:
+        _sizes_from_tensors(cfg, hf_sd)
     return cfg, hf_to_native_state_dict(cfg, hf_sd)

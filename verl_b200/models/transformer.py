@@ -364,6 +364,9 @@ class CausalLM(nn.Module):
         ``lo .. hi - 1``; the embedding lives on the first stage, final norm and head on the last). ``layers[i]`` is then
         decoder layer ``lo + i`` (``layer_offset``)."""
         super().__init__()
+        if cfg.is_layer_list:
+            raise NotImplementedError(f"{cfg.model_type}: layer-list models are built by build_model and served by the "
+                                      "rollout engine; there is no training path for them")
         self.cfg = cfg
         self.value_head = value_head or cfg.num_labels == 1
         lo, hi = layer_range if layer_range is not None else (0, cfg.num_hidden_layers)
@@ -514,9 +517,23 @@ class CausalLM(nn.Module):
         return self.logprob_entropy(hidden, labels, temperature)
 
 
+def model_class(cfg: ModelConfig):
+    """Module class of an architecture."""
+    if cfg.is_layer_list:
+        from .hybrid import HybridLM
+
+        return HybridLM
+    return CausalLM
+
+
 def build_model(cfg: ModelConfig, dtype=torch.bfloat16, device="cpu", value_head: bool = False, seed: int = 0,
-                init: bool = True) -> CausalLM:
-    m = CausalLM(cfg, dtype=dtype, device=device, value_head=value_head)
+                init: bool = True) -> nn.Module:
+    if cfg.is_layer_list:
+        if value_head:
+            raise NotImplementedError(f"{cfg.model_type}: layer-list models have no value head")
+        m = model_class(cfg)(cfg, dtype=dtype, device=device)
+    else:
+        m = CausalLM(cfg, dtype=dtype, device=device, value_head=value_head)
     if init:
         m.init_weights(seed)
     return m

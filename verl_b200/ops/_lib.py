@@ -45,6 +45,14 @@ _SIGS = {
     "vb_sumsq": ([P, I, L, P, P], I),
     "vb_clip_coef": ([P, F, F, P, P, P, P], I),
     "vb_cast_f32_bf16": ([P, P, L, P], I),
+    # layer-list decoders
+    "vb_embed_scaled": ([P, P, P, I, I, F, I, P], I),
+    "vb_add_rmsnorm": ([P, L, P, P, P, I, I, F, I, P], I),
+    "vb_clamped_glu": ([P, L, P, I, I, F, F, I, P], I),
+    "vb_qk_norm_kv_write": ([P, L, P, P, P, P, P, I, I, I, I, I, I, F, I, P], I),
+    "vb_gemm_simt": ([P, P, P, P, I, I, I, L, L, L, I, I, P], I),
+    "vb_paged_attention_simt": ([P, L, P, P, P, I, P, P, I, I, I, I, I, I, I, F, I, I, P, I, P, L, I, P], I),
+    "vb_delta_rule": ([P, L, P, P, P, P, P, P, P, P, P, P, P, P, L, I, I, I, I, I, I, I, I, F, I, P], I),
     # rl ops
     "vb_ppo_loss": ([P, P, P, P, P, P, P, P, P, P, L, F, F, F, F, I, F, F, P], I),
     "vb_gae": ([P, P, P, P, P, I, I, F, F, P], I),

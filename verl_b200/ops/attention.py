@@ -204,3 +204,68 @@ def paged_decode_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torc
         s = torch.einsum("hgd,hld->hgl", qq, kk) * scale
         out[b] = torch.einsum("hgl,hld->hgd", torch.softmax(s, -1), vv).reshape(Hq, D).to(q.dtype)
     return out
+
+
+# ------------------------------------------- paged attention of layer-list decoders (windows, kept keys, distance bias)
+def qk_norm_kv_write(qkv: torch.Tensor, q_weight: torch.Tensor | None, k_weight: torch.Tensor | None, slots: torch.Tensor,
+                     k_cache: torch.Tensor, v_cache: torch.Tensor, heads: int, eps: float) -> torch.Tensor:
+    """``qkv`` [T, q | k | v | padding]: RMS norm of q and of k over the whole projection (all heads at once; no weights =
+    no norm), k and v to their places in the paged caches [NB, Hk, BS, D] / [NB, Hk, BS, Dv] (slot < 0: no write).
+    Returns q [T, heads, D], a view of ``qkv`` (normalised in place on CUDA)."""
+    _, Hk, BS, D = k_cache.shape
+    Dv = v_cache.shape[3]
+    T, nq, nk = qkv.shape[0], heads * D, Hk * D
+    if qkv.is_cuda:
+        rc = _lib.fn("vb_qk_norm_kv_write")(qkv.data_ptr(), qkv.stride(0), _lib.ptr(q_weight), _lib.ptr(k_weight),
+                                            slots.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), T, heads, Hk, D, Dv, BS,
+                                            float(eps), int(qkv.dtype == torch.float32), _lib.stream())
+        _lib.check(rc, "vb_qk_norm_kv_write")
+        return qkv[:, :nq].view(T, heads, D)
+    from .nn import _rmsnorm_ref
+
+    q, k, v = qkv[:, :nq], qkv[:, nq : nq + nk], qkv[:, nq + nk : nq + nk + Hk * Dv]
+    if q_weight is not None:
+        q, k = _rmsnorm_ref(q, q_weight, eps), _rmsnorm_ref(k, k_weight, eps)
+    kv_cache_write(k.reshape(T, Hk, D), v.reshape(T, Hk, Dv), slots, k_cache, v_cache)
+    return q.reshape(T, heads, D)
+
+
+def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor,
+                    cu_q: torch.Tensor, seq_lens: torch.Tensor, max_q: int, *, scale: float, window: int = 0,
+                    keep_first: int = 0, bias: torch.Tensor | None = None, impl: str = "auto") -> torch.Tensor:
+    """Causal attention of ragged queries (the last ``cu_q[b + 1] - cu_q[b]`` positions of every sequence) over the paged
+    cache, which holds the new tokens already. q [T, Hq, D]; caches [NB, Hk, BS, D] / [NB, Hk, BS, Dv]; ``seq_lens``
+    [B] = tokens of each sequence including the new ones. ``window`` > 0: position i sees j <= i with i - j < window or
+    j < keep_first. ``bias`` fp32 [Hq, L]: ``bias[h, min(i - j, L - 1)]`` is added to the scaled score. -> [T, Hq * Dv]."""
+    T, Hq, D = q.shape
+    Hk, BS, Dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
+    B = seq_lens.numel()
+    out = torch.empty((T, Hq * Dv), dtype=q.dtype, device=q.device)
+    if q.is_cuda:
+        f32 = q.dtype == torch.float32
+        L = 0 if bias is None else bias.shape[1]
+        rc = _lib.fn("vb_paged_attention_simt")(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
+                                                block_table.data_ptr(), block_table.stride(0), cu_q.data_ptr(),
+                                                seq_lens.data_ptr(), T, B, Hq, Hk, D, Dv, BS, float(scale), window, keep_first,
+                                                _lib.ptr(bias), L, out.data_ptr(), out.stride(0), int(f32), _lib.stream())
+        _lib.check(rc, "vb_paged_attention_simt")
+        return out
+    G = Hq // Hk
+    cu, lens = cu_q.tolist(), seq_lens.tolist()
+    for b in range(B):
+        lo, hi, n = cu[b], cu[b + 1], lens[b]
+        if hi == lo:
+            continue
+        blocks = block_table[b, : (n + BS - 1) // BS].long()
+        kk = k_cache[blocks].permute(1, 0, 2, 3).reshape(Hk, -1, D)[:, :n].float().repeat_interleave(G, 0)
+        vv = v_cache[blocks].permute(1, 0, 2, 3).reshape(Hk, -1, Dv)[:, :n].float().repeat_interleave(G, 0)
+        s = torch.einsum("qhd,hkd->hqk", q[lo:hi].float(), kk) * scale
+        dist = torch.arange(n - (hi - lo), n, device=q.device)[:, None] - torch.arange(n, device=q.device)[None]
+        seen = dist >= 0
+        if window > 0:
+            seen &= (dist < window) | (torch.arange(n, device=q.device)[None] < keep_first)
+        if bias is not None:
+            s = s + bias[:, dist.clamp(0, bias.shape[1] - 1)]
+        s = s.masked_fill(~seen, float("-inf"))
+        out[lo:hi] = torch.einsum("hqk,hkd->qhd", torch.softmax(s, -1), vv).reshape(hi - lo, -1).to(q.dtype)
+    return out

@@ -52,6 +52,8 @@ def gemm(
                 out.copy_(res)
             return out
         return res.to(out_dtype)
+    if _needs_simt(a, b) and not (a_mn or b_mn or accumulate):
+        return _gemm_simt(a, b, bias, out, out_dtype)
     if a.dtype != torch.bfloat16 or b.dtype != torch.bfloat16:
         raise TypeError("gemm expects bf16 operands on CUDA")
     _check_2d(a, "a")
@@ -73,6 +75,26 @@ def gemm(
         _lib.status_word(a.device).data_ptr(), stream,
     )
     _lib.check(rc, "vb_gemm_bf16")
+    return out
+
+
+def _needs_simt(a: torch.Tensor, b: torch.Tensor) -> bool:
+    """32-bit operands (true fp32 products), or bf16 rows that TMA cannot describe (row length not a multiple of 8)."""
+    if a.dtype != b.dtype:
+        return False
+    return a.dtype == torch.float32 or (a.dtype == torch.bfloat16 and (a.stride(0) % 8 != 0 or b.stride(0) % 8 != 0))
+
+
+def _gemm_simt(a, b, bias, out, out_dtype):
+    f32 = a.dtype == torch.float32
+    if out is None:
+        out = torch.empty((a.shape[0], b.shape[0]), dtype=torch.float32 if f32 else out_dtype, device=a.device)
+    if a.stride(1) != 1 or b.stride(1) != 1 or out.stride(1) != 1 or (f32 and out.dtype != torch.float32):
+        raise TypeError("gemm: unit inner strides are required, and fp32 operands give an fp32 result")
+    rc = _lib.fn("vb_gemm_simt")(a.data_ptr(), b.data_ptr(), out.data_ptr(), _lib.ptr(bias), a.shape[0], b.shape[0],
+                                 a.shape[1], a.stride(0), b.stride(0), out.stride(0), int(f32),
+                                 int(out.dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "vb_gemm_simt")
     return out
 
 

@@ -269,3 +269,47 @@ def embedding(ids: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
     if weight.is_cuda:
         return _EmbeddingFn.apply(ids.contiguous(), weight)
     return F.embedding(ids, weight)
+
+
+# ------------------------------------------------- 32-bit residual stream (inference only)
+def embedding_scaled(ids: torch.Tensor, weight: torch.Tensor, scale: float) -> torch.Tensor:
+    """fp32 residual stream ``weight[ids] * scale`` [T, H]."""
+    if not weight.is_cuda:
+        return F.embedding(ids, weight).float() * scale
+    T, H = ids.numel(), weight.shape[1]
+    res = torch.empty((T, H), dtype=torch.float32, device=weight.device)
+    rc = _lib.fn("vb_embed_scaled")(ids.data_ptr(), weight.data_ptr(), res.data_ptr(), T, H, float(scale),
+                                    int(weight.dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "vb_embed_scaled")
+    return res
+
+
+def add_rmsnorm(delta: torch.Tensor | None, residual: torch.Tensor, weight: torch.Tensor, eps: float) -> torch.Tensor:
+    """Adds ``delta`` to the fp32 ``residual`` [T, H] IN PLACE and returns rmsnorm(residual) * weight in the weight's
+    dtype: :func:`rmsnorm` for a residual stream that stays in 32 bits."""
+    if not residual.is_cuda:
+        if delta is not None:
+            residual += delta.float()
+        return _rmsnorm_ref(residual, weight, eps).to(weight.dtype)
+    T, H = residual.shape
+    y = torch.empty((T, H), dtype=weight.dtype, device=residual.device)
+    rc = _lib.fn("vb_add_rmsnorm")(_lib.ptr(delta), 0 if delta is None else delta.stride(0), residual.data_ptr(),
+                                   weight.data_ptr(), y.data_ptr(), T, H, float(eps), int(weight.dtype == torch.float32),
+                                   _lib.stream())
+    _lib.check(rc, "vb_add_rmsnorm")
+    return y
+
+
+def clamped_glu(gate_up: torch.Tensor, ff: int, limit: float, alpha: float) -> torch.Tensor:
+    """``gate_up`` rows hold [gate (ff) | up (ff) | padding]. With g = min(gate, limit), u = clamp(up, -limit, limit):
+    ``g * sigmoid(alpha * g) * (u + 1)`` [T, ff]."""
+    if not gate_up.is_cuda:
+        g = gate_up[:, :ff].float().clamp(max=limit)
+        u = gate_up[:, ff : 2 * ff].float().clamp(-limit, limit)
+        return (g * torch.sigmoid(alpha * g) * (u + 1)).to(gate_up.dtype)
+    T = gate_up.shape[0]
+    y = torch.empty((T, ff), dtype=gate_up.dtype, device=gate_up.device)
+    rc = _lib.fn("vb_clamped_glu")(gate_up.data_ptr(), gate_up.stride(0), y.data_ptr(), T, ff, float(limit), float(alpha),
+                                   int(gate_up.dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "vb_clamped_glu")
+    return y

@@ -4,10 +4,11 @@ Replaces the vLLM / SGLang servers the reference launches (verl/workers/rollout/
 vllm_async_server.py, sglang_rollout/*). The scheduler and block manager are C++
 (``csrc/scheduler.cpp``); the model runner executes the same transformer weights as the training
 engine with the hand-written kernels: prefill = packed varlen attention + KV-cache write, decode =
-paged-KV attention, one CUDA graph per padded batch size, sampling fused into one kernel that also
+paged-KV attention (layer-list models: every mixer works on the ragged step against its pages or its state), one CUDA graph per padded batch size, sampling fused into one kernel that also
 returns the log-prob of the sampled token (what the trainer stores as ``rollout_log_probs``).
 
 Token-in / token-out API: :meth:`add_request`, :meth:`step`, :meth:`generate`, :meth:`abort_request`,
+:meth:`feed` (given tokens in, logits out: replays),
 :meth:`sleep` / :meth:`wake_up` (drop / re-create the KV cache), :meth:`update_weights`.
 """
 
@@ -26,6 +27,7 @@ import torch
 from .. import ops
 from ..models import CausalLM, ModelConfig
 from ..models.hf_io import hf_to_native_state_dict
+from ..models.hybrid import RaggedBatch, StateCache
 from ..ops import _lib
 
 
@@ -94,6 +96,8 @@ def _sched_lib():
         lib.vb_sched_stats.argtypes, lib.vb_sched_stats.restype = [P, P], None
         lib.vb_sched_reserve_burst.argtypes, lib.vb_sched_reserve_burst.restype = [P, I], I
         lib.vb_sched_commit_burst.argtypes, lib.vb_sched_commit_burst.restype = [P, P, I, P, P, P], None
+        lib.vb_sched_feed.argtypes, lib.vb_sched_feed.restype = [P, I, P, P, P], I
+        lib.vb_sched_step_slots.argtypes, lib.vb_sched_step_slots.restype = [P, P], None
         lib.vb_sched_step_limits.argtypes, lib.vb_sched_step_limits.restype = [P, P], None
         lib._sched_bound = True
     return lib
@@ -121,6 +125,7 @@ class Scheduler:
         self.done = np.zeros(cap_s, np.int32)
         self.accepted = np.zeros(cap_s, np.int32)
         self.limits = np.zeros(cap_s, np.int32)
+        self.state_slots = np.full(cap_s, -1, np.int32)
 
     def __del__(self):
         try:
@@ -157,6 +162,23 @@ class Scheduler:
         if got > 1:
             self._fetch()
         return got
+
+    _FEED_ERRORS = {-1: "a request twice in one step, an empty entry, or more tokens than a step may hold",
+                    -2: "a sequence longer than max_model_len", -3: "more live requests than max_num_seqs",
+                    -4: "not enough free cache pages"}
+
+    def feed(self, sids: list[int], chunks: list[list[int]]) -> tuple[int, int]:
+        """Plan a step of exactly these tokens (new sequences start here). Returns (sequences, tokens)."""
+        ids, counts = np.asarray(sids, np.int64), np.asarray([len(c) for c in chunks], np.int32)
+        toks = np.asarray([t for c in chunks for t in c], np.int32)
+        rc = self.lib.vb_sched_feed(self.h, len(sids), ids.ctypes.data, counts.ctypes.data, toks.ctypes.data)
+        if rc:
+            raise ValueError(f"step refused: {self._FEED_ERRORS.get(rc, rc)}")
+        return len(sids), self._fetch()
+
+    def step_state_slots(self, n: int) -> np.ndarray:
+        self.lib.vb_sched_step_slots(self.h, self.state_slots.ctypes.data)
+        return self.state_slots[:n]
 
     def step_limits(self, n: int) -> np.ndarray:
         self.lib.vb_sched_step_limits(self.h, self.limits.ctypes.data)
@@ -233,7 +255,8 @@ class NativeRolloutEngine:
         self.max_model_len = max_model_len
         self.max_num_batched_tokens = max(max_num_batched_tokens, 16)
         self.block_size = block_size
-        self.enable_prefix_caching = enable_prefix_caching
+        # pages of a shared prefix say nothing about the recurrent state behind it
+        self.enable_prefix_caching = enable_prefix_caching and not self.cfg.has_recurrent_state
         # mixture-of-experts models: keep, per request, the experts every INPUT token was routed to in every layer
         # (``TokenOutput.routed_experts [prompt + response tokens, layers, top-k]``; the trainer replays them, router
         # replay mode R3). Tokens served from the prefix cache are never routed, so the cache is off while recording.
@@ -249,16 +272,23 @@ class NativeRolloutEngine:
         self.k_cache: list = []
         self._kv_store = None  # one allocation behind the per-layer K / V views
         self.v_cache: list = []
+        self.state_cache: Optional[StateCache] = None  # layer-list models: pages and recurrent state per layer
+        self.embed_itemsize = self.dtype.itemsize
         self.sched: Optional[Scheduler] = None
         self.requests: dict[int, _Request] = {}
         self._mmreq: dict[int, dict] = {}  # per-request multimodal state of vision-language models
         self.by_rid: dict[str, int] = {}
+        self._fed: dict[str, int] = {}  # requests whose tokens the caller brings (feed)
         self._next_sid = 0
         self._graphs: dict[int, tuple] = {}
         self._capture_sizes = cudagraph_capture_sizes
         self.step_counter = torch.zeros(1, dtype=torch.long, device=self.device)
         self.stats = {"steps": 0, "prefill_tokens": 0, "decode_tokens": 0, "decode_steps": 0, "step_s": 0.0,
                       "decode_wait_s": 0.0, "prefill_s": 0.0}
+        if self.cfg.is_layer_list:
+            if self.tp > 1:
+                raise NotImplementedError(f"{self.cfg.model_type}: layer-list models run on one GPU per replica")
+            self.model.refresh()
         if self.tp > 1 and self.on_gpu:
             if tp_comm is None:
                 raise ValueError("a tensor-parallel rollout replica on CUDA needs its peer-memory communicator (tp_comm)")
@@ -275,6 +305,8 @@ class NativeRolloutEngine:
     # ----------------------------------------------------------------- memory
     def _page_bytes(self) -> int:
         c = self.cfg
+        if c.is_layer_list:
+            return max(StateCache.page_bytes(c, self.block_size, self.embed_itemsize), 1)
         return 2 * c.num_hidden_layers * c.num_key_value_heads * self.block_size * c.head_dim * 2
 
     def wake_up(self, tags: Optional[list] = None):
@@ -282,13 +314,15 @@ class NativeRolloutEngine:
         reference's multi-stage wake-up; weights are owned by the caller, so only "kv_cache" acts here."""
         if tags is not None and "kv_cache" not in tags:
             return
-        if self.sched is not None and self.k_cache:
+        if self.sched is not None and (self.k_cache or self.state_cache is not None):
             return
         if self._num_blocks_arg is not None:
             nb = self._num_blocks_arg
         elif self.on_gpu:
             free, total = torch.cuda.mem_get_info(self.device)
             budget = int(min(free * 0.9, total * self.gpu_memory_utilization))
+            if self.cfg.is_layer_list:
+                budget -= self.max_num_seqs * StateCache.slot_bytes(self.cfg, self.embed_itemsize)
             nb = max(budget // self._page_bytes(), 64)
             nb = min(nb, self.max_num_seqs * ((self.max_model_len + self.block_size - 1) // self.block_size) + 64)
         else:
@@ -301,6 +335,16 @@ class NativeRolloutEngine:
             nb = int(t.item())
         self.num_blocks = int(nb)
         c = self.cfg
+        if c.is_layer_list:
+            self.state_cache = StateCache(c, self.num_blocks, self.block_size, self.max_num_seqs, self.dtype, self.device)
+        else:
+            self._alloc_kv_pages()
+        self.sched = Scheduler(self.num_blocks, self.block_size, self.max_num_seqs, self.max_num_batched_tokens,
+                               self.max_model_len, self.enable_prefix_caching)
+        self._graphs = {}
+
+    def _alloc_kv_pages(self):
+        c = self.cfg
         shape = (self.num_blocks, c.num_key_value_heads, self.block_size, c.head_dim)
         # ONE allocation for the K and V pages of all layers: freeing it on sleep() is one driver call instead of one
         # per layer and side (with peer access enabled every cudaFree of a large block is expensive)
@@ -308,15 +352,14 @@ class NativeRolloutEngine:
         self._kv_store = torch.zeros((2 * L,) + shape, dtype=self.dtype, device=self.device)
         self.k_cache = [self._kv_store[i] for i in range(L)]
         self.v_cache = [self._kv_store[L + i] for i in range(L)]
-        self.sched = Scheduler(self.num_blocks, self.block_size, self.max_num_seqs, self.max_num_batched_tokens,
-                               self.max_model_len, self.enable_prefix_caching)
-        self._graphs = {}
 
     def sleep(self):
         """Free the KV cache (and captured graphs). Running requests must have been drained or aborted."""
         self.abort_all_requests()
+        self._fed = {}
         self.k_cache, self.v_cache, self._graphs = [], [], {}
         self._kv_store = None
+        self.state_cache = None
         self.sched = None
         if self.on_gpu:
             torch.cuda.empty_cache()
@@ -340,6 +383,8 @@ class NativeRolloutEngine:
         for k, v in native.items():
             if k in own:
                 own[k].data.copy_(v.to(own[k].dtype))
+        if self.cfg.is_layer_list:
+            self.model.refresh()
         self.refresh_quantization()
         self.clear_kv_cache()
 
@@ -479,6 +524,10 @@ class NativeRolloutEngine:
 
         # routed experts (no grouped fp8 GEMM) and the two-matrix xIELU MLP stay in bf16: for those models the
         # attention projections alone are quantised
+        if self.cfg.is_layer_list:
+            for w in self.model.projection_weights():
+                self._fp8[id(w)] = fp8.quantize_weight(w.data)
+            return
         dense_mlp = not self.cfg.is_moe and self.cfg.mlp_gated
         for layer in self.model.layers:
             ws = [layer.self_attn.qkv_proj.weight, layer.self_attn.o_proj.weight]
@@ -588,7 +637,9 @@ class NativeRolloutEngine:
 
     # ------------------------------------------------------------------ decode
     @torch.no_grad()
-    def _decode_forward(self, ids, positions, slots, block_table, seq_lens, splits, work):
+    def _decode_forward(self, ids, positions, slots, block_table, seq_lens, splits, work, ragged=None):
+        if self.cfg.is_layer_list:
+            return self._final_logits(self.model.run(ids, ragged, self.state_cache, self._mm))
         h = ops.embedding(ids, self.model.embed_tokens.weight)
 
         def attend(li, layer, x):
@@ -621,6 +672,8 @@ class NativeRolloutEngine:
                   ("lens", np.int32, (B,), 1), ("temp", np.float32, (B,), 1.0), ("topk", np.int32, (B,), -1),
                   ("topp", np.float32, (B,), 1.0), ("limit", np.int32, (B,), 0), ("alive", np.int32, (B,), 0),
                   ("flags", np.int32, (B,), 0), ("bpos", np.int32, (1,), 0), ("bt", np.int32, (B, mb), 0)]
+        if c.is_layer_list:
+            fields.append(("state", np.int32, (B,), -1))
         off, layout = 0, {}
         for name, dt, shape, _ in fields:
             nb = int(np.prod(shape)) * np.dtype(dt).itemsize
@@ -658,9 +711,14 @@ class NativeRolloutEngine:
                                             self.max_model_len, dev)
         st["splits"], st["work"] = splits, work
         eos = -1 if self.eos is None else int(self.eos)
+        ragged = None
+        if c.is_layer_list:  # one token per sequence
+            ragged = RaggedBatch(torch.arange(B + 1, dtype=torch.int32, device=dev), 1, st["lens"], st["slots"], st["bt"],
+                                 st["state"], self.max_model_len)
 
         def run():
-            logits = self._decode_forward(st["ids"], st["pos"], st["slots"], st["bt"], st["lens"], splits, work)
+            logits = self._decode_forward(st["ids"], st["pos"], st["slots"], st["bt"], st["lens"], splits, work, ragged)
+            st["logits"] = logits  # kept: feed() reads them after a replay
             if self.record_routing:  # before decode_advance moves the burst position on
                 st["ring_rt"].index_copy_(0, st["bpos"].long(), self._routing_snapshot().unsqueeze(0))
             ops.sample(logits, temperature=st["temp"], top_k=st["topk"], top_p=st["topp"], seed=self.seed,
@@ -708,6 +766,9 @@ class NativeRolloutEngine:
     @torch.no_grad()
     def _prefill_forward(self, seq_idx: list[int], tok_lo: list[int]):
         """Run the scheduled prefill chunks. Returns logits [num_prefill_seqs, V] at each chunk's last token."""
+        if self.cfg.is_layer_list:
+            last = np.cumsum([int(self.sched.seq_ntok[i]) for i in seq_idx]) - 1
+            return self._ragged_forward(seq_idx, tok_lo, last)
         sc, c, dev = self.sched, self.cfg, self.device
         ids_l, pos_l, slot_l, cu, ctx_lens = [], [], [], [0], []
         for i, lo in zip(seq_idx, tok_lo):
@@ -794,7 +855,108 @@ class NativeRolloutEngine:
         last = torch.tensor([b - 1 for b in cu[1:]], dtype=torch.long, device=dev)
         return self._final_logits(x[last])
 
+    @torch.no_grad()
+    def _ragged_forward(self, seq_idx: list[int], tok_lo: list[int], rows) -> torch.Tensor:
+        """Layer-list models: one forward over the planned tokens of the given sequences, prompt portions and single
+        tokens together. Returns logits [len(rows), V] at the token rows ``rows`` of this step."""
+        sc, dev = self.sched, self.device
+        counts = [int(sc.seq_ntok[i]) for i in seq_idx]
+        tok = np.concatenate([np.arange(lo, lo + n) for lo, n in zip(tok_lo, counts)])
+        cu = np.concatenate([[0], np.cumsum(counts)])
+        si = np.asarray(seq_idx)
+        ctx = int(sc.seq_total[si].max())
+        nb = (ctx + self.block_size - 1) // self.block_size
+        # one staging copy: int64 fields, then int32 fields
+        wide = [sc.tokens[tok], sc.slots[tok], np.asarray(rows, np.int64)]
+        narrow = [cu, sc.seq_total[si], sc.step_state_slots(int(si.max()) + 1)[si], sc.block_tables[si, :nb].ravel()]
+        buf = np.concatenate([np.concatenate(wide).astype(np.int64).view(np.int32),
+                              np.concatenate(narrow).astype(np.int32)])
+        d = torch.from_numpy(buf).to(dev)
+        T, B, R = len(tok), len(seq_idx), len(wide[2])
+        w = d[: 2 * (2 * T + R)].view(torch.int64)
+        x = d[2 * (2 * T + R) :]
+        batch = RaggedBatch(x[: B + 1], max(counts), x[B + 1 : 2 * B + 1], w[T : 2 * T], x[3 * B + 1 :].view(B, nb),
+                            x[2 * B + 1 : 3 * B + 1], ctx)
+        h = self.model.run(w[:T], batch, self.state_cache, self._mm, observe=getattr(self, "observe_layers", None))
+        return self._final_logits(h[w[2 * T :]]) if R else h.new_zeros((0, self.cfg.vocab_size), dtype=torch.float32)
+
     # -------------------------------------------------------------------- step
+    def _run_decode_batch(self, dec: list[int], tok_lo: list[int], steps: int, sps: list):
+        """Launch ``steps`` decode steps of the planned sequences ``dec`` (CUDA graph of the padded batch size)."""
+        sc, nd = self.sched, len(dec)
+        st, graph, run = self._get_graph(self._pad_batch(nd))
+        di = np.asarray(dec)
+        sids_d = sc.seq_ids[di]
+        t_idx = np.asarray([tok_lo[i] for i in dec])
+        hp, pad = st["host"], st["pad"]
+        sig = (nd, sids_d.tobytes())
+        fresh = st["sig"] != sig  # batch membership changed: rewrite the padding and the per-request constants
+        dec_pos = sc.positions[t_idx]
+        if self._mmreq:  # after its images a request's text positions are offset (all three RoPE axes are equal then)
+            dec_pos = dec_pos + np.asarray([self._mmreq.get(int(sid), {}).get("delta", 0) for sid in sids_d])
+        cols = [("ids", sc.tokens[t_idx]), ("pos", dec_pos), ("slots", sc.slots[t_idx]), ("bt", sc.block_tables[di]),
+                ("lens", sc.seq_total[di])]
+        if self.cfg.is_layer_list:
+            cols.append(("state", sc.step_state_slots(int(di.max()) + 1)[di]))
+        for name, arr in cols:
+            hp[name][:nd] = arr
+            if fresh:
+                hp[name][nd:] = pad[name]
+        if fresh:
+            for name, vals in (("temp", [p.temperature for p in sps]), ("topk", [p.top_k for p in sps]),
+                               ("topp", [p.top_p for p in sps]), ("flags", [int(p.ignore_eos) for p in sps]),
+                               ("limit", sc.step_limits(int(di.max()) + 1)[di]), ("alive", 1)):
+                hp[name][:nd] = vals
+                hp[name][nd:] = pad[name]
+            st["sig"] = sig
+        st["dev_buf"].copy_(st["host_buf"], non_blocking=True)
+        for _ in range(steps):
+            if graph is not None:
+                graph.replay()
+            else:
+                run()
+        return st, t_idx
+
+    @torch.no_grad()
+    def feed(self, entries: list[tuple[str, list[int], list[int]]], end: Iterable[str] = ()) -> Optional[torch.Tensor]:
+        """One step of given tokens: ``entries`` = (request id, its next tokens, the places among them whose logits are
+        wanted). A request is admitted at its first entry and keeps its pages and state until it is named in ``end`` (after
+        the step). All entries run as one batch, through the same paths as generation: single tokens of running requests
+        as a decode step, anything else as one ragged forward. Returns fp32 logits [wanted, V] in order, or None. Does
+        not mix with :meth:`step`: generation requests must have finished."""
+        if not self.cfg.is_layer_list:
+            raise NotImplementedError("feed() serves layer-list models")
+        if self.requests.keys() - self._fed.values():
+            raise RuntimeError("feed() cannot run while generation requests are unfinished")
+        if self.sched is None:
+            self.wake_up()
+        out = None
+        if entries:
+            sids = [self._fed.get(rid, self._next_sid + i) for i, (rid, _, _) in enumerate(entries)]
+            n, T = self.sched.feed(sids, [list(t) for _, t, _ in entries])
+            for sid, (rid, toks, _) in zip(sids, entries):
+                if rid not in self._fed:
+                    self._fed[rid] = sid
+                    self.requests[sid] = _Request(rid, sid, SamplingParams(temperature=0.0, ignore_eos=True), len(toks))
+                    self.by_rid[rid] = sid
+            self._next_sid += len(entries)
+            counts = [len(t) for _, t, _ in entries]
+            lo = np.concatenate([[0], np.cumsum(counts)])[:-1]
+            rows = [int(a) + int(w) for a, (_, _, want) in zip(lo, entries) for w in want]
+            if not self.sched.seq_prefill[:n].any():
+                st, _ = self._run_decode_batch(list(range(n)), lo.tolist(), 1, [self.requests[s].params for s in sids])
+                out = st["logits"][rows] if rows else None
+            else:
+                logits = self._ragged_forward(list(range(n)), lo.tolist(), rows)
+                out = logits if rows else None
+            self.sched.commit(np.full(n, -1, np.int64), np.zeros(n, np.int32))
+        for rid in end:
+            sid = self._fed.pop(rid)
+            self.requests.pop(sid)
+            self.by_rid.pop(rid)
+            self.sched.remove(sid)
+        return out
+
     @torch.no_grad()
     def step(self) -> list[TokenOutput]:
         """One scheduler iteration. Returns the requests that finished in it."""
@@ -810,45 +972,21 @@ class NativeRolloutEngine:
             lo += int(sc.seq_ntok[i])
         dec = [i for i in range(n) if not sc.seq_prefill[i]]
         pre = [i for i in range(n) if sc.seq_prefill[i]]
+        if pre and self.cfg.is_layer_list:  # decoding sequences join the prompt portions in one ragged forward
+            dec, pre = [], list(range(n))
         new_tokens = np.full(n, -1, np.int64)
         new_lps = np.zeros(n, np.float32)
         dev = self.device
         burst = None
         if dec:
             nd = len(dec)
-            B = self._pad_batch(nd)
-            st, graph, run = self._get_graph(B)
             di = np.asarray(dec)
             sids_d = sc.seq_ids[di]
             sps = [self.requests[int(sid)].params for sid in sids_d]
             k = 1
             if not pre and self.decode_burst > 1 and not any(p.stop_token_ids for p in sps):
                 k = sc.reserve_burst(self.decode_burst)
-            t_idx = np.asarray([tok_lo[i] for i in dec])
-            hp, pad = st["host"], st["pad"]
-            sig = (nd, sids_d.tobytes())
-            fresh = st["sig"] != sig  # batch membership changed: rewrite the padding and the per-request constants
-            dec_pos = sc.positions[t_idx]
-            if self._mmreq:  # after its images a request's text positions are offset (all three RoPE axes are equal then)
-                dec_pos = dec_pos + np.asarray([self._mmreq.get(int(sid), {}).get("delta", 0) for sid in sids_d])
-            for name, arr in (("ids", sc.tokens[t_idx]), ("pos", dec_pos), ("slots", sc.slots[t_idx]),
-                              ("bt", sc.block_tables[di]), ("lens", sc.seq_total[di])):
-                hp[name][:nd] = arr
-                if fresh:
-                    hp[name][nd:] = pad[name]
-            if fresh:
-                for name, vals in (("temp", [p.temperature for p in sps]), ("topk", [p.top_k for p in sps]),
-                                   ("topp", [p.top_p for p in sps]), ("flags", [int(p.ignore_eos) for p in sps]),
-                                   ("limit", sc.step_limits(n)[di]), ("alive", 1)):
-                    hp[name][:nd] = vals
-                    hp[name][nd:] = pad[name]
-                st["sig"] = sig
-            st["dev_buf"].copy_(st["host_buf"], non_blocking=True)
-            for _ in range(k):
-                if graph is not None:
-                    graph.replay()
-                else:
-                    run()
+            st, t_idx = self._run_decode_batch(dec, tok_lo, k, sps)
             st["out_host"].copy_(st["out_dev"], non_blocking=True)
             if self.record_routing:
                 st["rt_host"].copy_(st["ring_rt"], non_blocking=True)

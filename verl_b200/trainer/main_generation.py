@@ -32,7 +32,7 @@ DEFAULTS = {
 
 def run_generation(config) -> list[dict]:
     from ..rollout import NativeRolloutEngine, SamplingParams
-    from ..models.transformer import CausalLM
+    from ..models import build_model
     from ..utils.dataset.rl_dataset import _read_rows
     from ..workers.engine_workers import resolve_model_config
     from .main_ppo import build_tokenizer
@@ -41,7 +41,7 @@ def run_generation(config) -> list[dict]:
     model_cfg, state = resolve_model_config(config.model)
     tok = build_tokenizer(config.model, model_cfg)
     dtype = torch.bfloat16 if dev.type == "cuda" else torch.float32
-    model = CausalLM(model_cfg, dtype=dtype, device=dev)
+    model = build_model(model_cfg, dtype=dtype, device=dev, init=False)
     if state is not None:
         model.load_state_dict({k: v.to(dtype) for k, v in state.items()}, strict=False)
     else:

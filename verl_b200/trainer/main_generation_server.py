@@ -27,7 +27,7 @@ DEFAULTS["rollout"].update(num_replicas=1, server_address="127.0.0.1", max_concu
 
 
 def _engine_factory(config, dev):
-    from ..models.transformer import CausalLM
+    from ..models import build_model
     from ..rollout import NativeRolloutEngine
     from ..workers.engine_workers import resolve_model_config
 
@@ -36,7 +36,7 @@ def _engine_factory(config, dev):
     rc = config.rollout
 
     def build():
-        model = CausalLM(model_cfg, dtype=dtype, device=dev)
+        model = build_model(model_cfg, dtype=dtype, device=dev, init=False)
         if state is not None:
             model.load_state_dict({k: v.to(dtype) for k, v in state.items()}, strict=False)
         else:
