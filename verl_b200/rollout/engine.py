@@ -946,6 +946,8 @@ class NativeRolloutEngine:
             if not self.sched.seq_prefill[:n].any():
                 st, _ = self._run_decode_batch(list(range(n)), lo.tolist(), 1, [self.requests[s].params for s in sids])
                 out = st["logits"][rows] if rows else None
+                if self.on_gpu:  # the pinned step description is rewritten by the next step
+                    torch.cuda.current_stream(self.device).synchronize()
             else:
                 logits = self._ragged_forward(list(range(n)), lo.tolist(), rows)
                 out = logits if rows else None
