@@ -207,6 +207,27 @@ __global__ void decode_merge_kernel(const float* __restrict__ o_part, const floa
   out[(long long)b * out_stride + (long long)hq * D + d] = __float2bfloat16(l > 0.f ? o / l : 0.f);
 }
 
+// The same for any head size: one warp per (sequence, query head).
+__global__ void decode_merge_any_kernel(const float* __restrict__ o_part, const float* __restrict__ ml_part, int Hq, int D,
+                                        int num_splits, __nv_bfloat16* __restrict__ out, long long out_stride) {
+  const int b = blockIdx.x, hq = blockIdx.y;
+  const long long base = ((long long)b * Hq + hq) * num_splits;
+  float m = -INFINITY, l = 0.f;
+  for (int s = 0; s < num_splits; ++s) m = fmaxf(m, ml_part[(base + s) * 2]);
+  for (int s = 0; s < num_splits; ++s) {
+    const float ms = ml_part[(base + s) * 2];
+    l += ms == -INFINITY ? 0.f : ml_part[(base + s) * 2 + 1] * __expf(ms - m);
+  }
+  for (int d = threadIdx.x; d < D; d += blockDim.x) {
+    float o = 0.f;
+    for (int s = 0; s < num_splits; ++s) {
+      const float ms = ml_part[(base + s) * 2];
+      if (ms != -INFINITY) o += o_part[(base + s) * D + d] * __expf(ms - m);
+    }
+    out[(long long)b * out_stride + (long long)hq * D + d] = __float2bfloat16(l > 0.f ? o / l : 0.f);
+  }
+}
+
 // k, v: [T, Hk, D] (token stride given); slot = block * block_size + offset, slot < 0 skips the token.
 __global__ void kv_write_kernel(const __nv_bfloat16* __restrict__ k, const __nv_bfloat16* __restrict__ v,
                                 long long k_stride, long long v_stride, const long long* __restrict__ slots,
@@ -250,6 +271,13 @@ int vb_decode_merge_128(const float* o_part, const float* ml_part, int B, int Hq
                         long long out_stride, cudaStream_t stream) {
   decode_merge_kernel<128><<<dim3(B, Hq), 128, 0, stream>>>(o_part, ml_part, Hq, num_splits, (__nv_bfloat16*)out,
                                                             out_stride);
+  return (int)cudaGetLastError();
+}
+
+int vb_decode_merge(const float* o_part, const float* ml_part, int B, int Hq, int D, int num_splits, void* out,
+                    long long out_stride, cudaStream_t stream) {
+  decode_merge_any_kernel<<<dim3(B, Hq), D <= 64 ? 64 : 128, 0, stream>>>(o_part, ml_part, Hq, D, num_splits,
+                                                                          (__nv_bfloat16*)out, out_stride);
   return (int)cudaGetLastError();
 }
 

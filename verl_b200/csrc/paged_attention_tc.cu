@@ -16,6 +16,11 @@
 //                one CTA's softmax chain overlaps the other's loads and MMAs
 //   warp 5     : TMEM allocation + single-thread tcgen05.mma issue
 //
+// The EXT variant serves layer-list decoders: head sizes up to 128 with separate key and value sizes (TMA fills the
+// missing columns with zeros), a sliding window with kept first keys (only the chunks in sight are visited), a
+// per-distance bias, and weights that stay close to fp32: with up to 8 query heads per KV head, rows G .. 2G-1 of the
+// P operand hold the remainders that rounding the weights to bf16 leaves, and their products are added.
+//
 // V needs no transpose: [keys, dims] with dims contiguous is exactly an "MN-major" A operand.
 // All waits are bounded; on expiry the status word is set and the CTA leaves through its teardown.
 #include "common.cuh"
@@ -53,7 +58,29 @@ struct DecodeTcParams {
   float* o_part;
   float* ml_part;
   int* status;
+  // EXT only
+  int D, Dv, window, keep_first, bias_len;
+  const float* bias;  // [Hq, bias_len] or null
 };
+
+// Chunks a decode query at position seq_len - 1 visits: [0, keep) and [win, ...); without a window all of them.
+struct TcRange {
+  int keep, win, total;
+  __device__ __forceinline__ int at(int c) const { return c < keep ? c : win + c - keep; }
+};
+template <bool EXT>
+__device__ __forceinline__ TcRange tc_range(const DecodeTcParams& p, int seq_len) {
+  TcRange r;
+  const int chunks = (seq_len + TC_CHUNK - 1) / TC_CHUNK;
+  r.keep = 0;
+  r.win = 0;
+  if (EXT && p.window > 0) {
+    r.keep = min((p.keep_first + TC_CHUNK - 1) / TC_CHUNK, chunks);
+    r.win = max(max(seq_len - p.window, 0) / TC_CHUNK, r.keep);
+  }
+  r.total = r.keep + max(chunks - r.win, 0);
+  return r;
+}
 
 // byte offset of element (row r, col k) inside a K-major, 128-byte-swizzled operand of `rows` rows whose
 // k extent is split in 64-element blocks of rows*128 bytes
@@ -377,7 +404,9 @@ constexpr int TCP_SMEM = TCP_RED_OFF + 2 * TC_NH * 4 * 4 + 1024;
 
 struct TcItem {
   int b, h, split, seq_len, c_begin, n_chunks;
+  TcRange range;
 };
+template <bool EXT>
 __device__ __forceinline__ TcItem tc_item(const DecodeTcParams& p, int item) {
   TcItem it;
   it.split = item % p.num_splits;
@@ -385,13 +414,15 @@ __device__ __forceinline__ TcItem tc_item(const DecodeTcParams& p, int item) {
   it.h = bh % p.Hk;
   it.b = bh / p.Hk;
   it.seq_len = p.seq_lens[it.b];
-  const int chunks_total = (it.seq_len + TC_CHUNK - 1) / TC_CHUNK;
+  it.range = tc_range<EXT>(p, it.seq_len);
+  const int chunks_total = it.range.total;
   const int per_split = (chunks_total + p.num_splits - 1) / p.num_splits;
   it.c_begin = it.split * per_split;
   it.n_chunks = max(min(chunks_total, it.c_begin + per_split) - it.c_begin, 0);
   return it;
 }
 
+template <bool EXT>
 __global__ void __launch_bounds__(TC_THREADS, 2)
 paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                                const DecodeTcParams p, const int num_items) {
@@ -414,6 +445,7 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
   float (*red2_s)[4] = reinterpret_cast<float (*)[4]>(smem + TCP_RED_OFF + TC_NH * 16);
 
   const int G = p.Hq / p.Hk;
+  const int D = EXT ? p.D : TC_D, Dv = EXT ? p.Dv : TC_D;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int pages_per_chunk = TC_CHUNK / p.block_size;
 
@@ -455,7 +487,7 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
     uint32_t tg = 0, ig = 0;
     bool ok = true;
     for (int item = blockIdx.x; ok && item < num_items; item += gridDim.x) {
-      const TcItem it = tc_item(p, item);
+      const TcItem it = tc_item<EXT>(p, item);
       if (it.n_chunks <= 0) continue;
       const int qb = 0;
       // the Q operand is free once the QK MMAs of the previous item have completed
@@ -470,11 +502,11 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
       good = __shfl_sync(0xffffffffu, good, 0);
       if (!good) break;
       {
-        const __nv_bfloat16* qrow = p.q + (long long)it.b * p.q_stride + (long long)it.h * G * TC_D;
+        const __nv_bfloat16* qrow = p.q + (long long)it.b * p.q_stride + (long long)it.h * G * D;
         uint8_t* qdst = q_s + qb * Q_BYTES;
-        for (int idx = lane; idx < G * (TC_D / 8); idx += 32) {
-          const int g = idx / (TC_D / 8), c8 = idx % (TC_D / 8);
-          const uint4 v = *reinterpret_cast<const uint4*>(qrow + g * TC_D + c8 * 8);
+        for (int idx = lane; idx < G * (D / 8); idx += 32) {
+          const int g = idx / (D / 8), c8 = idx % (D / 8);
+          const uint4 v = *reinterpret_cast<const uint4*>(qrow + g * D + c8 * 8);
           *reinterpret_cast<uint4*>(qdst + sw128_off(g, c8 * 8, TC_NH)) = v;
         }
         fence_proxy_async_smem();
@@ -482,11 +514,14 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
         if (lane == 0) mbar_arrive(&q_full[qb]);
       }
       const int n_pages = (it.seq_len + p.block_size - 1) / p.block_size;
-      const int page_base = it.c_begin * pages_per_chunk;
       const int* bt = p.block_table + (long long)it.b * p.max_blocks;
-      const int cnt = min(min(it.n_chunks * pages_per_chunk, n_pages - page_base), TC_BT_MAX);
+      const int cnt = min(it.n_chunks * pages_per_chunk, TC_BT_MAX);
+      // page of the item's i-th one; pages past the end of the sequence re-read its last page (masked later)
+      auto page_at = [&](int i) {
+        return min(it.range.at(it.c_begin + i / pages_per_chunk) * pages_per_chunk + i % pages_per_chunk, n_pages - 1);
+      };
       __syncwarp();
-      for (int i = lane; i < cnt; i += 32) bt_s[i] = bt[page_base + i];
+      for (int i = lane; i < cnt; i += 32) bt_s[i] = bt[page_at(i)];
       __syncwarp();
       if (lane == 0) {
         for (int t = 0; t < 2 * it.n_chunks; ++t, ++tg) {
@@ -501,11 +536,9 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
           mbar_arrive_expect_tx(&full[s], STAGE_BYTES_TC);
           uint8_t* dst = stage0 + s * STAGE_BYTES_TC;
           const CUtensorMap* tm = (t & 1) ? &tmV : &tmK;
-          const int page0 = (it.c_begin + (t >> 1)) * pages_per_chunk;
           for (int pg = 0; pg < pages_per_chunk; ++pg) {
-            const int pi = min(page0 + pg, n_pages - 1);
-            const int rel = pi - page_base;
-            const int blk = rel < TC_BT_MAX ? bt_s[rel] : bt[pi];
+            const int rel = (t >> 1) * pages_per_chunk + pg;
+            const int blk = rel < TC_BT_MAX ? bt_s[rel] : bt[page_at(rel)];
             const int row = (blk * p.Hk + it.h) * p.block_size;
             const int off = pg * p.block_size * 128;
             tma_load_2d(dst + off, tm, &full[s], 0, row);
@@ -525,7 +558,7 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
       uint32_t tg = 0, cg = 0, ig = 0;
       bool ok = true;
       for (int item = blockIdx.x; ok && item < num_items; item += gridDim.x) {
-        const TcItem it = tc_item(p, item);
+        const TcItem it = tc_item<EXT>(p, item);
         if (it.n_chunks <= 0) continue;
         const int qb = 0;
         if (*abort_flag || !mbar_wait(&q_full[qb], ig & 1)) {
@@ -599,7 +632,7 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
     bool ok = true;
     uint32_t cg = 0;
     for (int item = blockIdx.x; ok && item < num_items; item += gridDim.x) {
-      const TcItem it = tc_item(p, item);
+      const TcItem it = tc_item<EXT>(p, item);
       float m_run[TC_NH], l_run[TC_NH], o_acc[TC_NH];
 #pragma unroll
       for (int g = 0; g < TC_NH; ++g) {
@@ -626,12 +659,17 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
 #pragma unroll
           for (int g = 0; g < 16; ++g) sr[g] = 0;
         }
-        const int key = (it.c_begin + c) * TC_CHUNK + tid;
-        const bool valid = key < it.seq_len;
+        const int key = it.range.at(it.c_begin + c) * TC_CHUNK + tid;
+        const int dist = it.seq_len - 1 - key;
+        const bool valid = dist >= 0 && (!EXT || p.window <= 0 || dist < p.window || key < p.keep_first);
+        const float* brow = EXT && p.bias != nullptr
+                                ? p.bias + (long long)it.h * G * p.bias_len + max(min(dist, p.bias_len - 1), 0)
+                                : nullptr;
         float sc[TC_NH];
 #pragma unroll
         for (int g = 0; g < TC_NH; ++g) {
           sc[g] = valid ? __uint_as_float(sr[g]) * p.scale : -INFINITY;
+          if (EXT && brow != nullptr && g < G) sc[g] += __ldg(brow + g * p.bias_len);
           if (g < G) {
             const float wm = warp_reduce_max(sc[g]);
             if (lane == 0) red_s[g][warp] = wm;
@@ -648,7 +686,11 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
             alpha[g] = __expf(m_run[g] - nm);
             const float pv = valid ? __expf(sc[g] - nm) : 0.f;
             m_run[g] = nm;
-            *reinterpret_cast<__nv_bfloat16*>(pbuf + sw128_off(g, tid, TC_NH)) = __float2bfloat16(pv);
+            const __nv_bfloat16 ph = __float2bfloat16(pv);
+            *reinterpret_cast<__nv_bfloat16*>(pbuf + sw128_off(g, tid, TC_NH)) = ph;
+            if (EXT)
+              *reinterpret_cast<__nv_bfloat16*>(pbuf + sw128_off(G + g, tid, TC_NH)) =
+                  __float2bfloat16(pv - __bfloat162float(ph));
             const float ws = warp_reduce_sum(pv);
             if (lane == 0) red2_s[g][warp] = ws;
           }
@@ -681,26 +723,34 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
           tmem_ld_32x16(tmem_base + lane_base + 32 + i * TC_NH, orr);
           tmem_ld_wait();
 #pragma unroll
-          for (int g = 0; g < TC_NH; ++g)
-            if (g < G) o_acc[g] = o_acc[g] * alpha_cur[g] + __uint_as_float(orr[g]);
+          for (int g = 0; g < TC_NH; ++g) {
+            if (g >= G) continue;
+            float x = __uint_as_float(orr[g]);
+            if (EXT) {
+#pragma unroll
+              for (int k = 1; k <= TC_NH / 2; ++k)  // column G + g, without dynamic register indexing
+                if (k == G && g + k < TC_NH) x += __uint_as_float(orr[(g + k) & (TC_NH - 1)]);
+            }
+            o_acc[g] = o_acc[g] * alpha_cur[g] + x;
+          }
         }
 #pragma unroll
         for (int g = 0; g < TC_NH; ++g) alpha_cur[g] = alpha_nxt[g];
         ok = bar_and_128(ok);
       }
       cg += it.n_chunks;
-      if (ok) {
+      if (ok && tid < Dv) {
         const int d = tid;
 #pragma unroll
         for (int g = 0; g < TC_NH; ++g) {
           if (g < G) {
             const int hq = it.h * G + g;
             if (p.num_splits == 1) {
-              p.out[(long long)it.b * p.out_stride + (long long)hq * TC_D + d] =
+              p.out[(long long)it.b * p.out_stride + (long long)hq * Dv + d] =
                   __float2bfloat16(l_run[g] > 0.f ? o_acc[g] / l_run[g] : 0.f);
             } else {
               const long long base = ((long long)it.b * p.Hq + hq) * p.num_splits + it.split;
-              p.o_part[base * TC_D + d] = o_acc[g];
+              p.o_part[base * Dv + d] = o_acc[g];
               if (d == 0) {
                 p.ml_part[base * 2] = m_run[g];
                 p.ml_part[base * 2 + 1] = l_run[g];
@@ -777,11 +827,11 @@ extern "C" int vb_paged_decode_tc(const void* q, long long q_stride, const void*
   if (persist && items > 2 * vb_num_sms() && (q_stride & 7) == 0 && (reinterpret_cast<uintptr_t>(q) & 15) == 0) {
     static bool attr2_set = false;
     if (!attr2_set) {
-      VB_CUDA_CHECK(cudaFuncSetAttribute(paged_decode_tc_persist_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+      VB_CUDA_CHECK(cudaFuncSetAttribute(paged_decode_tc_persist_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          TCP_SMEM));
       attr2_set = true;
     }
-    rc = (int)vb_launch_pdl(paged_decode_tc_persist_kernel, dim3(2 * vb_num_sms()), dim3(TC_THREADS), TCP_SMEM, stream,
+    rc = (int)vb_launch_pdl(paged_decode_tc_persist_kernel<false>, dim3(2 * vb_num_sms()), dim3(TC_THREADS), TCP_SMEM, stream,
                             1, tmK, tmV, p, items);
   } else {
     dim3 grid(B, Hk, num_splits);
@@ -791,4 +841,63 @@ extern "C" int vb_paged_decode_tc(const void* q, long long q_stride, const void*
   if (rc == 0) rc = (int)cudaGetLastError();
   if (rc || num_splits == 1) return rc;
   return vb_decode_merge_128(p.o_part, p.ml_part, B, Hq, num_splits, out, out_stride, stream);
+}
+
+int vb_decode_merge(const float* o_part, const float* ml_part, int B, int Hq, int D, int num_splits, void* out,
+                    long long out_stride, cudaStream_t stream);
+
+// Returns 1 if vb_paged_decode_window supports this configuration.
+extern "C" int vb_paged_decode_window_supported(int Hq, int Hk, int D, int Dv, int block_size) {
+  return D >= 8 && D <= TC_D && Dv >= 8 && Dv <= TC_D && (D & 7) == 0 && (Dv & 7) == 0 && Hk > 0 && Hq / Hk <= TC_NH / 2 &&
+         vb_paged_decode_tc_supported(Hq, Hk, TC_D, block_size);
+}
+
+// One query token per sequence over caches [num_blocks, Hk, block_size, D | Dv] bf16, at position seq_lens[b] - 1:
+//   window > 0: key j is visible when seq_len - 1 - j < window or j < keep_first (0: every key)
+//   bias [Hq, bias_len] fp32 or null: bias[h][min(seq_len - 1 - j, bias_len - 1)] is added to the scaled score
+// work: fp32 scratch of B * Hq * num_splits * (Dv + 2) floats (unused when num_splits == 1).
+extern "C" int vb_paged_decode_window(const void* q, long long q_stride, const void* kc, const void* vc, int num_blocks,
+                                      const int* block_table, int max_blocks, const int* seq_lens, int B, int Hq, int Hk,
+                                      int D, int Dv, int block_size, float scale, int window, int keep_first,
+                                      const float* bias, int bias_len, int num_splits, void* out, long long out_stride,
+                                      float* work, int* status, cudaStream_t stream) {
+  if (B <= 0) return 0;
+  if (!vb_paged_decode_window_supported(Hq, Hk, D, Dv, block_size) || (q_stride & 7) != 0 ||
+      (reinterpret_cast<uintptr_t>(q) & 15) != 0 || num_splits < 1 || (num_splits > 1 && work == nullptr) ||
+      (bias != nullptr && bias_len <= 0))
+    return -3;
+  CUtensorMap tmK, tmV;
+  const uint64_t rows = (uint64_t)num_blocks * Hk * block_size;
+  int rc = vb_make_tmap_2d(&tmK, kc, 2, D, rows, (uint64_t)D * 2, 64, block_size);
+  if (rc) return rc;
+  rc = vb_make_tmap_2d(&tmV, vc, 2, Dv, rows, (uint64_t)Dv * 2, 64, block_size);
+  if (rc) return rc;
+  static bool attr_set = false;
+  if (!attr_set) {
+    VB_CUDA_CHECK(cudaFuncSetAttribute(paged_decode_tc_persist_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                       TCP_SMEM));
+    attr_set = true;
+  }
+  DecodeTcParams p{};
+  p.q = reinterpret_cast<const __nv_bfloat16*>(q);
+  p.q_stride = q_stride;
+  p.block_table = block_table;
+  p.max_blocks = max_blocks;
+  p.seq_lens = seq_lens;
+  p.Hq = Hq; p.Hk = Hk; p.block_size = block_size;
+  p.scale = scale;
+  p.num_splits = num_splits;
+  p.out = reinterpret_cast<__nv_bfloat16*>(out);
+  p.out_stride = out_stride;
+  p.o_part = work;
+  p.ml_part = work ? work + (long long)B * Hq * num_splits * Dv : nullptr;
+  p.status = status;
+  p.D = D; p.Dv = Dv; p.window = window; p.keep_first = keep_first; p.bias_len = bias_len; p.bias = bias;
+  const int items = B * Hk * num_splits, slots = 2 * vb_num_sms();
+  rc = (int)vb_launch_pdl(paged_decode_tc_persist_kernel<true>, dim3(items < slots ? items : slots), dim3(TC_THREADS),
+                          TCP_SMEM, stream, 1, tmK, tmV, p, items);
+  vb_count_launch(num_splits > 1 ? 2 : 1);
+  if (rc == 0) rc = (int)cudaGetLastError();
+  if (rc || num_splits == 1) return rc;
+  return vb_decode_merge(p.o_part, p.ml_part, B, Hq, Dv, num_splits, out, out_stride, stream);
 }

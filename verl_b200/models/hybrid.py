@@ -95,7 +95,7 @@ class AttentionMixer(nn.Module):
         q = ops.qk_norm_kv_write(qkv, *norms, batch.slots, cache[0], cache[1], s.heads, self.eps)
         o = ops.paged_attention(q, cache[0], cache[1], batch.block_table, batch.cu_q, batch.seq_lens, batch.max_q,
                                 scale=s.scale, window=s.window, keep_first=s.keep_first,
-                                bias=self.bias if s.bias_rows else None)
+                                bias=self.bias if s.bias_rows else None, max_ctx=batch.max_ctx)
         return mm(o, self.o_proj.weight)
 
 

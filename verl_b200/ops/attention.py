@@ -232,11 +232,16 @@ def qk_norm_kv_write(qkv: torch.Tensor, q_weight: torch.Tensor | None, k_weight:
 
 def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor,
                     cu_q: torch.Tensor, seq_lens: torch.Tensor, max_q: int, *, scale: float, window: int = 0,
-                    keep_first: int = 0, bias: torch.Tensor | None = None, impl: str = "auto") -> torch.Tensor:
+                    keep_first: int = 0, bias: torch.Tensor | None = None, max_ctx: int = 0,
+                    impl: str = "auto") -> torch.Tensor:
     """Causal attention of ragged queries (the last ``cu_q[b + 1] - cu_q[b]`` positions of every sequence) over the paged
     cache, which holds the new tokens already. q [T, Hq, D]; caches [NB, Hk, BS, D] / [NB, Hk, BS, Dv]; ``seq_lens``
     [B] = tokens of each sequence including the new ones. ``window`` > 0: position i sees j <= i with i - j < window or
-    j < keep_first. ``bias`` fp32 [Hq, L]: ``bias[h, min(i - j, L - 1)]`` is added to the scaled score. -> [T, Hq * Dv]."""
+    j < keep_first. ``bias`` fp32 [Hq, L]: ``bias[h, min(i - j, L - 1)]`` is added to the scaled score. ``max_ctx``: bound
+    of ``seq_lens``. -> [T, Hq * Dv].
+
+    ``impl``: "tc" = tcgen05 kernels (bf16, head sizes up to 128 in multiples of 8, block size a power of two in 8..128;
+    one token per sequence: up to 8 query heads per KV head), "simt" = CUDA-core kernel, "auto" = "tc" where it applies."""
     T, Hq, D = q.shape
     Hk, BS, Dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
     B = seq_lens.numel()
@@ -244,11 +249,34 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     if q.is_cuda:
         f32 = q.dtype == torch.float32
         L = 0 if bias is None else bias.shape[1]
-        rc = _lib.fn("vb_paged_attention_simt")(q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(),
-                                                block_table.data_ptr(), block_table.stride(0), cu_q.data_ptr(),
-                                                seq_lens.data_ptr(), T, B, Hq, Hk, D, Dv, BS, float(scale), window, keep_first,
-                                                _lib.ptr(bias), L, out.data_ptr(), out.stride(0), int(f32), _lib.stream())
-        _lib.check(rc, "vb_paged_attention_simt")
+        if max_q == 1:
+            tc = _lib.fn("vb_paged_decode_window_supported")(Hq, Hk, D, Dv, BS)
+        else:
+            tc = _lib.fn("vb_paged_flash_supported")(Hq, Hk, D, Dv, BS, L)
+        tc = bool(tc) and not f32 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
+        if impl == "tc" and not tc:
+            raise ValueError(f"tensor-core attention does not support Hq={Hq} Hk={Hk} D={D} Dv={Dv} block_size={BS}")
+        args = (q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr())
+        table = (block_table.data_ptr(), block_table.stride(0))
+        mask = (float(scale), window, keep_first, _lib.ptr(bias), L)
+        dst = (out.data_ptr(), out.stride(0))
+        if tc and impl != "simt" and max_q == 1:
+            seen = max_ctx or block_table.shape[1] * BS
+            if window > 0:
+                seen = min(seen, window + keep_first + 128)
+            splits = _lib.fn("vb_decode_num_splits")(B, Hk, seen)
+            work = torch.empty(B * Hq * splits * (Dv + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
+            rc = _lib.fn("vb_paged_decode_window")(*args, k_cache.shape[0], *table, seq_lens.data_ptr(), B, Hq, Hk, D, Dv, BS,
+                                                   *mask, splits, *dst, _lib.ptr(work),
+                                                   _lib.status_word(q.device).data_ptr(), _lib.stream())
+        elif tc and impl != "simt":
+            rc = _lib.fn("vb_paged_flash")(*args, k_cache.shape[0], *table, cu_q.data_ptr(), seq_lens.data_ptr(), T, B, max_q,
+                                           Hq, Hk, D, Dv, BS, *mask, *dst, _lib.status_word(q.device).data_ptr(),
+                                           _lib.stream())
+        else:
+            rc = _lib.fn("vb_paged_attention_simt")(*args, *table, cu_q.data_ptr(), seq_lens.data_ptr(), T, B, Hq, Hk, D, Dv, BS,
+                                                    *mask, *dst, int(f32), _lib.stream())
+        _lib.check(rc, "paged_attention")
         return out
     G = Hq // Hk
     cu, lens = cu_q.tolist(), seq_lens.tolist()
