@@ -68,6 +68,11 @@ def parse_args():
     ap.add_argument("--lora-rank", type=int, default=0, help="variant: LoRA training (not the headline configuration)")
     ap.add_argument("--prefix-sharing", action="store_true",
                     help="variant: the log-prob passes evaluate each prompt once for its n samples (use_prefix_grouper)")
+    ap.add_argument("--serving", default="", metavar="PRESET",
+                    help="instead of the RL step: prefill and decode throughput of this layer-list model beside --serving-vs")
+    ap.add_argument("--serving-vs", default="llama-3-8b", metavar="PRESET")
+    ap.add_argument("--serving-layers", type=int, default=6, help="layers of both models (their widths are the presets')")
+    ap.add_argument("--serving-kernels", action="store_true", help="also every kernel beside its counterpart")
     args = ap.parse_args()
     if args.prompts_per_gpu is None:
         args.prompts_per_gpu = 16 if args.config == 1 else 32
@@ -205,6 +210,11 @@ def main():
         from baseline import stock_libs
 
         stock_libs.main(args)
+        return
+    if args.serving:
+        from verl_b200.rollout import serving_bench
+
+        serving_bench.main(args)
         return
     import torch
     import torch.distributed as dist

@@ -13,8 +13,23 @@
 // read and write the ring without ordering between its blocks. A sequence whose first token has position 0 starts from
 // zero state whatever its slot holds; slot < 0 marks a padding row.
 //
-// Kernels: delta_prep (convolution, silu, unit norms, gates of every token) -> delta_scan (state carried through the
-// tokens in registers, fp32) -> gated_norm; delta_step does all of it for sequences that bring one token each.
+// Kernels:
+//   delta_step   one token per sequence: everything fused (decode)
+//   delta_prep   convolution, silu, unit norms, gates of every token, then either
+//     delta_scan   token by token, state in registers, fp32 throughout (32-bit mode, short portions, any head size), or
+//     delta_chunk_prep + delta_chunk_scan   chunks of 64 tokens on the tensor cores (bf16 serving)
+//   gated_norm   the output norm and gate
+//
+// Chunked form. With G_t the running sum of log decays inside a chunk, S0 the state in front of it and u_t the write of
+// token t, unrolling the recurrence gives
+//     u_t = beta_t (v_t - e^{G_t} S0^T k_t - sum_{s<t} e^{G_t - G_s} (k_t . k_s) u_s)       i.e. (I + A) U = B (V - ...)
+//     o_t = e^{G_t} S0^T q_t + sum_{s<=t} e^{G_t - G_s} (q_t . k_s) u_s
+//     S   = e^{G_last} S0 + sum_s e^{G_last - G_s} k_s u_s^T
+// delta_chunk_prep computes T = (I + A)^-1 B and the matrix P of the second sum for all chunks in parallel;
+// delta_chunk_scan walks a sequence's chunks with S in fp32 accumulators. Precision: the convolved q and k are bf16
+// activations and enter the products unnormalised, their fp32 unit-norm factors multiply the results; every other
+// operand (S, T, P, U and the right-hand side) is split into two bf16 terms, so that products carry about 16 bits of
+// both operands and sums are fp32.
 #include "common.cuh"
 #include "host_utils.h"
 
@@ -42,7 +57,8 @@ struct DeltaParams {
   const int* cu_q;         // [B + 1]
   const int* seq_lens;     // [B] tokens of the sequence up to and including this step's
   const int* slots;        // [B]
-  float* qkv;              // [T, C] fp32 (scan path)
+  void* qkv;               // [T, C]: fp32, unit q and k (scan path); bf16, unnormalised (chunk path)
+  float* unit;             // [T, 2 Hk] fp32 factors that make q (times D^-1/2) and k unit vectors (chunk path)
   float* gates;            // [T, 2 H] fp32: beta | log decay (scan path)
   void* out;               // [T, out_stride]
   long long out_stride;
@@ -54,7 +70,7 @@ struct DeltaParams {
 // One warp per (sequence, tile of tokens, head row); lanes across the head's channels, a sliding window of inputs in
 // registers. Head rows: Hk of q, Hk of k, H of v; one more row does the gates.
 constexpr int DP_TT = 32;  // tokens per tile
-template <typename T, int TAPS, int CPL>
+template <typename T, int TAPS, int CPL, bool CHUNK>
 __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaParams p) {
   pdl_trigger();
   pdl_wait();
@@ -109,14 +125,23 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaParams p) {
 #pragma unroll
       for (int j = TAPS - 1; j > 0; --j) hist[j][i] = hist[j - 1][i];
       y[i] = silu_f(a);
+      if (CHUNK) y[i] = __bfloat162float(__float2bfloat16(y[i]));  // the norm is that of the stored vector
       ss += y[i] * y[i];  // channels past the head give silu(0) = 0
     }
     float mul = 1.f;
     if (qk) mul = qscale / sqrtf(warp_reduce_sum(ss) + UNIT_EPS);
-    float* dst = p.qkv + (long long)(first + t) * C + c0;
+    if (CHUNK) {
+      __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.qkv) + (long long)(first + t) * C + c0;
 #pragma unroll
-    for (int i = 0; i < CPL; ++i)
-      if (lane + 32 * i < size) dst[lane + 32 * i] = y[i] * mul;
+      for (int i = 0; i < CPL; ++i)
+        if (lane + 32 * i < size) dst[lane + 32 * i] = __float2bfloat16(y[i]);
+      if (qk && lane == 0) p.unit[(long long)(first + t) * 2 * p.Hk + r] = mul;
+    } else {
+      float* dst = static_cast<float*>(p.qkv) + (long long)(first + t) * C + c0;
+#pragma unroll
+      for (int i = 0; i < CPL; ++i)
+        if (lane + 32 * i < size) dst[lane + 32 * i] = y[i] * mul;
+    }
   }
 }
 
@@ -132,6 +157,17 @@ __device__ __forceinline__ float sum8(float v) {  // over groups of eight lanes
   v += __shfl_xor_sync(0xffffffffu, v, 2);
   v += __shfl_xor_sync(0xffffffffu, v, 4);
   return v;
+}
+
+// The last convolution inputs of a sequence: its channels are dealt out over the `parts` CTAs that work on it.
+template <typename T>
+__device__ __forceinline__ void store_ring(const DeltaParams& p, int first, int n, int start, int slot, int part, int parts) {
+  const int C = 2 * p.Hk * p.D + p.H * p.V;
+  const T* proj = static_cast<const T*>(p.proj) + (long long)first * p.stride;
+  T* ring = static_cast<T*>(p.ring) + (long long)slot * p.taps * C;
+  for (int c = part * blockDim.x + threadIdx.x; c < C; c += parts * blockDim.x)
+    for (int t = max(0, n - p.taps); t < n; ++t)
+      ring[(long long)((start + t) % p.taps) * C + c] = proj[(long long)t * p.stride + c];
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -166,7 +202,7 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaParam
     const int row = 4 * (r + 8 * (i >> 2)) + (i & 3);
     S[i] = (start > 0 && col_on && row < p.D) ? st[row] : 0.f;
   }
-  const float* qkv = p.qkv + (long long)first * C;
+  const float* qkv = static_cast<const float*>(p.qkv) + (long long)first * C;
   const float* gates = p.gates + (long long)first * 2 * p.H;
   auto stage = [&](int blk) {
     const int buf = blk & 1, t0 = blk * DS_TB;
@@ -249,13 +285,427 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaParam
     const int row = 4 * (r + 8 * (i >> 2)) + (i & 3);
     if (col_on && row < p.D) st[row] = S[i];
   }
-  // the last convolution inputs: the channels are dealt out over the CTAs of the sequence
-  const T* proj = static_cast<const T*>(p.proj) + (long long)first * p.stride;
-  T* ring = static_cast<T*>(p.ring) + (long long)slot * p.taps * C;
-  const int parts = gridDim.x * gridDim.y, part = blockIdx.y * gridDim.x + blockIdx.x;
-  for (int c = part * DS_THREADS + tid; c < C; c += parts * DS_THREADS)
-    for (int t = max(0, n - p.taps); t < n; ++t)
-      ring[(long long)((start + t) % p.taps) * C + c] = proj[(long long)t * p.stride + c];
+  store_ring<T>(p, first, n, start, slot, blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y);
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// Chunked form on the tensor cores. Chunk c of sequence b has index (cu_q[b] / 64) + b + c: distinct for all chunks, at
+// most T / 64 + B of them.
+constexpr int DC = 64;             // tokens per chunk
+constexpr int DC_VB = 64;          // state columns per CTA
+constexpr int DC_MAT = DC * DC;    // one bf16 term of T or P
+// scratch of one (chunk, head): T hi | T lo | P hi | P lo (bf16 [64][64] each), then fp32 vectors
+//   e^{G_t} / |k_t|,  e^{G_t} D^{-1/2} / |q_t|,  e^{G_last - G_t} / |k_t|,  [e^{G_last}, unused ...]
+constexpr int DC_VEC_OFF = 4 * DC_MAT * 2;
+constexpr int DC_BYTES = DC_VEC_OFF + 4 * DC * 4;
+
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const __nv_bfloat16* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(smem_u32(p)) : "memory");
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const __nv_bfloat16* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(smem_u32(p)) : "memory");
+}
+__device__ __forceinline__ void mma16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void cp_async16(void* dst, const void* src, bool on) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(on ? 16 : 0) : "memory");
+}
+// x = hi + lo, both bf16, for two neighbours packed into 32 bits
+__device__ __forceinline__ void split2(float x0, float x1, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16x2(x0, x1);
+  lo = pack_bf16x2(x0 - __uint_as_float(hi << 16), x1 - __uint_as_float(hi & 0xffff0000u));
+}
+// Fragment addresses. A [16 x 16] at (row, col) of a row-major tile:
+template <int PITCH>
+__device__ __forceinline__ const __nv_bfloat16* frag_a(const __nv_bfloat16* t, int row, int col, int lane) {
+  return t + (row + (lane & 15)) * PITCH + col + (lane >> 4) * 8;
+}
+// A^T: the tile stores [k][m]; the result is the [16 m x 16 k] operand (ldsm4t)
+template <int PITCH>
+__device__ __forceinline__ const __nv_bfloat16* frag_at(const __nv_bfloat16* t, int m, int k, int lane) {
+  return t + (k + ((lane >> 4) & 1) * 8 + (lane & 7)) * PITCH + m + ((lane >> 3) & 1) * 8;
+}
+// B of two neighbouring n-tiles, stored [k][n] (ldsm4t)
+template <int PITCH>
+__device__ __forceinline__ const __nv_bfloat16* frag_b(const __nv_bfloat16* t, int k, int n, int lane) {
+  return t + (k + (lane & 15)) * PITCH + n + (lane >> 4) * 8;
+}
+// B of two neighbouring n-tiles, stored [n][k] (ldsm4)
+template <int PITCH>
+__device__ __forceinline__ const __nv_bfloat16* frag_bn(const __nv_bfloat16* t, int k, int n, int lane) {
+  return t + (n + ((lane >> 4) & 1) * 8 + (lane & 7)) * PITCH + k + ((lane >> 3) & 1) * 8;
+}
+
+// One CTA of four warps per (chunk, head): T = (I + A)^-1 diag(beta) and P.
+template <int DP>
+__global__ void __launch_bounds__(128) delta_chunk_prep_kernel(const DeltaParams p, uint8_t* __restrict__ scratch) {
+  constexpr int PI = DP + 8, AP = DC + 4, TP = DC + 8;
+  extern __shared__ uint8_t smb[];
+  __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smb);
+  __nv_bfloat16* q_s = k_s + DC * PI;
+  float* a_s = reinterpret_cast<float*>(q_s + DC * PI);                      // [64][AP]
+  float* G_s = a_s + DC * AP;                                                // [64]
+  float *b_s = G_s + DC, *nk_s = b_s + DC, *nq_s = nk_s + DC;
+  __nv_bfloat16* t_s = k_s;                                                  // T hi | lo [64][TP] over k_s / q_s, later
+  pdl_trigger();
+  pdl_wait();
+  const int idx = blockIdx.x, h = blockIdx.y;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  int lo = 0, hi = p.B - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if ((p.cu_q[mid] >> 6) + mid <= idx) lo = mid; else hi = mid - 1;
+  }
+  const int b = lo, first = p.cu_q[b], n = p.cu_q[b + 1] - first, t0 = (idx - (first >> 6) - b) * DC;
+  if (t0 >= n || p.slots[b] < 0) return;
+  const int hk = h / (p.H / p.Hk), C = 2 * p.Hk * p.D + p.H * p.V;
+  const __nv_bfloat16* y = static_cast<const __nv_bfloat16*>(p.qkv) + (long long)(first + t0) * C + hk * p.D;
+  for (int i = tid; i < DC * (DP / 8); i += 128) {
+    const int t = i / (DP / 8), d = i % (DP / 8) * 8;
+    const bool on = t0 + t < n && d < p.D;
+    const __nv_bfloat16* src = on ? y + (long long)t * C + d : y;
+    cp_async16(q_s + t * PI + d, src, on);
+    cp_async16(k_s + t * PI + d, src + p.Hk * p.D, on);
+  }
+  cp_async_commit();
+  if (tid < DC) {
+    const bool on = t0 + tid < n;
+    const long long t = first + t0 + tid;
+    G_s[tid] = on ? p.gates[t * 2 * p.H + p.H + h] : 0.f;
+    b_s[tid] = on ? p.gates[t * 2 * p.H + h] : 0.f;
+    nq_s[tid] = on ? p.unit[t * 2 * p.Hk + hk] : 0.f;
+    nk_s[tid] = on ? p.unit[t * 2 * p.Hk + p.Hk + hk] : 0.f;
+  }
+  __syncthreads();
+  if (warp == 0) {  // running sums of the log decays, two tokens per lane
+    const float x0 = G_s[2 * lane], x1 = G_s[2 * lane + 1];
+    float s = x0 + x1;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float v = __shfl_up_sync(0xffffffffu, s, o);
+      if (lane >= o) s += v;
+    }
+    G_s[2 * lane] = s - x1;
+    G_s[2 * lane + 1] = s;
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+  uint8_t* dst = scratch + ((long long)idx * p.H + h) * DC_BYTES;
+  if (tid < DC) {
+    float* vec = reinterpret_cast<float*>(dst + DC_VEC_OFF);
+    const float g = G_s[tid], gl = G_s[DC - 1], eg = expf(g);
+    vec[tid] = eg * nk_s[tid];
+    vec[DC + tid] = eg * nq_s[tid];
+    vec[2 * DC + tid] = expf(gl - g) * nk_s[tid];
+    if (tid == 0) vec[3 * DC] = expf(gl);
+  }
+  // Gram matrices of this warp's 16 rows, columns up to the diagonal block
+  float kk[8][4] = {}, qk[8][4] = {};
+  const int nt_end = 2 * (warp + 1);
+#pragma unroll
+  for (int k = 0; k < DP / 16; ++k) {
+    uint32_t ak[4], aq[4];
+    ldsm4(ak, frag_a<PI>(k_s, warp * 16, k * 16, lane));
+    ldsm4(aq, frag_a<PI>(q_s, warp * 16, k * 16, lane));
+#pragma unroll
+    for (int nt = 0; nt < 8; nt += 2) {
+      if (nt < nt_end) {
+        uint32_t bb[4];
+        ldsm4(bb, frag_bn<PI>(k_s, k * 16, nt * 8, lane));
+        mma16(kk[nt], ak, bb[0], bb[1]);
+        mma16(kk[nt + 1], ak, bb[2], bb[3]);
+        mma16(qk[nt], aq, bb[0], bb[1]);
+        mma16(qk[nt + 1], aq, bb[2], bb[3]);
+      }
+    }
+  }
+  uint32_t* P_hi = reinterpret_cast<uint32_t*>(dst) + DC_MAT;  // 32-bit words: T hi, T lo take DC_MAT of them
+  uint32_t* P_lo = P_hi + DC_MAT / 2;
+#pragma unroll
+  for (int nt = 0; nt < 8; ++nt) {
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int t = warp * 16 + (lane >> 2) + 8 * half, s = nt * 8 + (lane & 3) * 2;
+      float pv[2], av[2];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const float dec = s + e <= t ? expf(G_s[t] - G_s[s + e]) * nk_s[s + e] : 0.f;
+        pv[e] = dec * nq_s[t] * qk[nt][2 * half + e];
+        av[e] = s + e < t ? dec * nk_s[t] * b_s[t] * kk[nt][2 * half + e] : 0.f;
+      }
+      uint32_t ph, pl;
+      split2(pv[0], pv[1], ph, pl);
+      P_hi[(t * DC + s) >> 1] = ph;
+      P_lo[(t * DC + s) >> 1] = pl;
+      *reinterpret_cast<float2*>(a_s + t * AP + s) = make_float2(av[0], av[1]);
+    }
+  }
+  __syncthreads();
+  // forward substitution: thread j owns column j of (I + A)^-1
+  if (tid < DC) {
+    float x[DC];
+#pragma unroll
+    for (int i = 0; i < DC; ++i) {
+      float s0 = i == tid ? 1.f : 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
+#pragma unroll
+      for (int k = 0; k < i; k += 4) {
+        const float4 a = *reinterpret_cast<const float4*>(a_s + i * AP + k);  // entries from the diagonal on are zero
+        s0 = fmaf(-a.x, x[k], s0);
+        if (k + 1 < i) s1 = fmaf(-a.y, x[k + 1], s1);
+        if (k + 2 < i) s2 = fmaf(-a.z, x[k + 2], s2);
+        if (k + 3 < i) s3 = fmaf(-a.w, x[k + 3], s3);
+      }
+      x[i] = (s0 + s1) + (s2 + s3);
+    }
+    const float beta = b_s[tid];
+#pragma unroll
+    for (int i = 0; i < DC; ++i) {
+      const float v = x[i] * beta;
+      const __nv_bfloat16 vh = __float2bfloat16(v);
+      t_s[i * TP + tid] = vh;
+      t_s[(DC + i) * TP + tid] = __float2bfloat16(v - __bfloat162float(vh));
+    }
+  }
+  __syncthreads();
+  for (int i = tid; i < 2 * DC * 8; i += 128) {
+    const int r = i >> 3, c = (i & 7) * 8;
+    *reinterpret_cast<uint4*>(dst + (r * DC + c) * 2) = *reinterpret_cast<const uint4*>(t_s + r * TP + c);
+  }
+}
+
+// One CTA of eight warps per (sequence, head, 64 state columns): warp = (row slab wr of 16 tokens, column half wc of 32).
+// S [D, 64] stays in fp32 accumulators (warp (wr, wc) owns rows 32 wr .. of DP = 128, 16 wr .. of DP = 64) with a hi / lo
+// copy in shared memory for the next chunk's products.
+template <int DP>
+__global__ void __launch_bounds__(256, 1) delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch) {
+  constexpr int PI = DP + 8, XP = DC_VB + 8, MT = DP / 64;  // MT: 16-row tiles of S per warp
+  extern __shared__ uint8_t smb[];
+  __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smb);    // [2][64][PI]
+  __nv_bfloat16* q_s = k_s + 2 * DC * PI;                        // [2][64][PI]
+  __nv_bfloat16* v_s = q_s + 2 * DC * PI;                        // [2][64][XP]
+  __nv_bfloat16* T_s = v_s + 2 * DC * XP;                        // hi | lo [64][XP]
+  __nv_bfloat16* P_s = T_s + 2 * DC * XP;                        // hi | lo
+  __nv_bfloat16* x_s = P_s + 2 * DC * XP;                        // hi | lo: right-hand side, then U
+  __nv_bfloat16* w_s = x_s + 2 * DC * XP;                        // hi | lo: U scaled for the state
+  __nv_bfloat16* S_s = w_s + 2 * DC * XP;                        // hi | lo [DP][XP]
+  float* vec_s = reinterpret_cast<float*>(S_s + 2 * DP * XP);    // [2][4][64]
+  pdl_trigger();
+  pdl_wait();
+  const int v0 = blockIdx.x * DC_VB, h = blockIdx.y, b = blockIdx.z;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, wr = warp & 3, wc = warp >> 2;
+  const int first = p.cu_q[b], n = p.cu_q[b + 1] - first, slot = p.slots[b];
+  if (n <= 0 || slot < 0) return;
+  const int start = p.seq_lens[b] - n, hk = h / (p.H / p.Hk), C = 2 * p.Hk * p.D + p.H * p.V;
+  const __nv_bfloat16* y = static_cast<const __nv_bfloat16*>(p.qkv) + (long long)first * C;
+  const uint8_t* scr = scratch + ((long long)((first >> 6) + b) * p.H + h) * DC_BYTES;
+  const long long scr_step = (long long)p.H * DC_BYTES;
+  const int chunks = (n + DC - 1) / DC;
+
+  auto load_kqv = [&](int c) {
+    if (c < chunks) {
+      const int buf = c & 1, t0 = c * DC;
+      for (int i = tid; i < DC * (DP / 8); i += 256) {
+        const int t = i / (DP / 8), d = i % (DP / 8) * 8;
+        const bool on = t0 + t < n && d < p.D;
+        const __nv_bfloat16* src = y + (on ? (long long)(t0 + t) * C + hk * p.D + d : 0);
+        cp_async16(q_s + (buf * DC + t) * PI + d, src, on);
+        cp_async16(k_s + (buf * DC + t) * PI + d, src + p.Hk * p.D, on);
+      }
+      for (int i = tid; i < DC * (DC_VB / 8); i += 256) {
+        const int t = i / (DC_VB / 8), d = i % (DC_VB / 8) * 8;
+        const bool on = t0 + t < n && v0 + d < p.V;
+        cp_async16(v_s + (buf * DC + t) * XP + d,
+                   y + (on ? (long long)(t0 + t) * C + 2 * p.Hk * p.D + h * p.V + v0 + d : 0), on);
+      }
+      if (tid < DC) cp_async16(vec_s + buf * 4 * DC + tid * 4, scr + c * scr_step + DC_VEC_OFF + tid * 16, true);
+    }
+    cp_async_commit();
+  };
+  auto load_mat = [&](int c, __nv_bfloat16* dst, int off) {
+    if (c < chunks)
+      for (int i = tid; i < 2 * DC * 8; i += 256) {
+        const int r = i >> 3, k = (i & 7) * 8;
+        cp_async16(dst + r * XP + k, scr + c * scr_step + off + (r * DC + k) * 2, true);
+      }
+    cp_async_commit();
+  };
+  // accumulator element e of tile (mt, nt): row, column within the CTA's [DP, 64] block
+  auto s_row = [&](int mt, int e) { return wr * 16 * MT + mt * 16 + (lane >> 2) + 8 * (e >> 1); };
+  auto s_col = [&](int nt, int e) { return wc * 32 + nt * 8 + (lane & 3) * 2 + (e & 1); };
+  float S[MT][4][4];
+  float* st = p.state + ((long long)slot * p.H + h) * p.V * p.D;
+  load_kqv(0);
+  load_mat(0, T_s, 0);
+  load_mat(0, P_s, 2 * DC_MAT * 2);
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int d = s_row(mt, e), c = v0 + s_col(nt, e);
+        S[mt][nt][e] = start > 0 && d < p.D && c < p.V ? st[(long long)c * p.D + d] : 0.f;
+      }
+  auto publish_state = [&]() {
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          uint32_t hi, lo;
+          split2(S[mt][nt][2 * half], S[mt][nt][2 * half + 1], hi, lo);
+          __nv_bfloat16* d = S_s + s_row(mt, 2 * half) * XP + s_col(nt, 0);
+          *reinterpret_cast<uint32_t*>(d) = hi;
+          *reinterpret_cast<uint32_t*>(d + DP * XP) = lo;
+        }
+  };
+  publish_state();
+  cp_async_wait<2>();
+  __syncthreads();
+
+  for (int c = 0; c < chunks; ++c) {
+    const int buf = c & 1, t0 = c * DC;
+    const __nv_bfloat16 *kb = k_s + buf * DC * PI, *qb = q_s + buf * DC * PI, *vb = v_s + buf * DC * XP;
+    const float* vec = vec_s + buf * 4 * DC;
+    load_kqv(c + 1);
+    // 1. K S and Q S
+    float R[4][4] = {}, O[4][4] = {};
+#pragma unroll
+    for (int k = 0; k < DP / 16; ++k) {
+      uint32_t ak[4], aq[4];
+      ldsm4(ak, frag_a<PI>(kb, wr * 16, k * 16, lane));
+      ldsm4(aq, frag_a<PI>(qb, wr * 16, k * 16, lane));
+#pragma unroll
+      for (int part = 0; part < 2; ++part)
+#pragma unroll
+        for (int np = 0; np < 2; ++np) {
+          uint32_t bb[4];
+          ldsm4t(bb, frag_b<XP>(S_s + part * DP * XP, k * 16, wc * 32 + np * 16, lane));
+          mma16(R[2 * np], ak, bb[0], bb[1]);
+          mma16(R[2 * np + 1], ak, bb[2], bb[3]);
+          mma16(O[2 * np], aq, bb[0], bb[1]);
+          mma16(O[2 * np + 1], aq, bb[2], bb[3]);
+        }
+    }
+    // right-hand side v - e^G k S
+#pragma unroll
+    for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int t = wr * 16 + (lane >> 2) + 8 * half, col = s_col(nt, 0);
+        const uint32_t vv = *reinterpret_cast<const uint32_t*>(vb + t * XP + col);
+        const float ek = vec[t], eq = vec[DC + t];
+        uint32_t hi, lo;
+        split2(__uint_as_float(vv << 16) - ek * R[nt][2 * half], __uint_as_float(vv & 0xffff0000u) - ek * R[nt][2 * half + 1], hi,
+               lo);
+        *reinterpret_cast<uint32_t*>(x_s + t * XP + col) = hi;
+        *reinterpret_cast<uint32_t*>(x_s + (DC + t) * XP + col) = lo;
+        O[nt][2 * half] *= eq;
+        O[nt][2 * half + 1] *= eq;
+      }
+    cp_async_wait<2>();  // T of this chunk
+    __syncthreads();
+    // 2. U = T . rhs (lower triangular: this slab needs the token blocks 0 .. wr)
+    float U[4][4] = {};
+    auto tri = [&](float (&acc)[4][4], const __nv_bfloat16* m) {
+      for (int k = 0; k <= wr; ++k) {
+        uint32_t ah[4], al[4];
+        ldsm4(ah, frag_a<XP>(m, wr * 16, k * 16, lane));
+        ldsm4(al, frag_a<XP>(m + DC * XP, wr * 16, k * 16, lane));
+#pragma unroll
+        for (int np = 0; np < 2; ++np) {
+          uint32_t bh[4], bl[4];
+          ldsm4t(bh, frag_b<XP>(x_s, k * 16, wc * 32 + np * 16, lane));
+          ldsm4t(bl, frag_b<XP>(x_s + DC * XP, k * 16, wc * 32 + np * 16, lane));
+          mma16(acc[2 * np], ah, bh[0], bh[1]);
+          mma16(acc[2 * np + 1], ah, bh[2], bh[3]);
+          mma16(acc[2 * np], al, bh[0], bh[1]);
+          mma16(acc[2 * np + 1], al, bh[2], bh[3]);
+          mma16(acc[2 * np], ah, bl[0], bl[1]);
+          mma16(acc[2 * np + 1], ah, bl[2], bl[3]);
+        }
+      }
+    };
+    tri(U, T_s);
+    __syncthreads();  // every warp is done with the right-hand side and with T
+    load_mat(c + 1, T_s, 0);
+#pragma unroll
+    for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int t = wr * 16 + (lane >> 2) + 8 * half, col = s_col(nt, 0);
+        const float ce = vec[2 * DC + t];
+        uint32_t hi, lo;
+        split2(U[nt][2 * half], U[nt][2 * half + 1], hi, lo);
+        *reinterpret_cast<uint32_t*>(x_s + t * XP + col) = hi;
+        *reinterpret_cast<uint32_t*>(x_s + (DC + t) * XP + col) = lo;
+        split2(ce * U[nt][2 * half], ce * U[nt][2 * half + 1], hi, lo);
+        *reinterpret_cast<uint32_t*>(w_s + t * XP + col) = hi;
+        *reinterpret_cast<uint32_t*>(w_s + (DC + t) * XP + col) = lo;
+      }
+    cp_async_wait<2>();  // P of this chunk
+    __syncthreads();
+    // 3. output
+    tri(O, P_s);
+    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (long long)(first + t0) * p.out_stride + (long long)h * p.V + v0;
+#pragma unroll
+    for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int t = wr * 16 + (lane >> 2) + 8 * half, col = s_col(nt, 0);
+        if (t0 + t < n && v0 + col < p.V)
+          *reinterpret_cast<uint32_t*>(out + (long long)t * p.out_stride + col) = pack_bf16x2(O[nt][2 * half], O[nt][2 * half + 1]);
+      }
+    // 4. state
+    const float egl = vec[3 * DC];
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) S[mt][nt][e] *= egl;
+#pragma unroll
+    for (int k = 0; k < DC / 16; ++k) {
+      uint32_t a[MT][4];
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt) ldsm4t(a[mt], frag_at<PI>(kb, wr * 16 * MT + mt * 16, k * 16, lane));
+#pragma unroll
+      for (int part = 0; part < 2; ++part)
+#pragma unroll
+        for (int np = 0; np < 2; ++np) {
+          uint32_t bb[4];
+          ldsm4t(bb, frag_b<XP>(w_s + part * DC * XP, k * 16, wc * 32 + np * 16, lane));
+#pragma unroll
+          for (int mt = 0; mt < MT; ++mt) {
+            mma16(S[mt][2 * np], a[mt], bb[0], bb[1]);
+            mma16(S[mt][2 * np + 1], a[mt], bb[2], bb[3]);
+          }
+        }
+    }
+    publish_state();
+    cp_async_wait<1>();  // q, k, v of the next chunk
+    __syncthreads();
+    load_mat(c + 1, P_s, 2 * DC_MAT * 2);
+  }
+#pragma unroll
+  for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+    for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int d = s_row(mt, e), c = v0 + s_col(nt, e);
+        if (d < p.D && c < p.V) st[(long long)c * p.D + d] = S[mt][nt][e];
+      }
+  store_ring<__nv_bfloat16>(p, first, n, start, slot, blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y);
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -420,16 +870,16 @@ __global__ void __launch_bounds__(DD_THREADS) delta_step_kernel(const DeltaParam
   for (int c = tid; c < p.V; c += DD_THREADS) out[c] = dl_t<T>(o_s[c] * inv * dl_f<T>(w[c]) * silu_f(dl_f<T>(gate[c])));
 }
 
-template <typename T>
+template <typename T, bool CHUNK>
 static int run_prep(const DeltaParams& p, int max_q, cudaStream_t stream) {
   const dim3 g((max_q + DP_TT - 1) / DP_TT, (2 * p.Hk + p.H + 1 + 3) / 4, p.B), b(128);
   const int cpl = ((p.D > p.V ? p.D : p.V) + 31) / 32;
   cudaError_t e = cudaErrorInvalidValue;
 #define VB_PREP(TAPS)                                                                                      \
-  (cpl <= 1   ? vb_launch_pdl(delta_prep_kernel<T, TAPS, 1>, g, b, 0, stream, 1, p)                        \
-   : cpl <= 2 ? vb_launch_pdl(delta_prep_kernel<T, TAPS, 2>, g, b, 0, stream, 1, p)                        \
-   : cpl <= 4 ? vb_launch_pdl(delta_prep_kernel<T, TAPS, 4>, g, b, 0, stream, 1, p)                        \
-              : vb_launch_pdl(delta_prep_kernel<T, TAPS, 8>, g, b, 0, stream, 1, p))
+  (cpl <= 1   ? vb_launch_pdl(delta_prep_kernel<T, TAPS, 1, CHUNK>, g, b, 0, stream, 1, p)                        \
+   : cpl <= 2 ? vb_launch_pdl(delta_prep_kernel<T, TAPS, 2, CHUNK>, g, b, 0, stream, 1, p)                        \
+   : cpl <= 4 ? vb_launch_pdl(delta_prep_kernel<T, TAPS, 4, CHUNK>, g, b, 0, stream, 1, p)                        \
+              : vb_launch_pdl(delta_prep_kernel<T, TAPS, 8, CHUNK>, g, b, 0, stream, 1, p))
   e = p.taps <= 4 ? VB_PREP(4) : VB_PREP(8);
 #undef VB_PREP
   vb_count_launch();
@@ -459,8 +909,28 @@ static int run_step(const DeltaParams& p, cudaStream_t stream) {
   return (int)e;
 }
 
+template <int DP>
+static int run_chunks(const DeltaParams& p, int tokens, uint8_t* scratch, cudaStream_t stream) {
+  constexpr int PI = DP + 8, XP = DC_VB + 8;
+  const int smem1 = 2 * DC * PI * 2 + (DC * (DC + 4) + 4 * DC) * 4;
+  const int smem2 = (4 * DC * PI + 2 * DC * XP + 8 * DC * XP + 2 * DP * XP) * 2 + 8 * DC * 4;
+  static bool attr = false;
+  if (!attr) {
+    VB_CUDA_CHECK(cudaFuncSetAttribute(delta_chunk_prep_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem1));
+    VB_CUDA_CHECK(cudaFuncSetAttribute(delta_chunk_scan_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2));
+    attr = true;
+  }
+  cudaError_t e = vb_launch_pdl(delta_chunk_prep_kernel<DP>, dim3(tokens / DC + p.B, p.H), dim3(128), smem1, stream, 1, p,
+                                scratch);
+  if (e != cudaSuccess) return (int)e;
+  e = vb_launch_pdl(delta_chunk_scan_kernel<DP>, dim3((p.V + DC_VB - 1) / DC_VB, p.H, p.B), dim3(256), smem2, stream, 1, p,
+                    (const uint8_t*)scratch);
+  vb_count_launch(2);
+  return (int)e;
+}
+
 template <typename T>
-static int run_delta(const DeltaParams& p, int tokens, int max_q, cudaStream_t stream) {
+static int run_delta(const DeltaParams& p, int tokens, int max_q, uint8_t* chunk_scratch, cudaStream_t stream) {
   const int nr = p.D <= 32 ? 4 : p.D <= 64 ? 8 : p.D <= 128 ? 16 : 32;
   if (max_q == 1) {
     if (nr == 4) return run_step<T, 4>(p, stream);
@@ -468,10 +938,15 @@ static int run_delta(const DeltaParams& p, int tokens, int max_q, cudaStream_t s
     if (nr == 16) return run_step<T, 16>(p, stream);
     return run_step<T, 32>(p, stream);
   }
-  int rc = run_prep<T>(p, max_q, stream);
+  int rc = chunk_scratch ? run_prep<T, true>(p, max_q, stream) : run_prep<T, false>(p, max_q, stream);
   if (rc) return rc;
-  rc = nr == 4 ? run_scan<T, 4>(p, stream) : nr == 8 ? run_scan<T, 8>(p, stream) : nr == 16 ? run_scan<T, 16>(p, stream)
-                                                                                           : run_scan<T, 32>(p, stream);
+  if (chunk_scratch)
+    rc = p.D <= 64 ? run_chunks<64>(p, tokens, chunk_scratch, stream) : run_chunks<128>(p, tokens, chunk_scratch, stream);
+  else
+    rc = nr == 4    ? run_scan<T, 4>(p, stream)
+         : nr == 8  ? run_scan<T, 8>(p, stream)
+         : nr == 16 ? run_scan<T, 16>(p, stream)
+                    : run_scan<T, 32>(p, stream);
   if (rc) return rc;
   const long long warps = (long long)tokens * p.H;
   cudaError_t e = vb_launch_pdl(gated_norm_kernel<T>, dim3((unsigned)((warps + 3) / 4)), dim3(128), 0, stream, 1, p, tokens);
@@ -483,18 +958,30 @@ static int run_delta(const DeltaParams& p, int tokens, int max_q, cudaStream_t s
 
 using namespace vb;
 
-// Limits: D, V <= 256, taps <= 8. max_q == 1 (every sequence brings exactly one token) takes the fused step and does not
-// touch qkv / gates; otherwise qkv is fp32 scratch [T, 2 Hk D + H V] and gates fp32 scratch [T, 2 H].
+// 1 if the chunked form serves these sizes (bf16 only).
+extern "C" int vb_delta_chunk_supported(int D, int V) {
+  return D >= 8 && D <= 128 && (D & 7) == 0 && V >= 8 && V <= 256 && (V & 7) == 0;
+}
+// Bytes of chunk_scratch for T tokens of B sequences.
+extern "C" long long vb_delta_chunk_bytes(int T, int B, int H) { return (long long)(T / DC + B) * H * DC_BYTES; }
+
+// Limits: D, V <= 256, taps <= 8. max_q == 1 (every sequence brings exactly one token) takes the fused step and needs no
+// scratch. Otherwise gates is fp32 scratch [T, 2 H] and qkv scratch [T, 2 Hk D + H V]: fp32 for the token-by-token scan
+// (chunk_scratch and unit null), bf16 for the chunked form, with unit fp32 [T, 2 Hk] and chunk_scratch (16-byte aligned).
 extern "C" int vb_delta_rule(const void* proj, long long stride, const void* conv_w, const float* a_log,
                              const float* dt_bias, const void* norm_w, void* ring, float* state, const int* cu_q,
-                             const int* seq_lens, const int* slots, float* qkv, float* gates, void* out,
-                             long long out_stride, int T, int B, int max_q, int H, int Hk, int D, int V, int taps, float eps,
-                             int f32, cudaStream_t stream) {
+                             const int* seq_lens, const int* slots, void* qkv, float* unit, float* gates, void* chunk_scratch,
+                             void* out, long long out_stride, int T, int B, int max_q, int H, int Hk, int D, int V, int taps,
+                             float eps, int f32, cudaStream_t stream) {
   if (T <= 0 || B <= 0 || max_q <= 0) return 0;
   if (Hk <= 0 || H % Hk != 0 || D <= 0 || D > 256 || V <= 0 || V > 256 || taps < 1 || taps > 8 || B > 65535) return -3;
   if (max_q > 1 && (qkv == nullptr || gates == nullptr)) return -3;
-  DeltaParams p{proj, stride, conv_w, a_log, dt_bias, norm_w, ring, state, cu_q, seq_lens, slots, qkv, gates, out,
+  if (max_q > 1 && chunk_scratch != nullptr &&
+      (f32 || unit == nullptr || !vb_delta_chunk_supported(D, V) || (out_stride & 1) || (reinterpret_cast<uintptr_t>(qkv) & 15)))
+    return -3;
+  DeltaParams p{proj, stride, conv_w, a_log, dt_bias, norm_w, ring, state, cu_q, seq_lens, slots, qkv, unit, gates, out,
                 out_stride, B, H, Hk, D, V, taps, eps};
-  const int rc = f32 ? run_delta<float>(p, T, max_q, stream) : run_delta<__nv_bfloat16>(p, T, max_q, stream);
+  uint8_t* scr = reinterpret_cast<uint8_t*>(chunk_scratch);
+  const int rc = f32 ? run_delta<float>(p, T, max_q, nullptr, stream) : run_delta<__nv_bfloat16>(p, T, max_q, scr, stream);
   return rc ? rc : (int)cudaGetLastError();
 }

@@ -1,15 +1,17 @@
 // Prefill attention of layer-list decoders on tcgen05: ragged queries over the paged KV cache, with a sliding window,
 // kept first keys and a per-distance bias. Head sizes up to 128 (multiples of 8), bf16.
 //
-// One CTA per (sequence, query head, block of 128 queries). The CTA walks the 128-key chunks that some row of the block
-// may see: those of the kept first keys, then those of the window. Per chunk:
+// One CTA per (sequence, query head, block of 128 queries), two CTAs per SM: one's softmax overlaps the other's tensor
+// work. The CTA walks the 128-key chunks that some row of the block may see: those of the kept first keys, then those of
+// the window. Per chunk:
 //     S[128 q x 128 keys] = Q . K^T                       (tcgen05.mma, accumulator in TMEM)
-//     P = exp(S * scale + bias[distance] - rowmax)        (thread = query row)
-//     O_c[128 q x Dv]     = P . V                         (A operand = P in TMEM)
+//     P = exp(S * scale + bias[distance] - reference)     (thread = query row)
+//     O[128 q x Dv]      += P . V                         (A operand = P in TMEM, accumulator in TMEM)
 // The weights stay close to fp32: P is split into two bf16 terms (P = hi + lo) that are written over the columns of S
-// they came from, and both are multiplied with V. The running output lives in registers (flash rescale).
-// K / V pages arrive by per-CTA TMA loads through a ring of 32 KB slots; columns past a head's size are filled with zeros
-// by TMA, keys past the sequence or outside the mask get weight zero.
+// they came from, and both are multiplied with V. A row's reference is a running maximum that only moves when the
+// maximum has grown by more than 2^8 (the result does not depend on it), so O is rarely rescaled.
+// K / V pages arrive by per-CTA TMA loads; columns past a head's size are filled with zeros by TMA, keys past the sequence
+// or outside the mask get weight zero. Masks and the bias table are looked at only by the 32 x 32 blocks they reach.
 // Every wait is bounded; on expiry the status word is set and the CTA leaves through its teardown.
 #include "common.cuh"
 #include "host_utils.h"
@@ -18,12 +20,13 @@ namespace vb {
 
 constexpr int PF_M = 128, PF_N = 128;             // queries per CTA, keys per chunk
 constexpr int PF_TILE = 128 * 128 * 2;            // 32 KB: two 64-column halves of 16 KB
-constexpr int PF_SLOTS = 5;
 constexpr int PF_THREADS = 192;
-constexpr int PF_RING_OFF = PF_TILE;              // Q first
-constexpr int PF_BAR_OFF = PF_RING_OFF + PF_SLOTS * PF_TILE;
-constexpr int PF_BIAS_OFF = PF_BAR_OFF + 20 * 8 + 32;
-constexpr int PF_MAX_BIAS = 6144;                 // distances staged in shared memory
+constexpr int PF_K_OFF = PF_TILE;                 // Q first, then one K and one V tile
+constexpr int PF_V_OFF = 2 * PF_TILE;
+constexpr int PF_BAR_OFF = 3 * PF_TILE;
+constexpr int PF_BIAS_OFF = PF_BAR_OFF + 8 * 8 + 32;
+constexpr int PF_MAX_BIAS = 3072;                 // distances staged in shared memory
+constexpr float PF_SLACK = 8.f;                   // growth of the row maximum (log2) that is let through
 
 struct PagedFlashParams {
   const int* cu_q;         // [B + 1]
@@ -40,20 +43,15 @@ struct PagedFlashParams {
 // exp2 of the scaled scores: scale and bias are multiplied by log2(e) up front
 constexpr float LOG2E = 1.4426950408889634f;
 
-__global__ void __launch_bounds__(PF_THREADS, 1)
+__global__ void __launch_bounds__(PF_THREADS, 2)
 paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                    const __grid_constant__ CUtensorMap tmV, const PagedFlashParams p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  uint8_t* q_s = smem;
-  uint8_t* ring = smem + PF_RING_OFF;
-  uint64_t* full = reinterpret_cast<uint64_t*>(smem + PF_BAR_OFF);
-  uint64_t* empty = full + PF_SLOTS;
-  uint64_t* s_full = empty + PF_SLOTS;
-  uint64_t* p_ready = s_full + 2;
-  uint64_t* o_full = p_ready + 2;
-  uint64_t* q_full = o_full + 2;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(q_full + 1);
+  // barriers: [0] Q, [1] K full, [2] V full, [3] K empty, [4] V empty, [5] S full, [6] P ready, [7] O full
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + PF_BAR_OFF);
+  uint64_t *q_full = bars, *full = bars + 1, *empty = bars + 3, *s_full = bars + 5, *p_ready = bars + 6, *o_full = bars + 7;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 8);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   float* bias_s = reinterpret_cast<float*>(smem + PF_BIAS_OFF);
 
@@ -77,21 +75,12 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   auto chunk_at = [&](int c) { return c < keep_chunks ? c : win_chunk + c - keep_chunks; };
 
   if (tid == 0) {
-    for (int s = 0; s < PF_SLOTS; ++s) {
-      mbar_init(&full[s], 1);
-      mbar_init(&empty[s], 1);
-    }
-    for (int i = 0; i < 2; ++i) {
-      mbar_init(&s_full[i], 1);
-      mbar_init(&p_ready[i], 4);
-      mbar_init(&o_full[i], 1);
-    }
-    mbar_init(q_full, 1);
+    for (int i = 0; i < 8; ++i) mbar_init(&bars[i], i == 6 ? 4 : 1);
     *abort_flag = 0;
     mbar_fence_init();
   }
   if (warp == 5) {
-    tmem_alloc(tmem_slot, 512);
+    tmem_alloc(tmem_slot, 256);
     tmem_relinquish();
   }
   if (p.bias != nullptr)
@@ -99,7 +88,7 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem_base = *tmem_slot;
+  const uint32_t tmem_base = *tmem_slot;  // S / P: columns 0..127, O: 128..255
   pdl_trigger();  // TMEM is held: a dependent kernel may take what is left
   const int k_halves = p.D > 64 ? 2 : 1, v_halves = p.Dv > 64 ? 2 : 1;
 
@@ -110,20 +99,20 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       tma_prefetch_desc(&tmK);
       tma_prefetch_desc(&tmV);
       mbar_arrive_expect_tx(q_full, k_halves * 16384);
-      for (int x = 0; x < k_halves; ++x) tma_load_3d(q_s + x * 16384, &tmQ, q_full, x * 64, hq, q_first + r0);
+      for (int x = 0; x < k_halves; ++x) tma_load_3d(smem + x * 16384, &tmQ, q_full, x * 64, hq, q_first + r0);
       const int* bt = p.block_table + (long long)b * p.max_blocks;
       const int ppc = PF_N / p.block_size, n_pages = (seq_len + p.block_size - 1) / p.block_size;
       for (int t = 0; t < 2 * n_chunks; ++t) {
-        const int s = t % PF_SLOTS;
-        if (*abort_flag || !mbar_wait(&empty[s], ((t / PF_SLOTS) & 1) ^ 1)) {
+        const int s = t & 1;  // 0 = K, 1 = V
+        if (*abort_flag || !mbar_wait(&empty[s], ((t >> 1) & 1) ^ 1)) {
           report_error(p.status, ERR_WAIT_EMPTY, t);
           *abort_flag = 1;
           break;
         }
-        const int halves = (t & 1) ? v_halves : k_halves;
+        const int halves = s ? v_halves : k_halves;
         mbar_arrive_expect_tx(&full[s], halves * 16384);
-        uint8_t* dst = ring + s * PF_TILE;
-        const CUtensorMap* tm = (t & 1) ? &tmV : &tmK;
+        uint8_t* dst = smem + (s ? PF_V_OFF : PF_K_OFF);
+        const CUtensorMap* tm = s ? &tmV : &tmK;
         const int page0 = chunk_at(t >> 1) * ppc;
         for (int pg = 0; pg < ppc; ++pg) {
           // pages past the end re-read the last page: finite data, weight zero
@@ -138,200 +127,180 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     if (lane == 0) {
       const uint32_t idesc_qk = umma_idesc(1, 1, 0, 0, PF_M, PF_N);
       const uint32_t idesc_pv = umma_idesc(1, 1, 0, 1, PF_M, (uint32_t)((p.Dv + 15) / 16 * 16));
-      const uint32_t q_addr = smem_u32(q_s);
+      const uint32_t q_addr = smem_u32(smem), k_addr = q_addr + PF_K_OFF, v_addr = q_addr + PF_V_OFF;
       const int k_steps = (p.D + 15) / 16;
-      bool ok = !*abort_flag && mbar_wait(q_full, 0);
-      if (!ok) {
-        report_error(p.status, ERR_WAIT_FULL, 9000);
+      auto wait = [&](uint64_t* bar, uint32_t parity, int code, int detail) -> bool {
+        if (!*abort_flag && mbar_wait(bar, parity)) return true;
+        report_error(p.status, code, detail);
         *abort_flag = 1;
-      }
-      auto issue_qk = [&](int c) -> bool {
-        const int t = 2 * c, s = t % PF_SLOTS;
-        // the buffer holds P of chunk c - 2 until its P.V has completed
-        if (c >= 2 && (*abort_flag || !mbar_wait(&o_full[c & 1], ((c - 2) >> 1) & 1))) {
-          report_error(p.status, ERR_WAIT_TMEM_EMPTY, 2000 + c);
-          *abort_flag = 1;
-          return false;
-        }
-        if (*abort_flag || !mbar_wait(&full[s], (t / PF_SLOTS) & 1)) {
-          report_error(p.status, ERR_WAIT_FULL, t);
-          *abort_flag = 1;
-          return false;
-        }
+        return false;
+      };
+      bool ok = wait(q_full, 0, ERR_WAIT_FULL, 9000);
+      for (int c = 0; ok && c < n_chunks; ++c) {
+        ok = wait(&full[0], c & 1, ERR_WAIT_FULL, 2 * c);
+        // S takes the place of the previous chunk's P: that chunk's P.V must have completed
+        if (ok && c > 0) ok = wait(o_full, (c - 1) & 1, ERR_WAIT_TMEM_EMPTY, 2000 + c);
+        if (!ok) break;
         tc_fence_after();
-        const uint32_t k_addr = smem_u32(ring + s * PF_TILE);
         for (int k = 0; k < k_steps; ++k) {
           const uint32_t off = (k >> 2) * 16384 + (k & 3) * 32;
-          tc_mma_f16(tmem_base + (c & 1) * PF_N, umma_smem_desc(q_addr + off, 16, 1024),
-                     umma_smem_desc(k_addr + off, 16, 1024), idesc_qk, k != 0);
+          tc_mma_f16(tmem_base, umma_smem_desc(q_addr + off, 16, 1024), umma_smem_desc(k_addr + off, 16, 1024), idesc_qk,
+                     k != 0);
         }
-        tc_commit(&s_full[c & 1]);
-        tc_commit(&empty[s]);
-        return true;
-      };
-      if (ok) ok = issue_qk(0);
-      for (int c = 0; ok && c < n_chunks; ++c) {
-        if (c + 1 < n_chunks) ok = issue_qk(c + 1);
+        tc_commit(s_full);
+        tc_commit(&empty[0]);
+        ok = wait(&full[1], c & 1, ERR_WAIT_FULL, 2 * c + 1) && wait(p_ready, c & 1, ERR_WAIT_TMEM_EMPTY, c);
         if (!ok) break;
-        const int t = 2 * c + 1, s = t % PF_SLOTS;
-        if (*abort_flag || !mbar_wait(&full[s], (t / PF_SLOTS) & 1)) {
-          report_error(p.status, ERR_WAIT_FULL, t);
-          *abort_flag = 1;
-          break;
-        }
-        if (*abort_flag || !mbar_wait(&p_ready[c & 1], (c >> 1) & 1)) {
-          report_error(p.status, ERR_WAIT_TMEM_EMPTY, c);
-          *abort_flag = 1;
-          break;
-        }
         tc_fence_after();
-        const uint32_t v_addr = smem_u32(ring + s * PF_TILE);
-        const uint32_t p_tmem = tmem_base + (c & 1) * PF_N, d_tmem = tmem_base + 256 + (c & 1) * 128;
 #pragma unroll
         for (int k = 0; k < PF_N / 16; ++k) {
           const uint64_t bv = umma_smem_desc(v_addr + k * 2048, 16384, 1024);
-          const uint32_t a = p_tmem + (k >> 1) * 32 + (k & 1) * 8;  // per 32 keys: 16 columns of hi, 16 of lo
-          tc_mma_f16_ta(d_tmem, a, bv, idesc_pv, k != 0);
-          tc_mma_f16_ta(d_tmem, a + 16, bv, idesc_pv, 1);
+          const uint32_t a = tmem_base + (k >> 1) * 32 + (k & 1) * 8;  // per 32 keys: 16 columns of hi, 16 of lo
+          tc_mma_f16_ta(tmem_base + 128, a, bv, idesc_pv, c != 0 || k != 0);
+          tc_mma_f16_ta(tmem_base + 128, a + 16, bv, idesc_pv, 1);
         }
-        tc_commit(&o_full[c & 1]);
-        tc_commit(&empty[s]);
+        tc_commit(o_full);
+        tc_commit(&empty[1]);
       }
     }
   } else {
-    // ----------------------- softmax + accumulation (128 threads, thread = query row) -----------------------
-    const int r = tid, qpos = pos0 + r;
-    const uint32_t lane_base = ((uint32_t)(warp * 32)) << 16;
+    // ----------------------- softmax (128 threads, thread = query row) -----------------------
+    const int r = tid, qpos = pos0 + r, qw = pos0 + warp * 32;  // qw: first row of the warp
+    const uint32_t s_addr = tmem_base + (((uint32_t)(warp * 32)) << 16), o_addr = s_addr + 128;
     const float scale2 = p.scale * LOG2E;
-    const int sat = p.bias_len - 1;
-    const float bias_far = p.bias != nullptr ? bias_s[sat] : 0.f;
-    float o_acc[128];
-#pragma unroll
-    for (int i = 0; i < 128; ++i) o_acc[i] = 0.f;
-    float m_run = -INFINITY, l_run = 0.f;
-    float alpha_cur = 1.f, alpha_nxt = 1.f;
+    const bool biased = p.bias != nullptr;
+    const int sat = biased ? p.bias_len - 1 : 0;
+    const float bias_far = biased ? bias_s[sat] : 0.f;
+    float m_ref = -INFINITY, l_run = 0.f;
     bool ok = true;
 
-    auto softmax_chunk = [&](int c) -> float {
-      const int i = c & 1;
-      if (*abort_flag || !mbar_wait(&s_full[i], (c >> 1) & 1)) {
+    for (int c = 0; c < n_chunks; ++c) {
+      if (*abort_flag || !mbar_wait(s_full, c & 1)) {
         report_error(p.status, ERR_WAIT_TMEM_FULL, c);
         *abort_flag = 1;
         ok = false;
       }
+      ok = __all_sync(0xffffffffu, ok);  // the lanes of a warp share its TMEM accesses: they stop together
+      if (!ok) break;
+      tc_fence_after();
       const int c0 = chunk_at(c) * PF_N;
-      // key c0 + e is visible iff e < lim and (e >= wlo or e < kp)
-      const int lim = qpos - c0 + 1;
-      const int wlo = windowed ? qpos - p.window + 1 - c0 : -1;
-      const int kp = keep - c0;
-      const bool all = lim >= PF_N && (wlo <= 0 || kp >= PF_N);
-      const bool far = p.bias == nullptr || qpos - (c0 + PF_N - 1) >= sat;  // every distance is past the table
-      const bool plain = __all_sync(0xffffffffu, all && far);
-      const uint32_t s_addr = tmem_base + lane_base + i * PF_N;
-      // scaled, biased, masked score of element e
-      auto score = [&](uint32_t raw, int e) -> float {
-        float x = fmaf(__uint_as_float(raw), scale2, bias_far);
-        if (!plain) {
-          if (p.bias != nullptr) x = fmaf(__uint_as_float(raw), scale2, bias_s[max(0, min(qpos - c0 - e, sat))]);
-          if (!(e < lim && (e >= wlo || e < kp))) x = -INFINITY;
-        }
-        return x;
-      };
+      // 32-key groups, as this warp sees them: bit j of `none`: nothing visible; of `plain`: all visible, all far
+      uint32_t none = 0, plain = 0;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int k0 = c0 + 32 * j, dmin = qw - (k0 + 31), dmax = qw + 31 - k0;
+        if (dmax < 0 || (windowed && dmin >= p.window && k0 >= keep)) none |= 1u << j;
+        else if (dmin >= sat && dmin >= 0 && scale2 > 0.f && (!windowed || dmax < p.window || k0 + 31 < keep)) plain |= 1u << j;
+      }
+      // pass 1: row maximum. Blocks with masks or table distances leave their final scores in place of the raw ones.
       float cmax = -INFINITY;
-      if (ok) {
-        tc_fence_after();
 #pragma unroll 1
-        for (int j = 0; j < PF_N / 32; ++j) {
-          uint32_t v[32];
-          tmem_ld_32x32(s_addr + j * 32, v);
-          tmem_ld_wait();
-          if (plain) {
-            // scale2 may be negative: take both ends
-            float hi = __uint_as_float(v[0]), lo = hi;
+      for (int j = 0; j < 4; ++j) {
+        if (none >> j & 1) continue;
+        uint32_t v[32];
+        tmem_ld_32x32(s_addr + j * 32, v);
+        tmem_ld_wait();
+        float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+        if (plain >> j & 1) {
 #pragma unroll
-            for (int e = 1; e < 32; ++e) {
-              hi = fmaxf(hi, __uint_as_float(v[e]));
-              lo = fminf(lo, __uint_as_float(v[e]));
-            }
-            cmax = fmaxf(cmax, fmaf(scale2 >= 0.f ? hi : lo, scale2, bias_far));
-          } else {
+          for (int e = 0; e < 32; ++e) mx[e & 3] = fmaxf(mx[e & 3], __uint_as_float(v[e]));
+          cmax = fmaxf(cmax, fmaf(fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])), scale2, bias_far));
+        } else {
+          const int k0 = c0 + j * 32, dist0 = qpos - k0;
+          const int kp = keep - k0;
 #pragma unroll
-            for (int e = 0; e < 32; ++e) cmax = fmaxf(cmax, score(v[e], j * 32 + e));
+          for (int e = 0; e < 32; ++e) {
+            const int dist = dist0 - e;
+            const float bv = biased ? bias_s[max(0, min(dist, sat))] : 0.f;
+            const bool seen = dist >= 0 && (!windowed || dist < p.window || e < kp);
+            const float x = seen ? fmaf(__uint_as_float(v[e]), scale2, bv) : -INFINITY;
+            mx[e & 3] = fmaxf(mx[e & 3], x);
+            v[e] = __float_as_uint(x);
           }
+          tmem_st_32x32(s_addr + j * 32, v);
+          cmax = fmaxf(cmax, fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])));
         }
       }
-      const float m_new = fmaxf(m_run, cmax);
-      const float m_ref = (m_new == -INFINITY) ? 0.f : m_new;  // no visible key so far: avoid inf - inf
-      const float alpha = exp2f(m_run - m_ref);
-      float lsum = 0.f;
-      if (ok) {
+      tmem_st_wait();
+      // move the reference where the maximum has outgrown it
+      const bool move = cmax > m_ref + PF_SLACK || (m_ref == -INFINITY && cmax > -INFINITY);
+      if (__any_sync(0xffffffffu, move)) {
+        const float m_new = move ? cmax : m_ref;
+        const float alpha = move ? exp2f(m_ref - m_new) : 1.f;  // exp2(-inf) = 0: nothing seen before
+        l_run *= alpha;
+        m_ref = m_new;
+        if (c > 0) {  // S of this chunk was issued after the previous P.V had completed: O is at rest
 #pragma unroll 1
-        for (int j = 0; j < PF_N / 32; ++j) {
-          uint32_t v[32], w[32];
-          tmem_ld_32x32(s_addr + j * 32, v);
-          tmem_ld_wait();
-#pragma unroll
-          for (int e = 0; e < 32; e += 2) {
-            const float p0 = exp2f(score(v[e], j * 32 + e) - m_ref);
-            const float p1 = exp2f(score(v[e + 1], j * 32 + e + 1) - m_ref);
-            lsum += p0 + p1;
-            const __nv_bfloat162 h = __floats2bfloat162_rn(p0, p1);
-            const float2 hf = __bfloat1622float2(h);
-            w[e >> 1] = *reinterpret_cast<const uint32_t*>(&h);
-            w[16 + (e >> 1)] = pack_bf16x2(p0 - hf.x, p1 - hf.y);
-          }
-          tmem_st_32x32(s_addr + j * 32, w);
-        }
-        tmem_st_wait();
-      }
-      m_run = m_new;
-      l_run = l_run * alpha + lsum;
-      tc_fence_before();
-      __syncwarp();
-      if (lane == 0) mbar_arrive(&p_ready[i]);
-      return alpha;
-    };
-
-    alpha_cur = softmax_chunk(0);
-    for (int c = 0; c < n_chunks; ++c) {
-      const int i = c & 1;
-      if (c + 1 < n_chunks) alpha_nxt = softmax_chunk(c + 1);
-      if (ok && (*abort_flag || !mbar_wait(&o_full[i], (c >> 1) & 1))) {
-        report_error(p.status, ERR_WAIT_TMEM_FULL, 1000 + c);
-        *abort_flag = 1;
-        ok = false;
-      }
-      // the lanes of a warp share its TMEM loads: they stop together
-      ok = __all_sync(0xffffffffu, ok);
-      if (ok) {
-        tc_fence_after();
-        const uint32_t o_addr = tmem_base + lane_base + 256 + i * 128;
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          if (j * 32 < p.Dv) {
+          for (int j = 0; j * 32 < p.Dv; ++j) {
             uint32_t v[32];
             tmem_ld_32x32(o_addr + j * 32, v);
             tmem_ld_wait();
 #pragma unroll
-            for (int e = 0; e < 32; ++e) o_acc[j * 32 + e] = o_acc[j * 32 + e] * alpha_cur + __uint_as_float(v[e]);
+            for (int e = 0; e < 32; ++e) v[e] = __float_as_uint(__uint_as_float(v[e]) * alpha);
+            tmem_st_32x32(o_addr + j * 32, v);
           }
         }
       }
-      alpha_cur = alpha_nxt;
-      if (!ok) break;
+      const float ref = m_ref == -INFINITY ? 0.f : m_ref;
+      // pass 2: weights, hi and lo terms over the scores they came from
+      float ls[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 1
+      for (int j = 0; j < 4; ++j) {
+        uint32_t v[32];
+        if (none >> j & 1) {
+#pragma unroll
+          for (int e = 0; e < 32; ++e) v[e] = 0;
+        } else {
+          const bool pl = plain >> j & 1;
+          const float a = pl ? scale2 : 1.f, bb = pl ? bias_far - ref : -ref;
+          tmem_ld_32x32(s_addr + j * 32, v);
+          tmem_ld_wait();
+          uint32_t w[32];
+#pragma unroll
+          for (int e = 0; e < 32; e += 2) {
+            const float p0 = exp2f(fmaf(__uint_as_float(v[e]), a, bb)), p1 = exp2f(fmaf(__uint_as_float(v[e + 1]), a, bb));
+            ls[e >> 1 & 3] += p0 + p1;
+            const uint32_t h = pack_bf16x2(p0, p1);
+            w[e >> 1] = h;
+            w[16 + (e >> 1)] = pack_bf16x2(p0 - __uint_as_float(h << 16), p1 - __uint_as_float(h & 0xffff0000u));
+          }
+#pragma unroll
+          for (int e = 0; e < 32; ++e) v[e] = w[e];
+        }
+        tmem_st_32x32(s_addr + j * 32, v);
+      }
+      l_run += (ls[0] + ls[1]) + (ls[2] + ls[3]);
+      tmem_st_wait();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(p_ready);
     }
-    if (ok && r0 + r < n_q) {
+    if (ok && (*abort_flag || !mbar_wait(o_full, (n_chunks - 1) & 1))) {
+      report_error(p.status, ERR_WAIT_TMEM_FULL, 1000);
+      *abort_flag = 1;
+      ok = false;
+    }
+    ok = __all_sync(0xffffffffu, ok);
+    if (ok) {
+      tc_fence_after();
       const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
       __nv_bfloat16* dst = p.out + (long long)(q_first + r0 + r) * p.out_stride + (long long)hq * p.Dv;
+#pragma unroll 1
+      for (int j = 0; j * 32 < p.Dv; ++j) {
+        uint32_t v[32];
+        tmem_ld_32x32(o_addr + j * 32, v);
+        tmem_ld_wait();
+        if (r0 + r < n_q) {
 #pragma unroll
-      for (int j = 0; j < 16; ++j) {
-        if (j * 8 < p.Dv) {
-          uint4 w;
-          w.x = pack_bf16x2(o_acc[8 * j] * inv, o_acc[8 * j + 1] * inv);
-          w.y = pack_bf16x2(o_acc[8 * j + 2] * inv, o_acc[8 * j + 3] * inv);
-          w.z = pack_bf16x2(o_acc[8 * j + 4] * inv, o_acc[8 * j + 5] * inv);
-          w.w = pack_bf16x2(o_acc[8 * j + 6] * inv, o_acc[8 * j + 7] * inv);
-          reinterpret_cast<uint4*>(dst)[j] = w;
+          for (int k = 0; k < 4; ++k) {
+            if (j * 32 + k * 8 < p.Dv) {
+              float f[8];
+#pragma unroll
+              for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(v[8 * k + e]) * inv;
+              *reinterpret_cast<uint4*>(dst + j * 32 + k * 8) = make_uint4(
+                  pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
+            }
+          }
         }
       }
     }
@@ -341,7 +310,7 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   __syncthreads();
   if (warp == 5) {
     tc_fence_after();
-    tmem_dealloc(tmem_base, 512);
+    tmem_dealloc(tmem_base, 256);
   }
 }
 

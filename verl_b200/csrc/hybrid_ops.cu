@@ -137,9 +137,11 @@ __global__ void add_rmsnorm_kernel(const T* __restrict__ delta, long long delta_
 
 // ---------------------------------------------------------------------------------------------------------------
 // gu rows hold [gate (F) | up (F)]: g = min(gate, limit), u = clamp(up, -limit, limit), y = g sigmoid(alpha g) (u + 1).
+template <typename T>
 __device__ __forceinline__ float clamped_glu_1(float g, float u, float limit, float alpha) {
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
+  if (sizeof(T) == 2) return __fdividef(g, 1.f + __expf(-alpha * g)) * (u + 1.f);  // error far below a bf16 ulp
   return g / (1.f + expf(-alpha * g)) * (u + 1.f);
 }
 template <typename T>
@@ -157,14 +159,14 @@ __global__ void clamped_glu_kernel(const T* __restrict__ gu, long long stride, T
       ld8(gu + t * stride + c, g);
       ld8(gu + t * stride + F + c, u);
 #pragma unroll
-      for (int k = 0; k < 8; ++k) g[k] = clamped_glu_1(g[k], u[k], limit, alpha);
+      for (int k = 0; k < 8; ++k) g[k] = clamped_glu_1<T>(g[k], u[k], limit, alpha);
       st8(y + t * F + c, g);
     }
   } else {
     for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += step) {
       const long long t = i / F;
       const int c = (int)(i - t * F);
-      y[i] = from_f<T>(clamped_glu_1(to_f<T>(gu[t * stride + c]), to_f<T>(gu[t * stride + F + c]), limit, alpha));
+      y[i] = from_f<T>(clamped_glu_1<T>(to_f<T>(gu[t * stride + c]), to_f<T>(gu[t * stride + F + c]), limit, alpha));
     }
   }
 }

@@ -264,7 +264,9 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
             seen = max_ctx or block_table.shape[1] * BS
             if window > 0:
                 seen = min(seen, window + keep_first + 128)
-            splits = _lib.fn("vb_decode_num_splits")(B, Hk, seen)
+            # split the keys only as far as all pieces run at once (two CTAs per SM): windows leave few chunks to walk
+            sms = torch.cuda.get_device_properties(q.device).multi_processor_count
+            splits = max(1, min(2 * sms // (B * Hk), (seen + 127) // 128, 16))
             work = torch.empty(B * Hq * splits * (Dv + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
             rc = _lib.fn("vb_paged_decode_window")(*args, k_cache.shape[0], *table, seq_lens.data_ptr(), B, Hq, Hk, D, Dv, BS,
                                                    *mask, splits, *dst, _lib.ptr(work),

@@ -7,27 +7,42 @@ import torch.nn.functional as F
 
 from . import _lib
 
+CHUNK_MIN = 32  # portions of at least this many tokens take the chunked tensor-core form
+
 
 def delta_rule(proj: torch.Tensor, conv_w: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, norm_w: torch.Tensor,
                ring: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor, seq_lens: torch.Tensor, slots: torch.Tensor,
-               max_q: int, heads: int, kv_heads: int, dim: int, vdim: int, eps: float) -> torch.Tensor:
+               max_q: int, heads: int, kv_heads: int, dim: int, vdim: int, eps: float, impl: str = "auto") -> torch.Tensor:
     """Mixer output before its last projection, [T, heads * vdim].
 
     ``proj`` [T, q | k | v | gate | b | a (| padding)] of ragged sequences (``cu_q`` [B + 1]); ``seq_lens`` [B] = tokens of
     each sequence up to and including these; ``slots`` [B] int32 = state slot (< 0: padding row). Updates in place
     ``state`` fp32 [slots, heads, vdim, dim] and ``ring`` [slots, taps, channels] (convolution inputs, position p in row
-    p % taps). Sequences that start at position 0 ignore what their slot held. ``max_q`` == 1: one token per sequence."""
+    p % taps). Sequences that start at position 0 ignore what their slot held. ``max_q`` == 1: one token per sequence.
+
+    ``impl`` (portions longer than a token): "chunk" = chunks of 64 tokens on the tensor cores (bf16, head sizes in
+    multiples of 8, keys up to 128), "scan" = token by token in fp32, "auto" = "chunk" for bf16 portions of 32 tokens up."""
     T, B, taps = proj.shape[0], slots.numel(), conv_w.shape[1]
     C = 2 * kv_heads * dim + heads * vdim
     out = torch.empty((T, heads * vdim), dtype=proj.dtype, device=proj.device)
     if proj.is_cuda:
-        qkv = gates = None
+        qkv = gates = unit = scratch = None
         if max_q > 1:
-            qkv = torch.empty((T, C), dtype=torch.float32, device=proj.device)
-            gates = torch.empty((T, 2 * heads), dtype=torch.float32, device=proj.device)
+            can = proj.dtype == torch.bfloat16 and bool(_lib.fn("vb_delta_chunk_supported")(dim, vdim))
+            if impl == "chunk" and not can:
+                raise ValueError(f"the chunked delta rule does not support dim={dim} vdim={vdim} in {proj.dtype}")
+            chunk = can and (impl == "chunk" or (impl == "auto" and max_q >= CHUNK_MIN))
+            new = lambda *shape: torch.empty(shape, dtype=torch.float32, device=proj.device)  # noqa: E731
+            gates = new(T, 2 * heads)
+            if chunk:
+                qkv, unit = torch.empty((T, C), dtype=torch.bfloat16, device=proj.device), new(T, 2 * kv_heads)
+                scratch = torch.empty(_lib.fn("vb_delta_chunk_bytes")(T, B, heads), dtype=torch.uint8, device=proj.device)
+            else:
+                qkv = new(T, C)
         rc = _lib.fn("vb_delta_rule")(proj.data_ptr(), proj.stride(0), conv_w.data_ptr(), a_log.data_ptr(), dt_bias.data_ptr(),
                                       norm_w.data_ptr(), ring.data_ptr(), state.data_ptr(), cu_q.data_ptr(),
-                                      seq_lens.data_ptr(), slots.data_ptr(), _lib.ptr(qkv), _lib.ptr(gates), out.data_ptr(),
+                                      seq_lens.data_ptr(), slots.data_ptr(), _lib.ptr(qkv), _lib.ptr(unit), _lib.ptr(gates),
+                                      _lib.ptr(scratch), out.data_ptr(),
                                       out.stride(0), T, B, int(max_q), heads, kv_heads, dim, vdim, taps, float(eps),
                                       int(proj.dtype == torch.float32), _lib.stream())
         _lib.check(rc, "vb_delta_rule")

@@ -1,0 +1,236 @@
+"""Serving throughput of a layer-list model beside a homogeneous model of equal size: prefill and decode through the
+rollout engine (random weights), and every kernel of the layer beside its counterpart.
+
+    python bench.py --serving fuganex-8b [--serving-vs llama-3-8b] [--serving-layers 6] [--serving-kernels]
+
+All times are CUDA events after warm-up on inputs larger than L2 (or rotated over enough copies). Rooflines: bytes over
+the measured copy bandwidth, flops over the measured bf16 matrix throughput (``MEASURED_PEAKS.json``).
+"""
+
+from __future__ import annotations
+
+import json
+import os
+from pathlib import Path
+
+import torch
+
+from .. import ops
+from ..models import build_model, preset
+from ..ops import _lib
+from .engine import NativeRolloutEngine
+
+
+def _peaks() -> tuple[float, float, str]:
+    p = Path(__file__).resolve().parents[2] / "MEASURED_PEAKS.json"
+    if p.exists():
+        d = json.loads(p.read_text())
+        return d["hbm_gbs"], d["bf16_tflops"], "measured"
+    return 6650.0, 1590.0, "fallback"
+
+
+def time_us(fn, iters: int = 10, warmup: int = 3) -> float:
+    """Microseconds per call: the calls are captured into one CUDA graph, so host time is not measured."""
+    for _ in range(warmup):
+        fn()
+    torch.cuda.synchronize()
+    g = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(g):
+        for _ in range(iters):
+            fn()
+    g.replay()
+    torch.cuda.synchronize()
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    e0.record()
+    g.replay()
+    e1.record()
+    torch.cuda.synchronize()
+    return e0.elapsed_time(e1) / iters * 1e3
+
+
+def model_config(name: str, layers: int):
+    """The preset with ``layers`` layers (layer-list models: their first ``layers`` layers)."""
+    full = preset(name)
+    if full.is_layer_list:
+        return preset(name, layer_specs=full.layer_specs[:layers])
+    return preset(name, num_hidden_layers=layers)
+
+
+def bench_model(name: str, layers: int, prefills: list[tuple[int, int]], decodes: list[tuple[int, int]], iters: int) -> dict:
+    """Prefill of ``(prompts, length)`` and decode steps of ``(sequences, context)``: one engine per point."""
+    dev = torch.device("cuda")
+    cfg = model_config(name, layers)
+    model = build_model(cfg, dtype=torch.bfloat16, device=dev)
+    out = {"model": name, "layers": layers, "parameters_1e9": round(cfg.num_parameters() / 1e9, 3), "prefill": [], "decode": []}
+    gen = torch.Generator().manual_seed(0)
+    for B, n in prefills:
+        eng = NativeRolloutEngine(model, max_num_seqs=B, max_model_len=n + 16, max_num_batched_tokens=B * n,
+                                  num_blocks=B * (n // 16 + 2), enable_prefix_caching=False)
+        for i in range(B):
+            eng.add_request(str(i), torch.randint(100, cfg.vocab_size - 100, (n,), generator=gen).tolist(), {"max_tokens": 4})
+        k, _ = eng.sched.step()
+        assert k == B
+        lo = [i * n for i in range(B)]
+
+        def prefill():  # same pages, same states (they restart at position 0): the call repeats exactly
+            eng._prefill_forward(list(range(B)), lo)
+
+        for _ in range(3):
+            prefill()
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        for _ in range(iters):
+            prefill()
+        e1.record()
+        torch.cuda.synchronize()
+        ms = e0.elapsed_time(e1) / iters
+        out["prefill"].append({"prompts": B, "len": n, "ms": round(ms, 3), "tokens_per_s": round(B * n / ms * 1e3)})
+        eng.abort_all_requests()
+        eng.sleep()
+        del eng
+    for B, ctx in decodes:
+        eng = NativeRolloutEngine(model, max_num_seqs=B, max_model_len=ctx + 16, max_num_batched_tokens=8192,
+                                  num_blocks=B * (ctx // 16 + 2), enable_prefix_caching=False)
+        st, graph, _ = eng._get_graph(B)
+        per = (ctx + 15) // 16
+        # every row at context `ctx` on pages spread over the cache; not alive, so that replays do not advance
+        st["bt"][:, :per] = torch.randperm(B * per, device=dev).view(B, per).int()
+        st["lens"].fill_(ctx)
+        st["pos"].fill_(ctx - 1)
+        st["alive"].zero_()
+        st["slots"].fill_(-1)
+        if cfg.is_layer_list:
+            st["state"].copy_(torch.arange(B, dtype=torch.int32))
+        for _ in range(3):
+            graph.replay()
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        for _ in range(5 * iters):
+            graph.replay()
+        e1.record()
+        torch.cuda.synchronize()
+        us = e0.elapsed_time(e1) / (5 * iters) * 1e3
+        out["decode"].append({"sequences": B, "ctx": ctx, "us_per_step": round(us, 1), "tokens_per_s": round(B / us * 1e6)})
+        eng.sleep()
+        del eng
+    return out
+
+
+def _paged(B: int, n: int, bs: int, heads: int, dim: int):
+    per = (n + bs - 1) // bs
+    kc = torch.randn(B * per, heads, bs, dim, device="cuda", dtype=torch.bfloat16)
+    vc = torch.randn_like(kc)
+    bt = torch.randperm(B * per, device="cuda").view(B, per).int()
+    return kc, vc, bt
+
+
+@torch.no_grad()
+def bench_kernels(name: str, vs: str, B: int, n: int, DB: int, ctx: int) -> list[dict]:
+    """Kernel times of the layer-list model and of its counterparts: prefill of B x n tokens, decode of DB sequences."""
+    bw, tf, _ = _peaks()
+    cfg, ref = preset(name), preset(vs)
+    att = next(s.mixer for s in cfg.layer_specs if s.kind == "attention")
+    dl = next(s.mixer for s in cfg.layer_specs if s.kind == "delta")
+    glu = next(s.mlp for s in cfg.layer_specs if s.mlp is not None)
+    H, T, bf = cfg.hidden_size, B * n, torch.bfloat16
+    r = lambda *s: torch.randn(*s, device="cuda", dtype=bf)  # noqa: E731
+    rows = []
+
+    def add(kernel, us, nbytes=0.0, flops=0.0):
+        ideal = max(nbytes / bw / 1e3, flops / tf / 1e6)
+        rows.append({"kernel": kernel, "us": round(us, 1), "roofline_us": round(ideal, 1), "frac": round(ideal / us, 3)})
+
+    # norm with residual: fp32 stream against the bf16 stream of the homogeneous model
+    x, res32, res16, w = r(T, H), torch.randn(T, H, device="cuda"), r(T, H), r(H)
+    add("add_rmsnorm (fp32 residual)", time_us(lambda: ops.add_rmsnorm(x, res32, w, 1e-5)), T * H * 12)
+    add("  vs rmsnorm (bf16 residual)", time_us(lambda: ops.rmsnorm(x, w, 1e-5, res16)), T * H * 8)
+    gu = r(T, 2 * glu.ff)
+    add("clamped_glu", time_us(lambda: ops.clamped_glu(gu, glu.ff, glu.limit, glu.alpha)), T * glu.ff * 6)
+    add("  vs swiglu", time_us(lambda: ops.swiglu(gu)), T * glu.ff * 6)
+    del gu
+    # query / key norm and cache write against RoPE + cache write
+    kc, vc, bt = _paged(B, n, 16, att.kv_heads, att.dim)
+    slots = (bt.long()[:, :, None] * 16 + torch.arange(16, device="cuda")).view(B, -1)[:, :n].reshape(-1).contiguous()
+    qkv, qw, kw = r(T, att.q_size + 2 * att.k_size), r(att.q_size), r(att.k_size)
+    nb = T * (2 * att.q_size + 4 * att.k_size) * 2
+    add("qk_norm_kv_write", time_us(lambda: ops.qk_norm_kv_write(qkv, qw, kw, slots, kc, vc, att.heads, 1e-5)), nb)
+    cos, sin = ops.rope_tables(ref.head_dim, n, 1e6, "cuda")
+    pos = torch.arange(n, device="cuda").repeat(B)
+    hq, hk, d = att.heads, att.kv_heads, att.dim
+
+    def rope_write():
+        y = ops.rope_qkv(qkv, pos, cos, sin, hq, hk, d)
+        ops.kv_cache_write(y[:, att.q_size : att.q_size + att.k_size].view(T, hk, d),
+                           y[:, att.q_size + att.k_size :].view(T, hk, d), slots, kc, vc)
+
+    add("  vs rope + kv_cache_write", time_us(rope_write), nb)
+    # prefill attention
+    qkv.normal_()
+    q = qkv[:, : att.q_size].view(T, hq, d)
+    cu = torch.arange(B + 1, device="cuda", dtype=torch.int32) * n
+    lens = torch.full((B,), n, device="cuda", dtype=torch.int32)
+    bias = torch.randn(hq, int(att.bias_max) + 1, device="cuda")
+    i = torch.arange(n, dtype=torch.float64)
+    pairs = float((torch.minimum(i + 1, torch.full_like(i, att.window) + torch.minimum(
+        torch.full_like(i, att.keep_first), (i + 1 - att.window).clamp(min=0)))).sum())
+    kw_ = dict(scale=att.scale, window=att.window, keep_first=att.keep_first, bias=bias)
+    add(f"paged_flash (window {att.window}, bias)", time_us(
+        lambda: ops.paged_attention(q, kc, vc, bt, cu, lens, n, **kw_)), T * (2 * hq + 2 * hk) * d * 2, 4 * pairs * B * hq * d)
+    add("paged_flash (full causal, no bias)", time_us(
+        lambda: ops.paged_attention(q, kc, vc, bt, cu, lens, n, scale=att.scale)),
+        T * (2 * hq + 2 * hk) * d * 2, 2.0 * n * (n + 1) * B * hq * d)
+    k = qkv[:, att.q_size : att.q_size + att.k_size].view(T, hk, d)
+    v = qkv[:, att.q_size + att.k_size :].view(T, hk, d)
+    add("  vs flash_fwd (full causal)", time_us(lambda: ops.attention_varlen(q, k, v, cu, n)),
+        T * (2 * hq + 2 * hk) * d * 2, 2.0 * n * (n + 1) * B * hq * d)
+    # decode attention
+    kc, vc, bt = _paged(DB, ctx, 16, hk, d)
+    q1, cu1 = r(DB, hq, d), torch.arange(DB + 1, device="cuda", dtype=torch.int32)
+    lens = torch.full((DB,), ctx, device="cuda", dtype=torch.int32)
+    seen = min(ctx, att.window + att.keep_first)
+    add(f"paged_decode_window (window {att.window}, bias)", time_us(
+        lambda: ops.paged_attention(q1, kc, vc, bt, cu1, lens, 1, max_ctx=ctx, **kw_)), DB * seen * hk * d * 4)
+    splits, work = ops.decode_workspace(DB, hq, hk, d, ctx, "cuda")
+    add("  vs paged_decode_tc (full context)", time_us(
+        lambda: ops.paged_decode_attention(q1, kc, vc, bt, lens, num_splits=splits, work=work)), DB * ctx * hk * d * 4)
+    del kc, vc
+    # delta rule
+    proj = r(T, dl.proj_size)
+    conv, alog = r(dl.channels, dl.conv) * 0.5, torch.zeros(dl.heads, device="cuda")
+    nw, dt = r(dl.vdim), torch.full((dl.heads,), -3.0, device="cuda")
+    nslot = max(B, DB)
+    ring = r(nslot, dl.conv, dl.channels)
+    state = torch.zeros(nslot, dl.heads, dl.vdim, dl.dim, device="cuda")
+    sl = torch.arange(nslot, device="cuda", dtype=torch.int32)
+    lens = torch.full((B,), n, device="cuda", dtype=torch.int32)
+    dims = (dl.heads, dl.kv_heads, dl.dim, dl.vdim, 1e-5)
+    add("delta_rule prefill (conv, recurrence, gated norm)", time_us(
+        lambda: ops.delta_rule(proj, conv, alog, dt, nw, ring, state, cu, lens, sl[:B], n, *dims)),
+        T * (dl.proj_size + dl.out_size) * 2, 6.0 * T * dl.heads * dl.dim * dl.vdim)
+    lens = torch.full((DB,), ctx, device="cuda", dtype=torch.int32)
+    add("delta_rule decode (fused step)", time_us(
+        lambda: ops.delta_rule(proj[:DB], conv, alog, dt, nw, ring, state, cu1, lens, sl[:DB], 1, *dims)),
+        DB * (2 * 4 * dl.heads * dl.dim * dl.vdim + (dl.proj_size + dl.out_size + dl.conv * dl.channels) * 2))
+    return rows
+
+
+def main(args) -> dict:
+    torch.cuda.set_device(0)
+    _lib.load(build_if_missing=False)
+    L = args.serving_layers
+    bw, tf, kind = _peaks()
+    out = {"bench": "serving", "dtype": "bf16", "data": "random tokens, random-init weights",
+           "peaks": {"hbm_gbs": bw, "bf16_tflops": tf, "kind": kind}, "timer": "CUDA events; inputs larger than L2"}
+    prefills, decodes = [(8, 1024), (8, 2048), (2, 8192)], [(16, 2048), (128, 1024), (128, 4096)]
+    out["models"] = [bench_model(m, L, prefills, decodes, args.steps if args.steps > 2 else 5)
+                     for m in (args.serving, args.serving_vs)]
+    if args.serving_kernels:
+        out["kernels"] = {f"prefill {b}x{n}, decode {db}x{c}": bench_kernels(args.serving, args.serving_vs, b, n, db, c)
+                          for b, n, db, c in ((8, 2048, 128, 2048), (2, 8192, 32, 8192))}
+    code, blk, detail = _lib.read_status()
+    if code:
+        raise RuntimeError(f"a kernel gave up waiting: code {code} (block {blk}, detail {detail})")
+    print(json.dumps(out))
+    return out
