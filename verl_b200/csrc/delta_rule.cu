@@ -32,6 +32,7 @@
 // both operands and sums are fp32.
 #include "common.cuh"
 #include "host_utils.h"
+#include <type_traits>
 
 namespace vb {
 
@@ -41,9 +42,39 @@ template <typename T>
 __device__ __forceinline__ T dl_t(float v) { return static_cast<T>(v); }
 
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+// For results that are rounded to bf16: the fast exponential and quotient err far below one bf16 ulp.
+template <typename T>
+__device__ __forceinline__ float silu_t(float x) {
+  return sizeof(T) == 2 ? __fdividef(x, 1.f + __expf(-x)) : silu_f(x);
+}
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 constexpr float UNIT_EPS = 1e-6f;
+
+// N consecutive elements, N * sizeof(T) aligned (N a power of two, at most 16 bytes at once).
+template <typename T, int N>
+__device__ __forceinline__ void load_n(const T* p, float (&f)[N]) {
+  constexpr int W = sizeof(T) * N > 16 ? 16 / sizeof(T) : N;
+  struct alignas(sizeof(T) * W) Vec { T v[W]; };
+#pragma unroll
+  for (int i = 0; i < N / W; ++i) {
+    const Vec x = reinterpret_cast<const Vec*>(p)[i];
+#pragma unroll
+    for (int j = 0; j < W; ++j) f[i * W + j] = dl_f<T>(x.v[j]);
+  }
+}
+template <typename T, int N>
+__device__ __forceinline__ void store_n(T* p, const float (&f)[N]) {
+  constexpr int W = sizeof(T) * N > 16 ? 16 / sizeof(T) : N;
+  struct alignas(sizeof(T) * W) Vec { T v[W]; };
+#pragma unroll
+  for (int i = 0; i < N / W; ++i) {
+    Vec x;
+#pragma unroll
+    for (int j = 0; j < W; ++j) x.v[j] = dl_t<T>(f[i * W + j]);
+    reinterpret_cast<Vec*>(p)[i] = x;
+  }
+}
 
 struct DeltaParams {
   const void* proj;        // [T, stride]
@@ -68,8 +99,9 @@ struct DeltaParams {
 
 // ---------------------------------------------------------------------------------------------------------------
 // One warp per (sequence, tile of tokens, head row); lanes across the head's channels, a sliding window of inputs in
-// registers. Head rows: Hk of q, Hk of k, H of v; one more row does the gates.
-constexpr int DP_TT = 32;  // tokens per tile
+// registers. Head rows: Hk of q, Hk of k, H of v; a few more rows do the gates.
+constexpr int DP_TT = 64;  // tokens per tile
+constexpr int DP_GATE_ROWS = 8;  // warps that share a tile's gates
 template <typename T, int TAPS, int CPL, bool CHUNK>
 __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaParams p) {
   pdl_trigger();
@@ -78,12 +110,13 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaParams p) {
   const int first = p.cu_q[b], n = p.cu_q[b + 1] - first;
   const int t0 = blockIdx.x * DP_TT, t1 = min(n, t0 + DP_TT);
   const int slot = p.slots[b], rows = 2 * p.Hk + p.H;
-  if (t0 >= n || r > rows || slot < 0) return;
+  if (t0 >= n || r >= rows + DP_GATE_ROWS || slot < 0) return;
   const int start = p.seq_lens[b] - n;
   const int C = 2 * p.Hk * p.D + p.H * p.V;
   const T* proj = static_cast<const T*>(p.proj) + (long long)first * p.stride;
-  if (r == rows) {
-    for (int i = lane; i < (t1 - t0) * p.H; i += 32) {
+  if (r >= rows) {
+#pragma unroll 4
+    for (int i = (r - rows) * 32 + lane; i < (t1 - t0) * p.H; i += 32 * DP_GATE_ROWS) {
       const int t = t0 + i / p.H, h = i % p.H;
       const T* row = proj + (long long)t * p.stride + C + p.H * p.V;
       float* g = p.gates + (long long)(first + t) * 2 * p.H;
@@ -96,51 +129,82 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaParams p) {
   const int size = qk ? p.D : p.V, c0 = qk ? r * p.D : 2 * p.Hk * p.D + (r - 2 * p.Hk) * p.V;
   const T* ring = static_cast<const T*>(p.ring) + (long long)slot * p.taps * C + c0;
   const T* cw = static_cast<const T*>(p.conv_w) + (long long)c0 * p.taps;
+  // Lane l owns channels l * CPL .. of the head, loaded as one vector where sizes and strides allow.
+  const bool vec = ((p.D | p.V | C | (int)p.stride) & (CPL - 1)) == 0;
+  const int cl = lane * CPL;
+  auto row_in = [&](const T* row, float (&x)[CPL]) {
+    if (vec) {
+      if (cl < size) {
+        load_n<T, CPL>(row + cl, x);
+      } else {
+#pragma unroll
+        for (int i = 0; i < CPL; ++i) x[i] = 0.f;
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < CPL; ++i) x[i] = cl + i < size ? dl_f<T>(row[cl + i]) : 0.f;
+    }
+  };
   // w[j], hist[j]: tap and input of the token j places back; taps beyond p.taps stay zero
   float w[TAPS][CPL], hist[TAPS][CPL];
+  float wv[CPL * TAPS];
+  const bool wvec = vec && p.taps == TAPS;
+  if (wvec && cl < size) load_n<T, CPL * TAPS>(cw + cl * TAPS, wv);
 #pragma unroll
-  for (int j = 0; j < TAPS; ++j)
+  for (int j = 0; j < TAPS; ++j) {
+    const int t = t0 - j;
 #pragma unroll
     for (int i = 0; i < CPL; ++i) {
-      const int c = lane + 32 * i, t = t0 - j;
-      const bool on = c < size && j < p.taps;
-      w[j][i] = on ? dl_f<T>(cw[c * p.taps + p.taps - 1 - j]) : 0.f;
-      float x = 0.f;
-      if (on && j > 0) {
-        if (t >= 0) x = dl_f<T>(proj[(long long)t * p.stride + c0 + c]);
-        else if (start + t >= 0) x = dl_f<T>(ring[(long long)((start + t) % p.taps) * C + c]);
-      }
-      hist[j][i] = x;
+      w[j][i] = 0.f;
+      if (cl + i < size && j < p.taps) w[j][i] = wvec ? wv[i * TAPS + TAPS - 1 - j] : dl_f<T>(cw[(cl + i) * p.taps + p.taps - 1 - j]);
+      hist[j][i] = 0.f;
     }
+    if (j > 0 && j < p.taps) {
+      if (t >= 0) row_in(proj + (long long)t * p.stride + c0, hist[j]);
+      else if (start + t >= 0) row_in(ring + (long long)((start + t) % p.taps) * C, hist[j]);
+    }
+  }
   const float qscale = r < p.Hk ? 1.f / sqrtf((float)p.D) : 1.f;
-  for (int t = t0; t < t1; ++t) {
-    float y[CPL], ss = 0.f;
+  constexpr int PRE = 4;  // tokens whose loads are in flight together
+  for (int tb = t0; tb < t1; tb += PRE) {
+    float xin[PRE][CPL];
 #pragma unroll
-    for (int i = 0; i < CPL; ++i) {
-      const int c = lane + 32 * i;
-      hist[0][i] = c < size ? dl_f<T>(proj[(long long)t * p.stride + c0 + c]) : 0.f;
-      float a = 0.f;
+    for (int k = 0; k < PRE; ++k)
+      if (tb + k < t1) row_in(proj + (long long)(tb + k) * p.stride + c0, xin[k]);
 #pragma unroll
-      for (int j = TAPS - 1; j >= 0; --j) a = fmaf(w[j][i], hist[j][i], a);
+    for (int k = 0; k < PRE; ++k) {
+      const int t = tb + k;
+      if (t >= t1) break;
+      float y[CPL], ss = 0.f;
 #pragma unroll
-      for (int j = TAPS - 1; j > 0; --j) hist[j][i] = hist[j - 1][i];
-      y[i] = silu_f(a);
-      if (CHUNK) y[i] = __bfloat162float(__float2bfloat16(y[i]));  // the norm is that of the stored vector
-      ss += y[i] * y[i];  // channels past the head give silu(0) = 0
-    }
-    float mul = 1.f;
-    if (qk) mul = qscale / sqrtf(warp_reduce_sum(ss) + UNIT_EPS);
-    if (CHUNK) {
-      __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.qkv) + (long long)(first + t) * C + c0;
+      for (int i = 0; i < CPL; ++i) {
+        hist[0][i] = xin[k][i];
+        float a = 0.f;
 #pragma unroll
-      for (int i = 0; i < CPL; ++i)
-        if (lane + 32 * i < size) dst[lane + 32 * i] = __float2bfloat16(y[i]);
-      if (qk && lane == 0) p.unit[(long long)(first + t) * 2 * p.Hk + r] = mul;
-    } else {
-      float* dst = static_cast<float*>(p.qkv) + (long long)(first + t) * C + c0;
+        for (int j = TAPS - 1; j >= 0; --j) a = fmaf(w[j][i], hist[j][i], a);
 #pragma unroll
-      for (int i = 0; i < CPL; ++i)
-        if (lane + 32 * i < size) dst[lane + 32 * i] = y[i] * mul;
+        for (int j = TAPS - 1; j > 0; --j) hist[j][i] = hist[j - 1][i];
+        y[i] = CHUNK ? silu_t<T>(a) : silu_f(a);
+        if (CHUNK) y[i] = __bfloat162float(__float2bfloat16(y[i]));  // the norm is that of the stored vector
+        ss += y[i] * y[i];  // channels past the head give silu(0) = 0
+      }
+      float mul = 1.f;
+      if (qk) mul = qscale / sqrtf(warp_reduce_sum(ss) + UNIT_EPS);
+      typedef typename std::conditional<CHUNK, __nv_bfloat16, float>::type Y;
+      Y* dst = static_cast<Y*>(p.qkv) + (long long)(first + t) * C + c0 + cl;
+      if (!CHUNK) {
+#pragma unroll
+        for (int i = 0; i < CPL; ++i) y[i] *= mul;
+      } else if (qk && lane == 0) {
+        p.unit[(long long)(first + t) * 2 * p.Hk + r] = mul;
+      }
+      if (vec) {
+        if (cl < size) store_n<Y, CPL>(dst, y);
+      } else {
+#pragma unroll
+        for (int i = 0; i < CPL; ++i)
+          if (cl + i < size) dst[i] = dl_t<Y>(y[i]);
+      }
     }
   }
 }
@@ -723,12 +787,36 @@ __global__ void __launch_bounds__(128) gated_norm_kernel(const DeltaParams p, in
   const T* gate = static_cast<const T*>(p.proj) + t * p.stride + 2 * p.Hk * p.D + p.H * p.V + (long long)h * p.V;
   const T* w = static_cast<const T*>(p.norm_w);
   float ss = 0.f;
+  if ((p.V & 3) == 0 && ((p.stride | p.out_stride | (2 * p.Hk * p.D)) & 3) == 0) {
+    float x[2][4], g[2][4];  // V <= 256
+#pragma unroll
+    for (int k = 0; k < 2; ++k)
+      if (lane * 4 + 128 * k < p.V) {
+        load_n<T, 4>(o + lane * 4 + 128 * k, x[k]);
+        load_n<T, 4>(gate + lane * 4 + 128 * k, g[k]);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) ss += x[k][e] * x[k][e];
+      }
+    const float inv = 1.f / sqrtf(warp_reduce_sum(ss) / (float)p.V + p.eps);
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const int c = lane * 4 + 128 * k;
+      if (c < p.V) {
+        float wv[4];
+        load_n<T, 4>(w + c, wv);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) x[k][e] = x[k][e] * inv * wv[e] * silu_t<T>(g[k][e]);
+        store_n<T, 4>(o + c, x[k]);
+      }
+    }
+    return;
+  }
   for (int c = lane; c < p.V; c += 32) {
     const float x = dl_f<T>(o[c]);
     ss += x * x;
   }
   const float inv = 1.f / sqrtf(warp_reduce_sum(ss) / (float)p.V + p.eps);
-  for (int c = lane; c < p.V; c += 32) o[c] = dl_t<T>(dl_f<T>(o[c]) * inv * dl_f<T>(w[c]) * silu_f(dl_f<T>(gate[c])));
+  for (int c = lane; c < p.V; c += 32) o[c] = dl_t<T>(dl_f<T>(o[c]) * inv * dl_f<T>(w[c]) * silu_t<T>(dl_f<T>(gate[c])));
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -872,7 +960,7 @@ __global__ void __launch_bounds__(DD_THREADS) delta_step_kernel(const DeltaParam
 
 template <typename T, bool CHUNK>
 static int run_prep(const DeltaParams& p, int max_q, cudaStream_t stream) {
-  const dim3 g((max_q + DP_TT - 1) / DP_TT, (2 * p.Hk + p.H + 1 + 3) / 4, p.B), b(128);
+  const dim3 g((max_q + DP_TT - 1) / DP_TT, (2 * p.Hk + p.H + DP_GATE_ROWS + 3) / 4, p.B), b(128);
   const int cpl = ((p.D > p.V ? p.D : p.V) + 31) / 32;
   cudaError_t e = cudaErrorInvalidValue;
 #define VB_PREP(TAPS)                                                                                      \
