@@ -33,6 +33,10 @@ CONFIGS = {
                              vocab=200, width=64),
     "delta_only": config([delta(3, 1, 40, 16, 1), delta(1, 1, 64, 128, 5, ff=96)], vocab=200, width=80, eps=1e-5),
     "odd": config([attention(3, 3, 20, 12, 40, 9, bias_max=33.5, ff=52), delta(5, 5, 12, 20, 2, ff=44)], vocab=203, width=52),
+    # 16 query heads on one key head, a distance table past the tensor-core kernels' limit, windows longer than a chunk, kept
+    # tokens past a chunk, a vocabulary that is no multiple of anything
+    "reach": config([attention(16, 1, 16, 16, 140, 150, bias_max=4000, ff=64), delta(4, 4, 16, 32, 6),
+                     attention(4, 2, 32, 64, 130, 3, bias_max=200)], vocab=331),
     "wide_head": config([attention(2, 2, 144, 160, 64, 2, ff=64), delta(2, 1, 160, 136, 4)], vocab=128, width=128),
 }
 

@@ -103,7 +103,7 @@ struct DeltaParams {
 constexpr int DP_TT = 64;  // tokens per tile
 constexpr int DP_GATE_ROWS = 8;  // warps that share a tile's gates
 template <typename T, int TAPS, int CPL, bool CHUNK>
-__global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaParams p) {
+__global__ void __launch_bounds__(128, CPL * TAPS <= 16 ? 8 : 1) delta_prep_kernel(const DeltaParams p) {
   pdl_trigger();
   pdl_wait();
   const int lane = threadIdx.x & 31, r = blockIdx.y * 4 + (threadIdx.x >> 5), b = blockIdx.z;
@@ -166,11 +166,12 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaParams p) {
   }
   const float qscale = r < p.Hk ? 1.f / sqrtf((float)p.D) : 1.f;
   constexpr int PRE = 4;  // tokens whose loads are in flight together
+  const T* src = proj + (long long)t0 * p.stride + c0;
   for (int tb = t0; tb < t1; tb += PRE) {
     float xin[PRE][CPL];
 #pragma unroll
-    for (int k = 0; k < PRE; ++k)
-      if (tb + k < t1) row_in(proj + (long long)(tb + k) * p.stride + c0, xin[k]);
+    for (int k = 0; k < PRE; ++k, src += p.stride)
+      if (tb + k < t1) row_in(src, xin[k]);
 #pragma unroll
     for (int k = 0; k < PRE; ++k) {
       const int t = tb + k;
@@ -189,7 +190,7 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaParams p) {
         ss += y[i] * y[i];  // channels past the head give silu(0) = 0
       }
       float mul = 1.f;
-      if (qk) mul = qscale / sqrtf(warp_reduce_sum(ss) + UNIT_EPS);
+      if (qk) mul = qscale * rsqrtf(warp_reduce_sum(ss) + UNIT_EPS);
       typedef typename std::conditional<CHUNK, __nv_bfloat16, float>::type Y;
       Y* dst = static_cast<Y*>(p.qkv) + (long long)(first + t) * C + c0 + cl;
       if (!CHUNK) {
@@ -408,20 +409,19 @@ __device__ __forceinline__ const __nv_bfloat16* frag_bn(const __nv_bfloat16* t, 
   return t + (n + ((lane >> 4) & 1) * 8 + (lane & 7)) * PITCH + k + ((lane >> 3) & 1) * 8;
 }
 
-// One CTA of four warps per (chunk, head): T = (I + A)^-1 diag(beta) and P.
-template <int DP>
+// One CTA of four warps per (chunk, NH heads that share their q and k): T = (I + A)^-1 diag(beta) and P of each.
+template <int DP, int NH>
 __global__ void __launch_bounds__(128) delta_chunk_prep_kernel(const DeltaParams p, uint8_t* __restrict__ scratch) {
-  constexpr int PI = DP + 8, AP = DC + 4, TP = DC + 8;
+  constexpr int PI = DP + 8, AP = DC + 4;
   extern __shared__ uint8_t smb[];
   __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smb);
   __nv_bfloat16* q_s = k_s + DC * PI;
-  float* a_s = reinterpret_cast<float*>(q_s + DC * PI);                      // [64][AP]
-  float* G_s = a_s + DC * AP;                                                // [64]
-  float *b_s = G_s + DC, *nk_s = b_s + DC, *nq_s = nk_s + DC;
-  __nv_bfloat16* t_s = k_s;                                                  // T hi | lo [64][TP] over k_s / q_s, later
+  float* a_s = reinterpret_cast<float*>(q_s + DC * PI);  // [NH][64][AP]
+  float* G_s = a_s + NH * DC * AP;                       // [NH][64]
+  float *b_s = G_s + NH * DC, *nk_s = b_s + NH * DC, *nq_s = nk_s + DC;
   pdl_trigger();
   pdl_wait();
-  const int idx = blockIdx.x, h = blockIdx.y;
+  const int idx = blockIdx.x, h = blockIdx.y * NH;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   int lo = 0, hi = p.B - 1;
   while (lo < hi) {
@@ -443,33 +443,38 @@ __global__ void __launch_bounds__(128) delta_chunk_prep_kernel(const DeltaParams
   if (tid < DC) {
     const bool on = t0 + tid < n;
     const long long t = first + t0 + tid;
-    G_s[tid] = on ? p.gates[t * 2 * p.H + p.H + h] : 0.f;
-    b_s[tid] = on ? p.gates[t * 2 * p.H + h] : 0.f;
+#pragma unroll
+    for (int x = 0; x < NH; ++x) {
+      G_s[x * DC + tid] = on ? p.gates[t * 2 * p.H + p.H + h + x] : 0.f;
+      b_s[x * DC + tid] = on ? p.gates[t * 2 * p.H + h + x] : 0.f;
+    }
     nq_s[tid] = on ? p.unit[t * 2 * p.Hk + hk] : 0.f;
     nk_s[tid] = on ? p.unit[t * 2 * p.Hk + p.Hk + hk] : 0.f;
   }
   __syncthreads();
-  if (warp == 0) {  // running sums of the log decays, two tokens per lane
-    const float x0 = G_s[2 * lane], x1 = G_s[2 * lane + 1];
+  if (warp < NH) {  // running sums of the log decays, two tokens per lane
+    float* G = G_s + warp * DC;
+    const float x0 = G[2 * lane], x1 = G[2 * lane + 1];
     float s = x0 + x1;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
       const float v = __shfl_up_sync(0xffffffffu, s, o);
       if (lane >= o) s += v;
     }
-    G_s[2 * lane] = s - x1;
-    G_s[2 * lane + 1] = s;
+    G[2 * lane] = s - x1;
+    G[2 * lane + 1] = s;
   }
   cp_async_wait<0>();
   __syncthreads();
   uint8_t* dst = scratch + ((long long)idx * p.H + h) * DC_BYTES;
-  if (tid < DC) {
-    float* vec = reinterpret_cast<float*>(dst + DC_VEC_OFF);
-    const float g = G_s[tid], gl = G_s[DC - 1], eg = expf(g);
-    vec[tid] = eg * nk_s[tid];
-    vec[DC + tid] = eg * nq_s[tid];
-    vec[2 * DC + tid] = expf(gl - g) * nk_s[tid];
-    if (tid == 0) vec[3 * DC] = expf(gl);
+  if (tid < NH * DC) {
+    const int t = tid % DC;
+    float* vec = reinterpret_cast<float*>(dst + tid / DC * DC_BYTES + DC_VEC_OFF);
+    const float g = G_s[tid], gl = G_s[tid / DC * DC + DC - 1], eg = expf(g);
+    vec[t] = eg * nk_s[t];
+    vec[DC + t] = eg * nq_s[t];
+    vec[2 * DC + t] = expf(gl - g) * nk_s[t];
+    if (t == 0) vec[3 * DC] = expf(gl);
   }
   // Gram matrices of this warp's 16 rows, columns up to the diagonal block
   float kk[8][4] = {}, qk[8][4] = {};
@@ -491,37 +496,42 @@ __global__ void __launch_bounds__(128) delta_chunk_prep_kernel(const DeltaParams
       }
     }
   }
-  uint32_t* P_hi = reinterpret_cast<uint32_t*>(dst) + DC_MAT;  // 32-bit words: T hi, T lo take DC_MAT of them
-  uint32_t* P_lo = P_hi + DC_MAT / 2;
+#pragma unroll
+  for (int x = 0; x < NH; ++x)
 #pragma unroll
   for (int nt = 0; nt < 8; ++nt) {
+    uint32_t* P_hi = reinterpret_cast<uint32_t*>(dst + x * DC_BYTES) + DC_MAT;  // 32-bit words: T takes DC_MAT of them
+    uint32_t* P_lo = P_hi + DC_MAT / 2;
+    const float *G = G_s + x * DC, *beta = b_s + x * DC;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
       const int t = warp * 16 + (lane >> 2) + 8 * half, s = nt * 8 + (lane & 3) * 2;
       float pv[2], av[2];
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const float dec = s + e <= t ? expf(G_s[t] - G_s[s + e]) * nk_s[s + e] : 0.f;
+        const float dec = s + e <= t ? expf(G[t] - G[s + e]) * nk_s[s + e] : 0.f;
         pv[e] = dec * nq_s[t] * qk[nt][2 * half + e];
-        av[e] = s + e < t ? dec * nk_s[t] * b_s[t] * kk[nt][2 * half + e] : 0.f;
+        av[e] = s + e < t ? dec * nk_s[t] * beta[t] * kk[nt][2 * half + e] : 0.f;
       }
       uint32_t ph, pl;
       split2(pv[0], pv[1], ph, pl);
       P_hi[(t * DC + s) >> 1] = ph;
       P_lo[(t * DC + s) >> 1] = pl;
-      *reinterpret_cast<float2*>(a_s + t * AP + s) = make_float2(av[0], av[1]);
+      *reinterpret_cast<float2*>(a_s + (x * DC + t) * AP + s) = make_float2(av[0], av[1]);
     }
   }
   __syncthreads();
-  // forward substitution: thread j owns column j of (I + A)^-1
-  if (tid < DC) {
+  // forward substitution: a thread owns one column of (I + A)^-1
+  if (tid < NH * DC) {
+    const int col = tid % DC;
+    const float* A = a_s + tid / DC * DC * AP;
     float x[DC];
 #pragma unroll
     for (int i = 0; i < DC; ++i) {
-      float s0 = i == tid ? 1.f : 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
+      float s0 = i == col ? 1.f : 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
 #pragma unroll
       for (int k = 0; k < i; k += 4) {
-        const float4 a = *reinterpret_cast<const float4*>(a_s + i * AP + k);  // entries from the diagonal on are zero
+        const float4 a = *reinterpret_cast<const float4*>(A + i * AP + k);  // entries from the diagonal on are zero
         s0 = fmaf(-a.x, x[k], s0);
         if (k + 1 < i) s1 = fmaf(-a.y, x[k + 1], s1);
         if (k + 2 < i) s2 = fmaf(-a.z, x[k + 2], s2);
@@ -530,18 +540,14 @@ __global__ void __launch_bounds__(128) delta_chunk_prep_kernel(const DeltaParams
       x[i] = (s0 + s1) + (s2 + s3);
     }
     const float beta = b_s[tid];
+    __nv_bfloat16* t_hi = reinterpret_cast<__nv_bfloat16*>(dst + tid / DC * DC_BYTES) + col;
 #pragma unroll
-    for (int i = 0; i < DC; ++i) {
+    for (int i = 0; i < DC; ++i) {  // a warp stores 32 neighbouring columns
       const float v = x[i] * beta;
       const __nv_bfloat16 vh = __float2bfloat16(v);
-      t_s[i * TP + tid] = vh;
-      t_s[(DC + i) * TP + tid] = __float2bfloat16(v - __bfloat162float(vh));
+      t_hi[i * DC] = vh;
+      t_hi[DC_MAT + i * DC] = __float2bfloat16(v - __bfloat162float(vh));
     }
-  }
-  __syncthreads();
-  for (int i = tid; i < 2 * DC * 8; i += 128) {
-    const int r = i >> 3, c = (i & 7) * 8;
-    *reinterpret_cast<uint4*>(dst + (r * DC + c) * 2) = *reinterpret_cast<const uint4*>(t_s + r * TP + c);
   }
 }
 
@@ -773,50 +779,51 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_scan_kernel(const DeltaPar
 }
 
 // ---------------------------------------------------------------------------------------------------------------
-// out = rmsnorm(out) * w * silu(gate) per (token, head), in place. One warp each.
+// out = rmsnorm(out) * w * silu(gate) per (token, head), in place. A warp takes GN_T tokens of one head.
+constexpr int GN_T = 4;
 template <typename T>
-__global__ void __launch_bounds__(128) gated_norm_kernel(const DeltaParams p, int T_) {
+__global__ void __launch_bounds__(128) gated_norm_kernel(const DeltaParams p, int tokens) {
   pdl_trigger();
   pdl_wait();
-  const int lane = threadIdx.x & 31;
-  const long long i = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
-  if (i >= (long long)T_ * p.H) return;
-  const long long t = i / p.H;
-  const int h = (int)(i % p.H);
-  T* o = static_cast<T*>(p.out) + t * p.out_stride + (long long)h * p.V;
-  const T* gate = static_cast<const T*>(p.proj) + t * p.stride + 2 * p.Hk * p.D + p.H * p.V + (long long)h * p.V;
+  const int lane = threadIdx.x & 31, h = blockIdx.y * 4 + (threadIdx.x >> 5);
+  if (h >= p.H) return;
+  const int t0 = blockIdx.x * GN_T, cnt = min(GN_T, tokens - t0);
+  T* o = static_cast<T*>(p.out) + (long long)t0 * p.out_stride + (long long)h * p.V;
+  const T* gate = static_cast<const T*>(p.proj) + (long long)t0 * p.stride + 2 * p.Hk * p.D + p.H * p.V + (long long)h * p.V;
   const T* w = static_cast<const T*>(p.norm_w);
-  float ss = 0.f;
-  if ((p.V & 3) == 0 && ((p.stride | p.out_stride | (2 * p.Hk * p.D)) & 3) == 0) {
-    float x[2][4], g[2][4];  // V <= 256
+  const float inv_v = 1.f / (float)p.V;
+  const int c = lane * 4;
+  if (p.V <= 128 && ((p.V | (int)p.stride | (int)p.out_stride | (2 * p.Hk * p.D)) & 3) == 0) {
+    const bool on = c < p.V;
+    float x[GN_T][4] = {}, g[GN_T][4], wv[4];
+    if (on) load_n<T, 4>(w + c, wv);
 #pragma unroll
-    for (int k = 0; k < 2; ++k)
-      if (lane * 4 + 128 * k < p.V) {
-        load_n<T, 4>(o + lane * 4 + 128 * k, x[k]);
-        load_n<T, 4>(gate + lane * 4 + 128 * k, g[k]);
-#pragma unroll
-        for (int e = 0; e < 4; ++e) ss += x[k][e] * x[k][e];
+    for (int k = 0; k < GN_T; ++k)
+      if (on && k < cnt) {
+        load_n<T, 4>(o + k * p.out_stride + c, x[k]);
+        load_n<T, 4>(gate + k * p.stride + c, g[k]);
       }
-    const float inv = 1.f / sqrtf(warp_reduce_sum(ss) / (float)p.V + p.eps);
 #pragma unroll
-    for (int k = 0; k < 2; ++k) {
-      const int c = lane * 4 + 128 * k;
-      if (c < p.V) {
-        float wv[4];
-        load_n<T, 4>(w + c, wv);
+    for (int k = 0; k < GN_T; ++k) {
+      const float ss = x[k][0] * x[k][0] + x[k][1] * x[k][1] + x[k][2] * x[k][2] + x[k][3] * x[k][3];
+      const float inv = rsqrtf(warp_reduce_sum(ss) * inv_v + p.eps);
+      if (on && k < cnt) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) x[k][e] = x[k][e] * inv * wv[e] * silu_t<T>(g[k][e]);
-        store_n<T, 4>(o + c, x[k]);
+        store_n<T, 4>(o + k * p.out_stride + c, x[k]);
       }
     }
     return;
   }
-  for (int c = lane; c < p.V; c += 32) {
-    const float x = dl_f<T>(o[c]);
-    ss += x * x;
+  for (int k = 0; k < cnt; ++k, o += p.out_stride, gate += p.stride) {
+    float ss = 0.f;
+    for (int i = lane; i < p.V; i += 32) {
+      const float x = dl_f<T>(o[i]);
+      ss += x * x;
+    }
+    const float inv = rsqrtf(warp_reduce_sum(ss) * inv_v + p.eps);
+    for (int i = lane; i < p.V; i += 32) o[i] = dl_t<T>(dl_f<T>(o[i]) * inv * dl_f<T>(w[i]) * silu_t<T>(dl_f<T>(gate[i])));
   }
-  const float inv = 1.f / sqrtf(warp_reduce_sum(ss) / (float)p.V + p.eps);
-  for (int c = lane; c < p.V; c += 32) o[c] = dl_t<T>(dl_f<T>(o[c]) * inv * dl_f<T>(w[c]) * silu_t<T>(dl_f<T>(gate[c])));
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -952,7 +959,7 @@ __global__ void __launch_bounds__(DD_THREADS) delta_step_kernel(const DeltaParam
   __syncthreads();
   float ss = 0.f;
   for (int c = lane; c < p.V; c += 32) ss += o_s[c] * o_s[c];
-  const float inv = 1.f / sqrtf(warp_reduce_sum(ss) / (float)p.V + p.eps);
+  const float inv = rsqrtf(warp_reduce_sum(ss) * (1.f / (float)p.V) + p.eps);
   const T* gate = proj + C + (long long)h * p.V;
   const T* w = static_cast<const T*>(p.norm_w);
   for (int c = tid; c < p.V; c += DD_THREADS) out[c] = dl_t<T>(o_s[c] * inv * dl_f<T>(w[c]) * silu_f(dl_f<T>(gate[c])));
@@ -1000,16 +1007,20 @@ static int run_step(const DeltaParams& p, cudaStream_t stream) {
 template <int DP>
 static int run_chunks(const DeltaParams& p, int tokens, uint8_t* scratch, cudaStream_t stream) {
   constexpr int PI = DP + 8, XP = DC_VB + 8;
-  const int smem1 = 2 * DC * PI * 2 + (DC * (DC + 4) + 4 * DC) * 4;
+  const int nh = (p.H / p.Hk) % 2 == 0 ? 2 : 1;
+  const int smem1 = 2 * DC * PI * 2 + (nh * DC * (DC + 4) + (2 * nh + 2) * DC) * 4;
   const int smem2 = (4 * DC * PI + 2 * DC * XP + 8 * DC * XP + 2 * DP * XP) * 2 + 8 * DC * 4;
   static bool attr = false;
   if (!attr) {
-    VB_CUDA_CHECK(cudaFuncSetAttribute(delta_chunk_prep_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem1));
+    const int most = 2 * DC * PI * 2 + (2 * DC * (DC + 4) + 6 * DC) * 4;
+    VB_CUDA_CHECK(cudaFuncSetAttribute(delta_chunk_prep_kernel<DP, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, most));
+    VB_CUDA_CHECK(cudaFuncSetAttribute(delta_chunk_prep_kernel<DP, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, most));
     VB_CUDA_CHECK(cudaFuncSetAttribute(delta_chunk_scan_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2));
     attr = true;
   }
-  cudaError_t e = vb_launch_pdl(delta_chunk_prep_kernel<DP>, dim3(tokens / DC + p.B, p.H), dim3(128), smem1, stream, 1, p,
-                                scratch);
+  const dim3 g1(tokens / DC + p.B, p.H / nh);
+  cudaError_t e = nh == 2 ? vb_launch_pdl(delta_chunk_prep_kernel<DP, 2>, g1, dim3(128), smem1, stream, 1, p, scratch)
+                          : vb_launch_pdl(delta_chunk_prep_kernel<DP, 1>, g1, dim3(128), smem1, stream, 1, p, scratch);
   if (e != cudaSuccess) return (int)e;
   e = vb_launch_pdl(delta_chunk_scan_kernel<DP>, dim3((p.V + DC_VB - 1) / DC_VB, p.H, p.B), dim3(256), smem2, stream, 1, p,
                     (const uint8_t*)scratch);
@@ -1036,8 +1047,8 @@ static int run_delta(const DeltaParams& p, int tokens, int max_q, uint8_t* chunk
          : nr == 16 ? run_scan<T, 16>(p, stream)
                     : run_scan<T, 32>(p, stream);
   if (rc) return rc;
-  const long long warps = (long long)tokens * p.H;
-  cudaError_t e = vb_launch_pdl(gated_norm_kernel<T>, dim3((unsigned)((warps + 3) / 4)), dim3(128), 0, stream, 1, p, tokens);
+  cudaError_t e = vb_launch_pdl(gated_norm_kernel<T>, dim3((tokens + GN_T - 1) / GN_T, (p.H + 3) / 4), dim3(128), 0,
+                                stream, 1, p, tokens);
   vb_count_launch();
   return (int)e;
 }
