@@ -21,7 +21,7 @@ import numpy as np
 import torch
 import torch.distributed as dist
 
-from ..models import CausalLM, ModelConfig, preset
+from ..models import CausalLM, ModelConfig, build_model, preset
 from ..models.hf_io import load_hf_checkpoint
 from ..protocol import DataProto
 from ..single_controller.base import Dispatch, Worker, register
@@ -322,7 +322,7 @@ class ActorRolloutRefWorker(_WorkerBase):
         elif self._is_actor and self.world == 1 and not getattr(self, "_lora", False) and not self.actor_engine.model_parallel:
             self.rollout_model = self.actor_engine.model  # same tensors: weight sync is free
         else:
-            self.rollout_model = CausalLM(model_cfg, dtype=dtype, device=self.device)
+            self.rollout_model = build_model(model_cfg, dtype=dtype, device=self.device, init=False)
             if self._is_actor and not self.actor_engine.model_parallel:
                 self._bind_rollout_to_flat()
             elif self._is_actor:
