@@ -25,10 +25,10 @@
 //     u_t = beta_t (v_t - e^{G_t} S0^T k_t - sum_{s<t} e^{G_t - G_s} (k_t . k_s) u_s)       i.e. (I + A) U = B (V - ...)
 //     o_t = e^{G_t} S0^T q_t + sum_{s<=t} e^{G_t - G_s} (q_t . k_s) u_s
 //     S   = e^{G_last} S0 + sum_s e^{G_last - G_s} k_s u_s^T
-// delta_chunk_prep computes T = (I + A)^-1 B and the matrix P of the second sum for all chunks in parallel;
-// delta_chunk_scan walks a sequence's chunks with S in fp32 accumulators. Precision: the convolved q and k are bf16
+// delta_chunk_prep computes T = (I + A)^-1 B and, with P the matrix of the second sum, P T for all chunks in parallel;
+// delta_chunk_scan walks a sequence's chunks on tcgen05 with S in fp32 accumulators. Precision: the convolved q and k are bf16
 // activations and enter the products unnormalised, their fp32 unit-norm factors multiply the results; every other
-// operand (S, T, P, U and the right-hand side) is split into two bf16 terms, so that products carry about 16 bits of
+// operand (S, T, P T, U and the right-hand side) is split into two bf16 terms, so that products carry about 16 bits of
 // both operands and sums are fp32.
 #include "common.cuh"
 #include "host_utils.h"
@@ -357,10 +357,9 @@ __global__ void __launch_bounds__(DS_THREADS) delta_scan_kernel(const DeltaParam
 // Chunked form on the tensor cores. Chunk c of sequence b has index (cu_q[b] / 64) + b + c: distinct for all chunks, at
 // most T / 64 + B of them.
 constexpr int DC = 64;             // tokens per chunk
-constexpr int DC_VB = 64;          // state columns per CTA
 constexpr int DC_MAT = DC * DC;    // one bf16 term of T or P
-// scratch of one (chunk, head): T hi | T lo | P hi | P lo (bf16 [64][64] each), then fp32 vectors
-//   e^{G_t} / |k_t|,  e^{G_t} D^{-1/2} / |q_t|,  e^{G_last - G_t} / |k_t|,  [e^{G_last}, unused ...]
+// scratch of one (chunk, head): T hi | P T hi | T lo | P T lo (bf16 [64][64] each), then fp32 vectors [64]:
+//   e^{G_t} / |k_t|,  e^{G_t} D^{-1/2} / |q_t|,  e^{G_last - G_t} / |k_t|,  e^{G_last} (repeated)
 constexpr int DC_VEC_OFF = 4 * DC_MAT * 2;
 constexpr int DC_BYTES = DC_VEC_OFF + 4 * DC * 4;
 
@@ -393,32 +392,35 @@ template <int PITCH>
 __device__ __forceinline__ const __nv_bfloat16* frag_a(const __nv_bfloat16* t, int row, int col, int lane) {
   return t + (row + (lane & 15)) * PITCH + col + (lane >> 4) * 8;
 }
-// A^T: the tile stores [k][m]; the result is the [16 m x 16 k] operand (ldsm4t)
-template <int PITCH>
-__device__ __forceinline__ const __nv_bfloat16* frag_at(const __nv_bfloat16* t, int m, int k, int lane) {
-  return t + (k + ((lane >> 4) & 1) * 8 + (lane & 7)) * PITCH + m + ((lane >> 3) & 1) * 8;
-}
-// B of two neighbouring n-tiles, stored [k][n] (ldsm4t)
-template <int PITCH>
-__device__ __forceinline__ const __nv_bfloat16* frag_b(const __nv_bfloat16* t, int k, int n, int lane) {
-  return t + (k + (lane & 15)) * PITCH + n + (lane >> 4) * 8;
-}
 // B of two neighbouring n-tiles, stored [n][k] (ldsm4)
 template <int PITCH>
 __device__ __forceinline__ const __nv_bfloat16* frag_bn(const __nv_bfloat16* t, int k, int n, int lane) {
   return t + (n + ((lane >> 4) & 1) * 8 + (lane & 7)) * PITCH + k + ((lane >> 3) & 1) * 8;
 }
 
-// One CTA of four warps per (chunk, NH heads that share their q and k): T = (I + A)^-1 diag(beta) and P of each.
+// One CTA of four warps per (chunk, NH heads that share their q and k): T = (I + A)^-1 diag(beta) and P T of each.
+template <int DP, int NH>
+struct ChunkPrepSmem {
+  static constexpr int PI = DP + 8, AP = DC + 4;
+  static constexpr int KQ = 2 * DC * PI * 2, STAGE = NH * 2 * DC_MAT * 2;
+  static constexpr int A_OFF = STAGE > KQ ? STAGE : KQ;              // k, q, later P; then A, later T
+  static constexpr int G_OFF = A_OFF + NH * DC * AP * 4;
+  static constexpr int BYTES = G_OFF + (2 * NH + 2) * DC * 4;
+};
 template <int DP, int NH>
 __global__ void __launch_bounds__(128) delta_chunk_prep_kernel(const DeltaParams p, uint8_t* __restrict__ scratch) {
-  constexpr int PI = DP + 8, AP = DC + 4;
-  extern __shared__ uint8_t smb[];
+  using L = ChunkPrepSmem<DP, NH>;
+  constexpr int PI = L::PI, AP = L::AP;
+  extern __shared__ __align__(16) uint8_t smb[];
   __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smb);
   __nv_bfloat16* q_s = k_s + DC * PI;
-  float* a_s = reinterpret_cast<float*>(q_s + DC * PI);  // [NH][64][AP]
-  float* G_s = a_s + NH * DC * AP;                       // [NH][64]
+  __nv_bfloat16* p_s = k_s;                                            // P, then P T: NH x (hi | lo)
+  float* a_s = reinterpret_cast<float*>(smb + L::A_OFF);               // [NH][64][AP]
+  __nv_bfloat16* t_s = reinterpret_cast<__nv_bfloat16*>(smb + L::A_OFF);  // T: NH x (hi | lo)
+  float* G_s = reinterpret_cast<float*>(smb + L::G_OFF);               // [NH][64]
   float *b_s = G_s + NH * DC, *nk_s = b_s + NH * DC, *nq_s = nk_s + DC;
+  // staged matrices: [64][64] bf16, 16-byte groups swizzled by row
+  auto at = [](int m, int t, int c) { return m * DC_MAT + t * DC + (((c >> 3) ^ (t & 7)) << 3) + (c & 7); };
   pdl_trigger();
   pdl_wait();
   const int idx = blockIdx.x, h = blockIdx.y * NH;
@@ -474,7 +476,7 @@ __global__ void __launch_bounds__(128) delta_chunk_prep_kernel(const DeltaParams
     vec[t] = eg * nk_s[t];
     vec[DC + t] = eg * nq_s[t];
     vec[2 * DC + t] = expf(gl - g) * nk_s[t];
-    if (t == 0) vec[3 * DC] = expf(gl);
+    vec[3 * DC + t] = expf(gl);
   }
   // Gram matrices of this warp's 16 rows, columns up to the diagonal block
   float kk[8][4] = {}, qk[8][4] = {};
@@ -496,36 +498,38 @@ __global__ void __launch_bounds__(128) delta_chunk_prep_kernel(const DeltaParams
       }
     }
   }
+  __syncthreads();  // every warp is done with k_s and q_s
 #pragma unroll
-  for (int x = 0; x < NH; ++x)
-#pragma unroll
-  for (int nt = 0; nt < 8; ++nt) {
-    uint32_t* P_hi = reinterpret_cast<uint32_t*>(dst + x * DC_BYTES) + DC_MAT;  // 32-bit words: T takes DC_MAT of them
-    uint32_t* P_lo = P_hi + DC_MAT / 2;
+  for (int x = 0; x < NH; ++x) {
     const float *G = G_s + x * DC, *beta = b_s + x * DC;
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int t = warp * 16 + (lane >> 2) + 8 * half, s = nt * 8 + (lane & 3) * 2;
-      float pv[2], av[2];
+    for (int nt = 0; nt < 8; ++nt) {
 #pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const float dec = s + e <= t ? expf(G[t] - G[s + e]) * nk_s[s + e] : 0.f;
-        pv[e] = dec * nq_s[t] * qk[nt][2 * half + e];
-        av[e] = s + e < t ? dec * nk_s[t] * beta[t] * kk[nt][2 * half + e] : 0.f;
+      for (int half = 0; half < 2; ++half) {
+        const int t = warp * 16 + (lane >> 2) + 8 * half, s = nt * 8 + (lane & 3) * 2;
+        float pv[2] = {0.f, 0.f}, av[2] = {0.f, 0.f};
+        if (nt < nt_end) {
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const float dec = s + e <= t ? __expf(G[t] - G[s + e]) * nk_s[s + e] : 0.f;
+            pv[e] = dec * nq_s[t] * qk[nt][2 * half + e];
+            av[e] = s + e < t ? dec * nk_s[t] * beta[t] * kk[nt][2 * half + e] : 0.f;
+          }
+        }
+        uint32_t ph, pl;
+        split2(pv[0], pv[1], ph, pl);
+        *reinterpret_cast<uint32_t*>(p_s + at(2 * x, t, s)) = ph;
+        *reinterpret_cast<uint32_t*>(p_s + at(2 * x + 1, t, s)) = pl;
+        *reinterpret_cast<float2*>(a_s + (x * DC + t) * AP + s) = make_float2(av[0], av[1]);
       }
-      uint32_t ph, pl;
-      split2(pv[0], pv[1], ph, pl);
-      P_hi[(t * DC + s) >> 1] = ph;
-      P_lo[(t * DC + s) >> 1] = pl;
-      *reinterpret_cast<float2*>(a_s + (x * DC + t) * AP + s) = make_float2(av[0], av[1]);
     }
   }
   __syncthreads();
   // forward substitution: a thread owns one column of (I + A)^-1
+  float x[DC];
   if (tid < NH * DC) {
     const int col = tid % DC;
     const float* A = a_s + tid / DC * DC * AP;
-    float x[DC];
 #pragma unroll
     for (int i = 0; i < DC; ++i) {
       float s0 = i == col ? 1.f : 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
@@ -539,243 +543,347 @@ __global__ void __launch_bounds__(128) delta_chunk_prep_kernel(const DeltaParams
       }
       x[i] = (s0 + s1) + (s2 + s3);
     }
+  }
+  __syncthreads();  // A is read: T takes its place
+  if (tid < NH * DC) {
+    const int col = tid % DC, m = tid / DC * 2;
     const float beta = b_s[tid];
-    __nv_bfloat16* t_hi = reinterpret_cast<__nv_bfloat16*>(dst + tid / DC * DC_BYTES) + col;
 #pragma unroll
-    for (int i = 0; i < DC; ++i) {  // a warp stores 32 neighbouring columns
+    for (int i = 0; i < DC; ++i) {
       const float v = x[i] * beta;
       const __nv_bfloat16 vh = __float2bfloat16(v);
-      t_hi[i * DC] = vh;
-      t_hi[DC_MAT + i * DC] = __float2bfloat16(v - __bfloat162float(vh));
+      t_s[at(m, i, col)] = vh;
+      t_s[at(m + 1, i, col)] = __float2bfloat16(v - __bfloat162float(vh));
     }
+  }
+  __syncthreads();
+  // P T of this warp's rows, written over its rows of P
+#pragma unroll 1
+  for (int xh = 0; xh < NH; ++xh) {
+    float acc[8][4] = {};
+    for (int kt = 0; kt <= warp; ++kt) {
+      const int r = warp * 16 + (lane & 15), g = kt * 2 + (lane >> 4), kr = kt * 16 + (lane & 15);
+      uint32_t ah[4], al[4];
+      ldsm4(ah, p_s + at(2 * xh, r, g * 8));
+      ldsm4(al, p_s + at(2 * xh + 1, r, g * 8));
+#pragma unroll
+      for (int nt = 0; nt < 8; nt += 2) {
+        if (nt <= 2 * kt) {  // T is lower triangular
+          uint32_t bh[4], bl[4];
+          ldsm4t(bh, t_s + at(2 * xh, kr, nt * 8 + (lane >> 4) * 8));
+          ldsm4t(bl, t_s + at(2 * xh + 1, kr, nt * 8 + (lane >> 4) * 8));
+          mma16(acc[nt], ah, bh[0], bh[1]);
+          mma16(acc[nt + 1], ah, bh[2], bh[3]);
+          mma16(acc[nt], al, bh[0], bh[1]);
+          mma16(acc[nt + 1], al, bh[2], bh[3]);
+          mma16(acc[nt], ah, bl[0], bl[1]);
+          mma16(acc[nt + 1], ah, bl[2], bl[3]);
+        }
+      }
+    }
+    __syncwarp();
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int t = warp * 16 + (lane >> 2) + 8 * half, s = nt * 8 + (lane & 3) * 2;
+        uint32_t ph, pl;
+        split2(acc[nt][2 * half], acc[nt][2 * half + 1], ph, pl);
+        *reinterpret_cast<uint32_t*>(p_s + at(2 * xh, t, s)) = ph;
+        *reinterpret_cast<uint32_t*>(p_s + at(2 * xh + 1, t, s)) = pl;
+      }
+  }
+  __syncthreads();
+  // scratch order: T hi, P T hi, T lo, P T lo
+  for (int i = tid; i < NH * 4 * DC * 8; i += 128) {
+    const int m = i / (DC * 8), t = i / 8 % DC, c = i % 8, head = m >> 2, term = (m >> 1) & 1;
+    const __nv_bfloat16* src = (m & 1 ? p_s : t_s) + at(2 * head + term, t, c * 8);
+    *reinterpret_cast<uint4*>(dst + head * DC_BYTES + ((m & 3) * DC_MAT + t * DC + c * 8) * 2) =
+        *reinterpret_cast<const uint4*>(src);
   }
 }
 
-// One CTA of eight warps per (sequence, head, 64 state columns): warp = (row slab wr of 16 tokens, column half wc of 32).
-// S [D, 64] stays in fp32 accumulators (warp (wr, wc) owns rows 32 wr .. of DP = 128, 16 wr .. of DP = 64) with a hi / lo
-// copy in shared memory for the next chunk's products.
-template <int DP>
-__global__ void __launch_bounds__(256, 1) delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch) {
-  constexpr int PI = DP + 8, XP = DC_VB + 8, MT = DP / 64;  // MT: 16-row tiles of S per warp
+// One CTA of eight warps per (sequence, head, 128 state columns); tcgen05 with accumulators in TMEM:
+//     RQ [128 = K rows | Q rows, v]  = [K; Q] . S          (S hi + lo from shared memory)
+//     rhs                            = v - e^G k S          (rows of K)
+//     UO [128, v]                    = [T; P T] . rhs       (rows 0..63 = U, rows 64..127 = P U)
+//     S^T [v, d]                    += U'^T . K             (U' = e^{G_last - G} U / |k|, fp32 state in TMEM)
+// The MMAs are issued by one thread; between them all warps read their TMEM lanes, scale, split into hi and lo and write
+// the next operand. Warp w owns TMEM lanes 32 (w % 4) .. and the column half w / 4. K and Q of the next chunk arrive
+// while a chunk is worked on, T and P T of the next chunk once UO is done.
+constexpr int DT_THREADS = 256;
+constexpr int DT_KQ = 32768;                     // [K; Q]: two 64-column blocks of 128 rows x 128 bytes
+constexpr int DT_TP_OFF = 2 * DT_KQ;             // hi | lo, 16 KB each
+constexpr int DT_X_OFF = DT_TP_OFF + 32768;      // rhs, then U': hi | lo, [64 tokens][128 columns] in two column blocks
+constexpr int DT_S_OFF = DT_X_OFF + 32768;       // S^T: hi | lo, [128 v][128 d] in two column blocks each
+constexpr int DT_BAR_OFF = DT_S_OFF + 65536;
+constexpr int DT_SMEM = DT_BAR_OFF + 64 + 1024;
+
+__global__ void __launch_bounds__(DT_THREADS, 1)
+delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch, int* status) {
   extern __shared__ uint8_t smb[];
-  __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smb);    // [2][64][PI]
-  __nv_bfloat16* q_s = k_s + 2 * DC * PI;                        // [2][64][PI]
-  __nv_bfloat16* v_s = q_s + 2 * DC * PI;                        // [2][64][XP]
-  __nv_bfloat16* T_s = v_s + 2 * DC * XP;                        // hi | lo [64][XP]
-  __nv_bfloat16* P_s = T_s + 2 * DC * XP;                        // hi | lo
-  __nv_bfloat16* x_s = P_s + 2 * DC * XP;                        // hi | lo: right-hand side, then U
-  __nv_bfloat16* w_s = x_s + 2 * DC * XP;                        // hi | lo: U scaled for the state
-  __nv_bfloat16* S_s = w_s + 2 * DC * XP;                        // hi | lo [DP][XP]
-  float* vec_s = reinterpret_cast<float*>(S_s + 2 * DP * XP);    // [2][4][64]
-  pdl_trigger();
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smb) + 1023) & ~uintptr_t(1023));
+  uint64_t* bar = reinterpret_cast<uint64_t*>(smem + DT_BAR_OFF);
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bar + 1);
   pdl_wait();
-  const int v0 = blockIdx.x * DC_VB, h = blockIdx.y, b = blockIdx.z;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, wr = warp & 3, wc = warp >> 2;
+  const int v0 = blockIdx.x * 128, h = blockIdx.y, b = blockIdx.z;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, quad = warp & 3, half = warp >> 2;
   const int first = p.cu_q[b], n = p.cu_q[b + 1] - first, slot = p.slots[b];
-  if (n <= 0 || slot < 0) return;
+  if (n <= 0 || slot < 0) return;  // uniform for the CTA, before any barrier or allocation
   const int start = p.seq_lens[b] - n, hk = h / (p.H / p.Hk), C = 2 * p.Hk * p.D + p.H * p.V;
   const __nv_bfloat16* y = static_cast<const __nv_bfloat16*>(p.qkv) + (long long)first * C;
   const uint8_t* scr = scratch + ((long long)((first >> 6) + b) * p.H + h) * DC_BYTES;
   const long long scr_step = (long long)p.H * DC_BYTES;
   const int chunks = (n + DC - 1) / DC;
+  const int VC = min(128, p.V - v0);             // columns of this CTA
 
-  auto load_kqv = [&](int c) {
+  if (tid == 0) {
+    mbar_init(bar, 1);
+    mbar_fence_init();
+  }
+  if (warp == 0) {
+    tmem_alloc(tmem_slot, 512);
+    tmem_relinquish();
+  }
+  auto load_kq = [&](int c) {
     if (c < chunks) {
-      const int buf = c & 1, t0 = c * DC;
-      for (int i = tid; i < DC * (DP / 8); i += 256) {
-        const int t = i / (DP / 8), d = i % (DP / 8) * 8;
+      uint8_t* dst = smem + (c & 1) * DT_KQ;
+      const int t0 = c * DC, groups = p.D > 64 ? 16 : 8;
+      for (int i = tid; i < DC * groups; i += DT_THREADS) {
+        const int t = i / groups, d = i % groups * 8;
         const bool on = t0 + t < n && d < p.D;
         const __nv_bfloat16* src = y + (on ? (long long)(t0 + t) * C + hk * p.D + d : 0);
-        cp_async16(q_s + (buf * DC + t) * PI + d, src, on);
-        cp_async16(k_s + (buf * DC + t) * PI + d, src + p.Hk * p.D, on);
+        uint8_t* to = dst + (d >> 6) * 16384 + t * 128 + ((((d & 63) >> 3) ^ (t & 7)) << 4);
+        cp_async16(to, src + p.Hk * p.D, on);
+        cp_async16(to + DC * 128, src, on);
       }
-      for (int i = tid; i < DC * (DC_VB / 8); i += 256) {
-        const int t = i / (DC_VB / 8), d = i % (DC_VB / 8) * 8;
-        const bool on = t0 + t < n && v0 + d < p.V;
-        cp_async16(v_s + (buf * DC + t) * XP + d,
-                   y + (on ? (long long)(t0 + t) * C + 2 * p.Hk * p.D + h * p.V + v0 + d : 0), on);
-      }
-      if (tid < DC) cp_async16(vec_s + buf * 4 * DC + tid * 4, scr + c * scr_step + DC_VEC_OFF + tid * 16, true);
     }
     cp_async_commit();
   };
-  auto load_mat = [&](int c, __nv_bfloat16* dst, int off) {
+  auto load_tp = [&](int c) {
     if (c < chunks)
-      for (int i = tid; i < 2 * DC * 8; i += 256) {
-        const int r = i >> 3, k = (i & 7) * 8;
-        cp_async16(dst + r * XP + k, scr + c * scr_step + off + (r * DC + k) * 2, true);
+      for (int i = tid; i < 256 * 8; i += DT_THREADS) {  // 128 rows of hi, 128 rows of lo
+        const int r = i >> 3, g = i & 7;
+        cp_async16(smem + DT_TP_OFF + r * 128 + ((g ^ (r & 7)) << 4), scr + c * scr_step + r * 128 + g * 16, true);
       }
     cp_async_commit();
   };
-  // accumulator element e of tile (mt, nt): row, column within the CTA's [DP, 64] block
-  auto s_row = [&](int mt, int e) { return wr * 16 * MT + mt * 16 + (lane >> 2) + 8 * (e >> 1); };
-  auto s_col = [&](int nt, int e) { return wc * 32 + nt * 8 + (lane & 3) * 2 + (e & 1); };
-  float S[MT][4][4];
-  float* st = p.state + ((long long)slot * p.H + h) * p.V * p.D;
-  load_kqv(0);
-  load_mat(0, T_s, 0);
-  load_mat(0, P_s, 2 * DC_MAT * 2);
+  // 32 fp32 values as two bf16 terms into four 16-byte groups of a 128-byte row, starting at group g0
+  auto put32 = [&](uint8_t* hi_row, uint8_t* lo_row, int row, int g0, const float (&f)[32]) {
 #pragma unroll
-  for (int mt = 0; mt < MT; ++mt)
+    for (int g = 0; g < 4; ++g) {
+      uint32_t hi[4], lo[4];
 #pragma unroll
-    for (int nt = 0; nt < 4; ++nt)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int d = s_row(mt, e), c = v0 + s_col(nt, e);
-        S[mt][nt][e] = start > 0 && d < p.D && c < p.V ? st[(long long)c * p.D + d] : 0.f;
-      }
-  auto publish_state = [&]() {
-#pragma unroll
-    for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-      for (int nt = 0; nt < 4; ++nt)
-#pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          uint32_t hi, lo;
-          split2(S[mt][nt][2 * half], S[mt][nt][2 * half + 1], hi, lo);
-          __nv_bfloat16* d = S_s + s_row(mt, 2 * half) * XP + s_col(nt, 0);
-          *reinterpret_cast<uint32_t*>(d) = hi;
-          *reinterpret_cast<uint32_t*>(d + DP * XP) = lo;
-        }
+      for (int k = 0; k < 4; ++k) split2(f[8 * g + 2 * k], f[8 * g + 2 * k + 1], hi[k], lo[k]);
+      const int off = ((g0 + g) ^ (row & 7)) << 4;
+      *reinterpret_cast<uint4*>(hi_row + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      *reinterpret_cast<uint4*>(lo_row + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    }
   };
-  publish_state();
-  cp_async_wait<2>();
+  load_kq(0);
+  load_tp(0);
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *tmem_slot, my = tmem + ((uint32_t)(quad * 32) << 16);
+  const uint32_t RQ = 0, UO = 128, ST = 256;
+  pdl_trigger();  // TMEM is held
+
+  // the state: this thread's row v and column half, in steps of 32
+  const int row_v = quad * 32 + lane;
+  float* st = p.state + (((long long)slot * p.H + h) * p.V + v0 + row_v) * p.D;
+  uint8_t* s_hi = smem + DT_S_OFF + half * 16384 + row_v * 128;
+  const bool half_on = half * 64 < p.D;
+  float egl = __ldg(reinterpret_cast<const float*>(scr + DC_VEC_OFF) + 3 * DC);
+  if (half_on) {
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      float f[32];
+      uint32_t w[32];
+#pragma unroll
+      for (int e = 0; e < 32; ++e) {
+        const int d = half * 64 + j * 32 + e;
+        f[e] = start > 0 && row_v < VC && d < p.D ? st[d] : 0.f;
+        w[e] = __float_as_uint(f[e] * egl);
+      }
+      put32(s_hi, s_hi + 32768, row_v, j * 4, f);
+      tmem_st_32x32(my + ST + half * 64 + j * 32, w);
+    }
+    tmem_st_wait();
+  }
+  cp_async_wait<0>();
+  fence_proxy_async_smem();
+  tc_fence_before();
   __syncthreads();
 
+  const uint32_t base = smem_u32(smem);
+  const int k_steps = (p.D + 15) / 16;
+  const uint32_t nv = (uint32_t)((VC + 15) / 16 * 16), nd = (uint32_t)((p.D + 15) / 16 * 16);
+  const uint32_t id_rq = umma_idesc(1, 1, 0, 0, 128, nv);  // A, B K-major
+  const uint32_t id_uo = umma_idesc(1, 1, 0, 1, 128, nv);  // B MN-major
+  const uint32_t id_s = umma_idesc(1, 1, 1, 1, 128, nd);   // both MN-major
+  uint32_t phase = 0;
+  bool ok = true;
+  // every thread waits for the MMAs issued last; one failed wait ends the loop for the whole CTA
+  auto mma_done = [&](int detail) {
+    const bool good = mbar_wait(bar, phase);
+    if (!good) report_error(status, ERR_WAIT_TMEM_FULL, detail);
+    phase ^= 1;
+    tc_fence_after();
+    return good;
+  };
+
   for (int c = 0; c < chunks; ++c) {
-    const int buf = c & 1, t0 = c * DC;
-    const __nv_bfloat16 *kb = k_s + buf * DC * PI, *qb = q_s + buf * DC * PI, *vb = v_s + buf * DC * XP;
-    const float* vec = vec_s + buf * 4 * DC;
-    load_kqv(c + 1);
-    // 1. K S and Q S
-    float R[4][4] = {}, O[4][4] = {};
-#pragma unroll
-    for (int k = 0; k < DP / 16; ++k) {
-      uint32_t ak[4], aq[4];
-      ldsm4(ak, frag_a<PI>(kb, wr * 16, k * 16, lane));
-      ldsm4(aq, frag_a<PI>(qb, wr * 16, k * 16, lane));
-#pragma unroll
-      for (int part = 0; part < 2; ++part)
-#pragma unroll
-        for (int np = 0; np < 2; ++np) {
-          uint32_t bb[4];
-          ldsm4t(bb, frag_b<XP>(S_s + part * DP * XP, k * 16, wc * 32 + np * 16, lane));
-          mma16(R[2 * np], ak, bb[0], bb[1]);
-          mma16(R[2 * np + 1], ak, bb[2], bb[3]);
-          mma16(O[2 * np], aq, bb[0], bb[1]);
-          mma16(O[2 * np + 1], aq, bb[2], bb[3]);
+    const int t0 = c * DC;
+    const uint32_t kq = base + (c & 1) * DT_KQ;
+    if (tid == 0) {
+      tc_fence_after();
+#pragma unroll 1
+      for (int term = 0; term < 2; ++term)
+        for (int k = 0; k < k_steps; ++k) {
+          const uint32_t off = (k >> 2) * 16384 + (k & 3) * 32;
+          tc_mma_f16(tmem + RQ, umma_smem_desc(kq + off, 16, 1024),
+                     umma_smem_desc(base + DT_S_OFF + term * 32768 + off, 16, 1024), id_rq, term != 0 || k != 0);
         }
+      tc_commit(bar);
     }
-    // right-hand side v - e^G k S
+    load_kq(c + 1);
+    const float* vec = reinterpret_cast<const float*>(scr + c * scr_step + DC_VEC_OFF);
+    const int t = (quad & 1) * 32 + lane;        // this thread's token (rows 0..63 K / U, 64..127 Q / O)
+    const bool tok = t0 + t < n;
+    uint4 v[8];
+    float scale_a, scale_b = 0.f;                // rows of K: e^G / |k| and e^{G_last - G} / |k|; rows of Q: e^G / |q|
+    if (quad < 2) {
+      const __nv_bfloat16* vr = y + (long long)(t0 + t) * C + 2 * p.Hk * p.D + h * p.V + v0 + half * 64;
 #pragma unroll
-    for (int nt = 0; nt < 4; ++nt)
+      for (int g = 0; g < 8; ++g)
+        v[g] = tok && half * 64 + g * 8 < VC ? *reinterpret_cast<const uint4*>(vr + g * 8) : make_uint4(0, 0, 0, 0);
+      scale_a = __ldg(vec + t);
+      scale_b = __ldg(vec + 2 * DC + t);
+    } else {
+      scale_a = __ldg(vec + DC + t);
+    }
+    const float egl_next = c + 1 < chunks ? __ldg(reinterpret_cast<const float*>(scr + (c + 1) * scr_step + DC_VEC_OFF) + 3 * DC)
+                                          : 1.f;
+    ok = mma_done(4 * c) && ok;
+    // right-hand side
+    uint8_t* x_hi = smem + DT_X_OFF + half * 8192 + t * 128;
+    if (quad < 2) {
 #pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int t = wr * 16 + (lane >> 2) + 8 * half, col = s_col(nt, 0);
-        const uint32_t vv = *reinterpret_cast<const uint32_t*>(vb + t * XP + col);
-        const float ek = vec[t], eq = vec[DC + t];
-        uint32_t hi, lo;
-        split2(__uint_as_float(vv << 16) - ek * R[nt][2 * half], __uint_as_float(vv & 0xffff0000u) - ek * R[nt][2 * half + 1], hi,
-               lo);
-        *reinterpret_cast<uint32_t*>(x_s + t * XP + col) = hi;
-        *reinterpret_cast<uint32_t*>(x_s + (DC + t) * XP + col) = lo;
-        O[nt][2 * half] *= eq;
-        O[nt][2 * half + 1] *= eq;
-      }
-    cp_async_wait<2>();  // T of this chunk
-    __syncthreads();
-    // 2. U = T . rhs (lower triangular: this slab needs the token blocks 0 .. wr)
-    float U[4][4] = {};
-    auto tri = [&](float (&acc)[4][4], const __nv_bfloat16* m) {
-      for (int k = 0; k <= wr; ++k) {
-        uint32_t ah[4], al[4];
-        ldsm4(ah, frag_a<XP>(m, wr * 16, k * 16, lane));
-        ldsm4(al, frag_a<XP>(m + DC * XP, wr * 16, k * 16, lane));
+      for (int j = 0; j < 2; ++j) {
+        uint32_t r[32];
+        tmem_ld_32x32(my + RQ + half * 64 + j * 32, r);
+        tmem_ld_wait();
+        float f[32];
 #pragma unroll
-        for (int np = 0; np < 2; ++np) {
-          uint32_t bh[4], bl[4];
-          ldsm4t(bh, frag_b<XP>(x_s, k * 16, wc * 32 + np * 16, lane));
-          ldsm4t(bl, frag_b<XP>(x_s + DC * XP, k * 16, wc * 32 + np * 16, lane));
-          mma16(acc[2 * np], ah, bh[0], bh[1]);
-          mma16(acc[2 * np + 1], ah, bh[2], bh[3]);
-          mma16(acc[2 * np], al, bh[0], bh[1]);
-          mma16(acc[2 * np + 1], al, bh[2], bh[3]);
-          mma16(acc[2 * np], ah, bl[0], bl[1]);
-          mma16(acc[2 * np + 1], ah, bl[2], bl[3]);
-        }
-      }
-    };
-    tri(U, T_s);
-    __syncthreads();  // every warp is done with the right-hand side and with T
-    load_mat(c + 1, T_s, 0);
+        for (int g = 0; g < 4; ++g) {
+          const uint32_t* vw = reinterpret_cast<const uint32_t*>(&v[j * 4 + g]);
 #pragma unroll
-    for (int nt = 0; nt < 4; ++nt)
-#pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int t = wr * 16 + (lane >> 2) + 8 * half, col = s_col(nt, 0);
-        const float ce = vec[2 * DC + t];
-        uint32_t hi, lo;
-        split2(U[nt][2 * half], U[nt][2 * half + 1], hi, lo);
-        *reinterpret_cast<uint32_t*>(x_s + t * XP + col) = hi;
-        *reinterpret_cast<uint32_t*>(x_s + (DC + t) * XP + col) = lo;
-        split2(ce * U[nt][2 * half], ce * U[nt][2 * half + 1], hi, lo);
-        *reinterpret_cast<uint32_t*>(w_s + t * XP + col) = hi;
-        *reinterpret_cast<uint32_t*>(w_s + (DC + t) * XP + col) = lo;
-      }
-    cp_async_wait<2>();  // P of this chunk
-    __syncthreads();
-    // 3. output
-    tri(O, P_s);
-    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (long long)(first + t0) * p.out_stride + (long long)h * p.V + v0;
-#pragma unroll
-    for (int nt = 0; nt < 4; ++nt)
-#pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int t = wr * 16 + (lane >> 2) + 8 * half, col = s_col(nt, 0);
-        if (t0 + t < n && v0 + col < p.V)
-          *reinterpret_cast<uint32_t*>(out + (long long)t * p.out_stride + col) = pack_bf16x2(O[nt][2 * half], O[nt][2 * half + 1]);
-      }
-    // 4. state
-    const float egl = vec[3 * DC];
-#pragma unroll
-    for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-      for (int nt = 0; nt < 4; ++nt)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) S[mt][nt][e] *= egl;
-#pragma unroll
-    for (int k = 0; k < DC / 16; ++k) {
-      uint32_t a[MT][4];
-#pragma unroll
-      for (int mt = 0; mt < MT; ++mt) ldsm4t(a[mt], frag_at<PI>(kb, wr * 16 * MT + mt * 16, k * 16, lane));
-#pragma unroll
-      for (int part = 0; part < 2; ++part)
-#pragma unroll
-        for (int np = 0; np < 2; ++np) {
-          uint32_t bb[4];
-          ldsm4t(bb, frag_b<XP>(w_s + part * DC * XP, k * 16, wc * 32 + np * 16, lane));
-#pragma unroll
-          for (int mt = 0; mt < MT; ++mt) {
-            mma16(S[mt][2 * np], a[mt], bb[0], bb[1]);
-            mma16(S[mt][2 * np + 1], a[mt], bb[2], bb[3]);
+          for (int k = 0; k < 4; ++k) {
+            const int e = 8 * g + 2 * k;
+            const bool on = half * 64 + j * 32 + e < VC;  // columns past N of the MMA are not defined
+            f[e] = on ? __uint_as_float(vw[k] << 16) - scale_a * __uint_as_float(r[e]) : 0.f;
+            f[e + 1] = on ? __uint_as_float(vw[k] & 0xffff0000u) - scale_a * __uint_as_float(r[e + 1]) : 0.f;
           }
         }
-    }
-    publish_state();
-    cp_async_wait<1>();  // q, k, v of the next chunk
-    __syncthreads();
-    load_mat(c + 1, P_s, 2 * DC_MAT * 2);
-  }
-#pragma unroll
-  for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-    for (int nt = 0; nt < 4; ++nt)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int d = s_row(mt, e), c = v0 + s_col(nt, e);
-        if (d < p.D && c < p.V) st[(long long)c * p.D + d] = S[mt][nt][e];
+        put32(x_hi, x_hi + 16384, t, j * 4, f);
       }
-  store_ring<__nv_bfloat16>(p, first, n, start, slot, blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y);
+    }
+    cp_async_wait<1>();  // T and P T of this chunk (the newest group is K and Q of the next one)
+    fence_proxy_async_smem();
+    tc_fence_before();
+    if (!__syncthreads_and(ok)) break;
+    if (tid == 0) {
+      tc_fence_after();
+#pragma unroll 1
+      for (int term = 0; term < 3; ++term) {  // hi hi, lo hi, hi lo
+        const uint32_t a0 = base + DT_TP_OFF + (term == 1 ? 16384 : 0), b0 = base + DT_X_OFF + (term == 2 ? 16384 : 0);
+        for (int k = 0; k < DC / 16; ++k)
+          tc_mma_f16(tmem + UO, umma_smem_desc(a0 + k * 32, 16, 1024), umma_smem_desc(b0 + k * 2048, 8192, 1024), id_uo,
+                     term != 0 || k != 0);
+      }
+      tc_commit(bar);
+    }
+    ok = mma_done(4 * c + 1) && ok;
+    load_tp(c + 1);
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      uint32_t r[32];
+      tmem_ld_32x32(my + UO + half * 64 + j * 32, r);
+      tmem_ld_wait();
+      float f[32];
+      if (quad < 2) {
+#pragma unroll
+        for (int e = 0; e < 32; ++e) f[e] = half * 64 + j * 32 + e < VC ? scale_b * __uint_as_float(r[e]) : 0.f;
+        put32(x_hi, x_hi + 16384, t, j * 4, f);
+      } else {
+        uint32_t q[32];
+        tmem_ld_32x32(my + RQ + half * 64 + j * 32, q);
+        tmem_ld_wait();
+#pragma unroll
+        for (int e = 0; e < 32; ++e) f[e] = fmaf(scale_a, __uint_as_float(q[e]), __uint_as_float(r[e]));
+        __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (long long)(first + t0 + t) * p.out_stride +
+                             (long long)h * p.V + v0 + half * 64 + j * 32;
+        if (tok)
+#pragma unroll
+          for (int g = 0; g < 4; ++g)
+            if (half * 64 + j * 32 + g * 8 < VC)
+              *reinterpret_cast<uint4*>(out + g * 8) =
+                  make_uint4(pack_bf16x2(f[8 * g], f[8 * g + 1]), pack_bf16x2(f[8 * g + 2], f[8 * g + 3]),
+                             pack_bf16x2(f[8 * g + 4], f[8 * g + 5]), pack_bf16x2(f[8 * g + 6], f[8 * g + 7]));
+      }
+    }
+    fence_proxy_async_smem();
+    tc_fence_before();
+    if (!__syncthreads_and(ok)) break;
+    if (tid == 0) {
+      tc_fence_after();
+#pragma unroll 1
+      for (int term = 0; term < 2; ++term)
+        for (int k = 0; k < DC / 16; ++k)
+          tc_mma_f16(tmem + ST, umma_smem_desc(base + DT_X_OFF + term * 16384 + k * 2048, 8192, 1024),
+                     umma_smem_desc(kq + k * 2048, 16384, 1024), id_s, 1);
+      tc_commit(bar);
+    }
+    ok = mma_done(4 * c + 2) && ok;
+    const bool last = c + 1 == chunks;
+    if (half_on && ok) {
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        uint32_t r[32];
+        tmem_ld_32x32(my + ST + half * 64 + j * 32, r);
+        tmem_ld_wait();
+        float f[32];
+#pragma unroll
+        for (int e = 0; e < 32; ++e) f[e] = half * 64 + j * 32 + e < (int)nd ? __uint_as_float(r[e]) : 0.f;
+        if (last) {
+#pragma unroll
+          for (int e = 0; e < 32; ++e) {
+            const int d = half * 64 + j * 32 + e;
+            if (row_v < VC && d < p.D) st[d] = f[e];
+          }
+        } else {
+          put32(s_hi, s_hi + 32768, row_v, j * 4, f);
+#pragma unroll
+          for (int e = 0; e < 32; ++e) r[e] = __float_as_uint(f[e] * egl_next);
+          tmem_st_32x32(my + ST + half * 64 + j * 32, r);
+        }
+      }
+      tmem_st_wait();
+    }
+    cp_async_wait<1>();  // K and Q of the next chunk (the newest group is its T and P T)
+    fence_proxy_async_smem();
+    tc_fence_before();
+    if (!__syncthreads_and(ok)) break;
+  }
+  cp_async_wait<0>();
+  if (ok) store_ring<__nv_bfloat16>(p, first, n, start, slot, blockIdx.y * gridDim.x + blockIdx.x, gridDim.x * gridDim.y);
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 0) {
+    tc_fence_after();
+    tmem_dealloc(tmem, 512);
+  }
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -1004,32 +1112,40 @@ static int run_step(const DeltaParams& p, cudaStream_t stream) {
   return (int)e;
 }
 
-template <int DP>
-static int run_chunks(const DeltaParams& p, int tokens, uint8_t* scratch, cudaStream_t stream) {
-  constexpr int PI = DP + 8, XP = DC_VB + 8;
-  const int nh = (p.H / p.Hk) % 2 == 0 ? 2 : 1;
-  const int smem1 = 2 * DC * PI * 2 + (nh * DC * (DC + 4) + (2 * nh + 2) * DC) * 4;
-  const int smem2 = (4 * DC * PI + 2 * DC * XP + 8 * DC * XP + 2 * DP * XP) * 2 + 8 * DC * 4;
+template <int DP, int NH>
+static cudaError_t launch_chunk_prep(const DeltaParams& p, int tokens, uint8_t* scratch, cudaStream_t stream) {
+  constexpr int bytes = ChunkPrepSmem<DP, NH>::BYTES;
   static bool attr = false;
   if (!attr) {
-    const int most = 2 * DC * PI * 2 + (2 * DC * (DC + 4) + 6 * DC) * 4;
-    VB_CUDA_CHECK(cudaFuncSetAttribute(delta_chunk_prep_kernel<DP, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, most));
-    VB_CUDA_CHECK(cudaFuncSetAttribute(delta_chunk_prep_kernel<DP, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, most));
-    VB_CUDA_CHECK(cudaFuncSetAttribute(delta_chunk_scan_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem2));
+    cudaError_t e = cudaFuncSetAttribute(delta_chunk_prep_kernel<DP, NH>, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+    if (e != cudaSuccess) return e;
     attr = true;
   }
-  const dim3 g1(tokens / DC + p.B, p.H / nh);
-  cudaError_t e = nh == 2 ? vb_launch_pdl(delta_chunk_prep_kernel<DP, 2>, g1, dim3(128), smem1, stream, 1, p, scratch)
-                          : vb_launch_pdl(delta_chunk_prep_kernel<DP, 1>, g1, dim3(128), smem1, stream, 1, p, scratch);
+  return vb_launch_pdl(delta_chunk_prep_kernel<DP, NH>, dim3(tokens / DC + p.B, p.H / NH), dim3(128), bytes, stream, 1, p,
+                       scratch);
+}
+
+static int run_chunks(const DeltaParams& p, int tokens, uint8_t* scratch, int* status, cudaStream_t stream) {
+  static bool attr = false;
+  if (!attr) {
+    VB_CUDA_CHECK(cudaFuncSetAttribute(delta_chunk_scan_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, DT_SMEM));
+    attr = true;
+  }
+  const bool pairs = (p.H / p.Hk) % 2 == 0;
+  cudaError_t e = p.D <= 64 ? (pairs ? launch_chunk_prep<64, 2>(p, tokens, scratch, stream)
+                                     : launch_chunk_prep<64, 1>(p, tokens, scratch, stream))
+                            : (pairs ? launch_chunk_prep<128, 2>(p, tokens, scratch, stream)
+                                     : launch_chunk_prep<128, 1>(p, tokens, scratch, stream));
   if (e != cudaSuccess) return (int)e;
-  e = vb_launch_pdl(delta_chunk_scan_kernel<DP>, dim3((p.V + DC_VB - 1) / DC_VB, p.H, p.B), dim3(256), smem2, stream, 1, p,
-                    (const uint8_t*)scratch);
+  e = vb_launch_pdl(delta_chunk_scan_kernel, dim3((p.V + 127) / 128, p.H, p.B), dim3(DT_THREADS), DT_SMEM, stream, 1, p,
+                    (const uint8_t*)scratch, status);
   vb_count_launch(2);
   return (int)e;
 }
 
 template <typename T>
-static int run_delta(const DeltaParams& p, int tokens, int max_q, uint8_t* chunk_scratch, cudaStream_t stream) {
+static int run_delta(const DeltaParams& p, int tokens, int max_q, uint8_t* chunk_scratch, int* status,
+                     cudaStream_t stream) {
   const int nr = p.D <= 32 ? 4 : p.D <= 64 ? 8 : p.D <= 128 ? 16 : 32;
   if (max_q == 1) {
     if (nr == 4) return run_step<T, 4>(p, stream);
@@ -1040,7 +1156,7 @@ static int run_delta(const DeltaParams& p, int tokens, int max_q, uint8_t* chunk
   int rc = chunk_scratch ? run_prep<T, true>(p, max_q, stream) : run_prep<T, false>(p, max_q, stream);
   if (rc) return rc;
   if (chunk_scratch)
-    rc = p.D <= 64 ? run_chunks<64>(p, tokens, chunk_scratch, stream) : run_chunks<128>(p, tokens, chunk_scratch, stream);
+    rc = run_chunks(p, tokens, chunk_scratch, status, stream);
   else
     rc = nr == 4    ? run_scan<T, 4>(p, stream)
          : nr == 8  ? run_scan<T, 8>(p, stream)
@@ -1071,16 +1187,16 @@ extern "C" int vb_delta_rule(const void* proj, long long stride, const void* con
                              const float* dt_bias, const void* norm_w, void* ring, float* state, const int* cu_q,
                              const int* seq_lens, const int* slots, void* qkv, float* unit, float* gates, void* chunk_scratch,
                              void* out, long long out_stride, int T, int B, int max_q, int H, int Hk, int D, int V, int taps,
-                             float eps, int f32, cudaStream_t stream) {
+                             float eps, int f32, int* status, cudaStream_t stream) {
   if (T <= 0 || B <= 0 || max_q <= 0) return 0;
   if (Hk <= 0 || H % Hk != 0 || D <= 0 || D > 256 || V <= 0 || V > 256 || taps < 1 || taps > 8 || B > 65535) return -3;
   if (max_q > 1 && (qkv == nullptr || gates == nullptr)) return -3;
   if (max_q > 1 && chunk_scratch != nullptr &&
-      (f32 || unit == nullptr || !vb_delta_chunk_supported(D, V) || (out_stride & 1) || (reinterpret_cast<uintptr_t>(qkv) & 15)))
+      (f32 || unit == nullptr || !vb_delta_chunk_supported(D, V) || (out_stride & 7) || (reinterpret_cast<uintptr_t>(qkv) & 15)))
     return -3;
   DeltaParams p{proj, stride, conv_w, a_log, dt_bias, norm_w, ring, state, cu_q, seq_lens, slots, qkv, unit, gates, out,
                 out_stride, B, H, Hk, D, V, taps, eps};
   uint8_t* scr = reinterpret_cast<uint8_t*>(chunk_scratch);
-  const int rc = f32 ? run_delta<float>(p, T, max_q, nullptr, stream) : run_delta<__nv_bfloat16>(p, T, max_q, scr, stream);
+  const int rc = f32 ? run_delta<float>(p, T, max_q, nullptr, status, stream) : run_delta<__nv_bfloat16>(p, T, max_q, scr, status, stream);
   return rc ? rc : (int)cudaGetLastError();
 }

@@ -58,7 +58,7 @@ _SIGS = {
     "vb_paged_decode_window": ([P, L, P, P, I, P, I, P, I, I, I, I, I, I, F, I, I, P, I, I, P, L, P, P, P], I),
     "vb_delta_chunk_supported": ([I, I], I),
     "vb_delta_chunk_bytes": ([I, I, I], L),
-    "vb_delta_rule": ([P, L, P, P, P, P, P, P, P, P, P, P, P, P, P, P, L, I, I, I, I, I, I, I, I, F, I, P], I),
+    "vb_delta_rule": ([P, L, P, P, P, P, P, P, P, P, P, P, P, P, P, P, L, I, I, I, I, I, I, I, I, F, I, P, P], I),
     # rl ops
     "vb_ppo_loss": ([P, P, P, P, P, P, P, P, P, P, L, F, F, F, F, I, F, F, P], I),
     "vb_gae": ([P, P, P, P, P, I, I, F, F, P], I),

@@ -44,7 +44,7 @@ def delta_rule(proj: torch.Tensor, conv_w: torch.Tensor, a_log: torch.Tensor, dt
                                       seq_lens.data_ptr(), slots.data_ptr(), _lib.ptr(qkv), _lib.ptr(unit), _lib.ptr(gates),
                                       _lib.ptr(scratch), out.data_ptr(),
                                       out.stride(0), T, B, int(max_q), heads, kv_heads, dim, vdim, taps, float(eps),
-                                      int(proj.dtype == torch.float32), _lib.stream())
+                                      int(proj.dtype == torch.float32), _lib.status_word(proj.device).data_ptr(), _lib.stream())
         _lib.check(rc, "vb_delta_rule")
         return out
     cu, lens, sl = cu_q.tolist(), seq_lens.tolist(), slots.tolist()
