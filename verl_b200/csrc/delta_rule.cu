@@ -603,19 +603,19 @@ __global__ void __launch_bounds__(128) delta_chunk_prep_kernel(const DeltaParams
   }
 }
 
-// One CTA of eight warps per (sequence, head, 128 state columns); tcgen05 with accumulators in TMEM:
-//     RQ [128 = K rows | Q rows, v]  = [K; Q] . S          (S hi + lo from shared memory)
+// One CTA of sixteen warps per (sequence, head, 128 state columns); tcgen05 with accumulators in TMEM:
+//     RQ [128 = K rows | Q rows, 2 v] = [K; Q] . [S hi | S lo]   (from shared memory; the halves are added when read)
 //     rhs                            = v - e^G k S          (rows of K)
 //     UO [128, v]                    = [T; P T] . rhs       (rows 0..63 = U, rows 64..127 = P U)
 //     S^T [v, d]                    += U'^T . K             (U' = e^{G_last - G} U / |k|, fp32 state in TMEM)
 // The MMAs are issued by one thread; between them all warps read their TMEM lanes, scale, split into hi and lo and write
-// the next operand. Warp w owns TMEM lanes 32 (w % 4) .. and the column half w / 4. K and Q of the next chunk arrive
+// the next operand. Warp w owns TMEM lanes 32 (w % 4) .. and the 32 columns 32 (w / 4) .. of each accumulator. K and Q of the next chunk arrive
 // while a chunk is worked on, T and P T of the next chunk once UO is done.
-constexpr int DT_THREADS = 256;
+constexpr int DT_THREADS = 512;
 constexpr int DT_KQ = 32768;                     // [K; Q]: two 64-column blocks of 128 rows x 128 bytes
 constexpr int DT_TP_OFF = 2 * DT_KQ;             // hi | lo, 16 KB each
 constexpr int DT_X_OFF = DT_TP_OFF + 32768;      // rhs, then U': hi | lo, [64 tokens][128 columns] in two column blocks
-constexpr int DT_S_OFF = DT_X_OFF + 32768;       // S^T: hi | lo, [128 v][128 d] in two column blocks each
+constexpr int DT_S_OFF = DT_X_OFF + 32768;       // S^T [128 v][128 d]: per column block hi | lo
 constexpr int DT_BAR_OFF = DT_S_OFF + 65536;
 constexpr int DT_SMEM = DT_BAR_OFF + 64 + 1024;
 
@@ -627,7 +627,7 @@ delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bar + 1);
   pdl_wait();
   const int v0 = blockIdx.x * 128, h = blockIdx.y, b = blockIdx.z;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, quad = warp & 3, half = warp >> 2;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, quad = warp & 3, col0 = (warp >> 2) * 32;
   const int first = p.cu_q[b], n = p.cu_q[b + 1] - first, slot = p.slots[b];
   if (n <= 0 || slot < 0) return;  // uniform for the CTA, before any barrier or allocation
   const int start = p.seq_lens[b] - n, hk = h / (p.H / p.Hk), C = 2 * p.Hk * p.D + p.H * p.V;
@@ -686,28 +686,29 @@ delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = *tmem_slot, my = tmem + ((uint32_t)(quad * 32) << 16);
-  const uint32_t RQ = 0, UO = 128, ST = 256;
+  const uint32_t RQ = 0, UO = 256, ST = 384;
   pdl_trigger();  // TMEM is held
 
   // the state: this thread's row v and column half, in steps of 32
   const int row_v = quad * 32 + lane;
   float* st = p.state + (((long long)slot * p.H + h) * p.V + v0 + row_v) * p.D;
-  uint8_t* s_hi = smem + DT_S_OFF + half * 16384 + row_v * 128;
-  const bool half_on = half * 64 < p.D;
+  uint8_t* s_hi = smem + DT_S_OFF + (col0 >> 6) * 32768 + row_v * 128;
+  const int nd = p.D > 64 ? 128 : 64;            // columns past D are zero
+  const bool d_on = col0 < nd;
+  const int g0 = (col0 & 32) >> 3;  // first 16-byte group within a 128-byte row
   float egl = __ldg(reinterpret_cast<const float*>(scr + DC_VEC_OFF) + 3 * DC);
-  if (half_on) {
-#pragma unroll
-    for (int j = 0; j < 2; ++j) {
+  if (d_on) {
+    {
       float f[32];
       uint32_t w[32];
 #pragma unroll
       for (int e = 0; e < 32; ++e) {
-        const int d = half * 64 + j * 32 + e;
+        const int d = col0 + e;
         f[e] = start > 0 && row_v < VC && d < p.D ? st[d] : 0.f;
         w[e] = __float_as_uint(f[e] * egl);
       }
-      put32(s_hi, s_hi + 32768, row_v, j * 4, f);
-      tmem_st_32x32(my + ST + half * 64 + j * 32, w);
+      put32(s_hi, s_hi + 16384, row_v, g0, f);
+      tmem_st_32x32(my + ST + col0, w);
     }
     tmem_st_wait();
   }
@@ -718,19 +719,31 @@ delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch
 
   const uint32_t base = smem_u32(smem);
   const int k_steps = (p.D + 15) / 16;
-  const uint32_t nv = (uint32_t)((VC + 15) / 16 * 16), nd = (uint32_t)((p.D + 15) / 16 * 16);
-  const uint32_t id_rq = umma_idesc(1, 1, 0, 0, 128, nv);  // A, B K-major
-  const uint32_t id_uo = umma_idesc(1, 1, 0, 1, 128, nv);  // B MN-major
-  const uint32_t id_s = umma_idesc(1, 1, 1, 1, 128, nd);   // both MN-major
+  const uint32_t id_rq = umma_idesc(1, 1, 0, 0, 128, 256);           // A, B K-major
+  const uint32_t id_uo = umma_idesc(1, 1, 0, 1, 128, 128);           // B MN-major
+  const uint32_t id_s = umma_idesc(1, 1, 1, 1, 128, (uint32_t)nd);   // both MN-major
   uint32_t phase = 0;
   bool ok = true;
   // every thread waits for the MMAs issued last; one failed wait ends the loop for the whole CTA
   auto mma_done = [&](int detail) {
-    const bool good = mbar_wait(bar, phase);
+    bool good = false;  // a few products take microseconds: bounded by attempts, without reading the clock
+    for (int i = 0; i < (1 << 22) && !good; ++i) good = mbar_try_wait(bar, phase);
     if (!good) report_error(status, ERR_WAIT_TMEM_FULL, detail);
     phase ^= 1;
     tc_fence_after();
     return good;
+  };
+
+  auto read_rq = [&](float (&f)[32]) {
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      uint32_t a[16], l[16];
+      tmem_ld_32x16(my + RQ + col0 + 16 * j, a);
+      tmem_ld_32x16(my + RQ + 128 + col0 + 16 * j, l);
+      tmem_ld_wait();
+#pragma unroll
+      for (int e = 0; e < 16; ++e) f[16 * j + e] = __uint_as_float(a[e]) + __uint_as_float(l[e]);
+    }
   };
 
   for (int c = 0; c < chunks; ++c) {
@@ -738,26 +751,22 @@ delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch
     const uint32_t kq = base + (c & 1) * DT_KQ;
     if (tid == 0) {
       tc_fence_after();
-#pragma unroll 1
-      for (int term = 0; term < 2; ++term)
-        for (int k = 0; k < k_steps; ++k) {
-          const uint32_t off = (k >> 2) * 16384 + (k & 3) * 32;
-          tc_mma_f16(tmem + RQ, umma_smem_desc(kq + off, 16, 1024),
-                     umma_smem_desc(base + DT_S_OFF + term * 32768 + off, 16, 1024), id_rq, term != 0 || k != 0);
-        }
+      for (int k = 0; k < k_steps; ++k)
+        tc_mma_f16(tmem + RQ, umma_smem_desc(kq + (k >> 2) * 16384 + (k & 3) * 32, 16, 1024),
+                   umma_smem_desc(base + DT_S_OFF + (k >> 2) * 32768 + (k & 3) * 32, 16, 1024), id_rq, k != 0);
       tc_commit(bar);
     }
     load_kq(c + 1);
     const float* vec = reinterpret_cast<const float*>(scr + c * scr_step + DC_VEC_OFF);
     const int t = (quad & 1) * 32 + lane;        // this thread's token (rows 0..63 K / U, 64..127 Q / O)
     const bool tok = t0 + t < n;
-    uint4 v[8];
+    uint4 v[4];
     float scale_a, scale_b = 0.f;                // rows of K: e^G / |k| and e^{G_last - G} / |k|; rows of Q: e^G / |q|
     if (quad < 2) {
-      const __nv_bfloat16* vr = y + (long long)(t0 + t) * C + 2 * p.Hk * p.D + h * p.V + v0 + half * 64;
+      const __nv_bfloat16* vr = y + (long long)(t0 + t) * C + 2 * p.Hk * p.D + h * p.V + v0 + col0;
 #pragma unroll
-      for (int g = 0; g < 8; ++g)
-        v[g] = tok && half * 64 + g * 8 < VC ? *reinterpret_cast<const uint4*>(vr + g * 8) : make_uint4(0, 0, 0, 0);
+      for (int g = 0; g < 4; ++g)
+        v[g] = tok && col0 + g * 8 < VC ? *reinterpret_cast<const uint4*>(vr + g * 8) : make_uint4(0, 0, 0, 0);
       scale_a = __ldg(vec + t);
       scale_b = __ldg(vec + 2 * DC + t);
     } else {
@@ -767,26 +776,22 @@ delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch
                                           : 1.f;
     ok = mma_done(4 * c) && ok;
     // right-hand side
-    uint8_t* x_hi = smem + DT_X_OFF + half * 8192 + t * 128;
+    uint8_t* x_hi = smem + DT_X_OFF + (col0 >> 6) * 8192 + t * 128;
     if (quad < 2) {
-#pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        uint32_t r[32];
-        tmem_ld_32x32(my + RQ + half * 64 + j * 32, r);
-        tmem_ld_wait();
+      {
         float f[32];
+        read_rq(f);
 #pragma unroll
         for (int g = 0; g < 4; ++g) {
-          const uint32_t* vw = reinterpret_cast<const uint32_t*>(&v[j * 4 + g]);
+          const uint32_t* vw = reinterpret_cast<const uint32_t*>(&v[g]);
 #pragma unroll
           for (int k = 0; k < 4; ++k) {
             const int e = 8 * g + 2 * k;
-            const bool on = half * 64 + j * 32 + e < VC;  // columns past N of the MMA are not defined
-            f[e] = on ? __uint_as_float(vw[k] << 16) - scale_a * __uint_as_float(r[e]) : 0.f;
-            f[e + 1] = on ? __uint_as_float(vw[k] & 0xffff0000u) - scale_a * __uint_as_float(r[e + 1]) : 0.f;
+            f[e] = fmaf(-scale_a, f[e], __uint_as_float(vw[k] << 16));
+            f[e + 1] = fmaf(-scale_a, f[e + 1], __uint_as_float(vw[k] & 0xffff0000u));
           }
         }
-        put32(x_hi, x_hi + 16384, t, j * 4, f);
+        put32(x_hi, x_hi + 16384, t, g0, f);
       }
     }
     cp_async_wait<1>();  // T and P T of this chunk (the newest group is K and Q of the next one)
@@ -806,28 +811,25 @@ delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch
     }
     ok = mma_done(4 * c + 1) && ok;
     load_tp(c + 1);
-#pragma unroll
-    for (int j = 0; j < 2; ++j) {
+    {
       uint32_t r[32];
-      tmem_ld_32x32(my + UO + half * 64 + j * 32, r);
+      tmem_ld_32x32(my + UO + col0, r);
       tmem_ld_wait();
       float f[32];
       if (quad < 2) {
 #pragma unroll
-        for (int e = 0; e < 32; ++e) f[e] = half * 64 + j * 32 + e < VC ? scale_b * __uint_as_float(r[e]) : 0.f;
-        put32(x_hi, x_hi + 16384, t, j * 4, f);
+        for (int e = 0; e < 32; ++e) f[e] = scale_b * __uint_as_float(r[e]);
+        put32(x_hi, x_hi + 16384, t, g0, f);
       } else {
-        uint32_t q[32];
-        tmem_ld_32x32(my + RQ + half * 64 + j * 32, q);
-        tmem_ld_wait();
+        read_rq(f);
 #pragma unroll
-        for (int e = 0; e < 32; ++e) f[e] = fmaf(scale_a, __uint_as_float(q[e]), __uint_as_float(r[e]));
+        for (int e = 0; e < 32; ++e) f[e] = fmaf(scale_a, f[e], __uint_as_float(r[e]));
         __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (long long)(first + t0 + t) * p.out_stride +
-                             (long long)h * p.V + v0 + half * 64 + j * 32;
+                             (long long)h * p.V + v0 + col0;
         if (tok)
 #pragma unroll
           for (int g = 0; g < 4; ++g)
-            if (half * 64 + j * 32 + g * 8 < VC)
+            if (col0 + g * 8 < VC)
               *reinterpret_cast<uint4*>(out + g * 8) =
                   make_uint4(pack_bf16x2(f[8 * g], f[8 * g + 1]), pack_bf16x2(f[8 * g + 2], f[8 * g + 3]),
                              pack_bf16x2(f[8 * g + 4], f[8 * g + 5]), pack_bf16x2(f[8 * g + 6], f[8 * g + 7]));
@@ -847,26 +849,25 @@ delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch
     }
     ok = mma_done(4 * c + 2) && ok;
     const bool last = c + 1 == chunks;
-    if (half_on && ok) {
-#pragma unroll
-      for (int j = 0; j < 2; ++j) {
+    if (d_on && ok) {
+      {
         uint32_t r[32];
-        tmem_ld_32x32(my + ST + half * 64 + j * 32, r);
+        tmem_ld_32x32(my + ST + col0, r);
         tmem_ld_wait();
         float f[32];
 #pragma unroll
-        for (int e = 0; e < 32; ++e) f[e] = half * 64 + j * 32 + e < (int)nd ? __uint_as_float(r[e]) : 0.f;
+        for (int e = 0; e < 32; ++e) f[e] = __uint_as_float(r[e]);
         if (last) {
 #pragma unroll
           for (int e = 0; e < 32; ++e) {
-            const int d = half * 64 + j * 32 + e;
+            const int d = col0 + e;
             if (row_v < VC && d < p.D) st[d] = f[e];
           }
         } else {
-          put32(s_hi, s_hi + 32768, row_v, j * 4, f);
+          put32(s_hi, s_hi + 16384, row_v, g0, f);
 #pragma unroll
           for (int e = 0; e < 32; ++e) r[e] = __float_as_uint(f[e] * egl_next);
-          tmem_st_32x32(my + ST + half * 64 + j * 32, r);
+          tmem_st_32x32(my + ST + col0, r);
         }
       }
       tmem_st_wait();
