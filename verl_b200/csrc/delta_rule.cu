@@ -610,13 +610,15 @@ __global__ void __launch_bounds__(128) delta_chunk_prep_kernel(const DeltaParams
 //     S^T [v, d]                    += U'^T . K             (U' = e^{G_last - G} U / |k|, fp32 state in TMEM)
 // The MMAs are issued by one thread; between them all warps read their TMEM lanes, scale, split into hi and lo and write
 // the next operand. Warp w owns TMEM lanes 32 (w % 4) .. and the 32 columns 32 (w / 4) .. of each accumulator. K and Q of the next chunk arrive
-// while a chunk is worked on, T and P T of the next chunk once UO is done.
+// (and v) while a chunk is worked on, T and P T of the next chunk once UO is done; outputs leave through shared memory, so
+// that global accesses are whole rows.
 constexpr int DT_THREADS = 512;
 constexpr int DT_KQ = 32768;                     // [K; Q]: two 64-column blocks of 128 rows x 128 bytes
 constexpr int DT_TP_OFF = 2 * DT_KQ;             // hi | lo, 16 KB each
 constexpr int DT_X_OFF = DT_TP_OFF + 32768;      // rhs, then U': hi | lo, [64 tokens][128 columns] in two column blocks
 constexpr int DT_S_OFF = DT_X_OFF + 32768;       // S^T [128 v][128 d]: per column block hi | lo
-constexpr int DT_BAR_OFF = DT_S_OFF + 65536;
+constexpr int DT_V_OFF = DT_S_OFF + 65536;       // two chunks of v [64 tokens][128], 16-byte groups swizzled; then their outputs
+constexpr int DT_BAR_OFF = DT_V_OFF + 2 * 16384;
 constexpr int DT_SMEM = DT_BAR_OFF + 64 + 1024;
 
 __global__ void __launch_bounds__(DT_THREADS, 1)
@@ -656,6 +658,12 @@ delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch
         uint8_t* to = dst + (d >> 6) * 16384 + t * 128 + ((((d & 63) >> 3) ^ (t & 7)) << 4);
         cp_async16(to, src + p.Hk * p.D, on);
         cp_async16(to + DC * 128, src, on);
+      }
+      for (int i = tid; i < DC * 16; i += DT_THREADS) {
+        const int t = i >> 4, g = i & 15;
+        const bool on = t0 + t < n && g * 8 < VC;
+        cp_async16(smem + DT_V_OFF + (c & 1) * 16384 + t * 256 + ((g ^ (t & 7)) << 4),
+                   y + (on ? (long long)(t0 + t) * C + 2 * p.Hk * p.D + h * p.V + v0 + g * 8 : 0), on);
       }
     }
     cp_async_commit();
@@ -734,6 +742,19 @@ delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch
     return good;
   };
 
+  // this thread's token (TMEM rows 0..63: K and U, 64..127: Q and O) and its factors, loaded a chunk ahead. Rows of K:
+  // e^G / |k| and e^{G_last - G} / |k|; rows of Q: e^G / |q|. next_g: e^{G_last} of the chunk after.
+  const int t = (quad & 1) * 32 + lane;
+  float next_a = 0.f, next_b = 0.f, next_g = 1.f;
+  auto load_vec = [&](int c) {
+    if (c < chunks) {
+      const float* vec = reinterpret_cast<const float*>(scr + c * scr_step + DC_VEC_OFF);
+      next_a = __ldg(vec + (quad < 2 ? 0 : DC) + t);
+      next_b = __ldg(vec + 2 * DC + t);
+    }
+    next_g = c + 1 < chunks ? __ldg(reinterpret_cast<const float*>(scr + (c + 1) * scr_step + DC_VEC_OFF) + 3 * DC) : 1.f;
+  };
+  load_vec(0);
   auto read_rq = [&](float (&f)[32]) {
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
@@ -757,25 +778,11 @@ delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch
       tc_commit(bar);
     }
     load_kq(c + 1);
-    const float* vec = reinterpret_cast<const float*>(scr + c * scr_step + DC_VEC_OFF);
-    const int t = (quad & 1) * 32 + lane;        // this thread's token (rows 0..63 K / U, 64..127 Q / O)
-    const bool tok = t0 + t < n;
-    uint4 v[4];
-    float scale_a, scale_b = 0.f;                // rows of K: e^G / |k| and e^{G_last - G} / |k|; rows of Q: e^G / |q|
-    if (quad < 2) {
-      const __nv_bfloat16* vr = y + (long long)(t0 + t) * C + 2 * p.Hk * p.D + h * p.V + v0 + col0;
-#pragma unroll
-      for (int g = 0; g < 4; ++g)
-        v[g] = tok && col0 + g * 8 < VC ? *reinterpret_cast<const uint4*>(vr + g * 8) : make_uint4(0, 0, 0, 0);
-      scale_a = __ldg(vec + t);
-      scale_b = __ldg(vec + 2 * DC + t);
-    } else {
-      scale_a = __ldg(vec + DC + t);
-    }
-    const float egl_next = c + 1 < chunks ? __ldg(reinterpret_cast<const float*>(scr + (c + 1) * scr_step + DC_VEC_OFF) + 3 * DC)
-                                          : 1.f;
+    const float scale_a = next_a, scale_b = next_b, egl_next = next_g;
+    load_vec(c + 1);
     ok = mma_done(4 * c) && ok;
     // right-hand side
+    uint8_t* vrow = smem + DT_V_OFF + (c & 1) * 16384 + t * 256;
     uint8_t* x_hi = smem + DT_X_OFF + (col0 >> 6) * 8192 + t * 128;
     if (quad < 2) {
       {
@@ -783,7 +790,8 @@ delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch
         read_rq(f);
 #pragma unroll
         for (int g = 0; g < 4; ++g) {
-          const uint32_t* vw = reinterpret_cast<const uint32_t*>(&v[g]);
+          const uint4 v4 = *reinterpret_cast<const uint4*>(vrow + (((col0 >> 3) + g) ^ (t & 7)) * 16);
+          const uint32_t vw[4] = {v4.x, v4.y, v4.z, v4.w};
 #pragma unroll
           for (int k = 0; k < 4; ++k) {
             const int e = 8 * g + 2 * k;
@@ -810,7 +818,6 @@ delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch
       tc_commit(bar);
     }
     ok = mma_done(4 * c + 1) && ok;
-    load_tp(c + 1);
     {
       uint32_t r[32];
       tmem_ld_32x32(my + UO + col0, r);
@@ -824,15 +831,11 @@ delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch
         read_rq(f);
 #pragma unroll
         for (int e = 0; e < 32; ++e) f[e] = fmaf(scale_a, f[e], __uint_as_float(r[e]));
-        __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (long long)(first + t0 + t) * p.out_stride +
-                             (long long)h * p.V + v0 + col0;
-        if (tok)
 #pragma unroll
-          for (int g = 0; g < 4; ++g)
-            if (col0 + g * 8 < VC)
-              *reinterpret_cast<uint4*>(out + g * 8) =
-                  make_uint4(pack_bf16x2(f[8 * g], f[8 * g + 1]), pack_bf16x2(f[8 * g + 2], f[8 * g + 3]),
-                             pack_bf16x2(f[8 * g + 4], f[8 * g + 5]), pack_bf16x2(f[8 * g + 6], f[8 * g + 7]));
+        for (int g = 0; g < 4; ++g)
+          *reinterpret_cast<uint4*>(vrow + (((col0 >> 3) + g) ^ (t & 7)) * 16) =
+              make_uint4(pack_bf16x2(f[8 * g], f[8 * g + 1]), pack_bf16x2(f[8 * g + 2], f[8 * g + 3]),
+                         pack_bf16x2(f[8 * g + 4], f[8 * g + 5]), pack_bf16x2(f[8 * g + 6], f[8 * g + 7]));
       }
     }
     fence_proxy_async_smem();
@@ -846,6 +849,14 @@ delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch
           tc_mma_f16(tmem + ST, umma_smem_desc(base + DT_X_OFF + term * 16384 + k * 2048, 8192, 1024),
                      umma_smem_desc(kq + k * 2048, 16384, 1024), id_s, 1);
       tc_commit(bar);
+    }
+    load_tp(c + 1);
+    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (long long)(first + t0) * p.out_stride + (long long)h * p.V + v0;
+    for (int i = tid; i < DC * 16; i += DT_THREADS) {
+      const int tt = i >> 4, g = i & 15;
+      if (t0 + tt < n && g * 8 < VC)
+        *reinterpret_cast<uint4*>(out + (long long)tt * p.out_stride + g * 8) =
+            *reinterpret_cast<const uint4*>(smem + DT_V_OFF + (c & 1) * 16384 + tt * 256 + ((g ^ (tt & 7)) << 4));
     }
     ok = mma_done(4 * c + 2) && ok;
     const bool last = c + 1 == chunks;
