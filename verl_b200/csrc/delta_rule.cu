@@ -32,7 +32,6 @@
 // both operands and sums are fp32.
 #include "common.cuh"
 #include "host_utils.h"
-#include <type_traits>
 
 namespace vb {
 
@@ -97,12 +96,23 @@ struct DeltaParams {
   float eps;
 };
 
+__device__ __forceinline__ void cp_async4(float* dst, const float* src, bool on) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(on ? 4 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+__device__ __forceinline__ void cp_async16(void* dst, const void* src, bool on) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(on ? 16 : 0) : "memory");
+}
+
 // ---------------------------------------------------------------------------------------------------------------
 // One warp per (sequence, tile of tokens, head row); lanes across the head's channels, a sliding window of inputs in
 // registers. Head rows: Hk of q, Hk of k, H of v; a few more rows do the gates.
 constexpr int DP_TT = 64;  // tokens per tile
 constexpr int DP_GATE_ROWS = 8;  // warps that share a tile's gates
-template <typename T, int TAPS, int CPL, bool CHUNK>
+template <typename T, int TAPS, int CPL>
 __global__ void __launch_bounds__(128, CPL * TAPS <= 16 ? 8 : 1) delta_prep_kernel(const DeltaParams p) {
   pdl_trigger();
   pdl_wait();
@@ -185,37 +195,100 @@ __global__ void __launch_bounds__(128, CPL * TAPS <= 16 ? 8 : 1) delta_prep_kern
         for (int j = TAPS - 1; j >= 0; --j) a = fmaf(w[j][i], hist[j][i], a);
 #pragma unroll
         for (int j = TAPS - 1; j > 0; --j) hist[j][i] = hist[j - 1][i];
-        y[i] = CHUNK ? silu_t<T>(a) : silu_f(a);
-        if (CHUNK) y[i] = __bfloat162float(__float2bfloat16(y[i]));  // the norm is that of the stored vector
+        y[i] = silu_f(a);
         ss += y[i] * y[i];  // channels past the head give silu(0) = 0
       }
       float mul = 1.f;
       if (qk) mul = qscale * rsqrtf(warp_reduce_sum(ss) + UNIT_EPS);
-      typedef typename std::conditional<CHUNK, __nv_bfloat16, float>::type Y;
-      Y* dst = static_cast<Y*>(p.qkv) + (long long)(first + t) * C + c0 + cl;
-      if (!CHUNK) {
+      float* dst = static_cast<float*>(p.qkv) + (long long)(first + t) * C + c0 + cl;
 #pragma unroll
-        for (int i = 0; i < CPL; ++i) y[i] *= mul;
-      } else if (qk && lane == 0) {
-        p.unit[(long long)(first + t) * 2 * p.Hk + r] = mul;
-      }
+      for (int i = 0; i < CPL; ++i) y[i] *= mul;
       if (vec) {
-        if (cl < size) store_n<Y, CPL>(dst, y);
+        if (cl < size) store_n<float, CPL>(dst, y);
       } else {
 #pragma unroll
         for (int i = 0; i < CPL; ++i)
-          if (cl + i < size) dst[i] = dl_t<Y>(y[i]);
+          if (cl + i < size) dst[i] = y[i];
       }
     }
   }
 }
 
-__device__ __forceinline__ void cp_async4(float* dst, const float* src, bool on) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(on ? 4 : 0) : "memory");
+// The same for the chunked form, bf16: one CTA per (sequence, tile of tokens, 128 channels of one head row). The tile and
+// the taps in front of it come into shared memory with all loads in flight; a warp takes 16 tokens, a lane 4 channels.
+template <int TAPS>
+__global__ void __launch_bounds__(128) delta_prep_tile_kernel(const DeltaParams p) {
+  __shared__ __align__(16) __nv_bfloat16 x_s[DP_TT + TAPS - 1][128];
+  pdl_trigger();
+  pdl_wait();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, b = blockIdx.z;
+  const int first = p.cu_q[b], n = p.cu_q[b + 1] - first, t0 = blockIdx.x * DP_TT, t1 = min(n, t0 + DP_TT);
+  const int slot = p.slots[b];
+  if (t0 >= n || slot < 0) return;
+  const int start = p.seq_lens[b] - n, C = 2 * p.Hk * p.D + p.H * p.V, vb = (p.V + 127) / 128;
+  const __nv_bfloat16* proj = static_cast<const __nv_bfloat16*>(p.proj) + (long long)first * p.stride;
+  int r = blockIdx.y;
+  if (r == 2 * p.Hk + p.H * vb) {  // the gates
+    for (int i = tid; i < (t1 - t0) * p.H; i += 128) {
+      const int t = t0 + i / p.H, h = i % p.H;
+      const __nv_bfloat16* row = proj + (long long)t * p.stride + C + p.H * p.V;
+      float* g = p.gates + (long long)(first + t) * 2 * p.H;
+      g[h] = sigmoid_f(dl_f(row[h]));
+      g[p.H + h] = -expf(p.a_log[h]) * softplus_f(dl_f(row[p.H + h]) + p.dt_bias[h]);
+    }
+    return;
+  }
+  const bool qk = r < 2 * p.Hk;
+  const int rv = r - 2 * p.Hk;
+  const int c0 = qk ? r * p.D : 2 * p.Hk * p.D + rv / vb * p.V + rv % vb * 128;
+  const int size = qk ? p.D : min(128, p.V - rv % vb * 128);
+  const __nv_bfloat16* ring = static_cast<const __nv_bfloat16*>(p.ring) + (long long)slot * p.taps * C + c0;
+  for (int i = tid; i < (DP_TT + TAPS - 1) * 16; i += 128) {
+    const int k = i >> 4, c = (i & 15) * 8, t = t0 + k - (TAPS - 1);  // row k holds token t
+    const bool cur = t >= 0, past = !cur && start + t >= 0 && -t < p.taps;
+    const bool on = c < size && t < t1 && (cur || past);
+    const __nv_bfloat16* src = !on ? proj : cur ? proj + (long long)t * p.stride + c0 + c : ring + (long long)((start + t) % p.taps) * C + c;
+    cp_async16(&x_s[k][c], src, on);
+  }
+  cp_async_commit();
+  const int cl = lane * 4;
+  float w[TAPS][4];  // w[j]: tap of the token j places back
+  const __nv_bfloat16* cw = static_cast<const __nv_bfloat16*>(p.conv_w) + (long long)(c0 + cl) * p.taps;
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j][i] = cl < size && j < p.taps ? dl_f(cw[i * p.taps + p.taps - 1 - j]) : 0.f;
+  const float qscale = r < p.Hk ? 1.f / sqrtf((float)p.D) : 1.f;
+  cp_async_wait<0>();
+  __syncthreads();
+  const int base = warp * (DP_TT / 4);
+  float hist[TAPS][4];
+#pragma unroll
+  for (int j = 1; j < TAPS; ++j) load_n<__nv_bfloat16, 4>(&x_s[base + TAPS - 1 - j][cl], hist[j]);
+#pragma unroll 4
+  for (int k = 0; k < DP_TT / 4; ++k) {
+    const int t = t0 + base + k;
+    if (t >= t1) break;
+    load_n<__nv_bfloat16, 4>(&x_s[base + k + TAPS - 1][cl], hist[0]);
+    float y[4], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      float a = 0.f;
+#pragma unroll
+      for (int j = TAPS - 1; j >= 0; --j) a = fmaf(w[j][i], hist[j][i], a);
+#pragma unroll
+      for (int j = TAPS - 1; j > 0; --j) hist[j][i] = hist[j - 1][i];
+      y[i] = __bfloat162float(__float2bfloat16(silu_t<__nv_bfloat16>(a)));  // the norm is that of the stored vector
+      ss = fmaf(y[i], y[i], ss);
+    }
+    if (qk) {
+      ss = warp_reduce_sum(ss);
+      if (lane == 0) p.unit[(long long)(first + t) * 2 * p.Hk + r] = qscale * rsqrtf(ss + UNIT_EPS);
+    }
+    if (cl < size)
+      store_n<__nv_bfloat16, 4>(static_cast<__nv_bfloat16*>(p.qkv) + (long long)(first + t) * C + c0 + cl, y);
+  }
 }
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 __device__ __forceinline__ float sum8(float v) {  // over groups of eight lanes
   v += __shfl_xor_sync(0xffffffffu, v, 1);
@@ -379,9 +452,6 @@ __device__ __forceinline__ void mma16(float (&c)[4], const uint32_t (&a)[4], uin
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ void cp_async16(void* dst, const void* src, bool on) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(on ? 16 : 0) : "memory");
-}
 // x = hi + lo, both bf16, for two neighbours packed into 32 bits
 __device__ __forceinline__ void split2(float x0, float x1, uint32_t& hi, uint32_t& lo) {
   hi = pack_bf16x2(x0, x1);
@@ -396,6 +466,26 @@ __device__ __forceinline__ const __nv_bfloat16* frag_a(const __nv_bfloat16* t, i
 template <int PITCH>
 __device__ __forceinline__ const __nv_bfloat16* frag_bn(const __nv_bfloat16* t, int k, int n, int lane) {
   return t + (n + ((lane >> 4) & 1) * 8 + (lane & 7)) * PITCH + k + ((lane >> 3) & 1) * 8;
+}
+
+// Column `col` >= LO of the inverse of the unit lower triangular I + A (rows of A in shared memory, pitch AP).
+template <int LO, int AP>
+__device__ __forceinline__ void solve_columns(const float* A, int col, float (&x)[DC]) {
+#pragma unroll
+  for (int i = 0; i < LO; ++i) x[i] = 0.f;
+#pragma unroll
+  for (int i = LO; i < DC; ++i) {
+    float s0 = i == col ? 1.f : 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
+#pragma unroll
+    for (int k = LO; k < i; k += 4) {
+      const float4 a = *reinterpret_cast<const float4*>(A + i * AP + k);  // entries from the diagonal on are zero
+      s0 = fmaf(-a.x, x[k], s0);
+      if (k + 1 < i) s1 = fmaf(-a.y, x[k + 1], s1);
+      if (k + 2 < i) s2 = fmaf(-a.z, x[k + 2], s2);
+      if (k + 3 < i) s3 = fmaf(-a.w, x[k + 3], s3);
+    }
+    x[i] = (s0 + s1) + (s2 + s3);
+  }
 }
 
 // One CTA of four warps per (chunk, NH heads that share their q and k): T = (I + A)^-1 diag(beta) and P T of each.
@@ -525,24 +615,11 @@ __global__ void __launch_bounds__(128) delta_chunk_prep_kernel(const DeltaParams
     }
   }
   __syncthreads();
-  // forward substitution: a thread owns one column of (I + A)^-1
+  // forward substitution: a thread owns one column of (I + A)^-1. Columns from 32 on are zero above row 32.
   float x[DC];
   if (tid < NH * DC) {
-    const int col = tid % DC;
-    const float* A = a_s + tid / DC * DC * AP;
-#pragma unroll
-    for (int i = 0; i < DC; ++i) {
-      float s0 = i == col ? 1.f : 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
-#pragma unroll
-      for (int k = 0; k < i; k += 4) {
-        const float4 a = *reinterpret_cast<const float4*>(A + i * AP + k);  // entries from the diagonal on are zero
-        s0 = fmaf(-a.x, x[k], s0);
-        if (k + 1 < i) s1 = fmaf(-a.y, x[k + 1], s1);
-        if (k + 2 < i) s2 = fmaf(-a.z, x[k + 2], s2);
-        if (k + 3 < i) s3 = fmaf(-a.w, x[k + 3], s3);
-      }
-      x[i] = (s0 + s1) + (s2 + s3);
-    }
+    if (tid & 32) solve_columns<32, AP>(a_s + tid / DC * DC * AP, tid % DC, x);
+    else solve_columns<0, AP>(a_s + tid / DC * DC * AP, tid % DC, x);
   }
   __syncthreads();  // A is read: T takes its place
   if (tid < NH * DC) {
@@ -1085,16 +1162,16 @@ __global__ void __launch_bounds__(DD_THREADS) delta_step_kernel(const DeltaParam
   for (int c = tid; c < p.V; c += DD_THREADS) out[c] = dl_t<T>(o_s[c] * inv * dl_f<T>(w[c]) * silu_f(dl_f<T>(gate[c])));
 }
 
-template <typename T, bool CHUNK>
+template <typename T>
 static int run_prep(const DeltaParams& p, int max_q, cudaStream_t stream) {
   const dim3 g((max_q + DP_TT - 1) / DP_TT, (2 * p.Hk + p.H + DP_GATE_ROWS + 3) / 4, p.B), b(128);
   const int cpl = ((p.D > p.V ? p.D : p.V) + 31) / 32;
   cudaError_t e = cudaErrorInvalidValue;
 #define VB_PREP(TAPS)                                                                                      \
-  (cpl <= 1   ? vb_launch_pdl(delta_prep_kernel<T, TAPS, 1, CHUNK>, g, b, 0, stream, 1, p)                        \
-   : cpl <= 2 ? vb_launch_pdl(delta_prep_kernel<T, TAPS, 2, CHUNK>, g, b, 0, stream, 1, p)                        \
-   : cpl <= 4 ? vb_launch_pdl(delta_prep_kernel<T, TAPS, 4, CHUNK>, g, b, 0, stream, 1, p)                        \
-              : vb_launch_pdl(delta_prep_kernel<T, TAPS, 8, CHUNK>, g, b, 0, stream, 1, p))
+  (cpl <= 1   ? vb_launch_pdl(delta_prep_kernel<T, TAPS, 1>, g, b, 0, stream, 1, p)                        \
+   : cpl <= 2 ? vb_launch_pdl(delta_prep_kernel<T, TAPS, 2>, g, b, 0, stream, 1, p)                        \
+   : cpl <= 4 ? vb_launch_pdl(delta_prep_kernel<T, TAPS, 4>, g, b, 0, stream, 1, p)                        \
+              : vb_launch_pdl(delta_prep_kernel<T, TAPS, 8>, g, b, 0, stream, 1, p))
   e = p.taps <= 4 ? VB_PREP(4) : VB_PREP(8);
 #undef VB_PREP
   vb_count_launch();
@@ -1165,7 +1242,15 @@ static int run_delta(const DeltaParams& p, int tokens, int max_q, uint8_t* chunk
     if (nr == 16) return run_step<T, 16>(p, stream);
     return run_step<T, 32>(p, stream);
   }
-  int rc = chunk_scratch ? run_prep<T, true>(p, max_q, stream) : run_prep<T, false>(p, max_q, stream);
+  int rc;
+  if (chunk_scratch) {
+    const dim3 g((max_q + DP_TT - 1) / DP_TT, 2 * p.Hk + p.H * ((p.V + 127) / 128) + 1, p.B);
+    rc = (int)(p.taps <= 4 ? vb_launch_pdl(delta_prep_tile_kernel<4>, g, dim3(128), 0, stream, 1, p)
+                           : vb_launch_pdl(delta_prep_tile_kernel<8>, g, dim3(128), 0, stream, 1, p));
+    vb_count_launch();
+  } else {
+    rc = run_prep<T>(p, max_q, stream);
+  }
   if (rc) return rc;
   if (chunk_scratch)
     rc = run_chunks(p, tokens, chunk_scratch, status, stream);
@@ -1204,7 +1289,7 @@ extern "C" int vb_delta_rule(const void* proj, long long stride, const void* con
   if (Hk <= 0 || H % Hk != 0 || D <= 0 || D > 256 || V <= 0 || V > 256 || taps < 1 || taps > 8 || B > 65535) return -3;
   if (max_q > 1 && (qkv == nullptr || gates == nullptr)) return -3;
   if (max_q > 1 && chunk_scratch != nullptr &&
-      (f32 || unit == nullptr || !vb_delta_chunk_supported(D, V) || (out_stride & 7) || (reinterpret_cast<uintptr_t>(qkv) & 15)))
+      (f32 || unit == nullptr || !vb_delta_chunk_supported(D, V) || (out_stride & 7) || (stride & 7) || (reinterpret_cast<uintptr_t>(qkv) & 15)))
     return -3;
   DeltaParams p{proj, stride, conv_w, a_log, dt_bias, norm_w, ring, state, cu_q, seq_lens, slots, qkv, unit, gates, out,
                 out_stride, B, H, Hk, D, V, taps, eps};

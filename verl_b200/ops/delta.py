@@ -28,7 +28,7 @@ def delta_rule(proj: torch.Tensor, conv_w: torch.Tensor, a_log: torch.Tensor, dt
     if proj.is_cuda:
         qkv = gates = unit = scratch = None
         if max_q > 1:
-            can = proj.dtype == torch.bfloat16 and bool(_lib.fn("vb_delta_chunk_supported")(dim, vdim))
+            can = proj.dtype == torch.bfloat16 and proj.stride(0) % 8 == 0 and bool(_lib.fn("vb_delta_chunk_supported")(dim, vdim))
             if impl == "chunk" and not can:
                 raise ValueError(f"the chunked delta rule does not support dim={dim} vdim={vdim} in {proj.dtype}")
             chunk = can and (impl == "chunk" or (impl == "auto" and max_q >= CHUNK_MIN))
