@@ -468,26 +468,6 @@ __device__ __forceinline__ const __nv_bfloat16* frag_bn(const __nv_bfloat16* t, 
   return t + (n + ((lane >> 4) & 1) * 8 + (lane & 7)) * PITCH + k + ((lane >> 3) & 1) * 8;
 }
 
-// Column `col` >= LO of the inverse of the unit lower triangular I + A (rows of A in shared memory, pitch AP).
-template <int LO, int AP>
-__device__ __forceinline__ void solve_columns(const float* A, int col, float (&x)[DC]) {
-#pragma unroll
-  for (int i = 0; i < LO; ++i) x[i] = 0.f;
-#pragma unroll
-  for (int i = LO; i < DC; ++i) {
-    float s0 = i == col ? 1.f : 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
-#pragma unroll
-    for (int k = LO; k < i; k += 4) {
-      const float4 a = *reinterpret_cast<const float4*>(A + i * AP + k);  // entries from the diagonal on are zero
-      s0 = fmaf(-a.x, x[k], s0);
-      if (k + 1 < i) s1 = fmaf(-a.y, x[k + 1], s1);
-      if (k + 2 < i) s2 = fmaf(-a.z, x[k + 2], s2);
-      if (k + 3 < i) s3 = fmaf(-a.w, x[k + 3], s3);
-    }
-    x[i] = (s0 + s1) + (s2 + s3);
-  }
-}
-
 // One CTA of four warps per (chunk, NH heads that share their q and k): T = (I + A)^-1 diag(beta) and P T of each.
 template <int DP, int NH>
 struct ChunkPrepSmem {
@@ -615,15 +595,50 @@ __global__ void __launch_bounds__(128) delta_chunk_prep_kernel(const DeltaParams
     }
   }
   __syncthreads();
-  // forward substitution: a thread owns one column of (I + A)^-1. Columns from 32 on are zero above row 32.
-  float x[DC];
-  if (tid < NH * DC) {
-    if (tid & 32) solve_columns<32, AP>(a_s + tid / DC * DC * AP, tid % DC, x);
-    else solve_columns<0, AP>(a_s + tid / DC * DC * AP, tid % DC, x);
+  // forward substitution by blocks of 16 rows: a thread owns one column of (I + A)^-1, whose finished blocks replace the
+  // rows of A that have been read (rolled loops: straight-line code for all 64 rows runs at instruction-fetch speed)
+  const int col = tid % DC;
+  float* A = a_s + (NH == 1 ? 0 : tid / DC) * DC * AP;
+  const bool solver = tid < NH * DC;
+#pragma unroll 1
+  for (int I = 0; I < DC; I += 16) {
+    float r[16];
+    if (solver) {
+#pragma unroll
+      for (int e = 0; e < 16; ++e) r[e] = I + e == col ? 1.f : 0.f;
+#pragma unroll 1
+      for (int k = 0; k < I; k += 4) {
+        const float x0 = A[k * AP + col], x1 = A[(k + 1) * AP + col], x2 = A[(k + 2) * AP + col], x3 = A[(k + 3) * AP + col];
+#pragma unroll
+        for (int e = 0; e < 16; ++e) {
+          const float4 a = *reinterpret_cast<const float4*>(A + (I + e) * AP + k);
+          r[e] = fmaf(-a.x, x0, fmaf(-a.y, x1, fmaf(-a.z, x2, fmaf(-a.w, x3, r[e]))));
+        }
+      }
+#pragma unroll
+      for (int e = 1; e < 16; ++e)
+#pragma unroll
+        for (int f = 0; f < e; f += 4) {
+          const float4 a = *reinterpret_cast<const float4*>(A + (I + e) * AP + I + f);  // zero from the diagonal on
+          r[e] = fmaf(-a.x, r[f], r[e]);
+          if (f + 1 < e) r[e] = fmaf(-a.y, r[f + 1], r[e]);
+          if (f + 2 < e) r[e] = fmaf(-a.z, r[f + 2], r[e]);
+          if (f + 3 < e) r[e] = fmaf(-a.w, r[f + 3], r[e]);
+        }
+    }
+    __syncthreads();  // the rows I .. I + 15 of A are read
+    if (solver)
+#pragma unroll
+      for (int e = 0; e < 16; ++e) A[(I + e) * AP + col] = r[e];
   }
-  __syncthreads();  // A is read: T takes its place
-  if (tid < NH * DC) {
-    const int col = tid % DC, m = tid / DC * 2;
+  float x[DC];
+  if (solver) {
+#pragma unroll
+    for (int i = 0; i < DC; ++i) x[i] = A[i * AP + col];  // this thread's own column
+  }
+  __syncthreads();  // T takes the place of A
+  if (solver) {
+    const int m = tid / DC * 2;
     const float beta = b_s[tid];
 #pragma unroll
     for (int i = 0; i < DC; ++i) {
