@@ -195,7 +195,7 @@ def oracle_delta(proj, cw, a_log, dt_bias, nw, H, G, D, V, eps):
 
 
 @pytest.mark.parametrize("dtype,impl", [(F32, "scan"), (BF, "scan"), (BF, "chunk")])
-@pytest.mark.parametrize("H,G,D,V,taps", [(4, 2, 64, 32, 4), (2, 2, 40, 72, 3), (3, 1, 128, 128, 1), (2, 1, 96, 136, 8),
+@pytest.mark.parametrize("H,G,D,V,taps", [(6, 2, 56, 24, 4), (2, 2, 40, 72, 3), (3, 1, 128, 128, 1), (2, 1, 96, 136, 8),
                                           (5, 5, 12, 20, 2), (1, 1, 200, 256, 5)])
 def test_delta_rule(dtype, impl, H, G, D, V, taps):
     """A whole prompt, portions down to two tokens and single tokens give the same outputs and state; the state slots hold

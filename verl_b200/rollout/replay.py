@@ -61,7 +61,8 @@ def main(argv=None) -> int:
         if not line.strip():
             continue
         step = json.loads(line)
-        logits = eng.feed([(e["id"], e["tokens"], e["want"]) for e in step["entries"]], step.get("end") or [])
+        logits = eng.feed([(e["id"], e["tokens"], e["want"]) for e in step["entries"] if e["tokens"]],
+                          step.get("end") or [])
         if logits is not None:
             logits.cpu().numpy().astype(np.dtype("<f4"), copy=False).tofile(out / f"{step['step']}.f32")
         code, blk, detail = _lib.read_status(eng.device)
