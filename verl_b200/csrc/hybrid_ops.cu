@@ -1,5 +1,6 @@
-// Token-wise kernels of layer-list decoders (models/hybrid.py): 32-bit residual stream with fused add + RMSNorm, scaled
-// embedding, clamped GLU, whole-projection query / key norm fused with the paged KV write, a CUDA-core matrix product for
+// Token-wise kernels of layer-list decoders (models/hybrid.py): 32-bit residual stream with fused add + RMSNorm (of the
+// stream, or of what is added to it), scaled embedding, gated linear units, query / key norms over the projection or per head
+// with rotary positions, fused with the paged KV write, the same for latent attention, CUDA-core matrix products for
 // 32-bit weights (and for shapes that TMA cannot describe), and a CUDA-core paged attention that takes any head size.
 //
 // Every kernel is a template over the activation type (bf16 when serving, fp32 for the exact mode); arithmetic is fp32.
@@ -57,10 +58,10 @@ __device__ __forceinline__ float block_sum_all(float v, float* sh) {
 }
 
 // ---------------------------------------------------------------------------------------------------------------
-// res[t] = table[ids[t]] * scale, fp32.
+// res[t] = table[ids[t]] * scale, fp32; y (when given): the same in the table's type.
 template <typename T>
 __global__ void embed_scaled_kernel(const long long* __restrict__ ids, const T* __restrict__ table,
-                                    float* __restrict__ res, int H, float scale) {
+                                    float* __restrict__ res, T* __restrict__ y, int H, float scale) {
   pdl_trigger();
   pdl_wait();
   const T* src = table + ids[blockIdx.x] * (long long)H;
@@ -72,9 +73,14 @@ __global__ void embed_scaled_kernel(const long long* __restrict__ ids, const T* 
 #pragma unroll
       for (int i = 0; i < 8; ++i) f[i] *= scale;
       st8(dst + v * 8, f);
+      if (y) st8(y + (long long)blockIdx.x * H + v * 8, f);
     }
   } else {
-    for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = to_f<T>(src[i]) * scale;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+      const float f = to_f<T>(src[i]) * scale;
+      dst[i] = f;
+      if (y) y[(long long)blockIdx.x * H + i] = from_f<T>(f);
+    }
   }
 }
 
@@ -136,17 +142,99 @@ __global__ void add_rmsnorm_kernel(const T* __restrict__ delta, long long delta_
 }
 
 // ---------------------------------------------------------------------------------------------------------------
+// res += delta / sqrt(mean(delta^2) + eps) * w; y = res, or with fw: y = res / sqrt(mean(res^2) + eps) * fw * fscale.
+template <typename T>
+__global__ void rmsnorm_add_kernel(const T* __restrict__ delta, long long delta_stride, float* __restrict__ res,
+                                   const T* __restrict__ w, const T* __restrict__ fw, float fscale, T* __restrict__ y,
+                                   int H, float eps) {
+  extern __shared__ float row[];
+  __shared__ float sh[32];
+  pdl_trigger();
+  pdl_wait();
+  const T* d = delta + (long long)blockIdx.x * delta_stride;
+  float* r = res + (long long)blockIdx.x * H;
+  T* out = y + (long long)blockIdx.x * H;
+  const bool vec = (H & 7) == 0 && (delta_stride & 7) == 0;
+  float ss = 0.f;
+  if (vec) {
+    for (int v = threadIdx.x; v < (H >> 3); v += blockDim.x) {
+      float f[8];
+      ld8(d + v * 8, f);
+      st8(row + v * 8, f);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) ss += f[i] * f[i];
+    }
+  } else {
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+      const float f = to_f<T>(d[i]);
+      row[i] = f;
+      ss += f * f;
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum_all(ss, sh) / (float)H + eps);
+  ss = 0.f;
+  if (vec) {
+    for (int v = threadIdx.x; v < (H >> 3); v += blockDim.x) {  // the same elements this thread has stored
+      float f[8], g[8], x[8];
+      ld8(r + v * 8, x);
+      ld8(row + v * 8, f);
+      ld8(w + v * 8, g);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        x[i] += f[i] * inv * g[i];
+        ss += x[i] * x[i];
+      }
+      st8(r + v * 8, x);
+      if (fw) st8(row + v * 8, x); else st8(out + v * 8, x);
+    }
+  } else {
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+      const float x = r[i] + row[i] * inv * to_f<T>(w[i]);
+      r[i] = x;
+      ss += x * x;
+      if (fw) row[i] = x; else out[i] = from_f<T>(x);
+    }
+  }
+  if (fw == nullptr) return;
+  const float fi = fscale / sqrtf(block_sum_all(ss, sh) / (float)H + eps);
+  if (vec) {
+    for (int v = threadIdx.x; v < (H >> 3); v += blockDim.x) {
+      float f[8], g[8];
+      ld8(row + v * 8, f);
+      ld8(fw + v * 8, g);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) f[i] = f[i] * fi * g[i];
+      st8(out + v * 8, f);
+    }
+  } else {
+    for (int i = threadIdx.x; i < H; i += blockDim.x) out[i] = from_f<T>(row[i] * fi * to_f<T>(fw[i]));
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------------
 // gu rows hold [gate (F) | up (F)]: g = min(gate, limit), u = clamp(up, -limit, limit), y = g sigmoid(alpha g) (u + 1).
 template <typename T>
-__device__ __forceinline__ float clamped_glu_1(float g, float u, float limit, float alpha) {
-  g = fminf(g, limit);
-  u = fminf(fmaxf(u, -limit), limit);
-  if (sizeof(T) == 2) return __fdividef(g, 1.f + __expf(-alpha * g)) * (u + 1.f);  // error far below a bf16 ulp
-  return g / (1.f + expf(-alpha * g)) * (u + 1.f);
-}
+struct ClampedGlu {
+  float limit, alpha;
+  __device__ __forceinline__ float operator()(float g, float u) const {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    if (sizeof(T) == 2) return __fdividef(g, 1.f + __expf(-alpha * g)) * (u + 1.f);  // error far below a bf16 ulp
+    return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+  }
+};
+// y = gelu(gate) * up with the tanh form of gelu: 0.5 g (1 + tanh(z)) = g sigmoid(2 z), z = sqrt(2 / pi) (g + 0.044715 g^3)
 template <typename T>
-__global__ void clamped_glu_kernel(const T* __restrict__ gu, long long stride, T* __restrict__ y, long long total, int F,
-                                   float limit, float alpha) {
+struct GeluTanhGlu {
+  __device__ __forceinline__ float operator()(float g, float u) const {
+    const float z = 0.7978845608028654f * (g + 0.044715f * g * g * g);
+    if (sizeof(T) == 2) return __fdividef(g, 1.f + __expf(-2.f * z)) * u;
+    return 0.5f * g * (1.f + tanhf(z)) * u;
+  }
+};
+template <typename T, typename Act>
+__global__ void glu_kernel(const T* __restrict__ gu, long long stride, T* __restrict__ y, long long total, int F,
+                           const Act act) {
   pdl_trigger();
   pdl_wait();
   const long long step = (long long)gridDim.x * blockDim.x;
@@ -159,14 +247,14 @@ __global__ void clamped_glu_kernel(const T* __restrict__ gu, long long stride, T
       ld8(gu + t * stride + c, g);
       ld8(gu + t * stride + F + c, u);
 #pragma unroll
-      for (int k = 0; k < 8; ++k) g[k] = clamped_glu_1<T>(g[k], u[k], limit, alpha);
+      for (int k = 0; k < 8; ++k) g[k] = act(g[k], u[k]);
       st8(y + t * F + c, g);
     }
   } else {
     for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += step) {
       const long long t = i / F;
       const int c = (int)(i - t * F);
-      y[i] = from_f<T>(clamped_glu_1<T>(to_f<T>(gu[t * stride + c]), to_f<T>(gu[t * stride + F + c]), limit, alpha));
+      y[i] = from_f<T>(act(to_f<T>(gu[t * stride + c]), to_f<T>(gu[t * stride + F + c])));
     }
   }
 }
@@ -254,6 +342,232 @@ __global__ void qk_norm_kv_write_kernel(T* __restrict__ qkv, long long stride, c
 }
 
 // ---------------------------------------------------------------------------------------------------------------
+// Cosines and sines of position * f_i for the pairs i of a rotation, times `amp`, in shared memory. Angles are fp32.
+__device__ __forceinline__ void rotation_table(float2* cs, const float* __restrict__ freqs, int n, long long pos, float amp) {
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    float sn, c;
+    sincosf((float)pos * freqs[i], &sn, &c);
+    cs[i] = make_float2(c * amp, sn * amp);
+  }
+}
+constexpr int ROT_MAX = 256;  // pairs of a rotation
+
+// One block per token. qkv row = [q (Hq * D) | k (Hk * D) | v (Hk * Dv) | ...]: every q and k head is divided by its root mean
+// square and multiplied by the weight of size D that all heads share (no weights: left as it is), then its first 2 * n_rot
+// dimensions turn. q in place; k and v go to the token's place in the paged caches (slot < 0: no write).
+// VEC: 8 elements per lane, `lanes` lanes per head (adjacent pairs only). Otherwise a warp per head with its row in shared memory.
+template <typename T, bool VEC>
+__global__ void head_norm_rope_kv_write_kernel(T* __restrict__ qkv, long long stride, const T* __restrict__ qw,
+                                               const T* __restrict__ kw, const float* __restrict__ freqs, int n_rot,
+                                               int interleaved, float amp, const long long* __restrict__ positions,
+                                               const long long* __restrict__ slots, T* __restrict__ kc, T* __restrict__ vc,
+                                               int Hq, int Hk, int D, int Dv, int block_size, float eps, int lanes) {
+  __shared__ float2 cs[ROT_MAX];
+  extern __shared__ float rows[];
+  pdl_trigger();
+  pdl_wait();
+  T* base = qkv + (long long)blockIdx.x * stride;
+  const long long slot = slots[blockIdx.x];
+  const long long blk = slot / block_size, off = slot % block_size;
+  rotation_table(cs, freqs, n_rot, positions[blockIdx.x], amp);
+  __syncthreads();
+  auto k_dst = [&](int hk) { return kc + ((blk * Hk + hk) * block_size + off) * (long long)D; };
+  if (VEC) {
+    const int per_block = blockDim.x / lanes, sub = threadIdx.x / lanes, e0 = (threadIdx.x % lanes) * 8;
+    for (int h0 = 0; h0 < Hq + Hk; h0 += per_block) {  // uniform trip count: the lanes of a warp shuffle together
+      const int h = h0 + sub;
+      const bool on = h < Hq + Hk && e0 < D;
+      float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      T* src = base + (long long)h * D + e0;  // k follows q
+      if (on) ld8(src, f);
+      const T* w = h < Hq ? qw : kw;
+      if (qw != nullptr) {
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) ss += f[i] * f[i];
+        for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        const float inv = 1.f / sqrtf(ss / (float)D + eps);
+        if (on) {
+          float g[8];
+          ld8(w + e0, g);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) f[i] = f[i] * inv * g[i];
+        }
+      }
+      if (!on) continue;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        if ((e0 >> 1) + i < n_rot) {
+          const float2 c = cs[(e0 >> 1) + i];
+          const float u = f[2 * i], v = f[2 * i + 1];
+          f[2 * i] = u * c.x - v * c.y;
+          f[2 * i + 1] = v * c.x + u * c.y;
+        }
+      }
+      if (h < Hq) st8(src, f);
+      else if (slot >= 0) st8(k_dst(h - Hq) + e0, f);
+    }
+  } else {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    float* row = rows + warp * D;
+    for (int h = warp; h < Hq + Hk; h += blockDim.x >> 5) {
+      T* src = base + (long long)h * D;
+      const T* w = h < Hq ? qw : kw;
+      float ss = 0.f;
+      for (int d = lane; d < D; d += 32) {
+        const float f = to_f<T>(src[d]);
+        row[d] = f;
+        ss += f * f;
+      }
+      ss = warp_reduce_sum(ss);
+      __syncwarp();
+      const float inv = 1.f / sqrtf(ss / (float)D + eps);
+      auto at = [&](int d) { return w != nullptr ? row[d] * inv * to_f<T>(w[d]) : row[d]; };
+      if (h >= Hq && slot < 0) continue;
+      T* dst = h < Hq ? src : k_dst(h - Hq);
+      for (int d = lane; d < D; d += 32) {
+        float f = at(d);
+        if (d < 2 * n_rot) {
+          const int i = interleaved ? d >> 1 : d % n_rot;
+          const bool second = interleaved ? (d & 1) != 0 : d >= n_rot;
+          const float other = at(interleaved ? d ^ 1 : (second ? d - n_rot : d + n_rot));
+          f = second ? f * cs[i].x + other * cs[i].y : f * cs[i].x - other * cs[i].y;
+        }
+        dst[d] = from_f<T>(f);
+      }
+      __syncwarp();
+    }
+  }
+  if (slot < 0) return;
+  const T* v = base + (long long)(Hq + Hk) * D;
+  constexpr int W = VEC ? 8 : 1;
+  for (int i = threadIdx.x * W; i < Hk * Dv; i += blockDim.x * W) {
+    const int h = i / Dv, d = i - h * Dv;
+    T* dst = vc + ((blk * Hk + h) * block_size + off) * (long long)Dv + d;
+    if (VEC) {
+      float f[8];
+      ld8(v + i, f);
+      st8(dst, f);
+    } else {
+      *dst = v[i];
+    }
+  }
+}
+
+// One block per token. proj row = [q (H heads of dim + rot) | latent (rank) | rotated key (rot) | ...]: the rotated parts turn
+// (pair i = (i, i + rot / 2)), q in place; normed latent and rotated key go to the token's row of the pages.
+template <typename T, bool VEC>
+__global__ void latent_rope_write_kernel(T* __restrict__ proj, long long stride, const T* __restrict__ w,
+                                         const float* __restrict__ freqs, float amp, const long long* __restrict__ positions,
+                                         const long long* __restrict__ slots, T* __restrict__ pages, int width, int H, int dim,
+                                         int rot, int rank, float eps) {
+  __shared__ float2 cs[ROT_MAX];
+  __shared__ float sh[32];
+  pdl_trigger();
+  pdl_wait();
+  T* base = proj + (long long)blockIdx.x * stride;
+  const T* c = base + (long long)H * (dim + rot);
+  const long long slot = slots[blockIdx.x];
+  const int half = rot >> 1;
+  constexpr int W = VEC ? 8 : 1;
+  rotation_table(cs, freqs, half, positions[blockIdx.x], amp);
+  float ss = 0.f;
+  for (int i = threadIdx.x * W; i < rank; i += blockDim.x * W) {
+    float f[W];
+    if constexpr (VEC) ld8(c + i, f); else f[0] = to_f<T>(c[i]);
+#pragma unroll
+    for (int e = 0; e < W; ++e) ss += f[e] * f[e];
+  }
+  ss = block_sum_all(ss, sh);  // also orders the table before its readers
+  const float inv = 1.f / sqrtf(ss / (float)rank + eps);
+  T* dst = pages + slot * width;
+  // heads 0 .. H - 1: queries in place; head H: the key
+  for (int j = threadIdx.x; j < (H + 1) * (half / W); j += blockDim.x) {
+    const int h = j / (half / W), i = (j - h * (half / W)) * W;
+    const T* src = h < H ? base + (long long)h * (dim + rot) + dim : c + rank;
+    T* to = h < H ? base + (long long)h * (dim + rot) + dim : dst + rank;
+    if (h == H && slot < 0) continue;
+    float u[W], v[W], a[W], b[W];
+    if constexpr (VEC) {
+      ld8(src + i, u);
+      ld8(src + half + i, v);
+    } else {
+      u[0] = to_f<T>(src[i]);
+      v[0] = to_f<T>(src[half + i]);
+    }
+#pragma unroll
+    for (int e = 0; e < W; ++e) {
+      const float2 k = cs[i + e];
+      a[e] = u[e] * k.x - v[e] * k.y;
+      b[e] = v[e] * k.x + u[e] * k.y;
+    }
+    if constexpr (VEC) {
+      st8(to + i, a);
+      st8(to + half + i, b);
+    } else {
+      to[i] = from_f<T>(a[0]);
+      to[half + i] = from_f<T>(b[0]);
+    }
+  }
+  if (slot < 0) return;
+  for (int i = threadIdx.x * W; i < rank; i += blockDim.x * W) {
+    float f[W], g[W];
+    if constexpr (VEC) {
+      ld8(c + i, f);
+      ld8(w + i, g);
+    } else {
+      f[0] = to_f<T>(c[i]);
+      g[0] = to_f<T>(w[i]);
+    }
+#pragma unroll
+    for (int e = 0; e < W; ++e) f[e] = f[e] * inv * g[e];
+    if constexpr (VEC) st8(dst + i, f); else dst[i] = from_f<T>(f[0]);
+  }
+}
+
+// rows[ctx_cu[b] + i] = page row of token i of sequence b, in 16-byte units. One warp per row.
+__global__ void latent_gather_kernel(const uint4* __restrict__ pages, const int* __restrict__ block_table, int max_blocks,
+                                     const int* __restrict__ ctx_cu, uint4* __restrict__ rows, int total, int B, int units,
+                                     int block_size) {
+  pdl_trigger();
+  pdl_wait();
+  const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (r >= total) return;
+  int lo = 0, hi = B - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (ctx_cu[mid] <= r) lo = mid; else hi = mid - 1;
+  }
+  const int i = r - ctx_cu[lo];
+  const long long row = (long long)block_table[(long long)lo * max_blocks + i / block_size] * block_size + i % block_size;
+  for (int u = lane; u < units; u += 32) rows[(long long)r * units + u] = pages[row * units + u];
+}
+
+// out[t, h, n] = sum_k a[t, h, k] b_h[k, n] for n < N (b_h stored [N, K], or [K, N] with b_mn), times sigmoid(gate[t, h * N + n]);
+// then `tail` elements copied from a[t, h, K ...], then zeros up to `width`. fp32 sums, one thread per element.
+template <typename T>
+__global__ void head_gemm_simt_kernel(const T* __restrict__ a, long long a_t, long long a_h, const T* __restrict__ b, int b_mn,
+                                      T* __restrict__ out, long long o_t, long long o_h, const T* __restrict__ gate,
+                                      long long gate_stride, int K, int N, int tail, int width) {
+  pdl_trigger();
+  pdl_wait();
+  const int n = blockIdx.z * blockDim.x + threadIdx.x, h = blockIdx.y;
+  const long long t = blockIdx.x;
+  if (n >= width) return;
+  const T* ar = a + t * a_t + h * a_h;
+  float x = 0.f;
+  if (n < N) {
+    const T* br = b + (long long)h * N * K + (b_mn ? n : (long long)n * K);
+    const int step = b_mn ? N : 1;
+    for (int k = 0; k < K; ++k) x = fmaf(to_f<T>(ar[k]), to_f<T>(br[(long long)k * step]), x);
+    if (gate) x /= 1.f + expf(-to_f<T>(gate[t * gate_stride + (long long)h * N + n]));
+  } else if (n < N + tail) {
+    x = to_f<T>(ar[K + n - N]);
+  }
+  out[t * o_t + h * o_h + n] = from_f<T>(x);
+}
+
+// ---------------------------------------------------------------------------------------------------------------
 // C[M, N] = A[M, K] . B[N, K]^T (+ bias), fp32 accumulation on the CUDA cores. 64 x 64 tile, 4 x 4 per thread.
 template <typename TA, typename TC>
 __global__ void __launch_bounds__(256) gemm_simt_kernel(const TA* __restrict__ A, const TA* __restrict__ B,
@@ -299,19 +613,21 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const TA* __restrict__ A
 // ---------------------------------------------------------------------------------------------------------------
 // Paged attention over ragged queries on the CUDA cores: one warp per (token, query head), lanes across 32 keys for the
 // scores and across the value dims for the weighted sum. A query at position i sees key j <= i when window <= 0, or
-// i - j < window, or j < keep_first; bias[h][min(i - j, bias_len - 1)] is added to the scaled score.
+// i - j < window, or j < keep_first (chunk > 0: when i / chunk == j / chunk); bias[h][min(i - j, bias_len - 1)] is added to
+// the scaled score, softcap > 0 bounds it, exp(sink[h]) joins the denominator, sigmoid(gate) multiplies the result.
 struct PagedSimtParams {
   const int* cu_q;
   const int* seq_lens;
   const int* block_table;
-  long long q_stride, out_stride;
-  int max_blocks, B, Hq, Hk, D, Dv, block_size, window, keep_first, bias_len;
-  float scale;
-  const float* bias;
+  long long q_stride, out_stride, gate_stride;
+  int max_blocks, B, Hq, Hk, D, Dv, v_width, block_size, window, keep_first, chunk, bias_len;  // v_width: elements of a value row
+  float scale, softcap;
+  const float *bias, *sink;
+  const void* gate;  // [T, Hq * Dv] of the activation type, or null
 };
-constexpr int PS_WARPS = 4, PS_MAX_D = 512, PS_VREG = PS_MAX_D / 32;
+constexpr int PS_WARPS = 4, PS_MAX_D = 1024;
 
-template <typename T>
+template <typename T, int PS_VREG>
 __global__ void __launch_bounds__(PS_WARPS * 32)
 paged_attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ kc, const T* __restrict__ vc, T* __restrict__ out,
                        const PagedSimtParams p) {
@@ -334,11 +650,12 @@ paged_attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ kc, const 
   __syncwarp();
   const int* bt = p.block_table + (long long)b * p.max_blocks;
   const float* bias = p.bias ? p.bias + (long long)h * p.bias_len : nullptr;
-  float m = -INFINITY, l = 0.f, acc[PS_VREG];
+  float m = p.sink ? p.sink[h] : -INFINITY, l = p.sink ? 1.f : 0.f, acc[PS_VREG];
 #pragma unroll
   for (int i = 0; i < PS_VREG; ++i) acc[i] = 0.f;
   const int n = pos + 1;
-  const int w_lo = p.window > 0 ? max(0, n - p.window) : 0;      // first key of the window
+  // first key of the window or chunk
+  const int w_lo = p.window > 0 ? max(0, n - p.window) : p.chunk > 0 ? pos - pos % p.chunk : 0;
   const int keep = min(p.window > 0 ? p.keep_first : 0, w_lo);   // kept keys in front of it
   const int total = keep + n - w_lo;
   for (int c = 0; c < total; c += 32) {
@@ -354,6 +671,7 @@ paged_attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ kc, const 
       for (int d = 0; d < p.D; ++d) a = fmaf(q_s[warp][d], to_f<T>(kr[d]), a);
       s = a * p.scale;
       if (bias) s += bias[min(pos - key, p.bias_len - 1)];
+      if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
     }
     const float nm = fmaxf(m, warp_reduce_max(s));
     const float alpha = expf(m - nm);
@@ -365,7 +683,7 @@ paged_attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ kc, const 
     const int cnt = min(32, total - c);
     for (int j = 0; j < cnt; ++j) {
       const float wj = __shfl_sync(0xffffffffu, w, j);
-      const T* vr = vc + __shfl_sync(0xffffffffu, row, j) * p.Dv;
+      const T* vr = vc + __shfl_sync(0xffffffffu, row, j) * p.v_width;
 #pragma unroll
       for (int i = 0; i < PS_VREG; ++i)
         if (lane + 32 * i < p.Dv) acc[i] = fmaf(wj, to_f<T>(vr[lane + 32 * i]), acc[i]);
@@ -373,8 +691,13 @@ paged_attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ kc, const 
   }
   T* o = out + (long long)t * p.out_stride + (long long)h * p.Dv;
 #pragma unroll
-  for (int i = 0; i < PS_VREG; ++i)
-    if (lane + 32 * i < p.Dv) o[lane + 32 * i] = from_f<T>(acc[i] / l);
+  for (int i = 0; i < PS_VREG; ++i) {
+    const int d = lane + 32 * i;
+    if (d >= p.Dv) continue;
+    float x = acc[i] / l;
+    if (p.gate) x /= 1.f + expf(-to_f<T>(reinterpret_cast<const T*>(p.gate)[t * p.gate_stride + (long long)h * p.Dv + d]));
+    o[d] = from_f<T>(x);
+  }
 }
 
 }  // namespace vb
@@ -391,12 +714,13 @@ typedef __nv_bfloat16 bf16;
 
 static inline int row_threads(int n) { return n >= 2048 ? 256 : (n >= 1024 ? 128 : 64); }
 
-extern "C" int vb_embed_scaled(const long long* ids, const void* table, float* res, int T, int H, float scale, int f32,
-                               cudaStream_t stream) {
+extern "C" int vb_embed_scaled(const long long* ids, const void* table, float* res, void* y, int T, int H, float scale,
+                               int f32, cudaStream_t stream) {
   if (T <= 0) return 0;
   const dim3 g(T), b(row_threads(H));
-  if (f32) VB_DONE(vb_launch_pdl(embed_scaled_kernel<float>, g, b, 0, stream, 1, ids, (const float*)table, res, H, scale));
-  VB_DONE(vb_launch_pdl(embed_scaled_kernel<bf16>, g, b, 0, stream, 1, ids, (const bf16*)table, res, H, scale));
+  if (f32) VB_DONE(vb_launch_pdl(embed_scaled_kernel<float>, g, b, 0, stream, 1, ids, (const float*)table, res, (float*)y, H,
+                                scale));
+  VB_DONE(vb_launch_pdl(embed_scaled_kernel<bf16>, g, b, 0, stream, 1, ids, (const bf16*)table, res, (bf16*)y, H, scale));
 }
 
 extern "C" int vb_add_rmsnorm(const void* delta, long long delta_stride, float* res, const void* w, void* y, int T, int H,
@@ -418,19 +742,46 @@ extern "C" int vb_add_rmsnorm(const void* delta, long long delta_stride, float* 
                         (const bf16*)w, (bf16*)y, H, eps));
 }
 
-extern "C" int vb_clamped_glu(const void* gu, long long stride, void* y, int T, int F, float limit, float alpha, int f32,
-                              cudaStream_t stream) {
-  if (T <= 0 || F <= 0) return 0;
-  const long long total = (long long)T * F;
+template <typename T, typename Act>
+static int launch_glu(const void* gu, long long stride, void* y, int T_, int F, const Act& act, cudaStream_t stream) {
+  if (T_ <= 0 || F <= 0) return 0;
+  const long long total = (long long)T_ * F;
   long long blocks = (total / 8 + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   if (blocks < 1) blocks = 1;
-  const dim3 g((unsigned)blocks), b(256);
+  VB_DONE(vb_launch_pdl(glu_kernel<T, Act>, dim3((unsigned)blocks), dim3(256), 0, stream, 1, (const T*)gu, stride, (T*)y, total,
+                        F, act));
+}
+
+extern "C" int vb_clamped_glu(const void* gu, long long stride, void* y, int T, int F, float limit, float alpha, int f32,
+                              cudaStream_t stream) {
+  if (f32) return launch_glu<float>(gu, stride, y, T, F, ClampedGlu<float>{limit, alpha}, stream);
+  return launch_glu<bf16>(gu, stride, y, T, F, ClampedGlu<bf16>{limit, alpha}, stream);
+}
+
+extern "C" int vb_gelu_glu(const void* gu, long long stride, void* y, int T, int F, int f32, cudaStream_t stream) {
+  if (f32) return launch_glu<float>(gu, stride, y, T, F, GeluTanhGlu<float>{}, stream);
+  return launch_glu<bf16>(gu, stride, y, T, F, GeluTanhGlu<bf16>{}, stream);
+}
+
+// delta rows of delta_stride elements; fw null: y = the new residual in the activation type.
+extern "C" int vb_rmsnorm_add(const void* delta, long long delta_stride, float* res, const void* w, const void* fw, float fscale,
+                              void* y, int T, int H, float eps, int f32, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  const size_t smem = (size_t)H * 4;
+  if (smem > 160 * 1024) return -3;
+  const dim3 g(T), b(row_threads(H));
+  static bool attr = false;
+  if (!attr) {
+    VB_CUDA_CHECK(cudaFuncSetAttribute(rmsnorm_add_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
+    VB_CUDA_CHECK(cudaFuncSetAttribute(rmsnorm_add_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
+    attr = true;
+  }
   if (f32)
-    VB_DONE(vb_launch_pdl(clamped_glu_kernel<float>, g, b, 0, stream, 1, (const float*)gu, stride, (float*)y, total, F,
-                          limit, alpha));
-  VB_DONE(vb_launch_pdl(clamped_glu_kernel<bf16>, g, b, 0, stream, 1, (const bf16*)gu, stride, (bf16*)y, total, F, limit,
-                        alpha));
+    VB_DONE(vb_launch_pdl(rmsnorm_add_kernel<float>, g, b, smem, stream, 1, (const float*)delta, delta_stride, res,
+                          (const float*)w, (const float*)fw, fscale, (float*)y, H, eps));
+  VB_DONE(vb_launch_pdl(rmsnorm_add_kernel<bf16>, g, b, smem, stream, 1, (const bf16*)delta, delta_stride, res,
+                        (const bf16*)w, (const bf16*)fw, fscale, (bf16*)y, H, eps));
 }
 
 // qw / kw null: no norm (q untouched, k and v only written to the cache).
@@ -469,19 +820,99 @@ extern "C" int vb_gemm_simt(const void* A, const void* B, void* C, const void* b
                         (const bf16*)bias, M, N, K, lda, ldb, ldc));
 }
 
+// Caches [NB, Hk, block_size, D] and [NB, Hk, block_size, v_width] (the first Dv elements of a row are the value).
 extern "C" int vb_paged_attention_simt(const void* q, long long q_stride, const void* kc, const void* vc,
                                        const int* block_table, int max_blocks, const int* cu_q, const int* seq_lens,
-                                       int T, int B, int Hq, int Hk, int D, int Dv, int block_size, float scale,
-                                       int window, int keep_first, const float* bias, int bias_len, void* out,
+                                       int T, int B, int Hq, int Hk, int D, int Dv, int v_width, int block_size, float scale,
+                                       int window, int keep_first, int chunk, const float* bias, int bias_len,
+                                       float softcap, const float* sink, const void* gate, long long gate_stride, void* out,
                                        long long out_stride, int f32, cudaStream_t stream) {
   if (T <= 0 || B <= 0) return 0;
-  if (Hk <= 0 || Hq % Hk != 0 || D <= 0 || D > PS_MAX_D || Dv <= 0 || Dv > PS_MAX_D || (bias && bias_len <= 0)) return -3;
-  PagedSimtParams p{cu_q, seq_lens, block_table, q_stride, out_stride, max_blocks, B,          Hq,    Hk,  D,
-                    Dv,   block_size, window,    keep_first, bias_len, scale,      bias};
+  if (Hk <= 0 || Hq % Hk != 0 || D <= 0 || D > PS_MAX_D || Dv <= 0 || Dv > PS_MAX_D || v_width < Dv || (bias && bias_len <= 0))
+    return -3;
+  PagedSimtParams p{};
+  p.cu_q = cu_q; p.seq_lens = seq_lens; p.block_table = block_table;
+  p.q_stride = q_stride; p.out_stride = out_stride; p.gate_stride = gate_stride;
+  p.max_blocks = max_blocks; p.B = B; p.Hq = Hq; p.Hk = Hk; p.D = D; p.Dv = Dv; p.v_width = v_width; p.block_size = block_size;
+  p.window = window; p.keep_first = keep_first; p.chunk = chunk; p.bias_len = bias_len;
+  p.scale = scale; p.softcap = softcap; p.bias = bias; p.sink = sink; p.gate = gate;
   const dim3 g(T, (Hq + PS_WARPS - 1) / PS_WARPS), b(PS_WARPS * 32);
+#define VB_PSA(TT, V)                                                                                             \
+  VB_DONE(vb_launch_pdl(paged_attn_simt_kernel<TT, V>, g, b, 0, stream, 1, (const TT*)q, (const TT*)kc, (const TT*)vc, \
+                        (TT*)out, p))
+  if (f32) {
+    if (Dv <= 128) VB_PSA(float, 4);
+    VB_PSA(float, PS_MAX_D / 32);
+  }
+  if (Dv <= 128) VB_PSA(bf16, 4);
+  VB_PSA(bf16, PS_MAX_D / 32);
+#undef VB_PSA
+}
+
+// qw / kw null: no norm. freqs: n_rot fp32 angular frequencies (n_rot 0: no rotation).
+extern "C" int vb_head_norm_rope_kv_write(void* qkv, long long stride, const void* qw, const void* kw, const float* freqs,
+                                          int n_rot, int interleaved, float amp, const long long* positions,
+                                          const long long* slots, void* kc, void* vc, int T, int Hq, int Hk, int D, int Dv,
+                                          int block_size, float eps, int f32, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if ((qw == nullptr) != (kw == nullptr) || n_rot < 0 || n_rot > ROT_MAX || 2 * n_rot > D || D > PS_MAX_D) return -3;
+  const bool vec = (D & 7) == 0 && D <= 256 && (Dv & 7) == 0 && (stride & 7) == 0 && (interleaved || n_rot == 0) &&
+                   (reinterpret_cast<uintptr_t>(qkv) & 15) == 0;
+  int lanes = 1;
+  while (lanes * 8 < D) lanes *= 2;
+  const dim3 g(T), b(vec ? 256 : 128);
+  const size_t smem = vec ? 0 : 4 * (size_t)D * sizeof(float);
+#define VB_HNR(TT, V)                                                                                                  \
+  VB_DONE(vb_launch_pdl(head_norm_rope_kv_write_kernel<TT, V>, g, b, smem, stream, 1, (TT*)qkv, stride, (const TT*)qw, \
+                        (const TT*)kw, freqs, n_rot, interleaved, amp, positions, slots, (TT*)kc, (TT*)vc, Hq, Hk, D, Dv, \
+                        block_size, eps, lanes))
+  if (f32) {
+    if (vec) VB_HNR(float, true);
+    VB_HNR(float, false);
+  }
+  if (vec) VB_HNR(bf16, true);
+  VB_HNR(bf16, false);
+#undef VB_HNR
+}
+
+extern "C" int vb_latent_rope_write(void* proj, long long stride, const void* w, const float* freqs, float amp,
+                                    const long long* positions, const long long* slots, void* pages, int width, int T, int H,
+                                    int dim, int rot, int rank, float eps, int f32, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (rot < 0 || (rot & 1) || rot > 2 * ROT_MAX || rank <= 0 || width < rank + rot) return -3;
+  const bool vec = (rot & 15) == 0 && (dim & 7) == 0 && (rank & 7) == 0 && (width & 7) == 0 && (stride & 7) == 0 &&
+                   (reinterpret_cast<uintptr_t>(proj) & 15) == 0;
+  const dim3 g(T), b(128);
+#define VB_LRW(TT, V)                                                                                                  \
+  VB_DONE(vb_launch_pdl(latent_rope_write_kernel<TT, V>, g, b, 0, stream, 1, (TT*)proj, stride, (const TT*)w, freqs, amp, \
+                        positions, slots, (TT*)pages, width, H, dim, rot, rank, eps))
+  if (f32) {
+    if (vec) VB_LRW(float, true);
+    VB_LRW(float, false);
+  }
+  if (vec) VB_LRW(bf16, true);
+  VB_LRW(bf16, false);
+#undef VB_LRW
+}
+
+// row_bytes: bytes of a page row, a multiple of 16.
+extern "C" int vb_latent_gather(const void* pages, const int* block_table, int max_blocks, const int* ctx_cu, void* rows,
+                                int total, int B, int row_bytes, int block_size, cudaStream_t stream) {
+  if (total <= 0 || B <= 0) return 0;
+  if (row_bytes & 15) return -3;
+  VB_DONE(vb_launch_pdl(latent_gather_kernel, dim3((total + 7) / 8), dim3(256), 0, stream, 1, (const uint4*)pages, block_table,
+                        max_blocks, ctx_cu, (uint4*)rows, total, B, row_bytes / 16, block_size));
+}
+
+extern "C" int vb_head_gemm_simt(const void* a, long long a_t, long long a_h, const void* b, int b_mn, void* out, long long o_t,
+                                 long long o_h, const void* gate, long long gate_stride, int T, int H, int K, int N, int tail,
+                                 int width, int f32, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || H > 65535 || K <= 0 || width < N + tail) return -3;
+  const dim3 g(T, H, (width + 127) / 128), blk(128);
   if (f32)
-    VB_DONE(vb_launch_pdl(paged_attn_simt_kernel<float>, g, b, 0, stream, 1, (const float*)q, (const float*)kc,
-                          (const float*)vc, (float*)out, p));
-  VB_DONE(vb_launch_pdl(paged_attn_simt_kernel<bf16>, g, b, 0, stream, 1, (const bf16*)q, (const bf16*)kc,
-                        (const bf16*)vc, (bf16*)out, p));
+    VB_DONE(vb_launch_pdl(head_gemm_simt_kernel<float>, g, blk, 0, stream, 1, (const float*)a, a_t, a_h, (const float*)b, b_mn,
+                          (float*)out, o_t, o_h, (const float*)gate, gate_stride, K, N, tail, width));
+  VB_DONE(vb_launch_pdl(head_gemm_simt_kernel<bf16>, g, blk, 0, stream, 1, (const bf16*)a, a_t, a_h, (const bf16*)b, b_mn,
+                        (bf16*)out, o_t, o_h, (const bf16*)gate, gate_stride, K, N, tail, width));
 }

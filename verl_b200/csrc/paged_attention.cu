@@ -207,9 +207,10 @@ __global__ void decode_merge_kernel(const float* __restrict__ o_part, const floa
   out[(long long)b * out_stride + (long long)hq * D + d] = __float2bfloat16(l > 0.f ? o / l : 0.f);
 }
 
-// The same for any head size: one warp per (sequence, query head).
+// The same for any head size, times the sigmoid of a gate [B, Hq * D] (or null).
 __global__ void decode_merge_any_kernel(const float* __restrict__ o_part, const float* __restrict__ ml_part, int Hq, int D,
-                                        int num_splits, __nv_bfloat16* __restrict__ out, long long out_stride) {
+                                        int num_splits, __nv_bfloat16* __restrict__ out, long long out_stride,
+                                        const __nv_bfloat16* __restrict__ gate, long long gate_stride) {
   const int b = blockIdx.x, hq = blockIdx.y;
   const long long base = ((long long)b * Hq + hq) * num_splits;
   float m = -INFINITY, l = 0.f;
@@ -224,7 +225,9 @@ __global__ void decode_merge_any_kernel(const float* __restrict__ o_part, const 
       const float ms = ml_part[(base + s) * 2];
       if (ms != -INFINITY) o += o_part[(base + s) * D + d] * __expf(ms - m);
     }
-    out[(long long)b * out_stride + (long long)hq * D + d] = __float2bfloat16(l > 0.f ? o / l : 0.f);
+    o = l > 0.f ? o / l : 0.f;
+    if (gate) o = __fdividef(o, 1.f + __expf(-__bfloat162float(gate[(long long)b * gate_stride + (long long)hq * D + d])));
+    out[(long long)b * out_stride + (long long)hq * D + d] = __float2bfloat16(o);
   }
 }
 
@@ -275,9 +278,9 @@ int vb_decode_merge_128(const float* o_part, const float* ml_part, int B, int Hq
 }
 
 int vb_decode_merge(const float* o_part, const float* ml_part, int B, int Hq, int D, int num_splits, void* out,
-                    long long out_stride, cudaStream_t stream) {
-  decode_merge_any_kernel<<<dim3(B, Hq), D <= 64 ? 64 : 128, 0, stream>>>(o_part, ml_part, Hq, D, num_splits,
-                                                                          (__nv_bfloat16*)out, out_stride);
+                    long long out_stride, const void* gate, long long gate_stride, cudaStream_t stream) {
+  decode_merge_any_kernel<<<dim3(B, Hq), D <= 64 ? 64 : 128, 0, stream>>>(o_part, ml_part, Hq, D, num_splits, (__nv_bfloat16*)out,
+                                                                          out_stride, (const __nv_bfloat16*)gate, gate_stride);
   return (int)cudaGetLastError();
 }
 

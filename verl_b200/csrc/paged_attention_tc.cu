@@ -17,8 +17,9 @@
 //   warp 5     : TMEM allocation + single-thread tcgen05.mma issue
 //
 // The EXT variant serves layer-list decoders: head sizes up to 128 with separate key and value sizes (TMA fills the
-// missing columns with zeros), a sliding window with kept first keys (only the chunks in sight are visited), a
-// per-distance bias, and weights that stay close to fp32: with up to 8 query heads per KV head, rows G .. 2G-1 of the
+// missing columns with zeros), a sliding window with kept first keys or chunks of the sequence (only the key blocks in sight
+// are visited), a per-distance bias or a soft cap of the scores, a sink in the denominator, an output gate, and weights that
+// stay close to fp32: with up to 8 query heads per KV head, rows G .. 2G-1 of the
 // P operand hold the remainders that rounding the weights to bf16 leaves, and their products are added.
 //
 // V needs no transpose: [keys, dims] with dims contiguous is exactly an "MN-major" A operand.
@@ -59,9 +60,18 @@ struct DecodeTcParams {
   float* ml_part;
   int* status;
   // EXT only
-  int D, Dv, window, keep_first, bias_len;
+  int D, Dv, window, keep_first, chunk, bias_len;
   const float* bias;  // [Hq, bias_len] or null
+  float softcap;
+  const float* sink;          // [Hq] or null
+  const __nv_bfloat16* gate;  // [B, Hq * Dv] or null
+  long long gate_stride;
 };
+
+// First key that the query at position seq_len - 1 sees, kept ones apart.
+__device__ __forceinline__ int tc_first_key(const DecodeTcParams& p, int seq_len) {
+  return p.window > 0 ? max(seq_len - p.window, 0) : p.chunk > 0 ? (seq_len - 1) / p.chunk * p.chunk : 0;
+}
 
 // Chunks a decode query at position seq_len - 1 visits: [0, keep) and [win, ...); without a window all of them.
 struct TcRange {
@@ -74,9 +84,9 @@ __device__ __forceinline__ TcRange tc_range(const DecodeTcParams& p, int seq_len
   const int chunks = (seq_len + TC_CHUNK - 1) / TC_CHUNK;
   r.keep = 0;
   r.win = 0;
-  if (EXT && p.window > 0) {
-    r.keep = min((p.keep_first + TC_CHUNK - 1) / TC_CHUNK, chunks);
-    r.win = max(max(seq_len - p.window, 0) / TC_CHUNK, r.keep);
+  if (EXT && (p.window > 0 || p.chunk > 0)) {
+    r.keep = p.window > 0 ? min((p.keep_first + TC_CHUNK - 1) / TC_CHUNK, chunks) : 0;
+    r.win = max(tc_first_key(p, seq_len) / TC_CHUNK, r.keep);
   }
   r.total = r.keep + max(chunks - r.win, 0);
   return r;
@@ -639,7 +649,13 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
         m_run[g] = -INFINITY;
         l_run[g] = 0.f;
         o_acc[g] = 0.f;
+        // the sink is a key without a value: it counts once, in the first split
+        if (EXT && p.sink != nullptr && g < G && it.split == 0) {
+          m_run[g] = p.sink[it.h * G + g];
+          l_run[g] = 1.f;
+        }
       }
+      const int first = EXT ? tc_first_key(p, it.seq_len) : 0;
       float alpha_cur[TC_NH], alpha_nxt[TC_NH];
       const uint32_t cg0 = cg;
       auto softmax_chunk = [&](int c, float (&alpha)[TC_NH]) {
@@ -661,7 +677,7 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
         }
         const int key = it.range.at(it.c_begin + c) * TC_CHUNK + tid;
         const int dist = it.seq_len - 1 - key;
-        const bool valid = dist >= 0 && (!EXT || p.window <= 0 || dist < p.window || key < p.keep_first);
+        const bool valid = dist >= 0 && (!EXT || key >= first || (p.window > 0 && key < p.keep_first));
         const float* brow = EXT && p.bias != nullptr
                                 ? p.bias + (long long)it.h * G * p.bias_len + max(min(dist, p.bias_len - 1), 0)
                                 : nullptr;
@@ -669,6 +685,9 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
 #pragma unroll
         for (int g = 0; g < TC_NH; ++g) {
           sc[g] = valid ? __uint_as_float(sr[g]) * p.scale : -INFINITY;
+          // cap tanh(s / cap) = cap - 2 cap / (1 + e^(2 s / cap))
+          if (EXT && p.softcap > 0.f && g < G && valid)
+            sc[g] = p.softcap - __fdividef(2.f * p.softcap, 1.f + __expf(sc[g] * (2.f / p.softcap)));
           if (EXT && brow != nullptr && g < G) sc[g] += __ldg(brow + g * p.bias_len);
           if (g < G) {
             const float wm = warp_reduce_max(sc[g]);
@@ -746,8 +765,10 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
           if (g < G) {
             const int hq = it.h * G + g;
             if (p.num_splits == 1) {
-              p.out[(long long)it.b * p.out_stride + (long long)hq * Dv + d] =
-                  __float2bfloat16(l_run[g] > 0.f ? o_acc[g] / l_run[g] : 0.f);
+              float x = l_run[g] > 0.f ? o_acc[g] / l_run[g] : 0.f;
+              if (EXT && p.gate != nullptr)
+                x = __fdividef(x, 1.f + __expf(-__bfloat162float(p.gate[(long long)it.b * p.gate_stride + hq * Dv + d])));
+              p.out[(long long)it.b * p.out_stride + (long long)hq * Dv + d] = __float2bfloat16(x);
             } else {
               const long long base = ((long long)it.b * p.Hq + hq) * p.num_splits + it.split;
               p.o_part[base * Dv + d] = o_acc[g];
@@ -844,7 +865,7 @@ extern "C" int vb_paged_decode_tc(const void* q, long long q_stride, const void*
 }
 
 int vb_decode_merge(const float* o_part, const float* ml_part, int B, int Hq, int D, int num_splits, void* out,
-                    long long out_stride, cudaStream_t stream);
+                    long long out_stride, const void* gate, long long gate_stride, cudaStream_t stream);
 
 // Returns 1 if vb_paged_decode_window supports this configuration.
 extern "C" int vb_paged_decode_window_supported(int Hq, int Hk, int D, int Dv, int block_size) {
@@ -854,17 +875,21 @@ extern "C" int vb_paged_decode_window_supported(int Hq, int Hk, int D, int Dv, i
 
 // One query token per sequence over caches [num_blocks, Hk, block_size, D | Dv] bf16, at position seq_lens[b] - 1:
 //   window > 0: key j is visible when seq_len - 1 - j < window or j < keep_first (0: every key)
+//   chunk > 0: key j is visible when j / chunk == (seq_len - 1) / chunk (not together with a window)
 //   bias [Hq, bias_len] fp32 or null: bias[h][min(seq_len - 1 - j, bias_len - 1)] is added to the scaled score
+//   softcap > 0 (without bias): scores become softcap * tanh(score / softcap)
+//   sink [Hq] fp32 or null: exp(sink[h]) joins the denominator; gate [B, Hq * Dv] or null: its sigmoid multiplies the result
 // work: fp32 scratch of B * Hq * num_splits * (Dv + 2) floats (unused when num_splits == 1).
 extern "C" int vb_paged_decode_window(const void* q, long long q_stride, const void* kc, const void* vc, int num_blocks,
                                       const int* block_table, int max_blocks, const int* seq_lens, int B, int Hq, int Hk,
                                       int D, int Dv, int block_size, float scale, int window, int keep_first,
-                                      const float* bias, int bias_len, int num_splits, void* out, long long out_stride,
-                                      float* work, int* status, cudaStream_t stream) {
+                                      int chunk, const float* bias, int bias_len, float softcap, const float* sink,
+                                      const void* gate, long long gate_stride, int num_splits, void* out,
+                                      long long out_stride, float* work, int* status, cudaStream_t stream) {
   if (B <= 0) return 0;
   if (!vb_paged_decode_window_supported(Hq, Hk, D, Dv, block_size) || (q_stride & 7) != 0 ||
       (reinterpret_cast<uintptr_t>(q) & 15) != 0 || num_splits < 1 || (num_splits > 1 && work == nullptr) ||
-      (bias != nullptr && bias_len <= 0))
+      (bias != nullptr && bias_len <= 0) || (window > 0 && chunk > 0) || (softcap > 0.f && bias != nullptr))
     return -3;
   CUtensorMap tmK, tmV;
   const uint64_t rows = (uint64_t)num_blocks * Hk * block_size;
@@ -893,11 +918,14 @@ extern "C" int vb_paged_decode_window(const void* q, long long q_stride, const v
   p.ml_part = work ? work + (long long)B * Hq * num_splits * Dv : nullptr;
   p.status = status;
   p.D = D; p.Dv = Dv; p.window = window; p.keep_first = keep_first; p.bias_len = bias_len; p.bias = bias;
+  p.chunk = chunk; p.softcap = softcap; p.sink = sink;
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
+  p.gate_stride = gate_stride;
   const int items = B * Hk * num_splits, slots = 2 * vb_num_sms();
   rc = (int)vb_launch_pdl(paged_decode_tc_persist_kernel<true>, dim3(items < slots ? items : slots), dim3(TC_THREADS),
                           TCP_SMEM, stream, 1, tmK, tmV, p, items);
   vb_count_launch(num_splits > 1 ? 2 : 1);
   if (rc == 0) rc = (int)cudaGetLastError();
   if (rc || num_splits == 1) return rc;
-  return vb_decode_merge(p.o_part, p.ml_part, B, Hq, Dv, num_splits, out, out_stride, stream);
+  return vb_decode_merge(p.o_part, p.ml_part, B, Hq, Dv, num_splits, out, out_stride, gate, gate_stride, stream);
 }

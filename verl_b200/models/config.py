@@ -10,7 +10,7 @@ from dataclasses import asdict, dataclass, field
 from pathlib import Path
 from typing import Any
 
-from .layer_specs import AttentionSpec, DeltaSpec, GluSpec, LayerSpec
+from .layer_specs import (DESIGNS, AttentionSpec, DeltaSpec, Design, GluSpec, LatentSpec, LayerSpec, RotarySpec)
 
 _ARCH_TO_TYPE = {
     "LlamaForCausalLM": "llama",
@@ -32,7 +32,7 @@ _TYPE_TO_ARCH = {"llama": "LlamaForCausalLM", "qwen2": "Qwen2ForCausalLM", "qwen
                  "qwen2_5_vl": "Qwen2_5_VLForConditionalGeneration", "apertus": "ApertusForCausalLM",
                  "qwen3_vl": "Qwen3VLForConditionalGeneration", "qwen3_vl_moe": "Qwen3VLMoeForConditionalGeneration"}
 # designs whose config.json lists its layers one by one (``architecture`` instead of ``architectures``)
-_LAYER_LIST_ARCHS = {"Fuganex": "fuganex"}
+_LAYER_LIST_ARCHS = {"Fuganex": "fuganex", "Padodra": "padodra"}
 _VL_TYPES = ("qwen2_vl", "qwen2_5_vl", "qwen3_vl", "qwen3_vl_moe")
 
 
@@ -68,6 +68,7 @@ class ModelConfig:
     # layer-list designs: one LayerSpec per layer (empty: all layers alike, described by the fields above)
     layer_specs: tuple = ()
     embedding_scale: float = 1.0
+    logit_scale: float = 1.0
     extra: dict = field(default_factory=dict)
 
     def __post_init__(self):
@@ -91,6 +92,11 @@ class ModelConfig:
     @property
     def is_layer_list(self) -> bool:
         return bool(self.layer_specs)
+
+    @property
+    def design(self) -> Design:
+        """What the layer-list design fixes for all its models."""
+        return DESIGNS[self.model_type]
 
     @property
     def has_recurrent_state(self) -> bool:
@@ -206,12 +212,14 @@ class ModelConfig:
 
     @classmethod
     def _from_layer_list(cls, d: dict[str, Any]) -> "ModelConfig":
-        specs = tuple(LayerSpec.from_dict(x) for x in d["layers"])
+        model_type = _LAYER_LIST_ARCHS[d["architecture"]]
+        design = DESIGNS[model_type]
+        specs = tuple(LayerSpec.from_dict(x, design) for x in d["layers"])
         att = [s.mixer for s in specs if s.kind == "attention"]
         kw = {k: int(d[k]) for k in ("bos_token_id", "eos_token_id", "pad_token_id") if d.get(k) is not None}
         kw.setdefault("eos_token_id", None)
-        known = ("architecture", "vocab", "width", "layers", "norm", "embedding", *kw)
-        return cls(model_type=_LAYER_LIST_ARCHS[d["architecture"]], vocab_size=int(d["vocab"]), hidden_size=int(d["width"]),
+        known = ("architecture", "vocab", "width", "layers", "norm", "embedding", "logit_scale", *kw)
+        return cls(model_type=model_type, logit_scale=float(d["logit_scale"]) if design.logit_scale else 1.0, vocab_size=int(d["vocab"]), hidden_size=int(d["width"]),
                    intermediate_size=max([s.mlp.ff for s in specs if s.mlp] or [0]),
                    num_attention_heads=max([a.heads for a in att] or [1]),
                    num_key_value_heads=max([a.kv_heads for a in att] or [1]), head_dim=max([a.dim for a in att] or [1]),
@@ -223,6 +231,8 @@ class ModelConfig:
         d = {"architecture": arch, "vocab": self.vocab_size, "width": self.hidden_size,
              "layers": [s.to_dict() for s in self.layer_specs], "norm": {"eps": self.rms_norm_eps},
              "embedding": {"scale": self.embedding_scale}, **self.extra}
+        if self.design.logit_scale:
+            d["logit_scale"] = self.logit_scale
         for k in ("bos_token_id", "eos_token_id", "pad_token_id"):
             if getattr(self, k) is not None:
                 d[k] = getattr(self, k)
@@ -239,7 +249,7 @@ class ModelConfig:
         if self.is_layer_list:
             return self._to_layer_list()
         d = asdict(self)
-        del d["layer_specs"], d["embedding_scale"]
+        del d["layer_specs"], d["embedding_scale"], d["logit_scale"]
         extra = d.pop("extra")
         if self.model_type in _VL_TYPES:
             moe_keys = () if self.is_moe else ("num_experts", "num_experts_per_tok", "moe_intermediate_size", "norm_topk_prob",
@@ -284,6 +294,19 @@ def _fuganex_specs(groups: int, heads: int, kv_heads: int, dim: int, window: int
     delta = LayerSpec(DeltaSpec(d_heads, d_kv_heads, d_dim, d_dim, 4), mlp)
     att = LayerSpec(AttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, window, keep_first, 128.0, 32), mlp)
     return (delta, delta, att) * groups
+
+
+def _padodra_specs(groups: int, heads: int, kv_heads: int, dim: int, chunk: int, ff: int, latent: tuple) -> tuple:
+    """``groups`` x (two chunked attention layers, one latent attention layer), a feed-forward after each. ``latent``: heads,
+    unrotated and rotated head size, value size, rank."""
+    mlp = GluSpec(ff, act="gelu_tanh")
+    rot = RotarySpec(dim, 500000.0, True, (("factor", 8.0), ("high", 4.0), ("low", 1.0), ("original", 8192)))
+    att = AttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, qk_norm="head", rotary=rot, chunk=chunk, softcap=30.0,
+                        sink=True, gate=True)
+    h, d, r, v, rank = latent
+    yarn = RotarySpec(r, 10000.0, False, (("factor", 40.0), ("fast", 32.0), ("original", 4096), ("slow", 1.0)))
+    lat = LatentSpec(h, d, r, v, rank, (d + r) ** -0.5, yarn, True)
+    return (LayerSpec(att, mlp), LayerSpec(att, mlp), LayerSpec(lat, mlp)) * groups
 
 
 # Named architectures used by the benchmarks and tests (random-init, no download needed).
@@ -390,6 +413,13 @@ PRESETS: dict[str, dict] = {
     "fuganex-8b": dict(model_type="fuganex", vocab_size=128256, hidden_size=4096, eos_token_id=None, rms_norm_eps=1e-5,
                        num_attention_heads=32, num_key_value_heads=8, head_dim=128, intermediate_size=14336,
                        layer_specs=_fuganex_specs(10, 32, 8, 128, 1024, 4, 14336, 32, 16, 128)),
+    "tiny-padodra": dict(model_type="padodra", vocab_size=704, hidden_size=160, eos_token_id=2, rms_norm_eps=1e-6,
+                         embedding_scale=4.0, logit_scale=0.5,
+                         layer_specs=_padodra_specs(1, 4, 2, 48, 56, 288, (4, 32, 16, 40, 56))),
+    # real-model sizes for benchmarks: the widths of llama-3-8b, chunks of 2048, a rank of 512 in every third layer
+    "padodra-8b": dict(model_type="padodra", vocab_size=128256, hidden_size=4096, eos_token_id=None, rms_norm_eps=1e-5,
+                       num_attention_heads=32, num_key_value_heads=8, head_dim=128, intermediate_size=14336,
+                       layer_specs=_padodra_specs(10, 32, 8, 128, 2048, 14336, (32, 128, 64, 128, 512))),
     "llama-3-8b": dict(model_type="llama", vocab_size=128256, hidden_size=4096, intermediate_size=14336,
                        num_hidden_layers=32, num_attention_heads=32, num_key_value_heads=8, rope_theta=5e5,
                        rms_norm_eps=1e-5, eos_token_id=128001),

@@ -211,14 +211,19 @@ _LIST_TOP = {"embed_tokens.weight": "embed", "norm.weight": "final.norm", "lm_he
 _LIST_PLAIN = {"norm1.weight": "norm1", "norm2.weight": "norm2", "mlp.down_proj.weight": "mlp.down",
                "mixer.o_proj.weight": "mix.o", "mixer.q_norm.weight": "mix.q.norm", "mixer.k_norm.weight": "mix.k.norm",
                "mixer.rel": "mix.rel", "mixer.A_log": "mix.A_log", "mixer.dt_bias": "mix.dt_bias",
-               "mixer.norm.weight": "mix.norm"}
+               "mixer.norm.weight": "mix.norm", "mixer.sink": "mix.sink", "mixer.kv_norm.weight": "mix.dkv.norm"}
 
 
 def _list_fused(spec) -> dict[str, list[tuple[str, int]]]:
     """Native fused matrices of a layer: name -> [(checkpoint name, rows), ...] in row order."""
     m = spec.mixer
     if spec.kind == "attention":
-        out = {"mixer.qkv_proj.weight": [("mix.q", m.q_size), ("mix.k", m.k_size), ("mix.v", m.v_size)]}
+        out = {"mixer.qkv_proj.weight": [("mix.q", m.q_size), ("mix.k", m.k_size), ("mix.v", m.v_size)]
+               + ([("mix.g", m.out_size)] if m.gate else [])}
+    elif spec.kind == "latent_attention":
+        out = {"mixer.in_proj.weight": [("mix.q", m.q_size), ("mix.dkv", m.latent_size)]
+               + ([("mix.g", m.out_size)] if m.gate else []),
+               "mixer.kv_up_proj.weight": [("mix.uk", m.heads * m.dim), ("mix.uv", m.heads * m.vdim)]}
     else:
         qk, v = m.kv_heads * m.dim, m.heads * m.vdim
         out = {"mixer.in_proj.weight": [("mix.q", qk), ("mix.k", qk), ("mix.v", v), ("mix.g", v), ("mix.b", m.heads),

@@ -1,11 +1,17 @@
 """Decoders described layer by layer (``ModelConfig.layer_specs``): every layer has its own mixer, softmax attention over
-the paged KV cache or a gated delta rule with per-sequence state, and an optional clamped-GLU feed-forward.
+the paged KV cache, latent attention over pages of latents or a gated delta rule with per-sequence state, and an optional
+gated feed-forward.
 
 Served by the rollout engine like the homogeneous stacks of :mod:`.transformer`; there is no training path. The residual
-stream is fp32 and every norm is fused with the residual add in front of it:
+stream is fp32 and every norm is fused with the residual add beside it. Designs that norm what a sublayer reads:
 
     embedding * scale -> [ add + norm1 -> fused input projection -> mixer -> output projection
-                           -> add + norm2 -> gate|up -> clamped GLU -> down ] ... -> add + final norm -> head
+                           -> add + norm2 -> gate|up -> GLU -> down ] ... -> add + final norm -> head
+
+Designs that norm what a sublayer puts out (the last norm + add also computes the final norm):
+
+    embedding * scale -> [ fused input projection -> mixer -> output projection -> norm1 + add
+                           -> gate|up -> GLU -> down -> norm2 + add ] ... -> head
 """
 
 from __future__ import annotations
@@ -18,8 +24,13 @@ import torch.nn as nn
 
 from .. import ops
 from .config import ModelConfig
-from .layer_specs import AttentionSpec, DeltaSpec, GluSpec, LayerSpec, distance_buckets
+from .layer_specs import AttentionSpec, DeltaSpec, GluSpec, LatentSpec, LayerSpec, distance_buckets
 from .transformer import Linear, RMSNormWeight
+
+
+# Latent attention: portions of up to LATENT_SHORT tokens attend in the latent space (more arithmetic per key, no expansion);
+# longer ones expand keys and values of up to LATENT_GROUP context tokens at a time (or of one longer sequence).
+LATENT_SHORT, LATENT_GROUP = 32, 1 << 17
 
 
 def pad8(n: int) -> int:
@@ -28,8 +39,21 @@ def pad8(n: int) -> int:
 
 
 @dataclass
+class LatentPlan:
+    """How latent-attention layers run a step. The leading ``short_seqs`` sequences (``short_rows`` token rows, few new tokens
+    each) attend in the latent space, straight from the pages. The others get the keys and values of their whole context
+    expanded, group by group: (first sequence, end, ctx_cu = int32 [n + 1] boundaries of the contexts, their total, longest
+    portion)."""
+
+    short_seqs: int
+    short_rows: int
+    groups: tuple = ()
+
+
+@dataclass
 class RaggedBatch:
-    """One step: the new tokens of B sequences, described for the cache and state (all int32 except ``slots`` int64)."""
+    """One step: the new tokens of B sequences, described for the cache and state (all int32 except ``slots`` and
+    ``positions``, int64)."""
 
     cu_q: torch.Tensor         # [B + 1] boundaries of the new tokens
     max_q: int
@@ -38,11 +62,13 @@ class RaggedBatch:
     block_table: torch.Tensor  # [B, max_blocks]
     state_slots: torch.Tensor  # [B] recurrent-state slot (< 0: padding)
     max_ctx: int = 0           # longest sequence a replay of this step may see
-    work: dict = field(default_factory=dict)  # scratch owned by the caller (CUDA graphs)
+    positions: Optional[torch.Tensor] = None  # [T] position of each token
+    latent: Optional[LatentPlan] = None
 
 
 class StateCache:
-    """Cache of a layer-list model: K / V pages per attention layer, fp32 state and convolution ring per delta layer."""
+    """Cache of a layer-list model: K / V pages per attention layer, pages of latents and rotated keys per latent-attention
+    layer, fp32 state and convolution ring per delta layer."""
 
     def __init__(self, cfg: ModelConfig, num_blocks: int, block_size: int, num_slots: int, dtype, device):
         self.layers: list[tuple] = []
@@ -51,14 +77,16 @@ class StateCache:
             if spec.kind == "attention":
                 self.layers.append(tuple(torch.zeros((num_blocks, m.kv_heads, block_size, d), dtype=dtype, device=device)
                                          for d in (m.dim, m.vdim)))
+            elif spec.kind == "latent_attention":
+                self.layers.append((torch.zeros((num_blocks, block_size, pad8(m.latent_size)), dtype=dtype, device=device),))
             else:
                 self.layers.append((torch.zeros((num_slots, m.conv, m.channels), dtype=dtype, device=device),
                                     torch.zeros((num_slots, m.heads, m.vdim, m.dim), dtype=torch.float32, device=device)))
 
     @staticmethod
     def page_bytes(cfg: ModelConfig, block_size: int, itemsize: int) -> int:
-        return sum(s.mixer.kv_heads * (s.mixer.dim + s.mixer.vdim) for s in cfg.layer_specs
-                   if s.kind == "attention") * block_size * itemsize
+        per_token = {"attention": lambda m: m.kv_heads * (m.dim + m.vdim), "latent_attention": lambda m: pad8(m.latent_size)}
+        return sum(per_token[s.kind](s.mixer) for s in cfg.layer_specs if s.kind in per_token) * block_size * itemsize
 
     @staticmethod
     def slot_bytes(cfg: ModelConfig, itemsize: int) -> int:
@@ -66,15 +94,23 @@ class StateCache:
                    for m in (s.mixer for s in cfg.layer_specs if s.kind == "delta"))
 
 
+def rotary_frequencies(module: nn.Module, spec, device) -> None:
+    """The rotation's frequencies as the module's fp32 buffer ``rot_freqs``."""
+    module.register_buffer("rot_freqs", torch.tensor(spec.frequencies(), dtype=torch.float32, device=device), persistent=False)
+
+
 class AttentionMixer(nn.Module):
     def __init__(self, cfg: ModelConfig, spec: AttentionSpec, dtype, device):
         super().__init__()
         self.spec, self.eps = spec, cfg.rms_norm_eps
-        self.qkv_proj = Linear(cfg.hidden_size, pad8(spec.q_size + spec.k_size + spec.v_size), False, dtype, device)
+        self.qkv_proj = Linear(cfg.hidden_size, pad8(spec.proj_size), False, dtype, device)
         self.o_proj = Linear(spec.out_size, cfg.hidden_size, False, dtype, device)
         if spec.qk_norm:
-            self.q_norm = RMSNormWeight(spec.q_size, dtype, device)
-            self.k_norm = RMSNormWeight(spec.k_size, dtype, device)
+            self.q_norm, self.k_norm = (RMSNormWeight(n, dtype, device) for n in spec.norm_sizes)
+        if spec.sink:
+            self.sink = nn.Parameter(torch.zeros(spec.heads, dtype=torch.float32, device=device))
+        if spec.rotary is not None:
+            rotary_frequencies(self, spec.rotary, device)
         if spec.bias_rows:
             self.rel = nn.Parameter(torch.zeros(spec.bias_rows, spec.heads, dtype=torch.float32, device=device))
             buckets = torch.tensor(distance_buckets(spec.bias_rows, spec.bias_max), dtype=torch.long, device=device)
@@ -92,11 +128,61 @@ class AttentionMixer(nn.Module):
         s = self.spec
         norms = (self.q_norm.weight, self.k_norm.weight) if s.qk_norm else (None, None)
         qkv = mm(x, self.qkv_proj.weight)
-        q = ops.qk_norm_kv_write(qkv, *norms, batch.slots, cache[0], cache[1], s.heads, self.eps)
+        if s.qk_norm == "projection" and s.rotary is None:
+            q = ops.qk_norm_kv_write(qkv, *norms, batch.slots, cache[0], cache[1], s.heads, self.eps)
+        elif s.qk_norm != "projection":
+            q = ops.head_norm_rope_kv_write(qkv, *norms, self.rot_freqs if s.rotary else None, batch.positions, batch.slots,
+                                            cache[0], cache[1], s.heads, self.eps,
+                                            interleaved=s.rotary is not None and s.rotary.interleaved,
+                                            amplitude=s.rotary.amplitude if s.rotary else 1.0)
+        else:
+            raise NotImplementedError("rotary positions after a norm over the whole projection")
+        lo = s.q_size + s.k_size + s.v_size
         o = ops.paged_attention(q, cache[0], cache[1], batch.block_table, batch.cu_q, batch.seq_lens, batch.max_q,
                                 scale=s.scale, window=s.window, keep_first=s.keep_first,
-                                bias=self.bias if s.bias_rows else None, max_ctx=batch.max_ctx)
+                                bias=self.bias if s.bias_rows else None, max_ctx=batch.max_ctx, chunk=s.chunk,
+                                softcap=s.softcap, sink=self.sink if s.sink else None,
+                                gate=qkv[:, lo : lo + s.out_size] if s.gate else None)
         return mm(o, self.o_proj.weight)
+
+
+class LatentMixer(nn.Module):
+    def __init__(self, cfg: ModelConfig, spec: LatentSpec, dtype, device):
+        super().__init__()
+        self.spec, self.eps = spec, cfg.rms_norm_eps
+        self.in_proj = Linear(cfg.hidden_size, pad8(spec.proj_size), False, dtype, device)
+        self.kv_norm = RMSNormWeight(spec.kv_rank, dtype, device)
+        self.kv_up_proj = Linear(spec.kv_rank, pad8(spec.up_size), False, dtype, device)
+        self.o_proj = Linear(spec.out_size, cfg.hidden_size, False, dtype, device)
+        rotary_frequencies(self, spec.rotary, device)
+
+    def refresh(self):
+        pass
+
+    def forward(self, x, batch: RaggedBatch, cache, mm: Callable):
+        s, pages, plan = self.spec, cache[0], batch.latent
+        T = x.shape[0]
+        proj = mm(x, self.in_proj.weight)
+        ops.latent_rope_write(proj, self.kv_norm.weight, self.rot_freqs, batch.positions, batch.slots, pages, s.heads, s.dim,
+                              s.rot_dim, s.kv_rank, self.eps, amplitude=s.rotary.amplitude)
+        q = proj[:, : s.q_size].view(T, s.heads, s.dim + s.rot_dim)
+        lo = s.q_size + s.latent_size
+        gate = proj[:, lo : lo + s.out_size] if s.gate else None
+        out = torch.empty((T, s.out_size), dtype=x.dtype, device=x.device)
+        up = self.kv_up_proj.weight
+        uk = up[: s.heads * s.dim].view(s.heads, s.dim, s.kv_rank)
+        uv = up[s.heads * s.dim : s.up_size].view(s.heads, s.vdim, s.kv_rank)
+        n, B = plan.short_rows, plan.short_seqs
+        if n:  # scores and weighted sums over the latents themselves: W_uk moves to the queries, W_uv behind the sum
+            lat = ops.latent_attention(ops.latent_queries(q[:n], uk), pages, batch.block_table[:B], batch.cu_q[: B + 1],
+                                       batch.seq_lens[:B], s.kv_rank, scale=s.scale, max_ctx=batch.max_ctx)
+            ops.latent_values(lat, uv, None if gate is None else gate[:n], out[:n])
+        for b0, b1, ctx_cu, total, max_q in plan.groups:
+            rows = ops.latent_gather(pages, batch.block_table[b0:b1], ctx_cu, total)
+            kv = mm(rows[:, : s.kv_rank], up)
+            ops.latent_prefill(q, rows[:, s.kv_rank : s.latent_size], kv, batch.cu_q[b0 : b1 + 1], ctx_cu, max_q, s.dim,
+                               s.vdim, scale=s.scale, gate=gate, out=out)
+        return mm(out, self.o_proj.weight)
 
 
 class DeltaMixer(nn.Module):
@@ -128,7 +214,7 @@ class DeltaMixer(nn.Module):
         return mm(o, self.o_proj.weight)
 
 
-class ClampedGLU(nn.Module):
+class GatedMLP(nn.Module):
     def __init__(self, cfg: ModelConfig, spec: GluSpec, dtype, device):
         super().__init__()
         self.spec = spec
@@ -137,18 +223,22 @@ class ClampedGLU(nn.Module):
 
     def forward(self, x, mm: Callable):
         s = self.spec
-        return mm(ops.clamped_glu(mm(x, self.gate_up_proj.weight), s.ff, s.limit, s.alpha), self.down_proj.weight)
+        gu = mm(x, self.gate_up_proj.weight)
+        h = ops.gelu_tanh_glu(gu, s.ff) if s.act == "gelu_tanh" else ops.clamped_glu(gu, s.ff, s.limit, s.alpha)
+        return mm(h, self.down_proj.weight)
+
+
+_MIXERS = {"attention": AttentionMixer, "latent_attention": LatentMixer, "delta": DeltaMixer}
 
 
 class HybridLayer(nn.Module):
     def __init__(self, cfg: ModelConfig, spec: LayerSpec, dtype, device):
         super().__init__()
         self.norm1 = RMSNormWeight(cfg.hidden_size, dtype, device)
-        mixer = AttentionMixer if spec.kind == "attention" else DeltaMixer
-        self.mixer = mixer(cfg, spec.mixer, dtype, device)
+        self.mixer = _MIXERS[spec.kind](cfg, spec.mixer, dtype, device)
         if spec.mlp is not None:
             self.norm2 = RMSNormWeight(cfg.hidden_size, dtype, device)
-            self.mlp = ClampedGLU(cfg, spec.mlp, dtype, device)
+            self.mlp = GatedMLP(cfg, spec.mlp, dtype, device)
         else:
             self.norm2 = self.mlp = None
 
@@ -161,6 +251,13 @@ class HybridLM(nn.Module):
         self.layers = nn.ModuleList([HybridLayer(cfg, s, dtype, device) for s in cfg.layer_specs])
         self.norm = RMSNormWeight(cfg.hidden_size, dtype, device)
         self.lm_head = Linear(cfg.hidden_size, cfg.vocab_size, False, dtype, device)
+        # portions up to this many tokens run latent attention in the latent space; sizes without an expanded form: all
+        self.latent_short = LATENT_SHORT
+        for s in cfg.layer_specs:
+            m = s.mixer
+            if s.kind == "latent_attention" and not ops.latent_prefill_supported(m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank,
+                                                                                 dtype, device):
+                self.latent_short = 1 << 30
 
     def init_weights(self, seed: int = 0):
         dev = self.embed_tokens.weight.device
@@ -175,6 +272,9 @@ class HybridLM(nn.Module):
             elif isinstance(m, AttentionMixer) and m.spec.bias_rows:
                 with torch.no_grad():
                     m.rel.copy_(torch.empty(m.rel.shape, device=dev).normal_(0.0, 0.5, generator=gen))
+            if isinstance(m, AttentionMixer) and m.spec.sink:
+                with torch.no_grad():
+                    m.sink.copy_(torch.empty(m.sink.shape, device=dev).normal_(0.0, 1.0, generator=gen))
         self.refresh()
         return self
 
@@ -188,8 +288,35 @@ class HybridLM(nn.Module):
         return self.lm_head.weight
 
     def projection_weights(self) -> list[torch.Tensor]:
-        """Matrices of the layers (what weight quantisation applies to)."""
-        return [m.weight for layer in self.layers for m in layer.modules() if isinstance(m, Linear)]
+        """Matrices of the layers (what weight quantisation applies to). The projections out of the latent are left out: they
+        are applied to queries and to weighted sums as well as to the latents."""
+        return [m.weight for layer in self.layers for n, m in layer.named_modules()
+                if isinstance(m, Linear) and not n.endswith("kv_up_proj")]
+
+    def plan_latent(self, counts: list[int], ctx: list[int], boundaries: Callable) -> Optional[LatentPlan]:
+        """How latent-attention layers run a step of ``counts[i]`` new tokens in sequences of ``ctx[i]`` tokens, ordered by
+        :meth:`latent_order`. ``boundaries(list)``: int32 device tensor. None without such layers."""
+        if not any(s.kind == "latent_attention" for s in self.cfg.layer_specs):
+            return None
+        B = sum(c <= self.latent_short for c in counts)
+        groups, b0 = [], B
+        while b0 < len(counts):  # expanded keys and values are scratch: contexts are taken together up to a bound
+            b1, total = b0 + 1, ctx[b0]
+            while b1 < len(counts) and total + ctx[b1] <= LATENT_GROUP:
+                total += ctx[b1]
+                b1 += 1
+            cu = [0]
+            for c in ctx[b0:b1]:
+                cu.append(cu[-1] + c)
+            groups.append((b0, b1, boundaries(cu), total, max(counts[b0:b1])))
+            b0 = b1
+        return LatentPlan(B, sum(counts[:B]), tuple(groups))
+
+    def latent_order(self, counts: list[int]) -> Optional[list[int]]:
+        """Order of a step's sequences: those whose latent attention stays in the latent space first. None: any order."""
+        if all(s.kind != "latent_attention" for s in self.cfg.layer_specs):
+            return None
+        return sorted(range(len(counts)), key=lambda i: counts[i] > self.latent_short)
 
     def forward(self, *args, **kwargs):
         raise NotImplementedError(f"{self.cfg.model_type}: layer-list models are served by the rollout engine only "
@@ -198,10 +325,23 @@ class HybridLM(nn.Module):
     @torch.no_grad()
     def run(self, ids: torch.Tensor, batch: RaggedBatch, cache: StateCache, mm: Callable,
             observe: Optional[Callable] = None) -> torch.Tensor:
-        """Final-norm hidden states [T, H] of one step. ``mm(x, w)``: the engine's matrix product. ``observe(i, stream)``
+        """Final-norm hidden states [T, H] of one step (times the design's logit scale). ``mm(x, w)``: the engine's matrix product. ``observe(i, stream)``
         gets the residual stream after layer i (a copy; debugging and tests)."""
-        eps = self.cfg.rms_norm_eps
-        res = ops.embedding_scaled(ids, self.embed_tokens.weight, self.cfg.embedding_scale)
+        c, eps = self.cfg, self.cfg.rms_norm_eps
+        if c.design.norm == "post":
+            res, x = ops.embedding_scaled(ids, self.embed_tokens.weight, c.embedding_scale, with_copy=True)
+            last = len(self.layers) - 1
+            for i, layer in enumerate(self.layers):
+                subs = [(lambda v: layer.mixer(v, batch, cache.layers[i], mm), layer.norm1)]
+                if layer.mlp is not None:
+                    subs.append((lambda v: layer.mlp(v, mm), layer.norm2))
+                for k, (sub, norm) in enumerate(subs):
+                    final = self.norm.weight if i == last and k == len(subs) - 1 else None
+                    x = ops.rmsnorm_add(sub(x), res, norm.weight, eps, final_weight=final, final_scale=c.logit_scale)
+                if observe is not None:
+                    observe(i, res.clone())
+            return x
+        res = ops.embedding_scaled(ids, self.embed_tokens.weight, c.embedding_scale)
         pending = None  # output of the last sublayer, not yet added to the stream
         for i, layer in enumerate(self.layers):
             x = ops.add_rmsnorm(pending, res, layer.norm1.weight, eps)

@@ -3,12 +3,15 @@
 reference paths that exist for the CPU test tier."""
 
 from . import _lib
-from .attention import (attention_varlen, decode_workspace, kv_cache_write, paged_attention, paged_decode_attention,
-                        qk_norm_kv_write)
+from .attention import (attention_varlen, decode_workspace, head_norm_rope_kv_write, kv_cache_write, paged_attention,
+                        paged_decode_attention, qk_norm_kv_write)
 from .delta import delta_rule
 from .gemm import gemm, linear
+from .latent import (latent_attention, latent_gather, latent_prefill, latent_prefill_supported, latent_queries,
+                     latent_rope_write, latent_values)
 from .lmhead import lmhead_logprob_entropy
-from .nn import add_rmsnorm, clamped_glu, embedding, embedding_scaled, rmsnorm, rope_qkv, rope_tables, swiglu
+from .nn import (add_rmsnorm, clamped_glu, embedding, embedding_scaled, gelu_tanh_glu, rmsnorm, rmsnorm_add, rope_qkv,
+                 rope_tables, swiglu)
 from .rl import (PPO_METRIC_NAMES, adamw_step, clip_coef, decode_advance, gae, grpo_advantage, ppo_loss_fused, sample,
                  sumsq_into)
 
@@ -17,4 +20,6 @@ __all__ = [
     "attention_varlen", "paged_decode_attention", "kv_cache_write", "decode_workspace", "ppo_loss_fused", "gae",
     "grpo_advantage", "sample", "decode_advance", "adamw_step", "sumsq_into", "clip_coef", "PPO_METRIC_NAMES",
     "paged_attention", "qk_norm_kv_write", "delta_rule", "add_rmsnorm", "clamped_glu", "embedding_scaled",
+    "rmsnorm_add", "gelu_tanh_glu", "head_norm_rope_kv_write", "latent_attention", "latent_gather", "latent_prefill",
+    "latent_prefill_supported", "latent_queries", "latent_rope_write", "latent_values",
 ]

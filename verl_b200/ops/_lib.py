@@ -46,16 +46,28 @@ _SIGS = {
     "vb_clip_coef": ([P, F, F, P, P, P, P], I),
     "vb_cast_f32_bf16": ([P, P, L, P], I),
     # layer-list decoders
-    "vb_embed_scaled": ([P, P, P, I, I, F, I, P], I),
+    "vb_embed_scaled": ([P, P, P, P, I, I, F, I, P], I),
+    "vb_rmsnorm_add": ([P, L, P, P, P, F, P, I, I, F, I, P], I),
+    "vb_gelu_glu": ([P, L, P, I, I, I, P], I),
+    "vb_head_norm_rope_kv_write": ([P, L, P, P, P, I, I, F, P, P, P, P, I, I, I, I, I, I, F, I, P], I),
+    "vb_latent_rope_write": ([P, L, P, P, F, P, P, P, I, I, I, I, I, I, F, I, P], I),
+    "vb_head_gemm": ([P, L, L, P, I, P, L, L, P, L, I, I, I, I, I, I, P, P], I),
+    "vb_head_gemm_simt": ([P, L, L, P, I, P, L, L, P, L, I, I, I, I, I, I, I, P], I),
+    "vb_latent_decode_supported": ([I, I, I, I], I),
+    "vb_latent_decode_splits": ([I, I, I], I),
+    "vb_latent_decode": ([P, P, I, P, I, P, P, I, I, I, I, I, I, F, I, P, P, P, P], I),
+    "vb_latent_gather": ([P, P, I, P, P, I, I, I, I, P], I),
+    "vb_latent_flash_supported": ([I, I, I, I, I], I),
+    "vb_latent_flash": ([P, L, I, P, L, P, L, I, P, P, I, I, I, I, I, I, F, P, L, P, L, P, P], I),
     "vb_add_rmsnorm": ([P, L, P, P, P, I, I, F, I, P], I),
     "vb_clamped_glu": ([P, L, P, I, I, F, F, I, P], I),
     "vb_qk_norm_kv_write": ([P, L, P, P, P, P, P, I, I, I, I, I, I, F, I, P], I),
     "vb_gemm_simt": ([P, P, P, P, I, I, I, L, L, L, I, I, P], I),
-    "vb_paged_attention_simt": ([P, L, P, P, P, I, P, P, I, I, I, I, I, I, I, F, I, I, P, I, P, L, I, P], I),
+    "vb_paged_attention_simt": ([P, L, P, P, P, I, P, P, I, I, I, I, I, I, I, I, F, I, I, I, P, I, F, P, P, L, P, L, I, P], I),
     "vb_paged_flash_supported": ([I, I, I, I, I, I], I),
-    "vb_paged_flash": ([P, L, P, P, I, P, I, P, P, I, I, I, I, I, I, I, I, F, I, I, P, I, P, L, P, P], I),
+    "vb_paged_flash": ([P, L, P, P, I, P, I, P, P, I, I, I, I, I, I, I, I, F, I, I, I, P, I, F, P, P, L, P, L, P, P], I),
     "vb_paged_decode_window_supported": ([I, I, I, I, I], I),
-    "vb_paged_decode_window": ([P, L, P, P, I, P, I, P, I, I, I, I, I, I, F, I, I, P, I, I, P, L, P, P, P], I),
+    "vb_paged_decode_window": ([P, L, P, P, I, P, I, P, I, I, I, I, I, I, F, I, I, I, P, I, F, P, P, L, I, P, L, P, P, P], I),
     "vb_delta_chunk_supported": ([I, I], I),
     "vb_delta_chunk_bytes": ([I, I, I], L),
     "vb_delta_rule": ([P, L, P, P, P, P, P, P, P, P, P, P, P, P, P, P, L, I, I, I, I, I, I, I, I, F, I, P, P], I),

@@ -206,7 +206,7 @@ def paged_decode_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torc
     return out
 
 
-# ------------------------------------------- paged attention of layer-list decoders (windows, kept keys, distance bias)
+# ----------------- paged attention of layer-list decoders (windows, chunks, kept keys, distance bias, soft cap, sink, gate)
 def qk_norm_kv_write(qkv: torch.Tensor, q_weight: torch.Tensor | None, k_weight: torch.Tensor | None, slots: torch.Tensor,
                      k_cache: torch.Tensor, v_cache: torch.Tensor, heads: int, eps: float) -> torch.Tensor:
     """``qkv`` [T, q | k | v | padding]: RMS norm of q and of k over the whole projection (all heads at once; no weights =
@@ -230,15 +230,61 @@ def qk_norm_kv_write(qkv: torch.Tensor, q_weight: torch.Tensor | None, k_weight:
     return q.reshape(T, heads, D)
 
 
+def rotate_pairs(x: torch.Tensor, positions: torch.Tensor, freqs: torch.Tensor, interleaved: bool,
+                 amplitude: float = 1.0) -> torch.Tensor:
+    """fp32 rotary positions on the first ``2 * len(freqs)`` of the last dimension of x [T, ..., D] (reference form)."""
+    x, n = x.float(), freqs.numel()
+    a = (positions.float()[:, None] * freqs).view([x.shape[0]] + [1] * (x.dim() - 2) + [n])
+    c, s = a.cos() * amplitude, a.sin() * amplitude
+    r = x[..., : 2 * n]
+    u, v = (r[..., 0::2], r[..., 1::2]) if interleaved else (r[..., :n], r[..., n:])
+    u, v = u * c - v * s, v * c + u * s
+    r = torch.stack((u, v), -1).flatten(-2) if interleaved else torch.cat((u, v), -1)
+    return torch.cat((r, x[..., 2 * n :]), -1)
+
+
+def head_norm_rope_kv_write(qkv: torch.Tensor, q_weight: torch.Tensor | None, k_weight: torch.Tensor | None,
+                            freqs: torch.Tensor | None, positions: torch.Tensor, slots: torch.Tensor, k_cache: torch.Tensor,
+                            v_cache: torch.Tensor, heads: int, eps: float, *, interleaved: bool,
+                            amplitude: float = 1.0) -> torch.Tensor:
+    """``qkv`` [T, q | k | v | ...]: RMS norm of every q and k head (weights [D] shared by the heads; None = no norm), rotary
+    positions with the angles ``positions * freqs`` (fp32; None = none) on the first ``2 * len(freqs)`` dimensions, k and v
+    to their places in the paged caches [NB, Hk, BS, D] / [NB, Hk, BS, Dv] (slot < 0: no write). Returns q [T, heads, D], a
+    view of ``qkv`` (changed in place on CUDA)."""
+    _, Hk, BS, D = k_cache.shape
+    Dv = v_cache.shape[3]
+    T, nq, nk = qkv.shape[0], heads * D, Hk * D
+    if qkv.is_cuda:
+        rc = _lib.fn("vb_head_norm_rope_kv_write")(
+            qkv.data_ptr(), qkv.stride(0), _lib.ptr(q_weight), _lib.ptr(k_weight), _lib.ptr(freqs),
+            0 if freqs is None else freqs.numel(), int(interleaved), float(amplitude), positions.data_ptr(), slots.data_ptr(),
+            k_cache.data_ptr(), v_cache.data_ptr(), T, heads, Hk, D, Dv, BS, float(eps), int(qkv.dtype == torch.float32),
+            _lib.stream())
+        _lib.check(rc, "vb_head_norm_rope_kv_write")
+        return qkv[:, :nq].view(T, heads, D)
+    from .nn import _rmsnorm_ref
+
+    q, k, v = qkv[:, :nq].view(T, heads, D), qkv[:, nq : nq + nk].view(T, Hk, D), qkv[:, nq + nk : nq + nk + Hk * Dv]
+    if q_weight is not None:
+        q, k = (_rmsnorm_ref(x.float(), w.float(), eps) for x, w in ((q, q_weight), (k, k_weight)))
+    if freqs is not None:
+        q, k = (rotate_pairs(x, positions, freqs, interleaved, amplitude) for x in (q, k))
+    kv_cache_write(k.to(qkv.dtype), v.reshape(T, Hk, Dv), slots, k_cache, v_cache)
+    return q.to(qkv.dtype)
+
+
 def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor,
                     cu_q: torch.Tensor, seq_lens: torch.Tensor, max_q: int, *, scale: float, window: int = 0,
-                    keep_first: int = 0, bias: torch.Tensor | None = None, max_ctx: int = 0,
+                    keep_first: int = 0, bias: torch.Tensor | None = None, max_ctx: int = 0, chunk: int = 0,
+                    softcap: float = 0.0, sink: torch.Tensor | None = None, gate: torch.Tensor | None = None,
                     impl: str = "auto") -> torch.Tensor:
     """Causal attention of ragged queries (the last ``cu_q[b + 1] - cu_q[b]`` positions of every sequence) over the paged
     cache, which holds the new tokens already. q [T, Hq, D]; caches [NB, Hk, BS, D] / [NB, Hk, BS, Dv]; ``seq_lens``
     [B] = tokens of each sequence including the new ones. ``window`` > 0: position i sees j <= i with i - j < window or
-    j < keep_first. ``bias`` fp32 [Hq, L]: ``bias[h, min(i - j, L - 1)]`` is added to the scaled score. ``max_ctx``: bound
-    of ``seq_lens``. -> [T, Hq * Dv].
+    j < keep_first. ``bias`` fp32 [Hq, L]: ``bias[h, min(i - j, L - 1)]`` is added to the scaled score. ``chunk`` > 0:
+    position i sees j <= i with i // chunk == j // chunk (not together with a window). ``softcap`` > 0: scores become
+    ``softcap * tanh(score / softcap)`` (without a bias). ``sink`` fp32 [Hq]: exp(sink[h]) joins the softmax denominator.
+    ``gate`` [T, Hq * Dv]: the result is multiplied with its sigmoid. ``max_ctx``: bound of ``seq_lens``. -> [T, Hq * Dv].
 
     ``impl``: "tc" = tcgen05 kernels (bf16, head sizes up to 128 in multiples of 8, block size a power of two in 8..128;
     one token per sequence: up to 8 query heads per KV head), "simt" = CUDA-core kernel, "auto" = "tc" where it applies."""
@@ -246,6 +292,8 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     Hk, BS, Dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
     B = seq_lens.numel()
     out = torch.empty((T, Hq * Dv), dtype=q.dtype, device=q.device)
+    if (chunk > 0 and window > 0) or (softcap > 0 and bias is not None):
+        raise ValueError("paged_attention: chunk goes without window, and softcap without bias")
     if q.is_cuda:
         f32 = q.dtype == torch.float32
         L = 0 if bias is None else bias.shape[1]
@@ -254,16 +302,21 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         else:
             tc = _lib.fn("vb_paged_flash_supported")(Hq, Hk, D, Dv, BS, L)
         tc = bool(tc) and not f32 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
+        if gate is not None:
+            tc = tc and gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0
         if impl == "tc" and not tc:
             raise ValueError(f"tensor-core attention does not support Hq={Hq} Hk={Hk} D={D} Dv={Dv} block_size={BS}")
         args = (q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr())
         table = (block_table.data_ptr(), block_table.stride(0))
-        mask = (float(scale), window, keep_first, _lib.ptr(bias), L)
+        mask = (float(scale), window, keep_first, chunk, _lib.ptr(bias), L, float(softcap), _lib.ptr(sink), _lib.ptr(gate),
+                0 if gate is None else gate.stride(0))
         dst = (out.data_ptr(), out.stride(0))
         if tc and impl != "simt" and max_q == 1:
             seen = max_ctx or block_table.shape[1] * BS
             if window > 0:
                 seen = min(seen, window + keep_first + 128)
+            elif chunk > 0:
+                seen = min(seen, chunk + 128)
             # split the keys only as far as all pieces run at once (two CTAs per SM): windows leave few chunks to walk
             sms = torch.cuda.get_device_properties(q.device).multi_processor_count
             splits = max(1, min(2 * sms // (B * Hk), (seen + 127) // 128, 16))
@@ -276,7 +329,7 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                                            Hq, Hk, D, Dv, BS, *mask, *dst, _lib.status_word(q.device).data_ptr(),
                                            _lib.stream())
         else:
-            rc = _lib.fn("vb_paged_attention_simt")(*args, *table, cu_q.data_ptr(), seq_lens.data_ptr(), T, B, Hq, Hk, D, Dv, BS,
+            rc = _lib.fn("vb_paged_attention_simt")(*args, *table, cu_q.data_ptr(), seq_lens.data_ptr(), T, B, Hq, Hk, D, Dv, Dv, BS,
                                                     *mask, *dst, int(f32), _lib.stream())
         _lib.check(rc, "paged_attention")
         return out
@@ -294,8 +347,18 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         seen = dist >= 0
         if window > 0:
             seen &= (dist < window) | (torch.arange(n, device=q.device)[None] < keep_first)
+        if chunk > 0:
+            at = torch.arange(n, device=q.device) // chunk
+            seen &= at[n - (hi - lo) :, None] == at[None]
+        if softcap > 0:
+            s = softcap * torch.tanh(s / softcap)
         if bias is not None:
             s = s + bias[:, dist.clamp(0, bias.shape[1] - 1)]
         s = s.masked_fill(~seen, float("-inf"))
-        out[lo:hi] = torch.einsum("hqk,hkd->qhd", torch.softmax(s, -1), vv).reshape(hi - lo, -1).to(q.dtype)
+        if sink is not None:  # a key without a value
+            s = torch.cat((s, sink[:, None, None].expand(Hq, hi - lo, 1)), -1)
+        o = torch.einsum("hqk,hkd->qhd", torch.softmax(s, -1)[..., :n], vv).reshape(hi - lo, -1)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[lo:hi].float())
+        out[lo:hi] = o.to(q.dtype)
     return out

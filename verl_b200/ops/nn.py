@@ -272,16 +272,18 @@ def embedding(ids: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
 
 
 # ------------------------------------------------- 32-bit residual stream (inference only)
-def embedding_scaled(ids: torch.Tensor, weight: torch.Tensor, scale: float) -> torch.Tensor:
-    """fp32 residual stream ``weight[ids] * scale`` [T, H]."""
+def embedding_scaled(ids: torch.Tensor, weight: torch.Tensor, scale: float, with_copy: bool = False):
+    """fp32 residual stream ``weight[ids] * scale`` [T, H]; ``with_copy``: (stream, the same in the weight's dtype)."""
     if not weight.is_cuda:
-        return F.embedding(ids, weight).float() * scale
+        res = F.embedding(ids, weight).float() * scale
+        return (res, res.to(weight.dtype, copy=True)) if with_copy else res
     T, H = ids.numel(), weight.shape[1]
     res = torch.empty((T, H), dtype=torch.float32, device=weight.device)
-    rc = _lib.fn("vb_embed_scaled")(ids.data_ptr(), weight.data_ptr(), res.data_ptr(), T, H, float(scale),
+    y = torch.empty((T, H), dtype=weight.dtype, device=weight.device) if with_copy else None
+    rc = _lib.fn("vb_embed_scaled")(ids.data_ptr(), weight.data_ptr(), res.data_ptr(), _lib.ptr(y), T, H, float(scale),
                                     int(weight.dtype == torch.float32), _lib.stream())
     _lib.check(rc, "vb_embed_scaled")
-    return res
+    return (res, y) if with_copy else res
 
 
 def add_rmsnorm(delta: torch.Tensor | None, residual: torch.Tensor, weight: torch.Tensor, eps: float) -> torch.Tensor:
@@ -297,6 +299,37 @@ def add_rmsnorm(delta: torch.Tensor | None, residual: torch.Tensor, weight: torc
                                    weight.data_ptr(), y.data_ptr(), T, H, float(eps), int(weight.dtype == torch.float32),
                                    _lib.stream())
     _lib.check(rc, "vb_add_rmsnorm")
+    return y
+
+
+def rmsnorm_add(delta: torch.Tensor, residual: torch.Tensor, weight: torch.Tensor, eps: float, *,
+                final_weight: torch.Tensor | None = None, final_scale: float = 1.0) -> torch.Tensor:
+    """Adds rmsnorm(delta) * weight to the fp32 ``residual`` [T, H] IN PLACE. Returns the new residual in the weight's dtype,
+    or with ``final_weight`` rmsnorm(residual) * final_weight * final_scale."""
+    if not residual.is_cuda:
+        residual += _rmsnorm_ref(delta.float(), weight.float(), eps)
+        if final_weight is None:
+            return residual.to(weight.dtype, copy=True)
+        return (_rmsnorm_ref(residual, final_weight.float(), eps) * final_scale).to(weight.dtype)
+    T, H = residual.shape
+    y = torch.empty((T, H), dtype=weight.dtype, device=residual.device)
+    rc = _lib.fn("vb_rmsnorm_add")(delta.data_ptr(), delta.stride(0), residual.data_ptr(), weight.data_ptr(),
+                                   _lib.ptr(final_weight), float(final_scale), y.data_ptr(), T, H, float(eps),
+                                   int(weight.dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "vb_rmsnorm_add")
+    return y
+
+
+def gelu_tanh_glu(gate_up: torch.Tensor, ff: int) -> torch.Tensor:
+    """``gate_up`` rows hold [gate (ff) | up (ff) | padding]: gelu(gate) * up [T, ff] with the tanh form of gelu."""
+    if not gate_up.is_cuda:
+        g, u = gate_up[:, :ff].float(), gate_up[:, ff : 2 * ff].float()
+        return (F.gelu(g, approximate="tanh") * u).to(gate_up.dtype)
+    T = gate_up.shape[0]
+    y = torch.empty((T, ff), dtype=gate_up.dtype, device=gate_up.device)
+    rc = _lib.fn("vb_gelu_glu")(gate_up.data_ptr(), gate_up.stride(0), y.data_ptr(), T, ff,
+                                int(gate_up.dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "vb_gelu_glu")
     return y
 
 

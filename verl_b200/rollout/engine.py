@@ -714,7 +714,8 @@ class NativeRolloutEngine:
         ragged = None
         if c.is_layer_list:  # one token per sequence
             ragged = RaggedBatch(torch.arange(B + 1, dtype=torch.int32, device=dev), 1, st["lens"], st["slots"], st["bt"],
-                                 st["state"], self.max_model_len)
+                                 st["state"], self.max_model_len, st["pos"],
+                                 self.model.plan_latent([1] * B, [1] * B, lambda v: None))
 
         def run():
             logits = self._decode_forward(st["ids"], st["pos"], st["slots"], st["bt"], st["lens"], splits, work, ragged)
@@ -861,24 +862,33 @@ class NativeRolloutEngine:
         tokens together. Returns logits [len(rows), V] at the token rows ``rows`` of this step."""
         sc, dev = self.sched, self.device
         counts = [int(sc.seq_ntok[i]) for i in seq_idx]
+        order = self.model.latent_order(counts)
+        if order is not None and order != sorted(order):  # the rows move with their sequences
+            starts = np.concatenate([[0], np.cumsum(counts)])
+            moved = np.empty(starts[-1], np.int64)
+            moved[np.concatenate([np.arange(starts[i], starts[i + 1]) for i in order])] = np.arange(starts[-1])
+            rows = moved[np.asarray(rows, np.int64)]
+            seq_idx, tok_lo, counts = ([x[i] for i in order] for x in (seq_idx, tok_lo, counts))
         tok = np.concatenate([np.arange(lo, lo + n) for lo, n in zip(tok_lo, counts)])
         cu = np.concatenate([[0], np.cumsum(counts)])
         si = np.asarray(seq_idx)
         ctx = int(sc.seq_total[si].max())
         nb = (ctx + self.block_size - 1) // self.block_size
         # one staging copy: int64 fields, then int32 fields
-        wide = [sc.tokens[tok], sc.slots[tok], np.asarray(rows, np.int64)]
+        wide = [sc.tokens[tok], sc.slots[tok], sc.positions[tok], np.asarray(rows, np.int64)]
         narrow = [cu, sc.seq_total[si], sc.step_state_slots(int(si.max()) + 1)[si], sc.block_tables[si, :nb].ravel()]
         buf = np.concatenate([np.concatenate(wide).astype(np.int64).view(np.int32),
                               np.concatenate(narrow).astype(np.int32)])
         d = torch.from_numpy(buf).to(dev)
-        T, B, R = len(tok), len(seq_idx), len(wide[2])
-        w = d[: 2 * (2 * T + R)].view(torch.int64)
-        x = d[2 * (2 * T + R) :]
+        T, B, R = len(tok), len(seq_idx), len(wide[3])
+        w = d[: 2 * (3 * T + R)].view(torch.int64)
+        x = d[2 * (3 * T + R) :]
         batch = RaggedBatch(x[: B + 1], max(counts), x[B + 1 : 2 * B + 1], w[T : 2 * T], x[3 * B + 1 :].view(B, nb),
-                            x[2 * B + 1 : 3 * B + 1], ctx)
+                            x[2 * B + 1 : 3 * B + 1], ctx, w[2 * T : 3 * T],
+                            self.model.plan_latent(counts, sc.seq_total[si].tolist(),
+                                                   lambda v: torch.tensor(v, dtype=torch.int32, device=dev)))
         h = self.model.run(w[:T], batch, self.state_cache, self._mm, observe=getattr(self, "observe_layers", None))
-        return self._final_logits(h[w[2 * T :]]) if R else h.new_zeros((0, self.cfg.vocab_size), dtype=torch.float32)
+        return self._final_logits(h[w[3 * T :]]) if R else h.new_zeros((0, self.cfg.vocab_size), dtype=torch.float32)
 
     # -------------------------------------------------------------------- step
     def _run_decode_batch(self, dec: list[int], tok_lo: list[int], steps: int, sps: list):
