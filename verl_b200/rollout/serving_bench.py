@@ -131,8 +131,7 @@ def bench_kernels(name: str, vs: str, B: int, n: int, DB: int, ctx: int) -> list
     """Kernel times of the layer-list model and of its counterparts: prefill of B x n tokens, decode of DB sequences."""
     bw, tf, _ = _peaks()
     cfg, ref = preset(name), preset(vs)
-    att = next(s.mixer for s in cfg.layer_specs if s.kind == "attention")
-    dl = next(s.mixer for s in cfg.layer_specs if s.kind == "delta")
+    mixers = {s.kind: s.mixer for s in reversed(cfg.layer_specs)}
     glu = next(s.mlp for s in cfg.layer_specs if s.mlp is not None)
     H, T, bf = cfg.hidden_size, B * n, torch.bfloat16
     r = lambda *s: torch.randn(*s, device="cuda", dtype=bf)  # noqa: E731
@@ -144,21 +143,47 @@ def bench_kernels(name: str, vs: str, B: int, n: int, DB: int, ctx: int) -> list
 
     # norm with residual: fp32 stream against the bf16 stream of the homogeneous model
     x, res32, res16, w = r(T, H), torch.randn(T, H, device="cuda"), r(T, H), r(H)
-    add("add_rmsnorm (fp32 residual)", time_us(lambda: ops.add_rmsnorm(x, res32, w, 1e-5)), T * H * 12)
+    if cfg.design.norm == "post":
+        add("rmsnorm_add (fp32 residual)", time_us(lambda: ops.rmsnorm_add(x, res32, w, 1e-5)), T * H * 12)
+    else:
+        add("add_rmsnorm (fp32 residual)", time_us(lambda: ops.add_rmsnorm(x, res32, w, 1e-5)), T * H * 12)
     add("  vs rmsnorm (bf16 residual)", time_us(lambda: ops.rmsnorm(x, w, 1e-5, res16)), T * H * 8)
     gu = r(T, 2 * glu.ff)
-    add("clamped_glu", time_us(lambda: ops.clamped_glu(gu, glu.ff, glu.limit, glu.alpha)), T * glu.ff * 6)
+    if glu.act == "gelu_tanh":
+        add("gelu_tanh_glu", time_us(lambda: ops.gelu_tanh_glu(gu, glu.ff)), T * glu.ff * 6)
+    else:
+        add("clamped_glu", time_us(lambda: ops.clamped_glu(gu, glu.ff, glu.limit, glu.alpha)), T * glu.ff * 6)
     add("  vs swiglu", time_us(lambda: ops.swiglu(gu)), T * glu.ff * 6)
     del gu
-    # query / key norm and cache write against RoPE + cache write
-    kc, vc, bt = _paged(B, n, 16, att.kv_heads, att.dim)
-    slots = (bt.long()[:, :, None] * 16 + torch.arange(16, device="cuda")).view(B, -1)[:, :n].reshape(-1).contiguous()
-    qkv, qw, kw = r(T, att.q_size + 2 * att.k_size), r(att.q_size), r(att.k_size)
+    if "attention" in mixers:
+        _bench_attention(add, r, mixers["attention"], ref, B, n, DB, ctx)
+    if "latent_attention" in mixers:
+        _bench_latent(add, r, mixers["latent_attention"], B, n, DB, ctx)
+    if "delta" in mixers:
+        _bench_delta(add, r, mixers["delta"], B, n, DB, ctx)
+    return rows
+
+
+def _slots(bt, B: int, n: int):
+    return (bt.long()[:, :, None] * 16 + torch.arange(16, device="cuda")).view(B, -1)[:, :n].reshape(-1).contiguous()
+
+
+def _bench_attention(add, r, att, ref, B: int, n: int, DB: int, ctx: int) -> None:
+    T, hq, hk, d = B * n, att.heads, att.kv_heads, att.dim
+    # query / key norm (and rotation) with the cache write against RoPE + cache write
+    kc, vc, bt = _paged(B, n, 16, hk, d)
+    slots = _slots(bt, B, n)
+    qkv, (nqw, nkw) = r(T, att.q_size + 2 * att.k_size), att.norm_sizes
+    qw, kw = r(nqw), r(nkw)
     nb = T * (2 * att.q_size + 4 * att.k_size) * 2
-    add("qk_norm_kv_write", time_us(lambda: ops.qk_norm_kv_write(qkv, qw, kw, slots, kc, vc, att.heads, 1e-5)), nb)
-    cos, sin = ops.rope_tables(ref.head_dim, n, 1e6, "cuda")
     pos = torch.arange(n, device="cuda").repeat(B)
-    hq, hk, d = att.heads, att.kv_heads, att.dim
+    if att.qk_norm == "head":
+        freqs = torch.tensor(att.rotary.frequencies(), device="cuda")
+        add("head_norm_rope_kv_write", time_us(lambda: ops.head_norm_rope_kv_write(
+            qkv, qw, kw, freqs, pos, slots, kc, vc, hq, 1e-5, interleaved=att.rotary.interleaved)), nb)
+    else:
+        add("qk_norm_kv_write", time_us(lambda: ops.qk_norm_kv_write(qkv, qw, kw, slots, kc, vc, hq, 1e-5)), nb)
+    cos, sin = ops.rope_tables(ref.head_dim, n, 1e6, "cuda")
 
     def rope_write():
         y = ops.rope_qkv(qkv, pos, cos, sin, hq, hk, d)
@@ -171,14 +196,36 @@ def bench_kernels(name: str, vs: str, B: int, n: int, DB: int, ctx: int) -> list
     q = qkv[:, : att.q_size].view(T, hq, d)
     cu = torch.arange(B + 1, device="cuda", dtype=torch.int32) * n
     lens = torch.full((B,), n, device="cuda", dtype=torch.int32)
-    bias = torch.randn(hq, int(att.bias_max) + 1, device="cuda")
     i = torch.arange(n, dtype=torch.float64)
-    pairs = float((torch.minimum(i + 1, torch.full_like(i, att.window) + torch.minimum(
-        torch.full_like(i, att.keep_first), (i + 1 - att.window).clamp(min=0)))).sum())
-    kw_ = dict(scale=att.scale, window=att.window, keep_first=att.keep_first, bias=bias)
-    add(f"paged_flash (window {att.window}, bias)", time_us(
-        lambda: ops.paged_attention(q, kc, vc, bt, cu, lens, n, **kw_)), T * (2 * hq + 2 * hk) * d * 2, 4 * pairs * B * hq * d)
-    add("paged_flash (full causal, no bias)", time_us(
+    kw_, what = {"scale": att.scale}, []
+    if att.chunk:
+        pairs = float((i % att.chunk + 1).sum())
+        kw_["chunk"] = att.chunk
+        what.append(f"chunk {att.chunk}")
+    elif att.window:
+        pairs = float((torch.minimum(i + 1, torch.full_like(i, att.window) + torch.minimum(
+            torch.full_like(i, att.keep_first), (i + 1 - att.window).clamp(min=0)))).sum())
+        kw_ |= {"window": att.window, "keep_first": att.keep_first}
+        what.append(f"window {att.window}")
+    else:
+        pairs = float((i + 1).sum())
+    if att.bias_max:
+        kw_["bias"] = torch.randn(hq, int(att.bias_max) + 1, device="cuda")
+        what.append("bias")
+    if att.softcap:
+        kw_["softcap"] = att.softcap
+        what.append("softcap")
+    if att.sink:
+        kw_["sink"] = torch.randn(hq, device="cuda")
+        what.append("sink")
+    gate = r(max(T, DB), att.out_size) if att.gate else None
+    if att.gate:
+        what.append("gate")
+    what = ", ".join(what)
+    nbytes = T * ((3 if att.gate else 2) * hq + 2 * hk) * d * 2
+    add(f"paged_flash ({what})", time_us(lambda: ops.paged_attention(
+        q, kc, vc, bt, cu, lens, n, **kw_, gate=gate[:T] if att.gate else None)), nbytes, 4 * pairs * B * hq * d)
+    add("paged_flash (full causal, plain)", time_us(
         lambda: ops.paged_attention(q, kc, vc, bt, cu, lens, n, scale=att.scale)),
         T * (2 * hq + 2 * hk) * d * 2, 2.0 * n * (n + 1) * B * hq * d)
     k = qkv[:, att.q_size : att.q_size + att.k_size].view(T, hk, d)
@@ -189,14 +236,63 @@ def bench_kernels(name: str, vs: str, B: int, n: int, DB: int, ctx: int) -> list
     kc, vc, bt = _paged(DB, ctx, 16, hk, d)
     q1, cu1 = r(DB, hq, d), torch.arange(DB + 1, device="cuda", dtype=torch.int32)
     lens = torch.full((DB,), ctx, device="cuda", dtype=torch.int32)
-    seen = min(ctx, att.window + att.keep_first)
-    add(f"paged_decode_window (window {att.window}, bias)", time_us(
-        lambda: ops.paged_attention(q1, kc, vc, bt, cu1, lens, 1, max_ctx=ctx, **kw_)), DB * seen * hk * d * 4)
+    seen = (ctx - 1) % att.chunk + 1 if att.chunk else min(ctx, att.window + att.keep_first) if att.window else ctx
+    add(f"paged_decode_window ({what}: {seen} keys)", time_us(lambda: ops.paged_attention(
+        q1, kc, vc, bt, cu1, lens, 1, max_ctx=ctx, **kw_, gate=gate[:DB] if att.gate else None)), DB * seen * hk * d * 4)
     splits, work = ops.decode_workspace(DB, hq, hk, d, ctx, "cuda")
     add("  vs paged_decode_tc (full context)", time_us(
         lambda: ops.paged_decode_attention(q1, kc, vc, bt, lens, num_splits=splits, work=work)), DB * ctx * hk * d * 4)
-    del kc, vc
-    # delta rule
+
+
+def _bench_latent(add, r, m, B: int, n: int, DB: int, ctx: int) -> None:
+    T, h, D, width = B * n, m.heads, m.dim + m.rot_dim, (m.latent_size + 7) // 8 * 8
+    per = (n + 15) // 16
+    pages, bt = r(B * per, 16, width), torch.randperm(B * per, device="cuda").view(B, per).int()
+    proj, nw = r(T, m.proj_size), r(m.kv_rank)
+    freqs, pos, slots = torch.tensor(m.rotary.frequencies(), device="cuda"), torch.arange(n, device="cuda").repeat(B), _slots(bt, B, n)
+    add("latent_rope_write", time_us(lambda: ops.latent_rope_write(
+        proj, nw, freqs, pos, slots, pages, h, m.dim, m.rot_dim, m.kv_rank, 1e-5)), T * 4 * (h * m.rot_dim + m.latent_size))
+    proj.normal_()
+    q, gate = proj[:, : m.q_size].view(T, h, D), proj[:, m.q_size + m.latent_size :]
+    cu = torch.arange(B + 1, device="cuda", dtype=torch.int32) * n
+    up = r(m.up_size, m.kv_rank) * m.kv_rank ** -0.5
+    add("latent_gather", time_us(lambda: ops.latent_gather(pages, bt, cu, T)), T * width * 4)
+    rows = ops.latent_gather(pages, bt, cu, T)
+    add("up projection of the latents (gemm)", time_us(lambda: ops.gemm(rows[:, : m.kv_rank], up)),
+        2 * (T * (m.kv_rank + m.up_size) + m.up_size * m.kv_rank), 2.0 * T * m.up_size * m.kv_rank)
+    kv, out = ops.gemm(rows[:, : m.kv_rank], up), r(T, m.out_size)
+    add("latent_flash (full causal, gate)", time_us(lambda: ops.latent_prefill(
+        q, rows[:, m.kv_rank : m.latent_size], kv, cu, cu, n, m.dim, m.vdim, scale=m.scale, gate=gate, out=out)),
+        2 * T * (h * (D + m.dim + 3 * m.vdim) + m.rot_dim), float(n) * (n + 1) * B * h * (D + m.vdim))
+    per = (ctx + 15) // 16
+    pages, bt = r(DB * per, 16, width), torch.randperm(DB * per, device="cuda").view(DB, per).int()
+    lens, cu1 = torch.full((DB,), ctx, device="cuda", dtype=torch.int32), torch.arange(DB + 1, device="cuda", dtype=torch.int32)
+    uk, uv = up[: h * m.dim].view(h, m.dim, m.kv_rank), up[h * m.dim :].view(h, m.vdim, m.kv_rank)
+    # the weights of the per-head products rotate, so that they come from memory
+    uks, uvs = [uk.clone() for _ in range(40)], [uv.clone() for _ in range(40)]
+    turn = [0]
+
+    def at(ws):
+        turn[0] += 1
+        return ws[turn[0] % 40]
+
+    add("latent_queries (decode)", time_us(lambda: ops.latent_queries(q[:DB], at(uks)), iters=40),
+        2 * (h * m.dim * m.kv_rank + DB * h * (D + width)), 2.0 * DB * h * m.dim * m.kv_rank)
+    qa = ops.latent_queries(q[:DB], uk)
+    add("latent_decode", time_us(lambda: ops.latent_attention(qa, pages, bt, cu1, lens, m.kv_rank, scale=m.scale, max_ctx=ctx)),
+        2 * DB * (ctx * m.latent_size + h * (width + m.kv_rank)), 2.0 * DB * ctx * h * (m.latent_size + m.kv_rank))
+    lat = ops.latent_attention(qa, pages, bt, cu1, lens, m.kv_rank, scale=m.scale, max_ctx=ctx)
+    add("latent_values (decode, gate)", time_us(lambda: ops.latent_values(lat, at(uvs), gate[:DB], out[:DB]), iters=40),
+        2 * (h * m.vdim * m.kv_rank + DB * h * (m.kv_rank + 2 * m.vdim)), 2.0 * DB * h * m.vdim * m.kv_rank)
+    x, ws = r(DB, m.kv_rank), [uv.reshape(-1, m.kv_rank).clone() for _ in range(40)]
+    add("  vs gemm with a weight of that size", time_us(lambda: ops.gemm(x, at(ws)), iters=40),
+        2 * (h * m.vdim * m.kv_rank + DB * (m.kv_rank + h * m.vdim)), 2.0 * DB * h * m.vdim * m.kv_rank)
+
+
+def _bench_delta(add, r, dl, B: int, n: int, DB: int, ctx: int) -> None:
+    T = B * n
+    cu = torch.arange(B + 1, device="cuda", dtype=torch.int32) * n
+    cu1 = torch.arange(DB + 1, device="cuda", dtype=torch.int32)
     proj = r(T, dl.proj_size)
     conv, alog = r(dl.channels, dl.conv) * 0.5, torch.zeros(dl.heads, device="cuda")
     nw, dt = r(dl.vdim), torch.full((dl.heads,), -3.0, device="cuda")
@@ -213,7 +309,6 @@ def bench_kernels(name: str, vs: str, B: int, n: int, DB: int, ctx: int) -> list
     add("delta_rule decode (fused step)", time_us(
         lambda: ops.delta_rule(proj[:DB], conv, alog, dt, nw, ring, state, cu1, lens, sl[:DB], 1, *dims)),
         DB * (2 * 4 * dl.heads * dl.dim * dl.vdim + (dl.proj_size + dl.out_size + dl.conv * dl.channels) * 2))
-    return rows
 
 
 def main(args) -> dict:
