@@ -114,7 +114,7 @@ def test_latent_rotation_norm_and_cache_write(dtype, H, N, rot, rank):
     T, BS, pos0 = 19, 16, 700
     nq = H * (N + rot)
     proj, w = rand(T, (nq + rank + rot + 15) // 8 * 8, seed=1, dtype=dtype), rand(rank, seed=2, dtype=dtype)
-    pages = torch.zeros(4, BS, (rank + rot + 7) // 8 * 8, dtype=dtype).cuda()
+    pages = torch.zeros(4, BS, ops.latent_width(rank + rot), dtype=dtype).cuda()
     slots = torch.randperm(4 * BS, generator=torch.Generator().manual_seed(1))[:T]
     slots[5] = -1
     freqs, amp = O.yarn_frequencies(rot, 2000.0, M.YARN)
@@ -215,7 +215,7 @@ LATENT_SIZES = pytest.mark.parametrize("H,N,rot,V,rank,bs", [
 
 
 def latent_case(H, N, rot, V, rank, dtype, n=333, gain=1.0):
-    width = (rank + rot + 7) // 8 * 8
+    width = ops.latent_width(rank + rot)
     rows = torch.zeros(n, width, dtype=dtype)
     rows[:, :rank + rot] = rand(n, rank + rot, seed=1, dtype=dtype)
     q = rand(n, H, N + rot, seed=2, dtype=dtype, scale=gain)
@@ -289,7 +289,7 @@ def test_latent_attention_far_keys(form):
     """One key that outweighs all others, anywhere in the context: block, page and split borders, the first and last tokens."""
     H, N, rot, V, rank, n = 2, 16, 16, 16, 64, 700
     for j in (0, 1, 15, 16, 127, 128, 255, 256, 383, 511, 512, 640, 698, 699):
-        rows = torch.zeros(n, rank + rot, dtype=BF)
+        rows = torch.zeros(n, ops.latent_width(rank + rot), dtype=BF)
         rows[j, rank + 3], rows[j, 5] = 6.0, 1.0       # the rotated part stands out, the latent carries the value
         q = torch.zeros(n, H, N + rot, dtype=BF)
         q[:, :, N + 3] = 5.0
@@ -305,7 +305,7 @@ def test_latent_attention_far_keys(form):
             r = ops.latent_gather(pages, bt, ctx, n)
             kv = ops.gemm(r[:, :rank], torch.cat([uk.view(-1, rank), uv.view(-1, rank)]))
             out = torch.empty(n, H * V, dtype=BF, device="cuda")
-            ops.latent_prefill(q.cuda(), r[:, rank:], kv, i32(0, n), ctx, n, N, V, scale=1.0, gate=None, out=out)
+            ops.latent_prefill(q.cuda(), r[:, rank:rank + rot], kv, i32(0, n), ctx, n, N, V, scale=1.0, gate=None, out=out)
             if j > 0:  # the query before it does not see it
                 assert abs(float(out[j - 1].float().mean())) < 1e-2, j
         assert abs(float(out[-1].float().mean()) - 1.0) < 1e-2, j

@@ -3,16 +3,19 @@
 // head_gemm: out[t, h, :] = a[t, h, :] . B_h for every head h of ragged token rows, the up projections of latent attention
 // applied to queries (and to weighted sums, times the sigmoid of an output gate). One CTA per (head, 128 rows, 64 columns).
 //
-// latent_decode: paged attention whose one "key head" is the row of the cache itself: R = rank + rotated part numbers, the
+// latent_decode: paged attention whose one "key head" is the row of the cache itself: `width` numbers (a multiple of 64), the
 // first `rank` of them being the value as well, so a row is read once. One CTA per (query row, group of up to 32 heads,
-// split of the keys). Work is transposed as in paged_attention_tc.cu, 128 keys at a time:
-//     S^T[keys x heads]  = C[128 keys x R] . Q^T              (M = 128 keys, N = heads)
-//     O^T[rank x heads] += C^T[rank x 128 keys] . P           (M = 128 dims per block, N = 2 x heads)
-// The row tile stays in shared memory for both products, in pairs of 64-column parts (32 KB) that a ring of slots hands from
-// the producer to the tensor core; a pair's slot is free once its part of O^T has been added. P is two bf16 terms (hi in the
-// columns of the heads, lo behind them), so that the weights stay close to fp32; both land in accumulators of their own and
-// are added at the end. O^T accumulates in TMEM over all keys: a head's reference only moves when its maximum has grown by
-// more than 2^8, and every thread keeps the sum of its own keys' weights until the end.
+// split of the keys). Work is transposed as in paged_attention_tc.cu, 64 keys at a time:
+//     S^T[keys x heads]  = C[64 keys x width] . Q^T          (M = keys, N = heads)
+//     O^T[rank x heads] += C^T[rank x 64 keys] . P           (M = 128 dims per block, N = 2 x heads)
+// A stage holds 64 whole rows and serves both products; a second one loads meanwhile. A row is wide, so one copy takes all
+// 64-column parts of eight rows: a stage is [8 groups][parts][8 rows x 128 bytes], and both products address it through the
+// strides of their descriptors. The M = 128 of the first product spans a pair of stages; the half of S^T that belongs to the
+// chunk is used (TMEM lanes 0..63 for even chunks, 64..127 for odd ones), the other half is never read. So warps 0-1 take
+// the softmax of even chunks and warps 2-3 that of odd ones.
+// P is two bf16 terms (hi in the columns of the heads, lo behind them), so that the weights stay close to fp32; both land in
+// accumulators of their own and are added at the end. O^T accumulates in TMEM over all keys: a head's reference only moves
+// when its maximum has grown by more than 2^8, and every thread keeps the sum of its own keys' weights until the end.
 // Every wait is bounded; on expiry the status word is set and the CTA leaves through its teardown.
 #include "common.cuh"
 #include "host_utils.h"
@@ -163,29 +166,30 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
 }
 
 // ------------------------------------------------------------------------------------------------ attention on latents
-constexpr int LD_KEYS = 128, LD_THREADS = 192, LD_SLOT = 32768, LD_MAX_SLOTS = 6, LD_MAX_PAIRS = 5, LD_BT = 512;
+constexpr int LD_KEYS = 64, LD_THREADS = 192, LD_MAX_STAGES = 6, LD_MAX_PARTS = 10;
 constexpr float LD_SLACK = 8.f;
 constexpr float LD_LOG2E = 1.4426950408889634f, LD_LN2 = 0.6931471805599453f;
 
 struct LatentDecodeParams {
   const __nv_bfloat16* q;  // [T, H, width]
   const int *block_table, *cu_q, *seq_lens;
-  int max_blocks, T, B, H, width, rank, block_size, num_splits, slots;
+  int max_blocks, T, B, H, width, rank, block_size, num_splits, stages;
   float scale;
   __nv_bfloat16* out;      // [T, H, rank]
   float *o_part, *ml_part;
   int* status;
 };
 
-// shared memory behind the slots: Q, P, barriers, block table, reductions
+// shared memory: stages, Q, two P buffers, barriers, reductions
 template <int HB>
 struct LdCfg {
-  static constexpr int P_BYTES = 2 * HB * 256;
+  static constexpr int P_BYTES = 2 * HB * 128;
   static constexpr int TMEM = HB == 32 ? 512 : 256;      // S: 2 x HB columns, O: up to 4 x 2 HB
-  static constexpr int TAIL = 256 + LD_BT * 4 + 2 * HB * 16;
-  static __host__ __device__ int q_bytes(int pairs) { return pairs * HB * 256; }
-  static __host__ __device__ int bytes(int slots, int pairs) {
-    return slots * LD_SLOT + q_bytes(pairs) + P_BYTES + TAIL + 1024;
+  static constexpr int TAIL = 256 + 2 * HB * 16;
+  static __host__ __device__ int stage_bytes(int parts) { return parts * LD_KEYS * 128; }
+  static __host__ __device__ int q_bytes(int parts) { return parts * HB * 128; }
+  static __host__ __device__ int bytes(int stages, int parts) {
+    return stages * stage_bytes(parts) + q_bytes(parts) + 2 * P_BYTES + TAIL + 1024;
   }
 };
 
@@ -212,16 +216,15 @@ __global__ void __launch_bounds__(LD_THREADS, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecodeParams p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  const int parts = (p.width + 63) / 64, pairs = (parts + 1) / 2, v_pairs = (p.rank + 127) / 128;
-  const int slots = p.slots;
-  uint8_t* q_s = smem + slots * LD_SLOT;
-  uint8_t* p_s = q_s + LdCfg<HB>::q_bytes(pairs);
-  uint64_t* full = reinterpret_cast<uint64_t*>(p_s + LdCfg<HB>::P_BYTES);
-  uint64_t *empty = full + LD_MAX_SLOTS, *s_full = empty + LD_MAX_SLOTS, *p_ready = s_full + 2, *o_full = p_ready + 1;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(o_full + 1);
+  const int parts = p.width >> 6, v_blocks = (p.rank + 127) / 128, stages = p.stages;
+  const int stage_bytes = LdCfg<HB>::stage_bytes(parts);
+  uint8_t* q_s = smem + stages * stage_bytes;
+  uint8_t* p_s = q_s + LdCfg<HB>::q_bytes(parts);
+  uint64_t* full = reinterpret_cast<uint64_t*>(p_s + 2 * LdCfg<HB>::P_BYTES);
+  uint64_t *empty = full + LD_MAX_STAGES, *s_full = empty + LD_MAX_STAGES, *p_ready = s_full + 2, *o_full = p_ready + 2;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(o_full + 2);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  int* bt_s = reinterpret_cast<int*>(reinterpret_cast<uint8_t*>(full) + 256);
-  float(*red_s)[4] = reinterpret_cast<float(*)[4]>(bt_s + LD_BT);
+  float(*red_s)[4] = reinterpret_cast<float(*)[4]>(reinterpret_cast<uint8_t*>(full) + 256);
   float(*sum_s)[4] = red_s + HB;
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -229,14 +232,15 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
   const int nh = min(HB, p.H - h0);
 
   if (tid == 0) {
-    for (int s = 0; s < LD_MAX_SLOTS; ++s) {
+    for (int s = 0; s < LD_MAX_STAGES; ++s) {
       mbar_init(&full[s], 1);
       mbar_init(&empty[s], 1);
     }
-    mbar_init(&s_full[0], 1);
-    mbar_init(&s_full[1], 1);
-    mbar_init(p_ready, 4);
-    mbar_init(o_full, 1);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&s_full[i], 1);
+      mbar_init(&p_ready[i], 2);
+      mbar_init(&o_full[i], 1);
+    }
     *abort_flag = 0;
     mbar_fence_init();
   }
@@ -263,17 +267,13 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
   const int len = p.seq_lens[b] - (p.T != p.B ? p.cu_q[b + 1] - 1 - t : 0);  // keys that the row sees
   const int chunks = (len + LD_KEYS - 1) / LD_KEYS, per_split = (chunks + p.num_splits - 1) / p.num_splits;
   const int c_begin = split * per_split, n_chunks = max(min(chunks, c_begin + per_split) - c_begin, 0);
-  const int ppc = LD_KEYS / p.block_size, n_pages = (len + p.block_size - 1) / p.block_size;
-  const int* bt = p.block_table + (long long)b * p.max_blocks;
-  // pages past the end re-read the last page: finite data, weight zero
-  for (int i = tid; i < min(n_chunks * ppc, LD_BT); i += LD_THREADS) bt_s[i] = bt[min(c_begin * ppc + i, n_pages - 1)];
   {
     const __nv_bfloat16* q = p.q + ((long long)t * p.H + h0) * p.width;
-    const int per_row = pairs * 16;
+    const int per_row = parts * 8;
     for (int i = tid; i < HB * per_row; i += LD_THREADS) {
       const int r = i / per_row, k = (i - r * per_row) * 8;
       uint4 v = make_uint4(0, 0, 0, 0);
-      if (r < nh && k < p.width) v = *reinterpret_cast<const uint4*>(q + (long long)r * p.width + k);
+      if (r < nh) v = *reinterpret_cast<const uint4*>(q + (long long)r * p.width + k);
       *reinterpret_cast<uint4*>(q_s + sw128_at(r, k, HB)) = v;
     }
   }
@@ -281,38 +281,43 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
   __syncthreads();
 
   if (warp == 4) {
-    // ------------------------------- TMA producer: the pairs of a chunk, last one first -------------------------------
-    if (lane == 0 && n_chunks > 0) {
-      tma_prefetch_desc(&tmC);
-      int tile = 0;
-      bool ok = true;
-      for (int c = 0; ok && c < n_chunks; ++c) {
-        for (int pr = pairs - 1; pr >= 0; --pr, ++tile) {
-          const int s = tile % slots;
-          if (*abort_flag || !mbar_wait(&empty[s], ((tile / slots) & 1) ^ 1)) {
-            report_error(p.status, ERR_WAIT_EMPTY, tile);
-            *abort_flag = 1;
-            ok = false;
-            break;
-          }
-          const int halves = min(2, parts - 2 * pr);
-          mbar_arrive_expect_tx(&full[s], halves * 16384);
-          uint8_t* dst = smem + s * LD_SLOT;
-          for (int pg = 0; pg < ppc; ++pg) {
-            const int rel = c * ppc + pg;
-            const int row = (rel < LD_BT ? bt_s[rel] : bt[min(c_begin * ppc + rel, n_pages - 1)]) * p.block_size;
-            for (int x = 0; x < halves; ++x)
-              tma_load_2d(dst + x * 16384 + pg * p.block_size * 128, &tmC, &full[s], (2 * pr + x) * 64, row);
-          }
+    // ------------------------------- TMA producer: lane g copies rows 8 g .. 8 g + 7 of a chunk -------------------------------
+    if (lane == 0) tma_prefetch_desc(&tmC);
+    const int* bt = p.block_table + (long long)b * p.max_blocks;
+    const int last_page = (len + p.block_size - 1) / p.block_size - 1;
+    // first row of the lane's group; pages past the end re-read the last page: finite data, weight zero
+    auto row_of = [&](int c) {
+      const int key = (c_begin + c) * LD_KEYS + (lane & 7) * 8, page = key / p.block_size;
+      return bt[min(page, last_page)] * p.block_size + key - page * p.block_size;
+    };
+    int row = n_chunks > 0 ? row_of(0) : 0;
+    bool ok = true;
+    for (int c = 0; ok && c < n_chunks; ++c) {
+      const int s = c % stages, next = c + 1 < n_chunks ? row_of(c + 1) : 0;
+      int good = 1;  // lane 0 decides for the warp: the lanes must leave the loop together
+      if (lane == 0) {
+        good = (!*abort_flag && mbar_wait(&empty[s], ((c / stages) & 1) ^ 1)) ? 1 : 0;
+        if (good) {
+          mbar_arrive_expect_tx(&full[s], stage_bytes);
+        } else {
+          report_error(p.status, ERR_WAIT_EMPTY, c);
+          *abort_flag = 1;
         }
       }
+      ok = __shfl_sync(0xffffffffu, good, 0) != 0;
+      if (ok && lane < 8) tma_load_3d(smem + s * stage_bytes + lane * parts * 1024, &tmC, &full[s], 0, row, 0);
+      __syncwarp();
+      row = next;
     }
   } else if (warp == 5) {
     // -------------------------------- MMA issuer --------------------------------
     if (lane == 0 && n_chunks > 0) {
       constexpr uint32_t idesc_qk = umma_idesc(1, 1, 0, 0, 128, HB);      // A = rows (K-major), B = Q^T (K-major)
       constexpr uint32_t idesc_pv = umma_idesc(1, 1, 1, 0, 128, 2 * HB);  // A = rows (MN-major), B = P (K-major)
-      const uint32_t base = smem_u32(smem), q_addr = smem_u32(q_s), p_addr = smem_u32(p_s);
+      // descriptors of the first tiles; steps are added in units of 16 bytes
+      const uint32_t base = smem_u32(smem), group = parts * 1024, step = stage_bytes >> 4;
+      const uint64_t a_qk = umma_smem_desc(base, 16, group), b_qk = umma_smem_desc(smem_u32(q_s), 16, 1024);
+      const uint64_t a_pv = umma_smem_desc(base, 1024, group), b_pv = umma_smem_desc(smem_u32(p_s), 16, 1024);
       auto wait = [&](uint64_t* bar, uint32_t parity, int code, int detail) -> bool {
         if (!*abort_flag && mbar_wait(bar, parity)) return true;
         report_error(p.status, code, detail);
@@ -320,44 +325,45 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
         return false;
       };
       auto issue_qk = [&](int c) -> bool {
+        const int s = c % stages;
+        if (!wait(&full[s], (c / stages) & 1, ERR_WAIT_FULL, c)) return false;
+        tc_fence_after();
+        const uint64_t a = a_qk + (uint64_t)(s & ~1) * step;  // the pair of stages
         const uint32_t d = tmem + (c & 1) * HB;
-        for (int pr = pairs - 1; pr >= 0; --pr) {
-          const int tile = c * pairs + pairs - 1 - pr, s = tile % slots;
-          if (!wait(&full[s], (tile / slots) & 1, ERR_WAIT_FULL, tile)) return false;
-          tc_fence_after();
-          const int steps = min(8, (p.width - pr * 128 + 15) / 16);
-          for (int k = 0; k < steps; ++k)
-            tc_mma_f16(d, umma_smem_desc(base + s * LD_SLOT + (k >> 2) * 16384 + (k & 3) * 32, 16, 1024),
-                       umma_smem_desc(q_addr + (2 * pr + (k >> 2)) * (HB * 128) + (k & 3) * 32, 16, 1024), idesc_qk,
-                       pr != pairs - 1 || k != 0);
-          if (pr >= v_pairs) tc_commit(&empty[s]);  // no values in this pair
+        for (int x = 0; x < parts; ++x) {
+          const uint64_t ax = a + x * 64, bx = b_qk + x * (HB * 8);
+#pragma unroll
+          for (int k = 0; k < 4; ++k) tc_mma_f16(d, ax + 2 * k, bx + 2 * k, idesc_qk, x != 0 || k != 0);
         }
         tc_commit(&s_full[c & 1]);
         return true;
       };
-      const bool ahead = slots >= 2 * pairs;  // the next chunk's rows fit beside this one's
       bool ok = issue_qk(0);
       for (int c = 0; ok && c < n_chunks; ++c) {
-        if (ahead && c + 1 < n_chunks) ok = issue_qk(c + 1);
-        if (!ok || !wait(p_ready, c & 1, ERR_WAIT_TMEM_EMPTY, c)) break;
+        const int s = c % stages, n = (c + 1) % stages;
+        // the next chunk's scores first if its rows are there, so that its softmax can begin; else this chunk's values, so
+        // that its stage can be loaded again
+        const bool more = c + 1 < n_chunks, early = more && mbar_try_wait(&full[n], ((c + 1) / stages) & 1);
+        if (early) ok = issue_qk(c + 1);
+        if (!ok || !wait(&p_ready[c & 1], (c >> 1) & 1, ERR_WAIT_TMEM_EMPTY, c)) break;
         tc_fence_after();
-        for (int pr = v_pairs - 1; pr >= 0; --pr) {
-          const int s = (c * pairs + pairs - 1 - pr) % slots;
+        const uint64_t a = a_pv + (uint64_t)s * step, bp = b_pv + (c & 1) * (LdCfg<HB>::P_BYTES >> 4);
+        for (int v = 0; v < v_blocks; ++v) {
+          const uint32_t d = tmem + 2 * HB + v * 2 * HB;
 #pragma unroll
-          for (int k = 0; k < LD_KEYS / 16; ++k)
-            tc_mma_f16(tmem + 2 * HB + pr * 2 * HB, umma_smem_desc(base + s * LD_SLOT + k * 2048, 16384, 1024),
-                       umma_smem_desc(p_addr + (k >> 2) * (2 * HB * 128) + (k & 3) * 32, 16, 1024), idesc_pv,
-                       c != 0 || k != 0);
-          tc_commit(&empty[s]);
+          for (int k = 0; k < LD_KEYS / 16; ++k)  // 16 keys: two groups of rows
+            tc_mma_f16(d, a + v * 128 + k * 2 * (group >> 4), bp + 2 * k, idesc_pv, c != 0 || k != 0);
         }
-        tc_commit(o_full);
-        if (!ahead && c + 1 < n_chunks) ok = issue_qk(c + 1);
+        tc_commit(&empty[s]);
+        tc_commit(&o_full[c & 1]);
+        if (more && !early) ok = issue_qk(c + 1);
       }
     }
   } else {
     // ----------------------- softmax (thread = key), then output (thread = dim) -----------------------
     const uint32_t lanes = ((uint32_t)(warp * 32)) << 16, s_addr = tmem + lanes, o_addr = s_addr + 2 * HB;
     const float scale2 = p.scale * LD_LOG2E;
+    const int key = tid & 63;
     float ref[HB], sum[HB];  // of all keys: the reference; of this thread's keys: the sum of weights
 #pragma unroll
     for (int g = 0; g < HB; ++g) {
@@ -366,71 +372,94 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
     }
     bool ok = true;
     for (int c = 0; c < n_chunks; ++c) {
-      if (*abort_flag || !mbar_wait(&s_full[c & 1], (c >> 1) & 1) || (c > 0 && !mbar_wait(o_full, (c - 1) & 1))) {
-        report_error(p.status, ERR_WAIT_TMEM_FULL, c);
-        *abort_flag = 1;
-        ok = false;
-      }
-      ok = !ld_bar_or(!ok);  // all 128 threads stop together
-      if (!ok) break;
-      tc_fence_after();
-      uint32_t v[HB];
-      ld_cols<HB>(s_addr + (c & 1) * HB, v);
-      tmem_ld_wait();
-      const bool valid = (c_begin + c) * LD_KEYS + tid < len;
-      bool grown = false;
+      const bool mine = (warp >> 1) == (c & 1);
+      // stages come in pairs: an even chunk is in lanes 0..63, an odd one in lanes 64..127
       float sc[HB];
+      bool grown = false;
+      if (mine) {
+        // P of chunk c - 2 was read by its product
+        if (*abort_flag || !mbar_wait(&s_full[c & 1], (c >> 1) & 1) ||
+            (c > 1 && !mbar_wait(&o_full[c & 1], ((c >> 1) - 1) & 1))) {
+          report_error(p.status, ERR_WAIT_TMEM_FULL, c);
+          *abort_flag = 1;
+          ok = false;
+        }
+        ok = __all_sync(0xffffffffu, ok);  // the lanes of a warp share its TMEM accesses
+        if (ok) {
+          tc_fence_after();
+          uint32_t v[HB];
+          ld_cols<HB>(s_addr + (c & 1) * HB, v);
+          tmem_ld_wait();
+          const bool valid = (c_begin + c) * LD_KEYS + key < len;
 #pragma unroll
-      for (int g = 0; g < HB; ++g) {
-        sc[g] = valid ? __uint_as_float(v[g]) * scale2 : -INFINITY;
-        grown |= sc[g] > ref[g] + LD_SLACK;
+          for (int g = 0; g < HB; ++g) {
+            sc[g] = valid ? __uint_as_float(v[g]) * scale2 : -INFINITY;
+            grown |= sc[g] > ref[g] + LD_SLACK;
+          }
+        }
       }
-      if (ld_bar_or(grown)) {  // rare after the first chunk: find the maxima, move the references that were outgrown
+      if (ld_bar_or(grown || !ok)) {  // rare after the first chunk: move the references that were outgrown
+        // all 128 threads stop together
+        if (c > 0 && ok && (*abort_flag || !mbar_wait(&o_full[(c - 1) & 1], ((c - 1) >> 1) & 1))) {
+          report_error(p.status, ERR_WAIT_TMEM_FULL, 2000 + c);
+          *abort_flag = 1;
+          ok = false;
+        }
+        ok = !ld_bar_or(!ok);
+        if (!ok) break;
+        tc_fence_after();
         float alpha[HB];
+        if (mine) {
 #pragma unroll
-        for (int g = 0; g < HB; ++g) {
-          const float wm = warp_reduce_max(sc[g]);
-          if (lane == 0) red_s[g][warp] = wm;
+          for (int g = 0; g < HB; ++g) {
+            const float wm = warp_reduce_max(sc[g]);
+            if (lane == 0) red_s[g][warp & 1] = wm;
+          }
         }
         ld_bar();
 #pragma unroll
         for (int g = 0; g < HB; ++g) {
-          const float m = fmaxf(fmaxf(red_s[g][0], red_s[g][1]), fmaxf(red_s[g][2], red_s[g][3]));
+          const float m = fmaxf(red_s[g][0], red_s[g][1]);
           const bool move = m > ref[g] + LD_SLACK;
           alpha[g] = move ? exp2f(ref[g] - m) : 1.f;  // exp2(-inf) = 0: nothing seen before
           sum[g] *= alpha[g];
           ref[g] = move ? m : ref[g];
         }
         if (c > 0) {  // the previous chunk's product has completed: O is at rest
-          for (int pr = 0; pr < 2 * v_pairs; ++pr) {
+          for (int v = 0; v < 2 * v_blocks; ++v) {
             uint32_t o[HB];
-            ld_cols<HB>(o_addr + pr * HB, o);
+            ld_cols<HB>(o_addr + v * HB, o);
             tmem_ld_wait();
 #pragma unroll
             for (int g = 0; g < HB; ++g) o[g] = __float_as_uint(__uint_as_float(o[g]) * alpha[g]);
-            if constexpr (HB == 32) tmem_st_32x32(o_addr + pr * HB, o);
-            else tmem_st_32x16(o_addr + pr * HB, o);
+            if constexpr (HB == 32) tmem_st_32x32(o_addr + v * HB, o);
+            else tmem_st_32x16(o_addr + v * HB, o);
           }
           tmem_st_wait();
         }
+        tc_fence_before();
+        ld_bar();  // every lane's part of O is in place before the weights are handed over; red_s is free again
+        tc_fence_after();
       }
-      const uint32_t k_off = (uint32_t)((tid >> 6) * (2 * HB * 128) + (tid & 7) * 2), c16 = (tid & 63) >> 3;
+      if (!mine) continue;
+      uint8_t* pbuf = p_s + (c & 1) * LdCfg<HB>::P_BYTES + (key & 7) * 2;
+      const uint32_t c16 = key >> 3;
 #pragma unroll
       for (int g = 0; g < HB; ++g) {
         const float w = exp2f(sc[g] - ref[g]);
         sum[g] += w;
         const __nv_bfloat16 hi = __float2bfloat16(w);
-        const uint32_t off = k_off + (g >> 3) * 1024 + (g & 7) * 128 + ((c16 ^ (g & 7)) << 4);
-        *reinterpret_cast<__nv_bfloat16*>(p_s + off) = hi;
-        *reinterpret_cast<__nv_bfloat16*>(p_s + off + HB * 128) = __float2bfloat16(w - __bfloat162float(hi));
+        const uint32_t off = (g >> 3) * 1024 + (g & 7) * 128 + ((c16 ^ (g & 7)) << 4);
+        *reinterpret_cast<__nv_bfloat16*>(pbuf + off) = hi;
+        *reinterpret_cast<__nv_bfloat16*>(pbuf + off + HB * 128) = __float2bfloat16(w - __bfloat162float(hi));
       }
       fence_proxy_async_smem();
       tc_fence_before();
       __syncwarp();
-      if (lane == 0) mbar_arrive(p_ready);
+      if (lane == 0) mbar_arrive(&p_ready[c & 1]);
     }
     if (ok && n_chunks > 0) {
-      if (*abort_flag || !mbar_wait(o_full, (n_chunks - 1) & 1)) {
+      if (*abort_flag || !mbar_wait(&o_full[(n_chunks - 1) & 1], ((n_chunks - 1) >> 1) & 1)) {
         report_error(p.status, ERR_WAIT_TMEM_FULL, 1000);
         *abort_flag = 1;
         ok = false;
@@ -460,12 +489,12 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
       }
       if (n_chunks > 0) {
         tc_fence_after();
-        for (int pr = 0; pr < v_pairs; ++pr) {
+        for (int v = 0; v < v_blocks; ++v) {
           uint32_t hi[HB], lo[HB];
-          ld_cols<HB>(o_addr + pr * 2 * HB, hi);
-          ld_cols<HB>(o_addr + pr * 2 * HB + HB, lo);
+          ld_cols<HB>(o_addr + v * 2 * HB, hi);
+          ld_cols<HB>(o_addr + v * 2 * HB + HB, lo);
           tmem_ld_wait();
-          const int d = pr * 128 + tid;
+          const int d = v * 128 + tid;
           if (d < p.rank) {
 #pragma unroll
             for (int g = 0; g < HB; ++g) {
@@ -525,26 +554,26 @@ extern "C" int vb_head_gemm(const void* a, long long a_t, long long a_h, const v
 }
 
 static inline int ld_heads(int H) { return H <= 16 ? 16 : 32; }
-static int ld_slots(int hb, int pairs) {
-  int s = LD_MAX_SLOTS;
-  while (s > 0 && (hb == 32 ? LdCfg<32>::bytes(s, pairs) : LdCfg<16>::bytes(s, pairs)) > 227 * 1024) --s;
+// Stages (an even number: they are used in pairs) that fit beside Q and P; 0: none.
+static int ld_stages(int hb, int parts) {
+  int s = LD_MAX_STAGES;
+  while (s > 0 && (hb == 32 ? LdCfg<32>::bytes(s, parts) : LdCfg<16>::bytes(s, parts)) > 227 * 1024) s -= 2;
   return s;
 }
 
 extern "C" int vb_latent_decode_supported(int H, int width, int rank, int block_size) {
-  const int pairs = (width + 127) / 128;
-  return H > 0 && rank > 0 && rank <= 512 && width >= rank && (width & 7) == 0 && pairs <= LD_MAX_PAIRS && block_size >= 8 &&
-         block_size <= LD_KEYS && LD_KEYS % block_size == 0 && ld_slots(ld_heads(H), pairs) >= pairs;
+  return H > 0 && rank > 0 && rank <= 512 && width >= rank && (width & 63) == 0 && width / 64 <= LD_MAX_PARTS && block_size >= 8 &&
+         (block_size & (block_size - 1)) == 0 && ld_stages(ld_heads(H), width / 64) >= 2;
 }
 
-// Splits of the keys that fill the SMs (one CTA each) for T rows over up to `chunks` blocks of 128 keys.
+// Splits of the keys that fill the SMs (one CTA each) for T rows over up to `chunks` blocks of 64 keys.
 extern "C" int vb_latent_decode_splits(int T, int H, int chunks) {
   const int sms = vb_num_sms(), items = T * ((H + ld_heads(H) - 1) / ld_heads(H));
   int best = 1;
   float best_cost = 0.f;
   for (int s = 1; s <= 16 && s <= chunks; ++s) {
     const int waves = (items * s + sms - 1) / sms;
-    const float cost = waves * ((chunks + s - 1) / s + 1.5f) + (s > 1 ? 1.f + 0.02f * items * s / sms : 0.f);
+    const float cost = waves * ((chunks + s - 1) / s + 3.f) + (s > 1 ? 2.f + 0.04f * items * s / sms : 0.f);
     if (s == 1 || cost < best_cost) {
       best = s;
       best_cost = cost;
@@ -568,14 +597,15 @@ extern "C" int vb_latent_decode(const void* q, const void* pages, int num_blocks
       (num_splits > 1 && work == nullptr) || (reinterpret_cast<uintptr_t>(q) & 15))
     return -3;
   CUtensorMap tmC;
-  int rc = vb_make_tmap_2d(&tmC, pages, 2, (uint64_t)width, (uint64_t)num_blocks * block_size, (uint64_t)width * 2, 64, block_size);
+  // [64 columns] x [rows] x [parts]: one copy takes all parts of eight rows
+  const int hb = ld_heads(H), parts = width / 64, stages = ld_stages(hb, parts);
+  int rc = vb_make_tmap_3d(&tmC, pages, 2, 64, (uint64_t)num_blocks * block_size, parts, (uint64_t)width * 2, 128, 64, 8, parts);
   if (rc) return rc;
-  const int hb = ld_heads(H), pairs = (width + 127) / 128, slots = ld_slots(hb, pairs);
   LatentDecodeParams p{};
   p.q = reinterpret_cast<const __nv_bfloat16*>(q);
   p.block_table = block_table; p.cu_q = cu_q; p.seq_lens = seq_lens; p.max_blocks = max_blocks;
   p.T = T; p.B = B; p.H = H; p.width = width; p.rank = rank; p.block_size = block_size;
-  p.num_splits = num_splits; p.slots = slots; p.scale = scale;
+  p.num_splits = num_splits; p.stages = stages; p.scale = scale;
   p.out = reinterpret_cast<__nv_bfloat16*>(out);
   p.o_part = work;
   p.ml_part = work ? work + (long long)T * H * num_splits * rank : nullptr;
@@ -587,7 +617,7 @@ extern "C" int vb_latent_decode(const void* q, const void* pages, int num_blocks
     attr_set = true;
   }
   const dim3 grid(T, (H + hb - 1) / hb, num_splits);
-  const int smem = hb == 32 ? LdCfg<32>::bytes(slots, pairs) : LdCfg<16>::bytes(slots, pairs);
+  const int smem = hb == 32 ? LdCfg<32>::bytes(stages, parts) : LdCfg<16>::bytes(stages, parts);
   rc = hb == 32 ? (int)vb_launch_pdl(latent_decode_kernel<32>, grid, dim3(LD_THREADS), (size_t)smem, stream, 1, tmC, p)
                 : (int)vb_launch_pdl(latent_decode_kernel<16>, grid, dim3(LD_THREADS), (size_t)smem, stream, 1, tmC, p);
   vb_count_launch(num_splits > 1 ? 2 : 1);

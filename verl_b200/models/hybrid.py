@@ -78,14 +78,14 @@ class StateCache:
                 self.layers.append(tuple(torch.zeros((num_blocks, m.kv_heads, block_size, d), dtype=dtype, device=device)
                                          for d in (m.dim, m.vdim)))
             elif spec.kind == "latent_attention":
-                self.layers.append((torch.zeros((num_blocks, block_size, pad8(m.latent_size)), dtype=dtype, device=device),))
+                self.layers.append((torch.zeros((num_blocks, block_size, ops.latent_width(m.latent_size)), dtype=dtype, device=device),))
             else:
                 self.layers.append((torch.zeros((num_slots, m.conv, m.channels), dtype=dtype, device=device),
                                     torch.zeros((num_slots, m.heads, m.vdim, m.dim), dtype=torch.float32, device=device)))
 
     @staticmethod
     def page_bytes(cfg: ModelConfig, block_size: int, itemsize: int) -> int:
-        per_token = {"attention": lambda m: m.kv_heads * (m.dim + m.vdim), "latent_attention": lambda m: pad8(m.latent_size)}
+        per_token = {"attention": lambda m: m.kv_heads * (m.dim + m.vdim), "latent_attention": lambda m: ops.latent_width(m.latent_size)}
         return sum(per_token[s.kind](s.mixer) for s in cfg.layer_specs if s.kind in per_token) * block_size * itemsize
 
     @staticmethod

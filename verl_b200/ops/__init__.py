@@ -8,7 +8,7 @@ from .attention import (attention_varlen, decode_workspace, head_norm_rope_kv_wr
 from .delta import delta_rule
 from .gemm import gemm, linear
 from .latent import (latent_attention, latent_gather, latent_prefill, latent_prefill_supported, latent_queries,
-                     latent_rope_write, latent_values)
+                     latent_rope_write, latent_values, latent_width)
 from .lmhead import lmhead_logprob_entropy
 from .nn import (add_rmsnorm, clamped_glu, embedding, embedding_scaled, gelu_tanh_glu, rmsnorm, rmsnorm_add, rope_qkv,
                  rope_tables, swiglu)
@@ -21,5 +21,5 @@ __all__ = [
     "grpo_advantage", "sample", "decode_advance", "adamw_step", "sumsq_into", "clip_coef", "PPO_METRIC_NAMES",
     "paged_attention", "qk_norm_kv_write", "delta_rule", "add_rmsnorm", "clamped_glu", "embedding_scaled",
     "rmsnorm_add", "gelu_tanh_glu", "head_norm_rope_kv_write", "latent_attention", "latent_gather", "latent_prefill",
-    "latent_prefill_supported", "latent_queries", "latent_rope_write", "latent_values",
+    "latent_prefill_supported", "latent_queries", "latent_rope_write", "latent_values", "latent_width",
 ]

@@ -1,7 +1,7 @@
 """Latent attention over pages of latents (``csrc/latent_attention.cu``, ``csrc/flash_attention_paged.cu``).
 
 A page row holds one token: the normed latent (``rank`` numbers), the rotated key part all heads share, zeros up to a
-multiple of eight. Two forms of the same attention: short portions stay in the latent space (the up projection of the keys
+multiple of 64. Two forms of the same attention: short portions stay in the latent space (the up projection of the keys
 is applied to the queries, that of the values to the weighted sum), longer ones expand the keys and values of their context.
 """
 
@@ -11,6 +11,11 @@ import torch
 
 from . import _lib
 from .attention import rotate_pairs
+
+
+def latent_width(size: int) -> int:
+    """Numbers of a page row for ``size`` of latent and rotated part."""
+    return (size + 63) // 64 * 64
 
 
 def latent_prefill_supported(heads: int, dim: int, rot_dim: int, vdim: int, rank: int, dtype, device) -> bool:
@@ -25,7 +30,7 @@ def latent_rope_write(proj: torch.Tensor, norm_w: torch.Tensor, freqs: torch.Ten
                       amplitude: float = 1.0) -> None:
     """``proj`` [T, q (heads x [dim | rot_dim]) | latent (rank) | rotated key (rot_dim) | ...]: rotary positions (half layout)
     on the rotated parts, RMS norm of the latent, latent and rotated key to the token's place in ``pages``
-    [NB, BS, pad8(rank + rot_dim)] (slot < 0: no write). The query part of ``proj`` is changed in place."""
+    [NB, BS, latent_width(rank + rot_dim)] (slot < 0: no write). The query part of ``proj`` is changed in place."""
     T, nq = proj.shape[0], heads * (dim + rot_dim)
     if proj.is_cuda:
         rc = _lib.fn("vb_latent_rope_write")(proj.data_ptr(), proj.stride(0), norm_w.data_ptr(), freqs.data_ptr(),
@@ -46,11 +51,11 @@ def latent_rope_write(proj: torch.Tensor, norm_w: torch.Tensor, freqs: torch.Ten
 
 
 def latent_queries(q: torch.Tensor, uk: torch.Tensor, impl: str = "auto") -> torch.Tensor:
-    """q [T, H, dim + rot_dim], uk [H, dim, rank] -> [T, H, pad8(rank + rot_dim)]: queries against latents, rotated part."""
+    """q [T, H, dim + rot_dim], uk [H, dim, rank] -> [T, H, latent_width(rank + rot_dim)]: queries against latents, rotated part."""
     T, H, D = q.shape
     dim, rank = uk.shape[1:]
     rot = D - dim
-    width = (rank + rot + 7) // 8 * 8
+    width = latent_width(rank + rot)
     if q.is_cuda:
         out = torch.empty((T, H, width), dtype=q.dtype, device=q.device)
         _head_gemm(q, uk, out, True, dim, rank, rot, None, impl)
@@ -113,7 +118,7 @@ def latent_attention(q: torch.Tensor, pages: torch.Tensor, block_table: torch.Te
             raise ValueError(f"tensor-core latent attention does not support heads={H} width={width} rank={rank} block_size={BS}")
         out = torch.empty((T, H, rank), dtype=q.dtype, device=q.device)
         if tc and impl != "simt":
-            chunks = ((max_ctx or block_table.shape[1] * BS) + 127) // 128
+            chunks = ((max_ctx or block_table.shape[1] * BS) + 63) // 64
             splits = _lib.fn("vb_latent_decode_splits")(T, H, chunks)
             work = torch.empty(T * H * splits * (rank + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
             rc = _lib.fn("vb_latent_decode")(q.data_ptr(), pages.data_ptr(), NB, block_table.data_ptr(), block_table.stride(0),

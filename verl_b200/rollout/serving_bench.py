@@ -245,7 +245,7 @@ def _bench_attention(add, r, att, ref, B: int, n: int, DB: int, ctx: int) -> Non
 
 
 def _bench_latent(add, r, m, B: int, n: int, DB: int, ctx: int) -> None:
-    T, h, D, width = B * n, m.heads, m.dim + m.rot_dim, (m.latent_size + 7) // 8 * 8
+    T, h, D, width = B * n, m.heads, m.dim + m.rot_dim, ops.latent_width(m.latent_size)
     per = (n + 15) // 16
     pages, bt = r(B * per, 16, width), torch.randperm(B * per, device="cuda").view(B, per).int()
     proj, nw = r(T, m.proj_size), r(m.kv_rank)
