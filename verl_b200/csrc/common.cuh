@@ -70,6 +70,13 @@ __device__ __forceinline__ void vb_jitter(uint32_t salt) {
 __device__ __forceinline__ void vb_jitter(uint32_t) {}
 #endif
 
+// True in one lane of the (converged) warp.
+__device__ __forceinline__ bool elect_one() {
+  uint32_t r;
+  asm volatile("{\n\t.reg .pred p;\n\telect.sync _|p, 0xffffffff;\n\tselp.u32 %0, 1, 0, p;\n\t}" : "=r"(r));
+  return r != 0;
+}
+
 // ---------------------------------------------------------------------------
 // Programmatic dependent launch. A kernel launched with the programmatic-serialization attribute may start while
 // its predecessor in the stream still runs: what it does before pdl_wait() (barrier init, TMEM allocation,

@@ -10,9 +10,8 @@
 //     O^T[rank x heads] += C^T[rank x 64 keys] . P           (M = 128 dims per block, N = 2 x heads)
 // A stage holds 64 whole rows and serves both products; a second one loads meanwhile. A row is wide, so one copy takes all
 // 64-column parts of eight rows: a stage is [8 groups][parts][8 rows x 128 bytes], and both products address it through the
-// strides of their descriptors. The M = 128 of the first product spans a pair of stages; the half of S^T that belongs to the
-// chunk is used (TMEM lanes 0..63 for even chunks, 64..127 for odd ones), the other half is never read. So warps 0-1 take
-// the softmax of even chunks and warps 2-3 that of odd ones.
+// strides of their descriptors. (The tensor core reads the first operand of these narrow products slowly enough for its rows
+// to count: M = 64 for the scores. An accumulator of 64 rows lies in the first 16 lanes of each warp's 32.)
 // P is two bf16 terms (hi in the columns of the heads, lo behind them), so that the weights stay close to fp32; both land in
 // accumulators of their own and are added at the end. O^T accumulates in TMEM over all keys: a head's reference only moves
 // when its maximum has grown by more than 2^8, and every thread keeps the sum of its own keys' weights until the end.
@@ -166,7 +165,7 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
 }
 
 // ------------------------------------------------------------------------------------------------ attention on latents
-constexpr int LD_KEYS = 64, LD_THREADS = 192, LD_MAX_STAGES = 6, LD_MAX_PARTS = 10;
+constexpr int LD_KEYS = 64, LD_THREADS = 224, LD_MAX_STAGES = 6, LD_MAX_PARTS = 10;
 constexpr float LD_SLACK = 8.f;
 constexpr float LD_LOG2E = 1.4426950408889634f, LD_LN2 = 0.6931471805599453f;
 
@@ -238,7 +237,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
     }
     for (int i = 0; i < 2; ++i) {
       mbar_init(&s_full[i], 1);
-      mbar_init(&p_ready[i], 2);
+      mbar_init(&p_ready[i], 4);
       mbar_init(&o_full[i], 1);
     }
     *abort_flag = 0;
@@ -310,60 +309,59 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
       row = next;
     }
   } else if (warp == 5) {
-    // -------------------------------- MMA issuer --------------------------------
-    if (lane == 0 && n_chunks > 0) {
-      constexpr uint32_t idesc_qk = umma_idesc(1, 1, 0, 0, 128, HB);      // A = rows (K-major), B = Q^T (K-major)
-      constexpr uint32_t idesc_pv = umma_idesc(1, 1, 1, 0, 128, 2 * HB);  // A = rows (MN-major), B = P (K-major)
+    // -------------------------------- scores --------------------------------
+    // The products are small: issuing them takes longer than running them, so that scores and values have a warp each.
+    if (n_chunks > 0 && elect_one()) {
+      constexpr uint32_t idesc = umma_idesc(1, 1, 0, 0, LD_KEYS, HB);  // A = rows (K-major), B = Q^T (K-major)
       // descriptors of the first tiles; steps are added in units of 16 bytes
-      const uint32_t base = smem_u32(smem), group = parts * 1024, step = stage_bytes >> 4;
-      const uint64_t a_qk = umma_smem_desc(base, 16, group), b_qk = umma_smem_desc(smem_u32(q_s), 16, 1024);
-      const uint64_t a_pv = umma_smem_desc(base, 1024, group), b_pv = umma_smem_desc(smem_u32(p_s), 16, 1024);
-      auto wait = [&](uint64_t* bar, uint32_t parity, int code, int detail) -> bool {
-        if (!*abort_flag && mbar_wait(bar, parity)) return true;
-        report_error(p.status, code, detail);
-        *abort_flag = 1;
-        return false;
-      };
-      auto issue_qk = [&](int c) -> bool {
+      const uint64_t a0 = umma_smem_desc(smem_u32(smem), 16, parts * 1024), b0 = umma_smem_desc(smem_u32(q_s), 16, 1024);
+      for (int c = 0; c < n_chunks; ++c) {
         const int s = c % stages;
-        if (!wait(&full[s], (c / stages) & 1, ERR_WAIT_FULL, c)) return false;
+        // the rows are there, and the scores of chunk c - 2 have been read
+        if (*abort_flag || !mbar_wait(&full[s], (c / stages) & 1) || (c > 1 && !mbar_wait(&p_ready[c & 1], ((c >> 1) - 1) & 1))) {
+          report_error(p.status, ERR_WAIT_FULL, c);
+          *abort_flag = 1;
+          break;
+        }
         tc_fence_after();
-        const uint64_t a = a_qk + (uint64_t)(s & ~1) * step;  // the pair of stages
+        const uint64_t a = a0 + (uint64_t)s * (stage_bytes >> 4);
         const uint32_t d = tmem + (c & 1) * HB;
         for (int x = 0; x < parts; ++x) {
-          const uint64_t ax = a + x * 64, bx = b_qk + x * (HB * 8);
 #pragma unroll
-          for (int k = 0; k < 4; ++k) tc_mma_f16(d, ax + 2 * k, bx + 2 * k, idesc_qk, x != 0 || k != 0);
+          for (int k = 0; k < 4; ++k) tc_mma_f16(d, a + x * 64 + 2 * k, b0 + x * (HB * 8) + 2 * k, idesc, x != 0 || k != 0);
         }
         tc_commit(&s_full[c & 1]);
-        return true;
-      };
-      bool ok = issue_qk(0);
-      for (int c = 0; ok && c < n_chunks; ++c) {
-        const int s = c % stages, n = (c + 1) % stages;
-        // the next chunk's scores first if its rows are there, so that its softmax can begin; else this chunk's values, so
-        // that its stage can be loaded again
-        const bool more = c + 1 < n_chunks, early = more && mbar_try_wait(&full[n], ((c + 1) / stages) & 1);
-        if (early) ok = issue_qk(c + 1);
-        if (!ok || !wait(&p_ready[c & 1], (c >> 1) & 1, ERR_WAIT_TMEM_EMPTY, c)) break;
+      }
+    }
+  } else if (warp == 6) {
+    // -------------------------------- values --------------------------------
+    if (n_chunks > 0 && elect_one()) {
+      constexpr uint32_t idesc = umma_idesc(1, 1, 1, 0, 128, 2 * HB);  // A = rows (MN-major), B = P (K-major)
+      const uint32_t group = parts * 64;                               // 16-byte units from one group of rows to the next
+      const uint64_t a0 = umma_smem_desc(smem_u32(smem), 1024, parts * 1024), b0 = umma_smem_desc(smem_u32(p_s), 16, 1024);
+      for (int c = 0; c < n_chunks; ++c) {
+        const int s = c % stages;
+        if (*abort_flag || !mbar_wait(&p_ready[c & 1], (c >> 1) & 1)) {
+          report_error(p.status, ERR_WAIT_TMEM_EMPTY, c);
+          *abort_flag = 1;
+          break;
+        }
         tc_fence_after();
-        const uint64_t a = a_pv + (uint64_t)s * step, bp = b_pv + (c & 1) * (LdCfg<HB>::P_BYTES >> 4);
+        const uint64_t a = a0 + (uint64_t)s * (stage_bytes >> 4), bp = b0 + (c & 1) * (LdCfg<HB>::P_BYTES >> 4);
         for (int v = 0; v < v_blocks; ++v) {
-          const uint32_t d = tmem + 2 * HB + v * 2 * HB;
 #pragma unroll
           for (int k = 0; k < LD_KEYS / 16; ++k)  // 16 keys: two groups of rows
-            tc_mma_f16(d, a + v * 128 + k * 2 * (group >> 4), bp + 2 * k, idesc_pv, c != 0 || k != 0);
+            tc_mma_f16(tmem + 2 * HB + v * 2 * HB, a + v * 128 + k * 2 * group, bp + 2 * k, idesc, c != 0 || k != 0);
         }
         tc_commit(&empty[s]);
         tc_commit(&o_full[c & 1]);
-        if (more && !early) ok = issue_qk(c + 1);
       }
     }
   } else {
     // ----------------------- softmax (thread = key), then output (thread = dim) -----------------------
     const uint32_t lanes = ((uint32_t)(warp * 32)) << 16, s_addr = tmem + lanes, o_addr = s_addr + 2 * HB;
     const float scale2 = p.scale * LD_LOG2E;
-    const int key = tid & 63;
+    const int key = warp * 16 + lane;  // of the chunk: lanes 0..15
     float ref[HB], sum[HB];  // of all keys: the reference; of this thread's keys: the sum of weights
 #pragma unroll
     for (int g = 0; g < HB; ++g) {
@@ -372,30 +370,25 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
     }
     bool ok = true;
     for (int c = 0; c < n_chunks; ++c) {
-      const bool mine = (warp >> 1) == (c & 1);
-      // stages come in pairs: an even chunk is in lanes 0..63, an odd one in lanes 64..127
+      // P of chunk c - 2 was read by its product
+      if (*abort_flag || !mbar_wait(&s_full[c & 1], (c >> 1) & 1) || (c > 1 && !mbar_wait(&o_full[c & 1], ((c >> 1) - 1) & 1))) {
+        report_error(p.status, ERR_WAIT_TMEM_FULL, c);
+        *abort_flag = 1;
+        ok = false;
+      }
+      ok = __all_sync(0xffffffffu, ok);  // the lanes of a warp share its TMEM accesses
       float sc[HB];
       bool grown = false;
-      if (mine) {
-        // P of chunk c - 2 was read by its product
-        if (*abort_flag || !mbar_wait(&s_full[c & 1], (c >> 1) & 1) ||
-            (c > 1 && !mbar_wait(&o_full[c & 1], ((c >> 1) - 1) & 1))) {
-          report_error(p.status, ERR_WAIT_TMEM_FULL, c);
-          *abort_flag = 1;
-          ok = false;
-        }
-        ok = __all_sync(0xffffffffu, ok);  // the lanes of a warp share its TMEM accesses
-        if (ok) {
-          tc_fence_after();
-          uint32_t v[HB];
-          ld_cols<HB>(s_addr + (c & 1) * HB, v);
-          tmem_ld_wait();
-          const bool valid = (c_begin + c) * LD_KEYS + key < len;
+      if (ok) {
+        tc_fence_after();
+        uint32_t v[HB];
+        ld_cols<HB>(s_addr + (c & 1) * HB, v);
+        tmem_ld_wait();
+        const bool valid = lane < 16 && (c_begin + c) * LD_KEYS + key < len;
 #pragma unroll
-          for (int g = 0; g < HB; ++g) {
-            sc[g] = valid ? __uint_as_float(v[g]) * scale2 : -INFINITY;
-            grown |= sc[g] > ref[g] + LD_SLACK;
-          }
+        for (int g = 0; g < HB; ++g) {
+          sc[g] = valid ? __uint_as_float(v[g]) * scale2 : -INFINITY;
+          grown |= sc[g] > ref[g] + LD_SLACK;
         }
       }
       if (ld_bar_or(grown || !ok)) {  // rare after the first chunk: move the references that were outgrown
@@ -409,17 +402,15 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
         if (!ok) break;
         tc_fence_after();
         float alpha[HB];
-        if (mine) {
 #pragma unroll
-          for (int g = 0; g < HB; ++g) {
-            const float wm = warp_reduce_max(sc[g]);
-            if (lane == 0) red_s[g][warp & 1] = wm;
-          }
+        for (int g = 0; g < HB; ++g) {
+          const float wm = warp_reduce_max(sc[g]);
+          if (lane == 0) red_s[g][warp] = wm;
         }
         ld_bar();
 #pragma unroll
         for (int g = 0; g < HB; ++g) {
-          const float m = fmaxf(red_s[g][0], red_s[g][1]);
+          const float m = fmaxf(fmaxf(red_s[g][0], red_s[g][1]), fmaxf(red_s[g][2], red_s[g][3]));
           const bool move = m > ref[g] + LD_SLACK;
           alpha[g] = move ? exp2f(ref[g] - m) : 1.f;  // exp2(-inf) = 0: nothing seen before
           sum[g] *= alpha[g];
@@ -441,17 +432,18 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
         ld_bar();  // every lane's part of O is in place before the weights are handed over; red_s is free again
         tc_fence_after();
       }
-      if (!mine) continue;
-      uint8_t* pbuf = p_s + (c & 1) * LdCfg<HB>::P_BYTES + (key & 7) * 2;
-      const uint32_t c16 = key >> 3;
+      if (lane < 16) {
+        uint8_t* pbuf = p_s + (c & 1) * LdCfg<HB>::P_BYTES + (key & 7) * 2;
+        const uint32_t c16 = key >> 3;
 #pragma unroll
-      for (int g = 0; g < HB; ++g) {
-        const float w = exp2f(sc[g] - ref[g]);
-        sum[g] += w;
-        const __nv_bfloat16 hi = __float2bfloat16(w);
-        const uint32_t off = (g >> 3) * 1024 + (g & 7) * 128 + ((c16 ^ (g & 7)) << 4);
-        *reinterpret_cast<__nv_bfloat16*>(pbuf + off) = hi;
-        *reinterpret_cast<__nv_bfloat16*>(pbuf + off + HB * 128) = __float2bfloat16(w - __bfloat162float(hi));
+        for (int g = 0; g < HB; ++g) {
+          const float w = exp2f(sc[g] - ref[g]);
+          sum[g] += w;
+          const __nv_bfloat16 hi = __float2bfloat16(w);
+          const uint32_t off = (g >> 3) * 1024 + (g & 7) * 128 + ((c16 ^ (g & 7)) << 4);
+          *reinterpret_cast<__nv_bfloat16*>(pbuf + off) = hi;
+          *reinterpret_cast<__nv_bfloat16*>(pbuf + off + HB * 128) = __float2bfloat16(w - __bfloat162float(hi));
+        }
       }
       fence_proxy_async_smem();
       tc_fence_before();
@@ -554,10 +546,10 @@ extern "C" int vb_head_gemm(const void* a, long long a_t, long long a_h, const v
 }
 
 static inline int ld_heads(int H) { return H <= 16 ? 16 : 32; }
-// Stages (an even number: they are used in pairs) that fit beside Q and P; 0: none.
+// Stages that fit beside Q and P.
 static int ld_stages(int hb, int parts) {
   int s = LD_MAX_STAGES;
-  while (s > 0 && (hb == 32 ? LdCfg<32>::bytes(s, parts) : LdCfg<16>::bytes(s, parts)) > 227 * 1024) s -= 2;
+  while (s > 0 && (hb == 32 ? LdCfg<32>::bytes(s, parts) : LdCfg<16>::bytes(s, parts)) > 227 * 1024) --s;
   return s;
 }
 
