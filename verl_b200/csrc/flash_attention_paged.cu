@@ -117,7 +117,7 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
 
   if (warp == 4) {
     // ------------------------------- TMA producer -------------------------------
-    if (lane == 0) {
+    if (elect_one()) {
       tma_prefetch_desc(&tmQ);
       tma_prefetch_desc(&tmK);
       tma_prefetch_desc(&tmV);
@@ -157,7 +157,7 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     }
   } else if (warp == 5) {
     // -------------------------------- MMA issuer --------------------------------
-    if (lane == 0) {
+    if (elect_one()) {
       const uint32_t idesc_qk = umma_idesc(1, 1, 0, 0, PF_M, PF_N);
       const uint32_t idesc_pv = umma_idesc(1, 1, 0, 1, PF_M, (uint32_t)((p.Dv + 15) / 16 * 16));
       const uint32_t q_addr = smem_u32(smem), k_addr = q_addr + Cfg::K_OFF, v_addr = q_addr + Cfg::V_OFF;
@@ -206,6 +206,16 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     // soft cap, in log2 units: cap tanh(z) = cap - 2 cap / (1 + e^(2 z)), z = score / cap
     const float cap2 = p.softcap * LOG2E, cap_k = soft ? 2.f * LOG2E * p.scale / p.softcap : 0.f;
     auto capped = [&](float raw) { return cap2 - __fdividef(2.f * cap2, 1.f + exp2f(raw * cap_k)); };
+    // The same for |z| <= 0.7 without the special-function unit, which the exponentials keep busy: an odd polynomial fitted to
+    // tanh there (largest error 1e-7). Its coefficients carry cap and scale; they need a range in which z^9 does not underflow.
+    const float zs = soft ? p.scale / p.softcap : 0.f, z2 = zs * zs;
+    const bool poly_ok = soft && zs > 1e-3f && zs < 1e3f;
+    const float k0c = 0.999998495f * cap2 * zs, k1c = -0.33326973f * cap2 * zs * z2, k2c = 0.132574543f * cap2 * zs * z2 * z2,
+                k3c = -0.0501952428f * cap2 * zs * z2 * z2 * z2, k4c = 0.0131941733f * cap2 * zs * z2 * z2 * z2 * z2;
+    auto capped_small = [&](float raw) {
+      const float t = raw * raw;
+      return raw * fmaf(t, fmaf(t, fmaf(t, fmaf(t, k4c, k3c), k2c), k1c), k0c);
+    };
     const int sat = biased ? p.bias_len - 1 : 0;
     const float bias_far = biased ? bias_s[sat] : 0.f;
     // the sink is a key without a value: its weight starts the denominator
@@ -235,6 +245,7 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       }
       // pass 1: row maximum. Blocks with masks or table distances leave their final scores in place of the raw ones.
       float cmax = -INFINITY;
+      uint32_t small = 0;  // bit j: every score of the warp's block takes the polynomial
 #pragma unroll 1
       for (int j = 0; j < GROUPS; ++j) {
         if (none >> j & 1) continue;
@@ -246,7 +257,16 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
 #pragma unroll
           for (int e = 0; e < 32; ++e) mx[e & 3] = fmaxf(mx[e & 3], __uint_as_float(v[e]));
           const float top = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
-          cmax = fmaxf(cmax, soft ? capped(top) : fmaf(top, scale2, bias_far));
+          if (soft) {
+            float low[4] = {INFINITY, INFINITY, INFINITY, INFINITY};
+#pragma unroll
+            for (int e = 0; e < 32; ++e) low[e & 3] = fminf(low[e & 3], __uint_as_float(v[e]));
+            const float far = fmaxf(fabsf(top), fabsf(fminf(fminf(low[0], low[1]), fminf(low[2], low[3]))));
+            small |= (uint32_t)__all_sync(0xffffffffu, poly_ok && far * zs <= 0.7f) << j;
+            cmax = fmaxf(cmax, capped(top));
+          } else {
+            cmax = fmaxf(cmax, fmaf(top, scale2, bias_far));
+          }
         } else {
           const int k0 = c0 + j * 32, dist0 = qpos - k0;
           const int kp = keep - k0;
@@ -298,7 +318,10 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
           const float a = pl && !soft ? scale2 : 1.f, bb = pl ? bias_far - ref : -ref;
           tmem_ld_32x32(s_addr + j * 32, v);
           tmem_ld_wait();
-          if (pl && soft) {
+          if (small >> j & 1) {
+#pragma unroll
+            for (int e = 0; e < 32; ++e) v[e] = __float_as_uint(capped_small(__uint_as_float(v[e])));
+          } else if (pl && soft) {
 #pragma unroll
             for (int e = 0; e < 32; ++e) v[e] = __float_as_uint(capped(__uint_as_float(v[e])));
           }

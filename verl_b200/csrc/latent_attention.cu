@@ -72,7 +72,7 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
   pdl_wait();
 
   if (warp == 4) {
-    if (lane == 0) {
+    if (elect_one()) {
       for (int k = 0; k < steps; ++k) {
         const int s = k % HG_STAGES;
         if (*abort_flag || !mbar_wait(&empty[s], ((k / HG_STAGES) & 1) ^ 1)) {
@@ -88,7 +88,7 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
       }
     }
   } else if (warp == 5) {
-    if (lane == 0) {
+    if (elect_one()) {
       const uint32_t idesc = umma_idesc(1, 1, 0, p.b_mn ? 1 : 0, 128, 64), base = smem_u32(smem);
       for (int k = 0; k < steps; ++k) {
         const int s = k % HG_STAGES;

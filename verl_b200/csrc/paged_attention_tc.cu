@@ -216,7 +216,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
     }
   } else if (warp == 5) {
     // -------------------------------- MMA issuer --------------------------------
-    if (lane == 0 && n_chunks > 0) {
+    if (n_chunks > 0 && elect_one()) {
       constexpr uint32_t idesc_qk = umma_idesc(1, 1, 0, 0, 128, TC_NH);  // A = K (K-major), B = Q^T (K-major)
       constexpr uint32_t idesc_pv = umma_idesc(1, 1, 1, 0, 128, TC_NH);  // A = V (MN-major), B = P^T (K-major)
       const uint32_t q_addr = smem_u32(q_s);
@@ -562,7 +562,7 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
     }
   } else if (warp == 5) {
     // -------------------------------- MMA issuer --------------------------------
-    if (lane == 0) {
+    if (elect_one()) {
       constexpr uint32_t idesc_qk = umma_idesc(1, 1, 0, 0, 128, TC_NH);
       constexpr uint32_t idesc_pv = umma_idesc(1, 1, 1, 0, 128, TC_NH);
       uint32_t tg = 0, cg = 0, ig = 0;
