@@ -219,7 +219,7 @@ class ModelConfig:
         kw = {k: int(d[k]) for k in ("bos_token_id", "eos_token_id", "pad_token_id") if d.get(k) is not None}
         kw.setdefault("eos_token_id", None)
         known = ("architecture", "vocab", "width", "layers", "norm", "embedding", "logit_scale", *kw)
-        return cls(model_type=model_type, logit_scale=float(d["logit_scale"]) if design.logit_scale else 1.0, vocab_size=int(d["vocab"]), hidden_size=int(d["width"]),
+        return cls(model_type=model_type, logit_scale=float(d.get("logit_scale", 1.0)) if design.logit_scale else 1.0, vocab_size=int(d["vocab"]), hidden_size=int(d["width"]),
                    intermediate_size=max([s.mlp.ff for s in specs if s.mlp] or [0]),
                    num_attention_heads=max([a.heads for a in att] or [1]),
                    num_key_value_heads=max([a.kv_heads for a in att] or [1]), head_dim=max([a.dim for a in att] or [1]),
