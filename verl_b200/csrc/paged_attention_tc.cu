@@ -638,14 +638,15 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
     }
   } else {
     // ----------------------- softmax + accumulation (128 threads) -----------------------
+    constexpr int NG = EXT ? TC_NH / 2 : TC_NH;  // query heads per KV head at most
     const uint32_t lane_base = ((uint32_t)(warp * 32)) << 16;
     bool ok = true;
     uint32_t cg = 0;
     for (int item = blockIdx.x; ok && item < num_items; item += gridDim.x) {
       const TcItem it = tc_item<EXT>(p, item);
-      float m_run[TC_NH], l_run[TC_NH], o_acc[TC_NH];
+      float m_run[NG], l_run[NG], o_acc[NG];
 #pragma unroll
-      for (int g = 0; g < TC_NH; ++g) {
+      for (int g = 0; g < NG; ++g) {
         m_run[g] = -INFINITY;
         l_run[g] = 0.f;
         o_acc[g] = 0.f;
@@ -656,9 +657,9 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
         }
       }
       const int first = EXT ? tc_first_key(p, it.seq_len) : 0;
-      float alpha_cur[TC_NH], alpha_nxt[TC_NH];
+      float alpha_cur[NG], alpha_nxt[NG];
       const uint32_t cg0 = cg;
-      auto softmax_chunk = [&](int c, float (&alpha)[TC_NH]) {
+      auto softmax_chunk = [&](int c, float (&alpha)[NG]) {
         const uint32_t cc = cg0 + c;
         const int i = cc & 1;
         if (*abort_flag || !mbar_wait(&s_full[i], (cc >> 1) & 1)) {
@@ -681,9 +682,9 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
         const float* brow = EXT && p.bias != nullptr
                                 ? p.bias + (long long)it.h * G * p.bias_len + max(min(dist, p.bias_len - 1), 0)
                                 : nullptr;
-        float sc[TC_NH];
+        float sc[NG];
 #pragma unroll
-        for (int g = 0; g < TC_NH; ++g) {
+        for (int g = 0; g < NG; ++g) {
           sc[g] = valid ? __uint_as_float(sr[g]) * p.scale : -INFINITY;
           // cap tanh(s / cap) = cap - 2 cap / (1 + e^(2 s / cap))
           if (EXT && p.softcap > 0.f && g < G && valid)
@@ -697,7 +698,7 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
         bar_sync_128();
         uint8_t* pbuf = p_s + i * P_BYTES;
 #pragma unroll
-        for (int g = 0; g < TC_NH; ++g) {
+        for (int g = 0; g < NG; ++g) {
           alpha[g] = 1.f;
           if (g < G) {
             const float cm = fmaxf(fmaxf(red_s[g][0], red_s[g][1]), fmaxf(red_s[g][2], red_s[g][3]));
@@ -720,7 +721,7 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
         if (lane == 0) mbar_arrive(&p_ready[i]);
         bar_sync_128();
 #pragma unroll
-        for (int g = 0; g < TC_NH; ++g)
+        for (int g = 0; g < NG; ++g)
           if (g < G) l_run[g] = l_run[g] * alpha[g] + red2_s[g][0] + red2_s[g][1] + red2_s[g][2] + red2_s[g][3];
       };
       if (it.n_chunks > 0) {
@@ -742,7 +743,7 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
           tmem_ld_32x16(tmem_base + lane_base + 32 + i * TC_NH, orr);
           tmem_ld_wait();
 #pragma unroll
-          for (int g = 0; g < TC_NH; ++g) {
+          for (int g = 0; g < NG; ++g) {
             if (g >= G) continue;
             float x = __uint_as_float(orr[g]);
             if (EXT) {
@@ -754,14 +755,14 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
           }
         }
 #pragma unroll
-        for (int g = 0; g < TC_NH; ++g) alpha_cur[g] = alpha_nxt[g];
+        for (int g = 0; g < NG; ++g) alpha_cur[g] = alpha_nxt[g];
         ok = bar_and_128(ok);
       }
       cg += it.n_chunks;
       if (ok && tid < Dv) {
         const int d = tid;
 #pragma unroll
-        for (int g = 0; g < TC_NH; ++g) {
+        for (int g = 0; g < NG; ++g) {
           if (g < G) {
             const int hq = it.h * G + g;
             if (p.num_splits == 1) {
