@@ -201,7 +201,7 @@ def test_attention_small_scores_keep_their_differences():
     n, D = 260, 32
     q, k, v = rand(n, 2, D, seed=1, dtype=BF, scale=0.2), rand(n, 2, D, seed=2, dtype=BF, scale=0.2), rand(n, 2, D, seed=3, dtype=BF)
     kc, vc, bt = paged(k, v, 16)
-    for cap in (500.0, 50.0):
+    for cap in (500.0, 50.0, 4.0, 1.5):  # from far inside the cap to scores on both sides of it
         want = O.attend(q.float(), k.float(), v.float(), 3.0, O.causal_mask(n), cap).reshape(n, -1)
         for lo in (0, n - 1):
             close(ops.paged_attention(q[lo:].cuda(), kc, vc, bt, i32(0, n - lo), i32(n), n - lo, scale=3.0, softcap=cap),
