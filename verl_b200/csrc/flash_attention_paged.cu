@@ -128,7 +128,8 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       const int* bt = LATENT ? nullptr : p.block_table + (long long)b * p.max_blocks;
       const int ppc = LATENT ? 0 : PF_N / p.block_size;
       const int n_pages = LATENT ? 0 : (seq_len + p.block_size - 1) / p.block_size;
-      for (int t = 0; t < 2 * n_chunks; ++t) {
+      int t = 0;
+      for (; t < 2 * n_chunks; ++t) {
         const int s = t & 1;  // 0 = K, 1 = V
         if (*abort_flag || !mbar_wait(&empty[s], ((t >> 1) & 1) ^ 1)) {
           report_error(p.status, ERR_WAIT_EMPTY, t);
@@ -154,6 +155,9 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             tma_load_2d(dst + x * Cfg::KV_HALF + pg * p.block_size * 128, tm, &full[s], x * 64, row);
         }
       }
+      // no copy is in flight when the CTA ends, whatever ended it
+      mbar_wait(q_full, 0);
+      for (int i = max(t - 2, 0); i < t; ++i) mbar_wait(&full[i & 1], (i >> 1) & 1);
     }
   } else if (warp == 5) {
     // -------------------------------- MMA issuer --------------------------------

@@ -51,7 +51,7 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
   uint64_t *empty = full + HG_STAGES, *done = empty + HG_STAGES;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(done + 1);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int tid = threadIdx.x, warp = tid >> 5;
   const int h = blockIdx.y, m0 = blockIdx.z * 128, n0 = blockIdx.x * 64;
   const int steps = (p.K + 63) / 64;
 
@@ -73,7 +73,8 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
 
   if (warp == 4) {
     if (elect_one()) {
-      for (int k = 0; k < steps; ++k) {
+      int k = 0;
+      for (; k < steps; ++k) {
         const int s = k % HG_STAGES;
         if (*abort_flag || !mbar_wait(&empty[s], ((k / HG_STAGES) & 1) ^ 1)) {
           report_error(p.status, ERR_WAIT_EMPTY, k);
@@ -86,6 +87,7 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
         if (p.b_mn) tma_load_3d(dst + HG_A, &tmB, &full[s], n0, k * 64, h);
         else tma_load_3d(dst + HG_A, &tmB, &full[s], k * 64, n0, h);
       }
+      for (int i = max(k - HG_STAGES, 0); i < k; ++i) mbar_wait(&full[i % HG_STAGES], (i / HG_STAGES) & 1);  // none in flight
     }
   } else if (warp == 5) {
     if (elect_one()) {
@@ -291,6 +293,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
     };
     int row = n_chunks > 0 ? row_of(0) : 0;
     bool ok = true;
+    int issued = 0;
     for (int c = 0; ok && c < n_chunks; ++c) {
       const int s = c % stages, next = c + 1 < n_chunks ? row_of(c + 1) : 0;
       int good = 1;  // lane 0 decides for the warp: the lanes must leave the loop together
@@ -307,7 +310,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
       if (ok && lane < 8) tma_load_3d(smem + s * stage_bytes + lane * parts * 1024, &tmC, &full[s], 0, row, 0);
       __syncwarp();
       row = next;
+      issued += ok;
     }
+    // no copy is in flight when the CTA ends, whatever ended it
+    for (int i = max(issued - stages, 0); lane == 0 && i < issued; ++i) mbar_wait(&full[i % stages], (i / stages) & 1);
   } else if (warp == 5) {
     // -------------------------------- scores --------------------------------
     // The products are small: issuing them takes longer than running them, so that scores and values have a warp each.
