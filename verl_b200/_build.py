@@ -10,6 +10,7 @@ nvcc cross-compiles without a GPU, so this also runs on a CPU-only machine.
 
 from __future__ import annotations
 
+import fcntl
 import hashlib
 import os
 import shutil
@@ -112,17 +113,25 @@ def build(force: bool = False, verbose: bool = False, ptxas_verbose: bool = Fals
     if force:
         for f in obj_dir.glob("*.sha1"):
             f.unlink()
+    with open(obj_dir / ".lock", "w") as lock:  # processes that start together build one after the other
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return _build_locked(obj_dir, out, force, verbose, ptxas_verbose, flavour)
+
+
+def _build_locked(obj_dir: Path, out: Path, force: bool, verbose: bool, ptxas_verbose: bool, flavour: str) -> Path:
     cu, cpp = _sources()
     with ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 4)) as ex:
         objs = list(ex.map(lambda s: _compile_one(s, verbose, ptxas_verbose, flavour), cu + cpp))
     newest = max(o.stat().st_mtime for o in objs)
     if force or not out.exists() or out.stat().st_mtime < newest:
-        cmd = [_nvcc(), "-shared", "-o", str(out), *map(str, objs), "-lcudart", "-lpthread"]
+        part = out.with_suffix(".part")  # a library that exists is whole
+        cmd = [_nvcc(), "-shared", "-o", str(part), *map(str, objs), "-lcudart", "-lpthread"]
         if verbose:
             print(" ".join(cmd), flush=True)
         res = subprocess.run(cmd, capture_output=True, text=True)
         if res.returncode != 0:
             raise RuntimeError(f"link failed\n{res.stdout}\n{res.stderr}")
+        os.replace(part, out)
     return out
 
 
