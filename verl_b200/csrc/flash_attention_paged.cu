@@ -15,7 +15,8 @@
 // or outside the mask get weight zero. Masks and the bias table are looked at only by the 32 x 32 blocks they reach.
 // The LATENT variant serves latent attention: keys and values of all heads lie expanded in rows of scratch memory, sequence
 // after sequence, and a key is two parts: the head's own and the rotated one that all heads share. Its three 64-column parts
-// of Q and K leave room for two CTAs per SM with 64 keys a block.
+// of Q and K leave room for two CTAs per SM with 64 keys a block. Its contexts may start where the first query's window does:
+// only distances count.
 // Every wait is bounded; on expiry the status word is set and the CTA leaves through its teardown.
 #include "common.cuh"
 #include "host_utils.h"
@@ -48,8 +49,9 @@ struct PagedFlashParams {
   int max_blocks, Hq, Hk, D, Dv, block_size, window, keep_first, chunk, bias_len, max_qblocks;
   float scale, softcap;
   const float* sink;            // [Hq] or null
-  const __nv_bfloat16* gate;    // [T, Hq * Dv] or null
+  const __nv_bfloat16* gate;    // [T, Hq * Dv] (gate_w 1: [T, Hq]) or null
   long long gate_stride;
+  int gate_w;
   int* status;
   // LATENT only: D = the heads' own part of a key; contexts of the sequences in the expanded rows
   int rot;
@@ -86,10 +88,10 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   const int seq_len = LATENT ? p.ctx_cu[b + 1] - ctx0 : p.seq_lens[b];
   const int pos0 = seq_len - n_q + r0;                     // position of row 0
   const int pos1 = min(pos0 + PF_M, seq_len) - 1;          // last real row
-  const bool windowed = !LATENT && (p.window > 0 || p.chunk > 0);
+  const bool windowed = p.window > 0 || (!LATENT && p.chunk > 0);
   const int keep = !LATENT && p.window > 0 ? p.keep_first : 0;
   // first key that a query at position i sees, kept ones apart
-  auto first_key = [&](int i) { return p.window > 0 ? i - p.window + 1 : i - i % p.chunk; };
+  auto first_key = [&](int i) { return LATENT || p.window > 0 ? i - p.window + 1 : i - i % p.chunk; };
   // chunks to visit: [0, keep_chunks) and [win_chunk, last_chunk]
   const int last_chunk = pos1 / PF_N;
   const int keep_chunks = min((keep + PF_N - 1) / PF_N, last_chunk + 1);
@@ -223,7 +225,7 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     const int sat = biased ? p.bias_len - 1 : 0;
     const float bias_far = biased ? bias_s[sat] : 0.f;
     // the sink is a key without a value: its weight starts the denominator
-    const bool sunk = !LATENT && p.sink != nullptr;
+    const bool sunk = p.sink != nullptr;
     float m_ref = sunk ? p.sink[hq] * LOG2E : -INFINITY, l_run = sunk ? 1.f : 0.f;
     const int first = windowed ? first_key(qpos) : 0, first_lo = windowed ? first_key(qw) : 0,
               first_hi = windowed ? first_key(qw + 31) : 0;
@@ -357,9 +359,11 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     ok = __all_sync(0xffffffffu, ok);
     if (ok) {
       tc_fence_after();
-      const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      if (p.gate && p.gate_w == 1 && r0 + r < n_q)  // one number for the head
+        inv = __fdividef(inv, 1.f + __expf(-__bfloat162float(p.gate[(long long)(q_first + r0 + r) * p.gate_stride + hq])));
       const __nv_bfloat16* gate =
-          p.gate ? p.gate + (long long)(q_first + r0 + r) * p.gate_stride + (long long)hq * p.Dv : nullptr;
+          p.gate && p.gate_w != 1 ? p.gate + (long long)(q_first + r0 + r) * p.gate_stride + (long long)hq * p.Dv : nullptr;
       __nv_bfloat16* dst = p.out + (long long)(q_first + r0 + r) * p.out_stride + (long long)hq * p.Dv;
 #pragma unroll 1
       for (int j = 0; j * 32 < p.Dv; ++j) {
@@ -446,6 +450,7 @@ extern "C" int vb_paged_flash(const void* q, long long q_stride, const void* kc,
   p.scale = scale; p.softcap = softcap; p.sink = sink;
   p.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
   p.gate_stride = gate_stride;
+  p.gate_w = 0;
   p.status = status;
   const dim3 grid(p.max_qblocks, Hq, B);
   cudaError_t e = vb_launch_pdl(paged_flash_kernel<false>, grid, dim3(PF_THREADS), (size_t)smem, stream, 1, tmQ, tmK, tmV, tmQ,
@@ -461,14 +466,17 @@ extern "C" int vb_latent_flash_supported(int H, int dim, int rot, int vdim, int 
 
 // q [T, H, dim + rot] bf16 (token stride q_stride); the contexts' rotated key parts [N, rot] (row stride rot_stride) and
 // expanded rows [N, H * dim keys | H * vdim values] (row stride kv_stride), sequence b from row ctx_cu[b]; its queries are
-// the rows cu_q[b] .. cu_q[b + 1] - 1 of q, the last positions of its context. out, gate as above.
+// the rows cu_q[b] .. cu_q[b + 1] - 1 of q, the last positions of its context. out, window, sink as above; gate_w: numbers of the
+// gate per head, vdim or 1.
 extern "C" int vb_latent_flash(const void* q, long long q_stride, int T, const void* rot_keys, long long rot_stride,
                                const void* kv, long long kv_stride, int N, const int* cu_q, const int* ctx_cu, int B, int max_q,
-                               int H, int dim, int rot, int vdim, float scale, const void* gate, long long gate_stride, void* out,
-                               long long out_stride, int* status, cudaStream_t stream) {
+                               int H, int dim, int rot, int vdim, float scale, int window, const float* sink, const void* gate,
+                               long long gate_stride, int gate_w, void* out, long long out_stride, int* status,
+                               cudaStream_t stream) {
   if (B <= 0 || T <= 0 || max_q <= 0 || N <= 0) return 0;
   if (!vb_latent_flash_supported(H, dim, rot, vdim, 8) || (q_stride & 7) || (rot_stride & 7) || (kv_stride & 7) ||
-      (out_stride & 7) || B > 65535 || (gate != nullptr && ((gate_stride & 7) || (reinterpret_cast<uintptr_t>(gate) & 15))))
+      (out_stride & 7) || B > 65535 || (gate != nullptr && gate_w != 1 && gate_w != vdim) ||
+      (gate != nullptr && gate_w != 1 && ((gate_stride & 7) || (reinterpret_cast<uintptr_t>(gate) & 15))))
     return -3;
   const __nv_bfloat16 *qb = reinterpret_cast<const __nv_bfloat16*>(q), *kb = reinterpret_cast<const __nv_bfloat16*>(kv);
   const uint64_t head = (uint64_t)(dim + rot) * 2, row = (uint64_t)kv_stride * 2;
@@ -492,9 +500,10 @@ extern "C" int vb_latent_flash(const void* q, long long q_stride, int T, const v
   p.out_stride = out_stride;
   p.Hq = H; p.Hk = H; p.D = dim; p.rot = rot; p.Dv = vdim;
   p.max_qblocks = (max_q + PF_M - 1) / PF_M;
-  p.scale = scale;
+  p.scale = scale; p.window = window; p.sink = sink;
   p.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
   p.gate_stride = gate_stride;
+  p.gate_w = gate_w;
   p.status = status;
   const dim3 grid(p.max_qblocks, H, B);
   cudaError_t e = vb_launch_pdl(paged_flash_kernel<true>, grid, dim3(PF_THREADS), (size_t)smem, stream, 1, tmQ, tmK, tmV, tmQr,

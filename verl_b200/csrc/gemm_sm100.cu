@@ -1369,15 +1369,15 @@ extern "C" int vb_gemm_rs_bf16(const void* A, const void* B, const void* bias, i
 //     b_mn = 0: B = [E, N, K], C[rows of e] = A . B[e]^T;  b_mn = 1: B = [E, K, N], C = A . B[e].
 //   mode 2 (weight gradients): A stored [P, M], B stored [P, N] (a_mn = b_mn = 1), C = [E, M, N] fp32,
 //     C[e] += A[rows of e]^T . B[rows of e]; expert_off[E + 1] are the padded row offsets (multiples of 128).
-// N (K for b_mn) must be a multiple of 64 in mode 1 so that a tile never reads the next expert's matrix into the
-// contraction; M, N arbitrary otherwise. Nothing is read back to the host: routing stays on the device.
+// In mode 1 with b_mn, K must be a multiple of 64 so that a tile never reads the next expert's matrix into the contraction
+// (without b_mn its rows only reach columns that are not stored); M, N arbitrary otherwise. Nothing is read back to the host: routing stays on the device.
 extern "C" int vb_grouped_gemm_bf16(const void* A, const void* B, void* C, int M, int N, int K, long long lda,
                                     long long ldb, long long ldc, int a_mn, int b_mn, int out_fp32, int accumulate,
                                     int mode, int E, const int* blk_expert, const int* expert_off, int* status,
                                     cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0 || E <= 0) return 0;
   if ((lda & 7) || (ldb & 7)) return -3;
-  if (mode == 1 && (a_mn || blk_expert == nullptr || (M % BM) != 0 || ((b_mn ? K : N) % 64) != 0)) return -3;
+  if (mode == 1 && (a_mn || blk_expert == nullptr || (M % BM) != 0 || (b_mn && (K % 64) != 0))) return -3;
   if (mode == 2 && (!a_mn || !b_mn || !out_fp32 || !accumulate || expert_off == nullptr)) return -3;
   if (mode != 1 && mode != 2) return -3;
   GemmParams p{};

@@ -4,58 +4,10 @@
 // 32-bit weights (and for shapes that TMA cannot describe), and a CUDA-core paged attention that takes any head size.
 //
 // Every kernel is a template over the activation type (bf16 when serving, fp32 for the exact mode); arithmetic is fp32.
-#include "common.cuh"
 #include "host_utils.h"
+#include "rowwise.cuh"
 
 namespace vb {
-
-template <typename T>
-__device__ __forceinline__ float to_f(T v);
-template <>
-__device__ __forceinline__ float to_f<float>(float v) { return v; }
-template <>
-__device__ __forceinline__ float to_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
-template <typename T>
-__device__ __forceinline__ T from_f(float v);
-template <>
-__device__ __forceinline__ float from_f<float>(float v) { return v; }
-template <>
-__device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
-
-// Eight consecutive elements (16-byte aligned).
-__device__ __forceinline__ void ld8(const __nv_bfloat16* p, float (&f)[8]) {
-  const uint4 raw = *reinterpret_cast<const uint4*>(p);
-  const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const float2 x = __bfloat1622float2(h[i]);
-    f[2 * i] = x.x;
-    f[2 * i + 1] = x.y;
-  }
-}
-__device__ __forceinline__ void ld8(const float* p, float (&f)[8]) {
-  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
-  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
-  f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
-}
-__device__ __forceinline__ void st8(__nv_bfloat16* p, const float (&f)[8]) {
-  *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]),
-                                            pack_bf16x2(f[6], f[7]));
-}
-__device__ __forceinline__ void st8(float* p, const float (&f)[8]) {
-  reinterpret_cast<float4*>(p)[0] = make_float4(f[0], f[1], f[2], f[3]);
-  reinterpret_cast<float4*>(p)[1] = make_float4(f[4], f[5], f[6], f[7]);
-}
-
-// Sum over the block, the same value in every thread. `sh` holds 32 floats.
-__device__ __forceinline__ float block_sum_all(float v, float* sh) {
-  v = warp_reduce_sum(v);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = (blockDim.x + 31) >> 5;
-  __syncthreads();
-  if (lane == 0) sh[warp] = v;
-  __syncthreads();
-  return warp_reduce_sum(lane < nw ? sh[lane] : 0.f);
-}
 
 // ---------------------------------------------------------------------------------------------------------------
 // res[t] = table[ids[t]] * scale, fp32; y (when given): the same in the table's type.
@@ -84,8 +36,26 @@ __global__ void embed_scaled_kernel(const long long* __restrict__ ids, const T* 
   }
 }
 
+// res[t] = table[ids[t]] / sqrt(mean of its squares + eps) * w, fp32.
+template <typename T>
+__global__ void embed_normed_kernel(const long long* __restrict__ ids, const T* __restrict__ table, const T* __restrict__ w,
+                                    float* __restrict__ res, int H, float eps) {
+  __shared__ float sh[32];
+  pdl_trigger();
+  pdl_wait();
+  const T* src = table + ids[blockIdx.x] * (long long)H;
+  float* dst = res + (long long)blockIdx.x * H;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    const float f = to_f<T>(src[i]);
+    ss += f * f;
+  }
+  const float inv = 1.f / sqrtf(block_sum_all(ss, sh) / (float)H + eps);
+  for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = to_f<T>(src[i]) * inv * to_f<T>(w[i]);
+}
+
 // ---------------------------------------------------------------------------------------------------------------
-// res += delta (when given); y = res / sqrt(mean(res^2) + eps) * w. The residual stays fp32 in global memory; the row is
+// res += delta (when given); y = res / sqrt(mean(res^2) + eps) * w, or without w the residual. The residual stays fp32 in global memory; the row is
 // kept in shared memory between the two passes.
 template <typename T>
 __global__ void add_rmsnorm_kernel(const T* __restrict__ delta, long long delta_stride, float* __restrict__ res,
@@ -125,20 +95,7 @@ __global__ void add_rmsnorm_kernel(const T* __restrict__ delta, long long delta_
       ss += f * f;
     }
   }
-  ss = block_sum_all(ss, sh);
-  const float inv = 1.f / sqrtf(ss / (float)H + eps);
-  if (vec) {
-    for (int v = threadIdx.x; v < (H >> 3); v += blockDim.x) {  // the same elements this thread has stored
-      float f[8], g[8];
-      ld8(row + v * 8, f);
-      ld8(w + v * 8, g);
-#pragma unroll
-      for (int i = 0; i < 8; ++i) f[i] = f[i] * inv * g[i];
-      st8(out + v * 8, f);
-    }
-  } else {
-    for (int i = threadIdx.x; i < H; i += blockDim.x) out[i] = from_f<T>(row[i] * inv * to_f<T>(w[i]));
-  }
+  norm_row_out(row, ss, w, out, H, eps, vec, sh);
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -223,18 +180,24 @@ struct ClampedGlu {
     return g / (1.f + expf(-alpha * g)) * (u + 1.f);
   }
 };
-// y = gelu(gate) * up with the tanh form of gelu: 0.5 g (1 + tanh(z)) = g sigmoid(2 z), z = sqrt(2 / pi) (g + 0.044715 g^3)
+// y = gelu(gate) * up with the tanh form of gelu
 template <typename T>
 struct GeluTanhGlu {
+  __device__ __forceinline__ float operator()(float g, float u) const { return gelu_tanh<sizeof(T) == 2>(g) * u; }
+};
+// y = silu(gate) * up
+template <typename T>
+struct SiluGlu {
   __device__ __forceinline__ float operator()(float g, float u) const {
-    const float z = 0.7978845608028654f * (g + 0.044715f * g * g * g);
-    if (sizeof(T) == 2) return __fdividef(g, 1.f + __expf(-2.f * z)) * u;
-    return 0.5f * g * (1.f + tanhf(z)) * u;
+    if (sizeof(T) == 2) return __fdividef(g, 1.f + __expf(-g)) * u;
+    return g / (1.f + expf(-g)) * u;
   }
 };
-template <typename T, typename Act>
+// ROUTED: rows of a buffer sorted by expert. Gate and up of a row are multiplied with its scale first (when given); blocks of 128
+// rows without an expert are left out.
+template <typename T, typename Act, bool ROUTED>
 __global__ void glu_kernel(const T* __restrict__ gu, long long stride, T* __restrict__ y, long long total, int F,
-                           const Act act) {
+                           const Act act, const float* __restrict__ row_scale, const int* __restrict__ blk_expert) {
   pdl_trigger();
   pdl_wait();
   const long long step = (long long)gridDim.x * blockDim.x;
@@ -243,19 +206,50 @@ __global__ void glu_kernel(const T* __restrict__ gu, long long stride, T* __rest
     for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total / 8; i += step) {
       const long long t = i / nv;
       const int c = (int)(i - t * nv) * 8;
+      if (ROUTED && blk_expert[t >> 7] < 0) continue;
+      const float w = ROUTED && row_scale ? row_scale[t] : 1.f;
       float g[8], u[8];
       ld8(gu + t * stride + c, g);
       ld8(gu + t * stride + F + c, u);
 #pragma unroll
-      for (int k = 0; k < 8; ++k) g[k] = act(g[k], u[k]);
+      for (int k = 0; k < 8; ++k) g[k] = ROUTED ? act(g[k] * w, u[k] * w) : act(g[k], u[k]);
       st8(y + t * F + c, g);
     }
   } else {
     for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += step) {
       const long long t = i / F;
       const int c = (int)(i - t * F);
-      y[i] = from_f<T>(act(to_f<T>(gu[t * stride + c]), to_f<T>(gu[t * stride + F + c])));
+      if (ROUTED && blk_expert[t >> 7] < 0) continue;
+      const float w = ROUTED && row_scale ? row_scale[t] : 1.f;
+      y[i] = from_f<T>(act(to_f<T>(gu[t * stride + c]) * w, to_f<T>(gu[t * stride + F + c]) * w));
     }
+  }
+}
+
+// y[t] = gelu(g[t]) * table[ids[t]][lo ..]. One block per token.
+template <typename T>
+__global__ void gelu_rows_kernel(const T* __restrict__ g, long long g_stride, const long long* __restrict__ ids,
+                                 const T* __restrict__ table, long long table_stride, int lo, T* __restrict__ y, int n) {
+  pdl_trigger();
+  pdl_wait();
+  const T* e = table + ids[blockIdx.x] * table_stride + lo;
+  for (int i = threadIdx.x; i < n; i += blockDim.x)
+    y[(long long)blockIdx.x * n + i] = from_f<T>(gelu_tanh<sizeof(T) == 2>(to_f<T>(g[blockIdx.x * g_stride + i])) * to_f<T>(e[i]));
+}
+
+// x = cap * tanh(x / cap)
+__global__ void softcap_kernel(float* __restrict__ x, long long n, float cap) {
+  pdl_trigger();
+  pdl_wait();
+  const long long step = (long long)gridDim.x * blockDim.x, i0 = blockIdx.x * (long long)blockDim.x + threadIdx.x;
+  if ((n & 3) == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0) {
+    for (long long i = i0; i < n / 4; i += step) {
+      float4 v = reinterpret_cast<float4*>(x)[i];
+      v = make_float4(cap * tanhf(v.x / cap), cap * tanhf(v.y / cap), cap * tanhf(v.z / cap), cap * tanhf(v.w / cap));
+      reinterpret_cast<float4*>(x)[i] = v;
+    }
+  } else {
+    for (long long i = i0; i < n; i += step) x[i] = cap * tanhf(x[i] / cap);
   }
 }
 
@@ -354,14 +348,15 @@ constexpr int ROT_MAX = 256;  // pairs of a rotation
 
 // One block per token. qkv row = [q (Hq * D) | k (Hk * D) | v (Hk * Dv) | ...]: every q and k head is divided by its root mean
 // square and multiplied by the weight of size D that all heads share (no weights: left as it is), then its first 2 * n_rot
-// dimensions turn. q in place; k and v go to the token's place in the paged caches (slot < 0: no write).
+// dimensions turn. q in place; k and v go to the token's place in the paged caches (slot < 0: no write). v_off: where the
+// values start in the row (at the keys themselves when those are the values; they are only read).
 // VEC: 8 elements per lane, `lanes` lanes per head (adjacent pairs only). Otherwise a warp per head with its row in shared memory.
 template <typename T, bool VEC>
 __global__ void head_norm_rope_kv_write_kernel(T* __restrict__ qkv, long long stride, const T* __restrict__ qw,
                                                const T* __restrict__ kw, const float* __restrict__ freqs, int n_rot,
                                                int interleaved, float amp, const long long* __restrict__ positions,
                                                const long long* __restrict__ slots, T* __restrict__ kc, T* __restrict__ vc,
-                                               int Hq, int Hk, int D, int Dv, int block_size, float eps, int lanes) {
+                                               int Hq, int Hk, int D, int Dv, int block_size, int v_off, float eps, int lanes) {
   __shared__ float2 cs[ROT_MAX];
   extern __shared__ float rows[];
   pdl_trigger();
@@ -439,7 +434,7 @@ __global__ void head_norm_rope_kv_write_kernel(T* __restrict__ qkv, long long st
     }
   }
   if (slot < 0) return;
-  const T* v = base + (long long)(Hq + Hk) * D;
+  const T* v = base + v_off;
   constexpr int W = VEC ? 8 : 1;
   for (int i = threadIdx.x * W; i < Hk * Dv; i += blockDim.x * W) {
     const int h = i / Dv, d = i - h * Dv;
@@ -454,46 +449,54 @@ __global__ void head_norm_rope_kv_write_kernel(T* __restrict__ qkv, long long st
   }
 }
 
-// One block per token. proj row = [q (H heads of dim + rot) | latent (rank) | rotated key (rot) | ...]: the rotated parts turn
-// (pair i = (i, i + rot / 2)), q in place; normed latent and rotated key go to the token's row of the pages.
+// Turns `rot` numbers at src into dst, the threads of the block together with `n` heads `stride` apart; pair i = (2 i, 2 i + 1) or
+// (i, i + rot / 2). VEC: eight numbers at a time.
 template <typename T, bool VEC>
-__global__ void latent_rope_write_kernel(T* __restrict__ proj, long long stride, const T* __restrict__ w,
-                                         const float* __restrict__ freqs, float amp, const long long* __restrict__ positions,
-                                         const long long* __restrict__ slots, T* __restrict__ pages, int width, int H, int dim,
-                                         int rot, int rank, float eps) {
-  __shared__ float2 cs[ROT_MAX];
-  __shared__ float sh[32];
-  pdl_trigger();
-  pdl_wait();
-  T* base = proj + (long long)blockIdx.x * stride;
-  const T* c = base + (long long)H * (dim + rot);
-  const long long slot = slots[blockIdx.x];
+__device__ __forceinline__ void turn_heads(const T* src, T* dst, int n, long long src_stride, long long dst_stride, int rot,
+                                           bool interleaved, const float2* cs) {
   const int half = rot >> 1;
-  constexpr int W = VEC ? 8 : 1;
-  rotation_table(cs, freqs, half, positions[blockIdx.x], amp);
-  float ss = 0.f;
-  for (int i = threadIdx.x * W; i < rank; i += blockDim.x * W) {
-    float f[W];
-    if constexpr (VEC) ld8(c + i, f); else f[0] = to_f<T>(c[i]);
+  if (interleaved) {
+    constexpr int P = VEC ? 4 : 1;  // pairs at a time
+    const int per = half / P;
+    for (int j = threadIdx.x; j < n * per; j += blockDim.x) {
+      const int h = j / per, i = (j - h * per) * P;
+      const T* from = src + h * src_stride + 2 * i;
+      T* to = dst + h * dst_stride + 2 * i;
+      float f[2 * P];
+      if constexpr (VEC) {
+        ld8(from, f);
+      } else {
+        f[0] = to_f<T>(from[0]);
+        f[1] = to_f<T>(from[1]);
+      }
 #pragma unroll
-    for (int e = 0; e < W; ++e) ss += f[e] * f[e];
+      for (int e = 0; e < P; ++e) {
+        const float2 k = cs[i + e];
+        const float u = f[2 * e], v = f[2 * e + 1];
+        f[2 * e] = u * k.x - v * k.y;
+        f[2 * e + 1] = v * k.x + u * k.y;
+      }
+      if constexpr (VEC) {
+        st8(to, f);
+      } else {
+        to[0] = from_f<T>(f[0]);
+        to[1] = from_f<T>(f[1]);
+      }
+    }
+    return;
   }
-  ss = block_sum_all(ss, sh);  // also orders the table before its readers
-  const float inv = 1.f / sqrtf(ss / (float)rank + eps);
-  T* dst = pages + slot * width;
-  // heads 0 .. H - 1: queries in place; head H: the key
-  for (int j = threadIdx.x; j < (H + 1) * (half / W); j += blockDim.x) {
+  constexpr int W = VEC ? 8 : 1;
+  for (int j = threadIdx.x; j < n * (half / W); j += blockDim.x) {
     const int h = j / (half / W), i = (j - h * (half / W)) * W;
-    const T* src = h < H ? base + (long long)h * (dim + rot) + dim : c + rank;
-    T* to = h < H ? base + (long long)h * (dim + rot) + dim : dst + rank;
-    if (h == H && slot < 0) continue;
+    const T* from = src + h * src_stride;
+    T* to = dst + h * dst_stride;
     float u[W], v[W], a[W], b[W];
     if constexpr (VEC) {
-      ld8(src + i, u);
-      ld8(src + half + i, v);
+      ld8(from + i, u);
+      ld8(from + half + i, v);
     } else {
-      u[0] = to_f<T>(src[i]);
-      v[0] = to_f<T>(src[half + i]);
+      u[0] = to_f<T>(from[i]);
+      v[0] = to_f<T>(from[half + i]);
     }
 #pragma unroll
     for (int e = 0; e < W; ++e) {
@@ -509,14 +512,27 @@ __global__ void latent_rope_write_kernel(T* __restrict__ proj, long long stride,
       to[half + i] = from_f<T>(b[0]);
     }
   }
-  if (slot < 0) return;
-  for (int i = threadIdx.x * W; i < rank; i += blockDim.x * W) {
+}
+
+// dst = src / sqrt(mean(src^2) + eps) * w over the block (dst may be src).
+template <typename T, bool VEC>
+__device__ __forceinline__ void norm_to(const T* src, T* dst, const T* __restrict__ w, int n, float eps, float* sh) {
+  constexpr int W = VEC ? 8 : 1;
+  float ss = 0.f;
+  for (int i = threadIdx.x * W; i < n; i += blockDim.x * W) {
+    float f[W];
+    if constexpr (VEC) ld8(src + i, f); else f[0] = to_f<T>(src[i]);
+#pragma unroll
+    for (int e = 0; e < W; ++e) ss += f[e] * f[e];
+  }
+  const float inv = 1.f / sqrtf(block_sum_all(ss, sh) / (float)n + eps);
+  for (int i = threadIdx.x * W; i < n; i += blockDim.x * W) {
     float f[W], g[W];
     if constexpr (VEC) {
-      ld8(c + i, f);
+      ld8(src + i, f);
       ld8(w + i, g);
     } else {
-      f[0] = to_f<T>(c[i]);
+      f[0] = to_f<T>(src[i]);
       g[0] = to_f<T>(w[i]);
     }
 #pragma unroll
@@ -525,9 +541,48 @@ __global__ void latent_rope_write_kernel(T* __restrict__ proj, long long stride,
   }
 }
 
-// rows[ctx_cu[b] + i] = page row of token i of sequence b, in 16-byte units. One warp per row.
+// One block per token. proj row = [q (H heads of dim + rot), or the queries' latent (q_rank) | latent (rank) | rotated key (rot)
+// | ...]: the rotated parts turn, q in place; normed latent and rotated key go to the token's row of the pages; the queries'
+// latent is normed in place.
+template <typename T, bool VEC>
+__global__ void latent_rope_write_kernel(T* __restrict__ proj, long long stride, const T* __restrict__ w,
+                                         const float* __restrict__ freqs, float amp, int interleaved,
+                                         const long long* __restrict__ positions, const long long* __restrict__ slots,
+                                         T* __restrict__ pages, int width, int H, int dim, int rot, int rank, int q_rank,
+                                         const T* __restrict__ qw, float eps) {
+  __shared__ float2 cs[ROT_MAX];
+  __shared__ float sh[32];
+  pdl_trigger();
+  pdl_wait();
+  T* base = proj + (long long)blockIdx.x * stride;
+  const T* c = base + (q_rank ? q_rank : H * (dim + rot));
+  const long long slot = slots[blockIdx.x];
+  rotation_table(cs, freqs, rot >> 1, positions[blockIdx.x], amp);
+  __syncthreads();
+  T* dst = pages + slot * width;
+  turn_heads<T, VEC>(base + dim, base + dim, H, dim + rot, dim + rot, rot, interleaved, cs);
+  if (slot >= 0) turn_heads<T, VEC>(c + rank, dst + rank, 1, 0, 0, rot, interleaved, cs);
+  if (q_rank) norm_to<T, VEC>(base, base, qw, q_rank, eps, sh);
+  if (slot >= 0) norm_to<T, VEC>(c, dst, w, rank, eps, sh);  // uniform for the block
+}
+
+// The rotated parts of q rows [H heads of dim + rot | ...] turn in place. One block per token.
+template <typename T, bool VEC>
+__global__ void rotate_tails_kernel(T* __restrict__ q, long long stride, const float* __restrict__ freqs, float amp,
+                                    int interleaved, const long long* __restrict__ positions, int H, int dim, int rot) {
+  __shared__ float2 cs[ROT_MAX];
+  pdl_trigger();
+  pdl_wait();
+  rotation_table(cs, freqs, rot >> 1, positions[blockIdx.x], amp);
+  __syncthreads();
+  T* base = q + (long long)blockIdx.x * stride + dim;
+  turn_heads<T, VEC>(base, base, H, dim + rot, dim + rot, rot, interleaved, cs);
+}
+
+// rows[ctx_cu[b] + i] = page row of token i of sequence b, counted from the first of its last ctx_cu[b + 1] - ctx_cu[b] tokens
+// (of seq_lens[b]; null: from its first token), in 16-byte units. One warp per row.
 __global__ void latent_gather_kernel(const uint4* __restrict__ pages, const int* __restrict__ block_table, int max_blocks,
-                                     const int* __restrict__ ctx_cu, uint4* __restrict__ rows, int total, int B, int units,
+                                     const int* __restrict__ ctx_cu, const int* __restrict__ seq_lens, uint4* __restrict__ rows, int total, int B, int units,
                                      int block_size) {
   pdl_trigger();
   pdl_wait();
@@ -538,17 +593,18 @@ __global__ void latent_gather_kernel(const uint4* __restrict__ pages, const int*
     const int mid = (lo + hi + 1) >> 1;
     if (ctx_cu[mid] <= r) lo = mid; else hi = mid - 1;
   }
-  const int i = r - ctx_cu[lo];
+  const int i = r - ctx_cu[lo] + (seq_lens ? seq_lens[lo] - (ctx_cu[lo + 1] - ctx_cu[lo]) : 0);
   const long long row = (long long)block_table[(long long)lo * max_blocks + i / block_size] * block_size + i % block_size;
   for (int u = lane; u < units; u += 32) rows[(long long)r * units + u] = pages[row * units + u];
 }
 
-// out[t, h, n] = sum_k a[t, h, k] b_h[k, n] for n < N (b_h stored [N, K], or [K, N] with b_mn), times sigmoid(gate[t, h * N + n]);
+// out[t, h, n] = sum_k a[t, h, k] b_h[k, n] for n < N (b_h stored [N, K], or [K, N] with b_mn), times sigmoid(gate[t, h * N + n])
+// (gate_w 1: sigmoid(gate[t, h]));
 // then `tail` elements copied from a[t, h, K ...], then zeros up to `width`. fp32 sums, one thread per element.
 template <typename T>
 __global__ void head_gemm_simt_kernel(const T* __restrict__ a, long long a_t, long long a_h, const T* __restrict__ b, int b_mn,
                                       T* __restrict__ out, long long o_t, long long o_h, const T* __restrict__ gate,
-                                      long long gate_stride, int K, int N, int tail, int width) {
+                                      long long gate_stride, int gate_w, int K, int N, int tail, int width) {
   pdl_trigger();
   pdl_wait();
   const int n = blockIdx.z * blockDim.x + threadIdx.x, h = blockIdx.y;
@@ -560,7 +616,7 @@ __global__ void head_gemm_simt_kernel(const T* __restrict__ a, long long a_t, lo
     const T* br = b + (long long)h * N * K + (b_mn ? n : (long long)n * K);
     const int step = b_mn ? N : 1;
     for (int k = 0; k < K; ++k) x = fmaf(to_f<T>(ar[k]), to_f<T>(br[(long long)k * step]), x);
-    if (gate) x /= 1.f + expf(-to_f<T>(gate[t * gate_stride + (long long)h * N + n]));
+    if (gate) x /= 1.f + expf(-to_f<T>(gate[t * gate_stride + (gate_w == 1 ? h : (long long)h * N + n)]));
   } else if (n < N + tail) {
     x = to_f<T>(ar[K + n - N]);
   }
@@ -568,15 +624,22 @@ __global__ void head_gemm_simt_kernel(const T* __restrict__ a, long long a_t, lo
 }
 
 // ---------------------------------------------------------------------------------------------------------------
-// C[M, N] = A[M, K] . B[N, K]^T (+ bias), fp32 accumulation on the CUDA cores. 64 x 64 tile, 4 x 4 per thread.
+// C[M, N] = A[M, K] . B[N, K]^T (+ bias), fp32 accumulation on the CUDA cores. 64 x 64 tile, 4 x 4 per thread. blk_expert (or
+// null): B = [experts, N, K], the rows of A belong to experts in blocks of 128 (< 0: skipped).
 template <typename TA, typename TC>
 __global__ void __launch_bounds__(256) gemm_simt_kernel(const TA* __restrict__ A, const TA* __restrict__ B,
                                                         TC* __restrict__ C, const TA* __restrict__ bias, int M, int N,
-                                                        int K, long long lda, long long ldb, long long ldc) {
+                                                        int K, long long lda, long long ldb, long long ldc,
+                                                        const int* __restrict__ blk_expert) {
   __shared__ float As[16][68], Bs[16][68];
   pdl_trigger();
   pdl_wait();
   const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+  if (blk_expert) {
+    const int e = blk_expert[m0 >> 7];
+    if (e < 0) return;
+    B += (long long)e * N * ldb;
+  }
   const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
   float acc[4][4] = {};
   for (int k0 = 0; k0 < K; k0 += 16) {
@@ -705,15 +768,6 @@ paged_attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ kc, const 
 using namespace vb;
 typedef __nv_bfloat16 bf16;
 
-#define VB_DONE(e)                                   \
-  do {                                               \
-    cudaError_t _r = (e);                            \
-    vb_count_launch();                               \
-    return _r != cudaSuccess ? (int)_r : (int)cudaGetLastError(); \
-  } while (0)
-
-static inline int row_threads(int n) { return n >= 2048 ? 256 : (n >= 1024 ? 128 : 64); }
-
 extern "C" int vb_embed_scaled(const long long* ids, const void* table, float* res, void* y, int T, int H, float scale,
                                int f32, cudaStream_t stream) {
   if (T <= 0) return 0;
@@ -742,15 +796,57 @@ extern "C" int vb_add_rmsnorm(const void* delta, long long delta_stride, float* 
                         (const bf16*)w, (bf16*)y, H, eps));
 }
 
-template <typename T, typename Act>
-static int launch_glu(const void* gu, long long stride, void* y, int T_, int F, const Act& act, cudaStream_t stream) {
+template <typename T, bool ROUTED = false, typename Act>
+static int launch_glu(const void* gu, long long stride, void* y, int T_, int F, const Act& act, cudaStream_t stream,
+                      const float* row_scale = nullptr, const int* blk_expert = nullptr) {
   if (T_ <= 0 || F <= 0) return 0;
   const long long total = (long long)T_ * F;
   long long blocks = (total / 8 + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   if (blocks < 1) blocks = 1;
-  VB_DONE(vb_launch_pdl(glu_kernel<T, Act>, dim3((unsigned)blocks), dim3(256), 0, stream, 1, (const T*)gu, stride, (T*)y, total,
-                        F, act));
+  VB_DONE(vb_launch_pdl(glu_kernel<T, Act, ROUTED>, dim3((unsigned)blocks), dim3(256), 0, stream, 1, (const T*)gu, stride,
+                        (T*)y, total, F, act, row_scale, blk_expert));
+}
+
+// blk_expert (T / 128 of them) or null: rows of a buffer sorted by expert; row_scale [T] or null: see glu_kernel.
+extern "C" int vb_silu_glu(const void* gu, long long stride, void* y, int T, int F, const float* row_scale,
+                           const int* blk_expert, int f32, cudaStream_t stream) {
+  if (blk_expert) {
+    if (f32) return launch_glu<float, true>(gu, stride, y, T, F, SiluGlu<float>{}, stream, row_scale, blk_expert);
+    return launch_glu<bf16, true>(gu, stride, y, T, F, SiluGlu<bf16>{}, stream, row_scale, blk_expert);
+  }
+  if (row_scale) return -3;
+  if (f32) return launch_glu<float>(gu, stride, y, T, F, SiluGlu<float>{}, stream);
+  return launch_glu<bf16>(gu, stride, y, T, F, SiluGlu<bf16>{}, stream);
+}
+
+// y [T, n] = gelu(g) * table[ids, lo .. lo + n)
+extern "C" int vb_gelu_rows(const void* g, long long g_stride, const long long* ids, const void* table, long long table_stride,
+                            int lo, void* y, int T, int n, int f32, cudaStream_t stream) {
+  if (T <= 0 || n <= 0) return 0;
+  const dim3 grid(T), b(n >= 128 ? 128 : 64);
+  if (f32)
+    VB_DONE(vb_launch_pdl(gelu_rows_kernel<float>, grid, b, 0, stream, 1, (const float*)g, g_stride, ids, (const float*)table,
+                          table_stride, lo, (float*)y, n));
+  VB_DONE(vb_launch_pdl(gelu_rows_kernel<bf16>, grid, b, 0, stream, 1, (const bf16*)g, g_stride, ids, (const bf16*)table,
+                        table_stride, lo, (bf16*)y, n));
+}
+
+extern "C" int vb_softcap(float* x, long long n, float cap, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (!(cap > 0.f)) return -3;
+  long long blocks = (n + 1023) / 1024;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  VB_DONE(vb_launch_pdl(softcap_kernel, dim3((unsigned)blocks), dim3(256), 0, stream, 1, x, n, cap));
+}
+
+extern "C" int vb_embed_normed(const long long* ids, const void* table, const void* w, float* res, int T, int H, float eps,
+                               int f32, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  const dim3 g(T), b(row_threads(H));
+  if (f32)
+    VB_DONE(vb_launch_pdl(embed_normed_kernel<float>, g, b, 0, stream, 1, ids, (const float*)table, (const float*)w, res, H, eps));
+  VB_DONE(vb_launch_pdl(embed_normed_kernel<bf16>, g, b, 0, stream, 1, ids, (const bf16*)table, (const bf16*)w, res, H, eps));
 }
 
 extern "C" int vb_clamped_glu(const void* gu, long long stride, void* y, int T, int F, float limit, float alpha, int f32,
@@ -812,12 +908,25 @@ extern "C" int vb_gemm_simt(const void* A, const void* B, void* C, const void* b
   const dim3 g((N + 63) / 64, (M + 63) / 64), b(256);
   if (a_f32)
     VB_DONE(vb_launch_pdl(gemm_simt_kernel<float, float>, g, b, 0, stream, 1, (const float*)A, (const float*)B, (float*)C,
-                          (const float*)bias, M, N, K, lda, ldb, ldc));
+                          (const float*)bias, M, N, K, lda, ldb, ldc, (const int*)nullptr));
   if (out_f32)
     VB_DONE(vb_launch_pdl(gemm_simt_kernel<bf16, float>, g, b, 0, stream, 1, (const bf16*)A, (const bf16*)B, (float*)C,
-                          (const bf16*)bias, M, N, K, lda, ldb, ldc));
+                          (const bf16*)bias, M, N, K, lda, ldb, ldc, (const int*)nullptr));
   VB_DONE(vb_launch_pdl(gemm_simt_kernel<bf16, bf16>, g, b, 0, stream, 1, (const bf16*)A, (const bf16*)B, (bf16*)C,
-                        (const bf16*)bias, M, N, K, lda, ldb, ldc));
+                        (const bf16*)bias, M, N, K, lda, ldb, ldc, (const int*)nullptr));
+}
+
+// C[rows of e] = A[rows of e] . B[e]^T, B [E, N, K]; M a multiple of 128, blk_expert [M / 128].
+extern "C" int vb_grouped_gemm_simt(const void* A, const void* B, void* C, int M, int N, int K, const int* blk_expert, int f32,
+                                    cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (K <= 0 || (M & 127) || M / 64 > 65535 || blk_expert == nullptr) return -3;
+  const dim3 g((N + 63) / 64, M / 64), b(256);
+  if (f32)
+    VB_DONE(vb_launch_pdl(gemm_simt_kernel<float, float>, g, b, 0, stream, 1, (const float*)A, (const float*)B, (float*)C,
+                          (const float*)nullptr, M, N, K, (long long)K, (long long)K, (long long)N, blk_expert));
+  VB_DONE(vb_launch_pdl(gemm_simt_kernel<bf16, bf16>, g, b, 0, stream, 1, (const bf16*)A, (const bf16*)B, (bf16*)C,
+                        (const bf16*)nullptr, M, N, K, (long long)K, (long long)K, (long long)N, blk_expert));
 }
 
 // Caches [NB, Hk, block_size, D] and [NB, Hk, block_size, v_width] (the first Dv elements of a row are the value).
@@ -849,12 +958,15 @@ extern "C" int vb_paged_attention_simt(const void* q, long long q_stride, const 
 #undef VB_PSA
 }
 
-// qw / kw null: no norm. freqs: n_rot fp32 angular frequencies (n_rot 0: no rotation).
+// qw / kw null: no norm. freqs: n_rot fp32 angular frequencies (n_rot 0: no rotation). key_values: no v in the row, the values
+// are the keys before norm and rotation.
 extern "C" int vb_head_norm_rope_kv_write(void* qkv, long long stride, const void* qw, const void* kw, const float* freqs,
                                           int n_rot, int interleaved, float amp, const long long* positions,
                                           const long long* slots, void* kc, void* vc, int T, int Hq, int Hk, int D, int Dv,
-                                          int block_size, float eps, int f32, cudaStream_t stream) {
+                                          int block_size, int key_values, float eps, int f32, cudaStream_t stream) {
   if (T <= 0) return 0;
+  if (key_values && D != Dv) return -3;
+  const int v_off = (key_values ? Hq : Hq + Hk) * D;
   if ((qw == nullptr) != (kw == nullptr) || n_rot < 0 || n_rot > ROT_MAX || 2 * n_rot > D || D > PS_MAX_D) return -3;
   const bool vec = (D & 7) == 0 && D <= 256 && (Dv & 7) == 0 && (stride & 7) == 0 && (interleaved || n_rot == 0) &&
                    (reinterpret_cast<uintptr_t>(qkv) & 15) == 0;
@@ -865,7 +977,7 @@ extern "C" int vb_head_norm_rope_kv_write(void* qkv, long long stride, const voi
 #define VB_HNR(TT, V)                                                                                                  \
   VB_DONE(vb_launch_pdl(head_norm_rope_kv_write_kernel<TT, V>, g, b, smem, stream, 1, (TT*)qkv, stride, (const TT*)qw, \
                         (const TT*)kw, freqs, n_rot, interleaved, amp, positions, slots, (TT*)kc, (TT*)vc, Hq, Hk, D, Dv, \
-                        block_size, eps, lanes))
+                        block_size, v_off, eps, lanes))
   if (f32) {
     if (vec) VB_HNR(float, true);
     VB_HNR(float, false);
@@ -875,17 +987,20 @@ extern "C" int vb_head_norm_rope_kv_write(void* qkv, long long stride, const voi
 #undef VB_HNR
 }
 
-extern "C" int vb_latent_rope_write(void* proj, long long stride, const void* w, const float* freqs, float amp,
+// q_rank > 0 (and H 0): the row starts with the latent of the queries, normed in place with qw.
+extern "C" int vb_latent_rope_write(void* proj, long long stride, const void* w, const float* freqs, float amp, int interleaved,
                                     const long long* positions, const long long* slots, void* pages, int width, int T, int H,
-                                    int dim, int rot, int rank, float eps, int f32, cudaStream_t stream) {
+                                    int dim, int rot, int rank, int q_rank, const void* qw, float eps, int f32,
+                                    cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (rot < 0 || (rot & 1) || rot > 2 * ROT_MAX || rank <= 0 || width < rank + rot) return -3;
-  const bool vec = (rot & 15) == 0 && (dim & 7) == 0 && (rank & 7) == 0 && (width & 7) == 0 && (stride & 7) == 0 &&
-                   (reinterpret_cast<uintptr_t>(proj) & 15) == 0;
+  if (rot < 0 || (rot & 1) || rot > 2 * ROT_MAX || rank <= 0 || width < rank + rot || (q_rank > 0 && (H != 0 || qw == nullptr)))
+    return -3;
+  const bool vec = (rot & (interleaved ? 7 : 15)) == 0 && (dim & 7) == 0 && (rank & 7) == 0 && (q_rank & 7) == 0 &&
+                   (width & 7) == 0 && (stride & 7) == 0 && (reinterpret_cast<uintptr_t>(proj) & 15) == 0;
   const dim3 g(T), b(128);
 #define VB_LRW(TT, V)                                                                                                  \
   VB_DONE(vb_launch_pdl(latent_rope_write_kernel<TT, V>, g, b, 0, stream, 1, (TT*)proj, stride, (const TT*)w, freqs, amp, \
-                        positions, slots, (TT*)pages, width, H, dim, rot, rank, eps))
+                        interleaved, positions, slots, (TT*)pages, width, H, dim, rot, rank, q_rank, (const TT*)qw, eps))
   if (f32) {
     if (vec) VB_LRW(float, true);
     VB_LRW(float, false);
@@ -895,24 +1010,42 @@ extern "C" int vb_latent_rope_write(void* proj, long long stride, const void* w,
 #undef VB_LRW
 }
 
+extern "C" int vb_rotate_tails(void* q, long long stride, const float* freqs, float amp, int interleaved,
+                               const long long* positions, int T, int H, int dim, int rot, int f32, cudaStream_t stream) {
+  if (T <= 0 || H <= 0 || rot == 0) return 0;
+  if (rot < 0 || (rot & 1) || rot > 2 * ROT_MAX) return -3;
+  const bool vec = (rot & (interleaved ? 7 : 15)) == 0 && (dim & 7) == 0 && (stride & 7) == 0 &&
+                   (reinterpret_cast<uintptr_t>(q) & 15) == 0;
+  const dim3 g(T), b(128);
+#define VB_RT(TT, V) \
+  VB_DONE(vb_launch_pdl(rotate_tails_kernel<TT, V>, g, b, 0, stream, 1, (TT*)q, stride, freqs, amp, interleaved, positions, H, dim, rot))
+  if (f32) {
+    if (vec) VB_RT(float, true);
+    VB_RT(float, false);
+  }
+  if (vec) VB_RT(bf16, true);
+  VB_RT(bf16, false);
+#undef VB_RT
+}
+
 // row_bytes: bytes of a page row, a multiple of 16.
-extern "C" int vb_latent_gather(const void* pages, const int* block_table, int max_blocks, const int* ctx_cu, void* rows,
-                                int total, int B, int row_bytes, int block_size, cudaStream_t stream) {
+extern "C" int vb_latent_gather(const void* pages, const int* block_table, int max_blocks, const int* ctx_cu,
+                                const int* seq_lens, void* rows, int total, int B, int row_bytes, int block_size, cudaStream_t stream) {
   if (total <= 0 || B <= 0) return 0;
   if (row_bytes & 15) return -3;
   VB_DONE(vb_launch_pdl(latent_gather_kernel, dim3((total + 7) / 8), dim3(256), 0, stream, 1, (const uint4*)pages, block_table,
-                        max_blocks, ctx_cu, (uint4*)rows, total, B, row_bytes / 16, block_size));
+                        max_blocks, ctx_cu, seq_lens, (uint4*)rows, total, B, row_bytes / 16, block_size));
 }
 
 extern "C" int vb_head_gemm_simt(const void* a, long long a_t, long long a_h, const void* b, int b_mn, void* out, long long o_t,
-                                 long long o_h, const void* gate, long long gate_stride, int T, int H, int K, int N, int tail,
-                                 int width, int f32, cudaStream_t stream) {
+                                 long long o_h, const void* gate, long long gate_stride, int gate_w, int T, int H, int K, int N,
+                                 int tail, int width, int f32, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (H <= 0 || H > 65535 || K <= 0 || width < N + tail) return -3;
   const dim3 g(T, H, (width + 127) / 128), blk(128);
   if (f32)
     VB_DONE(vb_launch_pdl(head_gemm_simt_kernel<float>, g, blk, 0, stream, 1, (const float*)a, a_t, a_h, (const float*)b, b_mn,
-                          (float*)out, o_t, o_h, (const float*)gate, gate_stride, K, N, tail, width));
+                          (float*)out, o_t, o_h, (const float*)gate, gate_stride, gate_w, K, N, tail, width));
   VB_DONE(vb_launch_pdl(head_gemm_simt_kernel<bf16>, g, blk, 0, stream, 1, (const bf16*)a, a_t, a_h, (const bf16*)b, b_mn,
-                        (bf16*)out, o_t, o_h, (const bf16*)gate, gate_stride, K, N, tail, width));
+                        (bf16*)out, o_t, o_h, (const bf16*)gate, gate_stride, gate_w, K, N, tail, width));
 }

@@ -37,9 +37,9 @@ struct HeadGemmParams {
   long long a_t, a_h;
   __nv_bfloat16* out;
   long long o_t, o_h;
-  const __nv_bfloat16* gate;  // [T, H * N] or null
+  const __nv_bfloat16* gate;  // [T, H * N] (gate_w 1: [T, H]) or null
   long long gate_stride;
-  int T, K, N, tail, width, b_mn;
+  int gate_w, T, K, N, tail, width, b_mn;
   int* status;
 };
 
@@ -121,6 +121,9 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
     if (ok) {
       tc_fence_after();
       __nv_bfloat16* dst = p.out + t * p.o_t + h * p.o_h;
+      float head_gate = 1.f;
+      if (p.gate && p.gate_w == 1 && t < p.T)
+        head_gate = __fdividef(1.f, 1.f + __expf(-__bfloat162float(p.gate[t * p.gate_stride + h])));
 #pragma unroll 1
       for (int j = 0; j < 2; ++j) {
         uint32_t v[32];
@@ -133,8 +136,8 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
             if (n < p.N) {
               float f[8];
 #pragma unroll
-              for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(v[8 * c + e]);
-              if (p.gate) {
+              for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(v[8 * c + e]) * head_gate;
+              if (p.gate && p.gate_w != 1) {
                 const uint4 raw = *reinterpret_cast<const uint4*>(p.gate + t * p.gate_stride + (long long)h * p.N + n);
                 const uint32_t g[4] = {raw.x, raw.y, raw.z, raw.w};
 #pragma unroll
@@ -174,8 +177,9 @@ constexpr float LD_LOG2E = 1.4426950408889634f, LD_LN2 = 0.6931471805599453f;
 struct LatentDecodeParams {
   const __nv_bfloat16* q;  // [T, H, width]
   const int *block_table, *cu_q, *seq_lens;
-  int max_blocks, T, B, H, width, rank, block_size, num_splits, stages;
+  int max_blocks, T, B, H, width, rank, block_size, window, num_splits, stages;
   float scale;
+  const float* sink;       // [H] or null
   __nv_bfloat16* out;      // [T, H, rank]
   float *o_part, *ml_part;
   int* status;
@@ -266,8 +270,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
     b = lo;
   }
   const int len = p.seq_lens[b] - (p.T != p.B ? p.cu_q[b + 1] - 1 - t : 0);  // keys that the row sees
-  const int chunks = (len + LD_KEYS - 1) / LD_KEYS, per_split = (chunks + p.num_splits - 1) / p.num_splits;
-  const int c_begin = split * per_split, n_chunks = max(min(chunks, c_begin + per_split) - c_begin, 0);
+  const int key_lo = p.window > 0 ? max(len - p.window, 0) : 0, c_first = key_lo / LD_KEYS;  // first key that it sees
+  const int chunks = (len + LD_KEYS - 1) / LD_KEYS, per_split = (chunks - c_first + p.num_splits - 1) / p.num_splits;
+  const int c_begin = c_first + split * per_split, n_chunks = max(min(chunks, c_begin + per_split) - c_begin, 0);
   {
     const __nv_bfloat16* q = p.q + ((long long)t * p.H + h0) * p.width;
     const int per_row = parts * 8;
@@ -369,10 +374,12 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
     const float scale2 = p.scale * LD_LOG2E;
     const int key = warp * 16 + lane;  // of the chunk: lanes 0..15
     float ref[HB], sum[HB];  // of all keys: the reference; of this thread's keys: the sum of weights
+    // the sink is a key without a value: its weight starts the denominator (of one split, in one thread)
+    const bool sunk = p.sink != nullptr && split == 0;
 #pragma unroll
     for (int g = 0; g < HB; ++g) {
-      ref[g] = -INFINITY;
-      sum[g] = 0.f;
+      ref[g] = sunk && g < nh ? p.sink[h0 + g] * LD_LOG2E : -INFINITY;
+      sum[g] = sunk && g < nh && tid == 0 ? 1.f : 0.f;
     }
     bool ok = true;
     for (int c = 0; c < n_chunks; ++c) {
@@ -390,7 +397,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
         uint32_t v[HB];
         ld_cols<HB>(s_addr + (c & 1) * HB, v);
         tmem_ld_wait();
-        const bool valid = lane < 16 && (c_begin + c) * LD_KEYS + key < len;
+        const int at = (c_begin + c) * LD_KEYS + key;
+        const bool valid = lane < 16 && at < len && at >= key_lo;
 #pragma unroll
         for (int g = 0; g < HB; ++g) {
           sc[g] = valid ? __uint_as_float(v[g]) * scale2 : -INFINITY;
@@ -522,15 +530,15 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
 using namespace vb;
 
 // out[t, h, n] = sum_k a[t, h, k] B_h[n, k] for n < N (B stored [H, N, K], or [H, K, N] with b_mn), times
-// sigmoid(gate[t, h * N + n]) when gate is given; then `tail` elements a[t, h, K ...], then zeros up to `width`.
+// sigmoid(gate[t, h * N + n]) when gate is given (gate_w 1: sigmoid(gate[t, h])); then `tail` elements a[t, h, K ...], then zeros up to `width`.
 // bf16; K, N, width and all strides are multiples of 8, all bases 16-byte aligned.
 extern "C" int vb_head_gemm(const void* a, long long a_t, long long a_h, const void* b, int b_mn, void* out, long long o_t,
-                            long long o_h, const void* gate, long long gate_stride, int T, int H, int K, int N, int tail,
-                            int width, int* status, cudaStream_t stream) {
+                            long long o_h, const void* gate, long long gate_stride, int gate_w, int T, int H, int K, int N,
+                            int tail, int width, int* status, cudaStream_t stream) {
   if (T <= 0) return 0;
+  if (gate != nullptr && gate_w != 1 && (gate_w != N || (gate_stride & 7) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -3;
   if (H <= 0 || H > 65535 || K <= 0 || N <= 0 || (K & 7) || (N & 7) || (width & 7) || width < N + tail || (a_t & 7) ||
-      (a_h & 7) || (o_t & 7) || (o_h & 7) || (gate_stride & 7) || (T + 127) / 128 > 65535 ||
-      ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(gate)) & 15))
+      (a_h & 7) || (o_t & 7) || (o_h & 7) || (T + 127) / 128 > 65535 || (reinterpret_cast<uintptr_t>(out) & 15))
     return -3;
   CUtensorMap tmA, tmB;
   int rc = vb_make_tmap_3d(&tmA, a, 2, K, H, T, (uint64_t)a_h * 2, (uint64_t)a_t * 2, 64, 1, 128);
@@ -544,7 +552,7 @@ extern "C" int vb_head_gemm(const void* a, long long a_t, long long a_h, const v
     attr_set = true;
   }
   HeadGemmParams p{reinterpret_cast<const __nv_bfloat16*>(a), a_t, a_h, reinterpret_cast<__nv_bfloat16*>(out), o_t, o_h,
-                   reinterpret_cast<const __nv_bfloat16*>(gate), gate_stride, T, K, N, tail, width, b_mn, status};
+                   reinterpret_cast<const __nv_bfloat16*>(gate), gate_stride, gate_w, T, K, N, tail, width, b_mn, status};
   rc = (int)vb_launch_pdl(head_gemm_kernel, dim3((N + 63) / 64, H, (T + 127) / 128), dim3(HG_THREADS), HG_SMEM, stream, 1, tmA,
                           tmB, p);
   vb_count_launch();
@@ -584,12 +592,13 @@ int vb_decode_merge(const float* o_part, const float* ml_part, int B, int Hq, in
                     long long out_stride, const void* gate, long long gate_stride, cudaStream_t stream);
 
 // Row t of q [T, H, width] is one of the last positions of its sequence (cu_q [B + 1], seq_lens [B]; T == B: one row each) and
-// sees the page rows [num_blocks, block_size, width] up to its own; the first `rank` numbers of a row are the value.
+// sees the page rows [num_blocks, block_size, width] up to its own (window > 0: the last `window` of them); the first `rank`
+// numbers of a row are the value. sink [H] fp32 or null: exp(sink[h]) joins the denominator.
 // out [T, H, rank]. work: T * H * num_splits * (rank + 2) floats (unused when num_splits == 1).
 extern "C" int vb_latent_decode(const void* q, const void* pages, int num_blocks, const int* block_table, int max_blocks,
                                 const int* cu_q, const int* seq_lens, int T, int B, int H, int width, int rank,
-                                int block_size, float scale, int num_splits, void* out, float* work, int* status,
-                                cudaStream_t stream) {
+                                int block_size, float scale, int window, const float* sink, int num_splits, void* out,
+                                float* work, int* status, cudaStream_t stream) {
   if (T <= 0 || B <= 0) return 0;
   if (!vb_latent_decode_supported(H, width, rank, block_size) || num_splits < 1 || num_splits > 65535 ||
       (num_splits > 1 && work == nullptr) || (reinterpret_cast<uintptr_t>(q) & 15))
@@ -603,7 +612,7 @@ extern "C" int vb_latent_decode(const void* q, const void* pages, int num_blocks
   p.q = reinterpret_cast<const __nv_bfloat16*>(q);
   p.block_table = block_table; p.cu_q = cu_q; p.seq_lens = seq_lens; p.max_blocks = max_blocks;
   p.T = T; p.B = B; p.H = H; p.width = width; p.rank = rank; p.block_size = block_size;
-  p.num_splits = num_splits; p.stages = stages; p.scale = scale;
+  p.num_splits = num_splits; p.stages = stages; p.scale = scale; p.window = window; p.sink = sink;
   p.out = reinterpret_cast<__nv_bfloat16*>(out);
   p.o_part = work;
   p.ml_part = work ? work + (long long)T * H * num_splits * rank : nullptr;

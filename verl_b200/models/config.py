@@ -10,7 +10,8 @@ from dataclasses import asdict, dataclass, field
 from pathlib import Path
 from typing import Any
 
-from .layer_specs import (DESIGNS, AttentionSpec, DeltaSpec, Design, GluSpec, LatentSpec, LayerSpec, RotarySpec)
+from .layer_specs import (DESIGNS, AttentionSpec, DeltaSpec, Design, GluSpec, LatentSpec, LayerSpec, LruSpec, MoeSpec,
+                          RotarySpec)
 
 _ARCH_TO_TYPE = {
     "LlamaForCausalLM": "llama",
@@ -32,7 +33,7 @@ _TYPE_TO_ARCH = {"llama": "LlamaForCausalLM", "qwen2": "Qwen2ForCausalLM", "qwen
                  "qwen2_5_vl": "Qwen2_5_VLForConditionalGeneration", "apertus": "ApertusForCausalLM",
                  "qwen3_vl": "Qwen3VLForConditionalGeneration", "qwen3_vl_moe": "Qwen3VLMoeForConditionalGeneration"}
 # designs whose config.json lists its layers one by one (``architecture`` instead of ``architectures``)
-_LAYER_LIST_ARCHS = {"Fuganex": "fuganex", "Padodra": "padodra"}
+_LAYER_LIST_ARCHS = {"Fuganex": "fuganex", "Padodra": "padodra", "Golonex": "golonex"}
 _VL_TYPES = ("qwen2_vl", "qwen2_5_vl", "qwen3_vl", "qwen3_vl_moe")
 
 
@@ -69,12 +70,15 @@ class ModelConfig:
     layer_specs: tuple = ()
     embedding_scale: float = 1.0
     logit_scale: float = 1.0
+    logit_softcap: float = 0.0  # > 0: logits become softcap * tanh(logits / softcap)
+    side_dim: int = 0           # size of the per-token input of every layer (0 = none)
     extra: dict = field(default_factory=dict)
 
     def __post_init__(self):
         self.layer_specs = tuple(self.layer_specs)
         if self.layer_specs:
             self.num_hidden_layers = len(self.layer_specs)
+            self.tie_word_embeddings = self.design.tied
         if self.head_dim is None:
             self.head_dim = self.hidden_size // self.num_attention_heads
         if self.attention_bias is None:
@@ -101,7 +105,7 @@ class ModelConfig:
     @property
     def has_recurrent_state(self) -> bool:
         """Some layer carries a state per sequence that pages cannot share."""
-        return any(s.kind == "delta" for s in self.layer_specs)
+        return any(s.kind in ("delta", "rglru") for s in self.layer_specs)
 
     @property
     def mlp_gated(self) -> bool:
@@ -139,7 +143,13 @@ class ModelConfig:
         H, L = self.hidden_size, self.num_hidden_layers
         if self.is_layer_list:
             total = H + sum(s.num_parameters(H) for s in self.layer_specs)
-            return total + (2 * self.vocab_size * H if include_embedding else 0)
+            if self.design.embedding == "norm":
+                total += H
+            if self.side_dim:
+                total += L * (2 * H * self.side_dim + H)
+                if include_embedding:
+                    total += self.vocab_size * L * self.side_dim
+            return total + ((1 if self.tie_word_embeddings else 2) * self.vocab_size * H if include_embedding else 0)
         attn = H * (self.q_size + 2 * self.kv_size) + self.q_size * H
         if self.attention_bias:
             attn += self.q_size + 2 * self.kv_size
@@ -218,21 +228,38 @@ class ModelConfig:
         att = [s.mixer for s in specs if s.kind == "attention"]
         kw = {k: int(d[k]) for k in ("bos_token_id", "eos_token_id", "pad_token_id") if d.get(k) is not None}
         kw.setdefault("eos_token_id", None)
-        known = ("architecture", "vocab", "width", "layers", "norm", "embedding", "logit_scale", *kw)
-        return cls(model_type=model_type, logit_scale=float(d.get("logit_scale", 1.0)) if design.logit_scale else 1.0, vocab_size=int(d["vocab"]), hidden_size=int(d["width"]),
+        known = ["architecture", "vocab", "width", "layers", "norm", *kw]
+        if design.embedding == "scale":
+            known.append("embedding")
+            kw["embedding_scale"] = float(d["embedding"]["scale"])
+        if design.logit_scale:
+            known.append("logit_scale")
+            kw["logit_scale"] = float(d.get("logit_scale", 1.0))
+        if design.logit_softcap:
+            known.append("logit_softcap")
+            kw["logit_softcap"] = float(d.get("logit_softcap") or 0.0)
+        if design.side:
+            known.append("token_side")
+            kw["side_dim"] = int((d.get("token_side") or {}).get("dim") or 0)
+        return cls(model_type=model_type, vocab_size=int(d["vocab"]), hidden_size=int(d["width"]),
                    intermediate_size=max([s.mlp.ff for s in specs if s.mlp] or [0]),
                    num_attention_heads=max([a.heads for a in att] or [1]),
                    num_key_value_heads=max([a.kv_heads for a in att] or [1]), head_dim=max([a.dim for a in att] or [1]),
-                   rms_norm_eps=float(d["norm"]["eps"]), embedding_scale=float(d["embedding"]["scale"]),
+                   rms_norm_eps=float(d["norm"]["eps"]),
                    layer_specs=specs, extra={k: v for k, v in d.items() if k not in known}, **kw)
 
     def _to_layer_list(self) -> dict[str, Any]:
         arch = {v: k for k, v in _LAYER_LIST_ARCHS.items()}[self.model_type]
         d = {"architecture": arch, "vocab": self.vocab_size, "width": self.hidden_size,
-             "layers": [s.to_dict() for s in self.layer_specs], "norm": {"eps": self.rms_norm_eps},
-             "embedding": {"scale": self.embedding_scale}, **self.extra}
+             "layers": [s.to_dict() for s in self.layer_specs], "norm": {"eps": self.rms_norm_eps}, **self.extra}
+        if self.design.embedding == "scale":
+            d["embedding"] = {"scale": self.embedding_scale}
         if self.design.logit_scale:
             d["logit_scale"] = self.logit_scale
+        if self.logit_softcap:
+            d["logit_softcap"] = self.logit_softcap
+        if self.side_dim:
+            d["token_side"] = {"dim": self.side_dim}
         for k in ("bos_token_id", "eos_token_id", "pad_token_id"):
             if getattr(self, k) is not None:
                 d[k] = getattr(self, k)
@@ -249,7 +276,8 @@ class ModelConfig:
         if self.is_layer_list:
             return self._to_layer_list()
         d = asdict(self)
-        del d["layer_specs"], d["embedding_scale"], d["logit_scale"]
+        for k in ("layer_specs", "embedding_scale", "logit_scale", "logit_softcap", "side_dim"):
+            del d[k]
         extra = d.pop("extra")
         if self.model_type in _VL_TYPES:
             moe_keys = () if self.is_moe else ("num_experts", "num_experts_per_tok", "moe_intermediate_size", "norm_topk_prob",
@@ -302,11 +330,23 @@ def _padodra_specs(groups: int, heads: int, kv_heads: int, dim: int, chunk: int,
     mlp = GluSpec(ff, act="gelu_tanh")
     rot = RotarySpec(dim, 500000.0, True, (("factor", 8.0), ("high", 4.0), ("low", 1.0), ("original", 8192)))
     att = AttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, qk_norm="head", rotary=rot, chunk=chunk, softcap=30.0,
-                        sink=True, gate=True)
+                        sink=True, gate="element")
     h, d, r, v, rank = latent
     yarn = RotarySpec(r, 10000.0, False, (("factor", 40.0), ("fast", 32.0), ("original", 4096), ("slow", 1.0)))
-    lat = LatentSpec(h, d, r, v, rank, (d + r) ** -0.5, yarn, True)
+    lat = LatentSpec(h, d, r, v, rank, (d + r) ** -0.5, yarn, "element")
     return (LayerSpec(att, mlp), LayerSpec(att, mlp), LayerSpec(lat, mlp)) * groups
+
+
+def _golonex_specs(groups: int, heads: int, kv_heads: int, dim: int, window: int, lru: tuple, latent: tuple, moe: tuple) -> tuple:
+    """``groups`` x (recurrent block, latent attention, attention), a mixture of experts after each. ``lru``: width, blocks,
+    taps; ``latent``: heads, unrotated and rotated head size, value size, rank, rank of the queries; ``moe``: experts, experts
+    per token, their size, the shared unit's size."""
+    mlp = MoeSpec(*moe)
+    yarn = RotarySpec(dim // 2, 10000.0, True, (("factor", 8.0), ("fast", 32.0), ("original", 4096), ("slow", 1.0)))
+    att = AttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, window, qk_norm=None, rotary=yarn, key_values=True)
+    h, d, r, v, rank, q_rank = latent
+    lat = LatentSpec(h, d, r, v, rank, (d + r) ** -0.5, RotarySpec(r, 10000.0, True), "head", q_rank, window, True)
+    return (LayerSpec(LruSpec(*lru), mlp), LayerSpec(lat, mlp), LayerSpec(att, mlp)) * groups
 
 
 # Named architectures used by the benchmarks and tests (random-init, no download needed).
@@ -420,6 +460,15 @@ PRESETS: dict[str, dict] = {
     "padodra-8b": dict(model_type="padodra", vocab_size=128256, hidden_size=4096, eos_token_id=None, rms_norm_eps=1e-5,
                        num_attention_heads=32, num_key_value_heads=8, head_dim=128, intermediate_size=14336,
                        layer_specs=_padodra_specs(10, 32, 8, 128, 2048, 14336, (32, 128, 64, 128, 512))),
+    "tiny-golonex": dict(model_type="golonex", vocab_size=600, hidden_size=144, eos_token_id=2, rms_norm_eps=1e-6,
+                         logit_softcap=20.0, side_dim=16,
+                         layer_specs=_golonex_specs(1, 6, 3, 32, 50, (168, 3, 4), (4, 24, 16, 40, 64, 72), (6, 2, 104, 88))),
+    # real-model sizes for benchmarks: the widths of llama-3-8b, windows of 1024, its feed-forward cut into 16 experts
+    "golonex-8b": dict(model_type="golonex", vocab_size=128256, hidden_size=4096, eos_token_id=None, rms_norm_eps=1e-5,
+                       num_attention_heads=32, num_key_value_heads=8, head_dim=128, intermediate_size=896, logit_softcap=30.0,
+                       side_dim=256,
+                       layer_specs=_golonex_specs(10, 32, 8, 128, 1024, (4096, 16, 4), (32, 128, 64, 128, 512, 1536),
+                                                  (16, 4, 896, 3584))),
     "llama-3-8b": dict(model_type="llama", vocab_size=128256, hidden_size=4096, intermediate_size=14336,
                        num_hidden_layers=32, num_attention_heads=32, num_key_value_heads=8, rope_theta=5e5,
                        rms_norm_eps=1e-5, eos_token_id=128001),

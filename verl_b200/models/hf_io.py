@@ -16,6 +16,7 @@ from typing import Iterable, Iterator
 import torch
 
 from .config import ModelConfig
+from .layer_specs import MoeSpec
 
 
 _VIS_HF_TO_NATIVE = (("attn.qkv.", "qkv."), ("attn.proj.", "proj."), ("mlp.fc1.", "fc1."), ("mlp.fc2.", "fc2."),
@@ -207,35 +208,58 @@ def native_to_hf_items(cfg: ModelConfig, named: Iterable[tuple[str, torch.Tensor
 
 # ------------------------------------------------------------- layer-list checkpoints (models/hybrid.py)
 # native name -> checkpoint name of the tensors that are stored alike
-_LIST_TOP = {"embed_tokens.weight": "embed", "norm.weight": "final.norm", "lm_head.weight": "head"}
+_LIST_TOP = {"embed_tokens.weight": "embed", "norm.weight": "final.norm", "lm_head.weight": "head",
+             "embed_norm.weight": "embed.norm", "side_embed.weight": "side.embed"}
 _LIST_PLAIN = {"norm1.weight": "norm1", "norm2.weight": "norm2", "mlp.down_proj.weight": "mlp.down",
                "mixer.o_proj.weight": "mix.o", "mixer.q_norm.weight": "mix.q.norm", "mixer.k_norm.weight": "mix.k.norm",
                "mixer.rel": "mix.rel", "mixer.A_log": "mix.A_log", "mixer.dt_bias": "mix.dt_bias",
-               "mixer.norm.weight": "mix.norm", "mixer.sink": "mix.sink", "mixer.kv_norm.weight": "mix.dkv.norm"}
+               "mixer.norm.weight": "mix.norm", "mixer.sink": "mix.sink", "mixer.kv_norm.weight": "mix.dkv.norm",
+               "mixer.q_latent_norm.weight": "mix.dq.norm", "mixer.conv_w": "mix.conv", "mixer.conv_b": "mix.conv.b",
+               "mixer.lam": "mix.lam", "mlp.shared.down_proj.weight": "mlp.shared.down",
+               "side.gate_proj.weight": "side.gate", "side.out_proj.weight": "side.proj", "side.norm.weight": "side.norm"}
 
 
 def _list_fused(spec) -> dict[str, list[tuple[str, int]]]:
     """Native fused matrices of a layer: name -> [(checkpoint name, rows), ...] in row order."""
     m = spec.mixer
     if spec.kind == "attention":
-        out = {"mixer.qkv_proj.weight": [("mix.q", m.q_size), ("mix.k", m.k_size), ("mix.v", m.v_size)]
-               + ([("mix.g", m.out_size)] if m.gate else [])}
+        out = {"mixer.qkv_proj.weight": [("mix.q", m.q_size), ("mix.k", m.k_size)]
+               + ([] if m.key_values else [("mix.v", m.v_size)]) + ([("mix.g", m.out_size)] if m.gate else [])}
     elif spec.kind == "latent_attention":
-        out = {"mixer.in_proj.weight": [("mix.q", m.q_size), ("mix.dkv", m.latent_size)]
-               + ([("mix.g", m.out_size)] if m.gate else []),
+        out = {"mixer.in_proj.weight": [("mix.dq" if m.q_rank else "mix.q", m.q_in), ("mix.dkv", m.latent_size)]
+               + ([("mix.g", m.gate_size)] if m.gate else []),
                "mixer.kv_up_proj.weight": [("mix.uk", m.heads * m.dim), ("mix.uv", m.heads * m.vdim)]}
+        if m.q_rank:
+            out["mixer.q_up_proj.weight"] = [("mix.uq", m.q_size)]
+    elif spec.kind == "rglru":
+        out = {"mixer.in_proj.weight": [("mix.y", m.width), ("mix.x", m.width)],
+               "mixer.in_proj.bias": [("mix.y.b", m.width), ("mix.x.b", m.width)],
+               "mixer.gates": [("mix.ra", m.blocks), ("mix.ri", m.blocks)],
+               "mixer.gates_b": [("mix.ra.b", m.blocks), ("mix.ri.b", m.blocks)]}
     else:
         qk, v = m.kv_heads * m.dim, m.heads * m.vdim
         out = {"mixer.in_proj.weight": [("mix.q", qk), ("mix.k", qk), ("mix.v", v), ("mix.g", v), ("mix.b", m.heads),
                                         ("mix.a", m.heads)],
                "mixer.conv": [("mix.q.conv", qk), ("mix.k.conv", qk), ("mix.v.conv", v)]}
-    if spec.mlp is not None:
+    if isinstance(spec.mlp, MoeSpec):
+        out["mlp.router_proj.weight"] = [("mlp.router", spec.mlp.experts)]
+        if spec.mlp.shared_ff:
+            out["mlp.router_proj.weight"].append(("mlp.shared.sg", 1))
+            out["mlp.shared.gate_up_proj.weight"] = [(f"mlp.shared.{x}", spec.mlp.shared_ff) for x in ("gate", "up")]
+    elif spec.mlp is not None:
         out["mlp.gate_up_proj.weight"] = [("mlp.gate", spec.mlp.ff), ("mlp.up", spec.mlp.ff)]
     return out
 
 
+def _list_experts(spec) -> dict[str, list[str]]:
+    """Native stacks of expert matrices: name -> the checkpoint names of one expert's rows (``mlp.e<k>.`` in front)."""
+    return {"mlp.experts_gate_up": ["gate", "up"], "mlp.experts_down": ["down"]} if isinstance(spec.mlp, MoeSpec) else {}
+
+
 def _layer_list_to_native(cfg: ModelConfig, sd: dict[str, torch.Tensor]) -> dict[str, torch.Tensor]:
-    out = {n: sd[c] for n, c in _LIST_TOP.items()}
+    out = {n: sd[c] for n, c in _LIST_TOP.items() if c in sd}
+    if "embed_tokens.weight" not in out or "norm.weight" not in out:
+        raise KeyError("the checkpoint has no embedding or no final norm")
     for i, spec in enumerate(cfg.layer_specs):
         fused = _list_fused(spec)
         for n, parts in fused.items():
@@ -246,9 +270,12 @@ def _layer_list_to_native(cfg: ModelConfig, sd: dict[str, torch.Tensor]) -> dict
                     raise ValueError(f"l{i}.{c}: {t.shape[0]} rows, the configuration says {rows}")
                 ts.append(t)
             w = torch.cat(ts, 0)
-            if n.endswith("_proj.weight") and w.shape[0] % 8:  # padded with zero rows
-                w = torch.cat([w, w.new_zeros(8 - w.shape[0] % 8, w.shape[1])], 0)
+            if n.endswith(("_proj.weight", "_proj.bias")) and w.shape[0] % 8:  # padded with zero rows
+                w = torch.cat([w, w.new_zeros(8 - w.shape[0] % 8, *w.shape[1:])], 0)
             out[f"layers.{i}.{n}"] = w
+        for n, parts in _list_experts(spec).items():
+            out[f"layers.{i}.{n}"] = torch.stack([torch.cat([sd[f"l{i}.mlp.e{e}.{c}"] for c in parts], 0)
+                                                  for e in range(spec.mlp.experts)])
         for n, c in _LIST_PLAIN.items():
             if f"l{i}.{c}" in sd:
                 out[f"layers.{i}.{n}"] = sd[f"l{i}.{c}"]
@@ -262,6 +289,12 @@ def _layer_list_to_ckpt(cfg: ModelConfig, name: str, t: torch.Tensor) -> Iterato
     _, i, rest = name.split(".", 2)
     if rest in _LIST_PLAIN:
         yield f"l{i}.{_LIST_PLAIN[rest]}", t
+        return
+    experts = _list_experts(cfg.layer_specs[int(i)]).get(rest)
+    if experts:
+        for e in range(t.shape[0]):
+            for c, part in zip(experts, t[e].chunk(len(experts), 0)):
+                yield f"l{i}.mlp.e{e}.{c}", part
         return
     lo = 0
     for c, rows in _list_fused(cfg.layer_specs[int(i)])[rest]:

@@ -1,6 +1,6 @@
 """Decoders described layer by layer (``ModelConfig.layer_specs``): every layer has its own mixer, softmax attention over
-the paged KV cache, latent attention over pages of latents or a gated delta rule with per-sequence state, and an optional
-gated feed-forward.
+the paged KV cache, latent attention over pages of latents, a gated delta rule or a gated linear recurrent unit with
+per-sequence state, and an optional gated feed-forward or mixture of them.
 
 Served by the rollout engine like the homogeneous stacks of :mod:`.transformer`; there is no training path. The residual
 stream is fp32 and every norm is fused with the residual add beside it. Designs that norm what a sublayer reads:
@@ -12,10 +12,16 @@ Designs that norm what a sublayer puts out (the last norm + add also computes th
 
     embedding * scale -> [ fused input projection -> mixer -> output projection -> norm1 + add
                            -> gate|up -> GLU -> down -> norm2 + add ] ... -> head
+
+Layers with an input of their own per token read the stream behind the feed-forward as it is, and their normed output is added
+together with the next layer's norm1 (or the final norm):
+
+    [ ... add + copy -> gate -> gelu * side embedding -> out -> norm + add + next norm ]
 """
 
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field
 from typing import Callable, Optional
 
@@ -24,7 +30,7 @@ import torch.nn as nn
 
 from .. import ops
 from .config import ModelConfig
-from .layer_specs import AttentionSpec, DeltaSpec, GluSpec, LatentSpec, LayerSpec, distance_buckets
+from .layer_specs import AttentionSpec, DeltaSpec, GluSpec, LatentSpec, LayerSpec, LruSpec, MoeSpec, distance_buckets
 from .transformer import Linear, RMSNormWeight
 
 
@@ -43,11 +49,15 @@ class LatentPlan:
     """How latent-attention layers run a step. The leading ``short_seqs`` sequences (``short_rows`` token rows, few new tokens
     each) attend in the latent space, straight from the pages. The others get the keys and values of their whole context
     expanded, group by group: (first sequence, end, ctx_cu = int32 [n + 1] boundaries of the contexts, their total, longest
-    portion)."""
+    portion). ``windowed``: the same for layers with a window, by its size: a context is what the window reaches."""
 
     short_seqs: int
     short_rows: int
     groups: tuple = ()
+    windowed: dict = field(default_factory=dict)
+
+    def groups_of(self, window: int) -> tuple:
+        return self.windowed[window] if window else self.groups
 
 
 @dataclass
@@ -64,11 +74,12 @@ class RaggedBatch:
     max_ctx: int = 0           # longest sequence a replay of this step may see
     positions: Optional[torch.Tensor] = None  # [T] position of each token
     latent: Optional[LatentPlan] = None
+    singles: int = 0           # leading sequences with one new token each
 
 
 class StateCache:
     """Cache of a layer-list model: K / V pages per attention layer, pages of latents and rotated keys per latent-attention
-    layer, fp32 state and convolution ring per delta layer."""
+    layer, fp32 state and convolution ring per delta or recurrent-unit layer."""
 
     def __init__(self, cfg: ModelConfig, num_blocks: int, block_size: int, num_slots: int, dtype, device):
         self.layers: list[tuple] = []
@@ -80,8 +91,15 @@ class StateCache:
             elif spec.kind == "latent_attention":
                 self.layers.append((torch.zeros((num_blocks, block_size, ops.latent_width(m.latent_size)), dtype=dtype, device=device),))
             else:
-                self.layers.append((torch.zeros((num_slots, m.conv, m.channels), dtype=dtype, device=device),
-                                    torch.zeros((num_slots, m.heads, m.vdim, m.dim), dtype=torch.float32, device=device)))
+                channels, state = self._state(spec)
+                self.layers.append((torch.zeros((num_slots, m.conv, channels), dtype=dtype, device=device),
+                                    torch.zeros((num_slots, *state), dtype=torch.float32, device=device)))
+
+    @staticmethod
+    def _state(spec) -> tuple:
+        """Convolved channels and shape of the state of a recurrent layer."""
+        m = spec.mixer
+        return (m.width, (m.width,)) if spec.kind == "rglru" else (m.channels, (m.heads, m.vdim, m.dim))
 
     @staticmethod
     def page_bytes(cfg: ModelConfig, block_size: int, itemsize: int) -> int:
@@ -90,8 +108,12 @@ class StateCache:
 
     @staticmethod
     def slot_bytes(cfg: ModelConfig, itemsize: int) -> int:
-        return sum(m.conv * m.channels * itemsize + 4 * m.heads * m.vdim * m.dim
-                   for m in (s.mixer for s in cfg.layer_specs if s.kind == "delta"))
+        total = 0
+        for s in cfg.layer_specs:
+            if s.kind in ("delta", "rglru"):
+                channels, state = StateCache._state(s)
+                total += s.mixer.conv * channels * itemsize + 4 * math.prod(state)
+        return total
 
 
 def rotary_frequencies(module: nn.Module, spec, device) -> None:
@@ -134,7 +156,7 @@ class AttentionMixer(nn.Module):
             q = ops.head_norm_rope_kv_write(qkv, *norms, self.rot_freqs if s.rotary else None, batch.positions, batch.slots,
                                             cache[0], cache[1], s.heads, self.eps,
                                             interleaved=s.rotary is not None and s.rotary.interleaved,
-                                            amplitude=s.rotary.amplitude if s.rotary else 1.0)
+                                            amplitude=s.rotary.amplitude if s.rotary else 1.0, key_values=s.key_values)
         else:
             raise NotImplementedError("rotary positions after a norm over the whole projection")
         lo = s.q_size + s.k_size + s.v_size
@@ -154,6 +176,11 @@ class LatentMixer(nn.Module):
         self.kv_norm = RMSNormWeight(spec.kv_rank, dtype, device)
         self.kv_up_proj = Linear(spec.kv_rank, pad8(spec.up_size), False, dtype, device)
         self.o_proj = Linear(spec.out_size, cfg.hidden_size, False, dtype, device)
+        if spec.q_rank:
+            self.q_latent_norm = RMSNormWeight(spec.q_rank, dtype, device)
+            self.q_up_proj = Linear(spec.q_rank, pad8(spec.q_size), False, dtype, device)
+        if spec.sink:
+            self.sink = nn.Parameter(torch.zeros(spec.heads, dtype=torch.float32, device=device))
         rotary_frequencies(self, spec.rotary, device)
 
     def refresh(self):
@@ -163,11 +190,18 @@ class LatentMixer(nn.Module):
         s, pages, plan = self.spec, cache[0], batch.latent
         T = x.shape[0]
         proj = mm(x, self.in_proj.weight)
-        ops.latent_rope_write(proj, self.kv_norm.weight, self.rot_freqs, batch.positions, batch.slots, pages, s.heads, s.dim,
-                              s.rot_dim, s.kv_rank, self.eps, amplitude=s.rotary.amplitude)
-        q = proj[:, : s.q_size].view(T, s.heads, s.dim + s.rot_dim)
-        lo = s.q_size + s.latent_size
-        gate = proj[:, lo : lo + s.out_size] if s.gate else None
+        rot = dict(amplitude=s.rotary.amplitude, interleaved=s.rotary.interleaved)
+        ops.latent_rope_write(proj, self.kv_norm.weight, self.rot_freqs, batch.positions, batch.slots, pages,
+                              0 if s.q_rank else s.heads, s.dim, s.rot_dim, s.kv_rank, self.eps, **rot, q_rank=s.q_rank,
+                              q_norm_w=self.q_latent_norm.weight if s.q_rank else None)
+        q = proj
+        if s.q_rank:
+            q = mm(proj[:, : s.q_rank], self.q_up_proj.weight)
+            ops.rotate_tails(q, self.rot_freqs, batch.positions, s.heads, s.dim, s.rot_dim, **rot)
+        q = q[:, : s.q_size].view(T, s.heads, s.dim + s.rot_dim)
+        lo = s.q_in + s.latent_size
+        gate = proj[:, lo : lo + s.gate_size] if s.gate else None
+        sink = self.sink if s.sink else None
         out = torch.empty((T, s.out_size), dtype=x.dtype, device=x.device)
         up = self.kv_up_proj.weight
         uk = up[: s.heads * s.dim].view(s.heads, s.dim, s.kv_rank)
@@ -175,13 +209,14 @@ class LatentMixer(nn.Module):
         n, B = plan.short_rows, plan.short_seqs
         if n:  # scores and weighted sums over the latents themselves: W_uk moves to the queries, W_uv behind the sum
             lat = ops.latent_attention(ops.latent_queries(q[:n], uk), pages, batch.block_table[:B], batch.cu_q[: B + 1],
-                                       batch.seq_lens[:B], s.kv_rank, scale=s.scale, max_ctx=batch.max_ctx)
+                                       batch.seq_lens[:B], s.kv_rank, scale=s.scale, max_ctx=batch.max_ctx, window=s.window,
+                                       sink=sink)
             ops.latent_values(lat, uv, None if gate is None else gate[:n], out[:n])
-        for b0, b1, ctx_cu, total, max_q in plan.groups:
-            rows = ops.latent_gather(pages, batch.block_table[b0:b1], ctx_cu, total)
+        for b0, b1, ctx_cu, total, max_q in plan.groups_of(s.window):
+            rows = ops.latent_gather(pages, batch.block_table[b0:b1], ctx_cu, total, batch.seq_lens[b0:b1])
             kv = mm(rows[:, : s.kv_rank], up)
             ops.latent_prefill(q, rows[:, s.kv_rank : s.latent_size], kv, batch.cu_q[b0 : b1 + 1], ctx_cu, max_q, s.dim,
-                               s.vdim, scale=s.scale, gate=gate, out=out)
+                               s.vdim, scale=s.scale, gate=gate, out=out, window=s.window, sink=sink)
         return mm(out, self.o_proj.weight)
 
 
@@ -214,6 +249,38 @@ class DeltaMixer(nn.Module):
         return mm(o, self.o_proj.weight)
 
 
+class LruMixer(nn.Module):
+    def __init__(self, cfg: ModelConfig, spec: LruSpec, dtype, device):
+        super().__init__()
+        self.spec = spec
+        n = spec.block_size
+        self.in_proj = Linear(cfg.hidden_size, pad8(spec.proj_size), True, dtype, device)
+        self.conv_w = nn.Parameter(torch.zeros(spec.width, spec.conv, dtype=dtype, device=device))
+        self.conv_b = nn.Parameter(torch.zeros(spec.width, dtype=dtype, device=device))
+        self.gates = nn.Parameter(torch.zeros(2 * spec.blocks, n, n, dtype=dtype, device=device))  # decay | input
+        self.gates_b = nn.Parameter(torch.zeros(2 * spec.blocks, n, dtype=torch.float32, device=device))
+        self.lam = nn.Parameter(torch.zeros(spec.width, dtype=torch.float32, device=device))
+        self.o_proj = Linear(spec.out_size, cfg.hidden_size, False, dtype, device)
+
+    def reset_parameters(self, generator=None):
+        with torch.no_grad():
+            for w, fan in ((self.conv_w, self.spec.conv), (self.gates, self.spec.block_size)):
+                w.copy_(torch.empty(w.shape, device=w.device).normal_(0.0, fan ** -0.5, generator=generator))
+            # decays (at a gate of one) between 0.9 and 0.999
+            a = torch.empty(self.spec.width, device=self.lam.device).uniform_(0.9, 0.999, generator=generator)
+            self.lam.copy_(torch.log(torch.expm1(-torch.log(a) / self.spec.power)))
+
+    def refresh(self):
+        pass
+
+    def forward(self, x, batch: RaggedBatch, cache, mm: Callable):
+        s = self.spec
+        proj = mm(x, self.in_proj.weight, self.in_proj.bias)
+        o = ops.rglru(proj, self.conv_w, self.conv_b, self.gates, self.gates_b, self.lam, cache[0], cache[1], batch.cu_q,
+                      batch.seq_lens, batch.state_slots, batch.max_q, s.power, singles=batch.singles)
+        return mm(o, self.o_proj.weight)
+
+
 class GatedMLP(nn.Module):
     def __init__(self, cfg: ModelConfig, spec: GluSpec, dtype, device):
         super().__init__()
@@ -224,23 +291,79 @@ class GatedMLP(nn.Module):
     def forward(self, x, mm: Callable):
         s = self.spec
         gu = mm(x, self.gate_up_proj.weight)
-        h = ops.gelu_tanh_glu(gu, s.ff) if s.act == "gelu_tanh" else ops.clamped_glu(gu, s.ff, s.limit, s.alpha)
+        if s.act == "silu":
+            h = ops.silu_glu(gu, s.ff)
+        else:
+            h = ops.gelu_tanh_glu(gu, s.ff) if s.act == "gelu_tanh" else ops.clamped_glu(gu, s.ff, s.limit, s.alpha)
         return mm(h, self.down_proj.weight)
 
 
-_MIXERS = {"attention": AttentionMixer, "latent_attention": LatentMixer, "delta": DeltaMixer}
+class RoutedMLP(nn.Module):
+    """Mixture of gated linear units; its result is still in parts (:class:`~verl_b200.ops.moe.RoutedSum`), which the next
+    add + norm puts together."""
+
+    def __init__(self, cfg: ModelConfig, spec: MoeSpec, dtype, device):
+        super().__init__()
+        self.spec, H = spec, cfg.hidden_size
+        self.router_proj = Linear(H, pad8(spec.router_rows), False, dtype, device)  # router | gate of the shared unit
+        self.experts_gate_up = nn.Parameter(torch.zeros(spec.experts, 2 * spec.ff, H, dtype=dtype, device=device))
+        self.experts_down = nn.Parameter(torch.zeros(spec.experts, H, spec.ff, dtype=dtype, device=device))
+        if spec.shared_ff:
+            self.shared = GatedMLP(cfg, GluSpec(spec.shared_ff, act=spec.act), dtype, device)
+        # tokens per expert while a step is being routed; zero between steps
+        self.register_buffer("counters", torch.zeros(spec.experts + 1, dtype=torch.int32, device=device), persistent=False)
+
+    def reset_parameters(self, generator=None):
+        with torch.no_grad():
+            for w in (self.experts_gate_up, self.experts_down):
+                for e in range(w.shape[0]):
+                    w[e].copy_(torch.empty(w.shape[1:], device=w.device).normal_(0.0, 0.02, generator=generator))
+
+    def forward(self, x, mm: Callable):
+        s = self.spec
+        logits = ops.gemm(x, self.router_proj.weight, out_dtype=torch.float32)
+        routing = ops.moe_route(logits, s.experts, s.top, self.counters, score=s.score, renormalize=s.renormalize)
+        out = ops.moe_experts(x, routing, self.experts_gate_up, self.experts_down, s.act, weigh_input=s.weigh == "input")
+        return ops.RoutedSum(out, routing, s.weigh == "output", self.shared(x, mm) if s.shared_ff else None,
+                             logits[:, s.experts] if s.shared_ff else None)
+
+
+class SideInput(nn.Module):
+    """Input of a layer's own per token: the layer's part of the token's side embedding, gated by the stream."""
+
+    def __init__(self, cfg: ModelConfig, index: int, dtype, device):
+        super().__init__()
+        self.lo, self.dim = index * cfg.side_dim, cfg.side_dim
+        self.gate_proj = Linear(cfg.hidden_size, cfg.side_dim, False, dtype, device)
+        self.out_proj = Linear(cfg.side_dim, cfg.hidden_size, False, dtype, device)
+        self.norm = RMSNormWeight(cfg.hidden_size, dtype, device)
+
+    def forward(self, x, ids, table, mm: Callable):
+        g = ops.gelu_rows(mm(x, self.gate_proj.weight), ids, table, self.lo, self.dim)
+        return mm(g, self.out_proj.weight)
+
+
+_MIXERS = {"attention": AttentionMixer, "latent_attention": LatentMixer, "delta": DeltaMixer, "rglru": LruMixer}
+
+
+def add_norm(pending, res, weight, eps, dtype):
+    """Adds a sublayer's output (None: nothing) to the stream in place; the normed stream, or without a weight a copy."""
+    if isinstance(pending, ops.RoutedSum):
+        return ops.moe_combine(pending, res, weight, eps, dtype)
+    return ops.add_rmsnorm(pending, res, weight, eps, dtype)
 
 
 class HybridLayer(nn.Module):
-    def __init__(self, cfg: ModelConfig, spec: LayerSpec, dtype, device):
+    def __init__(self, cfg: ModelConfig, spec: LayerSpec, index: int, dtype, device):
         super().__init__()
         self.norm1 = RMSNormWeight(cfg.hidden_size, dtype, device)
         self.mixer = _MIXERS[spec.kind](cfg, spec.mixer, dtype, device)
         if spec.mlp is not None:
             self.norm2 = RMSNormWeight(cfg.hidden_size, dtype, device)
-            self.mlp = GatedMLP(cfg, spec.mlp, dtype, device)
+            self.mlp = (RoutedMLP if isinstance(spec.mlp, MoeSpec) else GatedMLP)(cfg, spec.mlp, dtype, device)
         else:
             self.norm2 = self.mlp = None
+        self.side = SideInput(cfg, index, dtype, device) if cfg.side_dim else None
 
 
 class HybridLM(nn.Module):
@@ -248,9 +371,15 @@ class HybridLM(nn.Module):
         super().__init__()
         self.cfg = cfg
         self.embed_tokens = nn.Embedding(cfg.vocab_size, cfg.hidden_size, dtype=dtype, device=device)
-        self.layers = nn.ModuleList([HybridLayer(cfg, s, dtype, device) for s in cfg.layer_specs])
+        if cfg.design.norm == "post" and (cfg.side_dim or any(isinstance(s.mlp, MoeSpec) for s in cfg.layer_specs)):
+            raise NotImplementedError("mixtures of experts and side inputs go with norms in front of the sublayers")
+        if cfg.design.embedding == "norm":
+            self.embed_norm = RMSNormWeight(cfg.hidden_size, dtype, device)
+        if cfg.side_dim:
+            self.side_embed = nn.Embedding(cfg.vocab_size, cfg.num_hidden_layers * cfg.side_dim, dtype=dtype, device=device)
+        self.layers = nn.ModuleList([HybridLayer(cfg, s, i, dtype, device) for i, s in enumerate(cfg.layer_specs)])
         self.norm = RMSNormWeight(cfg.hidden_size, dtype, device)
-        self.lm_head = Linear(cfg.hidden_size, cfg.vocab_size, False, dtype, device)
+        self.lm_head = None if cfg.tie_word_embeddings else Linear(cfg.hidden_size, cfg.vocab_size, False, dtype, device)
         # portions up to this many tokens run latent attention in the latent space; sizes without an expanded form: all
         self.latent_short = LATENT_SHORT
         for s in cfg.layer_specs:
@@ -264,15 +393,17 @@ class HybridLM(nn.Module):
         gen = torch.Generator(device=dev)
         gen.manual_seed(seed)
         with torch.no_grad():
-            w = self.embed_tokens.weight
-            w.copy_(torch.empty(w.shape, dtype=torch.float32, device=dev).normal_(0.0, 1.0, generator=gen))
+            for e in (self.embed_tokens, getattr(self, "side_embed", None)):
+                if e is not None:  # a table that is the output projection as well: logits of a size near one
+                    std = self.cfg.hidden_size ** -0.5 if self.cfg.tie_word_embeddings and e is self.embed_tokens else 1.0
+                    e.weight.copy_(torch.empty(e.weight.shape, dtype=torch.float32, device=dev).normal_(0.0, std, generator=gen))
         for m in self.modules():
-            if isinstance(m, (Linear, DeltaMixer)):
+            if isinstance(m, (Linear, DeltaMixer, LruMixer, RoutedMLP)):
                 m.reset_parameters(gen)
             elif isinstance(m, AttentionMixer) and m.spec.bias_rows:
                 with torch.no_grad():
                     m.rel.copy_(torch.empty(m.rel.shape, device=dev).normal_(0.0, 0.5, generator=gen))
-            if isinstance(m, AttentionMixer) and m.spec.sink:
+            if isinstance(m, (AttentionMixer, LatentMixer)) and m.spec.sink:
                 with torch.no_grad():
                     m.sink.copy_(torch.empty(m.sink.shape, device=dev).normal_(0.0, 1.0, generator=gen))
         self.refresh()
@@ -285,20 +416,29 @@ class HybridLM(nn.Module):
 
     @property
     def lm_head_weight(self) -> torch.Tensor:
-        return self.lm_head.weight
+        return self.embed_tokens.weight if self.lm_head is None else self.lm_head.weight
 
     def projection_weights(self) -> list[torch.Tensor]:
-        """Matrices of the layers (what weight quantisation applies to). The projections out of the latent are left out: they
-        are applied to queries and to weighted sums as well as to the latents."""
+        """Matrices of the layers (what weight quantisation applies to). Left out: the projections out of the latent, which are
+        applied to queries and to weighted sums as well as to the latents; routers, whose scores choose; the narrow matrices of
+        side inputs."""
         return [m.weight for layer in self.layers for n, m in layer.named_modules()
-                if isinstance(m, Linear) and not n.endswith("kv_up_proj")]
+                if isinstance(m, Linear) and not n.endswith(("kv_up_proj", "router_proj")) and not n.startswith("side.")]
 
     def plan_latent(self, counts: list[int], ctx: list[int], boundaries: Callable) -> Optional[LatentPlan]:
         """How latent-attention layers run a step of ``counts[i]`` new tokens in sequences of ``ctx[i]`` tokens, ordered by
         :meth:`latent_order`. ``boundaries(list)``: int32 device tensor. None without such layers."""
-        if not any(s.kind == "latent_attention" for s in self.cfg.layer_specs):
+        windows = {s.mixer.window for s in self.cfg.layer_specs if s.kind == "latent_attention"}
+        if not windows:
             return None
         B = sum(c <= self.latent_short for c in counts)
+        full = self._latent_groups(B, counts, ctx, boundaries) if 0 in windows else ()
+        return LatentPlan(B, sum(counts[:B]), full,
+                          {w: self._latent_groups(B, counts, [min(n, c + w - 1) for n, c in zip(ctx, counts)], boundaries)
+                           for w in sorted(windows - {0})})
+
+    @staticmethod
+    def _latent_groups(B: int, counts: list[int], ctx: list[int], boundaries: Callable) -> tuple:
         groups, b0 = [], B
         while b0 < len(counts):  # expanded keys and values are scratch: contexts are taken together up to a bound
             b1, total = b0 + 1, ctx[b0]
@@ -310,13 +450,15 @@ class HybridLM(nn.Module):
                 cu.append(cu[-1] + c)
             groups.append((b0, b1, boundaries(cu), total, max(counts[b0:b1])))
             b0 = b1
-        return LatentPlan(B, sum(counts[:B]), tuple(groups))
+        return tuple(groups)
 
     def latent_order(self, counts: list[int]) -> Optional[list[int]]:
-        """Order of a step's sequences: those whose latent attention stays in the latent space first. None: any order."""
-        if all(s.kind != "latent_attention" for s in self.cfg.layer_specs):
+        """Order of a step's sequences: those whose latent attention stays in the latent space first, and where recurrent units
+        step single tokens together, those before all others. None: any order."""
+        kinds = {s.kind for s in self.cfg.layer_specs}
+        if not kinds & {"latent_attention", "rglru"}:
             return None
-        return sorted(range(len(counts)), key=lambda i: counts[i] > self.latent_short)
+        return sorted(range(len(counts)), key=lambda i: (counts[i] > self.latent_short, "rglru" in kinds and counts[i] > 1))
 
     def forward(self, *args, **kwargs):
         raise NotImplementedError(f"{self.cfg.model_type}: layer-list models are served by the rollout engine only "
@@ -325,9 +467,9 @@ class HybridLM(nn.Module):
     @torch.no_grad()
     def run(self, ids: torch.Tensor, batch: RaggedBatch, cache: StateCache, mm: Callable,
             observe: Optional[Callable] = None) -> torch.Tensor:
-        """Final-norm hidden states [T, H] of one step (times the design's logit scale). ``mm(x, w)``: the engine's matrix product. ``observe(i, stream)``
-        gets the residual stream after layer i (a copy; debugging and tests)."""
-        c, eps = self.cfg, self.cfg.rms_norm_eps
+        """Final-norm hidden states [T, H] of one step (times the design's logit scale). ``mm(x, w)`` or ``mm(x, w, bias)``: the
+        engine's matrix product. ``observe(i, stream)`` gets the residual stream after layer i (a copy; debugging and tests)."""
+        c, eps, dtype = self.cfg, self.cfg.rms_norm_eps, self.embed_tokens.weight.dtype
         if c.design.norm == "post":
             res, x = ops.embedding_scaled(ids, self.embed_tokens.weight, c.embedding_scale, with_copy=True)
             last = len(self.layers) - 1
@@ -341,14 +483,23 @@ class HybridLM(nn.Module):
                 if observe is not None:
                     observe(i, res.clone())
             return x
-        res = ops.embedding_scaled(ids, self.embed_tokens.weight, c.embedding_scale)
-        pending = None  # output of the last sublayer, not yet added to the stream
+        if c.design.embedding == "norm":
+            res = ops.embedding_normed(ids, self.embed_tokens.weight, self.embed_norm.weight, eps)
+        else:
+            res = ops.embedding_scaled(ids, self.embed_tokens.weight, c.embedding_scale)
+        x = ops.add_rmsnorm(None, res, self.layers[0].norm1.weight, eps)
         for i, layer in enumerate(self.layers):
-            x = ops.add_rmsnorm(pending, res, layer.norm1.weight, eps)
+            # the norm that the next sublayer (or the head) reads through
+            after = (self.layers[i + 1].norm1 if i + 1 < len(self.layers) else self.norm).weight
             pending = layer.mixer(x, batch, cache.layers[i], mm)
             if layer.mlp is not None:
-                x = ops.add_rmsnorm(pending, res, layer.norm2.weight, eps)
+                x = add_norm(pending, res, layer.norm2.weight, eps, dtype)
                 pending = layer.mlp(x, mm)
+            if layer.side is not None:
+                y = layer.side(add_norm(pending, res, None, eps, dtype), ids, self.side_embed.weight, mm)
+                x = ops.rmsnorm_add(y, res, layer.side.norm.weight, eps, final_weight=after)
+            else:
+                x = add_norm(pending, res, after, eps, dtype)
             if observe is not None:
-                observe(i, res + pending.float())
-        return ops.add_rmsnorm(pending, res, self.norm.weight, eps)
+                observe(i, res.clone())
+        return x

@@ -1,8 +1,9 @@
 """Per-layer descriptions of decoders whose layers differ from one another (``ModelConfig.layer_specs``).
 
-A layer is a mixer (softmax attention, latent attention or a gated delta rule, each with its own sizes) and an optional
-feed-forward. The specs carry every size and constant of a mechanism, so that another design can combine them differently;
-what a design fixes instead of writing it in its config.json is in ``DESIGNS``."""
+A layer is a mixer (softmax attention, latent attention, a gated delta rule or a gated linear recurrent unit, each with its own
+sizes) and an optional feed-forward (a gated linear unit or a mixture of them). The specs carry every size and constant of a
+mechanism, so that another design can combine them differently; what a design fixes instead of writing it in its config.json
+is in ``DESIGNS``."""
 
 from __future__ import annotations
 
@@ -76,7 +77,8 @@ class AttentionSpec:
     ``chunk`` positions, counted from the start of the sequence. ``bias_rows`` / ``bias_max``: learned distance
     bias per head, added to the scaled score (``bias_rows`` 0 = none); see :func:`distance_buckets`. ``softcap`` > 0: scaled
     scores become ``softcap * tanh(score / softcap)``. ``sink``: a learned number per head whose exponential joins the
-    softmax denominator. ``gate``: the heads are multiplied with the sigmoid of a projection of the mixer's input."""
+    softmax denominator. ``gate``: the heads are multiplied with the sigmoid of a projection of the mixer's input, element by
+    element ("element"). ``key_values``: the values are the keys as projected, before the rotation (no value projection)."""
 
     heads: int
     kv_heads: int
@@ -93,7 +95,8 @@ class AttentionSpec:
     chunk: int = 0
     softcap: float = 0.0
     sink: bool = False
-    gate: bool = False
+    gate: Optional[str] = None
+    key_values: bool = False
 
     @property
     def q_size(self) -> int:
@@ -105,7 +108,8 @@ class AttentionSpec:
 
     @property
     def v_size(self) -> int:
-        return self.kv_heads * self.vdim
+        """Rows of the value projection."""
+        return 0 if self.key_values else self.kv_heads * self.vdim
 
     @property
     def out_size(self) -> int:
@@ -126,7 +130,8 @@ class AttentionSpec:
 class LatentSpec:
     """Latent attention: every head's keys (their unrotated ``dim``) and values are projections of one normed latent of
     ``kv_rank`` numbers per token; ``rot_dim`` rotated key dimensions are shared by all heads. Latent and rotated part are
-    what the cache holds. Full causal. ``gate`` as in :class:`AttentionSpec`."""
+    what the cache holds. ``q_rank`` > 0: the queries are projections of a normed latent of their own. ``window`` (0 = full
+    causal) and ``sink`` as in :class:`AttentionSpec`; ``gate`` as there, or one number per head ("head")."""
 
     heads: int
     dim: int
@@ -135,11 +140,19 @@ class LatentSpec:
     kv_rank: int
     scale: float
     rotary: RotarySpec
-    gate: bool = False
+    gate: Optional[str] = None
+    q_rank: int = 0
+    window: int = 0
+    sink: bool = False
 
     @property
     def q_size(self) -> int:
         return self.heads * (self.dim + self.rot_dim)
+
+    @property
+    def q_in(self) -> int:
+        """Rows of the input projection that the queries come from: the queries themselves, or their latent."""
+        return self.q_rank or self.q_size
 
     @property
     def latent_size(self) -> int:
@@ -151,9 +164,13 @@ class LatentSpec:
         return self.heads * self.vdim
 
     @property
+    def gate_size(self) -> int:
+        return {None: 0, "element": self.out_size, "head": self.heads}[self.gate]
+
+    @property
     def proj_size(self) -> int:
-        """q | latent, rotated key (| output gate)."""
-        return self.q_size + self.latent_size + (self.out_size if self.gate else 0)
+        """q or its latent | latent, rotated key (| output gate)."""
+        return self.q_in + self.latent_size + self.gate_size
 
     @property
     def up_size(self) -> int:
@@ -187,14 +204,68 @@ class DeltaSpec:
 
 
 @dataclass(frozen=True)
+class LruSpec:
+    """Recurrent block with a real-gated linear recurrent unit (Griffin): a gelu branch times a branch that runs through a short
+    convolution of ``conv`` taps (without activation) and the recurrence ``S = a S + sqrt(1 - a^2) i u`` per channel, with
+    ``log a = -power * r * softplus(lam)``; the gates r and i are projections of u in ``blocks`` equal parts."""
+
+    width: int
+    blocks: int
+    conv: int
+    power: float = 8.0
+
+    @property
+    def block_size(self) -> int:
+        return self.width // self.blocks
+
+    @property
+    def proj_size(self) -> int:
+        """gelu branch | recurrent branch."""
+        return 2 * self.width
+
+    @property
+    def out_size(self) -> int:
+        return self.width
+
+
+@dataclass(frozen=True)
 class GluSpec:
     """Gated linear unit. ``act`` "clamped": ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``,
-    ``g * sigmoid(alpha * g) * (u + 1)``; "gelu_tanh": ``gelu(gate) * up`` with the tanh form of gelu."""
+    ``g * sigmoid(alpha * g) * (u + 1)``; "gelu_tanh": ``gelu(gate) * up`` with the tanh form of gelu; "silu":
+    ``silu(gate) * up``."""
 
     ff: int
     limit: float = 0.0
     alpha: float = 1.702
     act: str = "clamped"
+
+    def num_parameters(self, width: int) -> int:
+        return 3 * width * self.ff
+
+
+@dataclass(frozen=True)
+class MoeSpec:
+    """Mixture of ``experts`` gated linear units of ``ff``, ``top`` of them per token. Router scores: "sigmoid" or "softmax" of
+    the logits, computed in fp32; the ``top`` largest are chosen and weigh as they are (``renormalize``: divided by their sum).
+    ``weigh`` "input": an expert runs on its weight times the token, "output": its result is multiplied. ``shared_ff`` > 0: a
+    unit of that size runs for every token, its result multiplied with the sigmoid of a projection to one number."""
+
+    experts: int
+    top: int
+    ff: int
+    shared_ff: int = 0
+    act: str = "silu"
+    score: str = "sigmoid"
+    renormalize: bool = False
+    weigh: str = "input"
+
+    @property
+    def router_rows(self) -> int:
+        """Router | gate of the shared unit."""
+        return self.experts + (1 if self.shared_ff else 0)
+
+    def num_parameters(self, width: int) -> int:
+        return width * (self.router_rows + 3 * (self.experts * self.ff + self.shared_ff))
 
 
 @dataclass(frozen=True)
@@ -205,25 +276,35 @@ class Design:
     norm: str = "pre"
     mask: str = "window"
     qk_norm: Optional[str] = "projection"
-    interleaved: bool = False  # rotary layout of attention layers (latent attention: always halves)
+    interleaved: bool = False  # rotary layout of attention layers
     sink: bool = False
-    gate: bool = False
+    gate: Optional[str] = None
+    key_values: bool = False
+    latent_interleaved: bool = False  # the same of latent attention
+    latent_sink: bool = False
+    latent_gate: Optional[str] = None
     act: str = "clamped"
+    embedding: str = "scale"   # "scale": times a factor of config.json, "norm": RMS norm
+    tied: bool = False         # the embedding table is the output projection
     logit_scale: bool = False  # config.json has a factor for the logits
+    logit_softcap: bool = False  # config.json has a soft cap for the logits
+    side: bool = False         # layers add an input of their own per token (config.json: its size)
 
 
 DESIGNS: dict[str, Design] = {
     "fuganex": Design(),
-    "padodra": Design(norm="post", mask="chunk", qk_norm="head", interleaved=True, sink=True, gate=True, act="gelu_tanh",
-                      logit_scale=True),
+    "padodra": Design(norm="post", mask="chunk", qk_norm="head", interleaved=True, sink=True, gate="element",
+                      latent_gate="element", act="gelu_tanh", logit_scale=True),
+    "golonex": Design(qk_norm=None, interleaved=True, key_values=True, latent_interleaved=True, latent_sink=True,
+                      latent_gate="head", act="silu", embedding="norm", tied=True, logit_softcap=True, side=True),
 }
-_KINDS = {AttentionSpec: "attention", LatentSpec: "latent_attention", DeltaSpec: "delta"}
+_KINDS = {AttentionSpec: "attention", LatentSpec: "latent_attention", DeltaSpec: "delta", LruSpec: "rglru"}
 
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: Union[AttentionSpec, LatentSpec, DeltaSpec]
-    mlp: Optional[GluSpec] = None
+    mixer: Union[AttentionSpec, LatentSpec, DeltaSpec, LruSpec]
+    mlp: Union[GluSpec, MoeSpec, None] = None
 
     @property
     def kind(self) -> str:
@@ -240,25 +321,41 @@ class LayerSpec:
                                   0 if chunked else size, int(mask.get("keep_first") or 0), float(m.get("bias_max") or 0.0),
                                   qk_norm=design.qk_norm, chunk=size if chunked else 0,
                                   rotary=RotarySpec.from_dict(m["rot"], design.interleaved) if m.get("rot") else None,
-                                  softcap=float(m.get("softcap") or 0.0), sink=design.sink, gate=design.gate)
+                                  softcap=float(m.get("softcap") or 0.0), sink=design.sink, gate=design.gate,
+                                  key_values=design.key_values)
             if mixer.rotary is not None and mixer.rotary.dims > mixer.dim:
                 raise ValueError(f"{mixer.rotary.dims} rotated dimensions in heads of {mixer.dim}")
+            if mixer.key_values and mixer.vdim != mixer.dim:
+                raise ValueError(f"values of {mixer.vdim} that are the keys of {mixer.dim}")
         elif d["type"] == "latent_attention":
             mixer = LatentSpec(int(m["heads"]), int(m["dim"]), int(m["rot_dim"]), int(m["vdim"]), int(m["kv_rank"]),
-                               float(m["scale"]), RotarySpec.from_dict(m["rot"], False), design.gate)
+                               float(m["scale"]), RotarySpec.from_dict(m["rot"], design.latent_interleaved),
+                               design.latent_gate, int(m.get("q_rank") or 0), int((m.get("mask") or {}).get("size") or 0),
+                               design.latent_sink)
             if mixer.rotary.dims != mixer.rot_dim:
                 raise ValueError(f"{mixer.rotary.dims} rotated dimensions in a rotated part of {mixer.rot_dim}")
         elif d["type"] == "delta":
             mixer = DeltaSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), int(m["conv"]))
+        elif d["type"] == "rglru":
+            mixer = LruSpec(int(m["width"]), int(m["blocks"]), int(m["conv"]))
+            if mixer.width % mixer.blocks:
+                raise ValueError(f"a width of {mixer.width} is not a multiple of {mixer.blocks} blocks")
         else:
             raise ValueError(f"unknown layer type {d['type']!r} (known: {', '.join(_KINDS.values())})")
-        if mixer.heads % getattr(mixer, "kv_heads", 1):
+        if getattr(mixer, "heads", 0) % getattr(mixer, "kv_heads", 1):
             raise ValueError(f"{mixer.heads} heads are not a multiple of {mixer.kv_heads} key/value heads")
         mlp = d.get("mlp")
         if mlp is not None:
-            if mlp.get("kind", "dense") != "dense":
-                raise ValueError(f"unknown feed-forward kind {mlp['kind']!r} (known: dense)")
-            mlp = GluSpec(int(mlp["ff"]), float(mlp["limit"]) if design.act == "clamped" else 0.0, act=design.act)
+            kind = mlp.get("kind", "dense")
+            if kind == "moe" and design.act == "silu":
+                mlp = MoeSpec(int(mlp["router"]["experts"]), int(mlp["router"]["top"]), int(mlp["expert"]["ff"]),
+                              int((mlp.get("shared") or {}).get("ff") or 0), act=design.act)
+                if not 0 < mlp.top <= mlp.experts:
+                    raise ValueError(f"{mlp.top} of {mlp.experts} experts")
+            elif kind == "dense":
+                mlp = GluSpec(int(mlp["ff"]), float(mlp["limit"]) if design.act == "clamped" else 0.0, act=design.act)
+            else:
+                raise ValueError(f"unknown feed-forward kind {kind!r} (known: dense, and moe where the units are silu)")
         return cls(mixer, mlp)
 
     def to_dict(self) -> dict[str, Any]:
@@ -268,7 +365,7 @@ class LayerSpec:
             if m.chunk:
                 mix["mask"] = {"size": m.chunk}
             elif m.window or m.keep_first:
-                mix["mask"] = {"size": m.window, "keep_first": m.keep_first}
+                mix["mask"] = {"size": m.window, **({"keep_first": m.keep_first} if m.keep_first or not m.key_values else {})}
             if m.bias_max:
                 mix["bias_max"] = int(m.bias_max) if m.bias_max == int(m.bias_max) else m.bias_max
             if m.rotary is not None:
@@ -278,10 +375,20 @@ class LayerSpec:
         elif self.kind == "latent_attention":
             mix = {"heads": m.heads, "dim": m.dim, "rot_dim": m.rot_dim, "vdim": m.vdim, "kv_rank": m.kv_rank,
                    "scale": m.scale, "rot": m.rotary.to_dict()}
+            if m.q_rank:
+                mix["q_rank"] = m.q_rank
+            if m.window:
+                mix["mask"] = {"size": m.window}
+        elif self.kind == "rglru":
+            mix = {"width": m.width, "blocks": m.blocks, "conv": m.conv}
         else:
             mix = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "conv": m.conv}
         mlp = None
-        if self.mlp is not None:
+        if isinstance(self.mlp, MoeSpec):
+            mlp = {"kind": "moe", "expert": {"ff": self.mlp.ff}, "router": {"experts": self.mlp.experts, "top": self.mlp.top}}
+            if self.mlp.shared_ff:
+                mlp["shared"] = {"ff": self.mlp.shared_ff}
+        elif self.mlp is not None:
             mlp = {"kind": "dense", "ff": self.mlp.ff}
             if self.mlp.act == "clamped":
                 mlp["limit"] = self.mlp.limit
@@ -296,11 +403,15 @@ class LayerSpec:
         if self.kind == "attention":
             n += m.bias_rows * m.heads + sum(m.norm_sizes) + (m.heads if m.sink else 0)
         elif self.kind == "latent_attention":
-            n += m.kv_rank + m.up_size * m.kv_rank
+            n += m.kv_rank + m.up_size * m.kv_rank + (m.heads if m.sink else 0)
+            if m.q_rank:
+                n += m.q_rank + m.q_size * m.q_rank
+        elif self.kind == "rglru":  # biases of the branches, convolution, gates, lam
+            n += m.width * (2 + m.conv + 1 + 2 * (m.block_size + 1) + 1)
         else:
             n += m.channels * m.conv + 2 * m.heads + m.vdim
         if self.mlp is not None:
-            n += width + 3 * width * self.mlp.ff
+            n += width + self.mlp.num_parameters(width)
         return n
 
 

@@ -1,12 +1,15 @@
 """Architecture registry (verl/models/registry.py:43-63): HF ``architectures`` name -> the native model family.
 
 The reference maps an architecture to Megatron ``Parallel*ForCausalLMRmPadPP`` classes; here every supported family is
-one :class:`CausalLM` parameterised by :class:`ModelConfig`, so the registry resolves to a builder instead."""
+one :class:`CausalLM` (layer-list designs: one :class:`HybridLM`) parameterised by :class:`ModelConfig`, so the registry
+resolves to a builder instead."""
 
 from __future__ import annotations
 
 from functools import partial
 from typing import Callable, Optional
+
+from .config import _LAYER_LIST_ARCHS
 
 _ARCH_TO_FAMILY = {
     "LlamaForCausalLM": "llama",
@@ -17,6 +20,7 @@ _ARCH_TO_FAMILY = {
     "LlamaForTokenClassification": "llama",
     "Qwen2ForTokenClassification": "qwen2",
     "Qwen3ForTokenClassification": "qwen3",
+    **_LAYER_LIST_ARCHS,
 }
 
 

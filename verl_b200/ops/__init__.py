@@ -8,10 +8,12 @@ from .attention import (attention_varlen, decode_workspace, head_norm_rope_kv_wr
 from .delta import delta_rule
 from .gemm import gemm, linear
 from .latent import (latent_attention, latent_gather, latent_prefill, latent_prefill_supported, latent_queries,
-                     latent_rope_write, latent_values, latent_width)
+                     latent_rope_write, latent_values, latent_width, rotate_tails)
 from .lmhead import lmhead_logprob_entropy
-from .nn import (add_rmsnorm, clamped_glu, embedding, embedding_scaled, gelu_tanh_glu, rmsnorm, rmsnorm_add, rope_qkv,
-                 rope_tables, swiglu)
+from .lru import rglru
+from .moe import RoutedSum, moe_combine, moe_experts, moe_route
+from .nn import (add_rmsnorm, clamped_glu, embedding, embedding_normed, embedding_scaled, gelu_rows, gelu_tanh_glu, rmsnorm,
+                 rmsnorm_add, rope_qkv, rope_tables, silu_glu, softcap_, swiglu)
 from .rl import (PPO_METRIC_NAMES, adamw_step, clip_coef, decode_advance, gae, grpo_advantage, ppo_loss_fused, sample,
                  sumsq_into)
 
@@ -21,5 +23,6 @@ __all__ = [
     "grpo_advantage", "sample", "decode_advance", "adamw_step", "sumsq_into", "clip_coef", "PPO_METRIC_NAMES",
     "paged_attention", "qk_norm_kv_write", "delta_rule", "add_rmsnorm", "clamped_glu", "embedding_scaled",
     "rmsnorm_add", "gelu_tanh_glu", "head_norm_rope_kv_write", "latent_attention", "latent_gather", "latent_prefill",
-    "latent_prefill_supported", "latent_queries", "latent_rope_write", "latent_values", "latent_width",
+    "latent_prefill_supported", "latent_queries", "latent_rope_write", "latent_values", "latent_width", "rotate_tails",
+    "embedding_normed", "silu_glu", "gelu_rows", "softcap_", "rglru", "RoutedSum", "moe_route", "moe_experts", "moe_combine",
 ]

@@ -49,16 +49,27 @@ _SIGS = {
     "vb_embed_scaled": ([P, P, P, P, I, I, F, I, P], I),
     "vb_rmsnorm_add": ([P, L, P, P, P, F, P, I, I, F, I, P], I),
     "vb_gelu_glu": ([P, L, P, I, I, I, P], I),
-    "vb_head_norm_rope_kv_write": ([P, L, P, P, P, I, I, F, P, P, P, P, I, I, I, I, I, I, F, I, P], I),
-    "vb_latent_rope_write": ([P, L, P, P, F, P, P, P, I, I, I, I, I, I, F, I, P], I),
-    "vb_head_gemm": ([P, L, L, P, I, P, L, L, P, L, I, I, I, I, I, I, P, P], I),
-    "vb_head_gemm_simt": ([P, L, L, P, I, P, L, L, P, L, I, I, I, I, I, I, I, P], I),
+    "vb_silu_glu": ([P, L, P, I, I, P, P, I, P], I),
+    "vb_gelu_rows": ([P, L, P, P, L, I, P, I, I, I, P], I),
+    "vb_softcap": ([P, L, F, P], I),
+    "vb_embed_normed": ([P, P, P, P, I, I, F, I, P], I),
+    "vb_head_norm_rope_kv_write": ([P, L, P, P, P, I, I, F, P, P, P, P, I, I, I, I, I, I, I, F, I, P], I),
+    "vb_latent_rope_write": ([P, L, P, P, F, I, P, P, P, I, I, I, I, I, I, I, P, F, I, P], I),
+    "vb_rotate_tails": ([P, L, P, F, I, P, I, I, I, I, I, P], I),
+    "vb_head_gemm": ([P, L, L, P, I, P, L, L, P, L, I, I, I, I, I, I, I, P, P], I),
+    "vb_head_gemm_simt": ([P, L, L, P, I, P, L, L, P, L, I, I, I, I, I, I, I, I, P], I),
+    "vb_moe_route": ([P, L, I, I, I, I, I, P, P, P, P, I, P, P], I),
+    "vb_moe_gather": ([P, L, P, P, I, I, I, P, P, I, P], I),
+    "vb_moe_sum": ([P, P, P, I, P, L, P, L, P, P, P, I, I, F, I, P], I),
+    "vb_grouped_gemm_simt": ([P, P, P, I, I, I, P, I, P], I),
+    "vb_rglru_tc_supported": ([I, I], I),
+    "vb_rglru": ([P, L, P, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, P, P], I),
     "vb_latent_decode_supported": ([I, I, I, I], I),
     "vb_latent_decode_splits": ([I, I, I], I),
-    "vb_latent_decode": ([P, P, I, P, I, P, P, I, I, I, I, I, I, F, I, P, P, P, P], I),
-    "vb_latent_gather": ([P, P, I, P, P, I, I, I, I, P], I),
+    "vb_latent_decode": ([P, P, I, P, I, P, P, I, I, I, I, I, I, F, I, P, I, P, P, P, P], I),
+    "vb_latent_gather": ([P, P, I, P, P, P, I, I, I, I, P], I),
     "vb_latent_flash_supported": ([I, I, I, I, I], I),
-    "vb_latent_flash": ([P, L, I, P, L, P, L, I, P, P, I, I, I, I, I, I, F, P, L, P, L, P, P], I),
+    "vb_latent_flash": ([P, L, I, P, L, P, L, I, P, P, I, I, I, I, I, I, F, I, P, P, L, I, P, L, P, P], I),
     "vb_add_rmsnorm": ([P, L, P, P, P, I, I, F, I, P], I),
     "vb_clamped_glu": ([P, L, P, I, I, F, F, I, P], I),
     "vb_qk_norm_kv_write": ([P, L, P, P, P, P, P, I, I, I, I, I, I, F, I, P], I),

@@ -246,25 +246,28 @@ def rotate_pairs(x: torch.Tensor, positions: torch.Tensor, freqs: torch.Tensor, 
 def head_norm_rope_kv_write(qkv: torch.Tensor, q_weight: torch.Tensor | None, k_weight: torch.Tensor | None,
                             freqs: torch.Tensor | None, positions: torch.Tensor, slots: torch.Tensor, k_cache: torch.Tensor,
                             v_cache: torch.Tensor, heads: int, eps: float, *, interleaved: bool,
-                            amplitude: float = 1.0) -> torch.Tensor:
+                            amplitude: float = 1.0, key_values: bool = False) -> torch.Tensor:
     """``qkv`` [T, q | k | v | ...]: RMS norm of every q and k head (weights [D] shared by the heads; None = no norm), rotary
     positions with the angles ``positions * freqs`` (fp32; None = none) on the first ``2 * len(freqs)`` dimensions, k and v
-    to their places in the paged caches [NB, Hk, BS, D] / [NB, Hk, BS, Dv] (slot < 0: no write). Returns q [T, heads, D], a
-    view of ``qkv`` (changed in place on CUDA)."""
+    to their places in the paged caches [NB, Hk, BS, D] / [NB, Hk, BS, Dv] (slot < 0: no write). ``key_values``: there is no v,
+    the values are the keys before norm and rotation. Returns q [T, heads, D], a view of ``qkv`` (changed in place on CUDA)."""
     _, Hk, BS, D = k_cache.shape
     Dv = v_cache.shape[3]
     T, nq, nk = qkv.shape[0], heads * D, Hk * D
+    if key_values and Dv != D:
+        raise ValueError(f"values of {Dv} that are the keys of {D}")
     if qkv.is_cuda:
         rc = _lib.fn("vb_head_norm_rope_kv_write")(
             qkv.data_ptr(), qkv.stride(0), _lib.ptr(q_weight), _lib.ptr(k_weight), _lib.ptr(freqs),
             0 if freqs is None else freqs.numel(), int(interleaved), float(amplitude), positions.data_ptr(), slots.data_ptr(),
-            k_cache.data_ptr(), v_cache.data_ptr(), T, heads, Hk, D, Dv, BS, float(eps), int(qkv.dtype == torch.float32),
-            _lib.stream())
+            k_cache.data_ptr(), v_cache.data_ptr(), T, heads, Hk, D, Dv, BS, int(key_values), float(eps),
+            int(qkv.dtype == torch.float32), _lib.stream())
         _lib.check(rc, "vb_head_norm_rope_kv_write")
         return qkv[:, :nq].view(T, heads, D)
     from .nn import _rmsnorm_ref
 
-    q, k, v = qkv[:, :nq].view(T, heads, D), qkv[:, nq : nq + nk].view(T, Hk, D), qkv[:, nq + nk : nq + nk + Hk * Dv]
+    q, k = qkv[:, :nq].view(T, heads, D), qkv[:, nq : nq + nk].view(T, Hk, D)
+    v = k if key_values else qkv[:, nq + nk : nq + nk + Hk * Dv]
     if q_weight is not None:
         q, k = (_rmsnorm_ref(x.float(), w.float(), eps) for x, w in ((q, q_weight), (k, k_weight)))
     if freqs is not None:

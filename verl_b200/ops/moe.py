@@ -8,7 +8,10 @@ read back to the host (no per-expert Python loop, no ``.tolist()``): the padded 
 
 from __future__ import annotations
 
+from dataclasses import dataclass
+
 import torch
+import torch.nn.functional as F
 
 from . import _lib
 
@@ -117,3 +120,129 @@ def moe_mlp(x: torch.Tensor, top_i: torch.Tensor, top_w: torch.Tensor, gate_up: 
     out = grouped_linear(h, down, blk_expert, expert_off)
     picked = out.index_select(0, dest).view(T, k, H)
     return (picked * top_w.to(x.dtype).unsqueeze(-1)).sum(1)
+
+
+# ----------------------------------------------------------------- inference: routing, experts and their sum as fused kernels
+@dataclass
+class Routing:
+    """Experts of a step's tokens. ``idx`` / ``weight`` [T, top]: the chosen experts and their weights (fp32); ``dest`` [T, top]:
+    row of the pair in the buffer sorted by expert (``rows`` of them, every expert's share padded to :data:`BLK`);
+    ``blk_expert`` [rows / BLK]: expert of each block of rows (< 0: unused)."""
+
+    idx: torch.Tensor
+    weight: torch.Tensor
+    dest: torch.Tensor
+    blk_expert: torch.Tensor
+    rows: int
+
+
+@dataclass
+class RoutedSum:
+    """Result of a mixture in parts: rows of the sorted buffer ``out`` [rows, H], one per pair of ``routing`` (``weigh``: still to
+    be multiplied with its weight), and the ``shared`` unit's result [T, H] with the logit of its gate [T] (fp32)."""
+
+    out: torch.Tensor
+    routing: Routing
+    weigh: bool
+    shared: torch.Tensor | None = None
+    shared_logit: torch.Tensor | None = None
+
+
+def moe_route(logits: torch.Tensor, experts: int, top: int, counters: torch.Tensor, *, score: str = "sigmoid",
+              renormalize: bool = False) -> Routing:
+    """The ``top`` experts of every token by the fp32 ``logits`` [T, experts | ...]. ``counters``: int32 [experts + 1], zero
+    before and after."""
+    T = logits.shape[0]
+    # an expert's padding is at most BLK - 1 rows, and experts without a token have none
+    rows = (T * top + min(experts, T * top) * (BLK - 1)) // BLK * BLK
+    if score not in ("sigmoid", "softmax"):
+        raise ValueError(f"unknown router score {score!r}")
+    if logits.is_cuda:
+        new = lambda n, dt=torch.int32: torch.empty(n, dtype=dt, device=logits.device)  # noqa: E731
+        r = Routing(new((T, top)), new((T, top), torch.float32), new((T, top)), new(rows // BLK), rows)
+        rc = _lib.fn("vb_moe_route")(logits.data_ptr(), logits.stride(0), T, experts, top, int(score == "softmax"),
+                                     int(renormalize), r.idx.data_ptr(), r.weight.data_ptr(), r.dest.data_ptr(),
+                                     r.blk_expert.data_ptr(), rows // BLK, counters.data_ptr(), _lib.stream())
+        _lib.check(rc, "vb_moe_route")
+        return r
+    z = logits[:, :experts]
+    s = torch.sigmoid(z) if score == "sigmoid" else torch.softmax(z, -1)
+    idx = torch.sort(s, dim=-1, descending=True, stable=True).indices[:, :top]
+    w = s.gather(1, idx)
+    if renormalize:
+        w = w / w.sum(-1, keepdim=True)
+    dest, blk_expert, _, P = moe_layout(idx, experts)
+    return Routing(idx, w, dest.view(T, top), blk_expert, P)
+
+
+def moe_experts(x: torch.Tensor, routing: Routing, gate_up: torch.Tensor, down: torch.Tensor, act: str, *,
+                weigh_input: bool) -> torch.Tensor:
+    """Gated linear units of the routed pairs: rows of the sorted buffer [rows, H] (other rows undefined). x [T, H], ``gate_up``
+    [E, 2 * ff, H], ``down`` [E, H, ff]. ``weigh_input``: a unit runs on weight * x, which is applied behind its first, linear,
+    product."""
+    if act != "silu":
+        raise ValueError(f"unknown activation of routed experts {act!r}")
+    T, H = x.shape
+    top, (E, N, _) = routing.idx.shape[1], gate_up.shape
+    ff = N // 2
+    if not x.is_cuda:
+        out = torch.zeros(routing.rows, H, dtype=x.dtype)
+        for e in range(E):
+            t, k = (routing.idx == e).nonzero(as_tuple=True)
+            gu = x[t].float() @ gate_up[e].float().t()
+            if weigh_input:
+                gu = gu * routing.weight[t, k][:, None]
+            h = (F.silu(gu[:, :ff]) * gu[:, ff:]).to(x.dtype)
+            out[routing.dest[t, k]] = (h.float() @ down[e].float().t()).to(x.dtype)
+        return out
+    f32, P = int(x.dtype == torch.float32), routing.rows
+    new = lambda *s, dt=x.dtype: torch.empty(s, dtype=dt, device=x.device)  # noqa: E731
+    xs, scale = new(P, H), new(P, dt=torch.float32)
+    rc = _lib.fn("vb_moe_gather")(x.data_ptr(), x.stride(0), routing.dest.data_ptr(), routing.weight.data_ptr(), T, top, H,
+                                  xs.data_ptr(), scale.data_ptr(), f32, _lib.stream())
+    _lib.check(rc, "vb_moe_gather")
+    gu = grouped_product(xs, gate_up, routing.blk_expert)
+    h = new(P, ff)
+    rc = _lib.fn("vb_silu_glu")(gu.data_ptr(), gu.stride(0), h.data_ptr(), P, ff, scale.data_ptr() if weigh_input else None,
+                                routing.blk_expert.data_ptr(), f32, _lib.stream())
+    _lib.check(rc, "vb_silu_glu")
+    return grouped_product(h, down, routing.blk_expert)
+
+
+def grouped_product(xs: torch.Tensor, weight: torch.Tensor, blk_expert: torch.Tensor) -> torch.Tensor:
+    """xs [P, K] times the matrix of each block's expert, weight [E, N, K] -> [P, N] (inference; rows of unused blocks undefined).
+    fp32, and sizes that the tensor cores do not take: CUDA cores."""
+    (P, K), (E, N, _) = xs.shape, weight.shape
+    y = torch.empty((P, N), dtype=xs.dtype, device=xs.device)
+    if xs.dtype == torch.bfloat16 and K % 8 == 0:
+        _grouped(xs, weight, y, P, N, K, False, False, False, 1, E, blk_expert, None)
+    else:
+        rc = _lib.fn("vb_grouped_gemm_simt")(xs.data_ptr(), weight.data_ptr(), y.data_ptr(), P, N, K, blk_expert.data_ptr(),
+                                             int(xs.dtype == torch.float32), _lib.stream())
+        _lib.check(rc, "vb_grouped_gemm_simt")
+    return y
+
+
+def moe_combine(parts: RoutedSum, residual: torch.Tensor, weight: torch.Tensor | None, eps: float,
+                dtype: torch.dtype) -> torch.Tensor:
+    """Adds the mixture's sum to the fp32 ``residual`` [T, H] IN PLACE; returns rmsnorm(residual) * weight, or without a weight
+    the residual, in ``dtype``."""
+    r = parts.routing
+    T, H = residual.shape
+    top = r.idx.shape[1]
+    if residual.is_cuda:
+        y = torch.empty((T, H), dtype=dtype, device=residual.device)
+        sh, lg = parts.shared, parts.shared_logit
+        rc = _lib.fn("vb_moe_sum")(parts.out.data_ptr(), r.dest.data_ptr(), r.weight.data_ptr() if parts.weigh else None, top,
+                                       _lib.ptr(sh), 0 if sh is None else sh.stride(0), _lib.ptr(lg),
+                                       0 if lg is None else lg.stride(0), residual.data_ptr(), _lib.ptr(weight), y.data_ptr(),
+                                       T, H, float(eps), int(dtype == torch.float32), _lib.stream())
+        _lib.check(rc, "vb_moe_sum")
+        return y
+    picked = parts.out[r.dest.reshape(-1)].view(T, top, H).float()
+    d = (picked * r.weight[..., None] if parts.weigh else picked).sum(1)
+    if parts.shared is not None:
+        d = d + parts.shared.float() * torch.sigmoid(parts.shared_logit.float())[:, None]
+    from .nn import add_rmsnorm
+
+    return add_rmsnorm(d, residual, weight, eps, dtype)

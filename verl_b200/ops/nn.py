@@ -286,17 +286,31 @@ def embedding_scaled(ids: torch.Tensor, weight: torch.Tensor, scale: float, with
     return (res, y) if with_copy else res
 
 
-def add_rmsnorm(delta: torch.Tensor | None, residual: torch.Tensor, weight: torch.Tensor, eps: float) -> torch.Tensor:
+def embedding_normed(ids: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, eps: float) -> torch.Tensor:
+    """fp32 residual stream rmsnorm(``table[ids]``) * ``weight`` [T, H]."""
+    if not table.is_cuda:
+        return _rmsnorm_ref(F.embedding(ids, table).float(), weight.float(), eps)
+    T, H = ids.numel(), table.shape[1]
+    res = torch.empty((T, H), dtype=torch.float32, device=table.device)
+    rc = _lib.fn("vb_embed_normed")(ids.data_ptr(), table.data_ptr(), weight.data_ptr(), res.data_ptr(), T, H, float(eps),
+                                    int(table.dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "vb_embed_normed")
+    return res
+
+
+def add_rmsnorm(delta: torch.Tensor | None, residual: torch.Tensor, weight: torch.Tensor | None, eps: float,
+                dtype: torch.dtype | None = None) -> torch.Tensor:
     """Adds ``delta`` to the fp32 ``residual`` [T, H] IN PLACE and returns rmsnorm(residual) * weight in the weight's
-    dtype: :func:`rmsnorm` for a residual stream that stays in 32 bits."""
+    dtype: :func:`rmsnorm` for a residual stream that stays in 32 bits. Without a weight: the residual itself in ``dtype``."""
+    dtype = weight.dtype if weight is not None else dtype
     if not residual.is_cuda:
         if delta is not None:
             residual += delta.float()
-        return _rmsnorm_ref(residual, weight, eps).to(weight.dtype)
+        return residual.to(dtype, copy=True) if weight is None else _rmsnorm_ref(residual, weight, eps).to(dtype)
     T, H = residual.shape
-    y = torch.empty((T, H), dtype=weight.dtype, device=residual.device)
+    y = torch.empty((T, H), dtype=dtype, device=residual.device)
     rc = _lib.fn("vb_add_rmsnorm")(_lib.ptr(delta), 0 if delta is None else delta.stride(0), residual.data_ptr(),
-                                   weight.data_ptr(), y.data_ptr(), T, H, float(eps), int(weight.dtype == torch.float32),
+                                   _lib.ptr(weight), y.data_ptr(), T, H, float(eps), int(dtype == torch.float32),
                                    _lib.stream())
     _lib.check(rc, "vb_add_rmsnorm")
     return y
@@ -331,6 +345,40 @@ def gelu_tanh_glu(gate_up: torch.Tensor, ff: int) -> torch.Tensor:
                                 int(gate_up.dtype == torch.float32), _lib.stream())
     _lib.check(rc, "vb_gelu_glu")
     return y
+
+
+def silu_glu(gate_up: torch.Tensor, ff: int) -> torch.Tensor:
+    """``gate_up`` rows hold [gate (ff) | up (ff) | padding]: silu(gate) * up [T, ff] (inference; see :func:`swiglu`)."""
+    if not gate_up.is_cuda:
+        return (F.silu(gate_up[:, :ff].float()) * gate_up[:, ff : 2 * ff].float()).to(gate_up.dtype)
+    T = gate_up.shape[0]
+    y = torch.empty((T, ff), dtype=gate_up.dtype, device=gate_up.device)
+    rc = _lib.fn("vb_silu_glu")(gate_up.data_ptr(), gate_up.stride(0), y.data_ptr(), T, ff, None, None,
+                                int(gate_up.dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "vb_silu_glu")
+    return y
+
+
+def gelu_rows(gate: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, lo: int, dim: int) -> torch.Tensor:
+    """gelu(``gate`` [T, dim]) (tanh form) times ``table[ids, lo : lo + dim]``."""
+    if not gate.is_cuda:
+        e = F.embedding(ids, table)[:, lo : lo + dim].float()
+        return (F.gelu(gate[:, :dim].float(), approximate="tanh") * e).to(gate.dtype)
+    y = torch.empty((gate.shape[0], dim), dtype=gate.dtype, device=gate.device)
+    rc = _lib.fn("vb_gelu_rows")(gate.data_ptr(), gate.stride(0), ids.data_ptr(), table.data_ptr(), table.stride(0), lo,
+                                 y.data_ptr(), gate.shape[0], dim, int(gate.dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "vb_gelu_rows")
+    return y
+
+
+def softcap_(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """fp32 ``x`` becomes ``cap * tanh(x / cap)`` in place."""
+    if not x.is_cuda:
+        return x.copy_(cap * torch.tanh(x / cap))
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise TypeError("softcap_ takes contiguous fp32")
+    _lib.check(_lib.fn("vb_softcap")(x.data_ptr(), x.numel(), float(cap), _lib.stream()), "vb_softcap")
+    return x
 
 
 def clamped_glu(gate_up: torch.Tensor, ff: int, limit: float, alpha: float) -> torch.Tensor:

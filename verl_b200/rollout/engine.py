@@ -622,6 +622,8 @@ class NativeRolloutEngine:
     def _final_logits(self, x):
         w = self.model.lm_head_weight
         logits = ops.gemm(x, w, out_dtype=torch.float32) if self.on_gpu else x.float() @ w.float().t()
+        if self.cfg.logit_softcap:
+            ops.softcap_(logits, self.cfg.logit_softcap)
         ban = getattr(self, "_banned_ids", None)
         if ban is None:
             # vision-language models: the image placeholder id stands for pixels and is never a token to generate (a
@@ -886,7 +888,8 @@ class NativeRolloutEngine:
         batch = RaggedBatch(x[: B + 1], max(counts), x[B + 1 : 2 * B + 1], w[T : 2 * T], x[3 * B + 1 :].view(B, nb),
                             x[2 * B + 1 : 3 * B + 1], ctx, w[2 * T : 3 * T],
                             self.model.plan_latent(counts, sc.seq_total[si].tolist(),
-                                                   lambda v: torch.tensor(v, dtype=torch.int32, device=dev)))
+                                                   lambda v: torch.tensor(v, dtype=torch.int32, device=dev)),
+                            next((i for i, n in enumerate(counts) if n > 1), len(counts)))
         h = self.model.run(w[:T], batch, self.state_cache, self._mm, observe=getattr(self, "observe_layers", None))
         return self._final_logits(h[w[3 * T :]]) if R else h.new_zeros((0, self.cfg.vocab_size), dtype=torch.float32)
 
