@@ -17,7 +17,9 @@ import torch
 
 from .. import ops
 from ..models import build_model, preset
+from ..models.layer_specs import MoeSpec
 from ..ops import _lib
+from ..ops import moe as moe_ops
 from .engine import NativeRolloutEngine
 
 
@@ -148,13 +150,24 @@ def bench_kernels(name: str, vs: str, B: int, n: int, DB: int, ctx: int) -> list
     else:
         add("add_rmsnorm (fp32 residual)", time_us(lambda: ops.add_rmsnorm(x, res32, w, 1e-5)), T * H * 12)
     add("  vs rmsnorm (bf16 residual)", time_us(lambda: ops.rmsnorm(x, w, 1e-5, res16)), T * H * 8)
-    gu = r(T, 2 * glu.ff)
-    if glu.act == "gelu_tanh":
+    routed = glu if isinstance(glu, MoeSpec) else None
+    ff = routed.shared_ff if routed else glu.ff
+    gu = r(T, 2 * ff)
+    if glu.act == "silu":
+        add(f"silu_glu ({ff})", time_us(lambda: ops.silu_glu(gu, ff)), T * ff * 6)
+    elif glu.act == "gelu_tanh":
         add("gelu_tanh_glu", time_us(lambda: ops.gelu_tanh_glu(gu, glu.ff)), T * glu.ff * 6)
     else:
         add("clamped_glu", time_us(lambda: ops.clamped_glu(gu, glu.ff, glu.limit, glu.alpha)), T * glu.ff * 6)
-    add("  vs swiglu", time_us(lambda: ops.swiglu(gu)), T * glu.ff * 6)
+    add("  vs swiglu", time_us(lambda: ops.swiglu(gu)), T * ff * 6)
     del gu
+    if cfg.side_dim:
+        _bench_side(add, r, cfg, T)
+    if routed:
+        _bench_moe(add, r, routed, H, T, f"prefill {T}")
+        _bench_moe(add, r, routed, H, DB, f"decode {DB}")
+    if "rglru" in mixers:
+        _bench_lru(add, r, mixers["rglru"], B, n, DB, ctx)
     if "attention" in mixers:
         _bench_attention(add, r, mixers["attention"], ref, B, n, DB, ctx)
     if "latent_attention" in mixers:
@@ -177,10 +190,14 @@ def _bench_attention(add, r, att, ref, B: int, n: int, DB: int, ctx: int) -> Non
     qw, kw = r(nqw), r(nkw)
     nb = T * (2 * att.q_size + 4 * att.k_size) * 2
     pos = torch.arange(n, device="cuda").repeat(B)
-    if att.qk_norm == "head":
+    if att.rotary is not None:
         freqs = torch.tensor(att.rotary.frequencies(), device="cuda")
-        add("head_norm_rope_kv_write", time_us(lambda: ops.head_norm_rope_kv_write(
-            qkv, qw, kw, freqs, pos, slots, kc, vc, hq, 1e-5, interleaved=att.rotary.interleaved)), nb)
+        if not att.qk_norm:
+            qw = kw = None
+        what = "no norm, values are the keys" if att.key_values else "norm per head"
+        add(f"head_norm_rope_kv_write ({what})", time_us(lambda: ops.head_norm_rope_kv_write(
+            qkv, qw, kw, freqs, pos, slots, kc, vc, hq, 1e-5, interleaved=att.rotary.interleaved, key_values=att.key_values)),
+            nb - (T * att.k_size * 2 if att.key_values else 0))
     else:
         add("qk_norm_kv_write", time_us(lambda: ops.qk_norm_kv_write(qkv, qw, kw, slots, kc, vc, hq, 1e-5)), nb)
     cos, sin = ops.rope_tables(ref.head_dim, n, 1e6, "cuda")
@@ -244,26 +261,49 @@ def _bench_attention(add, r, att, ref, B: int, n: int, DB: int, ctx: int) -> Non
         lambda: ops.paged_decode_attention(q1, kc, vc, bt, lens, num_splits=splits, work=work)), DB * ctx * hk * d * 4)
 
 
+def _seen(n: int, window: int) -> float:
+    """Pairs of a query and a key that it sees, for one prompt."""
+    i = torch.arange(1, n + 1, dtype=torch.float64)
+    return float((i.clamp(max=window) if window else i).sum())
+
+
 def _bench_latent(add, r, m, B: int, n: int, DB: int, ctx: int) -> None:
     T, h, D, width = B * n, m.heads, m.dim + m.rot_dim, ops.latent_width(m.latent_size)
     per = (n + 15) // 16
     pages, bt = r(B * per, 16, width), torch.randperm(B * per, device="cuda").view(B, per).int()
-    proj, nw = r(T, m.proj_size), r(m.kv_rank)
+    proj, nw, qw = r(T, (m.proj_size + 7) // 8 * 8), r(m.kv_rank), r(m.q_rank) if m.q_rank else None
     freqs, pos, slots = torch.tensor(m.rotary.frequencies(), device="cuda"), torch.arange(n, device="cuda").repeat(B), _slots(bt, B, n)
-    add("latent_rope_write", time_us(lambda: ops.latent_rope_write(
-        proj, nw, freqs, pos, slots, pages, h, m.dim, m.rot_dim, m.kv_rank, 1e-5)), T * 4 * (h * m.rot_dim + m.latent_size))
+    q = r(T, m.q_size) if m.q_rank else proj
+    lens = torch.full((B,), n, device="cuda", dtype=torch.int32)
+    rot = dict(interleaved=m.rotary.interleaved)
+    add("latent_rope_write" + (" (with the norm of the queries' latent)" if m.q_rank else ""), time_us(lambda: ops.latent_rope_write(
+        proj, nw, freqs, pos, slots, pages, 0 if m.q_rank else h, m.dim, m.rot_dim, m.kv_rank, 1e-5, q_rank=m.q_rank, q_norm_w=qw,
+        **rot)), T * 4 * ((m.q_rank or h * m.rot_dim) + m.latent_size))
+    if m.q_rank:
+        add("rotate_tails (queries)", time_us(lambda: ops.rotate_tails(q, freqs, pos, h, m.dim, m.rot_dim, **rot)),
+            T * 4 * h * m.rot_dim)
     proj.normal_()
-    q, gate = proj[:, : m.q_size].view(T, h, D), proj[:, m.q_size + m.latent_size :]
+    q.normal_()
+    q, gate = q[:, : m.q_size].view(T, h, D), proj[:, m.q_in + m.latent_size : m.proj_size] if m.gate else None
+    sink = torch.randn(h, device="cuda") if m.sink else None
+    kw = dict(scale=m.scale, window=m.window, sink=sink)
+    what = ", ".join([f"window {m.window}" if m.window else "full causal"] + ["sink"] * m.sink
+                     + [f"gate per {m.gate}"] * (m.gate is not None))
     cu = torch.arange(B + 1, device="cuda", dtype=torch.int32) * n
     up = r(m.up_size, m.kv_rank) * m.kv_rank ** -0.5
-    add("latent_gather", time_us(lambda: ops.latent_gather(pages, bt, cu, T)), T * width * 4)
+    add("latent_gather", time_us(lambda: ops.latent_gather(pages, bt, cu, T, lens)), T * width * 4)
     rows = ops.latent_gather(pages, bt, cu, T)
     add("up projection of the latents (gemm)", time_us(lambda: ops.gemm(rows[:, : m.kv_rank], up)),
         2 * (T * (m.kv_rank + m.up_size) + m.up_size * m.kv_rank), 2.0 * T * m.up_size * m.kv_rank)
     kv, out = ops.gemm(rows[:, : m.kv_rank], up), r(T, m.out_size)
-    add("latent_flash (full causal, gate)", time_us(lambda: ops.latent_prefill(
-        q, rows[:, m.kv_rank : m.latent_size], kv, cu, cu, n, m.dim, m.vdim, scale=m.scale, gate=gate, out=out)),
-        2 * T * (h * (D + m.dim + 3 * m.vdim) + m.rot_dim), float(n) * (n + 1) * B * h * (D + m.vdim))
+    nbytes = 2 * T * (h * (D + m.dim + 2 * m.vdim) + m.rot_dim + m.gate_size)
+    flops = 2.0 * _seen(n, m.window) * B * h * (D + m.vdim)
+    add(f"latent_flash ({what})", time_us(lambda: ops.latent_prefill(
+        q, rows[:, m.kv_rank : m.latent_size], kv, cu, cu, n, m.dim, m.vdim, gate=gate, out=out, **kw)), nbytes, flops)
+    if m.window or m.sink:
+        add("  vs latent_flash (full causal, plain)", time_us(lambda: ops.latent_prefill(
+            q, rows[:, m.kv_rank : m.latent_size], kv, cu, cu, n, m.dim, m.vdim, scale=m.scale, gate=None, out=out)), nbytes,
+            2.0 * _seen(n, 0) * B * h * (D + m.vdim))
     per = (ctx + 15) // 16
     pages, bt = r(DB * per, 16, width), torch.randperm(DB * per, device="cuda").view(DB, per).int()
     lens, cu1 = torch.full((DB,), ctx, device="cuda", dtype=torch.int32), torch.arange(DB + 1, device="cuda", dtype=torch.int32)
@@ -279,14 +319,109 @@ def _bench_latent(add, r, m, B: int, n: int, DB: int, ctx: int) -> None:
     add("latent_queries (decode)", time_us(lambda: ops.latent_queries(q[:DB], at(uks)), iters=40),
         2 * (h * m.dim * m.kv_rank + DB * h * (D + width)), 2.0 * DB * h * m.dim * m.kv_rank)
     qa = ops.latent_queries(q[:DB], uk)
-    add("latent_decode", time_us(lambda: ops.latent_attention(qa, pages, bt, cu1, lens, m.kv_rank, scale=m.scale, max_ctx=ctx)),
-        2 * DB * (ctx * m.latent_size + h * (width + m.kv_rank)), 2.0 * DB * ctx * h * (m.latent_size + m.kv_rank))
-    lat = ops.latent_attention(qa, pages, bt, cu1, lens, m.kv_rank, scale=m.scale, max_ctx=ctx)
-    add("latent_values (decode, gate)", time_us(lambda: ops.latent_values(lat, at(uvs), gate[:DB], out[:DB]), iters=40),
-        2 * (h * m.vdim * m.kv_rank + DB * h * (m.kv_rank + 2 * m.vdim)), 2.0 * DB * h * m.vdim * m.kv_rank)
+    seen = min(ctx, m.window) if m.window else ctx
+    decode = lambda **k: ops.latent_attention(qa, pages, bt, cu1, lens, m.kv_rank, max_ctx=ctx, **k)  # noqa: E731
+
+    def cost(keys):
+        return 2 * DB * (keys * m.latent_size + h * (width + m.kv_rank)), 2.0 * DB * keys * h * (m.latent_size + m.kv_rank)
+
+    add(f"latent_decode ({what}: {seen} keys)", time_us(lambda: decode(**kw)), *cost(seen))
+    if m.window or m.sink:
+        add("  vs latent_decode (full context)", time_us(lambda: decode(scale=m.scale)), *cost(ctx))
+    lat = decode(**kw)
+    add("latent_values (decode, gate)", time_us(lambda: ops.latent_values(
+        lat, at(uvs), None if gate is None else gate[:DB], out[:DB]), iters=40),
+        2 * (h * m.vdim * m.kv_rank + DB * (h * (m.kv_rank + m.vdim) + m.gate_size)), 2.0 * DB * h * m.vdim * m.kv_rank)
     x, ws = r(DB, m.kv_rank), [uv.reshape(-1, m.kv_rank).clone() for _ in range(40)]
     add("  vs gemm with a weight of that size", time_us(lambda: ops.gemm(x, at(ws)), iters=40),
         2 * (h * m.vdim * m.kv_rank + DB * (m.kv_rank + h * m.vdim)), 2.0 * DB * h * m.vdim * m.kv_rank)
+
+
+def _bench_side(add, r, cfg, T: int) -> None:
+    H, d, L = cfg.hidden_size, cfg.side_dim, 6
+    table, ids, g = r(cfg.vocab_size, L * d), torch.randint(cfg.vocab_size, (T,), device="cuda"), r(T, d)
+    x, y, w, res = r(T, H), r(T, H), r(H), torch.randn(T, H, device="cuda")
+    wg, wp = r(d, H) * 0.02, r(H, d) * 0.02
+    add("side gate (gemm)", time_us(lambda: ops.gemm(x, wg)), 2 * (T * (H + d) + H * d), 2.0 * T * H * d)
+    add("gelu_rows", time_us(lambda: ops.gelu_rows(g, ids, table, d, d)), 6 * T * d)
+    add("side output (gemm)", time_us(lambda: ops.gemm(g, wp)), 2 * (T * (H + d) + H * d), 2.0 * T * H * d)
+    add("rmsnorm_add with the next norm (fp32 residual)", time_us(lambda: ops.rmsnorm_add(y, res, w, 1e-5, final_weight=w)), T * H * 12)
+
+
+def _bench_moe(add, r, m, H: int, T: int, tag: str) -> None:
+    E, top, ff = m.experts, m.top, m.ff
+    x, logits, res, w = r(T, H), torch.randn(T, (m.router_rows + 7) // 8 * 8, device="cuda"), torch.randn(T, H, device="cuda"), r(H)
+    counters = torch.zeros(E + 1, dtype=torch.int32, device="cuda")
+    wr = r(logits.shape[1], H) * 0.02
+    copies = 1 if T > 2048 else 8  # decode: the weights rotate, so that they come from memory
+    gus, downs = [r(E, 2 * ff, H) * 0.02 for _ in range(copies)], [r(E, H, ff) * 0.02 for _ in range(copies)]
+    turn = [0]
+
+    def at(ws):
+        turn[0] += 1
+        return ws[turn[0] % len(ws)]
+
+    add(f"router (gemm, fp32 out), {tag}", time_us(lambda: ops.gemm(x, wr, out_dtype=torch.float32)),
+        2 * (T * H + wr.numel()) + 4 * logits.numel(), 2.0 * T * wr.numel())
+    route = lambda: ops.moe_route(logits, E, top, counters, score=m.score)  # noqa: E731
+    add(f"moe_route, {tag}", time_us(route), 4 * T * (E + 3 * top))
+    rt = route()
+    top_i = rt.idx.long()
+    add("  vs moe_layout of the homogeneous models", time_us(lambda: moe_ops.moe_layout(top_i, E)), 4 * T * (E + 3 * top))
+    pairs, P = T * top, rt.rows
+    used = int((torch.bincount(rt.idx.flatten(), minlength=E) > 0).sum())
+    xs, scale, h = r(P, H), torch.rand(P, device="cuda"), r(P, ff)
+    f = _lib.fn
+    add(f"moe_gather, {tag}", time_us(lambda: f("vb_moe_gather")(
+        x.data_ptr(), H, rt.dest.data_ptr(), rt.weight.data_ptr(), T, top, H, xs.data_ptr(), scale.data_ptr(), 0, _lib.stream())),
+        2 * H * (T + pairs))
+    tok, dest = torch.arange(pairs, device="cuda") // top, rt.dest.flatten().long()
+    add("  vs index_copy of the homogeneous models", time_us(
+        lambda: torch.zeros((P, H), dtype=x.dtype, device="cuda").index_copy(0, dest, x.index_select(0, tok))), 2 * H * (T + pairs))
+    add(f"grouped gate|up, {tag}", time_us(lambda: moe_ops.grouped_product(xs, at(gus), rt.blk_expert), iters=16),
+        2 * (pairs * (H + 2 * ff) + used * 2 * ff * H), 4.0 * pairs * H * ff)
+    dense = [r(2 * ff * (top if T > 2048 else E), H) * 0.02 for _ in range(copies)]
+    add("  vs gemm of that size", time_us(lambda: ops.gemm(x, at(dense)), iters=16),
+        2 * (T * (H + dense[0].shape[0]) + dense[0].numel()), 2.0 * T * dense[0].numel())
+    del dense
+    gu = moe_ops.grouped_product(xs, gus[0], rt.blk_expert)
+    add(f"silu_glu of the routed rows, {tag}", time_us(lambda: f("vb_silu_glu")(
+        gu.data_ptr(), 2 * ff, h.data_ptr(), P, ff, scale.data_ptr(), rt.blk_expert.data_ptr(), 0, _lib.stream())), pairs * ff * 6)
+    add(f"grouped down, {tag}", time_us(lambda: moe_ops.grouped_product(h, at(downs), rt.blk_expert), iters=16),
+        2 * (pairs * (H + ff) + used * ff * H), 2.0 * pairs * H * ff)
+    out = moe_ops.grouped_product(h, downs[0], rt.blk_expert)
+    parts = ops.RoutedSum(out, rt, False, r(T, H), logits[:, E])
+    add(f"moe_combine (+ shared, residual, copy), {tag}", time_us(lambda: ops.moe_combine(parts, res, None, 1e-5, x.dtype)),
+        2 * H * (pairs + T) + 10 * T * H)
+    tw = rt.weight.to(x.dtype).unsqueeze(-1)
+    add("  vs sum and residual of the homogeneous models", time_us(lambda: ops.rmsnorm(
+        (out.index_select(0, dest).view(T, top, H) * tw).sum(1), w, 1e-5, x)), 2 * H * (pairs + T) + 6 * T * H)
+
+
+def _bench_lru(add, r, m, B: int, n: int, DB: int, ctx: int) -> None:
+    T, W = B * n, m.width
+    proj, gates = r(T, m.proj_size), r(2 * m.blocks, m.block_size, m.block_size) * m.block_size ** -0.5
+    gb, lam = torch.randn(2 * m.blocks, m.block_size, device="cuda"), torch.rand(W, device="cuda") * 6 - 5
+    conv, cb, nslot = r(W, m.conv) * 0.5, r(W), max(B, DB)
+    ring, state = r(nslot, m.conv, W), torch.zeros(nslot, W, device="cuda")
+    sl = torch.arange(nslot, device="cuda", dtype=torch.int32)
+    cu = torch.arange(B + 1, device="cuda", dtype=torch.int32) * n
+    lens = torch.full((B,), n, device="cuda", dtype=torch.int32)
+    add("rglru prefill (conv, gates, recurrence)", time_us(
+        lambda: ops.rglru(proj, conv, cb, gates, gb, lam, ring, state, cu, lens, sl[:B], n)),
+        T * 3 * W * 2, 4.0 * T * W * m.block_size)
+    cu1, lens1 = torch.arange(DB + 1, device="cuda", dtype=torch.int32), torch.full((DB,), ctx, device="cuda", dtype=torch.int32)
+    # weights, rings and states rotate, so that they come from memory
+    gs, rings, states = [gates.clone() for _ in range(16)], [ring.clone() for _ in range(16)], [state.clone() for _ in range(16)]
+    turn = [0]
+
+    def step():
+        turn[0] += 1
+        i = turn[0] % 16
+        return ops.rglru(proj[:DB], conv, cb, gs[i], gb, lam, rings[i], states[i], cu1, lens1, sl[:DB], 1)
+
+    add("rglru decode (conv, fused step)", time_us(step, iters=32),
+        2 * gates.numel() + DB * W * (3 * 2 + (m.conv + 1) * 2 + 8), 4.0 * DB * W * m.block_size)
 
 
 def _bench_delta(add, r, dl, B: int, n: int, DB: int, ctx: int) -> None:
