@@ -1216,7 +1216,7 @@ static int gemm_bf16_run(const void* A, const void* B, void* C, const void* bias
     const char* e = getenv("VERL_B200_SPLITK_CLUSTER");  // 0 = workspace + grid-barrier reduction (the older path)
     return !(e && e[0] == '0');
   }();
-  if (cluster_sk && splitk_mode != 0 && !accumulate && N > 128) {
+  if (cluster_sk && splitk_mode != 0 && !accumulate && (N > 128 || (!a_mn && !b_mn && M <= 256))) {
     // Skinny problems (decode projections): split K over the CTAs of a cluster and reduce through distributed shared
     // memory. Among tile widths {128, 64} and cluster sizes 2..8 take the pair that puts the most CTAs to work in ONE
     // wave: a cluster needs all its SMs free inside one GPC at once, so the number of co-resident clusters (asked

@@ -226,15 +226,29 @@ __global__ void glu_kernel(const T* __restrict__ gu, long long stride, T* __rest
   }
 }
 
-// y[t] = gelu(g[t]) * table[ids[t]][lo ..]. One block per token.
-template <typename T>
+// y[t] = gelu(g[t]) * table[ids[t]][lo ..]. V elements per thread.
+template <typename T, int V>
 __global__ void gelu_rows_kernel(const T* __restrict__ g, long long g_stride, const long long* __restrict__ ids,
-                                 const T* __restrict__ table, long long table_stride, int lo, T* __restrict__ y, int n) {
+                                 const T* __restrict__ table, long long table_stride, int lo, T* __restrict__ y, int n,
+                                 long long total) {
   pdl_trigger();
   pdl_wait();
-  const T* e = table + ids[blockIdx.x] * table_stride + lo;
-  for (int i = threadIdx.x; i < n; i += blockDim.x)
-    y[(long long)blockIdx.x * n + i] = from_f<T>(gelu_tanh<sizeof(T) == 2>(to_f<T>(g[blockIdx.x * g_stride + i])) * to_f<T>(e[i]));
+  const int per = n / V;
+  for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const long long t = i / per;
+    const int c = (int)(i - t * per) * V;
+    const T *src = g + t * g_stride + c, *e = table + ids[t] * table_stride + lo + c;
+    if constexpr (V == 8) {
+      float a[8], b[8];
+      ld8(src, a);
+      ld8(e, b);
+#pragma unroll
+      for (int k = 0; k < 8; ++k) a[k] = gelu_tanh<sizeof(T) == 2>(a[k]) * b[k];
+      st8(y + t * n + c, a);
+    } else {
+      y[t * n + c] = from_f<T>(gelu_tanh<sizeof(T) == 2>(to_f<T>(src[0])) * to_f<T>(e[0]));
+    }
+  }
 }
 
 // x = cap * tanh(x / cap)
@@ -824,12 +838,20 @@ extern "C" int vb_silu_glu(const void* gu, long long stride, void* y, int T, int
 extern "C" int vb_gelu_rows(const void* g, long long g_stride, const long long* ids, const void* table, long long table_stride,
                             int lo, void* y, int T, int n, int f32, cudaStream_t stream) {
   if (T <= 0 || n <= 0) return 0;
-  const dim3 grid(T), b(n >= 128 ? 128 : 64);
-  if (f32)
-    VB_DONE(vb_launch_pdl(gelu_rows_kernel<float>, grid, b, 0, stream, 1, (const float*)g, g_stride, ids, (const float*)table,
-                          table_stride, lo, (float*)y, n));
-  VB_DONE(vb_launch_pdl(gelu_rows_kernel<bf16>, grid, b, 0, stream, 1, (const bf16*)g, g_stride, ids, (const bf16*)table,
-                        table_stride, lo, (bf16*)y, n));
+  const bool vec = ((n | lo | g_stride | table_stride) & 7) == 0 &&
+                   ((reinterpret_cast<uintptr_t>(g) | reinterpret_cast<uintptr_t>(table)) & 15) == 0;
+  const long long total = (long long)T * n / (vec ? 8 : 1);
+  const dim3 grid((unsigned)min((total + 127) / 128, 148ll * 16)), b(128);
+#define VB_GR(TT, V)                                                                                                  \
+  VB_DONE(vb_launch_pdl(gelu_rows_kernel<TT, V>, grid, b, 0, stream, 1, (const TT*)g, g_stride, ids, (const TT*)table, \
+                        table_stride, lo, (TT*)y, n, total))
+  if (f32) {
+    if (vec) VB_GR(float, 8);
+    VB_GR(float, 1);
+  }
+  if (vec) VB_GR(bf16, 8);
+  VB_GR(bf16, 1);
+#undef VB_GR
 }
 
 extern "C" int vb_softcap(float* x, long long n, float cap, cudaStream_t stream) {

@@ -7,8 +7,8 @@
 //
 // lru_tc does all behind the convolution in one kernel (bf16). A CTA owns 128 channels of a block and walks a sequence, 64 tokens
 // at a time: Z^T[channels x tokens] = G[128 channels x n] . u^T on tcgen05 for both gates (weights stay in shared memory, tiles of
-// u arrive by TMA), then thread = channel: the terms of 32 tokens in registers, one dependent multiply-add per token, the carry
-// handed through shared memory to the four warps that hold the next 32 tokens. Neither gates nor decays reach memory. Steps of
+// u and of the gelu branch arrive by TMA), then thread = channel: the terms of 16 tokens in registers, one dependent multiply-add
+// per token, the carry handed through shared memory to the four warps that hold the next 16 tokens. Neither gates nor decays reach memory. Steps of
 // single tokens use the same kernel with sequences in place of tokens and the state in memory in place of the carry.
 // lru_gates and lru_scan are the same on CUDA cores (fp32, and sizes the other does not take).
 // Every wait is bounded; on expiry the status word is set and the CTA leaves through its teardown.
@@ -51,16 +51,16 @@ __device__ __forceinline__ void lru_terms(float zr, float zi, float u, float c, 
 // u[t, c] = bias[c] + sum over j of x[t - taps + 1 + j, c] w[c, j]. Thread: V channels, LC_TOKENS tokens in a row, whose earlier
 // inputs stay in registers (TAPS > 0). The row of a single token goes to its sequence's ring here; longer portions write theirs
 // behind the scan (other tokens still read the ring).
-constexpr int LC_TOKENS = 16;
+constexpr int LC_TOKENS = 16, LC_AHEAD = 8;
 template <typename T, int V, int TAPS>
 __global__ void lru_conv_kernel(const T* __restrict__ proj, const T* __restrict__ w, const T* __restrict__ bias,
-                                T* __restrict__ ring, T* __restrict__ u, const LruParams p) {
+                                T* __restrict__ ring, T* __restrict__ u, const int run, const LruParams p) {
   pdl_trigger();
   pdl_wait();
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
   if (c >= p.W) return;
   const T* x = proj + p.W;
-  const int t0 = blockIdx.x * LC_TOKENS, t1 = min(t0 + LC_TOKENS, p.T), taps = TAPS > 0 ? TAPS : p.taps;
+  const int t0 = blockIdx.x * run, t1 = min(t0 + run, p.T), taps = TAPS > 0 ? TAPS : p.taps;
   int b = seq_of(p.cu_q, p.B, t0);
   int first = 0, n_new = 0, start = 0, slot = 0;
   // input of token t's row `at` (before the portion: from the ring; before the sequence, or without a slot: zero)
@@ -88,6 +88,21 @@ __global__ void lru_conv_kernel(const T* __restrict__ proj, const T* __restrict_
 #pragma unroll
       for (int e = 0; e < V; ++e) wr[j][e] = to_f<T>(w[(long long)(c + e) * TAPS + j]);
   }
+  // u of token t from its input f and the inputs before it
+  auto shift = [&](int t, const float (&f)[V]) {
+    float acc[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      acc[e] = bias_r[e];
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) acc[e] = fmaf(hist[j][e], wr[j][e], acc[e]);
+      acc[e] = fmaf(f[e], wr[TAPS > 0 ? TAPS - 1 : 0][e], acc[e]);
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS - 1; ++j) hist[j][e] = hist[j + 1][e];
+      if (TAPS > 1) hist[TAPS > 1 ? TAPS - 2 : 0][e] = f[e];
+    }
+    if constexpr (V == 8) st8(u + (long long)t * p.W + c, acc); else u[(long long)t * p.W + c] = from_f<T>(acc[0]);
+  };
   bool fresh = true;
   for (int t = t0; t < t1; ++t) {
     if (fresh || p.cu_q[b + 1] <= t) {
@@ -102,28 +117,36 @@ __global__ void lru_conv_kernel(const T* __restrict__ proj, const T* __restrict_
       }
       fresh = false;
     }
-    float acc[V], f[V];
+    if constexpr (TAPS > 0 && V == 8 && sizeof(T) == 2) {
+      if (t + LC_AHEAD <= t1 && t + LC_AHEAD <= first + n_new && n_new > 1) {  // several inputs on their way at once
+        uint4 raw[LC_AHEAD];
 #pragma unroll
-    for (int e = 0; e < V; ++e) acc[e] = bias_r[e];
+        for (int i = 0; i < LC_AHEAD; ++i) raw[i] = __ldg(reinterpret_cast<const uint4*>(x + (t + i) * p.stride + c));
+#pragma unroll
+        for (int i = 0; i < LC_AHEAD; ++i) {
+          float f[V];
+          ld8(reinterpret_cast<const T*>(&raw[i]), f);
+          shift(t + i, f);
+        }
+        t += LC_AHEAD - 1;
+        continue;
+      }
+    }
+    float f[V];
     if constexpr (TAPS > 0) {
       load(t, f);
-#pragma unroll
-      for (int e = 0; e < V; ++e) {
-#pragma unroll
-        for (int j = 0; j < TAPS - 1; ++j) acc[e] = fmaf(hist[j][e], wr[j][e], acc[e]);
-        acc[e] = fmaf(f[e], wr[TAPS - 1][e], acc[e]);
-#pragma unroll
-        for (int j = 0; j + 1 < TAPS - 1; ++j) hist[j][e] = hist[j + 1][e];
-        if (TAPS > 1) hist[TAPS > 1 ? TAPS - 2 : 0][e] = f[e];
-      }
+      shift(t, f);
     } else {
+      float acc[V];
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc[e] = bias_r[e];
       for (int j = 0; j < taps; ++j) {
         load(t - taps + 1 + j, f);
 #pragma unroll
         for (int e = 0; e < V; ++e) acc[e] = fmaf(f[e], to_f<T>(w[(long long)(c + e) * taps + j]), acc[e]);
       }
+      if constexpr (V == 8) st8(u + (long long)t * p.W + c, acc); else u[(long long)t * p.W + c] = from_f<T>(acc[0]);
     }
-    if constexpr (V == 8) st8(u + (long long)t * p.W + c, acc); else u[(long long)t * p.W + c] = from_f<T>(acc[0]);
     if (n_new == 1 && slot >= 0) {
       T* dst = ring + ((long long)slot * taps + start % taps) * p.W + c;
       if constexpr (V == 8) {
@@ -191,20 +214,24 @@ __global__ void lru_scan_kernel(const T* __restrict__ proj, const float* __restr
 }
 
 // ------------------------------------------------------------------------------------------------ gates and recurrence, tcgen05
-constexpr int LT_EPI = 8, LT_THREADS = (LT_EPI + 2) * 32, LT_MAX_STAGES = 3, LT_TOKENS = 64, LT_STEP_TOKENS = 32;
+constexpr int LT_COLS = 16;  // tokens of a group of four warps
+constexpr int LT_MAX_STAGES = 3, LT_TOKENS = 64, LT_STEP_TOKENS = 32;
 constexpr float LT_LOG2E = 1.4426950408889634f;
 
 template <int NT>
 struct LtCfg {
+  static constexpr int GROUPS = NT / LT_COLS, EPI = 4 * GROUPS, THREADS = (EPI + 2) * 32;
   static constexpr int KB_W = 128 * 128, KB_U = NT * 128;  // bytes of 64 columns of a gate's weights, of a tile of u
   static constexpr int TMEM = 4 * NT;                      // two stages of both gates' logits
-  static constexpr int TAIL = 256 + 2 * 128 * 4;           // barriers, carries
-  static __host__ __device__ int bytes(int kb, int stages) { return 2 * kb * KB_W + stages * kb * KB_U + TAIL + 1024; }
+  static constexpr int TAIL = 512 + GROUPS * 128 * 4;      // barriers, carries
+  // a stage: the block's columns of u, 128 of the gelu branch
+  static __host__ __device__ int stage(int kb) { return (kb + 2) * KB_U; }
+  static __host__ __device__ int bytes(int kb, int stages) { return 2 * kb * KB_W + stages * stage(kb) + TAIL + 1024; }
 };
 
 struct LruTcParams {
   LruParams l;
-  const __nv_bfloat16 *proj, *u;
+  const __nv_bfloat16* proj;
   __nv_bfloat16 *ring, *out;
   int kb, tiles, stages, seq0;  // 64-column parts of a block, 128-channel tiles of a block, first sequence
   int steps;                    // STEP: rows (one token each)
@@ -216,18 +243,28 @@ __device__ __forceinline__ float sqrt_approx(float x) {
   asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+__device__ __forceinline__ float ex2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcp_approx(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 
-// The terms of the recurrence from the gates' logits and the input, and the gelu branch; cl = -power * softplus(lam) * log2(e).
-// The three sigmoids share one reciprocal: their denominators are bounded so that the product stays finite (below e^-28 a sigmoid
-// is nothing beside what it is added to or multiplied with here).
-__device__ __forceinline__ void lru_terms_fast(float zr, float zi, float u, float g, float cl, float& a, float& v, float& y) {
-  const float z = 0.7978845608028654f * (g + 0.044715f * g * g * g);
-  const float A = 1.f + exp2f(fminf(-zr * LT_LOG2E, 40.f)), B = 1.f + exp2f(fminf(-zi * LT_LOG2E, 40.f)),
-              C = 1.f + exp2f(fminf(-2.f * LT_LOG2E * z, 40.f));
-  const float ab = A * B, q = __fdividef(1.f, ab * C), qc = q * C;
-  y = g * q * ab;
+// The terms of the recurrence from the gates' logits and the input, and the gelu branch; nr, ni = the logits times -log2(e),
+// cl = -power * softplus(lam) * log2(e). The three sigmoids share one reciprocal: their denominators are bounded so that the
+// product stays finite (below e^-28 a sigmoid is nothing beside what it is added to or multiplied with here).
+__device__ __forceinline__ void lru_terms_fast(float nr, float ni, float u, float g, float cl, float& a, float& v, float& y) {
+  constexpr float K1 = -2.f * LT_LOG2E * 0.7978845608028654f, K3 = K1 * 0.044715f;
+  const float A = 1.f + ex2_approx(fminf(nr, 40.f)), B = 1.f + ex2_approx(fminf(ni, 40.f)),
+              C = 1.f + ex2_approx(fminf(g * fmaf(K3, g * g, K1), 40.f));
+  const float ab = A * B, q = rcp_approx(ab * C), qc = q * C;
+  y = g * (q * ab);
   const float la = cl * (qc * B);  // log2 of the decay
-  a = exp2f(la);
+  a = ex2_approx(la);
   // 1 - a^2 = -expm1(x), x = 2 ln(2) la: by its series near zero, where the difference would cancel
   const float x = 1.3862943611198906f * la;
   float e = fmaf(x, 1.f / 5040.f, 1.f / 720.f);
@@ -240,26 +277,21 @@ __device__ __forceinline__ void lru_terms_fast(float zr, float zi, float u, floa
   v = sqrt_approx(s) * (qc * A) * u;
 }
 
-template <int COLS>
-__device__ __forceinline__ void lt_cols(uint32_t addr, uint32_t (&v)[COLS]) {
-  if constexpr (COLS == 32) tmem_ld_32x32(addr, v);
-  else tmem_ld_32x16(addr, v);
-}
-
 template <int NT, bool STEP>
-__global__ void __launch_bounds__(LT_THREADS, 1)
-lru_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmU, const LruTcParams p) {
+__global__ void __launch_bounds__(LtCfg<NT>::THREADS, 1)
+lru_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmU,
+              const __grid_constant__ CUtensorMap tmY, const LruTcParams p) {
   using Cfg = LtCfg<NT>;
-  constexpr int COLS = NT / 2;  // tokens of one group of four warps
+  constexpr int GROUPS = Cfg::GROUPS, EPI = Cfg::EPI;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  const int kb = p.kb, stages = p.stages, u_off = 2 * kb * Cfg::KB_W, u_stage = kb * Cfg::KB_U;
-  uint64_t* w_full = reinterpret_cast<uint64_t*>(smem + u_off + stages * u_stage);
+  const int kb = p.kb, stages = p.stages, u_off = 2 * kb * Cfg::KB_W, stage_bytes = Cfg::stage(kb);
+  uint64_t* w_full = reinterpret_cast<uint64_t*>(smem + u_off + stages * stage_bytes);
   uint64_t *u_full = w_full + 1, *u_empty = u_full + LT_MAX_STAGES, *t_full = u_empty + LT_MAX_STAGES, *t_empty = t_full + 2,
            *carry = t_empty + 2;  // carry[group * 4 + warp of the group]
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(carry + 8);
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(carry + EPI);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  float* carry_s = reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(w_full) + 256);  // [group][channel]
+  float* carry_s = reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(w_full) + 512);  // [group][channel]
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int blk = blockIdx.x / p.tiles, m0 = (blockIdx.x - blk * p.tiles) * 128;  // first channel of the tile in its block
   const int W = p.l.W, n = p.l.n;
@@ -281,17 +313,17 @@ lru_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ C
     mbar_init(w_full, 1);
     for (int s = 0; s < LT_MAX_STAGES; ++s) {
       mbar_init(&u_full[s], 1);
-      mbar_init(&u_empty[s], LT_EPI);
+      mbar_init(&u_empty[s], EPI);
     }
     for (int i = 0; i < 2; ++i) {
       mbar_init(&t_full[i], 1);
-      mbar_init(&t_empty[i], LT_EPI);
+      mbar_init(&t_empty[i], EPI);
     }
-    for (int i = 0; i < 8; ++i) mbar_init(&carry[i], 1);
+    for (int i = 0; i < EPI; ++i) mbar_init(&carry[i], 1);
     *abort_flag = 0;
     mbar_fence_init();
   }
-  if (warp == LT_EPI + 1) {
+  if (warp == EPI + 1) {
     tmem_alloc(tmem_slot, Cfg::TMEM);
     tmem_relinquish();
   }
@@ -301,7 +333,7 @@ lru_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ C
   const uint32_t tmem = *tmem_slot;  // stage s: decay logits at s * 2 NT, input logits NT behind them
   pdl_trigger();
 
-  if (warp == LT_EPI) {
+  if (warp == EPI) {
     // ------------------------------- TMA producer -------------------------------
     if (elect_one()) {
       const int blocks = W / n;
@@ -317,15 +349,17 @@ lru_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ C
           *abort_flag = 1;
           break;
         }
-        mbar_arrive_expect_tx(&u_full[s], u_stage);
-        for (int k = 0; k < kb; ++k)
-          tma_load_3d(smem + u_off + s * u_stage + k * Cfg::KB_U, &tmU, &u_full[s], k * 64, blk, first + c * NT);
+        uint8_t* dst = smem + u_off + s * stage_bytes;
+        mbar_arrive_expect_tx(&u_full[s], stage_bytes);
+        for (int k = 0; k < kb; ++k) tma_load_3d(dst + k * Cfg::KB_U, &tmU, &u_full[s], k * 64, blk, first + c * NT);
+        for (int k = 0; k < 2; ++k)
+          tma_load_2d(dst + (kb + k) * Cfg::KB_U, &tmY, &u_full[s], blk * n + m0 + k * 64, first + c * NT);
       }
       // no copy is in flight when the CTA ends, whatever ended it
       mbar_wait(w_full, 0);
       for (int i = max(c - stages, 0); i < c; ++i) mbar_wait(&u_full[i % stages], (i / stages) & 1);
     }
-  } else if (warp == LT_EPI + 1) {
+  } else if (warp == EPI + 1) {
     // -------------------------------- MMA issuer --------------------------------
     if (elect_one()) {
       constexpr uint32_t idesc = umma_idesc(1, 1, 0, 0, 128, NT);  // A = weights, B = u, both K-major
@@ -345,7 +379,7 @@ lru_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ C
           for (int k = 0; k < k_steps; ++k)
             tc_mma_f16(tmem + (c & 1) * 2 * NT + g * NT,
                        umma_smem_desc(w_addr + (g * kb + (k >> 2)) * Cfg::KB_W + (k & 3) * 32, 16, 1024),
-                       umma_smem_desc(u_addr + s * u_stage + (k >> 2) * Cfg::KB_U + (k & 3) * 32, 16, 1024), idesc, k != 0);
+                       umma_smem_desc(u_addr + s * stage_bytes + (k >> 2) * Cfg::KB_U + (k & 3) * 32, 16, 1024), idesc, k != 0);
         tc_commit(&t_full[c & 1]);
       }
     }
@@ -354,25 +388,34 @@ lru_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ C
     const int group = warp >> 2, quad = warp & 3, row = quad * 32 + lane;  // row: channel of the tile
     const bool on = m0 + row < n;
     const int kc = on ? m0 + row : 0, ch = blk * n + kc;  // channel of the block, of the layer
-    const float br = p.l.gates_b[ch], bi = p.l.gates_b[W + ch], cl = -p.l.power * softplus_f(p.l.lam[ch]) * LT_LOG2E;
-    const __nv_bfloat16* y_src = p.proj + ch;
-    const uint32_t t_addr = tmem + (((uint32_t)(quad * 32)) << 16) + group * COLS;
-    const uint8_t* u_src = smem + u_off + (kc >> 6) * Cfg::KB_U + (kc & 7) * 2;
-    const int c16 = (kc & 63) >> 3;
+    const float br = -LT_LOG2E * p.l.gates_b[ch], bi = -LT_LOG2E * p.l.gates_b[W + ch],
+                cl = -p.l.power * softplus_f(p.l.lam[ch]) * LT_LOG2E;
+    const uint32_t t_addr = tmem + (((uint32_t)(quad * 32)) << 16) + group * LT_COLS;
+    // tiles are swizzled: element (row r, column k of a 64-column part) lies at (r / 8) * 1024 + (r % 8) * 128, in 16-byte piece
+    // (k / 8) ^ (r % 8); this group's rows start at a multiple of 8
+    const uint8_t *u_src = smem + u_off + (kc >> 6) * Cfg::KB_U + group * (LT_COLS / 8) * 1024 + (kc & 7) * 2,
+                  *y_src = smem + u_off + (kb + (row >> 6)) * Cfg::KB_U + group * (LT_COLS / 8) * 1024 + (row & 7) * 2;
+    const int cu = (kc & 63) >> 3, cy = (row & 63) >> 3;
     int slot = 0, len = 0;
-    float S = 0.f;
-    if (!STEP) {
+    float S = 0.f, S0[STEP ? LT_COLS : 1];
+    if constexpr (STEP) {  // state of the sequences, on its way while the gates are computed
+#pragma unroll
+      for (int j = 0; j < LT_COLS; ++j) {
+        const int t = first + group * LT_COLS + j;
+        S0[j] = 0.f;
+        if (t < first + nq && on) {
+          const int sl = p.l.slots[t];
+          if (sl >= 0 && p.l.seq_lens[t] > 1) S0[j] = p.l.state[(long long)sl * W + ch];
+        }
+      }
+    } else {
       slot = p.l.slots[b];
       len = p.l.seq_lens[b];
       if (group == 0 && slot >= 0 && len > nq) S = p.l.state[(long long)slot * W + ch];
     }
     bool ok = true;
     for (int c = 0; c < chunks; ++c) {
-      const int s = c % stages, tok0 = c * NT + group * COLS, live = max(min(nq - tok0, COLS), 0);
-      float y[COLS];
-#pragma unroll
-      for (int j = 0; j < COLS; ++j)
-        y[j] = j < live && on ? __bfloat162float(y_src[(long long)(first + tok0 + j) * p.l.stride]) : 0.f;
+      const int s = c % stages, tok0 = c * NT + group * LT_COLS, live = max(min(nq - tok0, LT_COLS), 0);
       if (*abort_flag || !mbar_wait(&u_full[s], (c / stages) & 1) || !mbar_wait(&t_full[c & 1], (c >> 1) & 1)) {
         report_error(p.status, ERR_WAIT_TMEM_FULL, c);
         *abort_flag = 1;
@@ -381,66 +424,79 @@ lru_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ C
       ok = __all_sync(0xffffffffu, ok);  // the lanes of a warp share its TMEM accesses: they stop together
       if (!ok) break;
       tc_fence_after();
-      float a[COLS], v[COLS];
+      float a[LT_COLS], v[LT_COLS], y[LT_COLS];
       {
-        uint32_t zr[COLS], zi[COLS];
-        lt_cols<COLS>(t_addr + (c & 1) * 2 * NT, zr);
-        lt_cols<COLS>(t_addr + (c & 1) * 2 * NT + NT, zi);
+        uint32_t zr[LT_COLS], zi[LT_COLS];
+        tmem_ld_32x16(t_addr + (c & 1) * 2 * NT, zr);
+        tmem_ld_32x16(t_addr + (c & 1) * 2 * NT + NT, zi);
         tmem_ld_wait();
         tc_fence_before();
         __syncwarp();
         if (lane == 0) mbar_arrive(&t_empty[c & 1]);
+        const uint8_t *us = u_src + s * stage_bytes, *ys = y_src + s * stage_bytes;
 #pragma unroll
-        for (int j = 0; j < COLS; ++j) {
-          const int r = group * COLS + j;  // row of the tile of u
-          const float u = __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(
-              u_src + s * u_stage + (r >> 3) * 1024 + (r & 7) * 128 + ((c16 ^ (r & 7)) << 4)));
-          lru_terms_fast(__uint_as_float(zr[j]) + br, __uint_as_float(zi[j]) + bi, u, y[j], cl, a[j], v[j], y[j]);
-          if (j >= live) {  // past the portion: the state stays
-            a[j] = 1.f;
-            v[j] = 0.f;
-          }
+        for (int j = 0; j < LT_COLS; ++j) {
+          const int at = (j >> 3) * 1024 + (j & 7) * 128;
+          const float u = __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(us + at + ((cu ^ (j & 7)) << 4)));
+          const float g = __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(ys + at + ((cy ^ (j & 7)) << 4)));
+          lru_terms_fast(fmaf(__uint_as_float(zr[j]), -LT_LOG2E, br), fmaf(__uint_as_float(zi[j]), -LT_LOG2E, bi), u, g, cl, a[j],
+                         v[j], y[j]);
         }
       }
       __syncwarp();
       if (lane == 0) mbar_arrive(&u_empty[s]);
-      if (STEP) {
+      if constexpr (STEP) {
 #pragma unroll
-        for (int j = 0; j < COLS; ++j) {
+        for (int j = 0; j < LT_COLS; ++j) {
           if (j < live && on) {
             const int t = first + tok0 + j, sl = p.l.slots[t];
-            float* st = p.l.state + (long long)max(sl, 0) * W + ch;
-            const float S1 = fmaf(a[j], sl >= 0 && p.l.seq_lens[t] > 1 ? *st : 0.f, v[j]);
-            if (sl >= 0) *st = S1;
+            const float S1 = fmaf(a[j], S0[j], v[j]);
+            if (sl >= 0) p.l.state[(long long)sl * W + ch] = S1;
             p.out[(long long)t * W + ch] = __float2bfloat16(sl >= 0 ? S1 * y[j] : 0.f);
           }
         }
         continue;
       }
-      if (group == 1 || c > 0) {  // from the group that holds the tokens before these
-        if (*abort_flag || !mbar_wait(&carry[(group ^ 1) * 4 + quad], (group == 1 ? c : c - 1) & 1)) {
+      if (live < LT_COLS) {  // past the portion the state stays
+#pragma unroll
+        for (int j = 0; j < LT_COLS; ++j)
+          if (j >= live) {
+            a[j] = 1.f;
+            v[j] = 0.f;
+          }
+      }
+      if (group > 0 || c > 0) {  // from the group that holds the tokens before these
+        const int from = group > 0 ? group - 1 : GROUPS - 1;
+        if (*abort_flag || !mbar_wait(&carry[from * 4 + quad], (group > 0 ? c : c - 1) & 1)) {
           report_error(p.status, ERR_WAIT_FLAG, c);
           *abort_flag = 1;
           ok = false;
         }
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
-        S = carry_s[(group ^ 1) * 128 + row];
+        S = carry_s[from * 128 + row];
       }
 #pragma unroll
-      for (int j = 0; j < COLS; ++j) {
+      for (int j = 0; j < LT_COLS; ++j) {
         S = fmaf(a[j], S, v[j]);
         a[j] = S;
       }
       carry_s[group * 128 + row] = S;
       __syncwarp();
       if (lane == 0) mbar_arrive(&carry[group * 4 + quad]);
+      __nv_bfloat16* dst = p.out + (long long)(first + tok0) * W + ch;
+      if (on) {
+        if (live == LT_COLS && slot >= 0) {
 #pragma unroll
-      for (int j = 0; j < COLS; ++j)
-        if (j < live && on)
-          p.out[(long long)(first + tok0 + j) * W + ch] = __float2bfloat16(slot >= 0 ? a[j] * y[j] : 0.f);
+          for (int j = 0; j < LT_COLS; ++j, dst += W) *dst = __float2bfloat16(a[j] * y[j]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < LT_COLS; ++j, dst += W)
+            if (j < live) *dst = __float2bfloat16(slot >= 0 ? a[j] * y[j] : 0.f);
+        }
+      }
     }
-    if (!STEP && ok && group == 1 && on && slot >= 0) {  // S: behind the last token
+    if (!STEP && ok && group == GROUPS - 1 && on && slot >= 0) {  // S: behind the last token
       p.l.state[(long long)slot * W + ch] = S;
       if (nq > 1) write_ring<__nv_bfloat16>(p.proj + W, p.ring, p.l, first, nq, len, slot, ch);
     }
@@ -448,7 +504,7 @@ lru_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ C
 
   tc_fence_before();
   __syncthreads();
-  if (warp == LT_EPI + 1) {
+  if (warp == EPI + 1) {
     tc_fence_after();
     tmem_dealloc(tmem, Cfg::TMEM);
   }
@@ -462,10 +518,11 @@ typedef __nv_bfloat16 bf16;
 template <typename T, int V>
 static cudaError_t launch_conv(const void* proj, const void* w, const void* bias, void* ring, void* u, const LruParams& p,
                                cudaStream_t stream) {
-  const int threads = p.W / V >= 256 ? 256 : 64;
-  const dim3 g((p.T + LC_TOKENS - 1) / LC_TOKENS, (p.W / V + threads - 1) / threads);
+  const int threads = p.W / V >= 256 ? 128 : 64;
+  const int run = p.T >= 8 * p.B ? LC_TOKENS : 1;  // mostly single tokens: nothing to keep from one to the next
+  const dim3 g((p.T + run - 1) / run, (p.W / V + threads - 1) / threads);
 #define VB_LC(N) vb_launch_pdl(lru_conv_kernel<T, V, N>, g, dim3(threads), 0, stream, 1, (const T*)proj, (const T*)w, (const T*)bias, \
-                               (T*)ring, (T*)u, p)
+                               (T*)ring, (T*)u, run, p)
   vb_count_launch();
   switch (p.taps) {
     case 1: return VB_LC(1);
@@ -501,10 +558,11 @@ extern "C" int vb_rglru_tc_supported(int W, int n) {
 }
 
 template <int NT, bool STEP>
-static int launch_tc(const CUtensorMap& tmW, LruTcParams p, int rows, cudaStream_t stream) {
-  CUtensorMap tmU;
+static int launch_tc(const CUtensorMap& tmW, const void* u, LruTcParams p, int rows, cudaStream_t stream) {
+  CUtensorMap tmU, tmY;
   const uint64_t n = p.l.n, W = p.l.W;
-  int rc = vb_make_tmap_3d(&tmU, p.u, 2, n, W / n, p.l.T, n * 2, W * 2, 64, 1, NT);
+  int rc = vb_make_tmap_3d(&tmU, u, 2, n, W / n, p.l.T, n * 2, W * 2, 64, 1, NT);
+  if (!rc) rc = vb_make_tmap_2d(&tmY, p.proj, 2, W, p.l.T, (uint64_t)p.l.stride * 2, 64, NT);
   if (rc) return rc;
   p.stages = lt_stages<NT>(p.kb);
   if (STEP) p.stages = 1;
@@ -513,8 +571,8 @@ static int launch_tc(const CUtensorMap& tmW, LruTcParams p, int rows, cudaStream
     VB_CUDA_CHECK(cudaFuncSetAttribute(lru_tc_kernel<NT, STEP>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
     attr_set = true;
   }
-  VB_DONE(vb_launch_pdl(lru_tc_kernel<NT, STEP>, dim3(p.tiles * (p.l.W / p.l.n), rows), dim3(LT_THREADS),
-                        (size_t)LtCfg<NT>::bytes(p.kb, p.stages), stream, 1, tmW, tmU, p));
+  VB_DONE(vb_launch_pdl(lru_tc_kernel<NT, STEP>, dim3(p.tiles * (p.l.W / p.l.n), rows), dim3(LtCfg<NT>::THREADS),
+                        (size_t)LtCfg<NT>::bytes(p.kb, p.stages), stream, 1, tmW, tmU, tmY, p));
 }
 
 // proj [T, stride] (gelu branch | recurrent branch), conv_w [W, taps], gates [2, W / n, n, n], gates_b [2, W], lam [W] fp32, ring
@@ -542,14 +600,14 @@ extern "C" int vb_rglru(const void* proj, long long stride, const void* conv_w, 
   if (rc) return rc;
   LruTcParams q{};
   q.l = p;
-  q.proj = (const bf16*)proj; q.u = (const bf16*)u; q.ring = (bf16*)ring; q.out = (bf16*)out;
+  q.proj = (const bf16*)proj; q.ring = (bf16*)ring; q.out = (bf16*)out;
   q.kb = (n + 63) / 64; q.tiles = (n + 127) / 128; q.status = status;
   if (singles > 0) {
     q.steps = singles;
-    rc = launch_tc<LT_STEP_TOKENS, true>(tmW, q, (singles + LT_STEP_TOKENS - 1) / LT_STEP_TOKENS, stream);
+    rc = launch_tc<LT_STEP_TOKENS, true>(tmW, u, q, (singles + LT_STEP_TOKENS - 1) / LT_STEP_TOKENS, stream);
     if (rc) return rc;
   }
   if (singles == B) return 0;
   q.seq0 = singles;
-  return launch_tc<LT_TOKENS, false>(tmW, q, B - singles, stream);
+  return launch_tc<LT_TOKENS, false>(tmW, u, q, B - singles, stream);
 }

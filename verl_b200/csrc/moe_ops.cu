@@ -251,9 +251,10 @@ extern "C" int vb_moe_route(const float* logits, long long stride, int T, int E,
   if (E <= 0 || E > MR_MAX_E || top <= 0 || top > MR_MAX_TOP || top > E ||
       (long long)nblk * MR_BLK + MR_BLK <= (long long)T * top + (long long)min(E, T * top) * (MR_BLK - 1))
     return -3;
-  const bool small = T <= 256;
-  MoeRouteParams p{logits, stride, T, E, top, softmax, renormalize, small ? T : 64, nblk, idx, dest, blk_expert, weight, counters};
-  const dim3 g(small ? 1 : (T + 63) / 64), b(small ? (T >= 32 ? 1024 : (T + 3) / 4 * 128) : 256);
+  const bool small = T <= 32;
+  const int per = small ? T : (T <= 4096 ? 8 : 64);
+  MoeRouteParams p{logits, stride, T, E, top, softmax, renormalize, per, nblk, idx, dest, blk_expert, weight, counters};
+  const dim3 g((T + per - 1) / per), b(small ? (T + 3) / 4 * 128 : 256);
 #define VB_MR(NV) e = vb_launch_pdl(moe_route_kernel<NV>, g, b, 0, stream, 1, p)
   cudaError_t e;
   if (E <= 32) VB_MR(1);

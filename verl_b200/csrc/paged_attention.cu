@@ -207,27 +207,46 @@ __global__ void decode_merge_kernel(const float* __restrict__ o_part, const floa
   out[(long long)b * out_stride + (long long)hq * D + d] = __float2bfloat16(l > 0.f ? o / l : 0.f);
 }
 
-// The same for any head size, times the sigmoid of a gate [B, Hq * D] (or null).
+// The same for any head size, times the sigmoid of a gate [B, Hq * D] (or null). Dynamic shared memory: num_splits floats.
 __global__ void decode_merge_any_kernel(const float* __restrict__ o_part, const float* __restrict__ ml_part, int Hq, int D,
                                         int num_splits, __nv_bfloat16* __restrict__ out, long long out_stride,
                                         const __nv_bfloat16* __restrict__ gate, long long gate_stride) {
+  extern __shared__ float weight[];  // of each split's partial result
   const int b = blockIdx.x, hq = blockIdx.y;
   const long long base = ((long long)b * Hq + hq) * num_splits;
+  const float2* ml = reinterpret_cast<const float2*>(ml_part) + base;
   float m = -INFINITY, l = 0.f;
-  for (int s = 0; s < num_splits; ++s) m = fmaxf(m, ml_part[(base + s) * 2]);
-  for (int s = 0; s < num_splits; ++s) {
-    const float ms = ml_part[(base + s) * 2];
-    l += ms == -INFINITY ? 0.f : ml_part[(base + s) * 2 + 1] * __expf(ms - m);
-  }
-  for (int d = threadIdx.x; d < D; d += blockDim.x) {
-    float o = 0.f;
+#pragma unroll 4
+  for (int s = 0; s < num_splits; ++s) m = fmaxf(m, ml[s].x);
+#pragma unroll 4
+  for (int s = 0; s < num_splits; ++s) l += ml[s].x == -INFINITY ? 0.f : ml[s].y * __expf(ml[s].x - m);
+  const float inv = l > 0.f ? 1.f / l : 0.f;
+  for (int s = threadIdx.x; s < num_splits; s += blockDim.x) weight[s] = ml[s].x == -INFINITY ? 0.f : __expf(ml[s].x - m) * inv;
+  __syncthreads();
+  const float* o_row = o_part + base * D;
+  const int step = (D & 3) == 0 ? 4 : 1;
+  for (int d = threadIdx.x * step; d < D; d += blockDim.x * step) {
+    float o[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
     for (int s = 0; s < num_splits; ++s) {
-      const float ms = ml_part[(base + s) * 2];
-      if (ms != -INFINITY) o += o_part[(base + s) * D + d] * __expf(ms - m);
+      const float w = weight[s];
+      if (w == 0.f) continue;  // nothing was written there
+      if (step == 4) {
+        const float4 f = *reinterpret_cast<const float4*>(o_row + (long long)s * D + d);
+        o[0] = fmaf(f.x, w, o[0]);
+        o[1] = fmaf(f.y, w, o[1]);
+        o[2] = fmaf(f.z, w, o[2]);
+        o[3] = fmaf(f.w, w, o[3]);
+      } else {
+        o[0] = fmaf(o_row[(long long)s * D + d], w, o[0]);
+      }
     }
-    o = l > 0.f ? o / l : 0.f;
-    if (gate) o = __fdividef(o, 1.f + __expf(-__bfloat162float(gate[(long long)b * gate_stride + (long long)hq * D + d])));
-    out[(long long)b * out_stride + (long long)hq * D + d] = __float2bfloat16(o);
+    for (int e = 0; e < step; ++e) {
+      float x = o[e];
+      if (gate)
+        x = __fdividef(x, 1.f + __expf(-__bfloat162float(gate[(long long)b * gate_stride + (long long)hq * D + d + e])));
+      out[(long long)b * out_stride + (long long)hq * D + d + e] = __float2bfloat16(x);
+    }
   }
 }
 
@@ -279,7 +298,7 @@ int vb_decode_merge_128(const float* o_part, const float* ml_part, int B, int Hq
 
 int vb_decode_merge(const float* o_part, const float* ml_part, int B, int Hq, int D, int num_splits, void* out,
                     long long out_stride, const void* gate, long long gate_stride, cudaStream_t stream) {
-  decode_merge_any_kernel<<<dim3(B, Hq), D <= 64 ? 64 : 128, 0, stream>>>(o_part, ml_part, Hq, D, num_splits, (__nv_bfloat16*)out,
+  decode_merge_any_kernel<<<dim3(B, Hq), D <= 256 ? 64 : 128, num_splits * sizeof(float), stream>>>(o_part, ml_part, Hq, D, num_splits, (__nv_bfloat16*)out,
                                                                           out_stride, (const __nv_bfloat16*)gate, gate_stride);
   return (int)cudaGetLastError();
 }
