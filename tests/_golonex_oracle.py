@@ -9,7 +9,7 @@ from __future__ import annotations
 
 import torch
 
-from _padodra_oracle import attend, gelu_tanh, plain_frequencies, rms_norm, rotate, sigmoid, yarn_frequencies  # noqa: F401
+from _padodra_oracle import attend, causal_mask, gelu_tanh, plain_frequencies, rms_norm, rotate, sigmoid, yarn_frequencies  # noqa: F401
 
 
 def window_mask(T, size):

@@ -167,29 +167,28 @@ __device__ __forceinline__ void write_ring(const T* __restrict__ x, T* __restric
     ring[((long long)slot * p.taps + pos % p.taps) * p.W + c] = x[(first + pos - (len - nq)) * p.stride + c];
 }
 
-// Decays and inputs [2, T, W] on the CUDA cores. One block per token and 128 channels.
+// Decays and inputs [2, T, W] on the CUDA cores. One block per token and 128 channels. gates null: ab holds the products.
 template <typename T>
 __global__ void lru_gates_kernel(const T* __restrict__ u, const T* __restrict__ gates, float* __restrict__ ab, const LruParams p) {
-  extern __shared__ float row[];
   pdl_trigger();
   pdl_wait();
-  const long long t = blockIdx.x;
-  for (int i = threadIdx.x; i < p.W; i += blockDim.x) row[i] = to_f<T>(u[t * p.W + i]);
-  __syncthreads();
   const int c = blockIdx.y * blockDim.x + threadIdx.x;
   if (c >= p.W) return;
-  const int blk = c / p.n;
-  const T *gr = gates + (long long)c * p.n, *gi = gr + (long long)p.W * p.n;
-  const float* ub = row + blk * p.n;
+  const T* ut = u + (long long)blockIdx.x * p.W;
+  float *pa = ab + (long long)blockIdx.x * p.W + c, *pv = pa + (long long)p.T * p.W;
   float zr = p.gates_b[c], zi = p.gates_b[p.W + c];
-  for (int k = 0; k < p.n; ++k) {
-    zr = fmaf(ub[k], to_f<T>(gr[k]), zr);
-    zi = fmaf(ub[k], to_f<T>(gi[k]), zi);
+  if (gates) {
+    const T *gr = gates + (long long)c * p.n, *gi = gr + (long long)p.W * p.n, *ub = ut + c / p.n * p.n;
+    for (int k = 0; k < p.n; ++k) {
+      const float f = to_f<T>(ub[k]);
+      zr = fmaf(f, to_f<T>(gr[k]), zr);
+      zi = fmaf(f, to_f<T>(gi[k]), zi);
+    }
+  } else {
+    zr += *pa;
+    zi += *pv;
   }
-  float a, v;
-  lru_terms(zr, zi, row[c], -p.power * softplus_f(p.lam[c]), a, v);
-  ab[t * p.W + c] = a;
-  ab[((long long)p.T + t) * p.W + c] = v;
+  lru_terms(zr, zi, to_f<T>(ut[c]), -p.power * softplus_f(p.lam[c]), *pa, *pv);
 }
 
 // One thread per sequence and channel.
@@ -535,10 +534,10 @@ static cudaError_t launch_conv(const void* proj, const void* w, const void* bias
 }
 
 template <typename T>
-static int rglru_simt(const void* proj, const void* gates, void* ring, void* u, float* ab, void* out, const LruParams& p,
+static int rglru_simt(const void* proj, const void* gates, void* ring, const void* u, float* ab, void* out, const LruParams& p,
                       cudaStream_t stream) {
-  cudaError_t e = vb_launch_pdl(lru_gates_kernel<T>, dim3(p.T, (p.W + 127) / 128), dim3(128), (size_t)p.W * 4, stream, 1,
-                                (const T*)u, (const T*)gates, ab, p);
+  cudaError_t e = vb_launch_pdl(lru_gates_kernel<T>, dim3(p.T, (p.W + 127) / 128), dim3(128), 0, stream, 1, (const T*)u,
+                                (const T*)gates, ab, p);
   vb_count_launch();
   if (e != cudaSuccess) return (int)e;
   VB_DONE(vb_launch_pdl(lru_scan_kernel<T>, dim3((p.W + 63) / 64, p.B), dim3(64), 0, stream, 1, (const T*)proj, (const float*)ab,
@@ -575,23 +574,32 @@ static int launch_tc(const CUtensorMap& tmW, const void* u, LruTcParams p, int r
                         (size_t)LtCfg<NT>::bytes(p.kb, p.stages), stream, 1, tmW, tmU, tmY, p));
 }
 
-// proj [T, stride] (gelu branch | recurrent branch), conv_w [W, taps], gates [2, W / n, n, n], gates_b [2, W], lam [W] fp32, ring
-// [slots, taps, W], state fp32 [slots, W], u [T, W] scratch, ab fp32 [2, T, W] scratch (without tc), out [T, W]. The leading
-// `singles` sequences have one token each.
-extern "C" int vb_rglru(const void* proj, long long stride, const void* conv_w, const void* conv_b, const void* gates,
-                        const float* gates_b, const float* lam, void* ring, float* state, const int* cu_q, const int* seq_lens,
-                        const int* slots, void* u, float* ab, void* out, int T, int B, int singles, int W, int n, int taps,
-                        float power, int f32, int tc, int* status, cudaStream_t stream) {
+// u [T, W]: the convolution of the recurrent branch of proj, alone.
+extern "C" int vb_rglru_conv(const void* proj, long long stride, const void* conv_w, const void* conv_b, void* ring, const int* cu_q,
+                             const int* seq_lens, const int* slots, void* u, int T, int B, int W, int taps, int f32,
+                             cudaStream_t stream) {
   if (T <= 0 || B <= 0) return 0;
-  if (W <= 0 || n <= 0 || W % n || taps <= 0 || B > 65535 || (W + 127) / 128 > 65535 || singles < 0 || singles > B ||
-      (!tc && (ab == nullptr || (size_t)W * 4 > 48 * 1024)) || (tc && (f32 || !vb_rglru_tc_supported(W, n))))
-    return -3;
-  LruParams p{cu_q, seq_lens, slots, T, B, W, n, taps, power, stride, gates_b, lam, state};
+  if (W <= 0 || taps <= 0) return -3;
+  LruParams p{cu_q, seq_lens, slots, T, B, W, W, taps, 0.f, stride, nullptr, nullptr, nullptr};
   const bool vec = (W & 7) == 0 && (stride & 7) == 0;
   cudaError_t e;
   if (f32) e = vec ? launch_conv<float, 8>(proj, conv_w, conv_b, ring, u, p, stream) : launch_conv<float, 1>(proj, conv_w, conv_b, ring, u, p, stream);
   else e = vec ? launch_conv<bf16, 8>(proj, conv_w, conv_b, ring, u, p, stream) : launch_conv<bf16, 1>(proj, conv_w, conv_b, ring, u, p, stream);
-  if (e != cudaSuccess) return (int)e;
+  return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
+}
+
+// Behind vb_rglru_conv. proj [T, stride] (gelu branch | recurrent branch), gates [2, W / n, n, n] (null: ab holds the products of u
+// with them), gates_b [2, W], lam [W] fp32, ring [slots, taps, W], state fp32 [slots, W], ab fp32 [2, T, W] scratch (without tc),
+// out [T, W]. The leading `singles` sequences have one token each.
+extern "C" int vb_rglru(const void* proj, long long stride, const void* gates, const float* gates_b,
+                        const float* lam, void* ring, float* state, const int* cu_q, const int* seq_lens, const int* slots, void* u,
+                        float* ab, void* out, int T, int B, int singles, int W, int n, int taps, float power, int f32, int tc,
+                        int* status, cudaStream_t stream) {
+  if (T <= 0 || B <= 0) return 0;
+  if (W <= 0 || n <= 0 || W % n || taps <= 0 || B > 65535 || (W + 127) / 128 > 65535 || singles < 0 || singles > B ||
+      (!tc && ab == nullptr) || (tc && (f32 || gates == nullptr || !vb_rglru_tc_supported(W, n))))
+    return -3;
+  LruParams p{cu_q, seq_lens, slots, T, B, W, n, taps, power, stride, gates_b, lam, state};
   if (f32) return rglru_simt<float>(proj, gates, ring, u, ab, out, p, stream);
   if (!tc) return rglru_simt<bf16>(proj, gates, ring, u, ab, out, p, stream);
   CUtensorMap tmW;

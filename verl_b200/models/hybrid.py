@@ -349,7 +349,7 @@ _MIXERS = {"attention": AttentionMixer, "latent_attention": LatentMixer, "delta"
 def add_norm(pending, res, weight, eps, dtype):
     """Adds a sublayer's output (None: nothing) to the stream in place; the normed stream, or without a weight a copy."""
     if isinstance(pending, ops.RoutedSum):
-        return ops.moe_combine(pending, res, weight, eps, dtype)
+        return ops.moe_combine(pending, res, weight, eps)
     return ops.add_rmsnorm(pending, res, weight, eps, dtype)
 
 

@@ -63,7 +63,8 @@ _SIGS = {
     "vb_moe_sum": ([P, P, P, I, P, L, P, L, P, P, P, I, I, F, I, P], I),
     "vb_grouped_gemm_simt": ([P, P, P, I, I, I, P, I, P], I),
     "vb_rglru_tc_supported": ([I, I], I),
-    "vb_rglru": ([P, L, P, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, P, P], I),
+    "vb_rglru_conv": ([P, L, P, P, P, P, P, P, P, I, I, I, I, I, P], I),
+    "vb_rglru": ([P, L, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, P, P], I),
     "vb_latent_decode_supported": ([I, I, I, I], I),
     "vb_latent_decode_splits": ([I, I, I], I),
     "vb_latent_decode": ([P, P, I, P, I, P, P, I, I, I, I, I, I, F, I, P, I, P, P, P, P], I),

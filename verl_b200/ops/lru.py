@@ -6,6 +6,7 @@ import torch
 import torch.nn.functional as F
 
 from . import _lib
+from .gemm import gemm
 
 
 def rglru(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, gates: torch.Tensor, gates_b: torch.Tensor,
@@ -22,25 +23,34 @@ def rglru(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, gates:
     row p % taps). Sequences that start at position 0 ignore what their slot held. ``max_q`` == 1: one token per sequence;
     otherwise the leading ``singles`` sequences have one.
 
-    ``impl``: "tc" = gates on the tensor cores, fused with the recurrence (bf16, blocks in multiples of 8 up to 512),
-    "simt" = CUDA cores, "auto" = "tc" where it applies."""
+    ``impl``: "tc" = gates on the tensor cores, fused with the recurrence (bf16, blocks in multiples of 8 up to 320),
+    "split" = the gates' products as plain matrix products (bf16, blocks in multiples of 8), "simt" = CUDA cores, "auto" = "tc"
+    where it applies, else "split"."""
     T, B, (W, taps) = proj.shape[0], slots.numel(), conv_w.shape
     n = gates.shape[1]
     if not proj.is_cuda:
         return _rglru_ref(proj, conv_w, conv_b, gates, gates_b, lam, ring, state, cu_q, seq_lens, slots, power)
-    f32 = proj.dtype == torch.float32
-    tc = not f32 and bool(_lib.fn("vb_rglru_tc_supported")(W, n)) and proj.stride(0) % 8 == 0
-    if impl == "tc" and not tc:
-        raise ValueError(f"the recurrent unit has no tensor-core form for width={W} block={n} in {proj.dtype}")
-    tc = tc and impl != "simt"
-    out, u = (torch.empty((T, W), dtype=proj.dtype, device=proj.device) for _ in range(2))
-    ab = None if tc else torch.empty((2, T, W), dtype=torch.float32, device=proj.device)
-    if max_q == 1:
-        singles = B
-    rc = _lib.fn("vb_rglru")(proj.data_ptr(), proj.stride(0), conv_w.data_ptr(), conv_b.data_ptr(), gates.data_ptr(),
-                             gates_b.data_ptr(), lam.data_ptr(), ring.data_ptr(), state.data_ptr(), cu_q.data_ptr(),
-                             seq_lens.data_ptr(), slots.data_ptr(), u.data_ptr(), _lib.ptr(ab), out.data_ptr(), T, B, singles, W,
-                             n, taps, float(power), int(f32), int(tc), _lib.status_word(proj.device).data_ptr(), _lib.stream())
+    f32, dev = proj.dtype == torch.float32, proj.device
+    mats = not f32 and n % 8 == 0 and proj.stride(0) % 8 == 0
+    tc = mats and bool(_lib.fn("vb_rglru_tc_supported")(W, n))
+    if (impl == "tc" and not tc) or (impl == "split" and not mats):
+        raise ValueError(f"the recurrent unit has no form {impl!r} for width={W} block={n} in {proj.dtype}")
+    tc = tc and impl in ("auto", "tc")
+    split = not tc and mats and impl != "simt"
+    out, u = (torch.empty((T, W), dtype=proj.dtype, device=dev) for _ in range(2))
+    common = (cu_q.data_ptr(), seq_lens.data_ptr(), slots.data_ptr(), u.data_ptr())
+    rc = _lib.fn("vb_rglru_conv")(proj.data_ptr(), proj.stride(0), conv_w.data_ptr(), conv_b.data_ptr(), ring.data_ptr(), *common,
+                                  T, B, W, taps, int(f32), _lib.stream())
+    _lib.check(rc, "vb_rglru_conv")
+    ab = None if tc else torch.empty((2, T, W), dtype=torch.float32, device=dev)
+    if split:
+        for g in range(2 * W // n):  # decay blocks, then input blocks
+            lo = g % (W // n) * n
+            gemm(u[:, lo : lo + n], gates[g], out=ab[g * n // W, :, lo : lo + n])
+    rc = _lib.fn("vb_rglru")(proj.data_ptr(), proj.stride(0), None if split else gates.data_ptr(), gates_b.data_ptr(),
+                             lam.data_ptr(), ring.data_ptr(), state.data_ptr(), *common, _lib.ptr(ab), out.data_ptr(), T, B,
+                             B if max_q == 1 else singles, W, n, taps, float(power), int(f32), int(tc),
+                             _lib.status_word(dev).data_ptr(), _lib.stream())
     _lib.check(rc, "vb_rglru")
     return out
 

@@ -223,11 +223,10 @@ def grouped_product(xs: torch.Tensor, weight: torch.Tensor, blk_expert: torch.Te
     return y
 
 
-def moe_combine(parts: RoutedSum, residual: torch.Tensor, weight: torch.Tensor | None, eps: float,
-                dtype: torch.dtype) -> torch.Tensor:
+def moe_combine(parts: RoutedSum, residual: torch.Tensor, weight: torch.Tensor | None, eps: float) -> torch.Tensor:
     """Adds the mixture's sum to the fp32 ``residual`` [T, H] IN PLACE; returns rmsnorm(residual) * weight, or without a weight
-    the residual, in ``dtype``."""
-    r = parts.routing
+    the residual, in the parts' dtype."""
+    r, dtype = parts.routing, parts.out.dtype
     T, H = residual.shape
     top = r.idx.shape[1]
     if residual.is_cuda:

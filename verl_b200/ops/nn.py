@@ -307,6 +307,8 @@ def add_rmsnorm(delta: torch.Tensor | None, residual: torch.Tensor, weight: torc
         if delta is not None:
             residual += delta.float()
         return residual.to(dtype, copy=True) if weight is None else _rmsnorm_ref(residual, weight, eps).to(dtype)
+    if delta is not None and delta.dtype != dtype:
+        raise TypeError(f"a sublayer's output in {delta.dtype} beside a norm in {dtype}")
     T, H = residual.shape
     y = torch.empty((T, H), dtype=dtype, device=residual.device)
     rc = _lib.fn("vb_add_rmsnorm")(_lib.ptr(delta), 0 if delta is None else delta.stride(0), residual.data_ptr(),

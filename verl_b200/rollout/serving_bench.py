@@ -391,7 +391,7 @@ def _bench_moe(add, r, m, H: int, T: int, tag: str) -> None:
         2 * (pairs * (H + ff) + used * ff * H), 2.0 * pairs * H * ff)
     out = moe_ops.grouped_product(h, downs[0], rt.blk_expert)
     parts = ops.RoutedSum(out, rt, False, r(T, H), logits[:, E])
-    add(f"moe_combine (+ shared, residual, copy), {tag}", time_us(lambda: ops.moe_combine(parts, res, None, 1e-5, x.dtype)),
+    add(f"moe_combine (+ shared, residual, copy), {tag}", time_us(lambda: ops.moe_combine(parts, res, None, 1e-5)),
         2 * H * (pairs + T) + 10 * T * H)
     tw = rt.weight.to(x.dtype).unsqueeze(-1)
     add("  vs sum and residual of the homogeneous models", time_us(lambda: ops.rmsnorm(
