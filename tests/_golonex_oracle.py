@@ -28,7 +28,7 @@ def softplus(z):
 
 
 def causal_conv(x, kernel, bias):
-    """x [T, C], kernel [C, taps]: tap j of the last column's taps - 1 - j predecessors; zeros before the start."""
+    """x [T, C], kernel [C, taps]: column j meets the input taps - 1 - j tokens back, if there is one."""
     T, taps = x.shape[0], kernel.shape[1]
     y = torch.zeros_like(x) + bias
     for j in range(taps):
@@ -149,7 +149,7 @@ MIXERS = {"attention": attention_mixer, "latent_attention": latent_mixer, "rglru
 
 
 def forward(cfg, weights, tokens, dtype=torch.float32, keep_layers=False):
-    """Logits [T, vocab] of one sequence (and the residual stream after every layer)."""
+    """Logits [T, vocab] of one sequence (and the stream behind each layer)."""
     def w(name):
         return weights[name].to(dtype)
 

@@ -259,7 +259,7 @@ def test_latent_window_edges(form):
     H, N, rot, V, rank = 2, 16, 16, 16, 64
     uk, uv = torch.zeros(H, N, rank, dtype=BF).cuda(), torch.zeros(H, V, rank, dtype=BF).cuda()
     uv[:, :, 5] = 1.0
-    for window, i in ((64, 63), (64, 64), (64, 700), (65, 128), (96, 95), (96, 96), (96, 300), (300, 640), (1, 130)):
+    for window, i in ((64, 63), (64, 64), (64, 700), (65, 128), (112, 111), (112, 112), (112, 300), (300, 640), (1, 130)):
         n, edge = i + 1, i - window + 1
         for j in {0, 1, edge - 1, edge, edge + 1, i - 1, i, i // 64 * 64, i // 64 * 64 - 1}:
             if not 0 <= j <= i:

@@ -174,7 +174,7 @@ def test_engine_portions_match_the_oracle(name, tmp_path):
     eng = M.engine(M.load_model(cfg, w, tmp_path, torch.float32, "cpu"))
     ids = tokens(75, cfg["vocab"])
     want = O.forward(cfg, w, ids)
-    for sizes in ([75], [1], [2], [40, 2, 33, 1]):  # the same engine: pages and slots are used again
+    for sizes in ([75], [1], [2], [40, 2, 33, 1]):  # the same engine: pages and slots a second time
         assert M.error(M.feed_portions(eng, "a", ids, sizes), want) < 1e-4, sizes
     assert eng.sched.stats()["free_pages"] == eng.num_blocks
 

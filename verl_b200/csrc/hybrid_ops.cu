@@ -55,8 +55,8 @@ __global__ void embed_normed_kernel(const long long* __restrict__ ids, const T* 
 }
 
 // ---------------------------------------------------------------------------------------------------------------
-// res += delta (when given); y = res / sqrt(mean(res^2) + eps) * w, or without w the residual. The residual stays fp32 in global memory; the row is
-// kept in shared memory between the two passes.
+// res += delta (when given); y = res / sqrt(mean(res^2) + eps) * w, or without w the residual. The residual stays fp32 in global
+// memory; the row is kept in shared memory between the two passes.
 template <typename T>
 __global__ void add_rmsnorm_kernel(const T* __restrict__ delta, long long delta_stride, float* __restrict__ res,
                                    const T* __restrict__ w, T* __restrict__ y, int H, float eps) {
@@ -596,8 +596,8 @@ __global__ void rotate_tails_kernel(T* __restrict__ q, long long stride, const f
 // rows[ctx_cu[b] + i] = page row of token i of sequence b, counted from the first of its last ctx_cu[b + 1] - ctx_cu[b] tokens
 // (of seq_lens[b]; null: from its first token), in 16-byte units. One warp per row.
 __global__ void latent_gather_kernel(const uint4* __restrict__ pages, const int* __restrict__ block_table, int max_blocks,
-                                     const int* __restrict__ ctx_cu, const int* __restrict__ seq_lens, uint4* __restrict__ rows, int total, int B, int units,
-                                     int block_size) {
+                                     const int* __restrict__ ctx_cu, const int* __restrict__ seq_lens, uint4* __restrict__ rows,
+                                     int total, int B, int units, int block_size) {
   pdl_trigger();
   pdl_wait();
   const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -1040,7 +1040,8 @@ extern "C" int vb_rotate_tails(void* q, long long stride, const float* freqs, fl
                    (reinterpret_cast<uintptr_t>(q) & 15) == 0;
   const dim3 g(T), b(128);
 #define VB_RT(TT, V) \
-  VB_DONE(vb_launch_pdl(rotate_tails_kernel<TT, V>, g, b, 0, stream, 1, (TT*)q, stride, freqs, amp, interleaved, positions, H, dim, rot))
+  VB_DONE(vb_launch_pdl(rotate_tails_kernel<TT, V>, g, b, 0, stream, 1, (TT*)q, stride, freqs, amp, interleaved, positions, H, \
+                        dim, rot))
   if (f32) {
     if (vec) VB_RT(float, true);
     VB_RT(float, false);
@@ -1052,7 +1053,8 @@ extern "C" int vb_rotate_tails(void* q, long long stride, const float* freqs, fl
 
 // row_bytes: bytes of a page row, a multiple of 16.
 extern "C" int vb_latent_gather(const void* pages, const int* block_table, int max_blocks, const int* ctx_cu,
-                                const int* seq_lens, void* rows, int total, int B, int row_bytes, int block_size, cudaStream_t stream) {
+                                const int* seq_lens, void* rows, int total, int B, int row_bytes, int block_size,
+                                cudaStream_t stream) {
   if (total <= 0 || B <= 0) return 0;
   if (row_bytes & 15) return -3;
   VB_DONE(vb_launch_pdl(latent_gather_kernel, dim3((total + 7) / 8), dim3(256), 0, stream, 1, (const uint4*)pages, block_table,

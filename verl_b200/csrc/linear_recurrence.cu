@@ -2,14 +2,14 @@
 //
 //   u = causal convolution of the recurrent branch (+ bias)              lru_conv
 //   r, i = sigmoid(block-wise projections of u + bias)
-//   a = exp(-power r softplus(lam)),  v = sqrt(1 - a^2) i u
+//   a = exp(-power softplus(lam) r),  v = i u sqrt(1 - a a)
 //   S = a S + v  token by token,  out = S gelu(gelu branch)
 //
 // lru_tc does all behind the convolution in one kernel (bf16). A CTA owns 128 channels of a block and walks a sequence, 64 tokens
 // at a time: Z^T[channels x tokens] = G[128 channels x n] . u^T on tcgen05 for both gates (weights stay in shared memory, tiles of
 // u and of the gelu branch arrive by TMA), then thread = channel: the terms of 16 tokens in registers, one dependent multiply-add
-// per token, the carry handed through shared memory to the four warps that hold the next 16 tokens. Neither gates nor decays reach memory. Steps of
-// single tokens use the same kernel with sequences in place of tokens and the state in memory in place of the carry.
+// per token, the carry handed through shared memory to the four warps that hold the next 16 tokens. Neither gates nor decays
+// reach memory. Steps of single tokens use the same kernel with sequences in place of tokens and the state in memory in place of the carry.
 // lru_gates and lru_scan are the same on CUDA cores (fp32, and sizes the other does not take).
 // Every wait is bounded; on expiry the status word is set and the CTA leaves through its teardown.
 //
@@ -520,8 +520,9 @@ static cudaError_t launch_conv(const void* proj, const void* w, const void* bias
   const int threads = p.W / V >= 256 ? 128 : 64;
   const int run = p.T >= 8 * p.B ? LC_TOKENS : 1;  // mostly single tokens: nothing to keep from one to the next
   const dim3 g((p.T + run - 1) / run, (p.W / V + threads - 1) / threads);
-#define VB_LC(N) vb_launch_pdl(lru_conv_kernel<T, V, N>, g, dim3(threads), 0, stream, 1, (const T*)proj, (const T*)w, (const T*)bias, \
-                               (T*)ring, (T*)u, run, p)
+#define VB_LC(N)                                                                                                              \
+  vb_launch_pdl(lru_conv_kernel<T, V, N>, g, dim3(threads), 0, stream, 1, (const T*)proj, (const T*)w, (const T*)bias, (T*)ring, \
+                (T*)u, run, p)
   vb_count_launch();
   switch (p.taps) {
     case 1: return VB_LC(1);
@@ -575,16 +576,18 @@ static int launch_tc(const CUtensorMap& tmW, const void* u, LruTcParams p, int r
 }
 
 // u [T, W]: the convolution of the recurrent branch of proj, alone.
-extern "C" int vb_rglru_conv(const void* proj, long long stride, const void* conv_w, const void* conv_b, void* ring, const int* cu_q,
-                             const int* seq_lens, const int* slots, void* u, int T, int B, int W, int taps, int f32,
+extern "C" int vb_rglru_conv(const void* proj, long long stride, const void* conv_w, const void* conv_b, void* ring,
+                             const int* cu_q, const int* seq_lens, const int* slots, void* u, int T, int B, int W, int taps, int f32,
                              cudaStream_t stream) {
   if (T <= 0 || B <= 0) return 0;
   if (W <= 0 || taps <= 0) return -3;
   LruParams p{cu_q, seq_lens, slots, T, B, W, W, taps, 0.f, stride, nullptr, nullptr, nullptr};
   const bool vec = (W & 7) == 0 && (stride & 7) == 0;
-  cudaError_t e;
-  if (f32) e = vec ? launch_conv<float, 8>(proj, conv_w, conv_b, ring, u, p, stream) : launch_conv<float, 1>(proj, conv_w, conv_b, ring, u, p, stream);
-  else e = vec ? launch_conv<bf16, 8>(proj, conv_w, conv_b, ring, u, p, stream) : launch_conv<bf16, 1>(proj, conv_w, conv_b, ring, u, p, stream);
+#define VB_CONV(TT)                                                      \
+  (vec ? launch_conv<TT, 8>(proj, conv_w, conv_b, ring, u, p, stream)    \
+       : launch_conv<TT, 1>(proj, conv_w, conv_b, ring, u, p, stream))
+  const cudaError_t e = f32 ? VB_CONV(float) : VB_CONV(bf16);
+#undef VB_CONV
   return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
 }
 
@@ -603,8 +606,8 @@ extern "C" int vb_rglru(const void* proj, long long stride, const void* gates, c
   if (f32) return rglru_simt<float>(proj, gates, ring, u, ab, out, p, stream);
   if (!tc) return rglru_simt<bf16>(proj, gates, ring, u, ab, out, p, stream);
   CUtensorMap tmW;
-  int rc = vb_make_tmap_3d(&tmW, gates, 2, (uint64_t)n, (uint64_t)n, (uint64_t)(2 * (W / n)), (uint64_t)n * 2, (uint64_t)n * n * 2, 64,
-                           128, 1);
+  const uint64_t n64 = n;
+  int rc = vb_make_tmap_3d(&tmW, gates, 2, n64, n64, (uint64_t)(2 * (W / n)), n64 * 2, n64 * n64 * 2, 64, 128, 1);
   if (rc) return rc;
   LruTcParams q{};
   q.l = p;

@@ -277,7 +277,7 @@ def _layer_list_to_native(cfg: ModelConfig, sd: dict[str, torch.Tensor]) -> dict
             out[f"layers.{i}.{n}"] = torch.stack([torch.cat([sd[f"l{i}.mlp.e{e}.{c}"] for c in parts], 0)
                                                   for e in range(spec.mlp.experts)])
         for n, c in _LIST_PLAIN.items():
-            if f"l{i}.{c}" in sd:
+            if f"l{i}.{c}" in sd and (spec.mlp is not None or n != "norm2.weight"):
                 out[f"layers.{i}.{n}"] = sd[f"l{i}.{c}"]
     return out
 

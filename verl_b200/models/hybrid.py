@@ -371,7 +371,8 @@ class HybridLM(nn.Module):
         super().__init__()
         self.cfg = cfg
         self.embed_tokens = nn.Embedding(cfg.vocab_size, cfg.hidden_size, dtype=dtype, device=device)
-        if cfg.design.norm == "post" and (cfg.side_dim or any(isinstance(s.mlp, MoeSpec) for s in cfg.layer_specs)):
+        routed = any(isinstance(s.mlp, MoeSpec) for s in cfg.layer_specs)
+        if cfg.design.norm == "post" and (cfg.side_dim or routed):
             raise NotImplementedError("mixtures of experts and side inputs go with norms in front of the sublayers")
         if cfg.design.embedding == "norm":
             self.embed_norm = RMSNormWeight(cfg.hidden_size, dtype, device)

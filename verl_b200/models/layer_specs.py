@@ -78,7 +78,7 @@ class AttentionSpec:
     bias per head, added to the scaled score (``bias_rows`` 0 = none); see :func:`distance_buckets`. ``softcap`` > 0: scaled
     scores become ``softcap * tanh(score / softcap)``. ``sink``: a learned number per head whose exponential joins the
     softmax denominator. ``gate``: the heads are multiplied with the sigmoid of a projection of the mixer's input, element by
-    element ("element"). ``key_values``: the values are the keys as projected, before the rotation (no value projection)."""
+    element ("element"). ``key_values``: no value projection, the unrotated key serves as the value too."""
 
     heads: int
     kv_heads: int
@@ -205,9 +205,9 @@ class DeltaSpec:
 
 @dataclass(frozen=True)
 class LruSpec:
-    """Recurrent block with a real-gated linear recurrent unit (Griffin): a gelu branch times a branch that runs through a short
-    convolution of ``conv`` taps (without activation) and the recurrence ``S = a S + sqrt(1 - a^2) i u`` per channel, with
-    ``log a = -power * r * softplus(lam)``; the gates r and i are projections of u in ``blocks`` equal parts."""
+    """Griffin's RG-LRU block. One branch is a gelu; the other is a short convolution of ``conv`` taps, giving u, and a diagonal
+    recurrence per channel: S decays by a = exp(-power * softplus(lam) * r) and takes in i * u, scaled by sqrt(1 - a * a). Decay
+    gate r and input gate i are sigmoids of u times block-diagonal matrices of ``blocks`` blocks. The branches are multiplied."""
 
     width: int
     blocks: int

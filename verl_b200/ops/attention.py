@@ -250,7 +250,7 @@ def head_norm_rope_kv_write(qkv: torch.Tensor, q_weight: torch.Tensor | None, k_
     """``qkv`` [T, q | k | v | ...]: RMS norm of every q and k head (weights [D] shared by the heads; None = no norm), rotary
     positions with the angles ``positions * freqs`` (fp32; None = none) on the first ``2 * len(freqs)`` dimensions, k and v
     to their places in the paged caches [NB, Hk, BS, D] / [NB, Hk, BS, Dv] (slot < 0: no write). ``key_values``: there is no v,
-    the values are the keys before norm and rotation. Returns q [T, heads, D], a view of ``qkv`` (changed in place on CUDA)."""
+    the keys' projection goes to the value cache as it is. Returns q [T, heads, D], a view of ``qkv`` (changed in place on CUDA)."""
     _, Hk, BS, D = k_cache.shape
     Dv = v_cache.shape[3]
     T, nq, nk = qkv.shape[0], heads * D, Hk * D

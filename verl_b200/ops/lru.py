@@ -18,8 +18,8 @@ def rglru(proj: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, gates:
     tokens of each sequence up to and including these; ``slots`` [B] int32 = state slot (< 0: padding row). u = causal
     convolution (``conv_w`` [W, taps], ``conv_b`` [W]) of the recurrent branch; r and i = sigmoid of the block-wise projections
     ``gates`` [2 * blocks, n, n] (decay, then input; [out, in]) with the biases ``gates_b`` [2 * blocks, n];
-    log a = -``power`` * r * softplus(``lam``); S = a * S + sqrt(1 - a^2) * i * u; output S * gelu(gelu branch). Gates, decay and
-    state are fp32. Updates in place ``state`` fp32 [slots, W] and ``ring`` [slots, taps, W] (convolution inputs, position p in
+    a = exp(-``power`` * softplus(``lam``) * r); S becomes a * S + v with v = i * u * sqrt(1 - a * a); output S * gelu(gelu branch).
+    Gates, decay and state are fp32. Updates in place ``state`` fp32 [slots, W] and ``ring`` [slots, taps, W] (convolution inputs, position p in
     row p % taps). Sequences that start at position 0 ignore what their slot held. ``max_q`` == 1: one token per sequence;
     otherwise the leading ``singles`` sequences have one.
 
