@@ -40,7 +40,8 @@ NVCC_FLAGS = [
 ]
 # Sources compiled without --use_fast_math: their exponentials, logarithms, divisions and roots feed recurrent state or
 # serve the 32-bit mode.
-PRECISE_SOURCES = {"hybrid_ops.cu", "delta_rule.cu", "moe_ops.cu", "linear_recurrence.cu"}
+PRECISE_SOURCES = {"hybrid_ops.cu", "delta_rule.cu", "moe_ops.cu", "linear_recurrence.cu",
+                   "gated_linear_attention.cu"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-pthread"]
 
 

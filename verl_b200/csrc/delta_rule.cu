@@ -32,48 +32,11 @@
 // both operands and sums are fp32.
 #include "common.cuh"
 #include "host_utils.h"
+#include "state_ops.cuh"
 
 namespace vb {
 
-template <typename T>
-__device__ __forceinline__ float dl_f(T v) { return static_cast<float>(v); }
-template <typename T>
-__device__ __forceinline__ T dl_t(float v) { return static_cast<T>(v); }
-
-__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
-// For results that are rounded to bf16: the fast exponential and quotient err far below one bf16 ulp.
-template <typename T>
-__device__ __forceinline__ float silu_t(float x) {
-  return sizeof(T) == 2 ? __fdividef(x, 1.f + __expf(-x)) : silu_f(x);
-}
-__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
-__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 constexpr float UNIT_EPS = 1e-6f;
-
-// N consecutive elements, N * sizeof(T) aligned (N a power of two, at most 16 bytes at once).
-template <typename T, int N>
-__device__ __forceinline__ void load_n(const T* p, float (&f)[N]) {
-  constexpr int W = sizeof(T) * N > 16 ? 16 / sizeof(T) : N;
-  struct alignas(sizeof(T) * W) Vec { T v[W]; };
-#pragma unroll
-  for (int i = 0; i < N / W; ++i) {
-    const Vec x = reinterpret_cast<const Vec*>(p)[i];
-#pragma unroll
-    for (int j = 0; j < W; ++j) f[i * W + j] = dl_f<T>(x.v[j]);
-  }
-}
-template <typename T, int N>
-__device__ __forceinline__ void store_n(T* p, const float (&f)[N]) {
-  constexpr int W = sizeof(T) * N > 16 ? 16 / sizeof(T) : N;
-  struct alignas(sizeof(T) * W) Vec { T v[W]; };
-#pragma unroll
-  for (int i = 0; i < N / W; ++i) {
-    Vec x;
-#pragma unroll
-    for (int j = 0; j < W; ++j) x.v[j] = dl_t<T>(f[i * W + j]);
-    reinterpret_cast<Vec*>(p)[i] = x;
-  }
-}
 
 struct DeltaParams {
   const void* proj;        // [T, stride]
@@ -95,17 +58,6 @@ struct DeltaParams {
   int B, H, Hk, D, V, taps;
   float eps;
 };
-
-__device__ __forceinline__ void cp_async4(float* dst, const float* src, bool on) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(on ? 4 : 0) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-
-__device__ __forceinline__ void cp_async16(void* dst, const void* src, bool on) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(on ? 16 : 0) : "memory");
-}
 
 // ---------------------------------------------------------------------------------------------------------------
 // One warp per (sequence, tile of tokens, head row); lanes across the head's channels, a sliding window of inputs in
@@ -290,13 +242,6 @@ __global__ void __launch_bounds__(128) delta_prep_tile_kernel(const DeltaParams 
   }
 }
 
-__device__ __forceinline__ float sum8(float v) {  // over groups of eight lanes
-  v += __shfl_xor_sync(0xffffffffu, v, 1);
-  v += __shfl_xor_sync(0xffffffffu, v, 2);
-  v += __shfl_xor_sync(0xffffffffu, v, 4);
-  return v;
-}
-
 // The last convolution inputs of a sequence: its channels are dealt out over the `parts` CTAs that work on it.
 template <typename T>
 __device__ __forceinline__ void store_ring(const DeltaParams& p, int first, int n, int start, int slot, int part, int parts) {
@@ -451,11 +396,6 @@ __device__ __forceinline__ void mma16(float (&c)[4], const uint32_t (&a)[4], uin
       "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-// x = hi + lo, both bf16, for two neighbours packed into 32 bits
-__device__ __forceinline__ void split2(float x0, float x1, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf16x2(x0, x1);
-  lo = pack_bf16x2(x0 - __uint_as_float(hi << 16), x1 - __uint_as_float(hi & 0xffff0000u));
 }
 // Fragment addresses. A [16 x 16] at (row, col) of a row-major tile:
 template <int PITCH>
@@ -991,54 +931,6 @@ delta_chunk_scan_kernel(const DeltaParams p, const uint8_t* __restrict__ scratch
 }
 
 // ---------------------------------------------------------------------------------------------------------------
-// out = rmsnorm(out) * w * silu(gate) per (token, head), in place. A warp takes GN_T tokens of one head.
-constexpr int GN_T = 4;
-template <typename T>
-__global__ void __launch_bounds__(128) gated_norm_kernel(const DeltaParams p, int tokens) {
-  pdl_trigger();
-  pdl_wait();
-  const int lane = threadIdx.x & 31, h = blockIdx.y * 4 + (threadIdx.x >> 5);
-  if (h >= p.H) return;
-  const int t0 = blockIdx.x * GN_T, cnt = min(GN_T, tokens - t0);
-  T* o = static_cast<T*>(p.out) + (long long)t0 * p.out_stride + (long long)h * p.V;
-  const T* gate = static_cast<const T*>(p.proj) + (long long)t0 * p.stride + 2 * p.Hk * p.D + p.H * p.V + (long long)h * p.V;
-  const T* w = static_cast<const T*>(p.norm_w);
-  const float inv_v = 1.f / (float)p.V;
-  const int c = lane * 4;
-  if (p.V <= 128 && ((p.V | (int)p.stride | (int)p.out_stride | (2 * p.Hk * p.D)) & 3) == 0) {
-    const bool on = c < p.V;
-    float x[GN_T][4] = {}, g[GN_T][4], wv[4];
-    if (on) load_n<T, 4>(w + c, wv);
-#pragma unroll
-    for (int k = 0; k < GN_T; ++k)
-      if (on && k < cnt) {
-        load_n<T, 4>(o + k * p.out_stride + c, x[k]);
-        load_n<T, 4>(gate + k * p.stride + c, g[k]);
-      }
-#pragma unroll
-    for (int k = 0; k < GN_T; ++k) {
-      const float ss = x[k][0] * x[k][0] + x[k][1] * x[k][1] + x[k][2] * x[k][2] + x[k][3] * x[k][3];
-      const float inv = rsqrtf(warp_reduce_sum(ss) * inv_v + p.eps);
-      if (on && k < cnt) {
-#pragma unroll
-        for (int e = 0; e < 4; ++e) x[k][e] = x[k][e] * inv * wv[e] * silu_t<T>(g[k][e]);
-        store_n<T, 4>(o + k * p.out_stride + c, x[k]);
-      }
-    }
-    return;
-  }
-  for (int k = 0; k < cnt; ++k, o += p.out_stride, gate += p.stride) {
-    float ss = 0.f;
-    for (int i = lane; i < p.V; i += 32) {
-      const float x = dl_f<T>(o[i]);
-      ss += x * x;
-    }
-    const float inv = rsqrtf(warp_reduce_sum(ss) * inv_v + p.eps);
-    for (int i = lane; i < p.V; i += 32) o[i] = dl_t<T>(dl_f<T>(o[i]) * inv * dl_f<T>(w[i]) * silu_t<T>(dl_f<T>(gate[i])));
-  }
-}
-
-// ---------------------------------------------------------------------------------------------------------------
 // Decode: one token per sequence, one CTA per (head, sequence), everything fused. The state columns are loaded before
 // the convolution so that the memory traffic is in flight while the small work runs.
 constexpr int DD_THREADS = 256, DD_NP = 4;
@@ -1275,10 +1167,8 @@ static int run_delta(const DeltaParams& p, int tokens, int max_q, uint8_t* chunk
          : nr == 16 ? run_scan<T, 16>(p, stream)
                     : run_scan<T, 32>(p, stream);
   if (rc) return rc;
-  cudaError_t e = vb_launch_pdl(gated_norm_kernel<T>, dim3((tokens + GN_T - 1) / GN_T, (p.H + 3) / 4), dim3(128), 0,
-                                stream, 1, p, tokens);
-  vb_count_launch();
-  return (int)e;
+  const T* gate = static_cast<const T*>(p.proj) + 2 * p.Hk * p.D + p.H * p.V;
+  return launch_gated_norm<T>(static_cast<T*>(p.out), p.out_stride, gate, p.stride, p.norm_w, p.H, p.V, p.eps, tokens, stream);
 }
 
 }  // namespace vb

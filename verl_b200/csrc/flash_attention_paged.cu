@@ -1,6 +1,6 @@
 // Prefill attention of layer-list decoders on tcgen05: ragged queries over the paged KV cache, with a sliding window and
 // kept first keys or chunks of the sequence, a per-distance bias or a soft cap of the scores, a sink in the denominator and
-// an output gate. Head sizes up to 128 (multiples of 8), bf16.
+// an output gate; with softmax weights or sigmoid ones. Head sizes up to 128 (multiples of 8), bf16.
 //
 // One CTA per (sequence, query head, block of 128 queries), two CTAs per SM: one's softmax overlaps the other's tensor
 // work. The CTA walks the 128-key blocks that some row of the block may see: those of the kept first keys, then those of
@@ -13,6 +13,9 @@
 // maximum has grown by more than 2^8 (the result does not depend on it), so O is rarely rescaled.
 // K / V pages arrive by per-CTA TMA loads; columns past a head's size are filled with zeros by TMA, keys past the sequence
 // or outside the mask get weight zero. Masks and the bias table are looked at only by the 32 x 32 blocks they reach.
+// The SIG variant weighs a key with the sigmoid of its score, less r1 ln(1 + r2 distance), plus a number of the head, without
+// reference, rescaling and denominator. The distance's part of the exponent comes from a table of the 255 distances between 128
+// queries and 128 keys, written anew for every block of keys.
 // The LATENT variant serves latent attention: keys and values of all heads lie expanded in rows of scratch memory, sequence
 // after sequence, and a key is two parts: the head's own and the rotated one that all heads share. Its three 64-column parts
 // of Q and K leave room for two CTAs per SM with 64 keys a block. Its contexts may start where the first query's window does:
@@ -53,6 +56,7 @@ struct PagedFlashParams {
   long long gate_stride;
   int gate_w;
   int* status;
+  const float *shift, *r1, *r2;  // [Hq]; SIG: shift, and r1, r2 or null
   // LATENT only: D = the heads' own part of a key; contexts of the sequences in the expanded rows
   int rot;
   const int* ctx_cu;       // [B + 1]
@@ -61,7 +65,20 @@ struct PagedFlashParams {
 // exp2 of the scaled scores: scale and bias are multiplied by log2(e) up front
 constexpr float LOG2E = 1.4426950408889634f;
 
-template <bool LATENT>
+constexpr int PF_TAB = 256;  // distances of a block of keys (SIG), double-buffered in place of the bias table
+
+// Barrier over the 128 threads of the first four warps that also and-reduces a predicate: they leave their loop together.
+__device__ __forceinline__ bool pf_bar_and(bool pred) {
+  uint32_t r;
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\tsetp.ne.u32 q, %1, 0;\n\tbarrier.red.and.pred p, 1, 128, q;\n\tselp.u32 %0, 1, 0, p;\n\t}"
+      : "=r"(r)
+      : "r"((uint32_t)pred)
+      : "memory");
+  return r != 0;
+}
+
+template <bool LATENT, bool SIG = false>
 __global__ void __launch_bounds__(PF_THREADS, 2)
 paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                    const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmQr,
@@ -231,6 +248,69 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
               first_hi = windowed ? first_key(qw + 31) : 0;
     bool ok = true;
 
+    if constexpr (SIG) {
+      static_assert(!LATENT, "sigmoid weights over the paged cache only");
+      l_run = 1.f;
+      const float shift2 = p.shift[hq] * LOG2E, r1 = p.r1 ? p.r1[hq] : 0.f, r2 = p.r1 ? p.r2[hq] : 0.f;
+      for (int c = 0; c < n_chunks; ++c) {
+        const int c0 = chunk_at(c) * PF_N;
+        // what the exponent of e^-(score + shift) takes from the distance d, at entry d - (distance of row 0 to the last key)
+        float* tab = bias_s + (c & 1) * PF_TAB;
+        for (int i = r; i < PF_TAB; i += 128)
+          tab[i] = fmaf(r1, __log2f(fmaf(r2, (float)max(pos0 - c0 - (PF_N - 1) + i, 0), 1.f)), -shift2);
+        ok = pf_bar_and(ok);  // the table is complete; a failed wait of the last round ends the loop for all
+        if (!ok) break;
+        if (*abort_flag || !mbar_wait(s_full, c & 1)) {
+          report_error(p.status, ERR_WAIT_TMEM_FULL, c);
+          *abort_flag = 1;
+          ok = false;
+        }
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) continue;  // to the barrier
+        tc_fence_after();
+        const float* row = tab + r + PF_N - 1;  // entry of key c0 + e: row[-e]
+#pragma unroll 1
+        for (int j = 0; j < GROUPS; ++j) {
+          const int k0 = c0 + 32 * j, dmin = qw - (k0 + 31), dmax = qw + 31 - k0;
+          uint32_t v[32];
+          if (dmax < 0 || (windowed && k0 + 31 < first_lo && k0 >= keep)) {
+#pragma unroll
+            for (int e = 0; e < 32; ++e) v[e] = 0;
+          } else {
+            tmem_ld_32x32(s_addr + j * 32, v);
+            tmem_ld_wait();
+            uint32_t seen = 0xffffffffu;  // bit e
+            if (dmin < 0 || (windowed && k0 < first_hi && k0 + 31 >= keep)) {
+              seen = 0;
+#pragma unroll
+              for (int e = 0; e < 32; ++e)
+                seen |= (uint32_t)(qpos >= k0 + e && (!windowed || k0 + e >= first || k0 + e < keep)) << e;
+            }
+            uint32_t w[32];
+#pragma unroll
+            for (int e = 0; e < 32; e += 2) {
+              // 1 / a and 1 / b from one reciprocal; weights below 2^-60 do not matter
+              float x0 = fminf(fmaf(__uint_as_float(v[e]), -scale2, row[-32 * j - e]), 60.f);
+              float x1 = fminf(fmaf(__uint_as_float(v[e + 1]), -scale2, row[-32 * j - e - 1]), 60.f);
+              x0 = seen >> e & 1 ? x0 : 60.f;
+              x1 = seen >> (e + 1) & 1 ? x1 : 60.f;
+              const float a = 1.f + exp2f(x0), b = 1.f + exp2f(x1), rc = __fdividef(1.f, a * b);
+              const float p0 = seen >> e & 1 ? b * rc : 0.f, p1 = seen >> (e + 1) & 1 ? a * rc : 0.f;
+              const uint32_t h = pack_bf16x2(p0, p1);
+              w[e >> 1] = h;
+              w[16 + (e >> 1)] = pack_bf16x2(p0 - __uint_as_float(h << 16), p1 - __uint_as_float(h & 0xffff0000u));
+            }
+#pragma unroll
+            for (int e = 0; e < 32; ++e) v[e] = w[e];
+          }
+          tmem_st_32x32(s_addr + j * 32, v);
+        }
+        tmem_st_wait();
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(p_ready);
+      }
+    } else
     for (int c = 0; c < n_chunks; ++c) {
       if (*abort_flag || !mbar_wait(s_full, c & 1)) {
         report_error(p.status, ERR_WAIT_TMEM_FULL, c);
@@ -412,17 +492,19 @@ extern "C" int vb_paged_flash_supported(int Hq, int Hk, int D, int Dv, int block
 
 // q [T, Hq, D] bf16 (token stride q_stride elements, a multiple of 8); caches [num_blocks, Hk, block_size, D | Dv]; the
 // queries of sequence b are the last cu_q[b + 1] - cu_q[b] of its seq_lens[b] positions; out [T, Hq * Dv]. Window (with kept
-// first keys) or chunk; bias or softcap; sink [Hq] fp32 and gate [T, Hq * Dv] bf16 or null.
+// first keys) or chunk; bias or softcap; sink [Hq] fp32 and gate [T, Hq * Dv] (gate_w 1: [T, Hq]) bf16 or null; shift [Hq] fp32
+// (without bias, softcap and sink) with r1, r2 [Hq] or null: sigmoid weights.
 extern "C" int vb_paged_flash(const void* q, long long q_stride, const void* kc, const void* vc, int num_blocks,
                               const int* block_table, int max_blocks, const int* cu_q, const int* seq_lens, int T, int B,
                               int max_q, int Hq, int Hk, int D, int Dv, int block_size, float scale, int window,
                               int keep_first, int chunk, const float* bias, int bias_len, float softcap, const float* sink,
-                              const void* gate, long long gate_stride, void* out, long long out_stride, int* status,
-                              cudaStream_t stream) {
+                              const float* shift, const float* r1, const float* r2, const void* gate, long long gate_stride,
+                              int gate_w, void* out, long long out_stride, int* status, cudaStream_t stream) {
   if (B <= 0 || T <= 0 || max_q <= 0) return 0;
   if (!vb_paged_flash_supported(Hq, Hk, D, Dv, block_size, bias_len) || (q_stride & 7) || (out_stride & 7) || B > 65535 ||
       (bias != nullptr && bias_len <= 0) || (window > 0 && chunk > 0) || (softcap > 0.f && bias != nullptr) ||
-      (gate != nullptr && ((gate_stride & 7) || (reinterpret_cast<uintptr_t>(gate) & 15))))
+      (gate != nullptr && gate_w != 1 && ((gate_stride & 7) || (reinterpret_cast<uintptr_t>(gate) & 15))) ||
+      (shift && (bias || sink || softcap > 0.f)) || (r1 && (!shift || !r2)))
     return -3;
   CUtensorMap tmQ, tmK, tmV;
   int rc = vb_make_tmap_3d(&tmQ, q, 2, (uint64_t)D, (uint64_t)Hq, (uint64_t)T, (uint64_t)D * 2, (uint64_t)q_stride * 2, 64, 1,
@@ -433,11 +515,13 @@ extern "C" int vb_paged_flash(const void* q, long long q_stride, const void* kc,
   if (rc) return rc;
   rc = vb_make_tmap_2d(&tmV, vc, 2, (uint64_t)Dv, rows, (uint64_t)Dv * 2, 64, block_size);
   if (rc) return rc;
-  const int smem = PfCfg<false>::BIAS_OFF + (bias ? bias_len * 4 : 0) + 1024;
+  const int smem = PfCfg<false>::BIAS_OFF + (shift ? 2 * PF_TAB * 4 : bias ? bias_len * 4 : 0) + 1024;
   static bool attr_set = false;
   if (!attr_set) {
     VB_CUDA_CHECK(cudaFuncSetAttribute(paged_flash_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                        PfCfg<false>::BIAS_OFF + PF_MAX_BIAS * 4 + 1024));
+    VB_CUDA_CHECK(cudaFuncSetAttribute(paged_flash_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                       PfCfg<false>::BIAS_OFF + 2 * PF_TAB * 4 + 1024));
     attr_set = true;
   }
   PagedFlashParams p{};
@@ -450,11 +534,14 @@ extern "C" int vb_paged_flash(const void* q, long long q_stride, const void* kc,
   p.scale = scale; p.softcap = softcap; p.sink = sink;
   p.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
   p.gate_stride = gate_stride;
-  p.gate_w = 0;
+  p.gate_w = gate_w;
+  p.shift = shift; p.r1 = r1; p.r2 = r2;
   p.status = status;
   const dim3 grid(p.max_qblocks, Hq, B);
-  cudaError_t e = vb_launch_pdl(paged_flash_kernel<false>, grid, dim3(PF_THREADS), (size_t)smem, stream, 1, tmQ, tmK, tmV, tmQ,
-                                tmK, p);
+  cudaError_t e = shift ? vb_launch_pdl(paged_flash_kernel<false, true>, grid, dim3(PF_THREADS), (size_t)smem, stream, 1, tmQ, tmK,
+                                        tmV, tmQ, tmK, p)
+                        : vb_launch_pdl(paged_flash_kernel<false>, grid, dim3(PF_THREADS), (size_t)smem, stream, 1, tmQ, tmK,
+                                        tmV, tmQ, tmK, p);
   vb_count_launch();
   return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
 }

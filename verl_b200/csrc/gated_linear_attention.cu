@@ -1,0 +1,718 @@
+// Gated linear attention over ragged batches with carried state (mixer of layer-list decoders).
+//
+// Per head with state S [D, V], decays a_t [D] (one per key channel), scaled q and plain k, v:
+//     S <- diag(a_t) S + k_t v_t^T;   o_t = S^T q_t
+// and the head's output is rmsnorm(o) * w * silu(gate). The decays come from a few numbers r per token that all heads share:
+//     z = W r + b,   a = sigmoid(z)^(1 / tau)
+//
+// Input row of a token (one projection GEMM): [q (H D) | k (H D) | v (H V) | gate (H V) | r (rank) | ...].
+// State of a sequence (slot s): fp32 state[s][H][V][D] (a column of S is contiguous). A sequence whose first token has position
+// 0 starts from zero state whatever its slot holds; slot < 0 marks a padding row.
+//
+// Kernels:
+//   gla_step    one token per sequence: everything fused (decode)
+//   gla_chunk   chunks of up to 64 tokens on the tensor cores (bf16 serving), gated_norm behind it
+//   gla_decay + gla_scan   token by token, state in registers, fp32 throughout (32-bit mode, sizes the chunks do not take)
+#include "common.cuh"
+#include "host_utils.h"
+#include "state_ops.cuh"
+
+namespace vb {
+
+struct GlaParams {
+  const void* proj;       // [T, stride]
+  long long stride;
+  const void* decay_w;    // [H D, rank]
+  const float* decay_b;   // [H D]
+  const void* norm_w;     // [V]
+  float* state;           // [slots, H, V, D]
+  const int* cu_q;        // [B + 1]
+  const int* seq_lens;    // [B] tokens of the sequence up to and including this step's
+  const int* slots;       // [B]
+  float* decay;           // [T, H D] fp32 (scan path)
+  void* out;              // [T, out_stride]
+  long long out_stride;
+  int H, D, V, rank, b0;  // b0: first sequence of a launch
+  float inv_tau, eps;
+};
+
+// log(sigmoid(z))
+__device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+
+// z of channel c from the token's numbers r (shared memory or global)
+template <typename T, typename R>
+__device__ __forceinline__ float decay_logit(const GlaParams& p, int c, const R* r) {
+  const T* w = static_cast<const T*>(p.decay_w) + (long long)c * p.rank;
+  float z = p.decay_b[c];
+  if ((p.rank & 7) == 0) {
+    for (int i = 0; i < p.rank; i += 8) {
+      float f[8];
+      load_n<T, 8>(w + i, f);
+#pragma unroll
+      for (int k = 0; k < 8; ++k) z = fmaf(f[k], dl_f<R>(r[i + k]), z);
+    }
+  } else {
+    for (int i = 0; i < p.rank; ++i) z = fmaf(dl_f<T>(w[i]), dl_f<R>(r[i]), z);
+  }
+  return z;
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// Decode: one CTA per (head, sequence). The state columns are loaded first, so that the memory traffic is in flight while the
+// decays are computed. Eight lanes share a column; lane r holds rows 4 (r + 8 i) + e.
+constexpr int GS_THREADS = 256, GS_NP = 4;
+template <typename T, int NR>
+__global__ void __launch_bounds__(GS_THREADS) gla_step_kernel(const GlaParams p) {
+  constexpr int DP = NR * 8;
+  extern __shared__ float sm[];
+  float* q_s = sm;            // [DP]
+  float* k_s = q_s + DP;      // [DP]
+  float* a_s = k_s + DP;      // [DP]
+  float* v_s = a_s + DP;      // [V]
+  float* o_s = v_s + p.V;     // [V]
+  float* r_s = o_s + p.V;     // [rank]
+  pdl_trigger();
+  pdl_wait();
+  const int h = blockIdx.x, b = p.b0 + blockIdx.y;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r = lane & 7, cw = warp * 4 + (lane >> 3);
+  const int slot = p.slots[b], pos = p.seq_lens[b] - 1, t = p.cu_q[b];
+  T* out = static_cast<T*>(p.out) + (long long)t * p.out_stride + (long long)h * p.V;
+  if (slot < 0) {
+    for (int c = tid; c < p.V; c += GS_THREADS) out[c] = dl_t<T>(0.f);
+    return;
+  }
+  const T* row = static_cast<const T*>(p.proj) + (long long)t * p.stride;
+  float* st = p.state + ((long long)slot * p.H + h) * p.V * p.D;
+  const bool vec = (p.D & 3) == 0;
+  auto load_cols = [&](int cbase, float (&S)[GS_NP][NR]) {
+#pragma unroll
+    for (int j = 0; j < GS_NP; ++j) {
+      const int col = cbase + j * 32 + cw;
+#pragma unroll
+      for (int i = 0; i < NR / 4; ++i) {
+        const int d = 4 * (r + 8 * i);
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (pos > 0 && col < p.V && d < p.D) {
+          const float* src = st + (long long)col * p.D + d;
+          if (vec) {
+            x = __ldcs(reinterpret_cast<const float4*>(src));
+          } else {
+            x.x = src[0];
+            if (d + 1 < p.D) x.y = src[1];
+            if (d + 2 < p.D) x.z = src[2];
+            if (d + 3 < p.D) x.w = src[3];
+          }
+        }
+        S[j][4 * i] = x.x; S[j][4 * i + 1] = x.y; S[j][4 * i + 2] = x.z; S[j][4 * i + 3] = x.w;
+      }
+    }
+  };
+  float S[GS_NP][NR];
+  load_cols(0, S);
+  const int HD = p.H * p.D, HV = p.H * p.V;
+  for (int i = tid; i < p.rank; i += GS_THREADS) r_s[i] = dl_f<T>(row[2 * (HD + HV) + i]);
+  const float qscale = 1.f / sqrtf((float)p.D);
+  for (int d = tid; d < DP; d += GS_THREADS) {
+    const bool on = d < p.D;
+    q_s[d] = on ? dl_f<T>(row[h * p.D + d]) * qscale : 0.f;
+    k_s[d] = on ? dl_f<T>(row[HD + h * p.D + d]) : 0.f;
+  }
+  for (int c = tid; c < p.V; c += GS_THREADS) v_s[c] = dl_f<T>(row[2 * HD + h * p.V + c]);
+  __syncthreads();
+  for (int d = tid; d < DP; d += GS_THREADS)
+    a_s[d] = d < p.D ? expf(log_sigmoid(decay_logit<T>(p, h * p.D + d, r_s)) * p.inv_tau) : 0.f;
+  __syncthreads();
+  float kv[NR], qv[NR], av[NR];
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int d = 4 * (r + 8 * (i >> 2)) + (i & 3);
+    kv[i] = k_s[d];
+    qv[i] = q_s[d];
+    av[i] = a_s[d];
+  }
+  for (int cbase = 0; cbase < p.V; cbase += GS_NP * 32) {
+    if (cbase > 0) load_cols(cbase, S);
+#pragma unroll
+    for (int j = 0; j < GS_NP; ++j) {
+      const int col = cbase + j * 32 + cw;
+      const float v = col < p.V ? v_s[col] : 0.f;
+      float o = 0.f;
+#pragma unroll
+      for (int i = 0; i < NR; ++i) {
+        S[j][i] = fmaf(kv[i], v, av[i] * S[j][i]);
+        o = fmaf(S[j][i], qv[i], o);
+      }
+      o = sum8(o);
+      if (col < p.V) {
+        if (r == 0) o_s[col] = o;
+#pragma unroll
+        for (int i = 0; i < NR / 4; ++i) {
+          const int d = 4 * (r + 8 * i);
+          if (d < p.D) {
+            const float4 x = make_float4(S[j][4 * i], S[j][4 * i + 1], S[j][4 * i + 2], S[j][4 * i + 3]);
+            float* dst = st + (long long)col * p.D + d;
+            if (vec) {
+              __stcs(reinterpret_cast<float4*>(dst), x);
+            } else {
+              dst[0] = x.x;
+              if (d + 1 < p.D) dst[1] = x.y;
+              if (d + 2 < p.D) dst[2] = x.z;
+              if (d + 3 < p.D) dst[3] = x.w;
+            }
+          }
+        }
+      }
+    }
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int c = lane; c < p.V; c += 32) ss += o_s[c] * o_s[c];
+  const float inv = 1.f / sqrtf(warp_reduce_sum(ss) / (float)p.V + p.eps);
+  const T* gate = row + 2 * HD + HV + (long long)h * p.V;
+  const T* w = static_cast<const T*>(p.norm_w);
+  for (int c = tid; c < p.V; c += GS_THREADS) out[c] = dl_t<T>(o_s[c] * inv * dl_f<T>(w[c]) * silu_f(dl_f<T>(gate[c])));
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// decay[t][c] = sigmoid(z)^(1 / tau). One CTA per (token, 128 channels).
+template <typename T>
+__global__ void __launch_bounds__(128) gla_decay_kernel(const GlaParams p) {
+  pdl_trigger();
+  pdl_wait();
+  const int c = blockIdx.y * 128 + threadIdx.x, HD = p.H * p.D;
+  const long long t = blockIdx.x;
+  if (c >= HD) return;
+  const T* r = static_cast<const T*>(p.proj) + t * p.stride + 2 * (HD + p.H * p.V);
+  p.decay[t * HD + c] = expf(log_sigmoid(decay_logit<T>(p, c, r)) * p.inv_tau);
+}
+
+// One CTA per (head, 32 state columns, sequence); the lanes of a column as above. Tokens come in blocks through shared memory.
+constexpr int GC_VB = 32, GC_TB = 16;
+template <typename T, int NR>
+__global__ void __launch_bounds__(GS_THREADS) gla_scan_kernel(const GlaParams p) {
+  constexpr int DP = NR * 8;
+  extern __shared__ float sm[];
+  float* q_s = sm;                       // [TB][DP]
+  float* k_s = q_s + GC_TB * DP;         // [TB][DP]
+  float* a_s = k_s + GC_TB * DP;         // [TB][DP]
+  float* v_s = a_s + GC_TB * DP;         // [TB][VB]
+  float* o_s = v_s + GC_TB * GC_VB;      // [TB][VB]
+  pdl_trigger();
+  pdl_wait();
+  const int h = blockIdx.x, v0 = blockIdx.y * GC_VB, b = p.b0 + blockIdx.z;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, r = lane & 7, col = warp * 4 + (lane >> 3);
+  const int first = p.cu_q[b], n = p.cu_q[b + 1] - first, slot = p.slots[b];
+  if (n <= 0 || slot < 0) return;
+  const int start = p.seq_lens[b] - n, HD = p.H * p.D;
+  const bool col_on = v0 + col < p.V;
+  float* st = p.state + (((long long)slot * p.H + h) * p.V + v0 + col) * p.D;
+  float S[NR];
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int d = 4 * (r + 8 * (i >> 2)) + (i & 3);
+    S[i] = (start > 0 && col_on && d < p.D) ? st[d] : 0.f;
+  }
+  const T* proj = static_cast<const T*>(p.proj) + (long long)first * p.stride;
+  const float* decay = p.decay + (long long)first * HD;
+  const float qscale = 1.f / sqrtf((float)p.D);
+  for (int t0 = 0; t0 < n; t0 += GC_TB) {
+    const int cnt = min(GC_TB, n - t0);
+    for (int i = tid; i < GC_TB * DP; i += GS_THREADS) {
+      const int t = i / DP, d = i % DP;
+      const bool on = t < cnt && d < p.D;
+      const T* row = proj + (long long)(t0 + t) * p.stride + h * p.D + d;
+      q_s[i] = on ? dl_f<T>(row[0]) * qscale : 0.f;
+      k_s[i] = on ? dl_f<T>(row[HD]) : 0.f;
+      a_s[i] = on ? decay[(long long)(t0 + t) * HD + h * p.D + d] : 0.f;
+    }
+    for (int i = tid; i < GC_TB * GC_VB; i += GS_THREADS) {
+      const int t = i / GC_VB, c = i % GC_VB;
+      v_s[i] = t < cnt && v0 + c < p.V ? dl_f<T>(proj[(long long)(t0 + t) * p.stride + 2 * HD + h * p.V + v0 + c]) : 0.f;
+    }
+    __syncthreads();
+    for (int t = 0; t < cnt; ++t) {
+      const float v = v_s[t * GC_VB + col];
+      float o = 0.f;
+#pragma unroll
+      for (int i = 0; i < NR / 4; ++i) {
+        const int at = t * DP + 4 * (r + 8 * i);
+        const float4 q4 = *reinterpret_cast<const float4*>(q_s + at), k4 = *reinterpret_cast<const float4*>(k_s + at),
+                     a4 = *reinterpret_cast<const float4*>(a_s + at);
+        S[4 * i] = fmaf(k4.x, v, a4.x * S[4 * i]);
+        S[4 * i + 1] = fmaf(k4.y, v, a4.y * S[4 * i + 1]);
+        S[4 * i + 2] = fmaf(k4.z, v, a4.z * S[4 * i + 2]);
+        S[4 * i + 3] = fmaf(k4.w, v, a4.w * S[4 * i + 3]);
+        o = fmaf(S[4 * i], q4.x, o);
+        o = fmaf(S[4 * i + 1], q4.y, o);
+        o = fmaf(S[4 * i + 2], q4.z, o);
+        o = fmaf(S[4 * i + 3], q4.w, o);
+      }
+      o = sum8(o);
+      if (r == 0) o_s[t * GC_VB + col] = o;
+    }
+    __syncthreads();
+    T* out = static_cast<T*>(p.out) + (long long)(first + t0) * p.out_stride + (long long)h * p.V + v0;
+    for (int i = tid; i < cnt * GC_VB; i += GS_THREADS) {
+      const int t = i / GC_VB, c = i % GC_VB;
+      if (v0 + c < p.V) out[(long long)t * p.out_stride + c] = dl_t<T>(o_s[i]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int d = 4 * (r + 8 * (i >> 2)) + (i & 3);
+    if (col_on && d < p.D) st[d] = S[i];
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// Chunked form on the tensor cores. With b_t the running sum of log decays inside a chunk (per channel), S0 the state in front
+// of it, Q~_t = q_t e^{b_t} and K~_s = k_s e^{-b_s}:
+//     o_t = S0^T Q~_t + sum_{s<=t} (Q~_t . K~_s) v_s,      S = e^{b_last} (S0 + sum_s K~_s v_s^T)
+// A chunk takes up to 64 tokens, fewer where a channel decays so far that e^{-b} would leave fp32's range: the walk then
+// goes on behind the tokens it has taken, whatever their number.
+//
+// One CTA of sixteen warps per (sequence, head, 128 state columns); tcgen05 with accumulators in TMEM (tokens = columns):
+//     Z^T [d, t]      = W . r^T                                  (W in TMEM; the decays' logits)
+//     P^T [s | s, t]  = [K~ hi; K~ lo] . (Q~ hi + Q~ lo)^T       (two partial sums of each score, added by the last product)
+//     S^T [v, d]     += V^T . (K~ hi + K~ lo)                    (fp32 state in TMEM, decayed when it is read)
+//     O^T [v, t]      = S0^T hi . (Q~ hi + Q~ lo)^T + S0^T lo . Q~ hi^T
+//     O^T [v, t]     += [V; V]^T . P hi + V^T . P lo             (P: causal part of the scores)
+// Every fp32 operand enters as two bf16 terms, so that products carry about 16 bits of both operands and sums are fp32; v and the
+// numbers r are bf16 activations. Warp w owns TMEM lanes 32 (w % 4) .. and a quarter of the columns of each accumulator. q, k and
+// r of the next chunk arrive while a chunk is worked on.
+constexpr int GK_C = 64, GK_THREADS = 512;
+constexpr int GK_Q_OFF = 0;                        // Q~: per 64 channels hi | lo, [64 tokens] x 128 bytes
+constexpr int GK_K_OFF = 32768;                    // K~: the same
+constexpr int GK_V_OFF = GK_K_OFF + 32768;         // v [64 tokens][128], two column blocks
+constexpr int GK_S_OFF = GK_V_OFF + 16384;         // S^T [128 v][128 d]: per 64 channels hi | lo
+constexpr int GK_P_OFF = GK_S_OFF + 65536;         // P hi [128 s][64 t] | P lo [64 s][64 t]; then the outputs [64 t][128 v]
+constexpr int GK_R_OFF = GK_P_OFF + 24576;         // q | k as they are, [64 tokens][128] each
+constexpr int GK_A_OFF = GK_R_OFF + 32768;         // r [64 tokens][64]
+constexpr int GK_SUM_OFF = GK_A_OFF + 8192;        // log decays of 16 tokens, [4][128] fp32
+constexpr int GK_DEC_OFF = GK_SUM_OFF + 2048;      // e^{b_last} [128]
+constexpr int GK_BAR_OFF = GK_DEC_OFF + 512;
+constexpr int GK_SMEM = GK_BAR_OFF + 64 + 1024;
+constexpr uint32_t GK_SC = 0, GK_O = 64, GK_ST = 128, GK_Z = 256, GK_W = 320;  // TMEM columns
+constexpr float GK_RANGE = 90.f;                   // log2 of the largest e^{-b}
+constexpr float GK_FLOOR = -64.f;                  // log2 of the strongest decay of a token: what is left does not show in fp32
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// log(sigmoid(z)): log(1 + u) = 2 atanh(u / (2 + u)), u = e^-|z| <= 1, by its series (relative error below 2e-7)
+__device__ __forceinline__ float log_sigmoid_fast(float z) {
+  const float u = __expf(-fabsf(z)), s = __fdividef(u, 2.f + u), t = s * s;
+  const float y = fmaf(t, fmaf(t, fmaf(t, fmaf(t, fmaf(t, 1.f / 11.f, 1.f / 9.f), 1.f / 7.f), 1.f / 5.f), 1.f / 3.f), 1.f);
+  return fminf(z, 0.f) - 2.f * s * y;
+}
+
+__global__ void __launch_bounds__(GK_THREADS, 1) gla_chunk_kernel(const GlaParams p, int* status) {
+  extern __shared__ uint8_t smb[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smb) + 1023) & ~uintptr_t(1023));
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + GK_BAR_OFF);  // Z, scores, state and O of the state, O
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 4);
+  int* far = reinterpret_cast<int*>(tmem_slot + 1);
+  float* sum_s = reinterpret_cast<float*>(smem + GK_SUM_OFF);
+  float* dec_s = reinterpret_cast<float*>(smem + GK_DEC_OFF);
+  pdl_wait();
+  const int v0 = blockIdx.x * 128, h = blockIdx.y, b = p.b0 + blockIdx.z;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, quad = warp & 3, grp = warp >> 2;
+  const int first = p.cu_q[b], n = p.cu_q[b + 1] - first, slot = p.slots[b];
+  if (n <= 0 || slot < 0) return;  // uniform for the CTA, before any barrier or allocation
+  const int start = p.seq_lens[b] - n, HD = p.H * p.D, HV = p.H * p.V;
+  const __nv_bfloat16* proj = static_cast<const __nv_bfloat16*>(p.proj) + (long long)first * p.stride;
+  const int VC = min(128, p.V - v0);             // columns of this CTA
+  const int nd = p.D > 64 ? 128 : 64;            // channels past D are zero
+
+  if (tid == 0) {
+    for (int i = 0; i < 4; ++i) mbar_init(&bars[i], 1);
+    *far = 0;
+    mbar_fence_init();
+  }
+  if (warp == 0) {
+    tmem_alloc(tmem_slot, 512);
+    tmem_relinquish();
+  }
+  // q, k, r of the tokens from t0 on
+  auto load_qk = [&](int t0) {
+    const int groups = nd >> 3;
+    for (int i = tid; i < GK_C * groups; i += GK_THREADS) {
+      const int t = i / groups, d = i % groups * 8;
+      const bool on = t0 + t < n && d < p.D;
+      const __nv_bfloat16* src = proj + (on ? (long long)(t0 + t) * p.stride + h * p.D + d : 0);
+      uint8_t* to = smem + GK_R_OFF + t * 256 + d * 2;
+      cp_async16(to, src, on);
+      cp_async16(to + 16384, on ? src + HD : src, on);
+    }
+    const __nv_bfloat16* r = proj + 2 * (HD + HV);
+    if ((p.rank & 7) == 0) {
+      const int t = tid >> 3, g = tid & 7;  // 64 tokens, 8 groups of eight
+      const bool on = t0 + t < n && g * 8 < p.rank;
+      cp_async16(smem + GK_A_OFF + t * 128 + ((g ^ (t & 7)) << 4), r + (on ? (long long)(t0 + t) * p.stride + g * 8 : 0), on);
+    } else {
+      for (int i = tid; i < GK_C * 64; i += GK_THREADS) {
+        const int t = i >> 6, c = i & 63;
+        const bool on = t0 + t < n && c < p.rank;
+        *reinterpret_cast<__nv_bfloat16*>(smem + GK_A_OFF + t * 128 + (((c >> 3) ^ (t & 7)) << 4) + (c & 7) * 2) =
+            on ? r[(long long)(t0 + t) * p.stride + c] : __float2bfloat16(0.f);
+      }
+    }
+    cp_async_commit();
+  };
+  auto load_v = [&](int t0) {
+    for (int i = tid; i < GK_C * 16; i += GK_THREADS) {
+      const int t = i >> 4, g = i & 15;
+      const bool on = t0 + t < n && g * 8 < VC;
+      cp_async16(smem + GK_V_OFF + (g >> 3) * 8192 + t * 128 + (((g & 7) ^ (t & 7)) << 4),
+                 proj + (on ? (long long)(t0 + t) * p.stride + 2 * HD + h * p.V + v0 + g * 8 : 0), on);
+    }
+    cp_async_commit();
+  };
+  load_qk(0);
+  load_v(0);
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *tmem_slot, my = tmem + ((uint32_t)(quad * 32) << 16);
+  pdl_trigger();  // TMEM is held
+
+  const int row = quad * 32 + lane;              // TMEM lane: channel d, state column v or token s
+  // this thread's channel: its row of W (by the first quarter of the warps) and its bias
+  const bool d_on = row < p.D;
+  const float bias = d_on ? p.decay_b[h * p.D + row] : 0.f;
+  const int r_steps = (p.rank + 15) / 16;
+  if (grp == 0) {
+    uint32_t w[32];
+    const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(p.decay_w) + (long long)(h * p.D + (d_on ? row : 0)) * p.rank;
+#pragma unroll
+    for (int i = 0; i < 32; ++i)
+      w[i] = pack_bf16x2(d_on && 2 * i < p.rank ? dl_f(src[2 * i]) : 0.f, d_on && 2 * i + 1 < p.rank ? dl_f(src[2 * i + 1]) : 0.f);
+    tmem_st_32x32(my + GK_W, w);
+  }
+  // 32 fp32 values as two bf16 terms into four 16-byte groups of a 128-byte row, starting at group g0
+  auto put32 = [&](uint8_t* hi_row, uint8_t* lo_row, int g0, const float (&f)[32]) {
+#pragma unroll
+    for (int g = 0; g < 4; ++g) {
+      uint32_t hi[4], lo[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) split2(f[8 * g + 2 * k], f[8 * g + 2 * k + 1], hi[k], lo[k]);
+      const int off = ((g0 + g) ^ (row & 7)) << 4;
+      *reinterpret_cast<uint4*>(hi_row + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      *reinterpret_cast<uint4*>(lo_row + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    }
+  };
+  // the state: this thread's column v and channels c0 .. c0 + 31
+  const int c0 = grp * 32;
+  const bool s_on = c0 < nd;
+  float* st = p.state + (((long long)slot * p.H + h) * p.V + v0 + row) * p.D;
+  uint8_t* s_hi = smem + GK_S_OFF + (c0 >> 6) * 32768 + row * 128;
+  if (s_on) {
+    float f[32];
+    uint32_t w[32];
+#pragma unroll
+    for (int e = 0; e < 32; ++e) {
+      f[e] = start > 0 && row < VC && c0 + e < p.D ? st[c0 + e] : 0.f;
+      w[e] = __float_as_uint(f[e]);
+    }
+    put32(s_hi, s_hi + 16384, (c0 & 32) >> 3, f);
+    tmem_st_32x32(my + GK_ST + c0, w);
+  }
+  tmem_st_wait();
+
+  const uint32_t base = smem_u32(smem);
+  const int k_steps = (p.D + 15) / 16;
+  constexpr uint32_t id_kk = umma_idesc(1, 1, 0, 0, 128, 64);           // both K-major
+  constexpr uint32_t id_mm = umma_idesc(1, 1, 1, 1, 128, 64);           // both MN-major
+  const uint32_t id_st = umma_idesc(1, 1, 1, 1, 128, (uint32_t)nd);
+  const bool issuer = warp == 0 && elect_one();
+  const float qscale = 1.f / sqrtf((float)p.D), rate = p.inv_tau * 1.4426950408889634f;
+  bool ok = true;
+  // every thread waits for products; one failed wait ends the loop for the whole CTA
+  auto wait = [&](int i, uint32_t parity, int detail) {
+    bool good = false;  // a few products take microseconds: bounded by attempts, without reading the clock
+    for (int a = 0; a < (1 << 22) && !good; ++a) good = mbar_try_wait(&bars[i], parity);
+    if (!good) report_error(status, ERR_WAIT_TMEM_FULL, detail);
+    tc_fence_after();
+    ok = good && ok;
+  };
+
+  int t0 = 0;
+  for (uint32_t it = 0; t0 < n; ++it) {
+    const uint32_t parity = it & 1;
+    cp_async_wait<1>();  // q, k and r (the newest group is v)
+    fence_proxy_async_smem();
+    tc_fence_before();
+    if (!__syncthreads_and(ok)) break;
+    if (issuer) {
+      tc_fence_after();
+      for (int k = 0; k < r_steps; ++k)
+        tc_mma_f16_ta(tmem + GK_Z, tmem + GK_W + k * 8, umma_smem_desc(base + GK_A_OFF + k * 32, 16, 1024), id_kk, k != 0);
+      tc_commit(&bars[0]);
+    }
+    wait(0, parity, 4 * it);
+    // running log2 decays of this thread's channel over its sixteen tokens
+    float lb[16];
+    {
+      uint32_t z[16];
+      tmem_ld_32x16(my + GK_Z + grp * 16, z);
+      tmem_ld_wait();
+      float run = 0.f;
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        const float l = fmaxf(log_sigmoid_fast(__uint_as_float(z[i]) + bias) * rate, GK_FLOOR);
+        run += d_on && t0 + grp * 16 + i < n ? l : 0.f;
+        lb[i] = run;
+      }
+      sum_s[grp * 128 + row] = run;
+    }
+    __syncthreads();
+    float total = 0.f;
+    {
+      float before = 0.f;
+#pragma unroll
+      for (int g = 0; g < 4; ++g) {
+        const float x = sum_s[g * 128 + row];
+        total += x;
+        if (g < grp) before += x;
+      }
+#pragma unroll
+      for (int i = 0; i < 16; ++i) lb[i] += before;
+    }
+    int cnt = min(GK_C, n - t0);  // tokens of this chunk
+    if (!__syncthreads_and(total >= -GK_RANGE)) {  // the largest power of two of them that stays within the range
+      int out = 0;
+#pragma unroll
+      for (int k = 0; k < 6; ++k) {
+        const int t = (1 << k) - 1;
+        if ((t >> 4) == grp && lb[t & 15] < -GK_RANGE) out |= 1 << k;
+      }
+      if (out) atomicOr(far, out);
+      __syncthreads();
+      out = *far;
+      int m = 1;
+      while (m < 32 && !(out & (2 * m))) m *= 2;
+      cnt = min(cnt, m);
+      __syncthreads();
+      if (tid == 0) *far = 0;
+    }
+    if (row < nd) {
+      const __nv_bfloat16* raw = reinterpret_cast<const __nv_bfloat16*>(smem + GK_R_OFF) + row;
+      uint8_t* qd = smem + GK_Q_OFF + (row >> 6) * 16384 + (row & 7) * 2;
+      const int g = (row & 63) >> 3;
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        const int t = grp * 16 + i;
+        const bool on = t < cnt;
+        const float q = on ? dl_f(raw[t * 128]) * qscale * ex2(lb[i]) : 0.f;
+        const float k = on ? dl_f(raw[8192 + t * 128]) * ex2(-lb[i]) : 0.f;
+        const __nv_bfloat16 qh = __float2bfloat16(q), kh = __float2bfloat16(k);
+        uint8_t* to = qd + t * 128 + ((g ^ (i & 7)) << 4);
+        *reinterpret_cast<__nv_bfloat16*>(to) = qh;
+        *reinterpret_cast<__nv_bfloat16*>(to + 8192) = __float2bfloat16(q - __bfloat162float(qh));
+        *reinterpret_cast<__nv_bfloat16*>(to + GK_K_OFF) = kh;
+        *reinterpret_cast<__nv_bfloat16*>(to + GK_K_OFF + 8192) = __float2bfloat16(k - __bfloat162float(kh));
+        if (t == cnt - 1) dec_s[row] = ex2(lb[i]);
+      }
+    }
+    cp_async_wait<0>();  // v
+    fence_proxy_async_smem();
+    tc_fence_before();
+    if (!__syncthreads_and(ok)) break;
+    if (issuer) {
+      tc_fence_after();
+      auto q_desc = [&](int term, int k) {
+        return umma_smem_desc(base + GK_Q_OFF + (k >> 2) * 16384 + term * 8192 + (k & 3) * 32, 16, 1024);
+      };
+      for (int term = 0; term < 2; ++term)
+        for (int k = 0; k < k_steps; ++k)
+          tc_mma_f16(tmem + GK_SC, umma_smem_desc(base + GK_K_OFF + (k >> 2) * 16384 + (k & 3) * 32, 16, 1024), q_desc(term, k),
+                     id_kk, term != 0 || k != 0);
+      tc_commit(&bars[1]);
+      for (int term = 0; term < 3; ++term)  // hi hi, hi lo, lo hi
+        for (int k = 0; k < k_steps; ++k)
+          tc_mma_f16(tmem + GK_O,
+                     umma_smem_desc(base + GK_S_OFF + (k >> 2) * 32768 + (term == 2 ? 16384 : 0) + (k & 3) * 32, 16, 1024),
+                     q_desc(term == 1, k), id_kk, term != 0 || k != 0);
+      for (int term = 0; term < 2; ++term)
+        for (int k = 0; k < GK_C / 16; ++k)
+          tc_mma_f16(tmem + GK_ST, umma_smem_desc(base + GK_V_OFF + k * 2048, 8192, 1024),
+                     umma_smem_desc(base + GK_K_OFF + term * 8192 + k * 2048, 16384, 1024), id_st, 1);
+      tc_commit(&bars[2]);
+    }
+    load_qk(t0 + cnt);
+    // scores: this thread's row s (hi or lo term of K~) and sixteen tokens t
+    wait(1, parity, 4 * it + 1);
+    {
+      uint32_t x[16];
+      tmem_ld_32x16(my + GK_SC + grp * 16, x);
+      tmem_ld_wait();
+      const int s = row & 63;
+      uint8_t* dst = smem + GK_P_OFF + row * 128;
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        uint32_t hi[4], lo[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const int e = 8 * j + 2 * k, t = grp * 16 + e;
+          split2(t >= s ? __uint_as_float(x[e]) : 0.f, t + 1 >= s ? __uint_as_float(x[e + 1]) : 0.f, hi[k], lo[k]);
+        }
+        const int off = ((2 * grp + j) ^ (row & 7)) << 4;
+        *reinterpret_cast<uint4*>(dst + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        if (quad < 2) *reinterpret_cast<uint4*>(dst + 16384 + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+      }
+    }
+    fence_proxy_async_smem();
+    tc_fence_before();
+    if (!__syncthreads_and(ok)) break;
+    if (issuer) {
+      tc_fence_after();
+      for (int k = 0; k < 12; ++k)  // P hi of both partial sums, P lo of the first
+        tc_mma_f16(tmem + GK_O, umma_smem_desc(base + GK_V_OFF + (k & 3) * 2048, 8192, 1024),
+                   umma_smem_desc(base + GK_P_OFF + k * 2048, 8192, 1024), id_mm, 1);
+      tc_commit(&bars[3]);
+    }
+    // the state behind the chunk
+    wait(2, parity, 4 * it + 2);
+    const bool last = t0 + cnt >= n;
+    if (s_on) {
+      uint32_t x[32];
+      tmem_ld_32x32(my + GK_ST + c0, x);
+      tmem_ld_wait();
+      float f[32];
+#pragma unroll
+      for (int e = 0; e < 32; e += 4) {
+        const float4 d4 = *reinterpret_cast<const float4*>(dec_s + c0 + e);
+        f[e] = __uint_as_float(x[e]) * d4.x;
+        f[e + 1] = __uint_as_float(x[e + 1]) * d4.y;
+        f[e + 2] = __uint_as_float(x[e + 2]) * d4.z;
+        f[e + 3] = __uint_as_float(x[e + 3]) * d4.w;
+      }
+      if (last) {
+        if (ok && row < VC)
+#pragma unroll
+          for (int e = 0; e < 32; ++e)
+            if (c0 + e < p.D) st[c0 + e] = f[e];
+      } else {
+        put32(s_hi, s_hi + 16384, (c0 & 32) >> 3, f);
+#pragma unroll
+        for (int e = 0; e < 32; ++e) x[e] = __float_as_uint(f[e]);
+        tmem_st_32x32(my + GK_ST + c0, x);
+      }
+      tmem_st_wait();
+    }
+    wait(3, parity, 4 * it + 3);
+    {
+      uint32_t x[16];
+      tmem_ld_32x16(my + GK_O + grp * 16, x);
+      tmem_ld_wait();
+      __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(smem + GK_P_OFF) + row;
+#pragma unroll
+      for (int e = 0; e < 16; ++e) o[(grp * 16 + e) * 128] = __float2bfloat16(__uint_as_float(x[e]));
+    }
+    if (!__syncthreads_and(ok)) break;
+    load_v(t0 + cnt);
+    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (long long)(first + t0) * p.out_stride + (long long)h * p.V + v0;
+    for (int i = tid; i < GK_C * 16; i += GK_THREADS) {
+      const int t = i >> 4, g = i & 15;
+      if (t < cnt && g * 8 < VC)
+        *reinterpret_cast<uint4*>(out + (long long)t * p.out_stride + g * 8) =
+            *reinterpret_cast<const uint4*>(smem + GK_P_OFF + t * 256 + g * 16);
+    }
+    t0 += cnt;
+  }
+  cp_async_wait<0>();
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 0) {
+    tc_fence_after();
+    tmem_dealloc(tmem, 512);
+  }
+}
+
+template <typename T, int NR>
+static int run_gla_step(const GlaParams& p, int B, cudaStream_t stream) {
+  const size_t smem = (3 * NR * 8 + 2 * p.V + p.rank) * sizeof(float);
+  cudaError_t e = vb_launch_pdl(gla_step_kernel<T, NR>, dim3(p.H, B), dim3(GS_THREADS), smem, stream, 1, p);
+  vb_count_launch();
+  return (int)e;
+}
+
+template <typename T, int NR>
+static int run_gla_scan(const GlaParams& p, int B, cudaStream_t stream) {
+  const size_t smem = (3 * GC_TB * NR * 8 + 2 * GC_TB * GC_VB) * sizeof(float);
+  static bool attr = false;
+  if (!attr) {
+    VB_CUDA_CHECK(cudaFuncSetAttribute(gla_scan_kernel<T, NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    attr = true;
+  }
+  const dim3 g(p.H, (p.V + GC_VB - 1) / GC_VB, B);
+  cudaError_t e = vb_launch_pdl(gla_scan_kernel<T, NR>, g, dim3(GS_THREADS), smem, stream, 1, p);
+  vb_count_launch();
+  return (int)e;
+}
+
+template <typename T>
+static int run_gla(GlaParams p, int T_, int B, int singles, int chunk, int* status, cudaStream_t stream) {
+  const int nr = p.D <= 32 ? 4 : p.D <= 64 ? 8 : p.D <= 128 ? 16 : 32;
+  int rc = 0;
+  if (singles > 0) {
+    rc = nr == 4    ? run_gla_step<T, 4>(p, singles, stream)
+         : nr == 8  ? run_gla_step<T, 8>(p, singles, stream)
+         : nr == 16 ? run_gla_step<T, 16>(p, singles, stream)
+                    : run_gla_step<T, 32>(p, singles, stream);
+    if (rc || singles == B) return rc;
+  }
+  p.b0 = singles;
+  if (chunk) {
+    static bool attr = false;
+    if (!attr) {
+      VB_CUDA_CHECK(cudaFuncSetAttribute(gla_chunk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, GK_SMEM));
+      attr = true;
+    }
+    const dim3 g((p.V + 127) / 128, p.H, B - singles);
+    rc = (int)vb_launch_pdl(gla_chunk_kernel, g, dim3(GK_THREADS), GK_SMEM, stream, 1, p, status);
+    vb_count_launch();
+  } else {
+    cudaError_t e = vb_launch_pdl(gla_decay_kernel<T>, dim3(T_, (p.H * p.D + 127) / 128), dim3(128), 0, stream, 1, p);
+    vb_count_launch();
+    if (e != cudaSuccess) return (int)e;
+    rc = nr == 4    ? run_gla_scan<T, 4>(p, B - singles, stream)
+         : nr == 8  ? run_gla_scan<T, 8>(p, B - singles, stream)
+         : nr == 16 ? run_gla_scan<T, 16>(p, B - singles, stream)
+                    : run_gla_scan<T, 32>(p, B - singles, stream);
+  }
+  if (rc) return rc;
+  // the leading sequences have one token each, which the step has finished
+  T* out = static_cast<T*>(p.out) + (long long)singles * p.out_stride;
+  const T* gate = static_cast<const T*>(p.proj) + (long long)singles * p.stride + 2 * p.H * p.D + p.H * p.V;
+  return launch_gated_norm<T>(out, p.out_stride, gate, p.stride, p.norm_w, p.H, p.V, p.eps, T_ - singles, stream);
+}
+
+}  // namespace vb
+
+using namespace vb;
+
+// 1 if the chunked form serves these sizes (bf16 only).
+extern "C" int vb_gla_chunk_supported(int H, int D, int V, int rank) {
+  return H > 0 && D >= 8 && D <= 128 && (D & 7) == 0 && V >= 8 && V <= 256 && (V & 7) == 0 && rank > 0 && rank <= 64;
+}
+
+// Limits: D, V <= 256, rank <= 4096. The leading `singles` sequences bring one token each (singles == B: all do); the others take the
+// chunked form (chunk) or the scan, with decay fp32 scratch [T, H D].
+extern "C" int vb_gla(const void* proj, long long stride, const void* decay_w, const float* decay_b, const void* norm_w,
+                      float* state, const int* cu_q, const int* seq_lens, const int* slots, float* decay, void* out,
+                      long long out_stride, int T, int B, int singles, int max_q, int H, int D, int V, int rank, float tau,
+                      float eps, int f32, int chunk, int* status, cudaStream_t stream) {
+  if (T <= 0 || B <= 0 || max_q <= 0) return 0;
+  if (H <= 0 || D <= 0 || D > 256 || V <= 0 || V > 256 || rank <= 0 || rank > 4096 || !(tau > 0.f) || singles < 0 || singles > B ||
+      B > 65535 || H > 65535 ||
+      (singles < B && (chunk ? !vb_gla_chunk_supported(H, D, V, rank) || f32 || (stride & 7) || (out_stride & 7) : decay == nullptr)))
+    return -3;
+  GlaParams p{proj, stride, decay_w, decay_b, norm_w, state, cu_q, seq_lens, slots, decay, out, out_stride, H, D, V, rank, 0,
+              1.f / tau, eps};
+  const int rc = f32 ? run_gla<float>(p, T, B, singles, chunk, status, stream)
+                     : run_gla<__nv_bfloat16>(p, T, B, singles, chunk, status, stream);
+  return rc ? rc : (int)cudaGetLastError();
+}

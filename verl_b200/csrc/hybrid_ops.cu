@@ -10,13 +10,15 @@
 namespace vb {
 
 // ---------------------------------------------------------------------------------------------------------------
-// res[t] = table[ids[t]] * scale, fp32; y (when given): the same in the table's type.
+// res[t] = table[ids[t]] * scale (+ pos[positions[t]], n_pos rows), fp32; y (when given): the same in the table's type.
 template <typename T>
 __global__ void embed_scaled_kernel(const long long* __restrict__ ids, const T* __restrict__ table,
-                                    float* __restrict__ res, T* __restrict__ y, int H, float scale) {
+                                    float* __restrict__ res, T* __restrict__ y, int H, float scale, const T* __restrict__ pos,
+                                    const long long* __restrict__ positions, int n_pos) {
   pdl_trigger();
   pdl_wait();
   const T* src = table + ids[blockIdx.x] * (long long)H;
+  const T* add = pos ? pos + max(min(positions[blockIdx.x], (long long)n_pos - 1), 0ll) * H : nullptr;
   float* dst = res + (long long)blockIdx.x * H;
   if ((H & 7) == 0) {
     for (int v = threadIdx.x; v < (H >> 3); v += blockDim.x) {
@@ -24,12 +26,18 @@ __global__ void embed_scaled_kernel(const long long* __restrict__ ids, const T* 
       ld8(src + v * 8, f);
 #pragma unroll
       for (int i = 0; i < 8; ++i) f[i] *= scale;
+      if (add) {
+        float g[8];
+        ld8(add + v * 8, g);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] += g[i];
+      }
       st8(dst + v * 8, f);
       if (y) st8(y + (long long)blockIdx.x * H + v * 8, f);
     }
   } else {
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
-      const float f = to_f<T>(src[i]) * scale;
+      const float f = to_f<T>(src[i]) * scale + (add ? to_f<T>(add[i]) : 0.f);
       dst[i] = f;
       if (y) y[(long long)blockIdx.x * H + i] = from_f<T>(f);
     }
@@ -99,73 +107,41 @@ __global__ void add_rmsnorm_kernel(const T* __restrict__ delta, long long delta_
 }
 
 // ---------------------------------------------------------------------------------------------------------------
-// res += delta / sqrt(mean(delta^2) + eps) * w; y = res, or with fw: y = res / sqrt(mean(res^2) + eps) * fw * fscale.
+// res += d / sqrt(mean(d^2) + eps) * w with d = delta, or with a gate delta * sigmoid(gate); y = res, or with fw:
+// y = res / sqrt(mean(res^2) + eps) * fw * fscale.
 template <typename T>
-__global__ void rmsnorm_add_kernel(const T* __restrict__ delta, long long delta_stride, float* __restrict__ res,
-                                   const T* __restrict__ w, const T* __restrict__ fw, float fscale, T* __restrict__ y,
-                                   int H, float eps) {
+__global__ void rmsnorm_add_kernel(const T* __restrict__ delta, long long delta_stride, const T* __restrict__ gate,
+                                   long long gate_stride, float* __restrict__ res, const T* __restrict__ w,
+                                   const T* __restrict__ fw, float fscale, T* __restrict__ y, int H, float eps, bool vec) {
   extern __shared__ float row[];
   __shared__ float sh[32];
   pdl_trigger();
   pdl_wait();
   const T* d = delta + (long long)blockIdx.x * delta_stride;
-  float* r = res + (long long)blockIdx.x * H;
-  T* out = y + (long long)blockIdx.x * H;
-  const bool vec = (H & 7) == 0 && (delta_stride & 7) == 0;
+  const T* g = gate ? gate + (long long)blockIdx.x * gate_stride : nullptr;
   float ss = 0.f;
   if (vec) {
     for (int v = threadIdx.x; v < (H >> 3); v += blockDim.x) {
       float f[8];
       ld8(d + v * 8, f);
+      if (g) {
+        float z[8];
+        ld8(g + v * 8, z);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] *= sigmoid_t<T>(z[i]);
+      }
       st8(row + v * 8, f);
 #pragma unroll
       for (int i = 0; i < 8; ++i) ss += f[i] * f[i];
     }
   } else {
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
-      const float f = to_f<T>(d[i]);
+      const float f = to_f<T>(d[i]) * (g ? sigmoid_t<T>(to_f<T>(g[i])) : 1.f);
       row[i] = f;
       ss += f * f;
     }
   }
-  const float inv = 1.f / sqrtf(block_sum_all(ss, sh) / (float)H + eps);
-  ss = 0.f;
-  if (vec) {
-    for (int v = threadIdx.x; v < (H >> 3); v += blockDim.x) {  // the same elements this thread has stored
-      float f[8], g[8], x[8];
-      ld8(r + v * 8, x);
-      ld8(row + v * 8, f);
-      ld8(w + v * 8, g);
-#pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        x[i] += f[i] * inv * g[i];
-        ss += x[i] * x[i];
-      }
-      st8(r + v * 8, x);
-      if (fw) st8(row + v * 8, x); else st8(out + v * 8, x);
-    }
-  } else {
-    for (int i = threadIdx.x; i < H; i += blockDim.x) {
-      const float x = r[i] + row[i] * inv * to_f<T>(w[i]);
-      r[i] = x;
-      ss += x * x;
-      if (fw) row[i] = x; else out[i] = from_f<T>(x);
-    }
-  }
-  if (fw == nullptr) return;
-  const float fi = fscale / sqrtf(block_sum_all(ss, sh) / (float)H + eps);
-  if (vec) {
-    for (int v = threadIdx.x; v < (H >> 3); v += blockDim.x) {
-      float f[8], g[8];
-      ld8(row + v * 8, f);
-      ld8(fw + v * 8, g);
-#pragma unroll
-      for (int i = 0; i < 8; ++i) f[i] = f[i] * fi * g[i];
-      st8(out + v * 8, f);
-    }
-  } else {
-    for (int i = threadIdx.x; i < H; i += blockDim.x) out[i] = from_f<T>(row[i] * fi * to_f<T>(fw[i]));
-  }
+  norm_row_add(row, ss, res + (long long)blockIdx.x * H, w, fw, fscale, y + (long long)blockIdx.x * H, H, eps, vec, sh);
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -226,6 +202,35 @@ __global__ void glu_kernel(const T* __restrict__ gu, long long stride, T* __rest
   }
 }
 
+// y[t][c] = act(x[t][c]), c < n: ACT 0: gelu with erf, 1: the square of relu. blk_expert (or null): see glu_kernel.
+template <typename T, int ACT>
+__global__ void activation_kernel(const T* __restrict__ x, long long stride, T* __restrict__ y, long long total, int n,
+                                  const int* __restrict__ blk_expert, bool vec) {
+  pdl_trigger();
+  pdl_wait();
+  const long long step = (long long)gridDim.x * blockDim.x, i0 = blockIdx.x * (long long)blockDim.x + threadIdx.x;
+  auto act = [](float z) {
+    if (ACT == 0) return 0.5f * z * (1.f + erff(z * 0.70710678118654752f));
+    const float r = fmaxf(z, 0.f);
+    return r * r;
+  };
+  const int per = vec ? n >> 3 : n;
+  for (long long i = i0; i < (vec ? total / 8 : total); i += step) {
+    const long long t = i / per;
+    if (blk_expert && blk_expert[t >> 7] < 0) continue;
+    if (vec) {
+      const int c = (int)(i - t * per) * 8;
+      float f[8];
+      ld8(x + t * stride + c, f);
+#pragma unroll
+      for (int k = 0; k < 8; ++k) f[k] = act(f[k]);
+      st8(y + t * n + c, f);
+    } else {
+      y[i] = from_f<T>(act(to_f<T>(x[t * stride + (i - t * n)])));
+    }
+  }
+}
+
 // y[t] = gelu(g[t]) * table[ids[t]][lo ..]. V elements per thread.
 template <typename T, int V>
 __global__ void gelu_rows_kernel(const T* __restrict__ g, long long g_stride, const long long* __restrict__ ids,
@@ -269,13 +274,14 @@ __global__ void softcap_kernel(float* __restrict__ x, long long n, float cap) {
 
 // ---------------------------------------------------------------------------------------------------------------
 // One block per token. qkv row = [q (Hq * D) | k (Hk * D) | v (Hk * Dv)]. With norm weights: q and k are divided by the
-// root mean square of the WHOLE projection (all heads together) and multiplied by their weights. q is normalised in
-// place; k and v go to the token's place in the paged caches ([NB, Hk, BS, D] / [NB, Hk, BS, Dv]; slot < 0: no write).
+// root mean square of the WHOLE projection (all heads together) and multiplied by their weights. With positions (of the
+// tokens), q is multiplied by 1 + coef ln(floor((position + 1) / every) + 1). q is changed in place; k and v go to the token's place in the paged caches ([NB, Hk, BS, D] / [NB, Hk, BS, Dv]; slot < 0: no write).
 template <typename T, bool VEC>
 __global__ void qk_norm_kv_write_kernel(T* __restrict__ qkv, long long stride, const T* __restrict__ qw,
                                         const T* __restrict__ kw, const long long* __restrict__ slots,
                                         T* __restrict__ kc, T* __restrict__ vc, int Hq, int Hk, int D, int Dv,
-                                        int block_size, float eps) {
+                                        int block_size, float eps, const long long* __restrict__ positions, float coef,
+                                        float every) {
   __shared__ float sh[32];
   pdl_trigger();
   pdl_wait();
@@ -285,6 +291,8 @@ __global__ void qk_norm_kv_write_kernel(T* __restrict__ qkv, long long stride, c
   const int nq = Hq * D, nk = Hk * D, nv = Hk * Dv;
   constexpr int W = VEC ? 8 : 1;
   float iq = 1.f, ik = 1.f;
+  const float temp =
+      positions ? 1.f + coef * logf((float)floor((double)(positions[blockIdx.x] + 1) / (double)every) + 1.f) : 1.f;
   if (qw != nullptr) {
     float sq = 0.f, sk = 0.f;
     for (int i = threadIdx.x * W; i < nq + nk; i += blockDim.x * W) {  // q and k are adjacent
@@ -304,16 +312,23 @@ __global__ void qk_norm_kv_write_kernel(T* __restrict__ qkv, long long stride, c
     sk = block_sum_all(sk, sh);
     iq = 1.f / sqrtf(sq / (float)nq + eps);
     ik = 1.f / sqrtf(sk / (float)nk + eps);
+  }
+  if (qw != nullptr || positions != nullptr) {
+    iq *= temp;
     for (int i = threadIdx.x * W; i < nq; i += blockDim.x * W) {
       if (VEC) {
         float f[8], g[8];
         ld8(q + i, f);
-        ld8(qw + i, g);
+        if (qw != nullptr) {
+          ld8(qw + i, g);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) f[e] = f[e] * iq * g[e];
+          for (int e = 0; e < 8; ++e) f[e] *= g[e];
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] *= iq;
         st8(q + i, f);
       } else {
-        q[i] = from_f<T>(to_f<T>(q[i]) * iq * to_f<T>(qw[i]));
+        q[i] = from_f<T>(to_f<T>(q[i]) * iq * (qw != nullptr ? to_f<T>(qw[i]) : 1.f));
       }
     }
   }
@@ -691,7 +706,8 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const TA* __restrict__ A
 // Paged attention over ragged queries on the CUDA cores: one warp per (token, query head), lanes across 32 keys for the
 // scores and across the value dims for the weighted sum. A query at position i sees key j <= i when window <= 0, or
 // i - j < window, or j < keep_first (chunk > 0: when i / chunk == j / chunk); bias[h][min(i - j, bias_len - 1)] is added to
-// the scaled score, softcap > 0 bounds it, exp(sink[h]) joins the denominator, sigmoid(gate) multiplies the result.
+// the scaled score, softcap > 0 bounds it, exp(sink[h]) joins the denominator, sigmoid(gate) multiplies the result. With shift
+// there is no softmax: a key weighs sigmoid(score - r1[h] ln(1 + r2[h] (i - j)) + shift[h]).
 struct PagedSimtParams {
   const int* cu_q;
   const int* seq_lens;
@@ -700,7 +716,9 @@ struct PagedSimtParams {
   int max_blocks, B, Hq, Hk, D, Dv, v_width, block_size, window, keep_first, chunk, bias_len;  // v_width: elements of a value row
   float scale, softcap;
   const float *bias, *sink;
-  const void* gate;  // [T, Hq * Dv] of the activation type, or null
+  const float *shift, *r1, *r2;  // [Hq] or null
+  const void* gate;  // [T, Hq * Dv] (gate_w 1: [T, Hq]) of the activation type, or null
+  int gate_w;
 };
 constexpr int PS_WARPS = 4, PS_MAX_D = 1024;
 
@@ -727,7 +745,9 @@ paged_attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ kc, const 
   __syncwarp();
   const int* bt = p.block_table + (long long)b * p.max_blocks;
   const float* bias = p.bias ? p.bias + (long long)h * p.bias_len : nullptr;
-  float m = p.sink ? p.sink[h] : -INFINITY, l = p.sink ? 1.f : 0.f, acc[PS_VREG];
+  const bool sig = p.shift != nullptr;
+  const float shift = sig ? p.shift[h] : 0.f, r1 = p.r1 ? p.r1[h] : 0.f, r2 = p.r1 ? p.r2[h] : 0.f;
+  float m = sig ? 0.f : p.sink ? p.sink[h] : -INFINITY, l = sig || p.sink ? 1.f : 0.f, acc[PS_VREG];
 #pragma unroll
   for (int i = 0; i < PS_VREG; ++i) acc[i] = 0.f;
   const int n = pos + 1;
@@ -749,14 +769,20 @@ paged_attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ kc, const 
       s = a * p.scale;
       if (bias) s += bias[min(pos - key, p.bias_len - 1)];
       if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
+      if (sig) s += shift - (p.r1 ? r1 * log1pf(r2 * (float)(pos - key)) : 0.f);
     }
-    const float nm = fmaxf(m, warp_reduce_max(s));
-    const float alpha = expf(m - nm);
-    const float w = valid ? expf(s - nm) : 0.f;
-    l = l * alpha + warp_reduce_sum(w);
-    m = nm;
+    float w;
+    if (sig) {
+      w = valid ? sigmoid_f(s) : 0.f;
+    } else {
+      const float nm = fmaxf(m, warp_reduce_max(s));
+      const float alpha = expf(m - nm);
+      w = valid ? expf(s - nm) : 0.f;
+      l = l * alpha + warp_reduce_sum(w);
+      m = nm;
 #pragma unroll
-    for (int i = 0; i < PS_VREG; ++i) acc[i] *= alpha;
+      for (int i = 0; i < PS_VREG; ++i) acc[i] *= alpha;
+    }
     const int cnt = min(32, total - c);
     for (int j = 0; j < cnt; ++j) {
       const float wj = __shfl_sync(0xffffffffu, w, j);
@@ -772,7 +798,8 @@ paged_attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ kc, const 
     const int d = lane + 32 * i;
     if (d >= p.Dv) continue;
     float x = acc[i] / l;
-    if (p.gate) x /= 1.f + expf(-to_f<T>(reinterpret_cast<const T*>(p.gate)[t * p.gate_stride + (long long)h * p.Dv + d]));
+    if (p.gate)
+      x /= 1.f + expf(-to_f<T>(reinterpret_cast<const T*>(p.gate)[t * p.gate_stride + (p.gate_w == 1 ? h : (long long)h * p.Dv + d)]));
     o[d] = from_f<T>(x);
   }
 }
@@ -782,13 +809,16 @@ paged_attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ kc, const 
 using namespace vb;
 typedef __nv_bfloat16 bf16;
 
+// pos (n_pos rows, with the tokens' positions) or null
 extern "C" int vb_embed_scaled(const long long* ids, const void* table, float* res, void* y, int T, int H, float scale,
-                               int f32, cudaStream_t stream) {
+                               const void* pos, const long long* positions, int n_pos, int f32, cudaStream_t stream) {
   if (T <= 0) return 0;
+  if (pos != nullptr && (positions == nullptr || n_pos <= 0)) return -3;
   const dim3 g(T), b(row_threads(H));
   if (f32) VB_DONE(vb_launch_pdl(embed_scaled_kernel<float>, g, b, 0, stream, 1, ids, (const float*)table, res, (float*)y, H,
-                                scale));
-  VB_DONE(vb_launch_pdl(embed_scaled_kernel<bf16>, g, b, 0, stream, 1, ids, (const bf16*)table, res, (bf16*)y, H, scale));
+                                scale, (const float*)pos, positions, n_pos));
+  VB_DONE(vb_launch_pdl(embed_scaled_kernel<bf16>, g, b, 0, stream, 1, ids, (const bf16*)table, res, (bf16*)y, H, scale,
+                        (const bf16*)pos, positions, n_pos));
 }
 
 extern "C" int vb_add_rmsnorm(const void* delta, long long delta_stride, float* res, const void* w, void* y, int T, int H,
@@ -832,6 +862,25 @@ extern "C" int vb_silu_glu(const void* gu, long long stride, void* y, int T, int
   if (row_scale) return -3;
   if (f32) return launch_glu<float>(gu, stride, y, T, F, SiluGlu<float>{}, stream);
   return launch_glu<bf16>(gu, stride, y, T, F, SiluGlu<bf16>{}, stream);
+}
+
+// y [T, n] = act of the first n elements of a row: 0 gelu with erf, 1 the square of relu. blk_expert (T / 128 of them) or null.
+extern "C" int vb_activation(const void* x, long long stride, void* y, int T, int n, int act, const int* blk_expert, int f32,
+                             cudaStream_t stream) {
+  if (T <= 0 || n <= 0) return 0;
+  if (act < 0 || act > 1) return -3;
+  const long long total = (long long)T * n;
+  const bool vec = ((n | stride) & 7) == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0;
+  const dim3 grid((unsigned)max(1ll, min((total / 8 + 255) / 256, 148ll * 16))), b(256);
+#define VB_ACT(TT, A) \
+  VB_DONE(vb_launch_pdl(activation_kernel<TT, A>, grid, b, 0, stream, 1, (const TT*)x, stride, (TT*)y, total, n, blk_expert, vec))
+  if (f32) {
+    if (act == 0) VB_ACT(float, 0);
+    VB_ACT(float, 1);
+  }
+  if (act == 0) VB_ACT(bf16, 0);
+  VB_ACT(bf16, 1);
+#undef VB_ACT
 }
 
 // y [T, n] = gelu(g) * table[ids, lo .. lo + n)
@@ -882,12 +931,15 @@ extern "C" int vb_gelu_glu(const void* gu, long long stride, void* y, int T, int
   return launch_glu<bf16>(gu, stride, y, T, F, GeluTanhGlu<bf16>{}, stream);
 }
 
-// delta rows of delta_stride elements; fw null: y = the new residual in the activation type.
-extern "C" int vb_rmsnorm_add(const void* delta, long long delta_stride, float* res, const void* w, const void* fw, float fscale,
-                              void* y, int T, int H, float eps, int f32, cudaStream_t stream) {
+// delta rows of delta_stride elements, gate rows (or null) of gate_stride; fw null: y = the new residual in the activation type.
+extern "C" int vb_rmsnorm_add(const void* delta, long long delta_stride, const void* gate, long long gate_stride, float* res,
+                              const void* w, const void* fw, float fscale, void* y, int T, int H, float eps, int f32,
+                              cudaStream_t stream) {
   if (T <= 0) return 0;
   const size_t smem = (size_t)H * 4;
   if (smem > 160 * 1024) return -3;
+  const bool vec = ((H | delta_stride | gate_stride) & 7) == 0 &&
+                   ((reinterpret_cast<uintptr_t>(delta) | reinterpret_cast<uintptr_t>(gate)) & 15) == 0;
   const dim3 g(T), b(row_threads(H));
   static bool attr = false;
   if (!attr) {
@@ -896,23 +948,23 @@ extern "C" int vb_rmsnorm_add(const void* delta, long long delta_stride, float* 
     attr = true;
   }
   if (f32)
-    VB_DONE(vb_launch_pdl(rmsnorm_add_kernel<float>, g, b, smem, stream, 1, (const float*)delta, delta_stride, res,
-                          (const float*)w, (const float*)fw, fscale, (float*)y, H, eps));
-  VB_DONE(vb_launch_pdl(rmsnorm_add_kernel<bf16>, g, b, smem, stream, 1, (const bf16*)delta, delta_stride, res,
-                        (const bf16*)w, (const bf16*)fw, fscale, (bf16*)y, H, eps));
+    VB_DONE(vb_launch_pdl(rmsnorm_add_kernel<float>, g, b, smem, stream, 1, (const float*)delta, delta_stride, (const float*)gate,
+                          gate_stride, res, (const float*)w, (const float*)fw, fscale, (float*)y, H, eps, vec));
+  VB_DONE(vb_launch_pdl(rmsnorm_add_kernel<bf16>, g, b, smem, stream, 1, (const bf16*)delta, delta_stride, (const bf16*)gate,
+                        gate_stride, res, (const bf16*)w, (const bf16*)fw, fscale, (bf16*)y, H, eps, vec));
 }
 
-// qw / kw null: no norm (q untouched, k and v only written to the cache).
+// qw / kw null: no norm (k and v only written to the cache). positions null: no factor of the queries.
 extern "C" int vb_qk_norm_kv_write(void* qkv, long long stride, const void* qw, const void* kw, const long long* slots,
                                    void* kc, void* vc, int T, int Hq, int Hk, int D, int Dv, int block_size, float eps,
-                                   int f32, cudaStream_t stream) {
+                                   const long long* positions, float coef, float every, int f32, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if ((qw == nullptr) != (kw == nullptr)) return -3;
+  if ((qw == nullptr) != (kw == nullptr) || !(every > 0.f)) return -3;
   const bool vec = (D & 7) == 0 && (Dv & 7) == 0 && (stride & 7) == 0;
   const dim3 g(T), b(row_threads(Hq * D));
 #define VB_QKN(TT, V)                                                                                              \
   VB_DONE(vb_launch_pdl(qk_norm_kv_write_kernel<TT, V>, g, b, 0, stream, 1, (TT*)qkv, stride, (const TT*)qw,       \
-                        (const TT*)kw, slots, (TT*)kc, (TT*)vc, Hq, Hk, D, Dv, block_size, eps))
+                        (const TT*)kw, slots, (TT*)kc, (TT*)vc, Hq, Hk, D, Dv, block_size, eps, positions, coef, every))
   if (f32) {
     if (vec) VB_QKN(float, true);
     VB_QKN(float, false);
@@ -956,9 +1008,11 @@ extern "C" int vb_paged_attention_simt(const void* q, long long q_stride, const 
                                        const int* block_table, int max_blocks, const int* cu_q, const int* seq_lens,
                                        int T, int B, int Hq, int Hk, int D, int Dv, int v_width, int block_size, float scale,
                                        int window, int keep_first, int chunk, const float* bias, int bias_len,
-                                       float softcap, const float* sink, const void* gate, long long gate_stride, void* out,
+                                       float softcap, const float* sink, const float* shift, const float* r1,
+                                       const float* r2, const void* gate, long long gate_stride, int gate_w, void* out,
                                        long long out_stride, int f32, cudaStream_t stream) {
   if (T <= 0 || B <= 0) return 0;
+  if ((shift && (bias || sink || softcap > 0.f)) || (r1 && (!shift || !r2))) return -3;
   if (Hk <= 0 || Hq % Hk != 0 || D <= 0 || D > PS_MAX_D || Dv <= 0 || Dv > PS_MAX_D || v_width < Dv || (bias && bias_len <= 0))
     return -3;
   PagedSimtParams p{};
@@ -967,6 +1021,7 @@ extern "C" int vb_paged_attention_simt(const void* q, long long q_stride, const 
   p.max_blocks = max_blocks; p.B = B; p.Hq = Hq; p.Hk = Hk; p.D = D; p.Dv = Dv; p.v_width = v_width; p.block_size = block_size;
   p.window = window; p.keep_first = keep_first; p.chunk = chunk; p.bias_len = bias_len;
   p.scale = scale; p.softcap = softcap; p.bias = bias; p.sink = sink; p.gate = gate;
+  p.shift = shift; p.r1 = r1; p.r2 = r2; p.gate_w = gate_w;
   const dim3 g(T, (Hq + PS_WARPS - 1) / PS_WARPS), b(PS_WARPS * 32);
 #define VB_PSA(TT, V)                                                                                             \
   VB_DONE(vb_launch_pdl(paged_attn_simt_kernel<TT, V>, g, b, 0, stream, 1, (const TT*)q, (const TT*)kc, (const TT*)vc, \

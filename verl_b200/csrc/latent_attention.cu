@@ -589,7 +589,7 @@ extern "C" int vb_latent_decode_splits(int T, int H, int chunks) {
 }
 
 int vb_decode_merge(const float* o_part, const float* ml_part, int B, int Hq, int D, int num_splits, void* out,
-                    long long out_stride, const void* gate, long long gate_stride, cudaStream_t stream);
+                    long long out_stride, const void* gate, long long gate_stride, int gate_w, cudaStream_t stream);
 
 // Row t of q [T, H, width] is one of the last positions of its sequence (cu_q [B + 1], seq_lens [B]; T == B: one row each) and
 // sees the page rows [num_blocks, block_size, width] up to its own (window > 0: the last `window` of them); the first `rank`
@@ -630,5 +630,5 @@ extern "C" int vb_latent_decode(const void* q, const void* pages, int num_blocks
   vb_count_launch(num_splits > 1 ? 2 : 1);
   if (rc == 0) rc = (int)cudaGetLastError();
   if (rc || num_splits == 1) return rc;
-  return vb_decode_merge(p.o_part, p.ml_part, T, H, rank, num_splits, out, (long long)H * rank, nullptr, 0, stream);
+  return vb_decode_merge(p.o_part, p.ml_part, T, H, rank, num_splits, out, (long long)H * rank, nullptr, 0, 0, stream);
 }

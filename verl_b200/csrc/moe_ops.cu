@@ -10,6 +10,7 @@ constexpr int MR_MAX_E = 512, MR_MAX_TOP = 32, MR_BLK = 128;
 
 struct MoeRouteParams {
   const float* logits;
+  const float* correction;  // [E] or null: joins the scores for the choice
   long long stride;
   int T, E, top, softmax, renormalize, per_block, nblk;
   int *idx, *dest, *blk_expert;  // [T, top], [T, top], [nblk]
@@ -53,7 +54,7 @@ __device__ __forceinline__ void fill_blocks(const int* off_s, int E, int* blk_ex
 
 // One warp per token. NV = scores per lane.
 template <int NV>
-__global__ void moe_route_kernel(const MoeRouteParams p) {
+__global__ void __launch_bounds__(1024) moe_route_kernel(const MoeRouteParams p) {
   __shared__ int hist[MR_MAX_E], base[MR_MAX_E + 1];
   pdl_trigger();
   pdl_wait();
@@ -80,18 +81,25 @@ __global__ void moe_route_kernel(const MoeRouteParams p) {
 #pragma unroll
       for (int i = 0; i < NV; ++i) s[i] = sigmoid_f(s[i]);
     }
-    // scores are never negative: -1 for what is no number (chosen last), -2 for what is taken or not there
+    // scores are never negative: -1 for what is no number (chosen last). c: what the choice goes by, -inf for what is taken or
+    // not there
+    float c[NV];
 #pragma unroll
-    for (int i = 0; i < NV; ++i) s[i] = i * 32 + lane >= p.E ? -2.f : (s[i] >= 0.f ? s[i] : -1.f);
+    for (int i = 0; i < NV; ++i) {
+      const int e = i * 32 + lane;
+      s[i] = s[i] >= 0.f ? s[i] : -1.f;
+      c[i] = e >= p.E ? -INFINITY : s[i] + (p.correction && s[i] >= 0.f ? p.correction[e] : 0.f);
+      if (e < p.E) c[i] = fmaxf(c[i], -3.0e38f);  // a correction that is no number, or minus infinity
+    }
     int my_e = 0;
     float my_w = 0.f, total = 0.f;
     for (int k = 0; k < p.top; ++k) {
-      float v = -3.f;
-      int e = 0;
+      float v = -INFINITY;
+      int e = p.E;
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
-        if (s[i] > v) {
-          v = s[i];
+        if (c[i] > v) {
+          v = c[i];
           e = i * 32 + lane;
         }
       }
@@ -104,9 +112,14 @@ __global__ void moe_route_kernel(const MoeRouteParams p) {
           e = oe;
         }
       }
+      float own = 0.f;
 #pragma unroll
       for (int i = 0; i < NV; ++i)
-        if (i * 32 + lane == e) s[i] = -2.f;
+        if (i * 32 + lane == e) {
+          c[i] = -INFINITY;
+          own = s[i];
+        }
+      v = __shfl_sync(0xffffffffu, own, e & 31);  // the score itself is the weight
       total += v;
       if (lane == k) {
         my_e = e;
@@ -116,7 +129,7 @@ __global__ void moe_route_kernel(const MoeRouteParams p) {
     if (lane < p.top) {
       const long long at = (long long)t * p.top + lane;
       p.idx[at] = my_e;
-      p.weight[at] = p.renormalize ? my_w / total : my_w;
+      p.weight[at] = p.renormalize ? my_w / (total + 1e-20f) : my_w;
       p.dest[at] = atomicAdd(&hist[my_e], 1);
     }
   }
@@ -184,13 +197,15 @@ __global__ void moe_gather_kernel(const T* __restrict__ x, long long stride, con
   }
 }
 
-// res[t] += sum over k of out[dest[t, k]] (* weight[t, k]) + shared[t] * sigmoid(logit[t]); y = res / sqrt(mean + eps) * w, or
-// without w the residual. One block per token.
+// d = sum over k of out[dest[t, k]] (* weight[t, k]) + shared[t] * sigmoid(logit[t]). Without post: res[t] += d,
+// y = res / sqrt(mean + eps) * w, or without w the residual. With post: d *= sigmoid(gate[t]) element by element (when given),
+// res += d / sqrt(mean(d^2) + eps) * post, y = res / sqrt(mean + eps) * w * scale. One block per token.
 template <typename T>
 __global__ void moe_combine_kernel(const T* __restrict__ out, const int* __restrict__ dest, const float* __restrict__ weight,
                                    int top, const T* __restrict__ shared, long long shared_stride,
-                                   const float* __restrict__ logit, long long logit_stride, float* __restrict__ res,
-                                   const T* __restrict__ w, T* __restrict__ y, int H, float eps) {
+                                   const float* __restrict__ logit, long long logit_stride, const T* __restrict__ gate,
+                                   long long gate_stride, const T* __restrict__ post, float* __restrict__ res,
+                                   const T* __restrict__ w, float scale, T* __restrict__ y, int H, float eps, bool vec) {
   extern __shared__ float row[];
   __shared__ float sh[32], wk[MR_MAX_TOP];
   __shared__ int from[MR_MAX_TOP];
@@ -204,13 +219,13 @@ __global__ void moe_combine_kernel(const T* __restrict__ out, const int* __restr
   __syncthreads();
   const float g = shared ? (logit ? sigmoid_f(logit[t * logit_stride]) : 1.f) : 0.f;
   const T* s = shared ? shared + t * shared_stride : nullptr;
+  const T* gt = gate ? gate + t * gate_stride : nullptr;
   float* r = res + t * H;
   float ss = 0.f;
-  const bool vec = (H & 7) == 0 && (shared_stride & 7) == 0;
   if (vec) {
     for (int v = threadIdx.x; v < (H >> 3); v += blockDim.x) {
-      float a[8], f[8];
-      ld8(r + v * 8, a);
+      float a[8] = {}, f[8];
+      if (!post) ld8(r + v * 8, a);
       if (s) {
         ld8(s + v * 8, f);
 #pragma unroll
@@ -221,21 +236,29 @@ __global__ void moe_combine_kernel(const T* __restrict__ out, const int* __restr
 #pragma unroll
         for (int i = 0; i < 8; ++i) a[i] = fmaf(f[i], wk[k], a[i]);
       }
-      st8(r + v * 8, a);
+      if (gt) {
+        ld8(gt + v * 8, f);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) a[i] *= sigmoid_t<T>(f[i]);
+      }
+      if (!post) st8(r + v * 8, a);
       st8(row + v * 8, a);
 #pragma unroll
       for (int i = 0; i < 8; ++i) ss += a[i] * a[i];
     }
   } else {
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
-      float a = r[i];
+      float a = post ? 0.f : r[i];
       if (s) a = fmaf(to_f<T>(s[i]), g, a);
       for (int k = 0; k < top; ++k) a = fmaf(to_f<T>(out[(long long)from[k] * H + i]), wk[k], a);
-      r[i] = row[i] = a;
+      if (gt) a *= sigmoid_t<T>(to_f<T>(gt[i]));
+      row[i] = a;
+      if (!post) r[i] = a;
       ss += a * a;
     }
   }
-  norm_row_out(row, ss, w, y + t * H, H, eps, vec, sh);
+  if (post) norm_row_add(row, ss, r, post, w, scale, y + t * H, H, eps, vec, sh);
+  else norm_row_out(row, ss, w, y + t * H, H, eps, vec, sh);
 }
 
 }  // namespace vb
@@ -245,15 +268,15 @@ typedef __nv_bfloat16 bf16;
 
 // logits fp32 [T, stride], the first E of a row; idx, weight, dest [T, top]; blk_expert [nblk], nblk * 128 rows being enough for
 // every expert's share rounded up to 128; counters [E + 1], zero before and after.
-extern "C" int vb_moe_route(const float* logits, long long stride, int T, int E, int top, int softmax, int renormalize, int* idx,
-                            float* weight, int* dest, int* blk_expert, int nblk, int* counters, cudaStream_t stream) {
+extern "C" int vb_moe_route(const float* logits, long long stride, int T, int E, int top, int softmax, int renormalize,
+                            const float* correction, int* idx, float* weight, int* dest, int* blk_expert, int nblk, int* counters, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (E <= 0 || E > MR_MAX_E || top <= 0 || top > MR_MAX_TOP || top > E ||
       (long long)nblk * MR_BLK + MR_BLK <= (long long)T * top + (long long)min(E, T * top) * (MR_BLK - 1))
     return -3;
   const bool small = T <= 32;
   const int per = small ? T : (T <= 4096 ? 8 : 64);
-  MoeRouteParams p{logits, stride, T, E, top, softmax, renormalize, per, nblk, idx, dest, blk_expert, weight, counters};
+  MoeRouteParams p{logits, correction, stride, T, E, top, softmax, renormalize, per, nblk, idx, dest, blk_expert, weight, counters};
   const dim3 g((T + per - 1) / per), b(small ? (T + 3) / 4 * 128 : 256);
 #define VB_MR(NV) e = vb_launch_pdl(moe_route_kernel<NV>, g, b, 0, stream, 1, p)
   cudaError_t e;
@@ -282,13 +305,17 @@ extern "C" int vb_moe_gather(const void* x, long long stride, const int* dest, c
                         scale));
 }
 
-// weight null: the rows of out are added as they are. shared null: none; logit null: its factor is one.
+// weight null: the rows of out are added as they are. shared null: none; logit null: its factor is one. post, gate, scale: see
+// moe_combine_kernel.
 extern "C" int vb_moe_sum(const void* out, const int* dest, const float* weight, int top, const void* shared,
-                              long long shared_stride, const float* logit, long long logit_stride, float* res, const void* w,
-                              void* y, int T, int H, float eps, int f32, cudaStream_t stream) {
+                          long long shared_stride, const float* logit, long long logit_stride, const void* gate,
+                          long long gate_stride, const void* post, float* res, const void* w, float scale, void* y, int T, int H,
+                          float eps, int f32, cudaStream_t stream) {
   if (T <= 0) return 0;
   const size_t smem = (size_t)H * 4;
-  if (smem > 160 * 1024 || top <= 0 || top > MR_MAX_TOP) return -3;
+  if (smem > 160 * 1024 || top <= 0 || top > MR_MAX_TOP || (gate && !post)) return -3;
+  const bool vec = ((H | shared_stride | gate_stride) & 7) == 0 &&
+                   ((reinterpret_cast<uintptr_t>(shared) | reinterpret_cast<uintptr_t>(gate)) & 15) == 0;
   static bool attr = false;
   if (!attr) {
     VB_CUDA_CHECK(cudaFuncSetAttribute(moe_combine_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024));
@@ -298,7 +325,9 @@ extern "C" int vb_moe_sum(const void* out, const int* dest, const float* weight,
   const dim3 g(T), b(row_threads(H));
   if (f32)
     VB_DONE(vb_launch_pdl(moe_combine_kernel<float>, g, b, smem, stream, 1, (const float*)out, dest, weight, top,
-                          (const float*)shared, shared_stride, logit, logit_stride, res, (const float*)w, (float*)y, H, eps));
+                          (const float*)shared, shared_stride, logit, logit_stride, (const float*)gate, gate_stride,
+                          (const float*)post, res, (const float*)w, scale, (float*)y, H, eps, vec));
   VB_DONE(vb_launch_pdl(moe_combine_kernel<bf16>, g, b, smem, stream, 1, (const bf16*)out, dest, weight, top, (const bf16*)shared,
-                        shared_stride, logit, logit_stride, res, (const bf16*)w, (bf16*)y, H, eps));
+                        shared_stride, logit, logit_stride, (const bf16*)gate, gate_stride, (const bf16*)post, res,
+                        (const bf16*)w, scale, (bf16*)y, H, eps, vec));
 }

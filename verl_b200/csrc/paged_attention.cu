@@ -207,10 +207,10 @@ __global__ void decode_merge_kernel(const float* __restrict__ o_part, const floa
   out[(long long)b * out_stride + (long long)hq * D + d] = __float2bfloat16(l > 0.f ? o / l : 0.f);
 }
 
-// The same for any head size, times the sigmoid of a gate [B, Hq * D] (or null). Dynamic shared memory: num_splits floats.
+// The same for any head size, times the sigmoid of a gate [B, Hq * D] (gate_w 1: [B, Hq]) or null. Dynamic shared memory: num_splits floats.
 __global__ void decode_merge_any_kernel(const float* __restrict__ o_part, const float* __restrict__ ml_part, int Hq, int D,
                                         int num_splits, __nv_bfloat16* __restrict__ out, long long out_stride,
-                                        const __nv_bfloat16* __restrict__ gate, long long gate_stride) {
+                                        const __nv_bfloat16* __restrict__ gate, long long gate_stride, int gate_w) {
   extern __shared__ float weight[];  // of each split's partial result
   const int b = blockIdx.x, hq = blockIdx.y;
   const long long base = ((long long)b * Hq + hq) * num_splits;
@@ -244,7 +244,8 @@ __global__ void decode_merge_any_kernel(const float* __restrict__ o_part, const 
     for (int e = 0; e < step; ++e) {
       float x = o[e];
       if (gate)
-        x = __fdividef(x, 1.f + __expf(-__bfloat162float(gate[(long long)b * gate_stride + (long long)hq * D + d + e])));
+        x = __fdividef(x, 1.f + __expf(-__bfloat162float(
+                                      gate[(long long)b * gate_stride + (gate_w == 1 ? hq : (long long)hq * D + d + e)])));
       out[(long long)b * out_stride + (long long)hq * D + d + e] = __float2bfloat16(x);
     }
   }
@@ -297,9 +298,9 @@ int vb_decode_merge_128(const float* o_part, const float* ml_part, int B, int Hq
 }
 
 int vb_decode_merge(const float* o_part, const float* ml_part, int B, int Hq, int D, int num_splits, void* out,
-                    long long out_stride, const void* gate, long long gate_stride, cudaStream_t stream) {
+                    long long out_stride, const void* gate, long long gate_stride, int gate_w, cudaStream_t stream) {
   decode_merge_any_kernel<<<dim3(B, Hq), D <= 256 ? 64 : 128, num_splits * sizeof(float), stream>>>(o_part, ml_part, Hq, D, num_splits, (__nv_bfloat16*)out,
-                                                                          out_stride, (const __nv_bfloat16*)gate, gate_stride);
+                                                                          out_stride, (const __nv_bfloat16*)gate, gate_stride, gate_w);
   return (int)cudaGetLastError();
 }
 

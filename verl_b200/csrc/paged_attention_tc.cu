@@ -64,8 +64,10 @@ struct DecodeTcParams {
   const float* bias;  // [Hq, bias_len] or null
   float softcap;
   const float* sink;          // [Hq] or null
-  const __nv_bfloat16* gate;  // [B, Hq * Dv] or null
+  const __nv_bfloat16* gate;  // [B, Hq * Dv] (gate_w 1: [B, Hq]) or null
   long long gate_stride;
+  int gate_w;
+  const float *shift, *r1, *r2;  // [Hq]; SIG: shift, and r1, r2 or null
 };
 
 // First key that the query at position seq_len - 1 sees, kept ones apart.
@@ -432,7 +434,9 @@ __device__ __forceinline__ TcItem tc_item(const DecodeTcParams& p, int item) {
   return it;
 }
 
-template <bool EXT>
+// SIG (with EXT): no softmax, a key weighs sigmoid(score - r1 ln(1 + r2 distance) + shift). The splits' results are sums then:
+// they get the reference 0 and the denominators 1, 0, 0, ..., with which the merge adds them up.
+template <bool EXT, bool SIG = false>
 __global__ void __launch_bounds__(TC_THREADS, 2)
 paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                                const DecodeTcParams p, const int num_items) {
@@ -651,7 +655,10 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
         l_run[g] = 0.f;
         o_acc[g] = 0.f;
         // the sink is a key without a value: it counts once, in the first split
-        if (EXT && p.sink != nullptr && g < G && it.split == 0) {
+        if (SIG) {
+          m_run[g] = 0.f;
+          l_run[g] = it.split == 0 ? 1.f : 0.f;
+        } else if (EXT && p.sink != nullptr && g < G && it.split == 0) {
           m_run[g] = p.sink[it.h * G + g];
           l_run[g] = 1.f;
         }
@@ -679,6 +686,29 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
         const int key = it.range.at(it.c_begin + c) * TC_CHUNK + tid;
         const int dist = it.seq_len - 1 - key;
         const bool valid = dist >= 0 && (!EXT || key >= first || (p.window > 0 && key < p.keep_first));
+        uint8_t* pbuf = p_s + i * P_BYTES;
+        if constexpr (SIG) {
+          const float d = (float)max(dist, 0);
+#pragma unroll
+          for (int g = 0; g < NG; ++g) {
+            alpha[g] = 1.f;
+            if (g < G) {
+              const int hq = it.h * G + g;
+              float x = fmaf(__uint_as_float(sr[g]), p.scale, __ldg(p.shift + hq));
+              if (p.r1 != nullptr) x -= __ldg(p.r1 + hq) * __logf(fmaf(__ldg(p.r2 + hq), d, 1.f));
+              const float pv = valid ? __fdividef(1.f, 1.f + __expf(fminf(-x, 60.f))) : 0.f;
+              const __nv_bfloat16 ph = __float2bfloat16(pv);
+              *reinterpret_cast<__nv_bfloat16*>(pbuf + sw128_off(g, tid, TC_NH)) = ph;
+              *reinterpret_cast<__nv_bfloat16*>(pbuf + sw128_off(G + g, tid, TC_NH)) =
+                  __float2bfloat16(pv - __bfloat162float(ph));
+            }
+          }
+          fence_proxy_async_smem();
+          tc_fence_before();
+          __syncwarp();
+          if (lane == 0) mbar_arrive(&p_ready[i]);
+          return;
+        }
         const float* brow = EXT && p.bias != nullptr
                                 ? p.bias + (long long)it.h * G * p.bias_len + max(min(dist, p.bias_len - 1), 0)
                                 : nullptr;
@@ -696,7 +726,6 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
           }
         }
         bar_sync_128();
-        uint8_t* pbuf = p_s + i * P_BYTES;
 #pragma unroll
         for (int g = 0; g < NG; ++g) {
           alpha[g] = 1.f;
@@ -768,7 +797,8 @@ paged_decode_tc_persist_kernel(const __grid_constant__ CUtensorMap tmK, const __
             if (p.num_splits == 1) {
               float x = l_run[g] > 0.f ? o_acc[g] / l_run[g] : 0.f;
               if (EXT && p.gate != nullptr)
-                x = __fdividef(x, 1.f + __expf(-__bfloat162float(p.gate[(long long)it.b * p.gate_stride + hq * Dv + d])));
+                x = __fdividef(x, 1.f + __expf(-__bfloat162float(
+                                              p.gate[(long long)it.b * p.gate_stride + (p.gate_w == 1 ? hq : hq * Dv + d)])));
               p.out[(long long)it.b * p.out_stride + (long long)hq * Dv + d] = __float2bfloat16(x);
             } else {
               const long long base = ((long long)it.b * p.Hq + hq) * p.num_splits + it.split;
@@ -866,7 +896,7 @@ extern "C" int vb_paged_decode_tc(const void* q, long long q_stride, const void*
 }
 
 int vb_decode_merge(const float* o_part, const float* ml_part, int B, int Hq, int D, int num_splits, void* out,
-                    long long out_stride, const void* gate, long long gate_stride, cudaStream_t stream);
+                    long long out_stride, const void* gate, long long gate_stride, int gate_w, cudaStream_t stream);
 
 // Returns 1 if vb_paged_decode_window supports this configuration.
 extern "C" int vb_paged_decode_window_supported(int Hq, int Hk, int D, int Dv, int block_size) {
@@ -879,18 +909,22 @@ extern "C" int vb_paged_decode_window_supported(int Hq, int Hk, int D, int Dv, i
 //   chunk > 0: key j is visible when j / chunk == (seq_len - 1) / chunk (not together with a window)
 //   bias [Hq, bias_len] fp32 or null: bias[h][min(seq_len - 1 - j, bias_len - 1)] is added to the scaled score
 //   softcap > 0 (without bias): scores become softcap * tanh(score / softcap)
-//   sink [Hq] fp32 or null: exp(sink[h]) joins the denominator; gate [B, Hq * Dv] or null: its sigmoid multiplies the result
+//   sink [Hq] fp32 or null: exp(sink[h]) joins the denominator
+//   shift [Hq] fp32 (without bias, softcap and sink): sigmoid weights; r1, r2 [Hq] or null: r1 ln(1 + r2 (seq_len - 1 - j)) off
+//   gate [B, Hq * Dv] (gate_w 1: [B, Hq]) or null: its sigmoid multiplies the result
 // work: fp32 scratch of B * Hq * num_splits * (Dv + 2) floats (unused when num_splits == 1).
 extern "C" int vb_paged_decode_window(const void* q, long long q_stride, const void* kc, const void* vc, int num_blocks,
                                       const int* block_table, int max_blocks, const int* seq_lens, int B, int Hq, int Hk,
                                       int D, int Dv, int block_size, float scale, int window, int keep_first,
                                       int chunk, const float* bias, int bias_len, float softcap, const float* sink,
-                                      const void* gate, long long gate_stride, int num_splits, void* out,
-                                      long long out_stride, float* work, int* status, cudaStream_t stream) {
+                                      const float* shift, const float* r1, const float* r2, const void* gate,
+                                      long long gate_stride, int gate_w, int num_splits, void* out, long long out_stride,
+                                      float* work, int* status, cudaStream_t stream) {
   if (B <= 0) return 0;
   if (!vb_paged_decode_window_supported(Hq, Hk, D, Dv, block_size) || (q_stride & 7) != 0 ||
       (reinterpret_cast<uintptr_t>(q) & 15) != 0 || num_splits < 1 || (num_splits > 1 && work == nullptr) ||
-      (bias != nullptr && bias_len <= 0) || (window > 0 && chunk > 0) || (softcap > 0.f && bias != nullptr))
+      (bias != nullptr && bias_len <= 0) || (window > 0 && chunk > 0) || (softcap > 0.f && bias != nullptr) ||
+      (shift && (bias || sink || softcap > 0.f)) || (r1 && (!shift || !r2)))
     return -3;
   CUtensorMap tmK, tmV;
   const uint64_t rows = (uint64_t)num_blocks * Hk * block_size;
@@ -902,6 +936,8 @@ extern "C" int vb_paged_decode_window(const void* q, long long q_stride, const v
   if (!attr_set) {
     VB_CUDA_CHECK(cudaFuncSetAttribute(paged_decode_tc_persist_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                        TCP_SMEM));
+    VB_CUDA_CHECK(cudaFuncSetAttribute(paged_decode_tc_persist_kernel<true, true>,
+                                       cudaFuncAttributeMaxDynamicSharedMemorySize, TCP_SMEM));
     attr_set = true;
   }
   DecodeTcParams p{};
@@ -922,11 +958,14 @@ extern "C" int vb_paged_decode_window(const void* q, long long q_stride, const v
   p.chunk = chunk; p.softcap = softcap; p.sink = sink;
   p.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
   p.gate_stride = gate_stride;
+  p.gate_w = gate_w;
+  p.shift = shift; p.r1 = r1; p.r2 = r2;
   const int items = B * Hk * num_splits, slots = 2 * vb_num_sms();
-  rc = (int)vb_launch_pdl(paged_decode_tc_persist_kernel<true>, dim3(items < slots ? items : slots), dim3(TC_THREADS),
-                          TCP_SMEM, stream, 1, tmK, tmV, p, items);
+  const dim3 grid(items < slots ? items : slots), block(TC_THREADS);
+  rc = (int)(shift ? vb_launch_pdl(paged_decode_tc_persist_kernel<true, true>, grid, block, TCP_SMEM, stream, 1, tmK, tmV, p, items)
+                   : vb_launch_pdl(paged_decode_tc_persist_kernel<true>, grid, block, TCP_SMEM, stream, 1, tmK, tmV, p, items));
   vb_count_launch(num_splits > 1 ? 2 : 1);
   if (rc == 0) rc = (int)cudaGetLastError();
   if (rc || num_splits == 1) return rc;
-  return vb_decode_merge(p.o_part, p.ml_part, B, Hq, Dv, num_splits, out, out_stride, gate, gate_stride, stream);
+  return vb_decode_merge(p.o_part, p.ml_part, B, Hq, Dv, num_splits, out, out_stride, gate, gate_stride, gate_w, stream);
 }

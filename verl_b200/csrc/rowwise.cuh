@@ -75,6 +75,58 @@ __device__ __forceinline__ void norm_row_out(const float* row, float ss, const T
   }
 }
 
+// The row in shared memory, of which every thread has stored the elements it reads here, with the sum of squares ss of this
+// thread's: res += row / sqrt(mean(row^2) + eps) * w; out = res, or with fw: res / sqrt(mean(res^2) + eps) * fw * fscale.
+template <typename T>
+__device__ __forceinline__ void norm_row_add(float* row, float ss, float* __restrict__ res, const T* __restrict__ w,
+                                             const T* __restrict__ fw, float fscale, T* __restrict__ out, int H, float eps,
+                                             bool vec, float* sh) {
+  const float inv = 1.f / sqrtf(block_sum_all(ss, sh) / (float)H + eps);
+  ss = 0.f;
+  if (vec) {
+    for (int v = threadIdx.x; v < (H >> 3); v += blockDim.x) {
+      float f[8], g[8], x[8];
+      ld8(res + v * 8, x);
+      ld8(row + v * 8, f);
+      ld8(w + v * 8, g);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        x[i] += f[i] * inv * g[i];
+        ss += x[i] * x[i];
+      }
+      st8(res + v * 8, x);
+      if (fw) st8(row + v * 8, x); else st8(out + v * 8, x);
+    }
+  } else {
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+      const float x = res[i] + row[i] * inv * to_f<T>(w[i]);
+      res[i] = x;
+      ss += x * x;
+      if (fw) row[i] = x; else out[i] = from_f<T>(x);
+    }
+  }
+  if (fw == nullptr) return;
+  const float fi = fscale / sqrtf(block_sum_all(ss, sh) / (float)H + eps);
+  if (vec) {
+    for (int v = threadIdx.x; v < (H >> 3); v += blockDim.x) {
+      float f[8], g[8];
+      ld8(row + v * 8, f);
+      ld8(fw + v * 8, g);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) f[i] = f[i] * fi * g[i];
+      st8(out + v * 8, f);
+    }
+  } else {
+    for (int i = threadIdx.x; i < H; i += blockDim.x) out[i] = from_f<T>(row[i] * fi * to_f<T>(fw[i]));
+  }
+}
+
+// 1 / (1 + e^-z) for the activation type: errors far below a bf16 ulp are let through.
+template <typename T>
+__device__ __forceinline__ float sigmoid_t(float z) {
+  return sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-z)) : 1.f / (1.f + expf(-z));
+}
+
 // gelu with tanh: 0.5 g (1 + tanh(z)) = g sigmoid(2 z), z = sqrt(2 / pi) (g + 0.044715 g^3). FAST: error far below a bf16 ulp.
 template <bool FAST>
 __device__ __forceinline__ float gelu_tanh(float g) {

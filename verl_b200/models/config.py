@@ -10,8 +10,8 @@ from dataclasses import asdict, dataclass, field
 from pathlib import Path
 from typing import Any
 
-from .layer_specs import (DESIGNS, AttentionSpec, DeltaSpec, Design, GluSpec, LatentSpec, LayerSpec, LruSpec, MoeSpec,
-                          RotarySpec)
+from .layer_specs import (DESIGNS, AttentionSpec, DeltaSpec, Design, GlaSpec, GluSpec, LatentSpec, LayerSpec, LruSpec, MlpSpec,
+                          MoeSpec, RotarySpec, weight_owner)
 
 _ARCH_TO_TYPE = {
     "LlamaForCausalLM": "llama",
@@ -33,7 +33,7 @@ _TYPE_TO_ARCH = {"llama": "LlamaForCausalLM", "qwen2": "Qwen2ForCausalLM", "qwen
                  "qwen2_5_vl": "Qwen2_5_VLForConditionalGeneration", "apertus": "ApertusForCausalLM",
                  "qwen3_vl": "Qwen3VLForConditionalGeneration", "qwen3_vl_moe": "Qwen3VLMoeForConditionalGeneration"}
 # designs whose config.json lists its layers one by one (``architecture`` instead of ``architectures``)
-_LAYER_LIST_ARCHS = {"Fuganex": "fuganex", "Padodra": "padodra", "Golonex": "golonex"}
+_LAYER_LIST_ARCHS = {"Fuganex": "fuganex", "Padodra": "padodra", "Golonex": "golonex", "Malinex": "malinex"}
 _VL_TYPES = ("qwen2_vl", "qwen2_5_vl", "qwen3_vl", "qwen3_vl_moe")
 
 
@@ -78,6 +78,8 @@ class ModelConfig:
         self.layer_specs = tuple(self.layer_specs)
         if self.layer_specs:
             self.num_hidden_layers = len(self.layer_specs)
+            for i in range(len(self.layer_specs)):
+                weight_owner(self.layer_specs, i)
             self.tie_word_embeddings = self.design.tied
         if self.head_dim is None:
             self.head_dim = self.hidden_size // self.num_attention_heads
@@ -105,7 +107,12 @@ class ModelConfig:
     @property
     def has_recurrent_state(self) -> bool:
         """Some layer carries a state per sequence that pages cannot share."""
-        return any(s.kind in ("delta", "rglru") for s in self.layer_specs)
+        return any(s.kind in ("delta", "gla", "rglru") for s in self.layer_specs)
+
+    @property
+    def has_position_table(self) -> bool:
+        """Positions are rows of a learned table: no sequence is longer than ``max_position_embeddings``."""
+        return self.is_layer_list and self.design.embedding == "positions"
 
     @property
     def mlp_gated(self) -> bool:
@@ -142,7 +149,9 @@ class ModelConfig:
     def num_parameters(self, include_embedding: bool = True) -> int:
         H, L = self.hidden_size, self.num_hidden_layers
         if self.is_layer_list:
-            total = H + sum(s.num_parameters(H) for s in self.layer_specs)
+            total = H + sum(s.num_parameters(H, self.design) for s in self.layer_specs)
+            if self.has_position_table and include_embedding:
+                total += self.max_position_embeddings * H
             if self.design.embedding == "norm":
                 total += H
             if self.side_dim:
@@ -232,6 +241,10 @@ class ModelConfig:
         if design.embedding == "scale":
             known.append("embedding")
             kw["embedding_scale"] = float(d["embedding"]["scale"])
+        elif design.embedding == "positions":
+            known.append("max_positions")
+            if d.get("max_positions") is not None:
+                kw["max_position_embeddings"] = int(d["max_positions"])
         if design.logit_scale:
             known.append("logit_scale")
             kw["logit_scale"] = float(d.get("logit_scale", 1.0))
@@ -254,6 +267,8 @@ class ModelConfig:
              "layers": [s.to_dict() for s in self.layer_specs], "norm": {"eps": self.rms_norm_eps}, **self.extra}
         if self.design.embedding == "scale":
             d["embedding"] = {"scale": self.embedding_scale}
+        elif self.has_position_table:
+            d["max_positions"] = self.max_position_embeddings
         if self.design.logit_scale:
             d["logit_scale"] = self.logit_scale
         if self.logit_softcap:

@@ -11,12 +11,12 @@ from __future__ import annotations
 
 import json
 from pathlib import Path
-from typing import Iterable, Iterator
+from typing import Iterable, Iterator, Optional
 
 import torch
 
 from .config import ModelConfig
-from .layer_specs import MoeSpec
+from .layer_specs import MlpSpec, MoeSpec, weight_owner
 
 
 _VIS_HF_TO_NATIVE = (("attn.qkv.", "qkv."), ("attn.proj.", "proj."), ("mlp.fc1.", "fc1."), ("mlp.fc2.", "fc2."),
@@ -209,22 +209,35 @@ def native_to_hf_items(cfg: ModelConfig, named: Iterable[tuple[str, torch.Tensor
 # ------------------------------------------------------------- layer-list checkpoints (models/hybrid.py)
 # native name -> checkpoint name of the tensors that are stored alike
 _LIST_TOP = {"embed_tokens.weight": "embed", "norm.weight": "final.norm", "lm_head.weight": "head",
-             "embed_norm.weight": "embed.norm", "side_embed.weight": "side.embed"}
+             "embed_norm.weight": "embed.norm", "side_embed.weight": "side.embed", "pos_embed.weight": "pos"}
 _LIST_PLAIN = {"norm1.weight": "norm1", "norm2.weight": "norm2", "mlp.down_proj.weight": "mlp.down",
                "mixer.o_proj.weight": "mix.o", "mixer.q_norm.weight": "mix.q.norm", "mixer.k_norm.weight": "mix.k.norm",
                "mixer.rel": "mix.rel", "mixer.A_log": "mix.A_log", "mixer.dt_bias": "mix.dt_bias",
                "mixer.norm.weight": "mix.norm", "mixer.sink": "mix.sink", "mixer.kv_norm.weight": "mix.dkv.norm",
                "mixer.q_latent_norm.weight": "mix.dq.norm", "mixer.conv_w": "mix.conv", "mixer.conv_b": "mix.conv.b",
                "mixer.lam": "mix.lam", "mlp.shared.down_proj.weight": "mlp.shared.down",
-               "side.gate_proj.weight": "side.gate", "side.out_proj.weight": "side.proj", "side.norm.weight": "side.norm"}
+               "side.gate_proj.weight": "side.gate", "side.out_proj.weight": "side.proj", "side.norm.weight": "side.norm",
+               "norm1b.weight": "norm1b", "norm2b.weight": "norm2b", "mixer.r1": "mix.r1", "mixer.r2": "mix.r2",
+               "mixer.shift": "mix.pb", "mixer.decay_w": "mix.a2", "mixer.decay_b": "mix.a2.b",
+               "mlp.correction": "mlp.correction"}
+# of the plain ones: what a layer without a feed-forward leaves out
+_LIST_SECOND = ("norm2.weight", "norm2b.weight")
 
 
-def _list_fused(spec) -> dict[str, list[tuple[str, int]]]:
-    """Native fused matrices of a layer: name -> [(checkpoint name, rows), ...] in row order."""
+def _list_fused(spec, gate: int = 0) -> dict[str, list[tuple[Optional[str], int]]]:
+    """Native fused matrices of a layer: name -> [(checkpoint name, rows), ...] in row order; no name: rows of zeros. ``gate``:
+    rows of the residual gates (0: none), behind the other rows of a sublayer's first matrix."""
     m = spec.mixer
     if spec.kind == "attention":
         out = {"mixer.qkv_proj.weight": [("mix.q", m.q_size), ("mix.k", m.k_size)]
-               + ([] if m.key_values else [("mix.v", m.v_size)]) + ([("mix.g", m.out_size)] if m.gate else [])}
+               + ([] if m.key_values else [("mix.v", m.v_size)]) + ([("mix.g", m.gate_size)] if m.gate else [])}
+        if m.qkv_bias:
+            out["mixer.qkv_proj.bias"] = ([("mix.q.b", m.q_size), ("mix.k.b", m.k_size)]
+                                          + ([] if m.key_values else [("mix.v.b", m.v_size)])
+                                          + ([(None, m.gate_size)] if m.gate else []))
+    elif spec.kind == "gla":
+        out = {"mixer.in_proj.weight": [("mix.q", m.qk_size), ("mix.k", m.qk_size), ("mix.v", m.out_size), ("mix.g", m.out_size),
+                                        ("mix.a1", m.rank)]}
     elif spec.kind == "latent_attention":
         out = {"mixer.in_proj.weight": [("mix.dq" if m.q_rank else "mix.q", m.q_in), ("mix.dkv", m.latent_size)]
                + ([("mix.g", m.gate_size)] if m.gate else []),
@@ -241,19 +254,49 @@ def _list_fused(spec) -> dict[str, list[tuple[str, int]]]:
         out = {"mixer.in_proj.weight": [("mix.q", qk), ("mix.k", qk), ("mix.v", v), ("mix.g", v), ("mix.b", m.heads),
                                         ("mix.a", m.heads)],
                "mixer.conv": [("mix.q.conv", qk), ("mix.k.conv", qk), ("mix.v.conv", v)]}
-    if isinstance(spec.mlp, MoeSpec):
-        out["mlp.router_proj.weight"] = [("mlp.router", spec.mlp.experts)]
-        if spec.mlp.shared_ff:
+    if gate:
+        _append_gate(out, next(n[: -len(".weight")] for n in out if n.endswith(("qkv_proj.weight", "in_proj.weight"))), "rg1", gate)
+    mlp = spec.mlp
+    if isinstance(mlp, MoeSpec):
+        out["mlp.router_proj.weight"] = [("mlp.router", mlp.experts)]
+        if mlp.shared_ff and mlp.shared_gate:
             out["mlp.router_proj.weight"].append(("mlp.shared.sg", 1))
-            out["mlp.shared.gate_up_proj.weight"] = [(f"mlp.shared.{x}", spec.mlp.shared_ff) for x in ("gate", "up")]
-    elif spec.mlp is not None:
-        out["mlp.gate_up_proj.weight"] = [("mlp.gate", spec.mlp.ff), ("mlp.up", spec.mlp.ff)]
+    unit, at = (mlp.shared, "mlp.shared") if isinstance(mlp, MoeSpec) else (mlp, "mlp")
+    first = None
+    if isinstance(unit, MlpSpec):
+        first = f"{at}.up_proj"
+        out[first + ".weight"] = [(f"{at}.up", unit.ff)]
+    elif unit is not None:
+        first = f"{at}.gate_up_proj"
+        out[first + ".weight"] = [(f"{at}.gate", unit.ff), (f"{at}.up", unit.ff)]
+    if gate and mlp is not None:
+        if first is None:  # a mixture without a shared unit
+            first = "mlp.gate_proj"
+            out[first + ".weight"] = []
+        _append_gate(out, first, "rg2", gate)
     return out
+
+
+def _append_gate(fused: dict, matrix: str, name: str, rows: int) -> None:
+    """The rows of a residual gate and their bias behind a fused matrix, from a multiple of 8 on."""
+    own = sum(n for _, n in fused[matrix + ".weight"])
+    bias = fused.setdefault(matrix + ".bias", [(None, own)] if own else [])
+    for parts, part in ((fused[matrix + ".weight"], name), (bias, name + ".b")):
+        if own % 8:
+            parts.append((None, 8 - own % 8))
+        parts.append((part, rows))
 
 
 def _list_experts(spec) -> dict[str, list[str]]:
     """Native stacks of expert matrices: name -> the checkpoint names of one expert's rows (``mlp.e<k>.`` in front)."""
-    return {"mlp.experts_gate_up": ["gate", "up"], "mlp.experts_down": ["down"]} if isinstance(spec.mlp, MoeSpec) else {}
+    if not isinstance(spec.mlp, MoeSpec):
+        return {}
+    first = {"mlp.experts_gate_up": ["gate", "up"]} if spec.mlp.gated else {"mlp.experts_up": ["up"]}
+    return {**first, "mlp.experts_down": ["down"]}
+
+
+def _gate_rows(cfg: ModelConfig) -> int:
+    return cfg.hidden_size if cfg.design.residual_gate else 0
 
 
 def _layer_list_to_native(cfg: ModelConfig, sd: dict[str, torch.Tensor]) -> dict[str, torch.Tensor]:
@@ -261,15 +304,18 @@ def _layer_list_to_native(cfg: ModelConfig, sd: dict[str, torch.Tensor]) -> dict
     if "embed_tokens.weight" not in out or "norm.weight" not in out:
         raise KeyError("the checkpoint has no embedding or no final norm")
     for i, spec in enumerate(cfg.layer_specs):
-        fused = _list_fused(spec)
+        if spec.weights_of is not None:
+            continue
+        fused = _list_fused(spec, _gate_rows(cfg))
         for n, parts in fused.items():
             ts = []
             for c, rows in parts:
-                t = sd[f"l{i}.{c}"]
-                if t.shape[0] != rows:
+                t = None if c is None else sd[f"l{i}.{c}"]
+                if t is not None and t.shape[0] != rows:
                     raise ValueError(f"l{i}.{c}: {t.shape[0]} rows, the configuration says {rows}")
-                ts.append(t)
-            w = torch.cat(ts, 0)
+                ts.append((t, rows))
+            like = next(t for t, _ in ts if t is not None)
+            w = torch.cat([like.new_zeros(rows, *like.shape[1:]) if t is None else t for t, rows in ts], 0)
             if n.endswith(("_proj.weight", "_proj.bias")) and w.shape[0] % 8:  # padded with zero rows
                 w = torch.cat([w, w.new_zeros(8 - w.shape[0] % 8, *w.shape[1:])], 0)
             out[f"layers.{i}.{n}"] = w
@@ -277,7 +323,7 @@ def _layer_list_to_native(cfg: ModelConfig, sd: dict[str, torch.Tensor]) -> dict
             out[f"layers.{i}.{n}"] = torch.stack([torch.cat([sd[f"l{i}.mlp.e{e}.{c}"] for c in parts], 0)
                                                   for e in range(spec.mlp.experts)])
         for n, c in _LIST_PLAIN.items():
-            if f"l{i}.{c}" in sd and (spec.mlp is not None or n != "norm2.weight"):
+            if f"l{i}.{c}" in sd and (spec.mlp is not None or n not in _LIST_SECOND):
                 out[f"layers.{i}.{n}"] = sd[f"l{i}.{c}"]
     return out
 
@@ -297,16 +343,26 @@ def _layer_list_to_ckpt(cfg: ModelConfig, name: str, t: torch.Tensor) -> Iterato
                 yield f"l{i}.mlp.e{e}.{c}", part
         return
     lo = 0
-    for c, rows in _list_fused(cfg.layer_specs[int(i)])[rest]:
-        yield f"l{i}.{c}", t[lo : lo + rows]
+    for c, rows in _list_fused(cfg.layer_specs[int(i)], _gate_rows(cfg))[rest]:
+        if c is not None:
+            yield f"l{i}.{c}", t[lo : lo + rows]
         lo += rows
 
 
 def _sizes_from_tensors(cfg: ModelConfig, sd: dict[str, torch.Tensor]) -> None:
-    """Sizes that only the tensors' shapes give: the rows of the distance-bias tables."""
-    cfg.layer_specs = tuple(
-        s.with_bias_rows(sd[f"l{i}.mix.rel"].shape[0] if f"l{i}.mix.rel" in sd else 0) if s.kind == "attention" else s
-        for i, s in enumerate(cfg.layer_specs))
+    """Sizes that only the tensors' shapes give: the rows of the distance-bias tables and of the position table, the ranks of
+    decays."""
+    specs = []
+    for i, s in enumerate(cfg.layer_specs):
+        j = weight_owner(cfg.layer_specs, i)
+        if s.kind == "attention":
+            s = s.with_sizes(bias_rows=sd[f"l{j}.mix.rel"].shape[0] if f"l{j}.mix.rel" in sd else 0)
+        elif s.kind == "gla":
+            s = s.with_sizes(rank=sd[f"l{j}.mix.a1"].shape[0])
+        specs.append(s)
+    cfg.layer_specs = tuple(specs)
+    if cfg.has_position_table:
+        cfg.max_position_embeddings = sd["pos"].shape[0]
 
 
 def _vis_native_to_hf(name: str, gated: bool = False) -> str:

@@ -1,6 +1,6 @@
-"""Decoders described layer by layer (``ModelConfig.layer_specs``): every layer has its own mixer, softmax attention over
-the paged KV cache, latent attention over pages of latents, a gated delta rule or a gated linear recurrent unit with
-per-sequence state, and an optional gated feed-forward or mixture of them.
+"""Decoders described layer by layer (``ModelConfig.layer_specs``): every layer has its own mixer, attention over the paged
+KV cache, latent attention over pages of latents, a gated delta rule, gated linear attention or a gated linear recurrent unit
+with per-sequence state, and an optional feed-forward or mixture of them.
 
 Served by the rollout engine like the homogeneous stacks of :mod:`.transformer`; there is no training path. The residual
 stream is fp32 and every norm is fused with the residual add beside it. Designs that norm what a sublayer reads:
@@ -12,6 +12,11 @@ Designs that norm what a sublayer puts out (the last norm + add also computes th
 
     embedding * scale -> [ fused input projection -> mixer -> output projection -> norm1 + add
                            -> gate|up -> GLU -> down -> norm2 + add ] ... -> head
+
+Designs that norm both, with a gate on what a sublayer puts out (its projection is part of the sublayer's first matrix):
+
+    embedding + position -> [ norm1 -> fused input projection -> mixer -> output projection -> gate, norm1b, add + norm2
+                              -> up -> activation -> down -> gate, norm2b, add + next norm ] ... -> head
 
 Layers with an input of their own per token read the stream behind the feed-forward as it is, and their normed output is added
 together with the next layer's norm1 (or the final norm):
@@ -30,7 +35,8 @@ import torch.nn as nn
 
 from .. import ops
 from .config import ModelConfig
-from .layer_specs import AttentionSpec, DeltaSpec, GluSpec, LatentSpec, LayerSpec, LruSpec, MoeSpec, distance_buckets
+from .layer_specs import (AttentionSpec, DeltaSpec, GlaSpec, GluSpec, LatentSpec, LayerSpec, LruSpec, MlpSpec, MoeSpec,
+                          distance_buckets, weight_owner)
 from .transformer import Linear, RMSNormWeight
 
 
@@ -79,7 +85,7 @@ class RaggedBatch:
 
 class StateCache:
     """Cache of a layer-list model: K / V pages per attention layer, pages of latents and rotated keys per latent-attention
-    layer, fp32 state and convolution ring per delta or recurrent-unit layer."""
+    layer, fp32 state (and a convolution ring where the layer convolves) per recurrent layer."""
 
     def __init__(self, cfg: ModelConfig, num_blocks: int, block_size: int, num_slots: int, dtype, device):
         self.layers: list[tuple] = []
@@ -92,14 +98,16 @@ class StateCache:
                 self.layers.append((torch.zeros((num_blocks, block_size, ops.latent_width(m.latent_size)), dtype=dtype, device=device),))
             else:
                 channels, state = self._state(spec)
-                self.layers.append((torch.zeros((num_slots, m.conv, channels), dtype=dtype, device=device),
-                                    torch.zeros((num_slots, *state), dtype=torch.float32, device=device)))
+                ring = (torch.zeros((num_slots, m.conv, channels), dtype=dtype, device=device),) if channels else ()
+                self.layers.append((*ring, torch.zeros((num_slots, *state), dtype=torch.float32, device=device)))
 
     @staticmethod
     def _state(spec) -> tuple:
         """Convolved channels and shape of the state of a recurrent layer."""
         m = spec.mixer
-        return (m.width, (m.width,)) if spec.kind == "rglru" else (m.channels, (m.heads, m.vdim, m.dim))
+        if spec.kind == "rglru":
+            return m.width, (m.width,)
+        return 0 if spec.kind == "gla" else m.channels, (m.heads, m.vdim, m.dim)
 
     @staticmethod
     def page_bytes(cfg: ModelConfig, block_size: int, itemsize: int) -> int:
@@ -110,9 +118,9 @@ class StateCache:
     def slot_bytes(cfg: ModelConfig, itemsize: int) -> int:
         total = 0
         for s in cfg.layer_specs:
-            if s.kind in ("delta", "rglru"):
+            if s.kind in ("delta", "gla", "rglru"):
                 channels, state = StateCache._state(s)
-                total += s.mixer.conv * channels * itemsize + 4 * math.prod(state)
+                total += (s.mixer.conv * channels * itemsize if channels else 0) + 4 * math.prod(state)
         return total
 
 
@@ -121,16 +129,45 @@ def rotary_frequencies(module: nn.Module, spec, device) -> None:
     module.register_buffer("rot_freqs", torch.tensor(spec.frequencies(), dtype=torch.float32, device=device), persistent=False)
 
 
-class AttentionMixer(nn.Module):
-    def __init__(self, cfg: ModelConfig, spec: AttentionSpec, dtype, device):
+class Sublayer(nn.Module):
+    """A mixer or feed-forward: its spec, and the rows of a residual gate (0: none) behind the ``own`` rows of its first matrix,
+    from a multiple of 8 on."""
+
+    def __init__(self, cfg: ModelConfig, spec, own: int):
         super().__init__()
         self.spec, self.eps = spec, cfg.rms_norm_eps
-        self.qkv_proj = Linear(cfg.hidden_size, pad8(spec.proj_size), False, dtype, device)
+        self.gate_rows = cfg.hidden_size if cfg.design.residual_gate else 0
+        self.own = own
+
+    def first_matrix(self, cfg: ModelConfig, bias: bool, dtype, device) -> Linear:
+        rows = pad8(self.own) + pad8(self.gate_rows) if self.gate_rows else pad8(self.own)
+        return Linear(cfg.hidden_size, rows, bias or self.gate_rows > 0, dtype, device)
+
+    def residual_gate(self, proj):
+        """Logits of the residual gate out of the first matrix' result, or None."""
+        lo = pad8(self.own)
+        return proj[:, lo : lo + self.gate_rows] if self.gate_rows else None
+
+
+class Mixer(Sublayer):
+    """``forward(x, batch, cache, mm)``: (result, logits of its residual gate or None)."""
+
+    def refresh(self):
+        """Derived tables, after the weights have changed."""
+
+
+class AttentionMixer(Mixer):
+    def __init__(self, cfg: ModelConfig, spec: AttentionSpec, dtype, device):
+        super().__init__(cfg, spec, spec.proj_size)
+        self.qkv_proj = self.first_matrix(cfg, spec.qkv_bias, dtype, device)
         self.o_proj = Linear(spec.out_size, cfg.hidden_size, False, dtype, device)
         if spec.qk_norm:
             self.q_norm, self.k_norm = (RMSNormWeight(n, dtype, device) for n in spec.norm_sizes)
         if spec.sink:
             self.sink = nn.Parameter(torch.zeros(spec.heads, dtype=torch.float32, device=device))
+        for n, on in (("r1", spec.log_bias), ("r2", spec.log_bias), ("shift", spec.weighting == "sigmoid")):
+            if on:
+                setattr(self, n, nn.Parameter(torch.zeros(spec.heads, dtype=torch.float32, device=device)))
         if spec.rotary is not None:
             rotary_frequencies(self, spec.rotary, device)
         if spec.bias_rows:
@@ -149,30 +186,34 @@ class AttentionMixer(nn.Module):
     def forward(self, x, batch: RaggedBatch, cache, mm: Callable):
         s = self.spec
         norms = (self.q_norm.weight, self.k_norm.weight) if s.qk_norm else (None, None)
-        qkv = mm(x, self.qkv_proj.weight)
-        if s.qk_norm == "projection" and s.rotary is None:
-            q = ops.qk_norm_kv_write(qkv, *norms, batch.slots, cache[0], cache[1], s.heads, self.eps)
-        elif s.qk_norm != "projection":
+        qkv = mm(x, self.qkv_proj.weight, self.qkv_proj.bias)
+        if s.rotary is None and (s.qk_norm == "projection" or s.q_temp is not None):
+            if s.qk_norm == "head":
+                raise NotImplementedError("a query temperature after a norm per head")
+            q = ops.qk_norm_kv_write(qkv, *norms, batch.slots, cache[0], cache[1], s.heads, self.eps, q_temp=s.q_temp,
+                                     positions=batch.positions)
+        elif s.qk_norm != "projection" and s.q_temp is None:
             q = ops.head_norm_rope_kv_write(qkv, *norms, self.rot_freqs if s.rotary else None, batch.positions, batch.slots,
                                             cache[0], cache[1], s.heads, self.eps,
                                             interleaved=s.rotary is not None and s.rotary.interleaved,
                                             amplitude=s.rotary.amplitude if s.rotary else 1.0, key_values=s.key_values)
         else:
-            raise NotImplementedError("rotary positions after a norm over the whole projection")
+            raise NotImplementedError("rotary positions after a norm over the whole projection, or with a query temperature")
         lo = s.q_size + s.k_size + s.v_size
         o = ops.paged_attention(q, cache[0], cache[1], batch.block_table, batch.cu_q, batch.seq_lens, batch.max_q,
                                 scale=s.scale, window=s.window, keep_first=s.keep_first,
                                 bias=self.bias if s.bias_rows else None, max_ctx=batch.max_ctx, chunk=s.chunk,
                                 softcap=s.softcap, sink=self.sink if s.sink else None,
-                                gate=qkv[:, lo : lo + s.out_size] if s.gate else None)
-        return mm(o, self.o_proj.weight)
+                                gate=qkv[:, lo : lo + s.gate_size] if s.gate else None,
+                                shift=self.shift if s.weighting == "sigmoid" else None,
+                                log_bias=(self.r1, self.r2) if s.log_bias else None)
+        return mm(o, self.o_proj.weight), self.residual_gate(qkv)
 
 
-class LatentMixer(nn.Module):
+class LatentMixer(Mixer):
     def __init__(self, cfg: ModelConfig, spec: LatentSpec, dtype, device):
-        super().__init__()
-        self.spec, self.eps = spec, cfg.rms_norm_eps
-        self.in_proj = Linear(cfg.hidden_size, pad8(spec.proj_size), False, dtype, device)
+        super().__init__(cfg, spec, spec.proj_size)
+        self.in_proj = self.first_matrix(cfg, False, dtype, device)
         self.kv_norm = RMSNormWeight(spec.kv_rank, dtype, device)
         self.kv_up_proj = Linear(spec.kv_rank, pad8(spec.up_size), False, dtype, device)
         self.o_proj = Linear(spec.out_size, cfg.hidden_size, False, dtype, device)
@@ -183,13 +224,10 @@ class LatentMixer(nn.Module):
             self.sink = nn.Parameter(torch.zeros(spec.heads, dtype=torch.float32, device=device))
         rotary_frequencies(self, spec.rotary, device)
 
-    def refresh(self):
-        pass
-
     def forward(self, x, batch: RaggedBatch, cache, mm: Callable):
         s, pages, plan = self.spec, cache[0], batch.latent
         T = x.shape[0]
-        proj = mm(x, self.in_proj.weight)
+        proj = mm(x, self.in_proj.weight, self.in_proj.bias)
         rot = dict(amplitude=s.rotary.amplitude, interleaved=s.rotary.interleaved)
         ops.latent_rope_write(proj, self.kv_norm.weight, self.rot_freqs, batch.positions, batch.slots, pages,
                               0 if s.q_rank else s.heads, s.dim, s.rot_dim, s.kv_rank, self.eps, **rot, q_rank=s.q_rank,
@@ -217,14 +255,13 @@ class LatentMixer(nn.Module):
             kv = mm(rows[:, : s.kv_rank], up)
             ops.latent_prefill(q, rows[:, s.kv_rank : s.latent_size], kv, batch.cu_q[b0 : b1 + 1], ctx_cu, max_q, s.dim,
                                s.vdim, scale=s.scale, gate=gate, out=out, window=s.window, sink=sink)
-        return mm(out, self.o_proj.weight)
+        return mm(out, self.o_proj.weight), self.residual_gate(proj)
 
 
-class DeltaMixer(nn.Module):
+class DeltaMixer(Mixer):
     def __init__(self, cfg: ModelConfig, spec: DeltaSpec, dtype, device):
-        super().__init__()
-        self.spec, self.eps = spec, cfg.rms_norm_eps
-        self.in_proj = Linear(cfg.hidden_size, pad8(spec.proj_size), False, dtype, device)
+        super().__init__(cfg, spec, spec.proj_size)
+        self.in_proj = self.first_matrix(cfg, False, dtype, device)
         self.conv = nn.Parameter(torch.zeros(spec.channels, spec.conv, dtype=dtype, device=device))
         self.A_log = nn.Parameter(torch.zeros(spec.heads, dtype=torch.float32, device=device))
         self.dt_bias = nn.Parameter(torch.zeros(spec.heads, dtype=torch.float32, device=device))
@@ -238,23 +275,43 @@ class DeltaMixer(nn.Module):
             self.A_log.copy_(torch.empty(self.spec.heads, device=dev).uniform_(1.0, 8.0, generator=generator).log())
             self.dt_bias.copy_(torch.empty(self.spec.heads, device=dev).uniform_(-5.0, -2.0, generator=generator))
 
-    def refresh(self):
-        pass
+    def forward(self, x, batch: RaggedBatch, cache, mm: Callable):
+        s = self.spec
+        proj = mm(x, self.in_proj.weight, self.in_proj.bias)
+        o = ops.delta_rule(proj, self.conv, self.A_log, self.dt_bias, self.norm.weight, cache[0], cache[1], batch.cu_q,
+                           batch.seq_lens, batch.state_slots, batch.max_q, s.heads, s.kv_heads, s.dim, s.vdim, self.eps)
+        return mm(o, self.o_proj.weight), self.residual_gate(proj)
+
+
+class GlaMixer(Mixer):
+    def __init__(self, cfg: ModelConfig, spec: GlaSpec, dtype, device):
+        super().__init__(cfg, spec, spec.proj_size)
+        self.in_proj = self.first_matrix(cfg, False, dtype, device)
+        self.decay_w = nn.Parameter(torch.zeros(spec.qk_size, spec.rank, dtype=dtype, device=device))
+        self.decay_b = nn.Parameter(torch.zeros(spec.qk_size, dtype=torch.float32, device=device))
+        self.norm = RMSNormWeight(spec.vdim, dtype, device)
+        self.o_proj = Linear(spec.out_size, cfg.hidden_size, False, dtype, device)
+
+    def reset_parameters(self, generator=None):
+        with torch.no_grad():
+            dev, n = self.decay_w.device, max(self.spec.rank, 1)
+            self.decay_w.copy_(torch.empty(self.decay_w.shape, device=dev).normal_(0.0, n ** -0.5, generator=generator))
+            self.decay_b.copy_(torch.empty(self.decay_b.shape, device=dev).uniform_(0.0, 4.0, generator=generator))
 
     def forward(self, x, batch: RaggedBatch, cache, mm: Callable):
         s = self.spec
-        proj = mm(x, self.in_proj.weight)
-        o = ops.delta_rule(proj, self.conv, self.A_log, self.dt_bias, self.norm.weight, cache[0], cache[1], batch.cu_q,
-                           batch.seq_lens, batch.state_slots, batch.max_q, s.heads, s.kv_heads, s.dim, s.vdim, self.eps)
-        return mm(o, self.o_proj.weight)
+        proj = mm(x, self.in_proj.weight, self.in_proj.bias)
+        o = ops.gated_linear_attention(proj, self.decay_w, self.decay_b, self.norm.weight, cache[0], batch.cu_q, batch.seq_lens,
+                                       batch.state_slots, batch.max_q, s.heads, s.dim, s.vdim, s.tau, self.eps,
+                                       singles=batch.singles)
+        return mm(o, self.o_proj.weight), self.residual_gate(proj)
 
 
-class LruMixer(nn.Module):
+class LruMixer(Mixer):
     def __init__(self, cfg: ModelConfig, spec: LruSpec, dtype, device):
-        super().__init__()
-        self.spec = spec
+        super().__init__(cfg, spec, spec.proj_size)
         n = spec.block_size
-        self.in_proj = Linear(cfg.hidden_size, pad8(spec.proj_size), True, dtype, device)
+        self.in_proj = self.first_matrix(cfg, True, dtype, device)
         self.conv_w = nn.Parameter(torch.zeros(spec.width, spec.conv, dtype=dtype, device=device))
         self.conv_b = nn.Parameter(torch.zeros(spec.width, dtype=dtype, device=device))
         self.gates = nn.Parameter(torch.zeros(2 * spec.blocks, n, n, dtype=dtype, device=device))  # decay | input
@@ -270,62 +327,91 @@ class LruMixer(nn.Module):
             a = torch.empty(self.spec.width, device=self.lam.device).uniform_(0.9, 0.999, generator=generator)
             self.lam.copy_(torch.log(torch.expm1(-torch.log(a) / self.spec.power)))
 
-    def refresh(self):
-        pass
-
     def forward(self, x, batch: RaggedBatch, cache, mm: Callable):
         s = self.spec
         proj = mm(x, self.in_proj.weight, self.in_proj.bias)
         o = ops.rglru(proj, self.conv_w, self.conv_b, self.gates, self.gates_b, self.lam, cache[0], cache[1], batch.cu_q,
                       batch.seq_lens, batch.state_slots, batch.max_q, s.power, singles=batch.singles)
-        return mm(o, self.o_proj.weight)
+        return mm(o, self.o_proj.weight), self.residual_gate(proj)
 
 
-class GatedMLP(nn.Module):
+class GatedMLP(Sublayer):
+    """``forward(x, mm)`` of a feed-forward: (result, logits of its residual gate or None)."""
+
     def __init__(self, cfg: ModelConfig, spec: GluSpec, dtype, device):
-        super().__init__()
-        self.spec = spec
-        self.gate_up_proj = Linear(cfg.hidden_size, pad8(2 * spec.ff), False, dtype, device)
+        super().__init__(cfg, spec, 2 * spec.ff)
+        self.gate_up_proj = self.first_matrix(cfg, False, dtype, device)
         self.down_proj = Linear(spec.ff, cfg.hidden_size, False, dtype, device)
 
     def forward(self, x, mm: Callable):
         s = self.spec
-        gu = mm(x, self.gate_up_proj.weight)
+        gu = mm(x, self.gate_up_proj.weight, self.gate_up_proj.bias)
         if s.act == "silu":
             h = ops.silu_glu(gu, s.ff)
         else:
             h = ops.gelu_tanh_glu(gu, s.ff) if s.act == "gelu_tanh" else ops.clamped_glu(gu, s.ff, s.limit, s.alpha)
-        return mm(h, self.down_proj.weight)
+        return mm(h, self.down_proj.weight), self.residual_gate(gu)
 
 
-class RoutedMLP(nn.Module):
-    """Mixture of gated linear units; its result is still in parts (:class:`~verl_b200.ops.moe.RoutedSum`), which the next
-    add + norm puts together."""
+class PlainMLP(Sublayer):
+    """Two matrices with an activation between them."""
+
+    def __init__(self, cfg: ModelConfig, spec: MlpSpec, dtype, device):
+        super().__init__(cfg, spec, spec.ff)
+        self.up_proj = self.first_matrix(cfg, False, dtype, device)
+        self.down_proj = Linear(spec.ff, cfg.hidden_size, False, dtype, device)
+
+    def forward(self, x, mm: Callable):
+        u = mm(x, self.up_proj.weight, self.up_proj.bias)
+        return mm(ops.activation(u, self.spec.ff, self.spec.act), self.down_proj.weight), self.residual_gate(u)
+
+
+class RoutedMLP(Sublayer):
+    """Mixture of experts; its result is still in parts (:class:`~verl_b200.ops.moe.RoutedSum`), which the next add + norm puts
+    together. The residual gate goes with the shared unit's first matrix, or has one of its own."""
 
     def __init__(self, cfg: ModelConfig, spec: MoeSpec, dtype, device):
-        super().__init__()
-        self.spec, H = spec, cfg.hidden_size
+        super().__init__(cfg, spec, 0)
+        H = cfg.hidden_size
         self.router_proj = Linear(H, pad8(spec.router_rows), False, dtype, device)  # router | gate of the shared unit
-        self.experts_gate_up = nn.Parameter(torch.zeros(spec.experts, 2 * spec.ff, H, dtype=dtype, device=device))
+        first = torch.zeros(spec.experts, (2 if spec.gated else 1) * spec.ff, H, dtype=dtype, device=device)
+        if spec.gated:
+            self.experts_gate_up = nn.Parameter(first)
+        else:
+            self.experts_up = nn.Parameter(first)
         self.experts_down = nn.Parameter(torch.zeros(spec.experts, H, spec.ff, dtype=dtype, device=device))
+        self.correction = (nn.Parameter(torch.zeros(spec.experts, dtype=torch.float32, device=device)) if spec.correction
+                           else None)
         if spec.shared_ff:
-            self.shared = GatedMLP(cfg, GluSpec(spec.shared_ff, act=spec.act), dtype, device)
+            self.shared = (GatedMLP if spec.gated else PlainMLP)(cfg, spec.shared, dtype, device)
+        elif self.gate_rows:
+            self.gate_proj = self.first_matrix(cfg, False, dtype, device)
         # tokens per expert while a step is being routed; zero between steps
         self.register_buffer("counters", torch.zeros(spec.experts + 1, dtype=torch.int32, device=device), persistent=False)
 
     def reset_parameters(self, generator=None):
         with torch.no_grad():
-            for w in (self.experts_gate_up, self.experts_down):
+            for w in (self.experts_first, self.experts_down):
                 for e in range(w.shape[0]):
                     w[e].copy_(torch.empty(w.shape[1:], device=w.device).normal_(0.0, 0.02, generator=generator))
+
+    @property
+    def experts_first(self):
+        return self.experts_gate_up if self.spec.gated else self.experts_up
 
     def forward(self, x, mm: Callable):
         s = self.spec
         logits = ops.gemm(x, self.router_proj.weight, out_dtype=torch.float32)
-        routing = ops.moe_route(logits, s.experts, s.top, self.counters, score=s.score, renormalize=s.renormalize)
-        out = ops.moe_experts(x, routing, self.experts_gate_up, self.experts_down, s.act, weigh_input=s.weigh == "input")
-        return ops.RoutedSum(out, routing, s.weigh == "output", self.shared(x, mm) if s.shared_ff else None,
-                             logits[:, s.experts] if s.shared_ff else None)
+        routing = ops.moe_route(logits, s.experts, s.top, self.counters, score=s.score, renormalize=s.renormalize,
+                                correction=self.correction)
+        out = ops.moe_experts(x, routing, self.experts_first, self.experts_down, s.act, weigh_input=s.weigh == "input")
+        shared = gate = None
+        if s.shared_ff:
+            shared, gate = self.shared(x, mm)
+        elif self.gate_rows:
+            gate = self.residual_gate(mm(x, self.gate_proj.weight, self.gate_proj.bias))
+        return ops.RoutedSum(out, routing, s.weigh == "output", shared,
+                             logits[:, s.experts] if s.shared_ff and s.shared_gate else None), gate
 
 
 class SideInput(nn.Module):
@@ -343,7 +429,8 @@ class SideInput(nn.Module):
         return mm(g, self.out_proj.weight)
 
 
-_MIXERS = {"attention": AttentionMixer, "latent_attention": LatentMixer, "delta": DeltaMixer, "rglru": LruMixer}
+_MIXERS = {"attention": AttentionMixer, "latent_attention": LatentMixer, "delta": DeltaMixer, "gla": GlaMixer, "rglru": LruMixer}
+_MLPS = {GluSpec: GatedMLP, MlpSpec: PlainMLP, MoeSpec: RoutedMLP}
 
 
 def add_norm(pending, res, weight, eps, dtype):
@@ -353,16 +440,26 @@ def add_norm(pending, res, weight, eps, dtype):
     return ops.add_rmsnorm(pending, res, weight, eps, dtype)
 
 
+def norm_add(pending, gate, res, weight, eps, **after):
+    """Adds the norm of a sublayer's output, times the sigmoid of ``gate`` where there is one, to the stream in place."""
+    if isinstance(pending, ops.RoutedSum):
+        return ops.moe_norm_add(pending, res, weight, eps, gate=gate, **after)
+    return ops.rmsnorm_add(pending, res, weight, eps, gate=gate, **after)
+
+
 class HybridLayer(nn.Module):
     def __init__(self, cfg: ModelConfig, spec: LayerSpec, index: int, dtype, device):
         super().__init__()
+        both = cfg.design.norm == "both"  # norm1, norm2 in front of the sublayers, norm1b, norm2b behind them
         self.norm1 = RMSNormWeight(cfg.hidden_size, dtype, device)
+        self.norm1b = RMSNormWeight(cfg.hidden_size, dtype, device) if both else None
         self.mixer = _MIXERS[spec.kind](cfg, spec.mixer, dtype, device)
         if spec.mlp is not None:
             self.norm2 = RMSNormWeight(cfg.hidden_size, dtype, device)
-            self.mlp = (RoutedMLP if isinstance(spec.mlp, MoeSpec) else GatedMLP)(cfg, spec.mlp, dtype, device)
+            self.norm2b = RMSNormWeight(cfg.hidden_size, dtype, device) if both else None
+            self.mlp = _MLPS[type(spec.mlp)](cfg, spec.mlp, dtype, device)
         else:
-            self.norm2 = self.mlp = None
+            self.norm2 = self.norm2b = self.mlp = None
         self.side = SideInput(cfg, index, dtype, device) if cfg.side_dim else None
 
 
@@ -372,13 +469,21 @@ class HybridLM(nn.Module):
         self.cfg = cfg
         self.embed_tokens = nn.Embedding(cfg.vocab_size, cfg.hidden_size, dtype=dtype, device=device)
         routed = any(isinstance(s.mlp, MoeSpec) for s in cfg.layer_specs)
-        if cfg.design.norm == "post" and (cfg.side_dim or routed):
+        if cfg.design.norm == "post" and routed or cfg.design.norm != "pre" and cfg.side_dim:
             raise NotImplementedError("mixtures of experts and side inputs go with norms in front of the sublayers")
+        if cfg.design.norm != "both" and cfg.design.residual_gate:
+            raise NotImplementedError("residual gates go with norms on both sides of the sublayers")
+        if cfg.has_position_table:
+            self.pos_embed = nn.Embedding(cfg.max_position_embeddings, cfg.hidden_size, dtype=dtype, device=device)
         if cfg.design.embedding == "norm":
             self.embed_norm = RMSNormWeight(cfg.hidden_size, dtype, device)
         if cfg.side_dim:
             self.side_embed = nn.Embedding(cfg.vocab_size, cfg.num_hidden_layers * cfg.side_dim, dtype=dtype, device=device)
-        self.layers = nn.ModuleList([HybridLayer(cfg, s, i, dtype, device) for i, s in enumerate(cfg.layer_specs)])
+        # a layer that uses another's weights has no module of its own; ``runs`` has the module of every layer
+        own = [weight_owner(cfg.layer_specs, i) for i in range(len(cfg.layer_specs))]
+        self.layers = nn.ModuleList([HybridLayer(cfg, s, i, dtype, device) if own[i] == i else None
+                                     for i, s in enumerate(cfg.layer_specs)])
+        self.runs = tuple(self.layers[j] for j in own)
         self.norm = RMSNormWeight(cfg.hidden_size, dtype, device)
         self.lm_head = None if cfg.tie_word_embeddings else Linear(cfg.hidden_size, cfg.vocab_size, False, dtype, device)
         # portions up to this many tokens run latent attention in the latent space; sizes without an expanded form: all
@@ -394,12 +499,13 @@ class HybridLM(nn.Module):
         gen = torch.Generator(device=dev)
         gen.manual_seed(seed)
         with torch.no_grad():
-            for e in (self.embed_tokens, getattr(self, "side_embed", None)):
+            for e in (self.embed_tokens, getattr(self, "side_embed", None), getattr(self, "pos_embed", None)):
                 if e is not None:  # a table that is the output projection as well: logits of a size near one
                     std = self.cfg.hidden_size ** -0.5 if self.cfg.tie_word_embeddings and e is self.embed_tokens else 1.0
+                    std = 0.3 if e is getattr(self, "pos_embed", None) else std
                     e.weight.copy_(torch.empty(e.weight.shape, dtype=torch.float32, device=dev).normal_(0.0, std, generator=gen))
         for m in self.modules():
-            if isinstance(m, (Linear, DeltaMixer, LruMixer, RoutedMLP)):
+            if isinstance(m, (Linear, DeltaMixer, GlaMixer, LruMixer, RoutedMLP)):
                 m.reset_parameters(gen)
             elif isinstance(m, AttentionMixer) and m.spec.bias_rows:
                 with torch.no_grad():
@@ -407,13 +513,21 @@ class HybridLM(nn.Module):
             if isinstance(m, (AttentionMixer, LatentMixer)) and m.spec.sink:
                 with torch.no_grad():
                     m.sink.copy_(torch.empty(m.sink.shape, device=dev).normal_(0.0, 1.0, generator=gen))
+            if isinstance(m, AttentionMixer):
+                with torch.no_grad():  # distance biases of a few units; about one key in e^4 weighs one half
+                    if m.spec.log_bias:
+                        m.r1.uniform_(0.0, 1.0, generator=gen)
+                        m.r2.uniform_(0.05, 0.5, generator=gen)
+                    if m.spec.weighting == "sigmoid":
+                        m.shift.fill_(-4.0)
         self.refresh()
         return self
 
     def refresh(self):
         """Derived tables, after the weights have changed."""
         for layer in self.layers:
-            layer.mixer.refresh()
+            if layer is not None:
+                layer.mixer.refresh()
 
     @property
     def lm_head_weight(self) -> torch.Tensor:
@@ -423,7 +537,7 @@ class HybridLM(nn.Module):
         """Matrices of the layers (what weight quantisation applies to). Left out: the projections out of the latent, which are
         applied to queries and to weighted sums as well as to the latents; routers, whose scores choose; the narrow matrices of
         side inputs."""
-        return [m.weight for layer in self.layers for n, m in layer.named_modules()
+        return [m.weight for layer in self.layers if layer is not None for n, m in layer.named_modules()
                 if isinstance(m, Linear) and not n.endswith(("kv_up_proj", "router_proj")) and not n.startswith("side.")]
 
     def plan_latent(self, counts: list[int], ctx: list[int], boundaries: Callable) -> Optional[LatentPlan]:
@@ -457,9 +571,10 @@ class HybridLM(nn.Module):
         """Order of a step's sequences: those whose latent attention stays in the latent space first, and where recurrent units
         step single tokens together, those before all others. None: any order."""
         kinds = {s.kind for s in self.cfg.layer_specs}
-        if not kinds & {"latent_attention", "rglru"}:
+        if not kinds & {"latent_attention", "gla", "rglru"}:
             return None
-        return sorted(range(len(counts)), key=lambda i: (counts[i] > self.latent_short, "rglru" in kinds and counts[i] > 1))
+        singles = bool(kinds & {"gla", "rglru"})
+        return sorted(range(len(counts)), key=lambda i: (counts[i] > self.latent_short, singles and counts[i] > 1))
 
     def forward(self, *args, **kwargs):
         raise NotImplementedError(f"{self.cfg.model_type}: layer-list models are served by the rollout engine only "
@@ -474,10 +589,10 @@ class HybridLM(nn.Module):
         if c.design.norm == "post":
             res, x = ops.embedding_scaled(ids, self.embed_tokens.weight, c.embedding_scale, with_copy=True)
             last = len(self.layers) - 1
-            for i, layer in enumerate(self.layers):
-                subs = [(lambda v: layer.mixer(v, batch, cache.layers[i], mm), layer.norm1)]
+            for i, layer in enumerate(self.runs):
+                subs = [(lambda v: layer.mixer(v, batch, cache.layers[i], mm)[0], layer.norm1)]
                 if layer.mlp is not None:
-                    subs.append((lambda v: layer.mlp(v, mm), layer.norm2))
+                    subs.append((lambda v: layer.mlp(v, mm)[0], layer.norm2))
                 for k, (sub, norm) in enumerate(subs):
                     final = self.norm.weight if i == last and k == len(subs) - 1 else None
                     x = ops.rmsnorm_add(sub(x), res, norm.weight, eps, final_weight=final, final_scale=c.logit_scale)
@@ -486,16 +601,30 @@ class HybridLM(nn.Module):
             return x
         if c.design.embedding == "norm":
             res = ops.embedding_normed(ids, self.embed_tokens.weight, self.embed_norm.weight, eps)
+        elif c.design.embedding == "positions":
+            res = ops.embedding_scaled(ids, self.embed_tokens.weight, c.embedding_scale, pos_table=self.pos_embed.weight,
+                                       positions=batch.positions)
         else:
             res = ops.embedding_scaled(ids, self.embed_tokens.weight, c.embedding_scale)
-        x = ops.add_rmsnorm(None, res, self.layers[0].norm1.weight, eps)
-        for i, layer in enumerate(self.layers):
+        x = ops.add_rmsnorm(None, res, self.runs[0].norm1.weight, eps)
+        last = len(self.runs) - 1
+        for i, layer in enumerate(self.runs):
             # the norm that the next sublayer (or the head) reads through
-            after = (self.layers[i + 1].norm1 if i + 1 < len(self.layers) else self.norm).weight
-            pending = layer.mixer(x, batch, cache.layers[i], mm)
+            after = (self.runs[i + 1].norm1 if i < last else self.norm).weight
+            pending, gate = layer.mixer(x, batch, cache.layers[i], mm)
+            if c.design.norm == "both":
+                end = {"final_weight": after, "final_scale": c.logit_scale if i == last else 1.0}
+                if layer.mlp is not None:
+                    x = norm_add(pending, gate, res, layer.norm1b.weight, eps, final_weight=layer.norm2.weight)
+                    x = norm_add(*layer.mlp(x, mm), res, layer.norm2b.weight, eps, **end)
+                else:
+                    x = norm_add(pending, gate, res, layer.norm1b.weight, eps, **end)
+                if observe is not None:
+                    observe(i, res.clone())
+                continue
             if layer.mlp is not None:
                 x = add_norm(pending, res, layer.norm2.weight, eps, dtype)
-                pending = layer.mlp(x, mm)
+                pending, _ = layer.mlp(x, mm)
             if layer.side is not None:
                 y = layer.side(add_norm(pending, res, None, eps, dtype), ids, self.side_embed.weight, mm)
                 x = ops.rmsnorm_add(y, res, layer.side.norm.weight, eps, final_weight=after)

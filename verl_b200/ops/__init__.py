@@ -7,13 +7,14 @@ from .attention import (attention_varlen, decode_workspace, head_norm_rope_kv_wr
                         paged_decode_attention, qk_norm_kv_write)
 from .delta import delta_rule
 from .gemm import gemm, linear
+from .gla import gated_linear_attention
 from .latent import (latent_attention, latent_gather, latent_prefill, latent_prefill_supported, latent_queries,
                      latent_rope_write, latent_values, latent_width, rotate_tails)
 from .lmhead import lmhead_logprob_entropy
 from .lru import rglru
-from .moe import RoutedSum, moe_combine, moe_experts, moe_route
-from .nn import (add_rmsnorm, clamped_glu, embedding, embedding_normed, embedding_scaled, gelu_rows, gelu_tanh_glu, rmsnorm,
-                 rmsnorm_add, rope_qkv, rope_tables, silu_glu, softcap_, swiglu)
+from .moe import RoutedSum, moe_combine, moe_experts, moe_norm_add, moe_route
+from .nn import (activation, add_rmsnorm, clamped_glu, embedding, embedding_normed, embedding_scaled, gelu_rows, gelu_tanh_glu,
+                 rmsnorm, rmsnorm_add, rope_qkv, rope_tables, silu_glu, softcap_, swiglu)
 from .rl import (PPO_METRIC_NAMES, adamw_step, clip_coef, decode_advance, gae, grpo_advantage, ppo_loss_fused, sample,
                  sumsq_into)
 
@@ -25,4 +26,5 @@ __all__ = [
     "rmsnorm_add", "gelu_tanh_glu", "head_norm_rope_kv_write", "latent_attention", "latent_gather", "latent_prefill",
     "latent_prefill_supported", "latent_queries", "latent_rope_write", "latent_values", "latent_width", "rotate_tails",
     "embedding_normed", "silu_glu", "gelu_rows", "softcap_", "rglru", "RoutedSum", "moe_route", "moe_experts", "moe_combine",
+    "activation", "gated_linear_attention", "moe_norm_add",
 ]

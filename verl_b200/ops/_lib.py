@@ -46,8 +46,9 @@ _SIGS = {
     "vb_clip_coef": ([P, F, F, P, P, P, P], I),
     "vb_cast_f32_bf16": ([P, P, L, P], I),
     # layer-list decoders
-    "vb_embed_scaled": ([P, P, P, P, I, I, F, I, P], I),
-    "vb_rmsnorm_add": ([P, L, P, P, P, F, P, I, I, F, I, P], I),
+    "vb_embed_scaled": ([P, P, P, P, I, I, F, P, P, I, I, P], I),
+    "vb_rmsnorm_add": ([P, L, P, L, P, P, P, F, P, I, I, F, I, P], I),
+    "vb_activation": ([P, L, P, I, I, I, P, I, P], I),
     "vb_gelu_glu": ([P, L, P, I, I, I, P], I),
     "vb_silu_glu": ([P, L, P, I, I, P, P, I, P], I),
     "vb_gelu_rows": ([P, L, P, P, L, I, P, I, I, I, P], I),
@@ -58,9 +59,9 @@ _SIGS = {
     "vb_rotate_tails": ([P, L, P, F, I, P, I, I, I, I, I, P], I),
     "vb_head_gemm": ([P, L, L, P, I, P, L, L, P, L, I, I, I, I, I, I, I, P, P], I),
     "vb_head_gemm_simt": ([P, L, L, P, I, P, L, L, P, L, I, I, I, I, I, I, I, I, P], I),
-    "vb_moe_route": ([P, L, I, I, I, I, I, P, P, P, P, I, P, P], I),
+    "vb_moe_route": ([P, L, I, I, I, I, I, P, P, P, P, P, I, P, P], I),
     "vb_moe_gather": ([P, L, P, P, I, I, I, P, P, I, P], I),
-    "vb_moe_sum": ([P, P, P, I, P, L, P, L, P, P, P, I, I, F, I, P], I),
+    "vb_moe_sum": ([P, P, P, I, P, L, P, L, P, L, P, P, P, F, P, I, I, F, I, P], I),
     "vb_grouped_gemm_simt": ([P, P, P, I, I, I, P, I, P], I),
     "vb_rglru_tc_supported": ([I, I], I),
     "vb_rglru_conv": ([P, L, P, P, P, P, P, P, P, I, I, I, I, I, P], I),
@@ -73,13 +74,15 @@ _SIGS = {
     "vb_latent_flash": ([P, L, I, P, L, P, L, I, P, P, I, I, I, I, I, I, F, I, P, P, L, I, P, L, P, P], I),
     "vb_add_rmsnorm": ([P, L, P, P, P, I, I, F, I, P], I),
     "vb_clamped_glu": ([P, L, P, I, I, F, F, I, P], I),
-    "vb_qk_norm_kv_write": ([P, L, P, P, P, P, P, I, I, I, I, I, I, F, I, P], I),
+    "vb_qk_norm_kv_write": ([P, L, P, P, P, P, P, I, I, I, I, I, I, F, P, F, F, I, P], I),
     "vb_gemm_simt": ([P, P, P, P, I, I, I, L, L, L, I, I, P], I),
-    "vb_paged_attention_simt": ([P, L, P, P, P, I, P, P, I, I, I, I, I, I, I, I, F, I, I, I, P, I, F, P, P, L, P, L, I, P], I),
+    "vb_paged_attention_simt": ([P, L, P, P, P, I, P, P, I, I, I, I, I, I, I, I, F, I, I, I, P, I, F, P, P, P, P, P, L, I, P, L, I, P], I),
     "vb_paged_flash_supported": ([I, I, I, I, I, I], I),
-    "vb_paged_flash": ([P, L, P, P, I, P, I, P, P, I, I, I, I, I, I, I, I, F, I, I, I, P, I, F, P, P, L, P, L, P, P], I),
+    "vb_paged_flash": ([P, L, P, P, I, P, I, P, P, I, I, I, I, I, I, I, I, F, I, I, I, P, I, F, P, P, P, P, P, L, I, P, L, P, P], I),
     "vb_paged_decode_window_supported": ([I, I, I, I, I], I),
-    "vb_paged_decode_window": ([P, L, P, P, I, P, I, P, I, I, I, I, I, I, F, I, I, I, P, I, F, P, P, L, I, P, L, P, P, P], I),
+    "vb_paged_decode_window": ([P, L, P, P, I, P, I, P, I, I, I, I, I, I, F, I, I, I, P, I, F, P, P, P, P, P, L, I, I, P, L, P, P, P], I),
+    "vb_gla_chunk_supported": ([I, I, I, I], I),
+    "vb_gla": ([P, L, P, P, P, P, P, P, P, P, P, L, I, I, I, I, I, I, I, I, F, F, I, I, P, P], I),
     "vb_delta_chunk_supported": ([I, I], I),
     "vb_delta_chunk_bytes": ([I, I, I], L),
     "vb_delta_rule": ([P, L, P, P, P, P, P, P, P, P, P, P, P, P, P, P, L, I, I, I, I, I, I, I, I, F, I, P, P], I),

@@ -208,24 +208,29 @@ def paged_decode_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torc
 
 # ----------------- paged attention of layer-list decoders (windows, chunks, kept keys, distance bias, soft cap, sink, gate)
 def qk_norm_kv_write(qkv: torch.Tensor, q_weight: torch.Tensor | None, k_weight: torch.Tensor | None, slots: torch.Tensor,
-                     k_cache: torch.Tensor, v_cache: torch.Tensor, heads: int, eps: float) -> torch.Tensor:
+                     k_cache: torch.Tensor, v_cache: torch.Tensor, heads: int, eps: float, *,
+                     q_temp: tuple | None = None, positions: torch.Tensor | None = None) -> torch.Tensor:
     """``qkv`` [T, q | k | v | padding]: RMS norm of q and of k over the whole projection (all heads at once; no weights =
     no norm), k and v to their places in the paged caches [NB, Hk, BS, D] / [NB, Hk, BS, Dv] (slot < 0: no write).
-    Returns q [T, heads, D], a view of ``qkv`` (normalised in place on CUDA)."""
+    ``q_temp`` (coef, every): the query at position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1). Returns q [T, heads, D], a view of ``qkv`` (normalised in place on CUDA)."""
     _, Hk, BS, D = k_cache.shape
     Dv = v_cache.shape[3]
     T, nq, nk = qkv.shape[0], heads * D, Hk * D
     if qkv.is_cuda:
         rc = _lib.fn("vb_qk_norm_kv_write")(qkv.data_ptr(), qkv.stride(0), _lib.ptr(q_weight), _lib.ptr(k_weight),
                                             slots.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), T, heads, Hk, D, Dv, BS,
-                                            float(eps), int(qkv.dtype == torch.float32), _lib.stream())
+                                            float(eps), None if q_temp is None else positions.data_ptr(),
+                                            *(q_temp or (0.0, 1.0)), int(qkv.dtype == torch.float32), _lib.stream())
         _lib.check(rc, "vb_qk_norm_kv_write")
         return qkv[:, :nq].view(T, heads, D)
     from .nn import _rmsnorm_ref
 
     q, k, v = qkv[:, :nq], qkv[:, nq : nq + nk], qkv[:, nq + nk : nq + nk + Hk * Dv]
     if q_weight is not None:
-        q, k = _rmsnorm_ref(q, q_weight, eps), _rmsnorm_ref(k, k_weight, eps)
+        q, k = _rmsnorm_ref(q.float(), q_weight.float(), eps), _rmsnorm_ref(k, k_weight, eps)
+    if q_temp is not None:
+        q = q.float() * (1 + q_temp[0] * torch.log(torch.floor((positions.double() + 1) / q_temp[1]) + 1)).float()[:, None]
+    q = q.to(qkv.dtype)
     kv_cache_write(k.reshape(T, Hk, D), v.reshape(T, Hk, Dv), slots, k_cache, v_cache)
     return q.reshape(T, heads, D)
 
@@ -280,14 +285,16 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                     cu_q: torch.Tensor, seq_lens: torch.Tensor, max_q: int, *, scale: float, window: int = 0,
                     keep_first: int = 0, bias: torch.Tensor | None = None, max_ctx: int = 0, chunk: int = 0,
                     softcap: float = 0.0, sink: torch.Tensor | None = None, gate: torch.Tensor | None = None,
-                    impl: str = "auto") -> torch.Tensor:
+                    shift: torch.Tensor | None = None, log_bias: tuple | None = None, impl: str = "auto") -> torch.Tensor:
     """Causal attention of ragged queries (the last ``cu_q[b + 1] - cu_q[b]`` positions of every sequence) over the paged
     cache, which holds the new tokens already. q [T, Hq, D]; caches [NB, Hk, BS, D] / [NB, Hk, BS, Dv]; ``seq_lens``
     [B] = tokens of each sequence including the new ones. ``window`` > 0: position i sees j <= i with i - j < window or
     j < keep_first. ``bias`` fp32 [Hq, L]: ``bias[h, min(i - j, L - 1)]`` is added to the scaled score. ``chunk`` > 0:
     position i sees j <= i with i // chunk == j // chunk (not together with a window). ``softcap`` > 0: scores become
     ``softcap * tanh(score / softcap)`` (without a bias). ``sink`` fp32 [Hq]: exp(sink[h]) joins the softmax denominator.
-    ``gate`` [T, Hq * Dv]: the result is multiplied with its sigmoid. ``max_ctx``: bound of ``seq_lens``. -> [T, Hq * Dv].
+    ``shift`` fp32 [Hq]: no softmax, a key weighs sigmoid(score + shift[h]) (without bias, soft cap and sink). ``log_bias`` = (r1,
+    r2), fp32 [Hq] each, only then: r1[h] * ln(1 + r2[h] * (i - j)) is taken off the scaled score. ``gate`` [T, Hq * Dv] or
+    [T, Hq]: the result is multiplied with its sigmoid. ``max_ctx``: bound of ``seq_lens``. -> [T, Hq * Dv].
 
     ``impl``: "tc" = tcgen05 kernels (bf16, head sizes up to 128 in multiples of 8, block size a power of two in 8..128;
     one token per sequence: up to 8 query heads per KV head), "simt" = CUDA-core kernel, "auto" = "tc" where it applies."""
@@ -297,6 +304,11 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     out = torch.empty((T, Hq * Dv), dtype=q.dtype, device=q.device)
     if (chunk > 0 and window > 0) or (softcap > 0 and bias is not None):
         raise ValueError("paged_attention: chunk goes without window, and softcap without bias")
+    if (shift is not None and (bias is not None or softcap > 0 or sink is not None)) or (log_bias is not None and shift is None):
+        raise ValueError("paged_attention: sigmoid weights go without bias table, soft cap and sink, a log bias only with them")
+    gate_w = 0 if gate is None else gate.shape[1] // Hq  # numbers of the gate per head
+    if gate is not None and gate.shape[1] not in (Hq, Hq * Dv):
+        raise ValueError(f"paged_attention: a gate of {gate.shape[1]} numbers for {Hq} heads of {Dv}")
     if q.is_cuda:
         f32 = q.dtype == torch.float32
         L = 0 if bias is None else bias.shape[1]
@@ -305,14 +317,15 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         else:
             tc = _lib.fn("vb_paged_flash_supported")(Hq, Hk, D, Dv, BS, L)
         tc = bool(tc) and not f32 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
-        if gate is not None:
+        if gate is not None and gate_w > 1:
             tc = tc and gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0
         if impl == "tc" and not tc:
             raise ValueError(f"tensor-core attention does not support Hq={Hq} Hk={Hk} D={D} Dv={Dv} block_size={BS}")
         args = (q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr())
         table = (block_table.data_ptr(), block_table.stride(0))
-        mask = (float(scale), window, keep_first, chunk, _lib.ptr(bias), L, float(softcap), _lib.ptr(sink), _lib.ptr(gate),
-                0 if gate is None else gate.stride(0))
+        r1, r2 = log_bias or (None, None)
+        mask = (float(scale), window, keep_first, chunk, _lib.ptr(bias), L, float(softcap), _lib.ptr(sink), _lib.ptr(shift),
+                _lib.ptr(r1), _lib.ptr(r2), _lib.ptr(gate), 0 if gate is None else gate.stride(0), gate_w)
         dst = (out.data_ptr(), out.stride(0))
         if tc and impl != "simt" and max_q == 1:
             seen = max_ctx or block_table.shape[1] * BS
@@ -357,11 +370,23 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
             s = softcap * torch.tanh(s / softcap)
         if bias is not None:
             s = s + bias[:, dist.clamp(0, bias.shape[1] - 1)]
+        if shift is not None:
+            if log_bias is not None:
+                r1, r2 = (r[:, None, None] for r in log_bias)
+                s = s - r1 * torch.log1p(r2 * dist.clamp(min=0))
+            w = torch.sigmoid(s + shift[:, None, None]).masked_fill(~seen, 0.0)
+            out[lo:hi] = _head_gate(torch.einsum("hqk,hkd->qhd", w, vv), None if gate is None else gate[lo:hi]).to(q.dtype)
+            continue
         s = s.masked_fill(~seen, float("-inf"))
         if sink is not None:  # a key without a value
             s = torch.cat((s, sink[:, None, None].expand(Hq, hi - lo, 1)), -1)
-        o = torch.einsum("hqk,hkd->qhd", torch.softmax(s, -1)[..., :n], vv).reshape(hi - lo, -1)
-        if gate is not None:
-            o = o * torch.sigmoid(gate[lo:hi].float())
-        out[lo:hi] = o.to(q.dtype)
+        o = torch.einsum("hqk,hkd->qhd", torch.softmax(s, -1)[..., :n], vv)
+        out[lo:hi] = _head_gate(o, None if gate is None else gate[lo:hi]).to(q.dtype)
     return out
+
+
+def _head_gate(o: torch.Tensor, gate: torch.Tensor | None) -> torch.Tensor:
+    """o [T, H, D] times the sigmoid of ``gate`` [T, H * D] or [T, H] -> [T, H * D]."""
+    if gate is not None:
+        o = o * torch.sigmoid(gate.float().view(o.shape[0], o.shape[1], -1))
+    return o.reshape(o.shape[0], -1)

@@ -167,7 +167,7 @@ def latent_attention(q: torch.Tensor, pages: torch.Tensor, block_table: torch.Te
         rc = _lib.fn("vb_paged_attention_simt")(q.data_ptr(), q.stride(0), pages.data_ptr(), pages.data_ptr(),
                                                 block_table.data_ptr(), block_table.stride(0), cu_q.data_ptr(),
                                                 seq_lens.data_ptr(), T, B, H, 1, width, rank, width, BS, float(scale), window,
-                                                0, 0, None, 0, 0.0, _lib.ptr(sink), None, 0, out.data_ptr(), out.stride(0),
+                                                0, 0, None, 0, 0.0, _lib.ptr(sink), None, None, None, None, 0, 0, out.data_ptr(), out.stride(0),
                                                 int(f32), _lib.stream())
         _lib.check(rc, "vb_paged_attention_simt")
         return out

@@ -14,6 +14,7 @@ import torch
 import torch.nn.functional as F
 
 from . import _lib
+from .nn import activation, add_rmsnorm, rmsnorm_add
 
 BLK = 128
 
@@ -139,7 +140,8 @@ class Routing:
 @dataclass
 class RoutedSum:
     """Result of a mixture in parts: rows of the sorted buffer ``out`` [rows, H], one per pair of ``routing`` (``weigh``: still to
-    be multiplied with its weight), and the ``shared`` unit's result [T, H] with the logit of its gate [T] (fp32)."""
+    be multiplied with its weight), and the ``shared`` unit's result [T, H] with the logit of its gate [T] (fp32; None: a factor of
+    one)."""
 
     out: torch.Tensor
     routing: Routing
@@ -149,9 +151,9 @@ class RoutedSum:
 
 
 def moe_route(logits: torch.Tensor, experts: int, top: int, counters: torch.Tensor, *, score: str = "sigmoid",
-              renormalize: bool = False) -> Routing:
-    """The ``top`` experts of every token by the fp32 ``logits`` [T, experts | ...]. ``counters``: int32 [experts + 1], zero
-    before and after."""
+              renormalize: bool = False, correction: torch.Tensor | None = None) -> Routing:
+    """The ``top`` experts of every token by the fp32 ``logits`` [T, experts | ...]. ``correction`` fp32 [experts]: added to the
+    scores for the choice, not for the weights. ``counters``: int32 [experts + 1], zero before and after."""
     T = logits.shape[0]
     # an expert's padding is at most BLK - 1 rows, and experts without a token have none
     rows = (T * top + min(experts, T * top) * (BLK - 1)) // BLK * BLK
@@ -161,38 +163,42 @@ def moe_route(logits: torch.Tensor, experts: int, top: int, counters: torch.Tens
         new = lambda n, dt=torch.int32: torch.empty(n, dtype=dt, device=logits.device)  # noqa: E731
         r = Routing(new((T, top)), new((T, top), torch.float32), new((T, top)), new(rows // BLK), rows)
         rc = _lib.fn("vb_moe_route")(logits.data_ptr(), logits.stride(0), T, experts, top, int(score == "softmax"),
-                                     int(renormalize), r.idx.data_ptr(), r.weight.data_ptr(), r.dest.data_ptr(),
+                                     int(renormalize), _lib.ptr(correction), r.idx.data_ptr(), r.weight.data_ptr(), r.dest.data_ptr(),
                                      r.blk_expert.data_ptr(), rows // BLK, counters.data_ptr(), _lib.stream())
         _lib.check(rc, "vb_moe_route")
         return r
     z = logits[:, :experts]
     s = torch.sigmoid(z) if score == "sigmoid" else torch.softmax(z, -1)
-    idx = torch.sort(s, dim=-1, descending=True, stable=True).indices[:, :top]
+    choice = s if correction is None else s + correction
+    idx = torch.sort(choice, dim=-1, descending=True, stable=True).indices[:, :top]
     w = s.gather(1, idx)
     if renormalize:
-        w = w / w.sum(-1, keepdim=True)
+        w = w / (w.sum(-1, keepdim=True) + 1e-20)
     dest, blk_expert, _, P = moe_layout(idx, experts)
     return Routing(idx, w, dest.view(T, top), blk_expert, P)
 
 
-def moe_experts(x: torch.Tensor, routing: Routing, gate_up: torch.Tensor, down: torch.Tensor, act: str, *,
+def moe_experts(x: torch.Tensor, routing: Routing, first: torch.Tensor, down: torch.Tensor, act: str, *,
                 weigh_input: bool) -> torch.Tensor:
-    """Gated linear units of the routed pairs: rows of the sorted buffer [rows, H] (other rows undefined). x [T, H], ``gate_up``
-    [E, 2 * ff, H], ``down`` [E, H, ff]. ``weigh_input``: a unit runs on weight * x, which is applied behind its first, linear,
-    product."""
-    if act != "silu":
+    """Units of the routed pairs: rows of the sorted buffer [rows, H] (other rows undefined). x [T, H], ``down`` [E, H, ff].
+    ``act`` "silu": gated linear units, ``first`` [E, 2 * ff, H] = gate | up; "gelu", "relu2": two matrices, ``first`` [E, ff, H].
+    ``weigh_input``: a gated unit runs on weight * x, which is applied behind its first, linear, product."""
+    if act not in ("silu", "gelu", "relu2"):
         raise ValueError(f"unknown activation of routed experts {act!r}")
+    gated = act == "silu"
+    if weigh_input and not gated:
+        raise NotImplementedError("experts of two matrices that run on weighted inputs")
     T, H = x.shape
-    top, (E, N, _) = routing.idx.shape[1], gate_up.shape
-    ff = N // 2
+    top, (E, N, _) = routing.idx.shape[1], first.shape
+    ff = N // 2 if gated else N
     if not x.is_cuda:
         out = torch.zeros(routing.rows, H, dtype=x.dtype)
         for e in range(E):
             t, k = (routing.idx == e).nonzero(as_tuple=True)
-            gu = x[t].float() @ gate_up[e].float().t()
+            gu = x[t].float() @ first[e].float().t()
             if weigh_input:
                 gu = gu * routing.weight[t, k][:, None]
-            h = (F.silu(gu[:, :ff]) * gu[:, ff:]).to(x.dtype)
+            h = (F.silu(gu[:, :ff]) * gu[:, ff:]).to(x.dtype) if gated else activation(gu, ff, act).to(x.dtype)
             out[routing.dest[t, k]] = (h.float() @ down[e].float().t()).to(x.dtype)
         return out
     f32, P = int(x.dtype == torch.float32), routing.rows
@@ -201,7 +207,9 @@ def moe_experts(x: torch.Tensor, routing: Routing, gate_up: torch.Tensor, down: 
     rc = _lib.fn("vb_moe_gather")(x.data_ptr(), x.stride(0), routing.dest.data_ptr(), routing.weight.data_ptr(), T, top, H,
                                   xs.data_ptr(), scale.data_ptr(), f32, _lib.stream())
     _lib.check(rc, "vb_moe_gather")
-    gu = grouped_product(xs, gate_up, routing.blk_expert)
+    gu = grouped_product(xs, first, routing.blk_expert)
+    if not gated:
+        return grouped_product(activation(gu, ff, act, routing.blk_expert), down, routing.blk_expert)
     h = new(P, ff)
     rc = _lib.fn("vb_silu_glu")(gu.data_ptr(), gu.stride(0), h.data_ptr(), P, ff, scale.data_ptr() if weigh_input else None,
                                 routing.blk_expert.data_ptr(), f32, _lib.stream())
@@ -226,22 +234,40 @@ def grouped_product(xs: torch.Tensor, weight: torch.Tensor, blk_expert: torch.Te
 def moe_combine(parts: RoutedSum, residual: torch.Tensor, weight: torch.Tensor | None, eps: float) -> torch.Tensor:
     """Adds the mixture's sum to the fp32 ``residual`` [T, H] IN PLACE; returns rmsnorm(residual) * weight, or without a weight
     the residual, in the parts' dtype."""
-    r, dtype = parts.routing, parts.out.dtype
-    T, H = residual.shape
-    top = r.idx.shape[1]
     if residual.is_cuda:
-        y = torch.empty((T, H), dtype=dtype, device=residual.device)
-        sh, lg = parts.shared, parts.shared_logit
-        rc = _lib.fn("vb_moe_sum")(parts.out.data_ptr(), r.dest.data_ptr(), r.weight.data_ptr() if parts.weigh else None, top,
-                                       _lib.ptr(sh), 0 if sh is None else sh.stride(0), _lib.ptr(lg),
-                                       0 if lg is None else lg.stride(0), residual.data_ptr(), _lib.ptr(weight), y.data_ptr(),
-                                       T, H, float(eps), int(dtype == torch.float32), _lib.stream())
-        _lib.check(rc, "vb_moe_sum")
-        return y
-    picked = parts.out[r.dest.reshape(-1)].view(T, top, H).float()
+        return _moe_sum(parts, residual, eps, weight)
+    return add_rmsnorm(_sum_ref(parts), residual, weight, eps, parts.out.dtype)
+
+
+def moe_norm_add(parts: RoutedSum, residual: torch.Tensor, weight: torch.Tensor, eps: float, *,
+                 final_weight: torch.Tensor | None = None, final_scale: float = 1.0,
+                 gate: torch.Tensor | None = None) -> torch.Tensor:
+    """:func:`~verl_b200.ops.nn.rmsnorm_add` of the mixture's sum."""
+    if residual.is_cuda:
+        return _moe_sum(parts, residual, eps, final_weight, weight, gate, final_scale)
+    y = rmsnorm_add(_sum_ref(parts), residual, weight, eps, final_weight=final_weight, final_scale=final_scale, gate=gate)
+    return y.to(parts.out.dtype)
+
+
+def _moe_sum(parts, residual, eps, weight, post=None, gate=None, scale=1.0):
+    r, dtype, (T, H) = parts.routing, parts.out.dtype, residual.shape
+    y = torch.empty((T, H), dtype=dtype, device=residual.device)
+    sh, lg = parts.shared, parts.shared_logit
+    rc = _lib.fn("vb_moe_sum")(parts.out.data_ptr(), r.dest.data_ptr(), r.weight.data_ptr() if parts.weigh else None,
+                               r.idx.shape[1], _lib.ptr(sh), 0 if sh is None else sh.stride(0), _lib.ptr(lg),
+                               0 if lg is None else lg.stride(0), _lib.ptr(gate), 0 if gate is None else gate.stride(0),
+                               _lib.ptr(post), residual.data_ptr(), _lib.ptr(weight), float(scale), y.data_ptr(), T, H, float(eps),
+                               int(dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "vb_moe_sum")
+    return y
+
+
+def _sum_ref(parts):
+    r = parts.routing
+    T, top = r.idx.shape
+    picked = parts.out[r.dest.reshape(-1)].view(T, top, -1).float()
     d = (picked * r.weight[..., None] if parts.weigh else picked).sum(1)
     if parts.shared is not None:
-        d = d + parts.shared.float() * torch.sigmoid(parts.shared_logit.float())[:, None]
-    from .nn import add_rmsnorm
-
-    return add_rmsnorm(d, residual, weight, eps, dtype)
+        factor = 1.0 if parts.shared_logit is None else torch.sigmoid(parts.shared_logit.float())[:, None]
+        d = d + parts.shared.float() * factor
+    return d

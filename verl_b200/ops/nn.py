@@ -272,16 +272,21 @@ def embedding(ids: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
 
 
 # ------------------------------------------------- 32-bit residual stream (inference only)
-def embedding_scaled(ids: torch.Tensor, weight: torch.Tensor, scale: float, with_copy: bool = False):
-    """fp32 residual stream ``weight[ids] * scale`` [T, H]; ``with_copy``: (stream, the same in the weight's dtype)."""
+def embedding_scaled(ids: torch.Tensor, weight: torch.Tensor, scale: float, with_copy: bool = False,
+                     pos_table: torch.Tensor | None = None, positions: torch.Tensor | None = None):
+    """fp32 residual stream ``weight[ids] * scale`` (``+ pos_table[positions]``, as it is) [T, H]; ``with_copy``: (stream, the same
+    in the weight's dtype). Positions past the table's end take its last row."""
     if not weight.is_cuda:
         res = F.embedding(ids, weight).float() * scale
+        if pos_table is not None:
+            res = res + pos_table[positions.clamp(max=pos_table.shape[0] - 1)].float()
         return (res, res.to(weight.dtype, copy=True)) if with_copy else res
     T, H = ids.numel(), weight.shape[1]
     res = torch.empty((T, H), dtype=torch.float32, device=weight.device)
     y = torch.empty((T, H), dtype=weight.dtype, device=weight.device) if with_copy else None
     rc = _lib.fn("vb_embed_scaled")(ids.data_ptr(), weight.data_ptr(), res.data_ptr(), _lib.ptr(y), T, H, float(scale),
-                                    int(weight.dtype == torch.float32), _lib.stream())
+                                    _lib.ptr(pos_table), None if pos_table is None else positions.data_ptr(),
+                                    0 if pos_table is None else pos_table.shape[0], int(weight.dtype == torch.float32), _lib.stream())
     _lib.check(rc, "vb_embed_scaled")
     return (res, y) if with_copy else res
 
@@ -319,17 +324,21 @@ def add_rmsnorm(delta: torch.Tensor | None, residual: torch.Tensor, weight: torc
 
 
 def rmsnorm_add(delta: torch.Tensor, residual: torch.Tensor, weight: torch.Tensor, eps: float, *,
-                final_weight: torch.Tensor | None = None, final_scale: float = 1.0) -> torch.Tensor:
+                final_weight: torch.Tensor | None = None, final_scale: float = 1.0,
+                gate: torch.Tensor | None = None) -> torch.Tensor:
     """Adds rmsnorm(delta) * weight to the fp32 ``residual`` [T, H] IN PLACE. Returns the new residual in the weight's dtype,
-    or with ``final_weight`` rmsnorm(residual) * final_weight * final_scale."""
+    or with ``final_weight`` rmsnorm(residual) * final_weight * final_scale. ``gate`` [T, H]: delta is multiplied with its sigmoid
+    first."""
     if not residual.is_cuda:
-        residual += _rmsnorm_ref(delta.float(), weight.float(), eps)
+        delta = delta.float() if gate is None else delta.float() * torch.sigmoid(gate.float())
+        residual += _rmsnorm_ref(delta, weight.float(), eps)
         if final_weight is None:
             return residual.to(weight.dtype, copy=True)
         return (_rmsnorm_ref(residual, final_weight.float(), eps) * final_scale).to(weight.dtype)
     T, H = residual.shape
     y = torch.empty((T, H), dtype=weight.dtype, device=residual.device)
-    rc = _lib.fn("vb_rmsnorm_add")(delta.data_ptr(), delta.stride(0), residual.data_ptr(), weight.data_ptr(),
+    rc = _lib.fn("vb_rmsnorm_add")(delta.data_ptr(), delta.stride(0), _lib.ptr(gate), 0 if gate is None else gate.stride(0),
+                                   residual.data_ptr(), weight.data_ptr(),
                                    _lib.ptr(final_weight), float(final_scale), y.data_ptr(), T, H, float(eps),
                                    int(weight.dtype == torch.float32), _lib.stream())
     _lib.check(rc, "vb_rmsnorm_add")
@@ -358,6 +367,24 @@ def silu_glu(gate_up: torch.Tensor, ff: int) -> torch.Tensor:
     rc = _lib.fn("vb_silu_glu")(gate_up.data_ptr(), gate_up.stride(0), y.data_ptr(), T, ff, None, None,
                                 int(gate_up.dtype == torch.float32), _lib.stream())
     _lib.check(rc, "vb_silu_glu")
+    return y
+
+
+_ACTS = {"gelu": 0, "relu2": 1}
+
+
+def activation(x: torch.Tensor, n: int, act: str, blk_expert: torch.Tensor | None = None) -> torch.Tensor:
+    """``act`` of the first ``n`` elements of the rows of x [T, n]: "gelu" (with erf) or "relu2", the square of relu. ``blk_expert``:
+    rows of a buffer sorted by expert; blocks of 128 rows without one are left out."""
+    if act not in _ACTS:
+        raise ValueError(f"unknown activation {act!r}")
+    if not x.is_cuda:
+        f = x[:, :n].float()
+        return (F.gelu(f) if act == "gelu" else torch.relu(f).square()).to(x.dtype)
+    y = torch.empty((x.shape[0], n), dtype=x.dtype, device=x.device)
+    rc = _lib.fn("vb_activation")(x.data_ptr(), x.stride(0), y.data_ptr(), x.shape[0], n, _ACTS[act], _lib.ptr(blk_expert),
+                                  int(x.dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "vb_activation")
     return y
 
 

@@ -252,7 +252,7 @@ class NativeRolloutEngine:
         self.dtype = model.embed_tokens.weight.dtype
         self.on_gpu = self.device.type == "cuda"
         self.max_num_seqs = max_num_seqs
-        self.max_model_len = max_model_len
+        self.max_model_len = min(max_model_len, model.cfg.max_position_embeddings) if model.cfg.has_position_table else max_model_len
         self.max_num_batched_tokens = max(max_num_batched_tokens, 16)
         self.block_size = block_size
         # pages of a shared prefix say nothing about the recurrent state behind it
