@@ -73,21 +73,32 @@ def clear_choices(cfg, t, g):
         elif n.endswith(".norm2"):
             w[:CODES] = 1
         elif n.endswith(".router"):
-            i = int(n[1:].split(".")[0])
-            E, top = w.shape[0], cfg["layers"][i]["mlp"]["router"]["top"]
+            E, top = w.shape[0], cfg["layers"][int(n[1:].split(".")[0])]["mlp"]["router"]["top"]
             corr = t[n.replace("router", "correction")]
-            corr.copy_(corr.to(torch.bfloat16))  # as it is stored
+            kinds = None
+            while kinds is None:
+                kinds = clear_kinds(corr, E, top, g)
+                if kinds is None:
+                    corr.copy_((torch.rand(E, generator=g) / E).to(torch.bfloat16))
             w[:] = 0
-            for c in range(CODES):
-                for _ in range(1000):
-                    z = torch.linspace(-1.2, 1.2, E)[torch.randperm(E, generator=g)]
-                    choice = [(torch.softmax(a * z, -1) + corr).sort(descending=True) for a in (1.0, 1.5, 2.0, 3.0, 4.0, 5.0)]
-                    chosen = {tuple(sorted(s.indices[:top].tolist())) for s in choice}
-                    if top == E or len(chosen) == 1 and all(float(s.values[top - 1] - s.values[top]) > 0.1 / E for s in choice):
-                        break
-                else:
-                    raise RuntimeError("no clear choice found")
-                w[:, c] = z
+            w[:, :CODES] = kinds.T
+
+
+def clear_kinds(corr, E, top, g):
+    """[CODES, E] logits whose choice is clear whatever the size of the stream, or None if none are found."""
+    out = []
+    corr.copy_(corr.to(torch.bfloat16))  # as it is stored
+    for _ in range(CODES):
+        for _ in range(200):
+            z = torch.linspace(-1.2, 1.2, E)[torch.randperm(E, generator=g)]
+            ranked = [(torch.softmax(a * z, -1) + corr).sort(descending=True) for a in (1.0, 1.5, 2.0, 3.0, 4.0, 5.0)]
+            chosen = {tuple(sorted(s.indices[:top].tolist())) for s in ranked}
+            if top == E or len(chosen) == 1 and all(float(s.values[top - 1] - s.values[top]) > 0.1 / E for s in ranked):
+                out.append(z)
+                break
+        else:
+            return None
+    return torch.stack(out)
 
 
 def weights(cfg, seed=0, dtype=torch.bfloat16, clear=True):

@@ -62,7 +62,7 @@ __device__ __forceinline__ float decay_logit(const GlaParams& p, int c, const R*
 // decays are computed. Eight lanes share a column; lane r holds rows 4 (r + 8 i) + e.
 constexpr int GS_THREADS = 256, GS_NP = 4;
 template <typename T, int NR>
-__global__ void __launch_bounds__(GS_THREADS) gla_step_kernel(const GlaParams p) {
+__global__ void __launch_bounds__(GS_THREADS, NR <= 16 ? 2 : 1) gla_step_kernel(const GlaParams p) {
   constexpr int DP = NR * 8;
   extern __shared__ float sm[];
   float* q_s = sm;            // [DP]
@@ -122,46 +122,47 @@ __global__ void __launch_bounds__(GS_THREADS) gla_step_kernel(const GlaParams p)
   for (int d = tid; d < DP; d += GS_THREADS)
     a_s[d] = d < p.D ? expf(log_sigmoid(decay_logit<T>(p, h * p.D + d, r_s)) * p.inv_tau) : 0.f;
   __syncthreads();
-  float kv[NR], qv[NR], av[NR];
-#pragma unroll
-  for (int i = 0; i < NR; ++i) {
-    const int d = 4 * (r + 8 * (i >> 2)) + (i & 3);
-    kv[i] = k_s[d];
-    qv[i] = q_s[d];
-    av[i] = a_s[d];
-  }
   for (int cbase = 0; cbase < p.V; cbase += GS_NP * 32) {
     if (cbase > 0) load_cols(cbase, S);
+    float v[GS_NP], o[GS_NP];
 #pragma unroll
     for (int j = 0; j < GS_NP; ++j) {
       const int col = cbase + j * 32 + cw;
-      const float v = col < p.V ? v_s[col] : 0.f;
-      float o = 0.f;
+      v[j] = col < p.V ? v_s[col] : 0.f;
+      o[j] = 0.f;
+    }
 #pragma unroll
-      for (int i = 0; i < NR; ++i) {
-        S[j][i] = fmaf(kv[i], v, av[i] * S[j][i]);
-        o = fmaf(S[j][i], qv[i], o);
-      }
-      o = sum8(o);
-      if (col < p.V) {
-        if (r == 0) o_s[col] = o;
+    for (int i = 0; i < NR / 4; ++i) {
+      const int d = 4 * (r + 8 * i);
+      const float4 q = *reinterpret_cast<const float4*>(q_s + d), k = *reinterpret_cast<const float4*>(k_s + d),
+                   a = *reinterpret_cast<const float4*>(a_s + d);
 #pragma unroll
-        for (int i = 0; i < NR / 4; ++i) {
-          const int d = 4 * (r + 8 * i);
-          if (d < p.D) {
-            const float4 x = make_float4(S[j][4 * i], S[j][4 * i + 1], S[j][4 * i + 2], S[j][4 * i + 3]);
-            float* dst = st + (long long)col * p.D + d;
-            if (vec) {
-              __stcs(reinterpret_cast<float4*>(dst), x);
-            } else {
-              dst[0] = x.x;
-              if (d + 1 < p.D) dst[1] = x.y;
-              if (d + 2 < p.D) dst[2] = x.z;
-              if (d + 3 < p.D) dst[3] = x.w;
-            }
+      for (int j = 0; j < GS_NP; ++j) {
+        float4 x = make_float4(S[j][4 * i], S[j][4 * i + 1], S[j][4 * i + 2], S[j][4 * i + 3]);
+        x.x = fmaf(k.x, v[j], a.x * x.x);
+        x.y = fmaf(k.y, v[j], a.y * x.y);
+        x.z = fmaf(k.z, v[j], a.z * x.z);
+        x.w = fmaf(k.w, v[j], a.w * x.w);
+        o[j] = fmaf(x.x, q.x, fmaf(x.y, q.y, fmaf(x.z, q.z, fmaf(x.w, q.w, o[j]))));
+        const int col = cbase + j * 32 + cw;
+        if (col < p.V && d < p.D) {
+          float* dst = st + (long long)col * p.D + d;
+          if (vec) {
+            __stcs(reinterpret_cast<float4*>(dst), x);
+          } else {
+            dst[0] = x.x;
+            if (d + 1 < p.D) dst[1] = x.y;
+            if (d + 2 < p.D) dst[2] = x.z;
+            if (d + 3 < p.D) dst[3] = x.w;
           }
         }
       }
+    }
+#pragma unroll
+    for (int j = 0; j < GS_NP; ++j) {
+      const float x = sum8(o[j]);
+      const int col = cbase + j * 32 + cw;
+      if (r == 0 && col < p.V) o_s[col] = x;
     }
   }
   __syncthreads();
@@ -278,8 +279,9 @@ __global__ void __launch_bounds__(GS_THREADS) gla_scan_kernel(const GlaParams p)
 //     O^T [v, t]      = S0^T hi . (Q~ hi + Q~ lo)^T + S0^T lo . Q~ hi^T
 //     O^T [v, t]     += [V; V]^T . P hi + V^T . P lo             (P: causal part of the scores)
 // Every fp32 operand enters as two bf16 terms, so that products carry about 16 bits of both operands and sums are fp32; v and the
-// numbers r are bf16 activations. Warp w owns TMEM lanes 32 (w % 4) .. and a quarter of the columns of each accumulator. q, k and
-// r of the next chunk arrive while a chunk is worked on.
+// numbers r are bf16 activations. Warp w owns TMEM lanes 32 (w % 4) .. and a quarter of the columns of each accumulator; three
+// warps issue the products. While the tensor cores work on a chunk, the decays of the next one are computed, and its q, k and r
+// arrive.
 constexpr int GK_C = 64, GK_THREADS = 512;
 constexpr int GK_Q_OFF = 0;                        // Q~: per 64 channels hi | lo, [64 tokens] x 128 bytes
 constexpr int GK_K_OFF = 32768;                    // K~: the same
@@ -301,18 +303,23 @@ __device__ __forceinline__ float ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-// log(sigmoid(z)): log(1 + u) = 2 atanh(u / (2 + u)), u = e^-|z| <= 1, by its series (relative error below 2e-7)
+// log(sigmoid(z)): log(1 + u) = 2 atanh(s), s = u / (2 + u), u = e^-|z| <= 1; atanh(s) / s by a polynomial in s^2 fitted on
+// [0, 1/9] (relative error 2e-8)
 __device__ __forceinline__ float log_sigmoid_fast(float z) {
   const float u = __expf(-fabsf(z)), s = __fdividef(u, 2.f + u), t = s * s;
-  const float y = fmaf(t, fmaf(t, fmaf(t, fmaf(t, fmaf(t, 1.f / 11.f, 1.f / 9.f), 1.f / 7.f), 1.f / 5.f), 1.f / 3.f), 1.f);
-  return fminf(z, 0.f) - 2.f * s * y;
+  const float y = fmaf(t, fmaf(t, fmaf(t, fmaf(t, 0.13433777f, 0.14116978f), 0.20003835f), 0.3333332f), 1.f);
+  return fmaf(-2.f * s, y, fminf(z, 0.f));
 }
 
+// ND: channels with those that are zero, 64 or 128
+template <int ND>
 __global__ void __launch_bounds__(GK_THREADS, 1) gla_chunk_kernel(const GlaParams p, int* status) {
   extern __shared__ uint8_t smb[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smb) + 1023) & ~uintptr_t(1023));
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + GK_BAR_OFF);  // Z, scores, state and O of the state, O
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 4);
+  // completed products: Z, scores, O of the state, state, O
+  enum { Z_DONE, SC_DONE, IN_DONE, ST_DONE, O_DONE, NBAR };
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + GK_BAR_OFF);
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + NBAR);
   int* far = reinterpret_cast<int*>(tmem_slot + 1);
   float* sum_s = reinterpret_cast<float*>(smem + GK_SUM_OFF);
   float* dec_s = reinterpret_cast<float*>(smem + GK_DEC_OFF);
@@ -324,10 +331,9 @@ __global__ void __launch_bounds__(GK_THREADS, 1) gla_chunk_kernel(const GlaParam
   const int start = p.seq_lens[b] - n, HD = p.H * p.D, HV = p.H * p.V;
   const __nv_bfloat16* proj = static_cast<const __nv_bfloat16*>(p.proj) + (long long)first * p.stride;
   const int VC = min(128, p.V - v0);             // columns of this CTA
-  const int nd = p.D > 64 ? 128 : 64;            // channels past D are zero
 
   if (tid == 0) {
-    for (int i = 0; i < 4; ++i) mbar_init(&bars[i], 1);
+    for (int i = 0; i < NBAR; ++i) mbar_init(&bars[i], 1);
     *far = 0;
     mbar_fence_init();
   }
@@ -335,17 +341,21 @@ __global__ void __launch_bounds__(GK_THREADS, 1) gla_chunk_kernel(const GlaParam
     tmem_alloc(tmem_slot, 512);
     tmem_relinquish();
   }
-  // q, k, r of the tokens from t0 on
+  // q and k of the tokens from t0 on; 16-byte groups of a row swapped by fours, so that two rows are read without conflicts
   auto load_qk = [&](int t0) {
-    const int groups = nd >> 3;
-    for (int i = tid; i < GK_C * groups; i += GK_THREADS) {
-      const int t = i / groups, d = i % groups * 8;
-      const bool on = t0 + t < n && d < p.D;
-      const __nv_bfloat16* src = proj + (on ? (long long)(t0 + t) * p.stride + h * p.D + d : 0);
-      uint8_t* to = smem + GK_R_OFF + t * 256 + d * 2;
+    constexpr int GROUPS = ND / 8;
+#pragma unroll
+    for (int i = tid; i < GK_C * GROUPS; i += GK_THREADS) {
+      const int t = i / GROUPS, g = i % GROUPS;
+      const bool on = t0 + t < n && g * 8 < p.D;
+      const __nv_bfloat16* src = proj + (on ? (long long)(t0 + t) * p.stride + h * p.D + g * 8 : 0);
+      uint8_t* to = smem + GK_R_OFF + t * 256 + ((g ^ (t & 4)) << 4);
       cp_async16(to, src, on);
       cp_async16(to + 16384, on ? src + HD : src, on);
     }
+    cp_async_commit();
+  };
+  auto load_r = [&](int t0) {
     const __nv_bfloat16* r = proj + 2 * (HD + HV);
     if ((p.rank & 7) == 0) {
       const int t = tid >> 3, g = tid & 7;  // 64 tokens, 8 groups of eight
@@ -362,6 +372,7 @@ __global__ void __launch_bounds__(GK_THREADS, 1) gla_chunk_kernel(const GlaParam
     cp_async_commit();
   };
   auto load_v = [&](int t0) {
+#pragma unroll
     for (int i = tid; i < GK_C * 16; i += GK_THREADS) {
       const int t = i >> 4, g = i & 15;
       const bool on = t0 + t < n && g * 8 < VC;
@@ -370,8 +381,8 @@ __global__ void __launch_bounds__(GK_THREADS, 1) gla_chunk_kernel(const GlaParam
     }
     cp_async_commit();
   };
+  load_r(0);
   load_qk(0);
-  load_v(0);
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -382,7 +393,6 @@ __global__ void __launch_bounds__(GK_THREADS, 1) gla_chunk_kernel(const GlaParam
   // this thread's channel: its row of W (by the first quarter of the warps) and its bias
   const bool d_on = row < p.D;
   const float bias = d_on ? p.decay_b[h * p.D + row] : 0.f;
-  const int r_steps = (p.rank + 15) / 16;
   if (grp == 0) {
     uint32_t w[32];
     const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(p.decay_w) + (long long)(h * p.D + (d_on ? row : 0)) * p.rank;
@@ -405,7 +415,7 @@ __global__ void __launch_bounds__(GK_THREADS, 1) gla_chunk_kernel(const GlaParam
   };
   // the state: this thread's column v and channels c0 .. c0 + 31
   const int c0 = grp * 32;
-  const bool s_on = c0 < nd;
+  const bool s_on = c0 < ND;
   float* st = p.state + (((long long)slot * p.H + h) * p.V + v0 + row) * p.D;
   uint8_t* s_hi = smem + GK_S_OFF + (c0 >> 6) * 32768 + row * 128;
   if (s_on) {
@@ -422,11 +432,16 @@ __global__ void __launch_bounds__(GK_THREADS, 1) gla_chunk_kernel(const GlaParam
   tmem_st_wait();
 
   const uint32_t base = smem_u32(smem);
-  const int k_steps = (p.D + 15) / 16;
+  constexpr int K_STEPS = ND / 16;
   constexpr uint32_t id_kk = umma_idesc(1, 1, 0, 0, 128, 64);           // both K-major
   constexpr uint32_t id_mm = umma_idesc(1, 1, 1, 1, 128, 64);           // both MN-major
-  const uint32_t id_st = umma_idesc(1, 1, 1, 1, 128, (uint32_t)nd);
-  const bool issuer = warp == 0 && elect_one();
+  constexpr uint32_t id_st = umma_idesc(1, 1, 1, 1, 128, ND);
+  // operands: a step of 32 bytes (K-major) or 2048 bytes (MN-major) adds to the address field of a descriptor
+  const uint64_t dq = umma_smem_desc(base + GK_Q_OFF, 16, 1024), dk = umma_smem_desc(base + GK_K_OFF, 16, 1024),
+                 dk_mn = umma_smem_desc(base + GK_K_OFF, 16384, 1024), ds = umma_smem_desc(base + GK_S_OFF, 16, 1024),
+                 dv = umma_smem_desc(base + GK_V_OFF, 8192, 1024), dp = umma_smem_desc(base + GK_P_OFF, 8192, 1024),
+                 da = umma_smem_desc(base + GK_A_OFF, 16, 1024);
+  const int r_steps = (p.rank + 15) / 16;
   const float qscale = 1.f / sqrtf((float)p.D), rate = p.inv_tau * 1.4426950408889634f;
   bool ok = true;
   // every thread waits for products; one failed wait ends the loop for the whole CTA
@@ -437,50 +452,39 @@ __global__ void __launch_bounds__(GK_THREADS, 1) gla_chunk_kernel(const GlaParam
     tc_fence_after();
     ok = good && ok;
   };
-
-  int t0 = 0;
-  for (uint32_t it = 0; t0 < n; ++it) {
-    const uint32_t parity = it & 1;
-    cp_async_wait<1>();  // q, k and r (the newest group is v)
-    fence_proxy_async_smem();
-    tc_fence_before();
-    if (!__syncthreads_and(ok)) break;
-    if (issuer) {
-      tc_fence_after();
-      for (int k = 0; k < r_steps; ++k)
-        tc_mma_f16_ta(tmem + GK_Z, tmem + GK_W + k * 8, umma_smem_desc(base + GK_A_OFF + k * 32, 16, 1024), id_kk, k != 0);
-      tc_commit(&bars[0]);
-    }
-    wait(0, parity, 4 * it);
-    // running log2 decays of this thread's channel over its sixteen tokens
-    float lb[16];
+  auto issue_z = [&]() {
+    for (int k = 0; k < r_steps; ++k) tc_mma_f16_ta(tmem + GK_Z, tmem + GK_W + k * 8, da + k * 2, id_kk, k != 0);
+    tc_commit(&bars[Z_DONE]);
+  };
+  // Running log2 decays of this thread's channel over its sixteen tokens of the chunk at t0; tokens that the chunk takes.
+  float lb[16];
+  auto decays = [&](int t0, uint32_t parity) {
+    wait(Z_DONE, parity, t0);
     {
       uint32_t z[16];
       tmem_ld_32x16(my + GK_Z + grp * 16, z);
       tmem_ld_wait();
+      const int in = d_on ? n - t0 - grp * 16 : 0;
       float run = 0.f;
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
         const float l = fmaxf(log_sigmoid_fast(__uint_as_float(z[i]) + bias) * rate, GK_FLOOR);
-        run += d_on && t0 + grp * 16 + i < n ? l : 0.f;
+        run += i < in ? l : 0.f;
         lb[i] = run;
       }
       sum_s[grp * 128 + row] = run;
     }
     __syncthreads();
-    float total = 0.f;
-    {
-      float before = 0.f;
+    float total = 0.f, before = 0.f;
 #pragma unroll
-      for (int g = 0; g < 4; ++g) {
-        const float x = sum_s[g * 128 + row];
-        total += x;
-        if (g < grp) before += x;
-      }
-#pragma unroll
-      for (int i = 0; i < 16; ++i) lb[i] += before;
+    for (int g = 0; g < 4; ++g) {
+      const float x = sum_s[g * 128 + row];
+      total += x;
+      if (g < grp) before += x;
     }
-    int cnt = min(GK_C, n - t0);  // tokens of this chunk
+#pragma unroll
+    for (int i = 0; i < 16; ++i) lb[i] += before;
+    int cnt = min(GK_C, n - t0);
     if (!__syncthreads_and(total >= -GK_RANGE)) {  // the largest power of two of them that stays within the range
       int out = 0;
 #pragma unroll
@@ -497,53 +501,96 @@ __global__ void __launch_bounds__(GK_THREADS, 1) gla_chunk_kernel(const GlaParam
       __syncthreads();
       if (tid == 0) *far = 0;
     }
-    if (row < nd) {
-      const __nv_bfloat16* raw = reinterpret_cast<const __nv_bfloat16*>(smem + GK_R_OFF) + row;
-      uint8_t* qd = smem + GK_Q_OFF + (row >> 6) * 16384 + (row & 7) * 2;
-      const int g = (row & 63) >> 3;
+    return cnt;
+  };
+
+  cp_async_wait<1>();  // r
+  fence_proxy_async_smem();
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 0 && elect_one()) {
+    tc_fence_after();
+    issue_z();
+  }
+  int t0 = 0, cnt = decays(0, 0);
+  load_r(cnt);
+  cp_async_wait<1>();  // q and k
+  __syncthreads();
+  load_v(0);
+  for (uint32_t it = 0; t0 < n; ++it) {
+    const uint32_t parity = it & 1;
+    // Q~ and K~: lanes in pairs, each lane two channels of eight tokens: the even one of the first eight of the sixteen
+    if (row < ND) {
+      const bool odd = lane & 1;
+      const int d = row & ~1, g = d >> 3;
 #pragma unroll
-      for (int i = 0; i < 16; ++i) {
-        const int t = grp * 16 + i;
-        const bool on = t < cnt;
-        const float q = on ? dl_f(raw[t * 128]) * qscale * ex2(lb[i]) : 0.f;
-        const float k = on ? dl_f(raw[8192 + t * 128]) * ex2(-lb[i]) : 0.f;
-        const __nv_bfloat16 qh = __float2bfloat16(q), kh = __float2bfloat16(k);
-        uint8_t* to = qd + t * 128 + ((g ^ (i & 7)) << 4);
-        *reinterpret_cast<__nv_bfloat16*>(to) = qh;
-        *reinterpret_cast<__nv_bfloat16*>(to + 8192) = __float2bfloat16(q - __bfloat162float(qh));
-        *reinterpret_cast<__nv_bfloat16*>(to + GK_K_OFF) = kh;
-        *reinterpret_cast<__nv_bfloat16*>(to + GK_K_OFF + 8192) = __float2bfloat16(k - __bfloat162float(kh));
-        if (t == cnt - 1) dec_s[row] = ex2(lb[i]);
+      for (int j = 0; j < 8; ++j) {
+        const float own = odd ? lb[8 + (j ^ 4)] : lb[j], give = odd ? lb[j] : lb[8 + (j ^ 4)];
+        const float got = __shfl_xor_sync(0xffffffffu, give, 1);
+        const float b0 = odd ? got : own, b1 = odd ? own : got;
+        const int t = grp * 16 + (odd ? 8 + (j ^ 4) : j);
+        const uint8_t* raw = smem + GK_R_OFF + t * 256 + ((g ^ (t & 4)) << 4) + (d & 7) * 2;
+        const uint32_t q2 = *reinterpret_cast<const uint32_t*>(raw), k2 = *reinterpret_cast<const uint32_t*>(raw + 16384);
+        const float e0 = ex2(b0), e1 = ex2(b1);
+        if (t == cnt - 1) *reinterpret_cast<float2*>(dec_s + d) = make_float2(e0, e1);
+        uint32_t qh = 0, ql = 0, kh = 0, kl = 0;
+        if (t < cnt) {
+          split2(__uint_as_float(q2 << 16) * (qscale * e0), __uint_as_float(q2 & 0xffff0000u) * (qscale * e1), qh, ql);
+          split2(__uint_as_float(k2 << 16) * ex2(-b0), __uint_as_float(k2 & 0xffff0000u) * ex2(-b1), kh, kl);
+        }
+        uint8_t* to = smem + (g >> 3) * 16384 + t * 128 + (((g & 7) ^ (t & 7)) << 4) + (d & 7) * 2;
+        *reinterpret_cast<uint32_t*>(to + GK_Q_OFF) = qh;
+        *reinterpret_cast<uint32_t*>(to + GK_Q_OFF + 8192) = ql;
+        *reinterpret_cast<uint32_t*>(to + GK_K_OFF) = kh;
+        *reinterpret_cast<uint32_t*>(to + GK_K_OFF + 8192) = kl;
       }
     }
-    cp_async_wait<0>();  // v
+    cp_async_wait<0>();  // v; r of the next chunk
     fence_proxy_async_smem();
     tc_fence_before();
     if (!__syncthreads_and(ok)) break;
-    if (issuer) {
-      tc_fence_after();
-      auto q_desc = [&](int term, int k) {
-        return umma_smem_desc(base + GK_Q_OFF + (k >> 2) * 16384 + term * 8192 + (k & 3) * 32, 16, 1024);
-      };
-      for (int term = 0; term < 2; ++term)
-        for (int k = 0; k < k_steps; ++k)
-          tc_mma_f16(tmem + GK_SC, umma_smem_desc(base + GK_K_OFF + (k >> 2) * 16384 + (k & 3) * 32, 16, 1024), q_desc(term, k),
-                     id_kk, term != 0 || k != 0);
-      tc_commit(&bars[1]);
-      for (int term = 0; term < 3; ++term)  // hi hi, hi lo, lo hi
-        for (int k = 0; k < k_steps; ++k)
-          tc_mma_f16(tmem + GK_O,
-                     umma_smem_desc(base + GK_S_OFF + (k >> 2) * 32768 + (term == 2 ? 16384 : 0) + (k & 3) * 32, 16, 1024),
-                     q_desc(term == 1, k), id_kk, term != 0 || k != 0);
-      for (int term = 0; term < 2; ++term)
-        for (int k = 0; k < GK_C / 16; ++k)
-          tc_mma_f16(tmem + GK_ST, umma_smem_desc(base + GK_V_OFF + k * 2048, 8192, 1024),
-                     umma_smem_desc(base + GK_K_OFF + term * 8192 + k * 2048, 16384, 1024), id_st, 1);
-      tc_commit(&bars[2]);
+    const int t1 = t0 + cnt;
+    if (warp == 0) {
+      if (elect_one()) {
+        tc_fence_after();
+        if (t1 < n) issue_z();
+#pragma unroll
+        for (int term = 0; term < 2; ++term)
+#pragma unroll
+          for (int k = 0; k < K_STEPS; ++k)
+            tc_mma_f16(tmem + GK_SC, dk + (k >> 2) * 1024 + (k & 3) * 2, dq + term * 512 + (k >> 2) * 1024 + (k & 3) * 2, id_kk,
+                       term != 0 || k != 0);
+        tc_commit(&bars[SC_DONE]);
+      }
+    } else if (warp == 1) {
+      if (elect_one()) {
+        tc_fence_after();
+#pragma unroll
+        for (int term = 0; term < 3; ++term)  // hi hi, hi lo, lo hi
+#pragma unroll
+          for (int k = 0; k < K_STEPS; ++k)
+            tc_mma_f16(tmem + GK_O, ds + (term == 2 ? 1024 : 0) + (k >> 2) * 2048 + (k & 3) * 2,
+                       dq + (term == 1 ? 512 : 0) + (k >> 2) * 1024 + (k & 3) * 2, id_kk, term != 0 || k != 0);
+        tc_commit(&bars[IN_DONE]);
+      }
+    } else if (warp == 2) {
+      if (elect_one()) {
+        tc_fence_after();
+#pragma unroll
+        for (int term = 0; term < 2; ++term)
+#pragma unroll
+          for (int k = 0; k < GK_C / 16; ++k)
+            tc_mma_f16(tmem + GK_ST, dv + k * 128, dk_mn + term * 512 + k * 128, id_st, 1);
+        tc_commit(&bars[ST_DONE]);
+      }
     }
-    load_qk(t0 + cnt);
+    __syncwarp();
+    load_qk(t1);
+    int next = 0;
+    if (t1 < n) next = decays(t1, parity ^ 1);
+    load_r(t1 + next);
     // scores: this thread's row s (hi or lo term of K~) and sixteen tokens t
-    wait(1, parity, 4 * it + 1);
+    wait(SC_DONE, parity, t0 + 1);
     {
       uint32_t x[16];
       tmem_ld_32x16(my + GK_SC + grp * 16, x);
@@ -566,16 +613,19 @@ __global__ void __launch_bounds__(GK_THREADS, 1) gla_chunk_kernel(const GlaParam
     fence_proxy_async_smem();
     tc_fence_before();
     if (!__syncthreads_and(ok)) break;
-    if (issuer) {
-      tc_fence_after();
-      for (int k = 0; k < 12; ++k)  // P hi of both partial sums, P lo of the first
-        tc_mma_f16(tmem + GK_O, umma_smem_desc(base + GK_V_OFF + (k & 3) * 2048, 8192, 1024),
-                   umma_smem_desc(base + GK_P_OFF + k * 2048, 8192, 1024), id_mm, 1);
-      tc_commit(&bars[3]);
+    if (warp == 1) {  // the one that has issued O of the state
+      if (elect_one()) {
+        tc_fence_after();
+#pragma unroll
+        for (int k = 0; k < 12; ++k)  // P hi of both partial sums, P lo of the first
+          tc_mma_f16(tmem + GK_O, dv + (k & 3) * 128, dp + k * 128, id_mm, 1);
+        tc_commit(&bars[O_DONE]);
+      }
     }
+    __syncwarp();
     // the state behind the chunk
-    wait(2, parity, 4 * it + 2);
-    const bool last = t0 + cnt >= n;
+    wait(ST_DONE, parity, t0 + 2);
+    wait(IN_DONE, parity, t0 + 3);
     if (s_on) {
       uint32_t x[32];
       tmem_ld_32x32(my + GK_ST + c0, x);
@@ -589,7 +639,7 @@ __global__ void __launch_bounds__(GK_THREADS, 1) gla_chunk_kernel(const GlaParam
         f[e + 2] = __uint_as_float(x[e + 2]) * d4.z;
         f[e + 3] = __uint_as_float(x[e + 3]) * d4.w;
       }
-      if (last) {
+      if (t1 >= n) {
         if (ok && row < VC)
 #pragma unroll
           for (int e = 0; e < 32; ++e)
@@ -602,7 +652,7 @@ __global__ void __launch_bounds__(GK_THREADS, 1) gla_chunk_kernel(const GlaParam
       }
       tmem_st_wait();
     }
-    wait(3, parity, 4 * it + 3);
+    wait(O_DONE, parity, t0 + 4);
     {
       uint32_t x[16];
       tmem_ld_32x16(my + GK_O + grp * 16, x);
@@ -611,16 +661,20 @@ __global__ void __launch_bounds__(GK_THREADS, 1) gla_chunk_kernel(const GlaParam
 #pragma unroll
       for (int e = 0; e < 16; ++e) o[(grp * 16 + e) * 128] = __float2bfloat16(__uint_as_float(x[e]));
     }
+    cp_async_wait<1>();  // q and k of the next chunk (the newest group is r)
+    tc_fence_before();
     if (!__syncthreads_and(ok)) break;
-    load_v(t0 + cnt);
+    load_v(t1);
     __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (long long)(first + t0) * p.out_stride + (long long)h * p.V + v0;
+#pragma unroll
     for (int i = tid; i < GK_C * 16; i += GK_THREADS) {
       const int t = i >> 4, g = i & 15;
       if (t < cnt && g * 8 < VC)
         *reinterpret_cast<uint4*>(out + (long long)t * p.out_stride + g * 8) =
             *reinterpret_cast<const uint4*>(smem + GK_P_OFF + t * 256 + g * 16);
     }
-    t0 += cnt;
+    t0 = t1;
+    cnt = next;
   }
   cp_async_wait<0>();
   tc_fence_before();
@@ -668,11 +722,13 @@ static int run_gla(GlaParams p, int T_, int B, int singles, int chunk, int* stat
   if (chunk) {
     static bool attr = false;
     if (!attr) {
-      VB_CUDA_CHECK(cudaFuncSetAttribute(gla_chunk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, GK_SMEM));
+      VB_CUDA_CHECK(cudaFuncSetAttribute(gla_chunk_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, GK_SMEM));
+      VB_CUDA_CHECK(cudaFuncSetAttribute(gla_chunk_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, GK_SMEM));
       attr = true;
     }
     const dim3 g((p.V + 127) / 128, p.H, B - singles);
-    rc = (int)vb_launch_pdl(gla_chunk_kernel, g, dim3(GK_THREADS), GK_SMEM, stream, 1, p, status);
+    rc = (int)(p.D <= 64 ? vb_launch_pdl(gla_chunk_kernel<64>, g, dim3(GK_THREADS), GK_SMEM, stream, 1, p, status)
+                         : vb_launch_pdl(gla_chunk_kernel<128>, g, dim3(GK_THREADS), GK_SMEM, stream, 1, p, status));
     vb_count_launch();
   } else {
     cudaError_t e = vb_launch_pdl(gla_decay_kernel<T>, dim3(T_, (p.H * p.D + 127) / 128), dim3(128), 0, stream, 1, p);

@@ -210,7 +210,7 @@ __global__ void activation_kernel(const T* __restrict__ x, long long stride, T* 
   pdl_wait();
   const long long step = (long long)gridDim.x * blockDim.x, i0 = blockIdx.x * (long long)blockDim.x + threadIdx.x;
   auto act = [](float z) {
-    if (ACT == 0) return 0.5f * z * (1.f + erff(z * 0.70710678118654752f));
+    if (ACT == 0) return gelu_erf<sizeof(T) == 2>(z);
     const float r = fmaxf(z, 0.f);
     return r * r;
   };
@@ -291,8 +291,9 @@ __global__ void qk_norm_kv_write_kernel(T* __restrict__ qkv, long long stride, c
   const int nq = Hq * D, nk = Hk * D, nv = Hk * Dv;
   constexpr int W = VEC ? 8 : 1;
   float iq = 1.f, ik = 1.f;
-  const float temp =
-      positions ? 1.f + coef * logf((float)floor((double)(positions[blockIdx.x] + 1) / (double)every) + 1.f) : 1.f;
+  __shared__ float temp;
+  if (positions != nullptr && threadIdx.x == 0)
+    temp = 1.f + coef * logf((float)floor((double)(positions[blockIdx.x] + 1) / (double)every) + 1.f);
   if (qw != nullptr) {
     float sq = 0.f, sk = 0.f;
     for (int i = threadIdx.x * W; i < nq + nk; i += blockDim.x * W) {  // q and k are adjacent
@@ -313,8 +314,11 @@ __global__ void qk_norm_kv_write_kernel(T* __restrict__ qkv, long long stride, c
     iq = 1.f / sqrtf(sq / (float)nq + eps);
     ik = 1.f / sqrtf(sk / (float)nk + eps);
   }
-  if (qw != nullptr || positions != nullptr) {
+  if (positions != nullptr) {
+    __syncthreads();
     iq *= temp;
+  }
+  if (qw != nullptr || positions != nullptr) {
     for (int i = threadIdx.x * W; i < nq; i += blockDim.x * W) {
       if (VEC) {
         float f[8], g[8];

@@ -134,6 +134,17 @@ __device__ __forceinline__ float gelu_tanh(float g) {
   if (FAST) return __fdividef(g, 1.f + __expf(-2.f * z));
   return 0.5f * g * (1.f + tanhf(z));
 }
+// gelu with erf: z Phi(z). FAST: erf by formula 7.1.26 of Abramowitz and Stegun, Handbook of Mathematical Functions (largest error
+// 1.5e-7).
+template <bool FAST>
+__device__ __forceinline__ float gelu_erf(float z) {
+  const float x = z * 0.70710678118654752f;
+  if (!FAST) return 0.5f * z * (1.f + erff(x));
+  const float a = fabsf(x), t = __fdividef(1.f, fmaf(0.3275911f, a, 1.f));
+  const float y = t * fmaf(t, fmaf(t, fmaf(t, fmaf(t, 1.061405429f, -1.453152027f), 1.421413741f), -0.284496736f), 0.254829592f);
+  const float tail = 0.5f * y * __expf(-a * a);  // 1 - Phi(|z|)
+  return z * (z < 0.f ? tail : 1.f - tail);
+}
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
 
 }  // namespace vb

@@ -6,7 +6,7 @@ checkpoint code. Mirrors the HF ``config.json`` fields of the supported families
 from __future__ import annotations
 
 import json
-from dataclasses import asdict, dataclass, field
+from dataclasses import asdict, dataclass, field, replace
 from pathlib import Path
 from typing import Any
 
@@ -364,6 +364,24 @@ def _golonex_specs(groups: int, heads: int, kv_heads: int, dim: int, window: int
     return (LayerSpec(LruSpec(*lru), mlp), LayerSpec(lat, mlp), LayerSpec(att, mlp)) * groups
 
 
+def _malinex_specs(groups: int, heads: int, kv_heads: int, dim: int, gla: tuple, ff: int, moe: tuple) -> tuple:
+    """``groups`` x (two layers of gated linear attention, one attention layer), a mixture of experts after each but the first, which
+    has a dense feed-forward; every second group uses the linear layers of the group before it again. ``gla``: heads, key and
+    value size, tau, rank; ``moe``: experts, experts per token, their size, the shared unit's size."""
+    mlp = MoeSpec(*moe, act="relu2", score="softmax", renormalize=True, weigh="output", gated=False, correction=True,
+                  shared_gate=False)
+    lin = LayerSpec(GlaSpec(*gla), mlp)
+    att = LayerSpec(AttentionSpec(heads, kv_heads, dim, dim, dim ** -0.5, gate="head", qkv_bias=True, q_temp=(0.1, 1024.0),
+                                  log_bias=True, weighting="sigmoid"), mlp)
+    out = []
+    for g in range(groups):
+        for k in (0, 1):
+            again = g % 2 and 3 * (g - 1) + k > 0
+            out.append(replace(lin, weights_of=3 * (g - 1) + k) if again else replace(lin, mlp=MlpSpec(ff)) if g + k == 0 else lin)
+        out.append(att)
+    return tuple(out)
+
+
 # Named architectures used by the benchmarks and tests (random-init, no download needed).
 PRESETS: dict[str, dict] = {
     "tiny-qwen2": dict(model_type="qwen2", vocab_size=2048, hidden_size=256, intermediate_size=688,
@@ -484,6 +502,14 @@ PRESETS: dict[str, dict] = {
                        side_dim=256,
                        layer_specs=_golonex_specs(10, 32, 8, 128, 1024, (4096, 16, 4), (32, 128, 64, 128, 512, 1536),
                                                   (16, 4, 896, 3584))),
+    "tiny-malinex": dict(model_type="malinex", vocab_size=616, hidden_size=136, eos_token_id=2, rms_norm_eps=1e-6, logit_scale=0.5,
+                         max_position_embeddings=1024,
+                         layer_specs=_malinex_specs(2, 6, 3, 24, (3, 24, 40, 8.0, 8), 296, (6, 2, 72, 104))),
+    # real-model sizes for benchmarks: the widths of llama-3-8b, its feed-forward cut into 16 experts
+    "malinex-8b": dict(model_type="malinex", vocab_size=128256, hidden_size=4096, eos_token_id=None, rms_norm_eps=1e-5,
+                       num_attention_heads=32, num_key_value_heads=8, head_dim=128, intermediate_size=896,
+                       max_position_embeddings=32768,
+                       layer_specs=_malinex_specs(10, 32, 8, 128, (32, 128, 128, 16.0, 16), 14336, (16, 4, 896, 3584))),
     "llama-3-8b": dict(model_type="llama", vocab_size=128256, hidden_size=4096, intermediate_size=14336,
                        num_hidden_layers=32, num_attention_heads=32, num_key_value_heads=8, rope_theta=5e5,
                        rms_norm_eps=1e-5, eos_token_id=128001),

@@ -17,7 +17,7 @@ import torch
 
 from .. import ops
 from ..models import build_model, preset
-from ..models.layer_specs import MoeSpec
+from ..models.layer_specs import PLAIN_ACTS, MoeSpec
 from ..ops import _lib
 from ..ops import moe as moe_ops
 from .engine import NativeRolloutEngine
@@ -145,7 +145,11 @@ def bench_kernels(name: str, vs: str, B: int, n: int, DB: int, ctx: int) -> list
 
     # norm with residual: fp32 stream against the bf16 stream of the homogeneous model
     x, res32, res16, w = r(T, H), torch.randn(T, H, device="cuda"), r(T, H), r(H)
-    if cfg.design.norm == "post":
+    if cfg.design.norm == "both":
+        g = r(T, H) if cfg.design.residual_gate else None
+        add("rmsnorm_add with " + ("gate and " if g is not None else "") + "next norm (fp32 residual)", time_us(
+            lambda: ops.rmsnorm_add(x, res32, w, 1e-5, final_weight=w, gate=g)), T * H * (14 if g is not None else 12))
+    elif cfg.design.norm == "post":
         add("rmsnorm_add (fp32 residual)", time_us(lambda: ops.rmsnorm_add(x, res32, w, 1e-5)), T * H * 12)
     else:
         add("add_rmsnorm (fp32 residual)", time_us(lambda: ops.add_rmsnorm(x, res32, w, 1e-5)), T * H * 12)
@@ -153,7 +157,9 @@ def bench_kernels(name: str, vs: str, B: int, n: int, DB: int, ctx: int) -> list
     routed = glu if isinstance(glu, MoeSpec) else None
     ff = routed.shared_ff if routed else glu.ff
     gu = r(T, 2 * ff)
-    if glu.act == "silu":
+    if glu.act in PLAIN_ACTS:
+        add(f"activation ({glu.act}, {ff})", time_us(lambda: ops.activation(gu, ff, glu.act)), T * ff * 4)
+    elif glu.act == "silu":
         add(f"silu_glu ({ff})", time_us(lambda: ops.silu_glu(gu, ff)), T * ff * 6)
     elif glu.act == "gelu_tanh":
         add("gelu_tanh_glu", time_us(lambda: ops.gelu_tanh_glu(gu, glu.ff)), T * glu.ff * 6)
@@ -163,6 +169,7 @@ def bench_kernels(name: str, vs: str, B: int, n: int, DB: int, ctx: int) -> list
     del gu
     if cfg.side_dim:
         _bench_side(add, r, cfg, T)
+    routed = routed or next((s.mlp for s in cfg.layer_specs if isinstance(s.mlp, MoeSpec)), None)
     if routed:
         _bench_moe(add, r, routed, H, T, f"prefill {T}")
         _bench_moe(add, r, routed, H, DB, f"decode {DB}")
@@ -174,6 +181,8 @@ def bench_kernels(name: str, vs: str, B: int, n: int, DB: int, ctx: int) -> list
         _bench_latent(add, r, mixers["latent_attention"], B, n, DB, ctx)
     if "delta" in mixers:
         _bench_delta(add, r, mixers["delta"], B, n, DB, ctx)
+    if "gla" in mixers:
+        _bench_gla(add, r, mixers["gla"], B, n, DB, ctx)
     return rows
 
 
@@ -199,7 +208,8 @@ def _bench_attention(add, r, att, ref, B: int, n: int, DB: int, ctx: int) -> Non
             qkv, qw, kw, freqs, pos, slots, kc, vc, hq, 1e-5, interleaved=att.rotary.interleaved, key_values=att.key_values)),
             nb - (T * att.k_size * 2 if att.key_values else 0))
     else:
-        add("qk_norm_kv_write", time_us(lambda: ops.qk_norm_kv_write(qkv, qw, kw, slots, kc, vc, hq, 1e-5)), nb)
+        add("qk_norm_kv_write" + (" with query temperature" if att.q_temp else ""), time_us(lambda: ops.qk_norm_kv_write(
+            qkv, qw, kw, slots, kc, vc, hq, 1e-5, q_temp=att.q_temp, positions=pos)), nb)
     cos, sin = ops.rope_tables(ref.head_dim, n, 1e6, "cuda")
 
     def rope_write():
@@ -235,11 +245,17 @@ def _bench_attention(add, r, att, ref, B: int, n: int, DB: int, ctx: int) -> Non
     if att.sink:
         kw_["sink"] = torch.randn(hq, device="cuda")
         what.append("sink")
-    gate = r(max(T, DB), att.out_size) if att.gate else None
+    if att.weighting == "sigmoid":
+        kw_["shift"] = torch.full((hq,), -4.0, device="cuda")
+        what.append("sigmoid")
+    if att.log_bias:
+        kw_["log_bias"] = (torch.rand(hq, device="cuda"), torch.rand(hq, device="cuda"))
+        what.append("log bias")
+    gate = r(max(T, DB), att.gate_size) if att.gate else None
     if att.gate:
-        what.append("gate")
+        what.append("gate" if att.gate == "element" else f"gate per {att.gate}")
     what = ", ".join(what)
-    nbytes = T * ((3 if att.gate else 2) * hq + 2 * hk) * d * 2
+    nbytes = T * ((2 * hq + 2 * hk) * d + att.gate_size) * 2
     add(f"paged_flash ({what})", time_us(lambda: ops.paged_attention(
         q, kc, vc, bt, cu, lens, n, **kw_, gate=gate[:T] if att.gate else None)), nbytes, 4 * pairs * B * hq * d)
     add("paged_flash (full causal, plain)", time_us(
@@ -354,7 +370,8 @@ def _bench_moe(add, r, m, H: int, T: int, tag: str) -> None:
     counters = torch.zeros(E + 1, dtype=torch.int32, device="cuda")
     wr = r(logits.shape[1], H) * 0.02
     copies = 1 if T > 2048 else 8  # decode: the weights rotate, so that they come from memory
-    gus, downs = [r(E, 2 * ff, H) * 0.02 for _ in range(copies)], [r(E, H, ff) * 0.02 for _ in range(copies)]
+    first = 2 * ff if m.gated else ff
+    gus, downs = [r(E, first, H) * 0.02 for _ in range(copies)], [r(E, H, ff) * 0.02 for _ in range(copies)]
     turn = [0]
 
     def at(ws):
@@ -363,7 +380,8 @@ def _bench_moe(add, r, m, H: int, T: int, tag: str) -> None:
 
     add(f"router (gemm, fp32 out), {tag}", time_us(lambda: ops.gemm(x, wr, out_dtype=torch.float32)),
         2 * (T * H + wr.numel()) + 4 * logits.numel(), 2.0 * T * wr.numel())
-    route = lambda: ops.moe_route(logits, E, top, counters, score=m.score)  # noqa: E731
+    corr = torch.rand(E, device="cuda") if m.correction else None
+    route = lambda: ops.moe_route(logits, E, top, counters, score=m.score, renormalize=m.renormalize, correction=corr)  # noqa: E731
     add(f"moe_route, {tag}", time_us(route), 4 * T * (E + 3 * top))
     rt = route()
     top_i = rt.idx.long()
@@ -378,21 +396,32 @@ def _bench_moe(add, r, m, H: int, T: int, tag: str) -> None:
     tok, dest = torch.arange(pairs, device="cuda") // top, rt.dest.flatten().long()
     add("  vs index_copy of the homogeneous models", time_us(
         lambda: torch.zeros((P, H), dtype=x.dtype, device="cuda").index_copy(0, dest, x.index_select(0, tok))), 2 * H * (T + pairs))
-    add(f"grouped gate|up, {tag}", time_us(lambda: moe_ops.grouped_product(xs, at(gus), rt.blk_expert), iters=16),
-        2 * (pairs * (H + 2 * ff) + used * 2 * ff * H), 4.0 * pairs * H * ff)
-    dense = [r(2 * ff * (top if T > 2048 else E), H) * 0.02 for _ in range(copies)]
+    add(f"grouped {'gate|up' if m.gated else 'up'}, {tag}", time_us(
+        lambda: moe_ops.grouped_product(xs, at(gus), rt.blk_expert), iters=16),
+        2 * (pairs * (H + first) + used * first * H), 2.0 * pairs * H * first)
+    dense = [r(first * (top if T > 2048 else E), H) * 0.02 for _ in range(copies)]
     add("  vs gemm of that size", time_us(lambda: ops.gemm(x, at(dense)), iters=16),
         2 * (T * (H + dense[0].shape[0]) + dense[0].numel()), 2.0 * T * dense[0].numel())
     del dense
     gu = moe_ops.grouped_product(xs, gus[0], rt.blk_expert)
-    add(f"silu_glu of the routed rows, {tag}", time_us(lambda: f("vb_silu_glu")(
-        gu.data_ptr(), 2 * ff, h.data_ptr(), P, ff, scale.data_ptr(), rt.blk_expert.data_ptr(), 0, _lib.stream())), pairs * ff * 6)
+    if m.gated:
+        add(f"silu_glu of the routed rows, {tag}", time_us(lambda: f("vb_silu_glu")(
+            gu.data_ptr(), 2 * ff, h.data_ptr(), P, ff, scale.data_ptr(), rt.blk_expert.data_ptr(), 0, _lib.stream())),
+            pairs * ff * 6)
+    else:
+        add(f"activation of the routed rows ({m.act}), {tag}", time_us(
+            lambda: ops.activation(gu, ff, m.act, rt.blk_expert)), pairs * ff * 4)
     add(f"grouped down, {tag}", time_us(lambda: moe_ops.grouped_product(h, at(downs), rt.blk_expert), iters=16),
         2 * (pairs * (H + ff) + used * ff * H), 2.0 * pairs * H * ff)
     out = moe_ops.grouped_product(h, downs[0], rt.blk_expert)
-    parts = ops.RoutedSum(out, rt, False, r(T, H), logits[:, E])
-    add(f"moe_combine (+ shared, residual, copy), {tag}", time_us(lambda: ops.moe_combine(parts, res, None, 1e-5)),
-        2 * H * (pairs + T) + 10 * T * H)
+    parts = ops.RoutedSum(out, rt, m.weigh == "output", r(T, H), logits[:, E] if m.shared_gate else None)
+    if m.shared_gate:
+        add(f"moe_combine (+ shared, residual, copy), {tag}", time_us(lambda: ops.moe_combine(parts, res, None, 1e-5)),
+            2 * H * (pairs + T) + 10 * T * H)
+    else:
+        g = r(T, H)
+        add(f"moe_norm_add (+ shared, gate, norm, residual, next norm), {tag}", time_us(
+            lambda: ops.moe_norm_add(parts, res, w, 1e-5, final_weight=w, gate=g)), 2 * H * (pairs + 2 * T) + 10 * T * H)
     tw = rt.weight.to(x.dtype).unsqueeze(-1)
     add("  vs sum and residual of the homogeneous models", time_us(lambda: ops.rmsnorm(
         (out.index_select(0, dest).view(T, top, H) * tw).sum(1), w, 1e-5, x)), 2 * H * (pairs + T) + 6 * T * H)
@@ -444,6 +473,24 @@ def _bench_delta(add, r, dl, B: int, n: int, DB: int, ctx: int) -> None:
     add("delta_rule decode (fused step)", time_us(
         lambda: ops.delta_rule(proj[:DB], conv, alog, dt, nw, ring, state, cu1, lens, sl[:DB], 1, *dims)),
         DB * (2 * 4 * dl.heads * dl.dim * dl.vdim + (dl.proj_size + dl.out_size + dl.conv * dl.channels) * 2))
+
+
+def _bench_gla(add, r, m, B: int, n: int, DB: int, ctx: int) -> None:
+    T, nslot = B * n, max(B, DB)
+    proj = r(T, m.proj_size)
+    w, b, nw = r(m.qk_size, m.rank) * m.rank ** -0.5, torch.rand(m.qk_size, device="cuda") * 4, r(m.vdim)
+    state = torch.zeros(nslot, m.heads, m.vdim, m.dim, device="cuda")
+    sl = torch.arange(nslot, device="cuda", dtype=torch.int32)
+    dims = (m.heads, m.dim, m.vdim, m.tau, 1e-5)
+    cu = torch.arange(B + 1, device="cuda", dtype=torch.int32) * n
+    lens = torch.full((B,), n, device="cuda", dtype=torch.int32)
+    add("gated linear attention prefill (chunks, gated norm)", time_us(
+        lambda: ops.gated_linear_attention(proj, w, b, nw, state, cu, lens, sl[:B], n, *dims)),
+        T * (m.proj_size + m.out_size) * 2, 4.0 * T * m.heads * m.dim * m.vdim)
+    cu1, lens1 = torch.arange(DB + 1, device="cuda", dtype=torch.int32), torch.full((DB,), ctx, device="cuda", dtype=torch.int32)
+    add("gated linear attention decode (fused step)", time_us(
+        lambda: ops.gated_linear_attention(proj[:DB], w, b, nw, state, cu1, lens1, sl[:DB], 1, *dims)),
+        DB * (2 * 4 * m.heads * m.dim * m.vdim + (m.proj_size + m.out_size) * 2))
 
 
 def main(args) -> dict:
