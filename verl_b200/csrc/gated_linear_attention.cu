@@ -272,417 +272,453 @@ __global__ void __launch_bounds__(GS_THREADS) gla_scan_kernel(const GlaParams p)
 // A chunk takes up to 64 tokens, fewer where a channel decays so far that e^{-b} would leave fp32's range: the walk then
 // goes on behind the tokens it has taken, whatever their number.
 //
-// One CTA of sixteen warps per (sequence, head, 128 state columns); tcgen05 with accumulators in TMEM (tokens = columns):
+// One CTA per (sequence, head, 128 state columns); tcgen05 with accumulators in TMEM (tokens = columns):
 //     Z^T [d, t]      = W . r^T                                  (W in TMEM; the decays' logits)
 //     P^T [s | s, t]  = [K~ hi; K~ lo] . (Q~ hi + Q~ lo)^T       (two partial sums of each score, added by the last product)
 //     S^T [v, d]     += V^T . (K~ hi + K~ lo)                    (fp32 state in TMEM, decayed when it is read)
-//     O^T [v, t]      = S0^T hi . (Q~ hi + Q~ lo)^T + S0^T lo . Q~ hi^T
+//     O^T [v, t]      = S0^T hi . (Q~ hi + Q~ lo)^T + S0^T lo . Q~ hi^T   (S0^T in TMEM)
 //     O^T [v, t]     += [V; V]^T . P hi + V^T . P lo             (P: causal part of the scores)
 // Every fp32 operand enters as two bf16 terms, so that products carry about 16 bits of both operands and sums are fp32; v and the
-// numbers r are bf16 activations. Warp w owns TMEM lanes 32 (w % 4) .. and a quarter of the columns of each accumulator; three
-// warps issue the products. While the tensor cores work on a chunk, the decays of the next one are computed, and its q, k and r
-// arrive.
-constexpr int GK_C = 64, GK_THREADS = 512;
-constexpr int GK_Q_OFF = 0;                        // Q~: per 64 channels hi | lo, [64 tokens] x 128 bytes
-constexpr int GK_K_OFF = 32768;                    // K~: the same
-constexpr int GK_V_OFF = GK_K_OFF + 32768;         // v [64 tokens][128], two column blocks
-constexpr int GK_S_OFF = GK_V_OFF + 16384;         // S^T [128 v][128 d]: per 64 channels hi | lo
-constexpr int GK_P_OFF = GK_S_OFF + 65536;         // P hi [128 s][64 t] | P lo [64 s][64 t]; then the outputs [64 t][128 v]
-constexpr int GK_R_OFF = GK_P_OFF + 24576;         // q | k as they are, [64 tokens][128] each
+// numbers r are bf16 activations.
+// Warps 0..15 make Q~ and K~ of chunk after chunk (two of them in shared memory), warps 16..23 turn scores into P, decay the state
+// and store the outputs, warp 24 issues the products (but Z, which warp 0 does). A warp reads the TMEM lanes 32 (w % 4) ..; those
+// of a group that share them have equal parts of the columns. q, k, v and r arrive by TMA.
+constexpr int GK_C = 64, GK_MAKERS = 512, GK_USERS = 256, GK_THREADS = GK_MAKERS + GK_USERS + 32;
+constexpr int GK_BUF = 32768;                      // Q~ or K~ of a chunk: per 64 channels hi | lo, [64 tokens] x 128 bytes
+constexpr int GK_Q_OFF = 0, GK_K_OFF = 2 * GK_BUF;
+constexpr int GK_V_OFF = GK_K_OFF + 2 * GK_BUF;    // v [64 tokens][128], two column blocks
+constexpr int GK_P_OFF = GK_V_OFF + 16384;         // P hi [128 s][64 t] | P lo [64 s][64 t]
+constexpr int GK_R_OFF = GK_P_OFF + 24576;         // q | k as they are, column blocks of 64: [64 tokens] x 128 bytes
 constexpr int GK_A_OFF = GK_R_OFF + 32768;         // r [64 tokens][64]
 constexpr int GK_SUM_OFF = GK_A_OFF + 8192;        // log decays of 16 tokens, [4][128] fp32
-constexpr int GK_DEC_OFF = GK_SUM_OFF + 2048;      // e^{b_last} [128]
-constexpr int GK_BAR_OFF = GK_DEC_OFF + 512;
-constexpr int GK_SMEM = GK_BAR_OFF + 64 + 1024;
-constexpr uint32_t GK_SC = 0, GK_O = 64, GK_ST = 128, GK_Z = 256, GK_W = 320;  // TMEM columns
-constexpr float GK_RANGE = 90.f;                   // log2 of the largest e^{-b}
-constexpr float GK_FLOOR = -64.f;                  // log2 of the strongest decay of a token: what is left does not show in fp32
+constexpr int GK_DEC_OFF = GK_SUM_OFF + 2048;      // e^{b_last} [128] of four chunks
+constexpr int GK_BAR_OFF = GK_DEC_OFF + 2048;
+constexpr int GK_SMEM = GK_BAR_OFF + 256 + 1024;
+constexpr uint32_t GK_SC = 0, GK_O = 64, GK_ST = 128, GK_Z = 256, GK_W = 320, GK_SH = 352, GK_SL = 416;  // TMEM columns
+constexpr float GK_RANGE = 90.f;                   // log2 of the largest e^{-b}: a stronger decay of one token does not show in fp32
 
 __device__ __forceinline__ float ex2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-// log(sigmoid(z)): log(1 + u) = 2 atanh(s), s = u / (2 + u), u = e^-|z| <= 1; atanh(s) / s by a polynomial in s^2 fitted on
-// [0, 1/9] (relative error 2e-8)
-__device__ __forceinline__ float log_sigmoid_fast(float z) {
-  const float u = __expf(-fabsf(z)), s = __fdividef(u, 2.f + u), t = s * s;
-  const float y = fmaf(t, fmaf(t, fmaf(t, fmaf(t, 0.13433777f, 0.14116978f), 0.20003835f), 0.3333332f), 1.f);
-  return fmaf(-2.f * s, y, fminf(z, 0.f));
+__device__ __forceinline__ float lg2(float x) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// Barrier of the threads that make Q~ and K~, which also and-reduces a predicate.
+__device__ __forceinline__ bool gk_bar_and(bool pred) {
+  uint32_t r;
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\tsetp.ne.u32 q, %1, 0;\n\tbarrier.red.and.pred p, 1, 512, q;\n\tselp.u32 %0, 1, 0, p;\n\t}"
+      : "=r"(r)
+      : "r"((uint32_t)pred)
+      : "memory");
+  return r != 0;
 }
 
 // ND: channels with those that are zero, 64 or 128
 template <int ND>
-__global__ void __launch_bounds__(GK_THREADS, 1) gla_chunk_kernel(const GlaParams p, int* status) {
+__global__ void __launch_bounds__(GK_THREADS, 1)
+gla_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
+                 const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmR, const GlaParams p, int* status) {
   extern __shared__ uint8_t smb[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smb) + 1023) & ~uintptr_t(1023));
-  // completed products: Z, scores, O of the state, state, O
-  enum { Z_DONE, SC_DONE, IN_DONE, ST_DONE, O_DONE, NBAR };
+  // Arrivals: by a copy (in), by the products (done), by the warps of a group. Barriers in pairs belong to chunks in turn.
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + GK_BAR_OFF);
+  uint64_t *r_in = bars, *qk_in = bars + 1, *v_in = bars + 2, *z_done = bars + 3, *sc_done = bars + 4, *s_done = bars + 5,
+           *o_done = bars + 7;                                                    // s_done: state and O of the state
+  uint64_t *qk_made = bars + 9, *p_made = bars + 11, *s_made = bars + 12, *o_read = bars + 13;
+  constexpr int NBAR = 14;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + NBAR);
-  int* far = reinterpret_cast<int*>(tmem_slot + 1);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  int* far = reinterpret_cast<int*>(tmem_slot + 2);
+  int* cnt_s = reinterpret_cast<int*>(tmem_slot + 4);  // [4] tokens of a chunk
   float* sum_s = reinterpret_cast<float*>(smem + GK_SUM_OFF);
-  float* dec_s = reinterpret_cast<float*>(smem + GK_DEC_OFF);
   pdl_wait();
   const int v0 = blockIdx.x * 128, h = blockIdx.y, b = p.b0 + blockIdx.z;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, quad = warp & 3, grp = warp >> 2;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, quad = warp & 3;
   const int first = p.cu_q[b], n = p.cu_q[b + 1] - first, slot = p.slots[b];
   if (n <= 0 || slot < 0) return;  // uniform for the CTA, before any barrier or allocation
-  const int start = p.seq_lens[b] - n, HD = p.H * p.D, HV = p.H * p.V;
-  const __nv_bfloat16* proj = static_cast<const __nv_bfloat16*>(p.proj) + (long long)first * p.stride;
+  const int start = p.seq_lens[b] - n;
   const int VC = min(128, p.V - v0);             // columns of this CTA
 
   if (tid == 0) {
-    for (int i = 0; i < NBAR; ++i) mbar_init(&bars[i], 1);
+    for (int i = 0; i < NBAR; ++i) mbar_init(&bars[i], i < 9 ? 1 : i < 11 ? GK_MAKERS / 32 : GK_USERS / 32);
+    *abort_flag = 0;
     *far = 0;
     mbar_fence_init();
   }
-  if (warp == 0) {
+  if (warp == 24) {
     tmem_alloc(tmem_slot, 512);
     tmem_relinquish();
   }
-  // q and k of the tokens from t0 on; 16-byte groups of a row swapped by fours, so that two rows are read without conflicts
-  auto load_qk = [&](int t0) {
-    constexpr int GROUPS = ND / 8;
-#pragma unroll
-    for (int i = tid; i < GK_C * GROUPS; i += GK_THREADS) {
-      const int t = i / GROUPS, g = i % GROUPS;
-      const bool on = t0 + t < n && g * 8 < p.D;
-      const __nv_bfloat16* src = proj + (on ? (long long)(t0 + t) * p.stride + h * p.D + g * 8 : 0);
-      uint8_t* to = smem + GK_R_OFF + t * 256 + ((g ^ (t & 4)) << 4);
-      cp_async16(to, src, on);
-      cp_async16(to + 16384, on ? src + HD : src, on);
-    }
-    cp_async_commit();
-  };
-  auto load_r = [&](int t0) {
-    const __nv_bfloat16* r = proj + 2 * (HD + HV);
-    if ((p.rank & 7) == 0) {
-      const int t = tid >> 3, g = tid & 7;  // 64 tokens, 8 groups of eight
-      const bool on = t0 + t < n && g * 8 < p.rank;
-      cp_async16(smem + GK_A_OFF + t * 128 + ((g ^ (t & 7)) << 4), r + (on ? (long long)(t0 + t) * p.stride + g * 8 : 0), on);
-    } else {
-      for (int i = tid; i < GK_C * 64; i += GK_THREADS) {
-        const int t = i >> 6, c = i & 63;
-        const bool on = t0 + t < n && c < p.rank;
-        *reinterpret_cast<__nv_bfloat16*>(smem + GK_A_OFF + t * 128 + (((c >> 3) ^ (t & 7)) << 4) + (c & 7) * 2) =
-            on ? r[(long long)(t0 + t) * p.stride + c] : __float2bfloat16(0.f);
-      }
-    }
-    cp_async_commit();
-  };
-  auto load_v = [&](int t0) {
-#pragma unroll
-    for (int i = tid; i < GK_C * 16; i += GK_THREADS) {
-      const int t = i >> 4, g = i & 15;
-      const bool on = t0 + t < n && g * 8 < VC;
-      cp_async16(smem + GK_V_OFF + (g >> 3) * 8192 + t * 128 + (((g & 7) ^ (t & 7)) << 4),
-                 proj + (on ? (long long)(t0 + t) * p.stride + 2 * HD + h * p.V + v0 + g * 8 : 0), on);
-    }
-    cp_async_commit();
-  };
-  load_r(0);
-  load_qk(0);
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = *tmem_slot, my = tmem + ((uint32_t)(quad * 32) << 16);
   pdl_trigger();  // TMEM is held
-
   const int row = quad * 32 + lane;              // TMEM lane: channel d, state column v or token s
-  // this thread's channel: its row of W (by the first quarter of the warps) and its bias
-  const bool d_on = row < p.D;
-  const float bias = d_on ? p.decay_b[h * p.D + row] : 0.f;
-  if (grp == 0) {
-    uint32_t w[32];
-    const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(p.decay_w) + (long long)(h * p.D + (d_on ? row : 0)) * p.rank;
-#pragma unroll
-    for (int i = 0; i < 32; ++i)
-      w[i] = pack_bf16x2(d_on && 2 * i < p.rank ? dl_f(src[2 * i]) : 0.f, d_on && 2 * i + 1 < p.rank ? dl_f(src[2 * i + 1]) : 0.f);
-    tmem_st_32x32(my + GK_W, w);
-  }
-  // 32 fp32 values as two bf16 terms into four 16-byte groups of a 128-byte row, starting at group g0
-  auto put32 = [&](uint8_t* hi_row, uint8_t* lo_row, int g0, const float (&f)[32]) {
-#pragma unroll
-    for (int g = 0; g < 4; ++g) {
-      uint32_t hi[4], lo[4];
-#pragma unroll
-      for (int k = 0; k < 4; ++k) split2(f[8 * g + 2 * k], f[8 * g + 2 * k + 1], hi[k], lo[k]);
-      const int off = ((g0 + g) ^ (row & 7)) << 4;
-      *reinterpret_cast<uint4*>(hi_row + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-      *reinterpret_cast<uint4*>(lo_row + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
-    }
+  auto wait = [&](uint64_t* bar, uint32_t parity, int detail) {
+    if (!*abort_flag && mbar_wait(bar, parity)) return true;
+    report_error(status, ERR_WAIT_TMEM_FULL, detail);
+    *abort_flag = 1;
+    return false;
   };
-  // the state: this thread's column v and channels c0 .. c0 + 31
-  const int c0 = grp * 32;
-  const bool s_on = c0 < ND;
-  float* st = p.state + (((long long)slot * p.H + h) * p.V + v0 + row) * p.D;
-  uint8_t* s_hi = smem + GK_S_OFF + (c0 >> 6) * 32768 + row * 128;
-  if (s_on) {
-    float f[32];
-    uint32_t w[32];
-#pragma unroll
-    for (int e = 0; e < 32; ++e) {
-      f[e] = start > 0 && row < VC && c0 + e < p.D ? st[c0 + e] : 0.f;
-      w[e] = __float_as_uint(f[e]);
-    }
-    put32(s_hi, s_hi + 16384, (c0 & 32) >> 3, f);
-    tmem_st_32x32(my + GK_ST + c0, w);
-  }
-  tmem_st_wait();
-
-  const uint32_t base = smem_u32(smem);
-  constexpr int K_STEPS = ND / 16;
-  constexpr uint32_t id_kk = umma_idesc(1, 1, 0, 0, 128, 64);           // both K-major
-  constexpr uint32_t id_mm = umma_idesc(1, 1, 1, 1, 128, 64);           // both MN-major
-  constexpr uint32_t id_st = umma_idesc(1, 1, 1, 1, 128, ND);
-  // operands: a step of 32 bytes (K-major) or 2048 bytes (MN-major) adds to the address field of a descriptor
-  const uint64_t dq = umma_smem_desc(base + GK_Q_OFF, 16, 1024), dk = umma_smem_desc(base + GK_K_OFF, 16, 1024),
-                 dk_mn = umma_smem_desc(base + GK_K_OFF, 16384, 1024), ds = umma_smem_desc(base + GK_S_OFF, 16, 1024),
-                 dv = umma_smem_desc(base + GK_V_OFF, 8192, 1024), dp = umma_smem_desc(base + GK_P_OFF, 8192, 1024),
-                 da = umma_smem_desc(base + GK_A_OFF, 16, 1024);
-  const int r_steps = (p.rank + 15) / 16;
-  const float qscale = 1.f / sqrtf((float)p.D), rate = p.inv_tau * 1.4426950408889634f;
-  bool ok = true;
-  // every thread waits for products; one failed wait ends the loop for the whole CTA
-  auto wait = [&](int i, uint32_t parity, int detail) {
-    bool good = false;  // a few products take microseconds: bounded by attempts, without reading the clock
-    for (int a = 0; a < (1 << 22) && !good; ++a) good = mbar_try_wait(&bars[i], parity);
-    if (!good) report_error(status, ERR_WAIT_TMEM_FULL, detail);
-    tc_fence_after();
-    ok = good && ok;
-  };
-  auto issue_z = [&]() {
-    for (int k = 0; k < r_steps; ++k) tc_mma_f16_ta(tmem + GK_Z, tmem + GK_W + k * 8, da + k * 2, id_kk, k != 0);
-    tc_commit(&bars[Z_DONE]);
-  };
-  // Running log2 decays of this thread's channel over its sixteen tokens of the chunk at t0; tokens that the chunk takes.
-  float lb[16];
-  auto decays = [&](int t0, uint32_t parity) {
-    wait(Z_DONE, parity, t0);
-    {
-      uint32_t z[16];
-      tmem_ld_32x16(my + GK_Z + grp * 16, z);
-      tmem_ld_wait();
-      const int in = d_on ? n - t0 - grp * 16 : 0;
-      float run = 0.f;
-#pragma unroll
-      for (int i = 0; i < 16; ++i) {
-        const float l = fmaxf(log_sigmoid_fast(__uint_as_float(z[i]) + bias) * rate, GK_FLOOR);
-        run += i < in ? l : 0.f;
-        lb[i] = run;
-      }
-      sum_s[grp * 128 + row] = run;
-    }
-    __syncthreads();
-    float total = 0.f, before = 0.f;
-#pragma unroll
-    for (int g = 0; g < 4; ++g) {
-      const float x = sum_s[g * 128 + row];
-      total += x;
-      if (g < grp) before += x;
-    }
-#pragma unroll
-    for (int i = 0; i < 16; ++i) lb[i] += before;
-    int cnt = min(GK_C, n - t0);
-    if (!__syncthreads_and(total >= -GK_RANGE)) {  // the largest power of two of them that stays within the range
-      int out = 0;
-#pragma unroll
-      for (int k = 0; k < 6; ++k) {
-        const int t = (1 << k) - 1;
-        if ((t >> 4) == grp && lb[t & 15] < -GK_RANGE) out |= 1 << k;
-      }
-      if (out) atomicOr(far, out);
-      __syncthreads();
-      out = *far;
-      int m = 1;
-      while (m < 32 && !(out & (2 * m))) m *= 2;
-      cnt = min(cnt, m);
-      __syncthreads();
-      if (tid == 0) *far = 0;
-    }
-    return cnt;
-  };
-
-  cp_async_wait<1>();  // r
-  fence_proxy_async_smem();
-  tc_fence_before();
-  __syncthreads();
-  if (warp == 0 && elect_one()) {
-    tc_fence_after();
-    issue_z();
-  }
-  int t0 = 0, cnt = decays(0, 0);
-  load_r(cnt);
-  cp_async_wait<1>();  // q and k
-  __syncthreads();
-  load_v(0);
-  for (uint32_t it = 0; t0 < n; ++it) {
-    const uint32_t parity = it & 1;
-    // Q~ and K~: lanes in pairs, each lane two channels of eight tokens: the even one of the first eight of the sixteen
-    if (row < ND) {
-      const bool odd = lane & 1;
-      const int d = row & ~1, g = d >> 3;
-#pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        const float own = odd ? lb[8 + (j ^ 4)] : lb[j], give = odd ? lb[j] : lb[8 + (j ^ 4)];
-        const float got = __shfl_xor_sync(0xffffffffu, give, 1);
-        const float b0 = odd ? got : own, b1 = odd ? own : got;
-        const int t = grp * 16 + (odd ? 8 + (j ^ 4) : j);
-        const uint8_t* raw = smem + GK_R_OFF + t * 256 + ((g ^ (t & 4)) << 4) + (d & 7) * 2;
-        const uint32_t q2 = *reinterpret_cast<const uint32_t*>(raw), k2 = *reinterpret_cast<const uint32_t*>(raw + 16384);
-        const float e0 = ex2(b0), e1 = ex2(b1);
-        if (t == cnt - 1) *reinterpret_cast<float2*>(dec_s + d) = make_float2(e0, e1);
-        uint32_t qh = 0, ql = 0, kh = 0, kl = 0;
-        if (t < cnt) {
-          split2(__uint_as_float(q2 << 16) * (qscale * e0), __uint_as_float(q2 & 0xffff0000u) * (qscale * e1), qh, ql);
-          split2(__uint_as_float(k2 << 16) * ex2(-b0), __uint_as_float(k2 & 0xffff0000u) * ex2(-b1), kh, kl);
-        }
-        uint8_t* to = smem + (g >> 3) * 16384 + t * 128 + (((g & 7) ^ (t & 7)) << 4) + (d & 7) * 2;
-        *reinterpret_cast<uint32_t*>(to + GK_Q_OFF) = qh;
-        *reinterpret_cast<uint32_t*>(to + GK_Q_OFF + 8192) = ql;
-        *reinterpret_cast<uint32_t*>(to + GK_K_OFF) = kh;
-        *reinterpret_cast<uint32_t*>(to + GK_K_OFF + 8192) = kl;
-      }
-    }
-    cp_async_wait<0>();  // v; r of the next chunk
+  // what a warp has written to shared memory and read from TMEM is done: tell the barrier
+  auto arrive = [&](uint64_t* bar) {
     fence_proxy_async_smem();
     tc_fence_before();
-    if (!__syncthreads_and(ok)) break;
-    const int t1 = t0 + cnt;
+    __syncwarp();
+    if (lane == 0) mbar_arrive(bar);
+  };
+
+  if (warp < 16) {
+    // ----------------------------- Q~ and K~ (thread = channel, 16 tokens) -----------------------------
+    const int grp = warp >> 2;
+    const bool d_on = row < p.D;
+    constexpr float LOG2E = 1.4426950408889634f;
+    const float bias = d_on ? p.decay_b[h * p.D + row] * LOG2E : 0.f;
+    const float qscale = 1.f / sqrtf((float)p.D);
+    const int r_steps = (p.rank + 15) / 16;
+    int loads_r = 0, loads_qk = 0;
+    auto load_r = [&](int t0) {
+      mbar_arrive_expect_tx(r_in, 8192);
+      tma_load_2d(smem + GK_A_OFF, &tmR, r_in, 0, first + t0);
+      ++loads_r;
+    };
     if (warp == 0) {
       if (elect_one()) {
-        tc_fence_after();
-        if (t1 < n) issue_z();
-#pragma unroll
-        for (int term = 0; term < 2; ++term)
-#pragma unroll
-          for (int k = 0; k < K_STEPS; ++k)
-            tc_mma_f16(tmem + GK_SC, dk + (k >> 2) * 1024 + (k & 3) * 2, dq + term * 512 + (k >> 2) * 1024 + (k & 3) * 2, id_kk,
-                       term != 0 || k != 0);
-        tc_commit(&bars[SC_DONE]);
+        tma_prefetch_desc(&tmQ);
+        tma_prefetch_desc(&tmK);
+        tma_prefetch_desc(&tmR);
+        load_r(0);
       }
-    } else if (warp == 1) {
-      if (elect_one()) {
-        tc_fence_after();
-#pragma unroll
-        for (int term = 0; term < 3; ++term)  // hi hi, hi lo, lo hi
-#pragma unroll
-          for (int k = 0; k < K_STEPS; ++k)
-            tc_mma_f16(tmem + GK_O, ds + (term == 2 ? 1024 : 0) + (k >> 2) * 2048 + (k & 3) * 2,
-                       dq + (term == 1 ? 512 : 0) + (k >> 2) * 1024 + (k & 3) * 2, id_kk, term != 0 || k != 0);
-        tc_commit(&bars[IN_DONE]);
-      }
-    } else if (warp == 2) {
-      if (elect_one()) {
-        tc_fence_after();
-#pragma unroll
-        for (int term = 0; term < 2; ++term)
-#pragma unroll
-          for (int k = 0; k < GK_C / 16; ++k)
-            tc_mma_f16(tmem + GK_ST, dv + k * 128, dk_mn + term * 512 + k * 128, id_st, 1);
-        tc_commit(&bars[ST_DONE]);
-      }
+      __syncwarp();
     }
-    __syncwarp();
-    load_qk(t1);
-    int next = 0;
-    if (t1 < n) next = decays(t1, parity ^ 1);
-    load_r(t1 + next);
-    // scores: this thread's row s (hi or lo term of K~) and sixteen tokens t
-    wait(SC_DONE, parity, t0 + 1);
-    {
-      uint32_t x[16];
-      tmem_ld_32x16(my + GK_SC + grp * 16, x);
-      tmem_ld_wait();
-      const int s = row & 63;
-      uint8_t* dst = smem + GK_P_OFF + row * 128;
+    if (grp == 0) {  // this channel's row of W
+      uint32_t w[32];
+      const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(p.decay_w) + (long long)(h * p.D + (d_on ? row : 0)) * p.rank;
 #pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        uint32_t hi[4], lo[4];
-#pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          const int e = 8 * j + 2 * k, t = grp * 16 + e;
-          split2(t >= s ? __uint_as_float(x[e]) : 0.f, t + 1 >= s ? __uint_as_float(x[e + 1]) : 0.f, hi[k], lo[k]);
-        }
-        const int off = ((2 * grp + j) ^ (row & 7)) << 4;
-        *reinterpret_cast<uint4*>(dst + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-        if (quad < 2) *reinterpret_cast<uint4*>(dst + 16384 + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
-      }
-    }
-    fence_proxy_async_smem();
-    tc_fence_before();
-    if (!__syncthreads_and(ok)) break;
-    if (warp == 1) {  // the one that has issued O of the state
-      if (elect_one()) {
-        tc_fence_after();
-#pragma unroll
-        for (int k = 0; k < 12; ++k)  // P hi of both partial sums, P lo of the first
-          tc_mma_f16(tmem + GK_O, dv + (k & 3) * 128, dp + k * 128, id_mm, 1);
-        tc_commit(&bars[O_DONE]);
-      }
-    }
-    __syncwarp();
-    // the state behind the chunk
-    wait(ST_DONE, parity, t0 + 2);
-    wait(IN_DONE, parity, t0 + 3);
-    if (s_on) {
-      uint32_t x[32];
-      tmem_ld_32x32(my + GK_ST + c0, x);
-      tmem_ld_wait();
-      float f[32];
-#pragma unroll
-      for (int e = 0; e < 32; e += 4) {
-        const float4 d4 = *reinterpret_cast<const float4*>(dec_s + c0 + e);
-        f[e] = __uint_as_float(x[e]) * d4.x;
-        f[e + 1] = __uint_as_float(x[e + 1]) * d4.y;
-        f[e + 2] = __uint_as_float(x[e + 2]) * d4.z;
-        f[e + 3] = __uint_as_float(x[e + 3]) * d4.w;
-      }
-      if (t1 >= n) {
-        if (ok && row < VC)
-#pragma unroll
-          for (int e = 0; e < 32; ++e)
-            if (c0 + e < p.D) st[c0 + e] = f[e];
-      } else {
-        put32(s_hi, s_hi + 16384, (c0 & 32) >> 3, f);
-#pragma unroll
-        for (int e = 0; e < 32; ++e) x[e] = __float_as_uint(f[e]);
-        tmem_st_32x32(my + GK_ST + c0, x);
-      }
+      for (int i = 0; i < 32; ++i)
+        w[i] = pack_bf16x2(d_on && 2 * i < p.rank ? dl_f(src[2 * i]) : 0.f, d_on && 2 * i + 1 < p.rank ? dl_f(src[2 * i + 1]) : 0.f);
+      tmem_st_32x32(my + GK_W, w);
       tmem_st_wait();
     }
-    wait(O_DONE, parity, t0 + 4);
-    {
+    constexpr uint32_t id_z = umma_idesc(1, 1, 0, 0, 128, 64);
+    const uint64_t da = umma_smem_desc(smem_u32(smem) + GK_A_OFF, 16, 1024);
+    bool ok = true;
+    int t0 = 0;
+    for (int c = 0; t0 < n; ++c) {
+      tc_fence_before();
+      ok = gk_bar_and(ok);  // everyone is through with q and k of the chunk before
+      if (!ok) break;
+      if (warp == 0) {
+        if (elect_one()) {
+          mbar_arrive_expect_tx(qk_in, 2 * (ND / 64) * 8192);
+#pragma unroll
+          for (int x = 0; x < ND / 64; ++x) {
+            tma_load_3d(smem + GK_R_OFF + x * 8192, &tmQ, qk_in, x * 64, h, first + t0);
+            tma_load_3d(smem + GK_R_OFF + 16384 + x * 8192, &tmK, qk_in, x * 64, h, first + t0);
+          }
+          ++loads_qk;
+          if (wait(r_in, c & 1, t0)) {
+            tc_fence_after();
+            for (int k = 0; k < r_steps; ++k) tc_mma_f16_ta(tmem + GK_Z, tmem + GK_W + k * 8, da + k * 2, id_z, k != 0);
+            tc_commit(z_done);
+          }
+        }
+        __syncwarp();
+      }
+      // running log2 decays of this thread's channel over its tokens
+      float lb[16];
+      ok = wait(z_done, c & 1, t0 + 1);
+      tc_fence_after();
+      {
+        uint32_t z[16];
+        tmem_ld_32x16(my + GK_Z + grp * 16, z);
+        tmem_ld_wait();
+        const int in = d_on ? n - t0 - grp * 16 : 0;
+        float run = 0.f;
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {  // log2 sigmoid(z) = min(z', 0) - log2(1 + 2^-|z'|), z' = z log2(e)
+          const float y = fmaf(__uint_as_float(z[i]), LOG2E, bias);
+          const float l = (fminf(y, 0.f) - lg2(1.f + ex2(-fabsf(y)))) * p.inv_tau;
+          run += i < in ? l : 0.f;
+          lb[i] = run;
+        }
+        sum_s[grp * 128 + row] = run;
+      }
+      gk_bar_and(true);
+      {
+        float before = 0.f;
+#pragma unroll
+        for (int g = 0; g < 3; ++g)
+          if (g < grp) before += sum_s[g * 128 + row];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) lb[i] += before;
+      }
+      int cnt = min(GK_C, n - t0);  // tokens of this chunk
+      if (!gk_bar_and(lb[15] >= -GK_RANGE)) {  // the largest power of two of them that stays within the range
+        int out = 0;
+#pragma unroll
+        for (int k = 0; k < 6; ++k) {
+          const int t = (1 << k) - 1;
+          if ((t >> 4) == grp && lb[t & 15] < -GK_RANGE) out |= 1 << k;
+        }
+        if (out) atomicOr(far, out);
+        gk_bar_and(true);
+        out = *far;
+        int m = 1;
+        while (m < 32 && !(out & (2 * m))) m *= 2;
+        cnt = min(cnt, m);
+#pragma unroll
+        for (int i = 0; i < 16; ++i) lb[i] = fmaxf(lb[i], -GK_RANGE);
+        gk_bar_and(true);
+        if (tid == 0) *far = 0;
+      }
+      const int t1 = t0 + cnt, buf = c & 1;
+      if (warp == 0) {
+        if (elect_one() && t1 < n) load_r(t1);
+        __syncwarp();
+      }
+      // everyone is through with chunk c - 2 (O is the last that is made of it)
+      if (c > 1) ok = wait(&o_done[buf], ((c >> 1) + 1) & 1, t0 + 2) && ok;
+      ok = wait(qk_in, c & 1, t0 + 3) && ok;
+      // lanes in pairs, each lane two channels of eight tokens: the even one the first eight of the sixteen
+      if (row < ND) {
+        const bool odd = lane & 1;
+        const int d = row & ~1, g = (d >> 3) & 7;
+        float* dec = reinterpret_cast<float*>(smem + GK_DEC_OFF) + (c & 3) * 128 + d;
+        uint8_t* dst = smem + buf * GK_BUF + (d >> 6) * 16384 + (d & 7) * 2;
+        const uint8_t* src = smem + GK_R_OFF + (d >> 6) * 8192 + (d & 7) * 2;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          const float own = odd ? lb[8 + (j ^ 4)] : lb[j], give = odd ? lb[j] : lb[8 + (j ^ 4)];
+          const float got = __shfl_xor_sync(0xffffffffu, give, 1);
+          const float b0 = odd ? got : own, b1 = odd ? own : got;
+          const int t = grp * 16 + (odd ? 8 + (j ^ 4) : j);
+          const int at = t * 128 + ((g ^ (t & 7)) << 4);
+          const uint32_t q2 = *reinterpret_cast<const uint32_t*>(src + at), k2 = *reinterpret_cast<const uint32_t*>(src + 16384 + at);
+          const float e0 = ex2(b0), e1 = ex2(b1);
+          if (t == cnt - 1) *reinterpret_cast<float2*>(dec) = make_float2(e0, e1);
+          uint32_t qh = 0, ql = 0, kh = 0, kl = 0;
+          if (t < cnt) {
+            split2(__uint_as_float(q2 << 16) * (qscale * e0), __uint_as_float(q2 & 0xffff0000u) * (qscale * e1), qh, ql);
+            split2(__uint_as_float(k2 << 16) * ex2(-b0), __uint_as_float(k2 & 0xffff0000u) * ex2(-b1), kh, kl);
+          }
+          *reinterpret_cast<uint32_t*>(dst + at + GK_Q_OFF) = qh;
+          *reinterpret_cast<uint32_t*>(dst + at + GK_Q_OFF + 8192) = ql;
+          *reinterpret_cast<uint32_t*>(dst + at + GK_K_OFF) = kh;
+          *reinterpret_cast<uint32_t*>(dst + at + GK_K_OFF + 8192) = kl;
+        }
+      }
+      if (tid == 0) cnt_s[c & 3] = cnt;
+      arrive(&qk_made[buf]);
+      t0 = t1;
+    }
+    // no copy is in flight when the CTA ends, whatever ended it
+    if (loads_qk > 0) mbar_wait(qk_in, (loads_qk - 1) & 1);
+    if (loads_r > 0) mbar_wait(r_in, (loads_r - 1) & 1);
+  } else if (warp < 24) {
+    // ------------------------- P, the state, the outputs (every warp on its own) -------------------------
+    const int half = (warp >> 2) & 1;
+    int loads_v = 0;
+    auto load_v = [&](int t0) {
+      if (warp == 16) {
+        if (elect_one()) {
+          mbar_arrive_expect_tx(v_in, 16384);
+          tma_load_3d(smem + GK_V_OFF, &tmV, v_in, v0, h, first + t0);
+          tma_load_3d(smem + GK_V_OFF + 8192, &tmV, v_in, v0 + 64, h, first + t0);
+          ++loads_v;
+        }
+        __syncwarp();
+      }
+    };
+    load_v(0);
+    float* st = p.state + (((long long)slot * p.H + h) * p.V + v0 + row) * p.D;
+    constexpr int SR = ND / 32;  // this thread's channels of column v, 16 at a time
+    // fp32 accumulator and two bf16 terms of 16 channels
+    auto put_state = [&](int c0, const float (&f)[16]) {
       uint32_t x[16];
-      tmem_ld_32x16(my + GK_O + grp * 16, x);
-      tmem_ld_wait();
-      __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(smem + GK_P_OFF) + row;
 #pragma unroll
-      for (int e = 0; e < 16; ++e) o[(grp * 16 + e) * 128] = __float2bfloat16(__uint_as_float(x[e]));
-    }
-    cp_async_wait<1>();  // q and k of the next chunk (the newest group is r)
-    tc_fence_before();
-    if (!__syncthreads_and(ok)) break;
-    load_v(t1);
-    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (long long)(first + t0) * p.out_stride + (long long)h * p.V + v0;
+      for (int e = 0; e < 16; ++e) x[e] = __float_as_uint(f[e]);
+      tmem_st_32x16(my + GK_ST + c0, x);
 #pragma unroll
-    for (int i = tid; i < GK_C * 16; i += GK_THREADS) {
-      const int t = i >> 4, g = i & 15;
-      if (t < cnt && g * 8 < VC)
-        *reinterpret_cast<uint4*>(out + (long long)t * p.out_stride + g * 8) =
-            *reinterpret_cast<const uint4*>(smem + GK_P_OFF + t * 256 + g * 16);
+      for (int e = 0; e < 8; ++e) split2(f[2 * e], f[2 * e + 1], x[e], x[8 + e]);
+      tmem_st_32x8(my + GK_SH + c0 / 2, x);
+      tmem_st_32x8(my + GK_SL + c0 / 2, x + 8);
+    };
+#pragma unroll
+    for (int k = 0; k < SR; ++k) {
+      const int c0 = (half * SR + k) * 16;
+      float f[16];
+#pragma unroll
+      for (int e = 0; e < 16; ++e) f[e] = start > 0 && row < VC && c0 + e < p.D ? st[c0 + e] : 0.f;
+      put_state(c0, f);
     }
-    t0 = t1;
-    cnt = next;
+    tmem_st_wait();
+    arrive(s_made);
+    int t0 = 0;
+    for (int c = 0; t0 < n; ++c) {
+      const int buf = c & 1;
+      // scores: this thread's row s (hi or lo term of K~) and 32 tokens t
+      if (!__all_sync(0xffffffffu, wait(&qk_made[buf], (c >> 1) & 1, t0 + 4) && wait(sc_done, c & 1, t0 + 5))) break;
+      tc_fence_after();
+      const int cnt = cnt_s[c & 3], t1 = t0 + cnt;
+      {
+        uint32_t x[32];
+        tmem_ld_32x32(my + GK_SC + half * 32, x);
+        tmem_ld_wait();
+        const int s = row & 63;
+        uint8_t* dst = smem + GK_P_OFF + row * 128;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          uint32_t hi[4], lo[4];
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const int e = 8 * j + 2 * k, t = half * 32 + e;
+            split2(t >= s ? __uint_as_float(x[e]) : 0.f, t + 1 >= s ? __uint_as_float(x[e + 1]) : 0.f, hi[k], lo[k]);
+          }
+          const int off = ((4 * half + j) ^ (row & 7)) << 4;
+          *reinterpret_cast<uint4*>(dst + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+          if (quad < 2) *reinterpret_cast<uint4*>(dst + 16384 + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+        }
+      }
+      arrive(p_made);
+      // the state behind the chunk
+      if (!__all_sync(0xffffffffu, wait(&s_done[buf], (c >> 1) & 1, t0 + 6))) break;
+      tc_fence_after();
+      const float* dec = reinterpret_cast<const float*>(smem + GK_DEC_OFF) + (c & 3) * 128;
+#pragma unroll
+      for (int k = 0; k < SR; ++k) {
+        const int c0 = (half * SR + k) * 16;
+        uint32_t x[16];
+        tmem_ld_32x16(my + GK_ST + c0, x);
+        tmem_ld_wait();
+        float f[16];
+#pragma unroll
+        for (int e = 0; e < 16; e += 4) {
+          const float4 d4 = *reinterpret_cast<const float4*>(dec + c0 + e);
+          f[e] = __uint_as_float(x[e]) * d4.x;
+          f[e + 1] = __uint_as_float(x[e + 1]) * d4.y;
+          f[e + 2] = __uint_as_float(x[e + 2]) * d4.z;
+          f[e + 3] = __uint_as_float(x[e + 3]) * d4.w;
+        }
+        if (t1 < n) {
+          put_state(c0, f);
+        } else if (row < VC) {
+#pragma unroll
+          for (int e = 0; e < 16; ++e)
+            if (c0 + e < p.D) st[c0 + e] = f[e];
+        }
+      }
+      tmem_st_wait();
+      arrive(s_made);
+      if (!__all_sync(0xffffffffu, wait(&o_done[buf], (c >> 1) & 1, t0 + 7))) break;
+      tc_fence_after();
+      if (t1 < n) load_v(t1);
+      // outputs: lanes in pairs, two columns v of one token each
+      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (long long)(first + t0 + half * 32 + (lane & 1)) * p.out_stride +
+                           (long long)h * p.V + v0 + (row & ~1);
+      const int left = (row & ~1) < VC ? cnt - half * 32 - (lane & 1) : 0;
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        uint32_t x[16];
+        tmem_ld_32x16(my + GK_O + half * 32 + 16 * k, x);
+        tmem_ld_wait();
+        if (k == 1) arrive(o_read);
+#pragma unroll
+        for (int e = 0; e < 16; e += 2) {
+          const bool odd = lane & 1;
+          const float got = __shfl_xor_sync(0xffffffffu, __uint_as_float(odd ? x[e] : x[e + 1]), 1);
+          const float own = __uint_as_float(odd ? x[e + 1] : x[e]);
+          if (16 * k + e < left) *reinterpret_cast<uint32_t*>(out) = odd ? pack_bf16x2(got, own) : pack_bf16x2(own, got);
+          out += 2 * p.out_stride;
+        }
+      }
+      t0 = t1;
+    }
+    if (loads_v > 0) mbar_wait(v_in, (loads_v - 1) & 1);
+  } else if (elect_one()) {
+    // ---------------------------------- products ----------------------------------
+    constexpr int K_STEPS = ND / 16;
+    constexpr uint32_t id_kk = umma_idesc(1, 1, 0, 0, 128, 64);           // both K-major
+    constexpr uint32_t id_mm = umma_idesc(1, 1, 1, 1, 128, 64);           // both MN-major
+    constexpr uint32_t id_st = umma_idesc(1, 1, 1, 1, 128, ND);
+    // a step of 32 bytes (K-major) or 2048 bytes (MN-major) adds to the address field of a descriptor
+    const uint32_t base = smem_u32(smem);
+    const uint64_t dq0 = umma_smem_desc(base + GK_Q_OFF, 16, 1024), dk0 = umma_smem_desc(base + GK_K_OFF, 16, 1024),
+                   dkt0 = umma_smem_desc(base + GK_K_OFF, 16384, 1024), dv = umma_smem_desc(base + GK_V_OFF, 8192, 1024),
+                   dp = umma_smem_desc(base + GK_P_OFF, 8192, 1024);
+    int t0 = 0;
+    for (int c = 0; t0 < n; ++c) {
+      const int buf = c & 1;
+      const uint64_t dq = dq0 + buf * (GK_BUF / 16), dk = dk0 + buf * (GK_BUF / 16), dkt = dkt0 + buf * (GK_BUF / 16);
+      if (!wait(&qk_made[buf], (c >> 1) & 1, t0 + 8)) break;
+      tc_fence_after();
+#pragma unroll
+      for (int term = 0; term < 2; ++term)
+#pragma unroll
+        for (int k = 0; k < K_STEPS; ++k)
+          tc_mma_f16(tmem + GK_SC, dk + (k >> 2) * 1024 + (k & 3) * 2, dq + term * 512 + (k >> 2) * 1024 + (k & 3) * 2, id_kk,
+                     term != 0 || k != 0);
+      tc_commit(sc_done);
+      if (!wait(v_in, c & 1, t0 + 9) || !wait(s_made, c & 1, t0 + 10)) break;
+      tc_fence_after();
+#pragma unroll
+      for (int term = 0; term < 2; ++term)
+#pragma unroll
+        for (int k = 0; k < GK_C / 16; ++k)
+          tc_mma_f16(tmem + GK_ST, dv + k * 128, dkt + term * 512 + k * 128, id_st, 1);
+      if (c > 0 && !wait(o_read, (c - 1) & 1, t0 + 11)) break;
+      tc_fence_after();
+#pragma unroll
+      for (int term = 0; term < 3; ++term)  // hi hi, hi lo, lo hi
+#pragma unroll
+        for (int k = 0; k < K_STEPS; ++k)
+          tc_mma_f16_ta(tmem + GK_O, tmem + (term == 2 ? GK_SL : GK_SH) + k * 8,
+                        dq + (term == 1 ? 512 : 0) + (k >> 2) * 1024 + (k & 3) * 2, id_kk, term != 0 || k != 0);
+      tc_commit(&s_done[buf]);
+      if (!wait(p_made, c & 1, t0 + 12)) break;
+      tc_fence_after();
+#pragma unroll
+      for (int k = 0; k < 12; ++k)  // P hi of both partial sums, P lo of the first
+        tc_mma_f16(tmem + GK_O, dv + (k & 3) * 128, dp + k * 128, id_mm, 1);
+      tc_commit(&o_done[buf]);
+      t0 += cnt_s[c & 3];
+    }
   }
-  cp_async_wait<0>();
   tc_fence_before();
   __syncthreads();
-  if (warp == 0) {
+  if (warp == 24) {
     tc_fence_after();
     tmem_dealloc(tmem, 512);
   }
+}
+
+// proj of T tokens; sequences from p.b0 on
+static int run_gla_chunks(const GlaParams& p, int T, int sequences, int* status, cudaStream_t stream) {
+  static bool attr = false;
+  if (!attr) {
+    VB_CUDA_CHECK(cudaFuncSetAttribute(gla_chunk_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, GK_SMEM));
+    VB_CUDA_CHECK(cudaFuncSetAttribute(gla_chunk_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, GK_SMEM));
+    attr = true;
+  }
+  const __nv_bfloat16* x = static_cast<const __nv_bfloat16*>(p.proj);
+  const uint64_t D = p.D, H = p.H, V = p.V, row = (uint64_t)p.stride * 2;
+  CUtensorMap tmQ, tmK, tmV, tmR;
+  int rc = vb_make_tmap_3d(&tmQ, x, 2, D, H, T, D * 2, row, 64, 1, GK_C);
+  if (!rc) rc = vb_make_tmap_3d(&tmK, x + H * D, 2, D, H, T, D * 2, row, 64, 1, GK_C);
+  if (!rc) rc = vb_make_tmap_3d(&tmV, x + 2 * H * D, 2, V, H, T, V * 2, row, 64, 1, GK_C);
+  if (!rc) rc = vb_make_tmap_2d(&tmR, x + 2 * H * (D + V), 2, p.rank, T, row, 64, GK_C);
+  if (rc) return rc;
+  const dim3 g((p.V + 127) / 128, p.H, sequences), blk(GK_THREADS);
+  rc = (int)(p.D <= 64 ? vb_launch_pdl(gla_chunk_kernel<64>, g, blk, GK_SMEM, stream, 1, tmQ, tmK, tmV, tmR, p, status)
+                       : vb_launch_pdl(gla_chunk_kernel<128>, g, blk, GK_SMEM, stream, 1, tmQ, tmK, tmV, tmR, p, status));
+  vb_count_launch();
+  return rc;
 }
 
 template <typename T, int NR>
@@ -720,16 +756,7 @@ static int run_gla(GlaParams p, int T_, int B, int singles, int chunk, int* stat
   }
   p.b0 = singles;
   if (chunk) {
-    static bool attr = false;
-    if (!attr) {
-      VB_CUDA_CHECK(cudaFuncSetAttribute(gla_chunk_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, GK_SMEM));
-      VB_CUDA_CHECK(cudaFuncSetAttribute(gla_chunk_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, GK_SMEM));
-      attr = true;
-    }
-    const dim3 g((p.V + 127) / 128, p.H, B - singles);
-    rc = (int)(p.D <= 64 ? vb_launch_pdl(gla_chunk_kernel<64>, g, dim3(GK_THREADS), GK_SMEM, stream, 1, p, status)
-                         : vb_launch_pdl(gla_chunk_kernel<128>, g, dim3(GK_THREADS), GK_SMEM, stream, 1, p, status));
-    vb_count_launch();
+    rc = run_gla_chunks(p, T_, B - singles, status, stream);
   } else {
     cudaError_t e = vb_launch_pdl(gla_decay_kernel<T>, dim3(T_, (p.H * p.D + 127) / 128), dim3(128), 0, stream, 1, p);
     vb_count_launch();
