@@ -281,9 +281,9 @@ __global__ void __launch_bounds__(GS_THREADS) gla_scan_kernel(const GlaParams p)
 // Every fp32 operand enters as two bf16 terms, so that products carry about 16 bits of both operands and sums are fp32; v and the
 // numbers r are bf16 activations.
 // Warps 0..15 make Q~ and K~ of chunk after chunk (two of them in shared memory), warps 16..23 turn scores into P, decay the state
-// and store the outputs, warp 24 issues the products (but Z, which warp 0 does). A warp reads the TMEM lanes 32 (w % 4) ..; those
-// of a group that share them have equal parts of the columns. q, k, v and r arrive by TMA.
-constexpr int GK_C = 64, GK_MAKERS = 512, GK_USERS = 256, GK_THREADS = GK_MAKERS + GK_USERS + 32;
+// and store the outputs, warp 24 issues the products (but Z, which warp 0 does), warp 25 fetches q and k. A warp reads the TMEM lanes
+// 32 (w % 4) ..; those of a group that share them have equal parts of the columns. q, k, v and r arrive by TMA.
+constexpr int GK_C = 64, GK_MAKERS = 512, GK_USERS = 256, GK_THREADS = GK_MAKERS + GK_USERS + 64;
 constexpr int GK_BUF = 32768;                      // Q~ or K~ of a chunk: per 64 channels hi | lo, [64 tokens] x 128 bytes
 constexpr int GK_Q_OFF = 0, GK_K_OFF = 2 * GK_BUF;
 constexpr int GK_V_OFF = GK_K_OFF + 2 * GK_BUF;    // v [64 tokens][128], two column blocks
@@ -382,7 +382,7 @@ gla_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     const float bias = d_on ? p.decay_b[h * p.D + row] * LOG2E : 0.f;
     const float qscale = 1.f / sqrtf((float)p.D);
     const int r_steps = (p.rank + 15) / 16;
-    int loads_r = 0, loads_qk = 0;
+    int loads_r = 0;
     auto load_r = [&](int t0) {
       mbar_arrive_expect_tx(r_in, 8192);
       tma_load_2d(smem + GK_A_OFF, &tmR, r_in, 0, first + t0);
@@ -390,8 +390,6 @@ gla_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     };
     if (warp == 0) {
       if (elect_one()) {
-        tma_prefetch_desc(&tmQ);
-        tma_prefetch_desc(&tmK);
         tma_prefetch_desc(&tmR);
         load_r(0);
       }
@@ -412,17 +410,10 @@ gla_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     int t0 = 0;
     for (int c = 0; t0 < n; ++c) {
       tc_fence_before();
-      ok = gk_bar_and(ok);  // everyone is through with q and k of the chunk before
+      ok = gk_bar_and(ok);  // everyone has read Z of the chunk before
       if (!ok) break;
       if (warp == 0) {
         if (elect_one()) {
-          mbar_arrive_expect_tx(qk_in, 2 * (ND / 64) * 8192);
-#pragma unroll
-          for (int x = 0; x < ND / 64; ++x) {
-            tma_load_3d(smem + GK_R_OFF + x * 8192, &tmQ, qk_in, x * 64, h, first + t0);
-            tma_load_3d(smem + GK_R_OFF + 16384 + x * 8192, &tmK, qk_in, x * 64, h, first + t0);
-          }
-          ++loads_qk;
           if (wait(r_in, c & 1, t0)) {
             tc_fence_after();
             for (int k = 0; k < r_steps; ++k) tc_mma_f16_ta(tmem + GK_Z, tmem + GK_W + k * 8, da + k * 2, id_z, k != 0);
@@ -501,13 +492,12 @@ gla_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
           const int t = grp * 16 + (odd ? 8 + (j ^ 4) : j);
           const int at = t * 128 + ((g ^ (t & 7)) << 4);
           const uint32_t q2 = *reinterpret_cast<const uint32_t*>(src + at), k2 = *reinterpret_cast<const uint32_t*>(src + 16384 + at);
-          const float e0 = ex2(b0), e1 = ex2(b1);
+          const bool on = t < cnt;  // other tokens: zeros
+          const float e0 = ex2(b0), e1 = ex2(b1), f0 = ex2(-b0), f1 = ex2(-b1), qs = on ? qscale : 0.f;
           if (t == cnt - 1) *reinterpret_cast<float2*>(dec) = make_float2(e0, e1);
-          uint32_t qh = 0, ql = 0, kh = 0, kl = 0;
-          if (t < cnt) {
-            split2(__uint_as_float(q2 << 16) * (qscale * e0), __uint_as_float(q2 & 0xffff0000u) * (qscale * e1), qh, ql);
-            split2(__uint_as_float(k2 << 16) * ex2(-b0), __uint_as_float(k2 & 0xffff0000u) * ex2(-b1), kh, kl);
-          }
+          uint32_t qh, ql, kh, kl;
+          split2(__uint_as_float(q2 << 16) * (qs * e0), __uint_as_float(q2 & 0xffff0000u) * (qs * e1), qh, ql);
+          split2(__uint_as_float(k2 << 16) * (on ? f0 : 0.f), __uint_as_float(k2 & 0xffff0000u) * (on ? f1 : 0.f), kh, kl);
           *reinterpret_cast<uint32_t*>(dst + at + GK_Q_OFF) = qh;
           *reinterpret_cast<uint32_t*>(dst + at + GK_Q_OFF + 8192) = ql;
           *reinterpret_cast<uint32_t*>(dst + at + GK_K_OFF) = kh;
@@ -519,7 +509,6 @@ gla_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       t0 = t1;
     }
     // no copy is in flight when the CTA ends, whatever ended it
-    if (loads_qk > 0) mbar_wait(qk_in, (loads_qk - 1) & 1);
     if (loads_r > 0) mbar_wait(r_in, (loads_r - 1) & 1);
   } else if (warp < 24) {
     // ------------------------- P, the state, the outputs (every warp on its own) -------------------------
@@ -538,25 +527,27 @@ gla_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     };
     load_v(0);
     float* st = p.state + (((long long)slot * p.H + h) * p.V + v0 + row) * p.D;
-    constexpr int SR = ND / 32;  // this thread's channels of column v, 16 at a time
-    // fp32 accumulator and two bf16 terms of 16 channels
-    auto put_state = [&](int c0, const float (&f)[16]) {
-      uint32_t x[16];
+    constexpr int SR = ND / 64;  // this thread's channels of column v, 32 at a time
+    // fp32 accumulator and two bf16 terms of 32 channels
+    auto put_state = [&](int c0, const uint32_t (&x)[32]) {
+      tmem_st_32x32(my + GK_ST + c0, x);
 #pragma unroll
-      for (int e = 0; e < 16; ++e) x[e] = __float_as_uint(f[e]);
-      tmem_st_32x16(my + GK_ST + c0, x);
+      for (int k = 0; k < 2; ++k) {
+        uint32_t y[16];
 #pragma unroll
-      for (int e = 0; e < 8; ++e) split2(f[2 * e], f[2 * e + 1], x[e], x[8 + e]);
-      tmem_st_32x8(my + GK_SH + c0 / 2, x);
-      tmem_st_32x8(my + GK_SL + c0 / 2, x + 8);
+        for (int e = 0; e < 8; ++e)
+          split2(__uint_as_float(x[16 * k + 2 * e]), __uint_as_float(x[16 * k + 2 * e + 1]), y[e], y[8 + e]);
+        tmem_st_32x8(my + GK_SH + c0 / 2 + 8 * k, y);
+        tmem_st_32x8(my + GK_SL + c0 / 2 + 8 * k, y + 8);
+      }
     };
 #pragma unroll
     for (int k = 0; k < SR; ++k) {
-      const int c0 = (half * SR + k) * 16;
-      float f[16];
+      const int c0 = (half * SR + k) * 32;
+      uint32_t x[32];
 #pragma unroll
-      for (int e = 0; e < 16; ++e) f[e] = start > 0 && row < VC && c0 + e < p.D ? st[c0 + e] : 0.f;
-      put_state(c0, f);
+      for (int e = 0; e < 32; ++e) x[e] = start > 0 && row < VC && c0 + e < p.D ? __float_as_uint(st[c0 + e]) : 0u;
+      put_state(c0, x);
     }
     tmem_st_wait();
     arrive(s_made);
@@ -593,25 +584,24 @@ gla_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       const float* dec = reinterpret_cast<const float*>(smem + GK_DEC_OFF) + (c & 3) * 128;
 #pragma unroll
       for (int k = 0; k < SR; ++k) {
-        const int c0 = (half * SR + k) * 16;
-        uint32_t x[16];
-        tmem_ld_32x16(my + GK_ST + c0, x);
+        const int c0 = (half * SR + k) * 32;
+        uint32_t x[32];
+        tmem_ld_32x32(my + GK_ST + c0, x);
         tmem_ld_wait();
-        float f[16];
 #pragma unroll
-        for (int e = 0; e < 16; e += 4) {
+        for (int e = 0; e < 32; e += 4) {
           const float4 d4 = *reinterpret_cast<const float4*>(dec + c0 + e);
-          f[e] = __uint_as_float(x[e]) * d4.x;
-          f[e + 1] = __uint_as_float(x[e + 1]) * d4.y;
-          f[e + 2] = __uint_as_float(x[e + 2]) * d4.z;
-          f[e + 3] = __uint_as_float(x[e + 3]) * d4.w;
+          x[e] = __float_as_uint(__uint_as_float(x[e]) * d4.x);
+          x[e + 1] = __float_as_uint(__uint_as_float(x[e + 1]) * d4.y);
+          x[e + 2] = __float_as_uint(__uint_as_float(x[e + 2]) * d4.z);
+          x[e + 3] = __float_as_uint(__uint_as_float(x[e + 3]) * d4.w);
         }
         if (t1 < n) {
-          put_state(c0, f);
+          put_state(c0, x);
         } else if (row < VC) {
 #pragma unroll
-          for (int e = 0; e < 16; ++e)
-            if (c0 + e < p.D) st[c0 + e] = f[e];
+          for (int e = 0; e < 32; ++e)
+            if (c0 + e < p.D) st[c0 + e] = __uint_as_float(x[e]);
         }
       }
       tmem_st_wait();
@@ -623,24 +613,41 @@ gla_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (long long)(first + t0 + half * 32 + (lane & 1)) * p.out_stride +
                            (long long)h * p.V + v0 + (row & ~1);
       const int left = (row & ~1) < VC ? cnt - half * 32 - (lane & 1) : 0;
+      uint32_t x[32];
+      tmem_ld_32x32(my + GK_O + half * 32, x);
+      tmem_ld_wait();
+      arrive(o_read);
 #pragma unroll
-      for (int k = 0; k < 2; ++k) {
-        uint32_t x[16];
-        tmem_ld_32x16(my + GK_O + half * 32 + 16 * k, x);
-        tmem_ld_wait();
-        if (k == 1) arrive(o_read);
-#pragma unroll
-        for (int e = 0; e < 16; e += 2) {
-          const bool odd = lane & 1;
-          const float got = __shfl_xor_sync(0xffffffffu, __uint_as_float(odd ? x[e] : x[e + 1]), 1);
-          const float own = __uint_as_float(odd ? x[e + 1] : x[e]);
-          if (16 * k + e < left) *reinterpret_cast<uint32_t*>(out) = odd ? pack_bf16x2(got, own) : pack_bf16x2(own, got);
-          out += 2 * p.out_stride;
-        }
+      for (int e = 0; e < 32; e += 2) {
+        const bool odd = lane & 1;
+        const float got = __shfl_xor_sync(0xffffffffu, __uint_as_float(odd ? x[e] : x[e + 1]), 1);
+        const float own = __uint_as_float(odd ? x[e + 1] : x[e]);
+        if (e < left) *reinterpret_cast<uint32_t*>(out) = odd ? pack_bf16x2(got, own) : pack_bf16x2(own, got);
+        out += 2 * p.out_stride;
       }
       t0 = t1;
     }
     if (loads_v > 0) mbar_wait(v_in, (loads_v - 1) & 1);
+  } else if (warp == 25) {
+    // ----------------------------------- q and k -----------------------------------
+    if (elect_one()) {
+      tma_prefetch_desc(&tmQ);
+      tma_prefetch_desc(&tmK);
+      int t0 = 0, c = 0;
+      for (; t0 < n; ++c) {
+        mbar_arrive_expect_tx(qk_in, 2 * (ND / 64) * 8192);
+#pragma unroll
+        for (int x = 0; x < ND / 64; ++x) {
+          tma_load_3d(smem + GK_R_OFF + x * 8192, &tmQ, qk_in, x * 64, h, first + t0);
+          tma_load_3d(smem + GK_R_OFF + 16384 + x * 8192, &tmK, qk_in, x * 64, h, first + t0);
+        }
+        if (!wait(&qk_made[c & 1], (c >> 1) & 1, t0 + 13)) {
+          mbar_wait(qk_in, c & 1);
+          break;
+        }
+        t0 += cnt_s[c & 3];
+      }
+    }
   } else if (elect_one()) {
     // ---------------------------------- products ----------------------------------
     constexpr int K_STEPS = ND / 16;
