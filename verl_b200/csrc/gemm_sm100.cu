@@ -875,13 +875,14 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
     *abort_flag = 0;
     mbar_fence_init();
   }
-  if (warp == 1) {
-    tmem_alloc_pair(tmem_slot, 2 * P_BN);
-    tmem_relinquish_pair();
-  }
+  // The pair allocates together, in the tensor memory of both SMs: not before both CTAs run. An allocation that one CTA made
+  // while the other was still being started has been seen to leave that one waiting for its columns for good.
+  cluster_sync_all();
+  if (warp == 1) tmem_alloc_pair(tmem_slot, 2 * P_BN);
   tc_fence_before();
   __syncthreads();
   cluster_sync_all();  // both CTAs' barriers are initialised and both allocations are done
+  if (warp == 1) tmem_relinquish_pair();
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
   pdl_trigger();  // TMEM is held: a dependent kernel may take what is left
